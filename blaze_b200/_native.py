@@ -19,7 +19,7 @@ import shutil
 import subprocess
 import sys
 from concurrent.futures import ThreadPoolExecutor
-from typing import List, Optional
+from typing import Dict, List, Optional, Sequence, Tuple
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 CSRC = os.path.join(ROOT, "csrc")
@@ -48,7 +48,7 @@ def _digest(paths: List[str]) -> str:
     for dp, _, fs in os.walk(os.path.join(CSRC, "include")):
         incs += [os.path.join(dp, f) for f in fs]
     for p in sorted(paths + incs):
-        h.update(p.encode())
+        h.update(os.path.relpath(p, ROOT).encode())      # a library stays valid when the tree moves
         with open(p, "rb") as f:
             h.update(f.read())
     return h.hexdigest()
@@ -62,54 +62,99 @@ def _stale(so: str, paths: List[str]) -> bool:
         return f.read().strip() != _digest(paths)
 
 
+def _compile(cu: List[str], verbose: bool = False, force: bool = False) -> List[str]:
+    """Object files of kernel sources; those whose source and headers have not changed are kept."""
+    nvcc = _nvcc()
+    if nvcc is None:
+        raise RuntimeError("nvcc not found; cannot build blaze_b200 kernels")
+    objdir = os.path.join(LIBDIR, "obj")
+    os.makedirs(objdir, exist_ok=True)
+
+    def one(src):
+        obj = os.path.join(objdir, os.path.basename(src) + ".o")
+        if not force and not _stale(obj, [src]):
+            return obj
+        cmd = [nvcc] + NVCC_FLAGS + ["-c", src, "-o", obj]
+        r = subprocess.run(cmd, capture_output=True, text=True)
+        if r.returncode != 0:
+            raise RuntimeError(f"nvcc failed for {src}:\n{r.stdout}\n{r.stderr}")
+        if verbose and r.stderr:
+            print(r.stderr, file=sys.stderr)
+        with open(obj + ".sha", "w") as f:
+            f.write(_digest([src]))
+        return obj
+
+    # the longest compilations first, so that none of them starts when the others are done
+    order = sorted(cu, key=lambda p: -os.path.getsize(p))
+    with ThreadPoolExecutor(max_workers=min(max(os.cpu_count() or 8, 8), len(cu))) as ex:
+        objs = list(ex.map(one, order))
+    return sorted(objs)
+
+
+def _link(so: str, cu: List[str], objs: List[str]) -> None:
+    part = f"{so}.{os.getpid()}.part"
+    r = subprocess.run([_nvcc(), "-shared", "-o", part] + objs + ["-gencode", "arch=compute_100a,code=sm_100a"],
+                       capture_output=True, text=True)
+    if r.returncode != 0:
+        raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+    os.replace(part, so)
+    with open(so + ".sha", "w") as f:
+        f.write(_digest(cu))
+
+
+def build_runtime(force: bool = False) -> None:
+    """The host runtime library, if out of date."""
+    os.makedirs(LIBDIR, exist_ok=True)
+    cpp = _sources("runtime", ".cpp")
+    if cpp and (force or _stale(RUNTIME_SO, cpp)):
+        cxx = shutil.which("g++") or "g++"
+        part = f"{RUNTIME_SO}.{os.getpid()}.part"
+        cmd = [cxx, "-O3", "-std=c++17", "-fPIC", "-shared", "-pthread", "-mavx2", "-mfma", "-ffp-contract=off",
+               "-I" + os.path.join(CSRC, "include"), "-o", part] + cpp
+        r = subprocess.run(cmd, capture_output=True, text=True)
+        if r.returncode != 0:
+            raise RuntimeError(f"g++ failed:\n{r.stdout}\n{r.stderr}")
+        os.replace(part, RUNTIME_SO)
+        with open(RUNTIME_SO + ".sha", "w") as f:
+            f.write(_digest(cpp))
+
+
 def build(force: bool = False, verbose: bool = False) -> None:
     """Compile everything that is out of date.  Raises on a compiler error."""
     os.makedirs(LIBDIR, exist_ok=True)
     cu = _sources("kernels", ".cu")
     if cu and (force or _stale(KERNELS_SO, cu)):
-        nvcc = _nvcc()
-        if nvcc is None:
-            raise RuntimeError("nvcc not found; cannot build blaze_b200 kernels")
-        objdir = os.path.join(LIBDIR, "obj")
-        os.makedirs(objdir, exist_ok=True)
+        _link(KERNELS_SO, cu, _compile(cu, verbose, force))
+    build_runtime(force)
 
-        def one(src):
-            obj = os.path.join(objdir, os.path.basename(src) + ".o")
-            cmd = [nvcc] + NVCC_FLAGS + ["-c", src, "-o", obj]
-            r = subprocess.run(cmd, capture_output=True, text=True)
-            if r.returncode != 0:
-                raise RuntimeError(f"nvcc failed for {src}:\n{r.stdout}\n{r.stderr}")
-            if verbose and r.stderr:
-                print(r.stderr, file=sys.stderr)
-            return obj
 
-        with ThreadPoolExecutor(max_workers=min(8, len(cu))) as ex:
-            objs = list(ex.map(one, cu))
-        r = subprocess.run([nvcc, "-shared", "-o", KERNELS_SO] + objs + ["-gencode", "arch=compute_100a,code=sm_100a"],
-                           capture_output=True, text=True)
-        if r.returncode != 0:
-            raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
-        with open(KERNELS_SO + ".sha", "w") as f:
-            f.write(_digest(cu))
-    cpp = _sources("runtime", ".cpp")
-    if cpp and (force or _stale(RUNTIME_SO, cpp)):
-        cxx = shutil.which("g++") or "g++"
-        cmd = [cxx, "-O3", "-std=c++17", "-fPIC", "-shared", "-pthread", "-mavx2", "-mfma", "-ffp-contract=off",
-               "-I" + os.path.join(CSRC, "include"), "-o", RUNTIME_SO] + cpp
-        r = subprocess.run(cmd, capture_output=True, text=True)
-        if r.returncode != 0:
-            raise RuntimeError(f"g++ failed:\n{r.stdout}\n{r.stderr}")
-        with open(RUNTIME_SO + ".sha", "w") as f:
-            f.write(_digest(cpp))
+def _part_so(sources: Sequence[str]) -> str:
+    """A library of some of the kernel sources (names without ``.cu``), built if needed: what one model family launches, for a
+    fresh checkout that has no complete library yet."""
+    cu = [os.path.join(CSRC, "kernels", n + ".cu") for n in sorted(sources)]
+    so = os.path.join(LIBDIR, "libblaze_kernels_" + hashlib.sha256(" ".join(sorted(sources)).encode()).hexdigest()[:8] + ".so")
+    os.makedirs(LIBDIR, exist_ok=True)
+    if _stale(so, cu):
+        _link(so, cu, _compile(cu))
+    return so
 
 
 _kernels = None
 _runtime = None
 
 
-def kernels() -> ctypes.CDLL:
-    """The CUDA kernel library.  Builds it when missing and nvcc is present; raises otherwise."""
+_parts: Dict[Tuple[str, ...], ctypes.CDLL] = {}
+
+
+def kernels(sources: Optional[Sequence[str]] = None) -> ctypes.CDLL:
+    """The CUDA kernel library.  Builds it when missing and nvcc is present; raises otherwise.  ``sources``: the kernel sources
+    the caller launches from; while the complete library is missing or out of date, a library of just these is built."""
     global _kernels
+    if sources is not None and _kernels is None and _stale(KERNELS_SO, _sources("kernels", ".cu")):
+        key = tuple(sorted(sources))
+        if key not in _parts:
+            _parts[key] = ctypes.CDLL(_part_so(key))
+        return _parts[key]
     if _kernels is None:
         if not os.path.exists(KERNELS_SO) or (os.environ.get("BLAZE_REBUILD") and _stale(KERNELS_SO, _sources("kernels", ".cu"))):
             build()
@@ -124,7 +169,7 @@ def runtime() -> ctypes.CDLL:
     global _runtime
     if _runtime is None:
         if not os.path.exists(RUNTIME_SO):
-            build()
+            build_runtime()
         _runtime = ctypes.CDLL(RUNTIME_SO)
     return _runtime
 

@@ -24,6 +24,8 @@ class SeqChunk:
     tokens: Sequence[int]     # new token ids (1 for decode, k+1 for verify, a chunk for prefill)
     start_pos: int            # position of tokens[0]  (== KV length before this step)
     want_logits: int = 1      # how many trailing rows need logits (0 = headless prefill chunk)
+    logit_at: Optional[Sequence[int]] = None         # rows of this chunk that need logits, in this order, when they are not the
+                                                     # trailing ones (scoring, replayed traces)
     pos3: Optional[Sequence[Sequence[int]]] = None   # M-RoPE: rotary positions (temporal, height, width) of the rows, 3 x n;
                                                      # None = all three equal start_pos + i + rope_delta
     rope_delta: int = 0       # added to the rotary position of text rows after image blocks (KV slots still follow start_pos)
@@ -154,7 +156,7 @@ def build_batch(chunks: Sequence[SeqChunk], block_table_host: np.ndarray, device
         slots[b] = c.slot
         q_start[b + 1] = r + n
         ctx_len[b] = c.start_pos + n
-        for j in range(n - c.want_logits, n):
+        for j in (range(n - c.want_logits, n) if c.logit_at is None else c.logit_at):
             logit_rows.append(r + j)
         r += n
         max_q = max(max_q, n)

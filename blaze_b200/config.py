@@ -37,6 +37,38 @@ class RopeConfig:
 
 
 @dataclass
+class DiffAttnSpec:
+    """Differential attention of one layer: two attention maps per head over the same values, the second subtracted from the
+    first with a learned weight."""
+    heads: int
+    kv_heads: int
+    dim: int                    # per map and head, queries and keys
+    vdim: int                   # per head, values
+    scale: float                # of the scores
+    diff: float                 # constant part of the second map's weight; the normed output is scaled by 1 - diff
+    window: int = 0             # a row sees itself and the window - 1 tokens before it (0: every token before it)
+
+    @property
+    def group(self) -> int:
+        return self.heads // self.kv_heads
+
+
+@dataclass
+class GluSpec:
+    """Dense feed-forward with a clamped gate and a clamped up projection."""
+    ff: int
+    limit: float
+
+
+@dataclass
+class LayerSpec:
+    """One entry of a configuration that describes its layers one by one."""
+    attn: DiffAttnSpec
+    mlp: Optional[GluSpec] = None          # None: the layer has no feed-forward
+    weights_of: Optional[int] = None       # the layer whose tensors this one uses (with a cache of its own)
+
+
+@dataclass
 class ModelConfig:
     architecture: str = "Qwen3ForCausalLM"
     model_type: str = "qwen3"
@@ -86,6 +118,12 @@ class ModelConfig:
     indexer_head_dim: int = 0
     indexer_budget: int = 0
     indexer_compress_ratio: int = 0
+    # models whose configuration lists its layers one by one, each with sizes of its own (Sevevik); the sizes above then hold
+    # those of the first layer
+    layer_specs: List[LayerSpec] = field(default_factory=list)
+    streams: int = 1                        # residual streams joined by learned static mixes
+    residual_mult: float = 1.0              # of every sublayer's output
+    embed_scale: float = 1.0
     # tokens
     eos_token_ids: List[int] = field(default_factory=list)
     bos_token_id: Optional[int] = None
@@ -122,6 +160,8 @@ class ModelConfig:
         return self.num_kv_heads * self.head_dim
 
     def layer_type(self, i: int) -> str:
+        if self.layer_specs:
+            return "diff_attention"
         return self.layer_types[i] if self.layer_types else "full_attention"
 
     def to_dict(self) -> Dict[str, Any]:
@@ -159,6 +199,8 @@ class ModelConfig:
 
     @classmethod
     def from_json(cls, raw: Dict[str, Any]) -> "ModelConfig":
+        if raw.get("architecture") == "Sevevik":
+            return cls._from_sevevik(raw)
         archs = raw.get("architectures") or ["Qwen3ForCausalLM"]
         t = raw.get("text_config", raw)
         g = lambda k, d=None: t.get(k, raw.get(k, d))  # noqa: E731
@@ -252,6 +294,56 @@ class ModelConfig:
         cfg.rope = rope
         return cfg
 
+    @classmethod
+    def _from_sevevik(cls, raw: Dict[str, Any]) -> "ModelConfig":
+        """The layer-by-layer configuration of the Sevevik design."""
+        specs: List[LayerSpec] = []
+        for i, e in enumerate(raw["layers"]):
+            if e["type"] != "attention":
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+            m = e["mixer"]
+            mask = m.get("mask") or {}
+            attn = DiffAttnSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                                scale=float(m["scale"]), diff=float(m["diff"]), window=int(mask.get("size") or 0))
+            mlp = None
+            if e.get("mlp") is not None:
+                if e["mlp"].get("kind", "dense") != "dense":
+                    raise ValueError(f"layer {i}: unknown feed-forward {e['mlp']['kind']!r}")
+                mlp = GluSpec(ff=int(e["mlp"]["ff"]), limit=float(e["mlp"]["limit"]))
+            wof = e.get("weights_of")
+            specs.append(LayerSpec(attn, mlp, None if wof is None else int(wof)))
+        if not specs:
+            raise ValueError("the configuration lists no layers")
+        _check_layers(specs)
+        return cls.of_layers(specs, architecture="Sevevik", model_type="sevevik", vocab_size=int(raw["vocab"]),
+                             hidden_size=int(raw["width"]), rms_norm_eps=float(raw["norm"]["eps"]), streams=int(raw.get("streams", 1)),
+                             residual_mult=float(raw.get("residual_mult", 1.0)),
+                             embed_scale=float((raw.get("embedding") or {}).get("scale", 1.0)),
+                             torch_dtype=str(raw.get("torch_dtype", "bfloat16")))
+
+    @classmethod
+    def of_layers(cls, specs: List[LayerSpec], **kw) -> "ModelConfig":
+        """A configuration from its layer list; the model-wide sizes that other parts read are those of the first layer."""
+        a, mlp = specs[0].attn, specs[0].mlp
+        return cls(layer_specs=specs, num_layers=len(specs), num_heads=a.heads, num_kv_heads=a.kv_heads, head_dim=a.dim,
+                   intermediate_size=mlp.ff if mlp else 0, qk_norm=False, layer_types=["diff_attention"] * len(specs), **kw)
+
+
+def _check_layers(specs: List[LayerSpec]) -> None:
+    """Refuse a layer list that no model of the design can have."""
+    for i, s in enumerate(specs):
+        a = s.attn
+        if min(a.heads, a.kv_heads, a.dim, a.vdim) < 1 or a.heads % a.kv_heads:
+            raise ValueError(f"layer {i}: {a.heads} query heads over {a.kv_heads} key/value heads of {a.dim} / {a.vdim}")
+        if a.window < 0:
+            raise ValueError(f"layer {i}: a window of {a.window}")
+        if s.weights_of is not None:
+            src = specs[s.weights_of] if 0 <= s.weights_of < len(specs) else None
+            if src is None or src.weights_of is not None:
+                raise ValueError(f"layer {i} uses the tensors of layer {s.weights_of}, which has none of its own")
+            if (src.attn, src.mlp) != (a, s.mlp):
+                raise ValueError(f"layer {i} differs from layer {s.weights_of}, whose tensors it uses")
+
 
 def inv_freq(cfg: ModelConfig, yarn_factor_override: Optional[float] = None):
     """Rotary inverse frequencies (fp32 list), with YaRN blending when enabled.
@@ -305,6 +397,23 @@ def named_config(name: str) -> ModelConfig:
         c.hc_count, c.hc_lowrank = 2, 8
         c.ple_layers, c.ngram_size, c.heads_per_ngram, c.ple_embed_dim, c.ple_conv_kernel = [0, 2], 3, 2, 16, 4
         c.eos_token_ids = [1]
+    elif n in ("tiny-sevevik",):
+        # the Sevevik layer kinds in miniature: unequal layers, one without a feed-forward, one that uses another's tensors
+        a = DiffAttnSpec(heads=4, kv_heads=2, dim=32, vdim=48, scale=0.2, diff=0.35, window=40)
+        b = DiffAttnSpec(heads=3, kv_heads=1, dim=16, vdim=64, scale=0.25, diff=0.2, window=24)
+        layers = [LayerSpec(a, GluSpec(320, 3.0)), LayerSpec(b), LayerSpec(a, GluSpec(320, 3.0), weights_of=0)]
+        return ModelConfig.of_layers(layers, architecture="Sevevik", model_type="sevevik", vocab_size=1024, hidden_size=192,
+                                     streams=3, residual_mult=0.8, embed_scale=6.0)
+    elif n in ("sevevik-8b", "sevevik-1b"):
+        # layers of a size that real models have (random weights: no checkpoint of the design at this size exists)
+        if n == "sevevik-8b":
+            a = DiffAttnSpec(heads=32, kv_heads=8, dim=64, vdim=128, scale=0.125, diff=0.5, window=1024)
+            ff, width, count = GluSpec(12288, 7.0), 4096, 36
+        else:
+            a = DiffAttnSpec(heads=16, kv_heads=8, dim=64, vdim=128, scale=0.125, diff=0.5, window=1024)
+            ff, width, count = GluSpec(6144, 7.0), 2048, 16
+        return ModelConfig.of_layers([LayerSpec(a, ff) for _ in range(count)], architecture="Sevevik", model_type="sevevik",
+                                     vocab_size=151936, hidden_size=width, streams=4, residual_mult=1.0, embed_scale=1.0)
     elif n in ("qwen3-8b",):
         c = ModelConfig(vocab_size=151936, hidden_size=4096, num_layers=36, num_heads=32, num_kv_heads=8,
                         head_dim=128, intermediate_size=12288, rope=RopeConfig(theta=1e6))

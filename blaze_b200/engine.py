@@ -138,7 +138,7 @@ class Engine:
                 kv_tokens = min(ecfg.max_seqs * ecfg.max_model_len, 1 << 16)
         self.num_pages = kv_tokens // PAGE + 1
         self.max_pages_per_seq = (ecfg.max_model_len + PAGE - 1) // PAGE
-        layout = "umma" if (self.device.type == "cuda" and ecfg.kv_dtype == "fp8" and model.ops.is_cuda) else "logical"
+        layout = "tiles" if (cfg.layer_specs and model.ops.is_cuda) else "umma" if (self.device.type == "cuda" and ecfg.kv_dtype == "fp8" and model.ops.is_cuda) else "logical"
         if ecfg.kv_rotate and cfg.head_dim & (cfg.head_dim - 1):
             raise ValueError("kv_rotate needs a power-of-two head_dim")
         model.kv_rotate = bool(ecfg.kv_rotate)      # read by the attention prep of both op sets
@@ -159,10 +159,11 @@ class Engine:
         self._last_greedy = None            # output of the last greedy decode step (source of token feedback)
         self._deferred: Dict[int, Tuple[int, int, int]] = {}   # slot -> (first row, first position, rows) of the last deferring step
         self.attn_group = 0
-        if model.ops.is_cuda:
+        if model.ops.is_cuda and not cfg.layer_specs:
             self.attn_group = max(max(cfg.num_heads // tpw, 1) // max(cfg.num_kv_heads // tpw, 1), 1)
         # the decode attention kernel covers head_dim 128; other head sizes run every sequence through the row-block kernel
-        self.attn_all_items = bool(model.ops.is_cuda and cfg.head_dim != 128)
+        # (differential attention sorts the rows itself: its layers may differ in group size)
+        self.attn_all_items = bool(model.ops.is_cuda and cfg.head_dim != 128 and not cfg.layer_specs)
         # Device status word, watched without a synchronisation of its own: after every step a 4-byte copy into this pinned
         # word is queued behind the step's kernels; whoever takes the step's results (and has synchronised for that)
         # calls check_status().  `status_source` replaces the device word in tests.
@@ -181,6 +182,11 @@ class Engine:
         self.kernel_launches = 0
 
     # ================================================================== page API
+    @property
+    def trees_ok(self) -> bool:
+        """Draft trees are verified by the attention kernels of plain softmax layers only."""
+        return not self.kv.gdn_layers and not self.model.cfg.layer_specs
+
     @property
     def free_tokens(self) -> int:
         return self.pages.free_count * PAGE
@@ -256,14 +262,19 @@ class Engine:
 
     # ================================================================== stepping
     def plan(self, items: Sequence[Tuple[Seq, Sequence[int], int]], defer_state: bool = False) -> List[SeqChunk]:
-        """items: (seq, new tokens, rows wanting logits).  Reserves pages and advances lengths.  ``defer_state``: the rows
+        """items: (seq, new tokens, rows wanting logits: how many of the last ones, or a list of places among the new tokens).
+        Reserves pages and advances lengths.  ``defer_state``: the rows
         are speculative — models with recurrent layers leave those sequences' state as it was, and ``commit_state`` advances
         it over the accepted rows afterwards."""
         chunks = []
         defer = bool(defer_state and self.kv.gdn_layers)
         for s, toks, want in items:
             self.reserve(s, s.length + len(toks))
-            chunks.append(SeqChunk(slot=s.row, tokens=list(toks), start_pos=s.length, want_logits=want, defer_state=defer))
+            at = None if isinstance(want, int) else [int(j) for j in want]
+            if at is not None and any(j < 0 or j >= len(toks) for j in at):
+                raise ValueError("logits wanted at a place outside the new tokens")
+            chunks.append(SeqChunk(slot=s.row, tokens=list(toks), start_pos=s.length, want_logits=want if at is None else len(at),
+                                   logit_at=at, defer_state=defer))
             s.length += len(toks)
         return chunks
 
@@ -289,8 +300,8 @@ class Engine:
         ``tokens[i]`` a drafted token whose parent row is ``parents[i] < i``.  Every row gets logits.  Row i's KV lands at
         slot ``length + i``; ``commit_tree`` moves the accepted path into place afterwards
         (reference: ``Engine::verify_many_tree``, crates/blaze/src/engine.rs :1401)."""
-        if self.kv.gdn_layers:
-            raise ValueError("draft trees need a model without recurrent (linear-attention) layers")
+        if not self.trees_ok:
+            raise ValueError("draft trees need a model without recurrent (linear-attention) layers and without differential attention")
         group = max(self.model.cfg.num_heads // max(self.model.cfg.num_kv_heads, 1), 1)
         chunks = []
         for s, toks, parents in items:
@@ -344,7 +355,7 @@ class Engine:
                 if c.defer_state:
                     self._deferred[c.slot] = (r, c.start_pos, len(c.tokens))
                 r += len(c.tokens)
-        plain = not any(c.rope_delta or c.pos3 is not None or c.embeds for c in chunks)     # captured steps carry text rows only
+        plain = not any(c.rope_delta or c.pos3 is not None or c.embeds or c.logit_at is not None for c in chunks)     # captured steps carry text rows only
         graphable = (plain and hidden_in is None and self.ecfg.use_graphs and self.device.type == "cuda" and decode_only
                      and mode == "greedy" and self.model.is_first_stage and self.model.is_last_stage and self.model.ops.is_cuda)
         # verify steps of equal-length chains (the scheduler pads drafts to one length) replay a captured graph as well

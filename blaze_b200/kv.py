@@ -9,6 +9,12 @@ Pages hold 16 tokens.  Two pool layouts exist:
   byte of token t, dim j at ``(t//8)*8*D + (j//16)*128 + (t%8)*16 + j%16``) followed by V transposed
   (``[head_dim][16 tokens]``), so that one 1-D bulk copy per (page, head) feeds both MMAs.
 
+* ``tiles`` — one tensor ``[pages, kv_heads, 16 * (2 * dim + vdim)]`` per differential-attention layer in bf16 or fp32: the keys
+  of map 1, the keys of map 2 and the values of the page's 16 tokens, each as 8-token x 8-element core matrices (element of token
+  t, dim j at ``(t // 8) * 8 * D + (j // 8) * 64 + (t % 8) * 8 + j % 8``, D rounded up to 16 and padded with zeros): 8 x 16 bytes
+  in a row is what ``ldmatrix`` and the tensor core's unswizzled operands both take.  The ``logical`` form of such a layer is
+  ``k [pages, 2 * kv_heads, 16, dim]`` (key head g's maps at 2g and 2g + 1) and ``v [pages, kv_heads, 16, vdim]``.
+
 The reference keeps one-token pages and several KV dtypes (``crates/blaze/src/model.rs:499-583``,
 ``alloc_kv`` :517); its page bookkeeping is in ``engine.rs:1083-1164``.
 """
@@ -26,7 +32,18 @@ from .config import ModelConfig
 PAGE = 16
 
 
+def pad16(n: int) -> int:
+    return (n + 15) // 16 * 16
+
+
+def diff_page_elems(spec) -> int:
+    """Elements of one (page, key/value head) block of the ``tiles`` layout."""
+    return PAGE * (2 * pad16(spec.dim) + pad16(spec.vdim))
+
+
 def kv_bytes_per_token(cfg: ModelConfig, kv_dtype: str, tp_world: int = 1) -> int:
+    if cfg.layer_specs:
+        return sum(s.attn.kv_heads * diff_page_elems(s.attn) for s in cfg.layer_specs) // PAGE * (4 if kv_dtype == "fp32" else 2)
     n_attn = sum(1 for i in range(cfg.num_layers) if cfg.layer_type(i) == "full_attention")
     kvh = max(cfg.num_kv_heads // tp_world, 1)
     if kv_dtype in FP4_KV:
@@ -72,6 +89,15 @@ class KVCache:
         self.k: Dict[int, torch.Tensor] = {}
         self.v: Dict[int, torch.Tensor] = {}
         self.kv: Dict[int, torch.Tensor] = {}
+        for i in (range(lo, hi) if cfg.layer_specs else ()):
+            a = cfg.layer_specs[i].attn
+            if kv_dtype not in ("fp32", "bf16"):
+                raise ValueError(f"differential attention keeps its keys and values in bf16 or fp32, not {kv_dtype}")
+            if layout == "tiles":
+                self.kv[i] = torch.zeros(num_pages, a.kv_heads, diff_page_elems(a), dtype=tdt, device=device)
+            else:
+                self.k[i] = torch.zeros(num_pages, 2 * a.kv_heads, PAGE, a.dim, dtype=tdt, device=device)
+                self.v[i] = torch.zeros(num_pages, a.kv_heads, PAGE, a.vdim, dtype=tdt, device=device)
         for i in self.attn_layers:
             if layout == "umma":
                 assert kv_dtype == "fp8"

@@ -16,6 +16,7 @@ import torch
 from . import log
 from .config import ModelConfig, named_config
 from .engine import Engine, EngineConfig
+from .models import model_class
 from .models.qwen3 import Model, TPInfo
 from .quant import Format
 from .sampler import SamplingParams
@@ -72,11 +73,15 @@ class LLM:
             if isinstance(model, Model):
                 self.model = model
             elif isinstance(model, ModelConfig):
-                self.model = Model.random_init(model, fmt, seed, self.device, dtype, tpi, first_layer=lo, last_layer=hi)
+                self.model = model_class(model).random_init(model, fmt, seed, self.device, dtype, tpi, first_layer=lo, last_layer=hi)
             elif os.path.isdir(model):
-                self.model = Model.load(model, self.device, dtype, tpi, first_layer=lo, last_layer=hi)
+                cfg = ModelConfig.load(model)
+                self.model = model_class(cfg).load(model, self.device, dtype, tpi, first_layer=lo, last_layer=hi, cfg=cfg)
             else:
-                self.model = Model.random_init(named_config(model), fmt, seed, self.device, dtype, tpi, first_layer=lo, last_layer=hi)
+                cfg = named_config(model)
+                self.model = model_class(cfg).random_init(cfg, fmt, seed, self.device, dtype, tpi, first_layer=lo, last_layer=hi)
+        if self.device.type == "cuda" and self.model.ops.is_cuda and dtype not in self.model.cuda_dtypes:
+            raise ValueError(f"the kernels of {self.model.cfg.architecture} do not run in {dtype}")
         cfg = self.model.cfg
         self.heat = None
         if expert_heat:
@@ -90,7 +95,8 @@ class LLM:
             with log.Stage("tune"):
                 tune_model(self.model, rows=sorted({min(max_seqs, 256), min(max_seqs, 64)}))
         if kv_cache_dtype == "auto":
-            kv_cache_dtype = "fp8" if (self.device.type == "cuda" and self.model.ops.is_cuda) else \
+            kv_cache_dtype = ("fp32" if dtype == torch.float32 else "bf16") if not self.model.fp8_pages else \
+                "fp8" if (self.device.type == "cuda" and self.model.ops.is_cuda) else \
                 ("fp32" if dtype == torch.float32 else "bf16")
         if kv_cache_dtype.startswith("nvfp4") and self.model.ops.is_cuda:
             raise ValueError(f"kv_cache_dtype {kv_cache_dtype!r}: the attention kernels read FP8 pages; NVFP4 pages run on the oracle op set")
@@ -99,9 +105,9 @@ class LLM:
                                                           kv_dtype=kv_cache_dtype, chunk=chunk, use_graphs=use_graphs,
                                                           kv_rotate=kv_rotate))
         eos = tuple(eos_ids) or tuple(cfg.eos_token_ids)
-        if self.model.cfg.has_hc and (drafter is not None or spec_method in ("mtp", "eagle", "dflash")):
+        if (self.model.cfg.has_hc or self.model.cfg.layer_specs) and (drafter is not None or spec_method in ("mtp", "eagle", "dflash")):
             # a drafter reads the target's hidden rows; a hyper-connection model hands out its streams instead
-            raise ValueError("model drafters are not built for hyper-connection models: use --spec-method ngram or suffix")
+            raise ValueError("model drafters are not built for hyper-connection and stream models: use --spec-method ngram or suffix")
         if drafter is None and spec_method in ("mtp", "eagle", "dflash"):
             from .models.drafter import build_drafter
             with log.Stage("drafter"):

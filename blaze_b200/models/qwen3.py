@@ -34,6 +34,22 @@ class Attn:
         self.kv_heads = 0
 
 
+class DiffAttn:
+    """Differential attention: ``qkv`` rows [q (head, map) | k (head, map) | v], ``lam`` the weight of the second map."""
+
+    def __init__(self, spec=None):
+        self.spec = spec                 # config.DiffAttnSpec
+        self.qkv: Linear = None
+        self.o: Linear = None
+        self.lam = 0.0
+
+    @staticmethod
+    def map_weight(lq1, lk1, lq2, lk2, diff: float) -> float:
+        """``exp(lq1 . lk1) - exp(lq2 . lk2) + diff``: one number for the layer."""
+        dot = lambda a, b: math.exp(float((a.double() * b.double()).sum()))      # noqa: E731
+        return dot(lq1, lk1) - dot(lq2, lk2) + diff
+
+
 class Gdn:
     def __init__(self):
         self.in_proj: Linear = None      # rows [q | k | v | z | b | a]
@@ -50,6 +66,15 @@ class DenseMlp:
     def __init__(self):
         self.gate_up: Linear = None
         self.down: Linear = None
+
+
+class ClampedGlu:
+    """Dense feed-forward ``down(g * sigmoid(1.702 g) * (u + 1))`` with g clamped from above and u on both sides."""
+
+    def __init__(self, limit: float = 0.0):
+        self.gate_up: Linear = None
+        self.down: Linear = None
+        self.limit = limit
 
 
 class Experts:
@@ -157,12 +182,22 @@ class TPInfo:
 
 
 class Model:
+    kernel_sources = None    # kernel sources a model class launches from (None: the complete library)
+    cuda_dtypes = (torch.bfloat16,)      # activation types the kernels of this class run in
+    fp8_pages = True         # the attention kernels of this class read FP8 pages
+
+    @classmethod
+    def _supports(cls, cfg: ModelConfig) -> None:
+        if cfg.layer_specs:
+            raise ValueError(f"{cfg.architecture} lists its layers one by one: use models.model_class(cfg)")
+
     def __init__(self, cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, tp: Optional[TPInfo] = None, ops=None,
                  first_layer: int = 0, last_layer: Optional[int] = None):
         from ..ops import get_ops
+        self._supports(cfg)
         self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
         self.tp = tp or TPInfo()
-        self.ops = ops or get_ops(device)
+        self.ops = ops or get_ops(device, sources=self.kernel_sources)
         self.layers: List[Layer] = []
         self.embed: torch.Tensor = None
         self.final_norm: torch.Tensor = None
@@ -673,6 +708,9 @@ class Model:
             o = ops.mul_sigmoid(o, gate.reshape(o.shape))
         return self._row_cut(A.o, o, o.shape[0], fused)
 
+    def _diff_attention(self, A: DiffAttn, h, batch, kv, gi):
+        return self.ops.linear(A.o, self.ops.diff_attention(self.ops.linear(A.qkv, h), A, batch, kv, gi, self.cfg.rms_norm_eps))
+
     def _gdn(self, G: Gdn, h, batch, kv, gi, fused=None):
         ops, cfg = self.ops, self.cfg
         dk, dv = cfg.linear_key_head_dim, cfg.linear_value_head_dim
@@ -724,6 +762,8 @@ class Model:
         """Returns (output, kind) with kind as in :meth:`forward`."""
         ops = self.ops
         tp = self.tp.world > 1
+        if isinstance(M, ClampedGlu):
+            return ops.linear(M.down, ops.linear_glu(M.gate_up, h, M.limit)), "full"
         if isinstance(M, DenseMlp):
             a = ops.linear_swiglu(M.gate_up, h, quant_for=M.down)
             return self._row_cut(M.down, a, a.rows if hasattr(a, "rows") else a.shape[0], fused)
@@ -791,7 +831,7 @@ class Model:
 
     def weight_bytes(self) -> int:
         n = 0
-        for L in self.layers:
+        for L in {id(L): L for L in self.layers}.values():       # layers may share their tensors
             for obj in (L.attn, L.gdn, L.mlp):
                 if obj is None:
                     continue

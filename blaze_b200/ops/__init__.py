@@ -10,9 +10,10 @@ import torch
 from .ref_ops import RefOps
 
 
-def get_ops(device, force_ref: bool = False):
+def get_ops(device, force_ref: bool = False, sources=None):
+    """``sources``: the kernel sources the caller launches from (None: all), see ``_native.kernels``."""
     dev = torch.device(device)
     if dev.type != "cuda" or force_ref:
         return RefOps()
     from .cuda_ops import CudaOps  # raises when the extension cannot be loaded
-    return CudaOps(dev)
+    return CudaOps(dev, sources)

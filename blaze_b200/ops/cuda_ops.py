@@ -31,13 +31,30 @@ def _ptr(t: Optional[torch.Tensor]) -> VP:
     return VP(0) if t is None else VP(t.data_ptr())
 
 
+class _Symbols:
+    """Entry points of a kernel library for declaring their types; those the library does not have are ignored here (calling one
+    raises)."""
+
+    class _Missing:
+        restype = argtypes = None
+
+    def __init__(self, lib):
+        self._lib = lib
+
+    def __getattr__(self, name):
+        try:
+            return getattr(self._lib, name)
+        except AttributeError:
+            return self._Missing()
+
+
 class CudaOps:
     is_cuda = True
     name = "sm100a"
 
-    def __init__(self, device):
+    def __init__(self, device, sources=None):
         self.device = torch.device(device)
-        self.lib = kernels()
+        self.lib = kernels(sources)
         self.launches = 0
         self._held_stream = None
         self._held_depth = 0
@@ -45,10 +62,10 @@ class CudaOps:
         self._scratch: Dict[str, torch.Tensor] = {}
         self._retired: list = []
         self._sm = torch.cuda.get_device_properties(self.device).multi_processor_count
-        lib = self.lib
+        lib = _Symbols(self.lib)           # a library of one model family has some of the entry points only
         lib.blz_gemm_tc.restype = _c.c_int
         lib.blz_gemm_tc.argtypes = [_c.c_int, VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_longlong, _c.c_int, _c.c_int,
-                                    _c.c_int, VP, VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_int, VP, _c.c_int, _c.c_int, _c.c_int, VP]
+                                    _c.c_int, VP, VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_int, VP, _c.c_int, _c.c_int, _c.c_int, _c.c_float, VP]
         lib.blz_gemm_wait_flags.restype = _c.c_int
         lib.blz_gemm_wait_flags.argtypes = [VP, VP, _c.c_int, _c.c_int]
         lib.blz_gemm_argmax_parts.argtypes = [VP, VP]
@@ -56,10 +73,10 @@ class CudaOps:
         lib.blz_gemm_wide.restype = _c.c_int
         lib.blz_gemm_wide.argtypes = [_c.c_int, VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_longlong, _c.c_int, _c.c_int,
                                       _c.c_int, VP, VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_int, VP, _c.c_longlong, VP,
-                                      _c.c_int, _c.c_int, _c.c_int, VP]
+                                      _c.c_int, _c.c_int, _c.c_int, _c.c_float, VP]
         lib.blz_gemm_sk.restype = _c.c_int
         lib.blz_gemm_sk.argtypes = [_c.c_int, VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_longlong, _c.c_int, _c.c_int,
-                                    _c.c_int, VP, VP, VP, VP, VP, _c.c_int, _c.c_int, VP]
+                                    _c.c_int, VP, VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_float, VP]
         lib.blz_gemm_fp8_block.restype = _c.c_int
         lib.blz_gemm_fp8_block.argtypes = [VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_longlong, _c.c_int, _c.c_int, _c.c_int,
                                            VP, _c.c_longlong, VP, VP, _c.c_int, VP]
@@ -106,7 +123,7 @@ class CudaOps:
                                      _c.c_int, VP, VP, VP, VP, VP, VP, _c.c_int, VP]
         lib.blz_gemm_narrow.restype = _c.c_int
         lib.blz_gemm_narrow.argtypes = [_c.c_int, VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_longlong, _c.c_int, _c.c_int, _c.c_int,
-                                        VP, VP, VP, VP, VP, _c.c_int, _c.c_int, VP]
+                                        VP, VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_float, VP]
         # dense layers with few rows (single-user decoding, verify steps) and a large weight take the features-on-lanes kernel
         # with the K range split over a cluster (blz_gemm_narrow).  Measured on B200, NVFP4, captured-graph timing, against the
         # one-CTA-per-tile kernel: 1-32 rows 24576x4096 21 -> 16 us, 4096x12288 19 -> 16 us, 17408x5120 18 -> 16 us, 6144x4096
@@ -143,6 +160,18 @@ class CudaOps:
         lib.blz_status_take.restype = _c.c_int
         lib.blz_status_peek_async.restype = _c.c_int
         lib.blz_status_peek_async.argtypes = [VP, VP]
+        # static residual streams, differential attention, 32-bit products
+        lib.blz_streams.argtypes = [VP, VP, VP, _c.c_int, _c.c_float, VP, VP, VP, VP, VP, _c.c_float, VP, VP, _c.c_int, _c.c_int, _c.c_int,
+                                    _c.c_int, _c.c_int, _c.c_int, VP]
+        lib.blz_norm_rows.argtypes = [VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_float, _c.c_int, VP]
+        lib.blz_gemm_simple.argtypes = [VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_int, _c.c_int, _c.c_int, _c.c_int,
+                                        _c.c_int, VP]
+        lib.blz_clamped_glu.argtypes = [VP, VP, _c.c_int, _c.c_int, _c.c_float, _c.c_int, VP]
+        lib.blz_diff_store.argtypes = [VP, _c.c_longlong, VP, _c.c_longlong, _c.c_longlong, VP] + [_c.c_int] * 6 + [VP]
+        common = [VP, _c.c_longlong, VP, VP, _c.c_longlong, _c.c_longlong, VP, _c.c_int, VP, VP, VP]
+        shape = [_c.c_int] * 7 + [_c.c_float] * 4
+        lib.blz_diff_plain.argtypes = common + [VP] + shape + [_c.c_int, VP]
+        lib.blz_diff_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
 
     # ------------------------------------------------------------------ plumbing
     def _stream(self) -> VP:
@@ -244,6 +273,11 @@ class CudaOps:
         def perm(t):
             return t if (order is None or t is None) else t.to(dev)[order]
 
+        if lin.fmt == Format.DENSE and lin.w.dtype == torch.float32:
+            if order is not None:
+                raise CudaError("32-bit weights are not interleaved: their gated activation is an op of its own")
+            return {"kind": 5, "w": lin.w.to(dev).contiguous(), "sf": None, "alpha": None,
+                    "bias": None if lin.bias is None else lin.bias.to(dev, torch.float32).contiguous()}
         if lin.fmt == Format.DENSE:
             pk = {"kind": 0, "w": perm(lin.w.to(dev, torch.bfloat16)).contiguous(), "sf": None, "alpha": None}
         elif lin.fmt == Format.NVFP4:
@@ -353,9 +387,39 @@ class CudaOps:
         act = self.linear(lin, x, swiglu=True)
         return self.quantize_rows(act, quant_for) if self._qmode(quant_for) else act
 
+    def _linear_simple(self, lin, pk, x, f32: bool, out=None):
+        """``x @ W^T`` on the CUDA cores: 32-bit weights, and bf16 rows too ragged for the TMA kernels."""
+        in32 = pk["kind"] == 5
+        if x.dtype != (torch.float32 if in32 else torch.bfloat16):
+            raise CudaError(f"{x.dtype} activations for {pk['w'].dtype} weights")
+        x = x.contiguous()
+        M = x.shape[0]
+        if out is None:
+            out = torch.empty(M, lin.N, dtype=torch.float32 if f32 else torch.bfloat16, device=self.device)
+        if M == 0:
+            return out
+        bias = pk["bias"].float() if pk["bias"] is not None else None
+        self._check(self.lib.blz_gemm_simple(_ptr(x), lin.K, _ptr(pk["w"]), lin.K, _ptr(out), out.stride(0), _ptr(bias), M, lin.N, lin.K,
+                                             int(in32), int(f32), self._stream()), "gemm_simple")
+        return out
+
+    def linear_glu(self, lin: Linear, x, limit: float):
+        """``g * sigmoid(1.702 g) * (u + 1)`` with ``g = min(x @ Wg^T, limit)`` and ``u`` = ``x @ Wu^T`` clamped to ``+-limit``, for a
+        stacked ``[gate; up]`` weight: in the GEMM's epilogue (fp32 accumulators) where the shape allows."""
+        if lin.w.dtype != torch.float32 and lin.N % 32 == 0 and lin.K % 16 == 0:
+            return self.linear(lin, x, swiglu=True, glu_limit=limit)
+        gu = self.linear(lin, x)
+        T, I = gu.shape[0], lin.N // 2
+        out = torch.empty(T, I, dtype=gu.dtype, device=self.device)
+        if T:
+            self._check(self.lib.blz_clamped_glu(_ptr(gu), _ptr(out), T, I, limit, int(gu.dtype == torch.float32), self._stream()), "clamped_glu")
+        return out
+
     def linear_argmax(self, lin: Linear, x, index_offset: int = 0, want_values: bool = False):
         """``argmax(x @ W^T)`` per row without writing the logits: the GEMM epilogue keeps the best (value, column) of each
         128-column tile and a small kernel merges the tiles (ties to the lower column, like ``argmax``)."""
+        if self.pack(lin)["kind"] == 5 or lin.K % 16:
+            return self.argmax(self.linear(lin, x, out_dtype=torch.float32), index_offset, want_values)
         M = x.rows if isinstance(x, QuantAct) else x.shape[0]
         tiles = (lin.N + 127) // 128
         val = self._buf("amax_val", tiles * max(M, 1) * 4).view(torch.float32)
@@ -393,12 +457,19 @@ class CudaOps:
         return out
 
     def linear(self, lin: Linear, x, out_dtype=None, out: Optional[torch.Tensor] = None, bn: int = 0, max_ctas: int = 0,
-               wide: Optional[bool] = None, ksplit: int = 0, swiglu: bool = False, argmax_parts=None, sk=None):
+               wide: Optional[bool] = None, ksplit: int = 0, swiglu: bool = False, argmax_parts=None, sk=None,
+               glu_limit: Optional[float] = None):
         """``wide``: None = choose; False = the 128-column kernel (needed by the fused all-reduce epilogue); True = insist on
         the wide-N kernel (raises when the shape is not covered).  ``sk``: None = choose; False = never; True or a K-slice
-        count 1..8 = the cluster split-K kernel (bf16 output, row-major weights)."""
+        count 1..8 = the cluster split-K kernel (bf16 output, row-major weights).  ``swiglu`` with ``glu_limit``: the clamped
+        gated activation instead of SwiGLU."""
         pk = self.pack(lin, swiglu=swiglu)
         kind = pk["kind"]
+        act, limit = int(swiglu) if glu_limit is None else 2, float(glu_limit or 0.0)
+        if kind == 5 or (kind == 0 and lin.K % 16):
+            if swiglu or argmax_parts is not None:
+                raise CudaError("the CUDA-core GEMM has the plain epilogue only")
+            return self._linear_simple(lin, pk, x, kind == 5 or out_dtype == torch.float32, out)
         f32 = out_dtype == torch.float32
         n_out = lin.N // 2 if swiglu else lin.N
         sfa = rs = None
@@ -446,7 +517,7 @@ class CudaOps:
                   and (not swiglu or ld_out % 8 == 0) and (sfa is None or sfa.numel() >= 512))
         if narrow:
             self._check(self.lib.blz_gemm_narrow(kind, _ptr(a), lda, _ptr(w), ldb, _ptr(out), ld_out, M, lin.N, lin.K, _ptr(rs),
-                                                 _ptr(pk["alpha"]), _ptr(pk["bias"]), _ptr(sfa), _ptr(pk["sf"]), 0, int(swiglu),
+                                                 _ptr(pk["alpha"]), _ptr(pk["bias"]), _ptr(sfa), _ptr(pk["sf"]), 0, act, limit,
                                                  self._stream()), f"gemm_narrow kind {kind}")
             return out
         sk_able = not f32 and argmax_parts is None and pending is None and not kt
@@ -470,7 +541,7 @@ class CudaOps:
             ks = 0 if sk is True else int(sk)
             self._check(self.lib.blz_gemm_sk(kind, _ptr(a), lda, _ptr(w), ldb, _ptr(out), ld_out, M, lin.N, lin.K,
                                              _ptr(rs), _ptr(pk["alpha"]), _ptr(pk["bias"]), _ptr(sfa), _ptr(pk["sf"]),
-                                             ks, int(swiglu), self._stream()), f"gemm_sk kind {kind}")
+                                             ks, act, limit, self._stream()), f"gemm_sk kind {kind}")
             return out
         if wide is None:
             # Measured on B200 (Qwen3-8B shapes, captured-graph timing): 256-feature tiles win for block-scaled prefill GEMMs
@@ -498,7 +569,7 @@ class CudaOps:
             self._check(self.lib.blz_gemm_wide(kind, _ptr(a), lda, _ptr(w), ldb, _ptr(out), out.stride(0), M, lin.N, lin.K,
                                                _ptr(rs), _ptr(pk["alpha"]), _ptr(pk["bias"]), _ptr(sfa), _ptr(pk["sf"]),
                                                int(f32), int(swap), ks, _ptr(ws), self.WIDE_WS_BYTES if ws is not None else 0,
-                                               _ptr(ctr), max_ctas, kt, int(swiglu), self._stream()), f"gemm_wide kind {kind}")
+                                               _ptr(ctr), max_ctas, kt, act, limit, self._stream()), f"gemm_wide kind {kind}")
             return out
         if argmax_parts is not None:
             rc = self.lib.blz_gemm_argmax_parts(_ptr(argmax_parts[0]), _ptr(argmax_parts[1]))
@@ -506,7 +577,7 @@ class CudaOps:
                 raise CudaError(f"blz_gemm_argmax_parts failed: {rc}")
         self._check(self.lib.blz_gemm_tc(kind, _ptr(a), lda, _ptr(w), ldb, _ptr(out), ld_out, M, lin.N, lin.K,
                                          _ptr(rs), _ptr(pk["alpha"]), _ptr(pk["bias"]), _ptr(sfa), _ptr(pk["sf"]),
-                                         int(f32), bn, max_ctas, VP(0), 0, kt, int(swiglu), self._stream()), f"gemm kind {kind}")
+                                         int(f32), bn, max_ctas, VP(0), 0, kt, act, limit, self._stream()), f"gemm kind {kind}")
         return out
 
     def silu_mul(self, gu, quant_for: Optional[Linear] = None):
@@ -651,6 +722,93 @@ class CudaOps:
                 self.launches += 1
         return out.view(T, Hq * D)
 
+    # ------------------------------------------------------------------ static residual streams
+    def streams_begin(self, table, tokens, scale: float, n: int):
+        """All ``n`` streams equal to the scaled embedding rows (read from the table where they are needed, not copied)."""
+        return (table, tokens, scale, n)
+
+    def _streams(self, src, y, prev, nxt, norm_w, eps, T, W, want_sum: bool, keep: bool):
+        from_embed = isinstance(src, tuple)
+        dt = torch.float32 if (src[0] if from_embed else y).dtype == torch.float32 else torch.bfloat16
+        if from_embed:
+            table, tokens, scale, S = src
+            streams = torch.empty(T, S, W, dtype=torch.float32, device=self.device) if keep else None
+        else:
+            table, tokens, scale, streams = None, None, 1.0, src
+            S = src.shape[1]
+        h = torch.empty(T, W, dtype=dt, device=self.device) if nxt is not None else None
+        total = torch.empty(T, W, dtype=torch.float32, device=self.device) if want_sum else None
+        self._check(self.lib.blz_streams(_ptr(streams), _ptr(table), _ptr(tokens), table.shape[0] if from_embed else 0, scale, _ptr(y),
+                                         _ptr(prev.mix if prev is not None else None), _ptr(prev.out if prev is not None else None),
+                                         _ptr(nxt.read if nxt is not None else None), _ptr(norm_w), eps, _ptr(h), _ptr(total), T, S, W,
+                                         int(from_embed), int(keep), int(dt == torch.float32), self._stream()), "streams")
+        return streams if keep else src, h, total
+
+    def streams_step(self, src, y, prev, nxt, norm_w, eps):
+        """Write the last sublayer's output ``y`` through ``prev``'s mix into the streams (``y`` None: there was none yet), then read
+        and normalise the next sublayer's input; returns (streams, input)."""
+        T, W = (src[1].numel(), src[0].shape[1]) if isinstance(src, tuple) else (src.shape[0], src.shape[2])
+        streams, h, _ = self._streams(src, y, prev, nxt, norm_w, eps, T, W, False, y is not None)
+        return streams, h
+
+    def streams_sum(self, src, y, prev):
+        """The sum of the streams after the sublayer whose output is ``y``, fp32 ``[T, W]``."""
+        T, W = (src[1].numel(), src[0].shape[1]) if isinstance(src, tuple) else (src.shape[0], src.shape[2])
+        return self._streams(src, y, prev, None, None, 0.0, T, W, True, False)[2]
+
+    def norm_rows(self, x, rows, w, eps, dtype):
+        """RMS norm of fp32 rows (those named by ``rows``) to ``dtype``."""
+        R = x.shape[0] if rows is None else rows.numel()
+        out = torch.empty(R, x.shape[1], dtype=dtype, device=self.device)
+        if R:
+            rows = None if rows is None else rows.to(torch.int32)
+            self._check(self.lib.blz_norm_rows(_ptr(x), _ptr(rows), _ptr(w), _ptr(out), R, x.shape[1], eps, int(dtype == torch.float32),
+                                               self._stream()), "norm_rows")
+        return out
+
+    # ------------------------------------------------------------------ differential attention
+    DIFF_SHORT_ROWS = 64       # sequences with new tokens * group up to this take the short-row kernel
+
+    def diff_attention(self, qkv, A, batch, kv, layer_idx, eps):
+        """Page write and differential attention of one layer; ``[T, heads * vdim]``, every head normed and scaled."""
+        a = A.spec
+        T = qkv.shape[0]
+        f32 = qkv.dtype == torch.float32
+        pool = kv.kv[layer_idx]
+        if kv.layout != "tiles" or pool.dtype != qkv.dtype:
+            raise CudaError(f"differential attention of {qkv.dtype} rows needs 'tiles' pages of that type")
+        out = torch.empty(T, a.heads * a.vdim, dtype=qkv.dtype, device=self.device)
+        B, bt = batch.slots.numel(), kv.block_table
+        st = self._stream()
+        self._check(self.lib.blz_diff_store(_ptr(qkv), qkv.stride(0), _ptr(pool), pool.stride(0), pool.stride(1), _ptr(batch.slot_mapping), T,
+                                            a.heads, a.kv_heads, a.dim, a.vdim, int(f32), st), "diff_store")
+        common = (_ptr(qkv), qkv.stride(0), _ptr(out), _ptr(pool), pool.stride(0), pool.stride(1), _ptr(bt), bt.stride(0),
+                  _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len))
+        shape = (T, B, a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.scale, A.lam, 1.0 - a.diff, eps)
+        if f32 or a.dim > 128 or a.vdim > 128:
+            self._check(self.lib.blz_diff_plain(*common, _ptr(batch.seq_of_row), *shape, int(f32), st), "diff_plain")
+            return out
+        group = a.group
+        lens = [(b - s) * group for s, b in zip(batch.h_q_start, batch.h_q_start[1:])]
+        small = [n for n in lens if 0 < n <= self.DIFF_SHORT_ROWS]
+        limit = self.DIFF_SHORT_ROWS
+        if len(small) < sum(1 for n in lens if n > 0):
+            small, limit = lens, 0x7FFFFFFF
+        if small:
+            rb = (max(small) + 15) // 16
+            toks = (max(small) + group - 1) // group
+            keys = min(batch.max_ctx, a.window + toks - 1) if a.window else batch.max_ctx
+            work = len(small) * a.kv_heads * rb
+            sp = max(1, min(4 * self._sm // work, (keys + 127) // 128, 32))
+            po = pm = None
+            if sp > 1:
+                n = B * a.kv_heads * rb * sp * 32
+                po = self._buf("diff_part_o", n * 128 * 4).view(torch.float32)
+                pm = self._buf("diff_part_ml", n * 2 * 4).view(torch.float32)
+                self.launches += 1
+            self._check(self.lib.blz_diff_short(*common, *shape, limit, rb, sp, _ptr(po), _ptr(pm), st), "diff_short")
+        return out
+
     # ------------------------------------------------------------------ head
     def argmax(self, logits, index_offset: int = 0, want_values: bool = False):
         R, V = logits.shape
@@ -715,7 +873,7 @@ class CudaOps:
         w = pk["w"]
         self._check(self.lib.blz_gemm_tc(kind, _ptr(data), lda, _ptr(w), w.shape[1] * w.element_size(), _ptr(out), out.stride(0),
                                          M_pad, pk["N"], pk["K"], _ptr(rs), _ptr(pk["alpha"]), VP(0), _ptr(sfa), _ptr(pk["sf"]),
-                                         0, 128, 0, _ptr(tile_expert), n_exp, 0, 0, self._stream()), "grouped gemm")
+                                         0, 128, 0, _ptr(tile_expert), n_exp, 0, 0, 0.0, self._stream()), "grouped gemm")
         return out
 
     def moe(self, x, topk_w, topk_id, experts):

@@ -174,7 +174,50 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     return out.to(q.dtype)
 
 
+def diff_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor, slots, q_start, ctx_len,
+                   scale: float, window: int, lam: float, post: float, eps: float) -> torch.Tensor:
+    """Differential attention of q ``[T, H, 2, d]``: per head two causal softmax maps (``window`` > 0: over the last ``window``
+    positions) on the keys ``[pages, 2 * G, 16, d]``, both over the values ``[pages, G, 16, e]``; the head's output is the
+    RMS-normed ``map 1 - lam * map 2`` times ``post``.  fp32 ``[T, H, e]``."""
+    T, H, _, d = q.shape
+    G, e = v_pool.shape[1], v_pool.shape[3]
+    out = torch.zeros(T, H, e, dtype=torch.float32, device=q.device)
+    for b, slot in enumerate(slots):
+        r0, r1 = q_start[b], q_start[b + 1]
+        ql, n = r1 - r0, ctx_len[b]
+        if ql <= 0:
+            continue
+        lo = max(n - ql - window + 1, 0) // PAGE if window else 0             # first page any of the rows can see
+        pages = block_table[slot, lo:(n + PAGE - 1) // PAGE].long()
+        m, base = n - lo * PAGE, lo * PAGE
+        K = k_pool[pages].float().permute(1, 0, 2, 3).reshape(G, 2, -1, d)[:, :, :m]
+        V = v_pool[pages].float().permute(1, 0, 2, 3).reshape(G, -1, e)[:, :m]
+        s = torch.einsum("qghmd,gmnd->gmhqn", q[r0:r1].float().view(ql, G, H // G, 2, d), K) * scale
+        pq = torch.arange(n - ql, n, device=q.device).view(ql, 1)
+        pk = torch.arange(base, n, device=q.device).view(1, m)
+        seen = pk <= pq
+        if window:
+            seen = seen & (pk > pq - window)
+        a = torch.einsum("gmhqn,gne->gmhqe", torch.softmax(s.masked_fill(~seen, float("-inf")), -1), V)
+        o = a[:, 0] - lam * a[:, 1]                                           # [G, h, q, e]
+        o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * post
+        out[r0:r1] = o.permute(2, 0, 1, 3).reshape(ql, H, e)
+    return out
+
+
+def streams_write(x: torch.Tensor, mix: torch.Tensor, out: torch.Tensor, y: torch.Tensor) -> torch.Tensor:
+    """Residual streams ``[T, S, W]`` after a sublayer: ``mix[from, to]`` of the old ones plus ``out[to] * y``."""
+    return torch.einsum("ab,taw->tbw", mix, x) + out.view(1, -1, 1) * y.float()[:, None]
+
+
 # ----------------------------------------------------------------------------------- MLP / MoE
+def clamped_glu(gu: torch.Tensor, limit: float) -> torch.Tensor:
+    """``[T, 2I]`` = ``[gate | up]`` -> ``g * sigmoid(1.702 g) * (u + 1)``, g = min(gate, limit), u = up clamped to +-limit."""
+    I = gu.shape[-1] // 2
+    g, u = gu[..., :I].clamp(max=limit), gu[..., I:].clamp(-limit, limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1)
+
+
 def silu_mul(gu: torch.Tensor) -> torch.Tensor:
     """``[T, 2I]`` laid out as ``[gate | up]`` → ``silu(gate) * up`` in the input dtype."""
     I = gu.shape[-1] // 2

@@ -81,6 +81,37 @@ class RefOps:
                                 tree_mask=getattr(batch, "tree_mask", None), allowed=allowed)
         return o.reshape(q.shape[0], -1)
 
+    # -------------------------------------------------------------- clamped GLU, static streams, differential attention
+    def linear_glu(self, lin: Linear, x, limit: float):
+        return ref.clamped_glu(self.linear(lin, x, torch.float32), limit).to(x.dtype)
+
+    def streams_begin(self, table, tokens, scale: float, n: int):
+        return (table[tokens.long()].float() * scale)[:, None].repeat(1, n, 1)
+
+    def streams_step(self, src, y, prev, nxt, norm_w, eps):
+        if y is not None:
+            src = ref.streams_write(src, prev.mix, prev.out, y)
+        u = torch.einsum("s,tsw->tw", nxt.read, src)
+        return src, self.norm_rows(u, None, norm_w, eps, nxt.dtype)
+
+    def streams_sum(self, src, y, prev):
+        return (ref.streams_write(src, prev.mix, prev.out, y) if y is not None else src).sum(1)
+
+    def norm_rows(self, x, rows, w, eps, dtype):
+        x = x if rows is None else x[rows.long()]
+        return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w).to(dtype)
+
+    def diff_attention(self, qkv, A, batch, kv, layer_idx, eps):
+        a = A.spec
+        T = qkv.shape[0]
+        nq, nk = a.heads * 2 * a.dim, a.kv_heads * 2 * a.dim
+        valid = batch.slot_mapping >= 0
+        ref.kv_write(kv.k[layer_idx], kv.v[layer_idx], qkv[valid, nq:nq + nk].reshape(-1, 2 * a.kv_heads, a.dim),
+                     qkv[valid, nq + nk:].reshape(-1, a.kv_heads, a.vdim), batch.slot_mapping[valid])
+        o = ref.diff_attention(qkv[:, :nq].reshape(T, a.heads, 2, a.dim), kv.k[layer_idx], kv.v[layer_idx], kv.block_table, batch.h_slots,
+                               batch.h_q_start, batch.h_ctx_len, a.scale, a.window, A.lam, 1.0 - a.diff, eps)
+        return o.reshape(T, -1).to(qkv.dtype)
+
     # -------------------------------------------------------------- MoE
     def router_topk(self, logits, k, renorm=True):
         return ref.router_topk(logits, k, renorm)

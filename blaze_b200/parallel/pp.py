@@ -36,6 +36,8 @@ def split_step(chunks: Sequence[SeqChunk], pp_chunk: int) -> List[List[SeqChunk]
     micro-batches run in order on every stage); only the piece that holds a chunk's last rows keeps its logit rows.
     Draft-tree and deferred-state chunks are never cut."""
     pp_chunk = max(int(pp_chunk), 1)
+    if any(c.logit_at is not None for c in chunks):
+        raise ValueError("pipeline stages return logits of the last rows of a chunk only")
     out: List[List[SeqChunk]] = []
     cur: List[SeqChunk] = []
     room = pp_chunk

@@ -46,7 +46,7 @@ class Leader:
         for r in gone:
             del self._sent[r]
         hid = None if hidden_in is None else (tuple(hidden_in.shape), str(hidden_in.dtype).replace("torch.", ""))
-        plan = ("step", mode, [(c.slot, list(c.tokens), c.start_pos, c.want_logits, c.parents, c.defer_state) for c in chunks],
+        plan = ("step", mode, [(c.slot, list(c.tokens), c.start_pos, c.want_logits, c.parents, c.defer_state, c.logit_at) for c in chunks],
                 changed, gone, feedback, self.tag, hid)
         self.group.broadcast_object(plan, 0)
         if hidden_in is not None:
@@ -104,7 +104,7 @@ def follow(llm) -> int:
                 s.pages = list(pg)
         for row in gone:
             eng.seqs.pop(row, None)
-        chunks = [SeqChunk(slot, toks, start, want, parents=parents, defer_state=defer) for slot, toks, start, want, parents, defer in raw]
+        chunks = [SeqChunk(slot, toks, start, want, parents=parents, defer_state=defer, logit_at=at) for slot, toks, start, want, parents, defer, at in raw]
         for c in chunks:                      # the follower's sequence lengths follow the plan (tree commits read them)
             s = eng.seqs.get(c.slot)
             if s is not None:

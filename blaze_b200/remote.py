@@ -43,6 +43,8 @@ def put_plan(chunks) -> bytes:
     """SeqChunk list → bytes: count, then per chunk (slot, start_pos, want_logits, n, tokens…)."""
     out = [struct.pack("<i", len(chunks))]
     for c in chunks:
+        if c.logit_at is not None:
+            raise ValueError("a remote stage returns logits of the last rows of a chunk only")
         toks = np.asarray(c.tokens, dtype=np.int32)
         out.append(struct.pack("<iiii", c.slot, c.start_pos, c.want_logits, toks.size))
         out.append(toks.tobytes())

@@ -1106,7 +1106,7 @@ class Scheduler:
         if cfg.spec_method == "ngram":
             eng = self.engine
             group = max(eng.model.cfg.num_heads // max(eng.model.cfg.num_kv_heads, 1), 1)
-            tree_rows = min(32, max(64 // group, 1)) if (cfg.draft_tree_width > 1 and not eng.kv.gdn_layers) else 0
+            tree_rows = min(32, max(64 // group, 1)) if (cfg.draft_tree_width > 1 and eng.trees_ok) else 0
             for a, k in zip(decoders, want):
                 if k <= 0:
                     continue
@@ -1128,7 +1128,7 @@ class Scheduler:
                         out[id(a)] = d
         elif self.drafter is not None:
             reqs = [(a, k) for a, k in zip(decoders, want) if k > 0]
-            if reqs and cfg.draft_tree_width > 1 and hasattr(self.drafter, "propose_tree") and not self.engine.kv.gdn_layers:
+            if reqs and cfg.draft_tree_width > 1 and hasattr(self.drafter, "propose_tree") and self.engine.trees_ok:
                 # trees grown by the drafter itself (EAGLE): verified with the tree rows of the target's attention
                 eng = self.engine
                 group = max(eng.model.cfg.num_heads // max(eng.model.cfg.num_kv_heads, 1), 1)

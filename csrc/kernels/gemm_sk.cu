@@ -18,6 +18,7 @@
 // Reference counterparts: the split-K small-m kernels of kernels/src/cuda/nvfp4_linear.cu (nvfp4_mma_kernel :185, split
 // over warps with a shared-memory reduce; tuner-chosen split :523), fp8_linear.cu :40/:159/:270, and the GEMM router
 // crates/blaze/src/linear.rs:535-760.
+#include "blaze/glu.cuh"
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
 
@@ -35,6 +36,7 @@ struct SkParams {
   int sf_col_tiles;          // 4-column scale tiles per 128-row tile along K
   int ks;                    // cluster size = number of K slices
   int act;                   // 1: B rows are [16 gate | 16 up] groups, C = silu(gate) * up, bf16 [M, N/2] (ks must be 1)
+  float act_limit;           // act 2: the clamp of glu.cuh
   int* status;
   unsigned* dbg;             // optional [gridDim.x] progress bits per CTA (diagnostics; null = off)
   unsigned long long* prof;  // optional [gridDim.x][16] time stamps per CTA (diagnostics; null = off)
@@ -255,7 +257,8 @@ gemm_sk_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
         __nv_bfloat16* dst = p.C + (size_t)row * p.ldc + col0 / 2;
         uint32_t pk[8];
 #pragma unroll
-        for (int i = 0; i < 16; i += 2) pk[i / 2] = pack_bf16x2(silu_mul_bf16(v[i], v[16 + i]), silu_mul_bf16(v[i + 1], v[17 + i]));
+        for (int i = 0; i < 16; i += 2) pk[i / 2] = p.act == 2 ? pack_bf16x2(clamped_glu_fast(v[i], v[16 + i], p.act_limit), clamped_glu_fast(v[i + 1], v[17 + i], p.act_limit))
+                                                               : pack_bf16x2(silu_mul_bf16(v[i], v[16 + i]), silu_mul_bf16(v[i + 1], v[17 + i]));
         if (vec) {
           *reinterpret_cast<uint4*>(dst) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
           *reinterpret_cast<uint4*>(dst + 8) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
@@ -480,7 +483,7 @@ BLZ_API int blz_gemm_sk_coresident(int kind, int ks) {
 // blz_gemm_tc (needs ks <= 4, N % 32 == 0 and ldc % 8 == 0).
 BLZ_API int blz_gemm_sk(int kind, const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M,
                         int N, int K, const float* row_scale, const float* alpha, const void* bias, const void* sfa,
-                        const void* sfb, int ks, int act, cudaStream_t stream) {
+                        const void* sfb, int ks, int act, float act_limit, cudaStream_t stream) {
   using namespace blz;
   if (M <= 0 || N <= 0 || K <= 0 || kind < 0 || kind > 3 || ks < 0 || ks > 8) return (int)cudaErrorInvalidValue;
   const int kmma = kind == 0 ? 16 : kind == 1 ? 64 : 32;
@@ -496,7 +499,7 @@ BLZ_API int blz_gemm_sk(int kind, const void* A, long long lda, const void* B, l
   p.row_scale = row_scale; p.alpha = alpha; p.bias = reinterpret_cast<const __nv_bfloat16*>(bias);
   p.sfa = reinterpret_cast<const uint8_t*>(sfa); p.sfb = reinterpret_cast<const uint8_t*>(sfb);
   p.sf_col_tiles = kind == 1 ? (K + 63) / 64 : kind == 2 ? (K + 127) / 128 : 0;
-  p.ks = ks; p.act = act;
+  p.ks = ks; p.act = act; p.act_limit = act_limit;
   p.status = status_word();
   p.dbg = g_sk_dbg;
   g_sk_dbg = nullptr;

@@ -14,6 +14,7 @@
 // Covers what the reference spreads over kernels/src/cuda/nvfp4_gemm.cu (w4a4_kernel :114, sm_120a-only
 // mma.sync), nvfp4_linear.cu (gemv / small-m mma kernels :49-:320), fp8_linear.cu (:40, :159, :270) and the
 // cuBLAS call in gemm.cu:55.
+#include "blaze/glu.cuh"
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
 
@@ -63,6 +64,7 @@ struct GemmParams {
   float* amax_val;           // arg-max epilogue (fp32 instantiation): per (N tile, row) best value ...
   int* amax_idx;             // ... and its column; C is not written.  Layout [N tiles][M].
   int act;                   // 1: B rows are [16 gate | 16 up] groups; the epilogue writes silu(gate) * up, bf16 [M, N/2]
+  float act_limit;           // act 2: the clamp of glu.cuh
   int b_kt;                  // > 0: B is tile-major, [N/128][b_kt][16 KB shared-memory image of a 128-row x 128-byte tile]
   const uint8_t* b_raw;      // base of B for the tile-major form (fetched with plain bulk copies, one per tile)
   int* status;
@@ -360,9 +362,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
               float a[2];
 #pragma unroll
               for (int j = 0; j < 2; ++j) {
-                const float g = bf2f(__float2bfloat16(fmaf(__uint_as_float(r[i + j]) * rs, sal[c * 32 + i + j], sbi[c * 32 + i + j])));
-                const float u = bf2f(__float2bfloat16(fmaf(__uint_as_float(r[16 + i + j]) * rs, sal[c * 32 + 16 + i + j], sbi[c * 32 + 16 + i + j])));
-                a[j] = g / (1.f + __expf(-g)) * u;
+                const float gf = fmaf(__uint_as_float(r[i + j]) * rs, sal[c * 32 + i + j], sbi[c * 32 + i + j]);
+                const float uf = fmaf(__uint_as_float(r[16 + i + j]) * rs, sal[c * 32 + 16 + i + j], sbi[c * 32 + 16 + i + j]);
+                if (p.act == 2) {
+                  a[j] = clamped_glu_fast(gf, uf, p.act_limit);
+                } else {
+                  const float g = bf2f(__float2bfloat16(gf)), u = bf2f(__float2bfloat16(uf));
+                  a[j] = g / (1.f + __expf(-g)) * u;
+                }
               }
               pk[i / 2] = pack_bf16x2(a[0], a[1]);
             }
@@ -614,12 +621,13 @@ BLZ_API int blz_gemm_push_rs(void* const* slots, void* const* flags, void* done_
 
 // kind: 0 bf16, 1 nvfp4, 2 mxfp8, 3 fp8.  A [M, K] and B [N, K] row-major (packed bytes for 4/8-bit kinds);
 // lda / ldb in BYTES.  out_f32: C is fp32, else bf16; ldc in elements.  bn: 128 or 256 (0 = choose).
-// act = 1: B's rows come in groups of [16 gate | 16 up] features and C is bf16 [M, N/2] = silu(gate) * up (ldc % 8 == 0).
+// act = 1: B's rows come in groups of [16 gate | 16 up] features and C is bf16 [M, N/2] = silu(gate) * up (ldc % 8 == 0);
+// act = 2: the clamped form of glu.cuh with act_limit.
 // b_kt > 0: B is the tile-major repack [ceil(N/128)][b_kt][128][128 bytes] (zero padded), b_kt = ceil(row bytes / 128).
 BLZ_API int blz_gemm_tc(int kind, const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
                         int M, int N, int K, const float* row_scale, const float* alpha, const void* bias,
                         const void* sfa, const void* sfb, int out_f32, int bn, int max_ctas, const int* tile_expert,
-                        int num_experts, int b_kt, int act, cudaStream_t stream) {
+                        int num_experts, int b_kt, int act, float act_limit, cudaStream_t stream) {
   using namespace blz;
   // snapshot and clear the one-shot arming first: an early return below must not leave it armed for an unrelated GEMM
   const FuseArgs fuse = g_fuse;
@@ -649,6 +657,7 @@ BLZ_API int blz_gemm_tc(int kind, const void* A, long long lda, const void* B, l
   p.b_kt = b_kt;
   p.b_raw = reinterpret_cast<const uint8_t*>(B);
   p.act = act;
+  p.act_limit = act_limit;
   if (act && (out_f32 || N % 32 || (ldc & 7) || tile_expert)) return (int)cudaErrorInvalidValue;
   if (b_kt > 0 && tile_expert) return (int)cudaErrorInvalidValue;
   p.mc_out = nullptr; p.done_ctr = nullptr; p.epoch = nullptr; p.spin_limit = 0; p.rank = 0; p.world = 1;

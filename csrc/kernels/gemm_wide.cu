@@ -19,6 +19,7 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 
+#include "blaze/glu.cuh"
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
 
@@ -43,6 +44,7 @@ struct WideParams {
   float* ws;                  // [tiles * ksplit][128][BN] fp32 partial tiles (ksplit > 1)
   unsigned* ctr;              // [tiles] arrival counters, zero between launches
   int act;                    // 1 (plain orientation): columns are [16 gate | 16 up] groups; C = silu(gate) * up, bf16 [tokens, N/2]
+  float act_limit;           // act 2: the clamp of glu.cuh
   int w_kt;                   // > 0: the weight operand is tile-major, [rows/128][w_kt][16 KB swizzled tile image]
   const uint8_t* w_raw;       // its base (fetched with plain bulk copies)
   int* status;
@@ -371,9 +373,14 @@ __global__ void __launch_bounds__(320, 1) gemm_wide_kernel(const __grid_constant
 #pragma unroll
                 for (int j = 0; j < 2; ++j) {
                   const int cg = half * CPT + gq + i + j, cu = cg + 16;
-                  const float g = bf2f(__float2bfloat16(fmaf(__uint_as_float(r[gq + i + j]) * ls, s_cs[cg], s_cb[cg])));
-                  const float u = bf2f(__float2bfloat16(fmaf(__uint_as_float(r[gq + 16 + i + j]) * ls, s_cs[cu], s_cb[cu])));
-                  a[j] = g / (1.f + __expf(-g)) * u;
+                  const float gf = fmaf(__uint_as_float(r[gq + i + j]) * ls, s_cs[cg], s_cb[cg]);
+                  const float uf = fmaf(__uint_as_float(r[gq + 16 + i + j]) * ls, s_cs[cu], s_cb[cu]);
+                  if (p.act == 2) {
+                    a[j] = clamped_glu_fast(gf, uf, p.act_limit);
+                  } else {
+                    const float g = bf2f(__float2bfloat16(gf)), u = bf2f(__float2bfloat16(uf));
+                    a[j] = g / (1.f + __expf(-g)) * u;
+                  }
                 }
                 pk[i / 2] = pack_bf16x2(a[0], a[1]);
               }
@@ -451,7 +458,7 @@ BLZ_API int blz_gemm_wide_ksplit(int tiles, int k_tiles, int sms) {
 BLZ_API int blz_gemm_wide(int kind, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M,
                           int N, int K, const float* row_scale, const float* alpha, const void* bias, const void* sfx,
                           const void* sfw, int out_f32, int swap, int ksplit, void* ws, long long ws_bytes, void* ctr,
-                          int max_ctas, int w_kt, int act, cudaStream_t stream) {
+                          int max_ctas, int w_kt, int act, float act_limit, cudaStream_t stream) {
   using namespace blz;
   // this kernel has no fused all-reduce / peer-wait / arg-max epilogue: a call armed for one is refused (and disarmed)
   if (gemm_oneshot_take_unsupported()) return (int)cudaErrorNotSupported;
@@ -477,6 +484,7 @@ BLZ_API int blz_gemm_wide(int kind, const void* X, long long ldx, const void* W,
   p.w_kt = w_kt;
   p.w_raw = reinterpret_cast<const uint8_t*>(W);
   p.act = act;
+  p.act_limit = act_limit;
   if (act && (swap || out_f32 || (ldc & 7))) return (int)cudaErrorInvalidValue;
   const void *A, *B;
   long long lda, ldb;

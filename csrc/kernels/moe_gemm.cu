@@ -27,6 +27,7 @@
 // role can have failed yet.  No TMA load is cluster-multicast.
 //
 // Reference counterparts: kernels/src/cuda/moe_narrow.cu (per-expert small-m kernels, :171-484) and moe_wide.cu (:125-313).
+#include "blaze/glu.cuh"
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
 
@@ -48,6 +49,7 @@ struct MoeGemmParams {
   int ks;                    // cluster size = K slices (1 = no cluster)
   int ft_per;                // feature tiles one CTA computes one after the other (1 when ks > 1)
   int act;                   // 1: SwiGLU epilogue, C is [rows, N / 2]
+  float act_limit;           // act 2: the clamp of glu.cuh
   int* status;
 };
 
@@ -253,7 +255,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__
           if (j < n) {
             const float x = fmaf(v[j] * al, s_rs[c0 + j], bs);
             const float o = __shfl_xor_sync(0xffffffffu, x, 16);
-            if (lane < 16 && c0 + j < rows) p.C[((size_t)mt * 128 + c0 + j) * p.ldc + fo] = __float2bfloat16(mg_silu_mul(x, o));
+            if (lane < 16 && c0 + j < rows) p.C[((size_t)mt * 128 + c0 + j) * p.ldc + fo] = __float2bfloat16(p.act == 2 ? clamped_glu_fast(x, o, p.act_limit) : mg_silu_mul(x, o));
           }
         }
       } else {
@@ -406,7 +408,7 @@ BLZ_API int blz_moe_gemm(int kind, const void* X, long long ldx, const void* W, 
   p.row_scale = row_scale; p.alpha = alpha;
   p.sfw = reinterpret_cast<const uint8_t*>(sfw); p.sfx = reinterpret_cast<const uint8_t*>(sfx);
   p.sf_col_tiles = kind == 1 ? (K + 63) / 64 : kind == 2 ? (K + 127) / 128 : 0;
-  p.tile_expert = tile_expert; p.tile_rows = tile_rows; p.act = act;
+  p.tile_expert = tile_expert; p.tile_rows = tile_rows; p.act = act; p.act_limit = 0.f;
   p.rows = 0; p.bias = nullptr; p.ks = 1;
   {
     // feature tiles per CTA: long enough streams to amortise a CTA's set-up, still at least four CTAs per row tile
@@ -441,10 +443,10 @@ BLZ_API int blz_moe_gemm(int kind, const void* X, long long ldx, const void* W, 
 // Dense layer at small batch: C[M, N] = (X[M, K] · W[N, K]^T) * row_scale[m] * alpha[n] (+ bias[n]) for M <= 128 rows, features on
 // the MMA lanes, the K range split over a cluster of ks CTAs (0 = choose: enough CTAs to cover the SMs twice, at most 8 and at
 // most one K block each).  Rows past M are never read (the tensor map ends at row M, the copy engine fills zeros); the scale
-// factors of X must be a whole 128-row tile.  act as in blz_moe_gemm.
+// factors of X must be a whole 128-row tile.  act as in blz_moe_gemm, or 2: the clamped form of glu.cuh with act_limit.
 BLZ_API int blz_gemm_narrow(int kind, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M,
                             int N, int K, const float* row_scale, const float* alpha, const void* bias, const void* sfx,
-                            const void* sfw, int ks, int act, cudaStream_t stream) {
+                            const void* sfw, int ks, int act, float act_limit, cudaStream_t stream) {
   using namespace blz;
   if (M <= 0) return 0;
   if (M > 128 || N <= 0 || K <= 0 || kind < 0 || kind > 2 || N % 128 || ks < 0 || ks > 8) return (int)cudaErrorInvalidValue;
@@ -465,7 +467,7 @@ BLZ_API int blz_gemm_narrow(int kind, const void* X, long long ldx, const void* 
   p.sfw = reinterpret_cast<const uint8_t*>(sfw); p.sfx = reinterpret_cast<const uint8_t*>(sfx);
   p.sf_col_tiles = kind == 1 ? (K + 63) / 64 : kind == 2 ? (K + 127) / 128 : 0;
   p.tile_expert = nullptr; p.tile_rows = nullptr; p.rows = M; p.bias = reinterpret_cast<const __nv_bfloat16*>(bias);
-  p.ks = ks; p.act = act; p.ft_per = 1;
+  p.ks = ks; p.act = act; p.act_limit = act_limit; p.ft_per = 1;
   p.status = status_word();
   CUtensorMap tmW, tmX;
   cudaError_t e;

@@ -223,7 +223,7 @@ def test_gemm_narrow_small_batch(ops, fmt, M, N, K, ks):
     wt = pk["w"]
     for _ in range(2):
         rc = ops.lib.blz_gemm_narrow(pk["kind"], ptr(a), lda, ptr(wt), wt.shape[1] * wt.element_size(), ptr(out), out.stride(0), M, N, K,
-                                     ptr(rs), ptr(pk["alpha"]), ptr(pk["bias"]), ptr(sfa), ptr(pk["sf"]), ks, 0,
+                                     ptr(rs), ptr(pk["alpha"]), ptr(pk["bias"]), ptr(sfa), ptr(pk["sf"]), ks, 0, 0.0,
                                      VP(torch.cuda.current_stream().cuda_stream))
         assert rc == 0
     y_tc = ops.linear(lin, xin, wide=False, sk=False)
