@@ -171,6 +171,7 @@ class CudaOps:
         common = [VP, _c.c_longlong, VP, VP, _c.c_longlong, _c.c_longlong, VP, _c.c_int, VP, VP, VP]
         shape = [_c.c_int] * 7 + [_c.c_float] * 4
         lib.blz_diff_plain.argtypes = common + [VP] + shape + [_c.c_int, VP]
+        lib.blz_diff_tc.argtypes = common + shape + [_c.c_int, _c.c_int, VP]
         lib.blz_diff_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
 
     # ------------------------------------------------------------------ plumbing
@@ -785,15 +786,16 @@ class CudaOps:
         common = (_ptr(qkv), qkv.stride(0), _ptr(out), _ptr(pool), pool.stride(0), pool.stride(1), _ptr(bt), bt.stride(0),
                   _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len))
         shape = (T, B, a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.scale, A.lam, 1.0 - a.diff, eps)
-        if f32 or a.dim > 128 or a.vdim > 128:
+        group = a.group
+        if f32 or a.dim > 128 or a.vdim > 128 or group > 128 or a.scale <= 0:
             self._check(self.lib.blz_diff_plain(*common, _ptr(batch.seq_of_row), *shape, int(f32), st), "diff_plain")
             return out
-        group = a.group
-        lens = [(b - s) * group for s, b in zip(batch.h_q_start, batch.h_q_start[1:])]
-        small = [n for n in lens if 0 < n <= self.DIFF_SHORT_ROWS]
+        lens = [b - s for s, b in zip(batch.h_q_start, batch.h_q_start[1:])]
         limit = self.DIFF_SHORT_ROWS
-        if len(small) < sum(1 for n in lens if n > 0):
-            small, limit = lens, 0x7FFFFFFF
+        small = [n * group for n in lens if 0 < n * group <= limit]
+        items = sum(-(-n // (128 // group)) for n in lens if n * group > limit)
+        if items:
+            self._check(self.lib.blz_diff_tc(*common, *shape, limit, items, st), "diff_tc")
         if small:
             rb = (max(small) + 15) // 16
             toks = (max(small) + group - 1) // group
