@@ -1,0 +1,229 @@
+"""A model design beside its closest relative at equal size: prefill and decode throughput of a few layers of real size (random
+weights, bf16), and every kernel that is the design's own beside the like kernel of the relative, with fractions of the measured
+peaks.  ``bench.py --design sevevik`` runs it: Sevevik against the Qwen3 decoder (equal width, heads, projections and
+feed-forward; the relative keeps FP8 pages, its only format on a GPU).
+
+Device-timed with CUDA events; kernels in captured graphs over buffers that together exceed L2.
+"""
+from __future__ import annotations
+
+from typing import Callable, Dict, List
+
+import torch
+
+from ..config import DiffAttnSpec, GluSpec, LayerSpec, ModelConfig, RopeConfig
+from .kernels import peaks
+
+# width, query heads, key/value heads, feed-forward
+SIZES = {"2048": (2048, 16, 8, 6144), "4096": (4096, 32, 8, 12288)}
+WINDOW = 1024
+
+
+def configs(size: str, layers: int, vocab: int) -> Dict[str, ModelConfig]:
+    W, H, G, ff = SIZES[size]
+    a = DiffAttnSpec(heads=H, kv_heads=G, dim=64, vdim=128, scale=0.125, diff=0.5, window=WINDOW)
+    sev = ModelConfig.of_layers([LayerSpec(a, GluSpec(ff, 7.0)) for _ in range(layers)], architecture="Sevevik", model_type="sevevik",
+                                vocab_size=vocab, hidden_size=W, streams=4)
+    qwen = ModelConfig(vocab_size=vocab, hidden_size=W, num_layers=layers, num_heads=H, num_kv_heads=G, head_dim=128,
+                       intermediate_size=ff, rope=RopeConfig(theta=1e6), layer_types=["full_attention"] * layers)
+    return {"sevevik": sev, "qwen3": qwen}
+
+
+def _events(fn: Callable[[], None], reps: int) -> float:
+    """Median milliseconds of ``fn``."""
+    fn()
+    torch.cuda.synchronize()
+    t = []
+    for _ in range(reps):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        t.append(a.elapsed_time(b))
+    return sorted(t)[len(t) // 2]
+
+
+def throughput(cfg: ModelConfig, steps: int, warmup: int, batch: int = 256, ctx: int = 1024) -> Dict[str, float]:
+    """Prefill tokens/s (8 prompts of 1024 in one step; one prompt of 8192) and decode tokens/s at ``batch`` x ``ctx``."""
+    from ..llm import LLM
+    longest = 8192
+    llm = LLM(cfg, device="cuda", kv_tokens=max(batch * (ctx + steps + warmup + 64), 2 * longest), max_seqs=batch, max_model_len=longest + 64,
+              enable_prefix_caching=False, seed=1, chunk=8192)
+    eng, V = llm.engine, cfg.vocab_size
+    g = torch.Generator().manual_seed(1)
+    out: Dict[str, float] = {}
+
+    def prefill(n_seqs, n):
+        prompts = torch.randint(0, V, (n_seqs, n), generator=g).tolist()
+
+        def once():
+            seqs = [eng.open_from() for _ in range(n_seqs)]
+            eng.forward(eng.plan([(s, p, 1) for s, p in zip(seqs, prompts)]), "greedy")
+            for s in seqs:
+                eng.close(s)
+        ms = _events(once, 5)
+        return {"ms": round(ms, 3), "tok_s": round(n_seqs * n / ms * 1e3)}
+    out["prefill_8x1024"] = prefill(8, 1024)
+    out["prefill_1x8192"] = prefill(1, 8192)
+    seqs = [eng.open_from() for _ in range(batch)]
+    for i in range(0, batch, 8):
+        part = seqs[i:i + 8]
+        eng.forward(eng.plan([(s, torch.randint(0, V, (ctx,), generator=g).tolist(), 0) for s in part]), "none")
+    zeros = [0]
+
+    def decode(feedback):
+        return eng.forward(eng.plan([(s, zeros, 1) for s in seqs]), "greedy", feedback=feedback)
+    for k in range(max(warmup, 3)):
+        decode(False)
+    torch.cuda.synchronize()
+    feed = eng.can_feed_back(batch)
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(steps):
+        decode(feed)
+    b.record()
+    torch.cuda.synchronize()
+    ms = a.elapsed_time(b) / steps
+    wbytes = llm.model.weight_bytes() - llm.model.embed.numel() * llm.model.embed.element_size()
+    out["decode_%dx%d" % (batch, ctx)] = {"ms": round(ms, 4), "tok_s": round(batch / ms * 1e3), "weight_mb": round(wbytes / 1e6), "captured": feed}
+    one = seqs[:1]
+    for s in seqs[1:]:
+        eng.close(s)
+    for _ in range(4):
+        eng.forward(eng.plan([(one[0], zeros, 1)]), "greedy")
+    torch.cuda.synchronize()
+    a.record()
+    for _ in range(steps):
+        eng.forward(eng.plan([(one[0], zeros, 1)]), "greedy", feedback=eng.can_feed_back(1))
+    b.record()
+    torch.cuda.synchronize()
+    out["decode_1x%d" % ctx] = {"ms": round(a.elapsed_time(b) / steps, 4)}
+    eng.check_status()
+    del llm, eng
+    torch.cuda.empty_cache()
+    return out
+
+
+def _graph_ms(calls: List[Callable[[], object]], reps: int = 7) -> float:
+    """Milliseconds per call of a captured graph of ``calls`` (each on buffers of its own)."""
+    for c in calls:
+        c()
+    torch.cuda.synchronize()
+    keep = []
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for c in calls:
+            keep.append(c())
+    return _events(graph.replay, reps) / len(calls)
+
+
+def _attention(ops, cfg: ModelConfig, B: int, qlen: int, ctx: int, copies: int):
+    """(attention calls, page-write calls, bytes of keys and values read, flops) of one layer."""
+    from ..batch import SeqChunk, build_batch
+    from ..kv import KVCache
+    sev = bool(cfg.layer_specs)
+    per = (ctx + 15) // 16 + 1
+    cfg.num_layers = 1
+    kvs = [KVCache(cfg, 1 + B * per, B, per, "bf16" if sev else "fp8", "cuda", "tiles" if sev else "umma") for _ in range(copies)]
+    G = cfg.num_kv_heads
+    for kv in kvs:
+        perm = torch.randperm(B * per, generator=torch.Generator().manual_seed(0)).tolist()
+        for b in range(B):
+            kv.set_pages(b, [1 + p for p in perm[b * per:(b + 1) * per]])
+        if sev:
+            kv.kv[0].normal_()
+        else:
+            kv.kv[0].copy_(torch.randint(0, 120, kv.kv[0].shape, dtype=torch.uint8, device="cuda"))
+    chunks = [SeqChunk(b, [0] * qlen, ctx - qlen) for b in range(B)]
+    batch = build_batch(chunks, kvs[0].block_table_host, "cuda", attn_group=0 if sev else cfg.num_heads // G)
+    T, H = B * qlen, cfg.num_heads
+    seen = lambda i: min(i + 1, WINDOW) if sev else i + 1      # noqa: E731
+    keys = sum(seen(i) for i in range(ctx - qlen, ctx))        # of one sequence's rows
+    first = max(ctx - qlen - WINDOW + 1, 0) if sev else 0
+    for kv in kvs:
+        _ = kv.block_table
+    if sev:
+        class A:
+            spec, lam = cfg.layer_specs[0].attn, 0.6
+        a = A.spec
+        qkv = torch.randn(T, a.heads * 2 * a.dim + a.kv_heads * (2 * a.dim + a.vdim), device="cuda").bfloat16()
+        calls = [lambda kv=kv: ops.diff_attention(qkv, A, batch, kv, 0, 1e-6, store=False) for kv in kvs]
+        write = [lambda kv=kv: ops.diff_store(qkv, A, batch, kv, 0) for kv in kvs]
+        flops = 2.0 * B * H * keys * (2 * a.dim + 2 * a.vdim)
+        return calls, write, B * (ctx - first) * G * (2 * a.dim + a.vdim) * 2.0, flops, T * qkv.shape[1] * 2.0
+    D = cfg.head_dim
+
+    class M:
+        inv_freq, rope_scale, kv_rotate = torch.ones(D // 2, device="cuda"), 1.0, False
+
+    class N:
+        heads, kv_heads, q_norm, k_norm = H, G, torch.ones(D, device="cuda").bfloat16(), torch.ones(D, device="cuda").bfloat16()
+    M.cfg = cfg
+    q = torch.randn(T, H, D, device="cuda").bfloat16()
+    qkv = torch.randn(T, (H + 2 * G) * D, device="cuda").bfloat16()
+    calls = [lambda kv=kv: ops.attention(q, M, batch, kv, 0, D ** -0.5) for kv in kvs]
+    write = [lambda kv=kv: ops.attn_prep_store(qkv, N, M, batch, kv, 0, None) for kv in kvs]
+    return calls, write, B * ctx * G * 2.0 * D, 4.0 * B * H * keys * D, T * qkv.shape[1] * 2.0
+
+
+def kernels(size: str) -> List[Dict]:
+    from ..linear import Linear
+    from ..models.sevevik import StaticStreams
+    from ..ops import get_ops
+    ops, pk = get_ops("cuda"), peaks()
+    W, H, G, ff = SIZES[size]
+    rows: List[Dict] = []
+
+    def add(name, model, ms, nbytes=0.0, flops=0.0):
+        bound = max(nbytes / pk["hbm_gbs"] / 1e6, flops / pk["bf16_tflops"] / 1e9)
+        rows.append({"kernel": name, "model": model, "us": round(ms * 1e3, 2), "roofline_frac": round(bound / ms, 3),
+                     "bound": "hbm" if nbytes / pk["hbm_gbs"] / 1e6 >= flops / pk["bf16_tflops"] / 1e9 else "bf16 tensor"})
+    for name, B, qlen, ctx, copies in (("attention decode 256x1024", 256, 1, 1024, 2), ("attention decode 32x1024", 32, 1, 1024, 8),
+                                       ("attention prefill 4x1024", 4, 1024, 1024, 4), ("attention prefill 1x8192", 1, 8192, 8192, 2)):
+        for model, cfg in configs(size, 1, 1024).items():
+            calls, write, kvb, flops, rowb = _attention(ops, cfg, B, qlen, ctx, copies)
+            out = B * qlen * H * 128 * 2.0
+            add(name, model, _graph_ms(calls), kvb + out + B * qlen * H * 128 * 2.0, flops)
+            if qlen == 1024 or B == 256:
+                add("page write " + name.split(" ", 1)[1], model, _graph_ms(write), 2 * rowb if model == "qwen3" else 2.0 * B * qlen * G * 256 * 2)
+            del calls, write
+            torch.cuda.empty_cache()
+    for T in (256, 8192):
+        n = max(2, int(400e6 // (T * W * 16)))
+        S = 4
+        w = StaticStreams(torch.randn(S), torch.randn(S, S), torch.randn(S), 1.0, "cuda", torch.bfloat16)
+        nw = torch.ones(W, device="cuda")
+        y = torch.randn(T, W, device="cuda").bfloat16()
+        xs = [torch.randn(T, S, W, device="cuda") for _ in range(n)]
+        add(f"streams + norm, {T} rows", "sevevik", _graph_ms([lambda x=x: ops.streams_step(x, y, w, w, nw, 1e-6) for x in xs]),
+            T * W * (2 * 4 * S + 2 + 2))
+        del xs
+        n = max(2, int(400e6 // (T * W * 4)))
+        rs = [torch.randn(T, W, device="cuda").bfloat16() for _ in range(n)]
+        nb = nw.bfloat16()
+        add(f"residual + norm, {T} rows", "qwen3", _graph_ms([lambda r=r: ops.norm(y, r, nb, 1e-6) for r in rs]), T * W * (2 + 2 + 2 + 2))
+        del rs
+        x = torch.randn(T, W, device="cuda").bfloat16()
+        ws = torch.randn(2 * ff, W, device="cuda") * 0.02
+        copies = max(1, min(8, int(300e6 // (2 * ff * W * 2)) + 1))
+        for model in ("sevevik", "qwen3"):
+            lins = [Linear.from_dense(ws) for _ in range(copies)]
+            f = (lambda l: ops.linear_glu(l, x, 7.0)) if model == "sevevik" else (lambda l: ops.linear_swiglu(l, x))
+            add(f"gate/up GEMM + activation, {T} rows", model, _graph_ms([lambda l=l: f(l) for l in lins]),
+                2.0 * (2 * ff * W + T * W + T * ff), 4.0 * T * ff * W)
+            del lins
+        del ws
+        torch.cuda.empty_cache()
+    assert ops.take_status() == 0
+    return rows
+
+
+def run(sizes, steps: int, warmup: int, layers: int = 8, vocab: int = 32768, kernels_only: bool = False) -> Dict:
+    res: Dict = {"design": "sevevik", "beside": "qwen3 (equal size, bf16 weights, FP8 pages)", "layers": layers, "vocab": vocab,
+                 "window": WINDOW, "data": "synthetic token ids, random-init weights", "throughput": {}, "kernels": {}}
+    for size in sizes:
+        res["kernels"][size] = kernels(size)
+        if not kernels_only:
+            res["throughput"][size] = {m: throughput(c, steps, warmup) for m, c in configs(size, layers, vocab).items()}
+    return res

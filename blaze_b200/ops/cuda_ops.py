@@ -770,19 +770,26 @@ class CudaOps:
     # ------------------------------------------------------------------ differential attention
     DIFF_SHORT_ROWS = 64       # sequences with new tokens * group up to this take the short-row kernel
 
-    def diff_attention(self, qkv, A, batch, kv, layer_idx, eps):
-        """Page write and differential attention of one layer; ``[T, heads * vdim]``, every head normed and scaled."""
+    def diff_store(self, qkv, A, batch, kv, layer_idx):
+        """The rows' keys and values into their pages."""
+        a, pool = A.spec, kv.kv[layer_idx]
+        if kv.layout != "tiles" or pool.dtype != qkv.dtype:
+            raise CudaError(f"differential attention of {qkv.dtype} rows needs 'tiles' pages of that type")
+        self._check(self.lib.blz_diff_store(_ptr(qkv), qkv.stride(0), _ptr(pool), pool.stride(0), pool.stride(1), _ptr(batch.slot_mapping),
+                                            qkv.shape[0], a.heads, a.kv_heads, a.dim, a.vdim, int(qkv.dtype == torch.float32),
+                                            self._stream()), "diff_store")
+
+    def diff_attention(self, qkv, A, batch, kv, layer_idx, eps, store: bool = True):
+        """Page write (``store``) and differential attention of one layer; ``[T, heads * vdim]``, every head normed and scaled."""
         a = A.spec
         T = qkv.shape[0]
         f32 = qkv.dtype == torch.float32
         pool = kv.kv[layer_idx]
-        if kv.layout != "tiles" or pool.dtype != qkv.dtype:
-            raise CudaError(f"differential attention of {qkv.dtype} rows needs 'tiles' pages of that type")
+        if store:
+            self.diff_store(qkv, A, batch, kv, layer_idx)
         out = torch.empty(T, a.heads * a.vdim, dtype=qkv.dtype, device=self.device)
         B, bt = batch.slots.numel(), kv.block_table
         st = self._stream()
-        self._check(self.lib.blz_diff_store(_ptr(qkv), qkv.stride(0), _ptr(pool), pool.stride(0), pool.stride(1), _ptr(batch.slot_mapping), T,
-                                            a.heads, a.kv_heads, a.dim, a.vdim, int(f32), st), "diff_store")
         common = (_ptr(qkv), qkv.stride(0), _ptr(out), _ptr(pool), pool.stride(0), pool.stride(1), _ptr(bt), bt.stride(0),
                   _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len))
         shape = (T, B, a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.scale, A.lam, 1.0 - a.diff, eps)
