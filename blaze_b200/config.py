@@ -404,16 +404,6 @@ def named_config(name: str) -> ModelConfig:
         layers = [LayerSpec(a, GluSpec(320, 3.0)), LayerSpec(b), LayerSpec(a, GluSpec(320, 3.0), weights_of=0)]
         return ModelConfig.of_layers(layers, architecture="Sevevik", model_type="sevevik", vocab_size=1024, hidden_size=192,
                                      streams=3, residual_mult=0.8, embed_scale=6.0)
-    elif n in ("sevevik-8b", "sevevik-1b"):
-        # layers of a size that real models have (random weights: no checkpoint of the design at this size exists)
-        if n == "sevevik-8b":
-            a = DiffAttnSpec(heads=32, kv_heads=8, dim=64, vdim=128, scale=0.125, diff=0.5, window=1024)
-            ff, width, count = GluSpec(12288, 7.0), 4096, 36
-        else:
-            a = DiffAttnSpec(heads=16, kv_heads=8, dim=64, vdim=128, scale=0.125, diff=0.5, window=1024)
-            ff, width, count = GluSpec(6144, 7.0), 2048, 16
-        return ModelConfig.of_layers([LayerSpec(a, ff) for _ in range(count)], architecture="Sevevik", model_type="sevevik",
-                                     vocab_size=151936, hidden_size=width, streams=4, residual_mult=1.0, embed_scale=1.0)
     elif n in ("qwen3-8b",):
         c = ModelConfig(vocab_size=151936, hidden_size=4096, num_layers=36, num_heads=32, num_kv_heads=8,
                         head_dim=128, intermediate_size=12288, rope=RopeConfig(theta=1e6))

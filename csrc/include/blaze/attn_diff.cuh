@@ -19,7 +19,6 @@ struct DiffParams {
   const int* slots;            // [B]
   const int* q_start;          // [B + 1]
   const int* ctx_len;          // [B]
-  const int* positions;        // [T]
   const int* seq_of_row;       // [T], -1 = padding
   const int* slot_mapping;     // [T], -1 = padding
   float* part_o;               // partial outputs of split key ranges

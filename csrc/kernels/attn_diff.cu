@@ -498,7 +498,7 @@ static blz::DiffParams diff_params(const void* qkv, long long ld, void* out, voi
   blz::DiffParams p;
   p.qkv = qkv; p.ld = ld; p.out = out; p.pool = pool; p.page_stride = page_stride; p.head_stride = head_stride;
   p.block_table = block_table; p.bt_stride = bt_stride; p.slots = slots; p.q_start = q_start; p.ctx_len = ctx_len;
-  p.positions = nullptr; p.seq_of_row = nullptr; p.slot_mapping = nullptr; p.part_o = p.part_ml = nullptr;
+  p.seq_of_row = nullptr; p.slot_mapping = nullptr; p.part_o = p.part_ml = nullptr;
   p.T = T; p.B = B; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window;
   p.scale = scale; p.lam = lam; p.post = post; p.eps = eps;
   p.max_rows = 0x7fffffff; p.row_blocks = p.splits = p.stages = 1;

@@ -153,7 +153,7 @@ def spec(heads, kv_heads, dim, vdim, window, scale=None, diff=0.3):
     return DiffAttnSpec(heads, kv_heads, dim, vdim, scale or dim ** -0.5, diff, window)
 
 
-SPECS = [(4, 4, 32, 64, 100), (4, 1, 16, 16, 24), (6, 2, 48, 80, 50), (8, 2, 64, 128, 200), (8, 1, 128, 128, 129), (4, 2, 40, 24, 33),
+SPECS = [(5, 5, 32, 64, 100), (4, 1, 16, 16, 24), (6, 2, 48, 80, 50), (8, 2, 64, 128, 200), (8, 1, 128, 128, 129), (4, 2, 40, 24, 33),
          (2, 2, 20, 36, 0), (3, 1, 64, 32, 1), (5, 1, 24, 120, 2), (2, 1, 144, 136, 40), (16, 1, 32, 32, 0), (40, 1, 16, 48, 90)]
 PORTIONS = {"whole": [10 ** 6], "pairs and more": [2, 37, 3, 130, 1], "decode": [150, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1]}
 
@@ -182,7 +182,7 @@ def test_attention_windows_and_far_keys(ops, case, portions, dtype):
     assert err.mean() < limit / 5
 
 
-@pytest.mark.parametrize("case", [(8, 2, 64, 128, 70), (4, 4, 32, 64, 0), (6, 2, 40, 24, 33)])
+@pytest.mark.parametrize("case", [(8, 2, 64, 128, 70), (3, 3, 32, 64, 0), (6, 2, 40, 24, 33)])
 def test_attention_batches_of_unequal_sequences(ops, case):
     """Long portions, short portions and single rows in one step; a freed sequence's pages serve the next one."""
     s = spec(*case)
