@@ -447,7 +447,7 @@ def self_spec(llm, ids, max_tokens: int, draft: int) -> int:
         while acc < draft and picks[acc] == drafts[acc]:
             acc += 1
         out.extend(int(t) for t in picks[:acc + 1])
-        if eng.kv.gdn_layers:
+        if eng.kv.state_layers:
             eng.commit_state([(s, acc + 1)])
         eng.truncate(s, base + acc + 1)
         rounds += 1

@@ -12,7 +12,7 @@ import json
 import math
 import os
 from dataclasses import dataclass, field, asdict
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Union
 
 
 @dataclass
@@ -48,24 +48,122 @@ class DiffAttnSpec:
     diff: float                 # constant part of the second map's weight; the normed output is scaled by 1 - diff
     window: int = 0             # a row sees itself and the window - 1 tokens before it (0: every token before it)
 
+    maps = 2                    # query / key maps per head
+
     @property
     def group(self) -> int:
         return self.heads // self.kv_heads
 
 
 @dataclass
+class RotarySpec:
+    """Rotary positions on the first ``dims`` dimensions of a head.  ``factor`` > 1 slows frequencies down by their wavelength:
+    those longer than ``original / low`` tokens by the whole factor, those shorter than ``original / high`` not at all, the ones
+    between by a blend."""
+    dims: int
+    base: float
+    interleaved: bool = True    # pairs (2i, 2i + 1); else (i, i + dims / 2)
+    factor: float = 1.0
+    low: float = 1.0
+    high: float = 4.0
+    original: float = 0.0       # 0: no scaling
+
+    def frequencies(self) -> List[float]:
+        out = []
+        for i in range(self.dims // 2):
+            f = self.base ** (-2.0 * i / self.dims)
+            if self.original:
+                turns = self.original * f / (2 * math.pi)          # full turns over the original context
+                if turns < self.low:
+                    f /= self.factor
+                elif turns <= self.high:
+                    keep = (turns - self.low) / (self.high - self.low) if self.high > self.low else 1.0
+                    f *= keep + (1 - keep) / self.factor
+            out.append(f)
+        return out
+
+
+@dataclass
+class SoftAttnSpec:
+    """Softmax attention of one layer over bf16 / fp32 pages, with the options of its designs."""
+    heads: int
+    kv_heads: int
+    dim: int                    # queries and keys
+    vdim: int                   # values
+    scale: float                # of the scores
+    rot: Optional[RotarySpec] = None
+    bias: bool = False          # q, k and v projections have biases
+    unit_rms: bool = False      # q and k heads divided by their root mean square after the rotation
+    sink: bool = False          # a learned term per head in the softmax's denominator
+    gate: bool = False          # heads multiplied by sigmoid of a projection of the layer's input
+    window: int = 0             # as in DiffAttnSpec
+    out_scale: float = 1.0      # of the mixer's output
+    maps = 1
+
+    @property
+    def group(self) -> int:
+        return self.heads // self.kv_heads
+
+
+@dataclass
+class DeltaSpec:
+    """Gated delta rule with one decay per head and key channel, and a gated norm per head."""
+    heads: int
+    kv_heads: int               # heads of q and k
+    dim: int
+    vdim: int
+    conv: int                   # taps of the convolution before it
+    out_scale: float = 1.0
+
+    @property
+    def conv_dim(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    @property
+    def state(self) -> int:
+        return self.dim
+
+
+@dataclass
+class StateSpaceSpec:
+    """Mamba-2 (state-space duality) mixer."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int                 # B / C pairs, each for heads / groups heads
+    norm_groups: int
+    conv: int
+    out_scale: float = 1.0
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_dim(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+
+@dataclass
 class GluSpec:
-    """Dense feed-forward with a clamped gate and a clamped up projection."""
+    """Dense gated feed-forward: with a clamped gate and a clamped up projection, or (no ``limit``) ``silu(gate) * up``."""
     ff: int
-    limit: float
+    limit: Optional[float] = None
 
 
 @dataclass
 class LayerSpec:
-    """One entry of a configuration that describes its layers one by one."""
-    attn: DiffAttnSpec
+    """One entry of a configuration that describes its layers one by one: an attention, a recurrence, or both side by side."""
+    attn: Union[DiffAttnSpec, SoftAttnSpec, None] = None
     mlp: Optional[GluSpec] = None          # None: the layer has no feed-forward
-    weights_of: Optional[int] = None       # the layer whose tensors this one uses (with a cache of its own)
+    weights_of: Optional[int] = None       # the layer whose tensors this one uses (with a cache and a state of its own)
+    rec: Union[DeltaSpec, StateSpaceSpec, None] = None
+
+    @property
+    def kind(self) -> str:
+        a = None if self.attn is None else "diff_attention" if self.attn.maps == 2 else "soft_attention"
+        r = None if self.rec is None else "state_space" if isinstance(self.rec, StateSpaceSpec) else "delta_rule"
+        return "+".join(k for k in (a, r) if k)
 
 
 @dataclass
@@ -118,12 +216,13 @@ class ModelConfig:
     indexer_head_dim: int = 0
     indexer_budget: int = 0
     indexer_compress_ratio: int = 0
-    # models whose configuration lists its layers one by one, each with sizes of its own (Sevevik); the sizes above then hold
-    # those of the first layer
+    # models whose configuration lists its layers one by one, each with sizes of its own (Sevevik, Niletar); the sizes above then
+    # hold those of the first layer
     layer_specs: List[LayerSpec] = field(default_factory=list)
     streams: int = 1                        # residual streams joined by learned static mixes
     residual_mult: float = 1.0              # of every sublayer's output
     embed_scale: float = 1.0
+    residual_alpha: float = 1.0             # post-norm residual: x <- norm(alpha * x + sublayer)
     # tokens
     eos_token_ids: List[int] = field(default_factory=list)
     bos_token_id: Optional[int] = None
@@ -161,7 +260,7 @@ class ModelConfig:
 
     def layer_type(self, i: int) -> str:
         if self.layer_specs:
-            return "diff_attention"
+            return self.layer_specs[i].kind
         return self.layer_types[i] if self.layer_types else "full_attention"
 
     def to_dict(self) -> Dict[str, Any]:
@@ -201,6 +300,8 @@ class ModelConfig:
     def from_json(cls, raw: Dict[str, Any]) -> "ModelConfig":
         if raw.get("architecture") == "Sevevik":
             return cls._from_sevevik(raw)
+        if raw.get("architecture") == "Niletar":
+            return cls._from_niletar(raw)
         archs = raw.get("architectures") or ["Qwen3ForCausalLM"]
         t = raw.get("text_config", raw)
         g = lambda k, d=None: t.get(k, raw.get(k, d))  # noqa: E731
@@ -305,15 +406,7 @@ class ModelConfig:
             mask = m.get("mask") or {}
             attn = DiffAttnSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
                                 scale=float(m["scale"]), diff=float(m["diff"]), window=int(mask.get("size") or 0))
-            mlp = None
-            if e.get("mlp") is not None:
-                if e["mlp"].get("kind", "dense") != "dense":
-                    raise ValueError(f"layer {i}: unknown feed-forward {e['mlp']['kind']!r}")
-                mlp = GluSpec(ff=int(e["mlp"]["ff"]), limit=float(e["mlp"]["limit"]))
-            wof = e.get("weights_of")
-            specs.append(LayerSpec(attn, mlp, None if wof is None else int(wof)))
-        if not specs:
-            raise ValueError("the configuration lists no layers")
+            specs.append(LayerSpec(attn, _dense_mlp(i, e, limit=True), _weights_of(e)))
         _check_layers(specs)
         return cls.of_layers(specs, architecture="Sevevik", model_type="sevevik", vocab_size=int(raw["vocab"]),
                              hidden_size=int(raw["width"]), rms_norm_eps=float(raw["norm"]["eps"]), streams=int(raw.get("streams", 1)),
@@ -322,26 +415,87 @@ class ModelConfig:
                              torch_dtype=str(raw.get("torch_dtype", "bfloat16")))
 
     @classmethod
+    def _from_niletar(cls, raw: Dict[str, Any]) -> "ModelConfig":
+        """The layer-by-layer configuration of the Niletar design."""
+        specs: List[LayerSpec] = []
+        for i, e in enumerate(raw["layers"]):
+            m, attn = e["mixer"], None
+            if e["type"] == "mamba2":
+                rec = StateSpaceSpec(heads=int(m["heads"]), vdim=int(m["vdim"]), state=int(m["state"]), groups=int(m["groups"]),
+                                     norm_groups=int(m["norm_groups"]), conv=int(m["conv"]))
+            elif e["type"] == "parallel":
+                l, r = m["left"], m["right"]
+                attn = SoftAttnSpec(heads=int(l["heads"]), kv_heads=int(l["kv_heads"]), dim=int(l["dim"]), vdim=int(l["vdim"]),
+                                    scale=float(l["scale"]), rot=_rotary(l.get("rot")), bias=True, unit_rms=True, sink=True, gate=True,
+                                    out_scale=float(m["left_scale"]))
+                rec = DeltaSpec(heads=int(r["heads"]), kv_heads=int(r["kv_heads"]), dim=int(r["dim"]), vdim=int(r["vdim"]),
+                                conv=int(r["conv"]), out_scale=float(m["right_scale"]))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+            specs.append(LayerSpec(attn, _dense_mlp(i, e, limit=False), _weights_of(e), rec))
+        _check_layers(specs)
+        return cls.of_layers(specs, architecture="Niletar", model_type="niletar", vocab_size=int(raw["vocab"]), hidden_size=int(raw["width"]),
+                             rms_norm_eps=float(raw["norm"]["eps"]), zero_centered_norm=True, residual_alpha=float(raw["postln_alpha"]),
+                             torch_dtype=str(raw.get("torch_dtype", "bfloat16")))
+
+    @classmethod
     def of_layers(cls, specs: List[LayerSpec], **kw) -> "ModelConfig":
         """A configuration from its layer list; the model-wide sizes that other parts read are those of the first layer."""
-        a, mlp = specs[0].attn, specs[0].mlp
-        return cls(layer_specs=specs, num_layers=len(specs), num_heads=a.heads, num_kv_heads=a.kv_heads, head_dim=a.dim,
-                   intermediate_size=mlp.ff if mlp else 0, qk_norm=False, layer_types=["diff_attention"] * len(specs), **kw)
+        a = next((s.attn for s in specs if s.attn is not None), None)
+        r, mlp = specs[0].rec, specs[0].mlp
+        heads = (a.heads, a.kv_heads, a.dim) if a is not None else (r.heads, r.heads, r.vdim)
+        return cls(layer_specs=specs, num_layers=len(specs), num_heads=heads[0], num_kv_heads=heads[1], head_dim=heads[2],
+                   intermediate_size=mlp.ff if mlp else 0, qk_norm=False, layer_types=[s.kind for s in specs], **kw)
+
+
+def _weights_of(entry: Dict[str, Any]) -> Optional[int]:
+    v = entry.get("weights_of")
+    return None if v is None else int(v)
+
+
+def _dense_mlp(i: int, entry: Dict[str, Any], limit: bool) -> Optional[GluSpec]:
+    m = entry.get("mlp")
+    if m is None:
+        return None
+    if m.get("kind", "dense") != "dense":
+        raise ValueError(f"layer {i}: unknown feed-forward {m['kind']!r}")
+    return GluSpec(ff=int(m["ff"]), limit=float(m["limit"]) if limit else None)
+
+
+def _rotary(rot: Optional[Dict[str, Any]]) -> Optional[RotarySpec]:
+    if not rot:
+        return None
+    r, sc = RotarySpec(dims=int(rot["dims"]), base=float(rot["base"])), rot.get("scaling")
+    if sc:
+        r.factor, r.low, r.high, r.original = (float(sc[k]) for k in ("factor", "low", "high", "original"))
+    return r
 
 
 def _check_layers(specs: List[LayerSpec]) -> None:
     """Refuse a layer list that no model of the design can have."""
+    if not specs:
+        raise ValueError("the configuration lists no layers")
     for i, s in enumerate(specs):
-        a = s.attn
-        if min(a.heads, a.kv_heads, a.dim, a.vdim) < 1 or a.heads % a.kv_heads:
-            raise ValueError(f"layer {i}: {a.heads} query heads over {a.kv_heads} key/value heads of {a.dim} / {a.vdim}")
-        if a.window < 0:
-            raise ValueError(f"layer {i}: a window of {a.window}")
+        a, r = s.attn, s.rec
+        if a is not None:
+            if min(a.heads, a.kv_heads, a.dim, a.vdim) < 1 or a.heads % a.kv_heads:
+                raise ValueError(f"layer {i}: {a.heads} query heads over {a.kv_heads} key/value heads of {a.dim} / {a.vdim}")
+            if a.window < 0:
+                raise ValueError(f"layer {i}: a window of {a.window}")
+            rot = getattr(a, "rot", None)
+            if rot is not None and (rot.dims % 2 or not 0 <= rot.dims <= a.dim):
+                raise ValueError(f"layer {i}: rotary positions on {rot.dims} of {a.dim} dimensions")
+        if r is not None:
+            groups = r.groups if isinstance(r, StateSpaceSpec) else r.kv_heads
+            if min(r.heads, groups, r.state, r.vdim, r.conv) < 1 or r.heads % groups:
+                raise ValueError(f"layer {i}: {r.heads} recurrent heads over {groups} groups, state {r.state} x {r.vdim}, {r.conv} taps")
+            if isinstance(r, StateSpaceSpec) and (r.norm_groups < 1 or r.inner % r.norm_groups):
+                raise ValueError(f"layer {i}: {r.inner} columns in {r.norm_groups} norm groups")
         if s.weights_of is not None:
             src = specs[s.weights_of] if 0 <= s.weights_of < len(specs) else None
             if src is None or src.weights_of is not None:
                 raise ValueError(f"layer {i} uses the tensors of layer {s.weights_of}, which has none of its own")
-            if (src.attn, src.mlp) != (a, s.mlp):
+            if (src.attn, src.rec, src.mlp) != (a, r, s.mlp):
                 raise ValueError(f"layer {i} differs from layer {s.weights_of}, whose tensors it uses")
 
 
@@ -404,6 +558,16 @@ def named_config(name: str) -> ModelConfig:
         layers = [LayerSpec(a, GluSpec(320, 3.0)), LayerSpec(b), LayerSpec(a, GluSpec(320, 3.0), weights_of=0)]
         return ModelConfig.of_layers(layers, architecture="Sevevik", model_type="sevevik", vocab_size=1024, hidden_size=192,
                                      streams=3, residual_mult=0.8, embed_scale=6.0)
+    elif n in ("tiny-niletar",):
+        # the Niletar layer kinds in miniature, one without a feed-forward, one that uses another's tensors
+        def mamba(**kw):
+            return StateSpaceSpec(**{**dict(heads=6, vdim=32, state=48, groups=2, norm_groups=3, conv=4), **kw})
+        a = SoftAttnSpec(heads=4, kv_heads=2, dim=32, vdim=48, scale=0.2, rot=RotarySpec(24, 1.0e4, factor=4.0, original=256.0), bias=True,
+                         unit_rms=True, sink=True, gate=True, out_scale=0.7)
+        d = DeltaSpec(heads=4, kv_heads=2, dim=32, vdim=40, conv=3, out_scale=0.4)
+        layers = [LayerSpec(a, GluSpec(320), None, d), LayerSpec(None, None, None, mamba()), LayerSpec(a, GluSpec(320), 0, d)]
+        return ModelConfig.of_layers(layers, architecture="Niletar", model_type="niletar", vocab_size=1024, hidden_size=192,
+                                     zero_centered_norm=True, residual_alpha=1.8)
     elif n in ("qwen3-8b",):
         c = ModelConfig(vocab_size=151936, hidden_size=4096, num_layers=36, num_heads=32, num_kv_heads=8,
                         head_dim=128, intermediate_size=12288, rope=RopeConfig(theta=1e6))

@@ -185,7 +185,7 @@ class Engine:
     @property
     def trees_ok(self) -> bool:
         """Draft trees are verified by the attention kernels of plain softmax layers only."""
-        return not self.kv.gdn_layers and not self.model.cfg.layer_specs
+        return not self.kv.state_layers and not self.model.cfg.layer_specs
 
     @property
     def free_tokens(self) -> int:
@@ -203,9 +203,9 @@ class Engine:
             s.length = snap.length
             s.shared = len(snap.pages)
             self.kv.set_pages(row, s.pages, 0)
-            if snap.state_row >= 0 and self.kv.gdn_layers:
+            if snap.state_row >= 0 and self.kv.state_layers:
                 self.kv.copy_state(snap.state_row, row)
-        elif self.kv.gdn_layers:
+        elif self.kv.state_layers:
             self.kv.zero_state(row)
         self.seqs[row] = s
         return s
@@ -228,7 +228,7 @@ class Engine:
         pg = s.pages[:n // PAGE]
         self.pages.retain(pg)
         row = -1
-        if with_state and self.kv.gdn_layers:
+        if with_state and self.kv.state_layers:
             if n != s.length:
                 # recurrent state is only valid at the sequence's current length
                 self.pages.release(pg)
@@ -267,7 +267,7 @@ class Engine:
         are speculative — models with recurrent layers leave those sequences' state as it was, and ``commit_state`` advances
         it over the accepted rows afterwards."""
         chunks = []
-        defer = bool(defer_state and self.kv.gdn_layers)
+        defer = bool(defer_state and self.kv.state_layers)
         for s, toks, want in items:
             self.reserve(s, s.length + len(toks))
             at = None if isinstance(want, int) else [int(j) for j in want]
@@ -282,7 +282,7 @@ class Engine:
         """items: (seq, rows kept) for sequences of the last step that ran with ``defer_state``: advance their recurrent
         state over the first ``rows kept`` rows of that step (the accepted tokens), reading the inputs the layers recorded
         (reference: ``Model::pre_verify`` / ``commit_replay``, crates/blaze/src/model.rs:3364, :3484)."""
-        if not self.kv.gdn_layers or not items:
+        if not self.kv.state_layers or not items:
             return
         chunks, rows = [], []
         for s, keep in items:
@@ -301,7 +301,7 @@ class Engine:
         slot ``length + i``; ``commit_tree`` moves the accepted path into place afterwards
         (reference: ``Engine::verify_many_tree``, crates/blaze/src/engine.rs :1401)."""
         if not self.trees_ok:
-            raise ValueError("draft trees need a model without recurrent (linear-attention) layers and without differential attention")
+            raise ValueError("draft trees need a model whose layers are all plain attention")
         group = max(self.model.cfg.num_heads // max(self.model.cfg.num_kv_heads, 1), 1)
         chunks = []
         for s, toks, parents in items:
@@ -447,7 +447,7 @@ class Engine:
         the rows of one sequence must fit the decode attention kernel's row tiers and the model must keep no recurrent state."""
         from .batch import SMALL_ROWS
         return bool(self.ecfg.use_graphs and self.ecfg.verify_graphs and self.device.type == "cuda" and self.model.ops.is_cuda
-                    and self.model.is_first_stage and self.model.is_last_stage and not self.kv.gdn_layers
+                    and self.model.is_first_stage and self.model.is_last_stage and not self.kv.state_layers
                     and not self.attn_all_items and rows_per_seq >= 1
                     and max(self.attn_group, 1) * rows_per_seq <= SMALL_ROWS
                     and self._bucket(seqs) * rows_per_seq <= self.ecfg.verify_graph_rows)

@@ -1,4 +1,4 @@
-"""Paged KV pools, block tables and recurrent (Gated DeltaNet) state rows.
+"""Paged KV pools, block tables and recurrent state rows.
 
 Pages hold 16 tokens.  Two pool layouts exist:
 
@@ -9,11 +9,14 @@ Pages hold 16 tokens.  Two pool layouts exist:
   byte of token t, dim j at ``(t//8)*8*D + (j//16)*128 + (t%8)*16 + j%16``) followed by V transposed
   (``[head_dim][16 tokens]``), so that one 1-D bulk copy per (page, head) feeds both MMAs.
 
-* ``tiles`` — one tensor ``[pages, kv_heads, 16 * (2 * dim + vdim)]`` per differential-attention layer in bf16 or fp32: the keys
-  of map 1, the keys of map 2 and the values of the page's 16 tokens, each as 8-token x 8-element core matrices (element of token
+* ``tiles`` — one tensor ``[pages, kv_heads, 16 * (maps * dim + vdim)]`` per layer of a layer-by-layer configuration in bf16 or
+  fp32: the keys of each map (two for differential attention) and the values of the page's 16 tokens, as 8-token x 8-element core matrices (element of token
   t, dim j at ``(t // 8) * 8 * D + (j // 8) * 64 + (t % 8) * 8 + j % 8``, D rounded up to 16 and padded with zeros): 8 x 16 bytes
   in a row is what ``ldmatrix`` and the tensor core's unswizzled operands both take.  The ``logical`` form of such a layer is
-  ``k [pages, 2 * kv_heads, 16, dim]`` (key head g's maps at 2g and 2g + 1) and ``v [pages, kv_heads, 16, vdim]``.
+  ``k [pages, maps * kv_heads, 16, dim]`` (two maps: key head g's at 2g and 2g + 1) and ``v [pages, kv_heads, 16, vdim]``.
+
+Recurrent layers (Gated DeltaNet, and the recurrences of a layer-by-layer configuration) keep one state row per sequence row: the
+last inputs of their convolution in the activation type and the recurrent state in fp32, of each layer's own sizes.
 
 The reference keeps one-token pages and several KV dtypes (``crates/blaze/src/model.rs:499-583``,
 ``alloc_kv`` :517); its page bookkeeping is in ``engine.rs:1083-1164``.
@@ -36,14 +39,15 @@ def pad16(n: int) -> int:
     return (n + 15) // 16 * 16
 
 
-def diff_page_elems(spec) -> int:
+def page_elems(spec) -> int:
     """Elements of one (page, key/value head) block of the ``tiles`` layout."""
-    return PAGE * (2 * pad16(spec.dim) + pad16(spec.vdim))
+    return PAGE * (spec.maps * pad16(spec.dim) + pad16(spec.vdim))
 
 
 def kv_bytes_per_token(cfg: ModelConfig, kv_dtype: str, tp_world: int = 1) -> int:
     if cfg.layer_specs:
-        return sum(s.attn.kv_heads * diff_page_elems(s.attn) for s in cfg.layer_specs) // PAGE * (4 if kv_dtype == "fp32" else 2)
+        attn = [s.attn for s in cfg.layer_specs if s.attn is not None]
+        return sum(a.kv_heads * page_elems(a) for a in attn) // PAGE * (4 if kv_dtype == "fp32" else 2)
     n_attn = sum(1 for i in range(cfg.num_layers) if cfg.layer_type(i) == "full_attention")
     kvh = max(cfg.num_kv_heads // tp_world, 1)
     if kv_dtype in FP4_KV:
@@ -92,11 +96,13 @@ class KVCache:
         for i in (range(lo, hi) if cfg.layer_specs else ()):
             a = cfg.layer_specs[i].attn
             if kv_dtype not in ("fp32", "bf16"):
-                raise ValueError(f"differential attention keeps its keys and values in bf16 or fp32, not {kv_dtype}")
+                raise ValueError(f"{cfg.architecture} keeps its keys and values in bf16 or fp32, not {kv_dtype}")
+            if a is None:
+                continue
             if layout == "tiles":
-                self.kv[i] = torch.zeros(num_pages, a.kv_heads, diff_page_elems(a), dtype=tdt, device=device)
+                self.kv[i] = torch.zeros(num_pages, a.kv_heads, page_elems(a), dtype=tdt, device=device)
             else:
-                self.k[i] = torch.zeros(num_pages, 2 * a.kv_heads, PAGE, a.dim, dtype=tdt, device=device)
+                self.k[i] = torch.zeros(num_pages, a.maps * a.kv_heads, PAGE, a.dim, dtype=tdt, device=device)
                 self.v[i] = torch.zeros(num_pages, a.kv_heads, PAGE, a.vdim, dtype=tdt, device=device)
         for i in self.attn_layers:
             if layout == "umma":
@@ -128,6 +134,12 @@ class KVCache:
                                                  dtype=act, device=device)
                 self.rec_state[i] = torch.zeros(self.state_rows, hv, cfg.linear_key_head_dim,
                                                 cfg.linear_value_head_dim, dtype=torch.float32, device=device)
+
+        rec = {i: cfg.layer_specs[i].rec for i in (range(lo, hi) if cfg.layer_specs else ()) if cfg.layer_specs[i].rec is not None}
+        for i, r in rec.items():
+            self.conv_state[i] = torch.zeros(self.state_rows, r.conv_dim, r.conv - 1, dtype=tdt, device=device)
+            self.rec_state[i] = torch.zeros(self.state_rows, r.heads, r.state, r.vdim, dtype=torch.float32, device=device)
+        self.state_layers = self.gdn_layers + list(rec)     # every layer with a recurrent state
 
         # sparse-attention indexer: the raw index key of every token, paged like K and V (shared prefixes share them)
         self.idx_k: Dict[int, torch.Tensor] = {}
@@ -188,15 +200,15 @@ class KVCache:
 
     # ------------------------------------------------------------------ recurrent state rows
     def copy_state(self, src: int, dst: int) -> None:
-        """Copy the GDN conv + recurrent state of row ``src`` to row ``dst`` (``model.rs:2718``)."""
-        for i in self.gdn_layers:
+        """Copy the conv + recurrent state of row ``src`` to row ``dst`` (``model.rs:2718``)."""
+        for i in self.state_layers:
             self.conv_state[i][dst].copy_(self.conv_state[i][src])
             self.rec_state[i][dst].copy_(self.rec_state[i][src])
         if self.ple is not None:
             self.ple.copy(src, dst)
 
     def zero_state(self, row: int) -> None:
-        for i in self.gdn_layers:
+        for i in self.state_layers:
             self.conv_state[i][row].zero_()
             self.rec_state[i][row].zero_()
         if self.ple is not None:

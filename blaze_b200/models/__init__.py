@@ -7,5 +7,8 @@ def model_class(cfg):
     if cfg.architecture == "Sevevik":
         from .sevevik import Sevevik
         return Sevevik
+    if cfg.architecture == "Niletar":
+        from .niletar import Niletar
+        return Niletar
     from .qwen3 import Model
     return Model

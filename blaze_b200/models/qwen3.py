@@ -62,6 +62,47 @@ class Gdn:
         self.v_heads = 0
 
 
+class SoftAttn:
+    """Softmax attention of a :class:`Mixer`: ``sink [heads]`` and ``freq [2, rotated / 2]`` (frequencies, and what rounding them to
+    32 bits left over), fp32; either may be None."""
+
+    def __init__(self, spec, device, sink=None):
+        self.spec = spec                 # config.SoftAttnSpec
+        self.sink = None if sink is None else sink.to(device, torch.float32).contiguous()
+        self.freq = None
+        if spec.rot is not None:
+            f = torch.tensor(spec.rot.frequencies(), dtype=torch.float64)
+            self.freq = torch.stack([f.float(), (f - f.float().double()).float()]).to(device)
+
+
+class Recurrence:
+    """Recurrent part of a :class:`Mixer`, ``kind`` "delta" (config.DeltaSpec) or "ssm" (config.StateSpaceSpec).  ``A`` is the positive
+    decay rate; decay, step and norm weights are fp32.  ``low`` (delta): from the low-rank inputs to [decay inputs | norm gates]."""
+
+    def __init__(self, spec, kind: str, norm_groups: int):
+        self.spec, self.kind, self.norm_groups = spec, kind, norm_groups
+        self.conv_w: torch.Tensor = None          # [conv_dim, taps], activation type
+        self.conv_b: Optional[torch.Tensor] = None
+        self.A = self.dt_bias = self.D = self.norm_w = None
+        self.low: Optional[Linear] = None
+
+
+class Mixer:
+    """The mixers of a layer on one input: a stacked input projection (``cols``: first column of each part), an attention and / or a
+    recurrence whose results lie side by side (scaled), and one output projection over both."""
+
+    def __init__(self):
+        self.in_proj: Linear = None
+        self.o: Linear = None
+        self.cols: Dict[str, int] = {}
+        self.low_width = 0               # columns of the low-rank inputs
+        self.attn: Optional[SoftAttn] = None
+        self.rec: Optional[Recurrence] = None
+
+    def linears(self) -> List[Linear]:
+        return [l for l in (self.in_proj, self.o, self.rec.low if self.rec is not None else None) if l is not None]
+
+
 class DenseMlp:
     def __init__(self):
         self.gate_up: Linear = None
@@ -115,6 +156,9 @@ class Layer:
         # Qwen4-Exp: hyper-connections around the two blocks (in place of the norms above) and an n-gram embedding
         self.hc_attn = self.hc_mlp = None
         self.ple = None
+        # post-norm designs: the mixers as one object, and the norms of the sums after them and after the feed-forward
+        self.mixer: Optional[Mixer] = None
+        self.mixer_norm = self.mlp_norm = None
 
 
 _PROFILE_PHASES = os.environ.get("BLAZE_PROFILE_PHASES", "0") == "1"
@@ -711,6 +755,20 @@ class Model:
     def _diff_attention(self, A: DiffAttn, h, batch, kv, gi):
         return self.ops.linear(A.o, self.ops.diff_attention(self.ops.linear(A.qkv, h), A, batch, kv, gi, self.cfg.rms_norm_eps))
 
+    def _mixer(self, M: Mixer, h, batch, kv, gi):
+        ops, eps = self.ops, self.cfg.rms_norm_eps
+        proj = ops.linear(M.in_proj, h)
+        n_attn = M.attn.spec.heads * M.attn.spec.vdim if M.attn is not None else 0
+        y = torch.empty(proj.shape[0], M.o.K, dtype=proj.dtype, device=proj.device)
+        if M.attn is not None:
+            ops.soft_attention(proj, M, batch, kv, gi, eps, y[:, :n_attn])
+        if M.rec is not None:
+            low = ops.linear(M.rec.low, proj[:, M.cols["low"]:M.cols["low"] + M.low_width]) if M.rec.low is not None else None
+            if batch.gdn_defer is not None:
+                self.gdn_records[gi] = (proj, low)      # what the recurrence consumed (see _gdn)
+            ops.recurrence(proj, low, M, batch, kv, gi, eps, y[:, n_attn:])
+        return ops.linear(M.o, y)
+
     def _gdn(self, G: Gdn, h, batch, kv, gi, fused=None):
         ops, cfg = self.ops, self.cfg
         dk, dv = cfg.linear_key_head_dim, cfg.linear_value_head_dim
@@ -727,17 +785,22 @@ class Model:
         return self._row_cut(G.out_proj, o, o.shape[0], fused)
 
     def gdn_replay(self, batch: StepBatch, rows: torch.Tensor, kv: KVCache) -> None:
-        """Advance the recurrent state of every GDN layer over ``rows`` (indices into the recorded step's rows, grouped by
+        """Advance the recurrent state of every recurrent layer over ``rows`` (indices into the recorded step's rows, grouped by
         sequence as ``batch`` describes) — the accepted prefix of a verify step whose state update was deferred
         (reference: ``commit_replay``, crates/blaze/src/model.rs:3484)."""
         idx = rows.long()
         for li, L in enumerate(self.layers):
             gi = self.first_layer + li
-            if L.gdn is None:
+            if L.gdn is None and (L.mixer is None or L.mixer.rec is None):
                 continue
             rec = self.gdn_records.get(gi)
             if rec is None:
                 raise RuntimeError("no deferred step to replay")
+            if L.mixer is not None:
+                proj, low = rec
+                self.ops.recurrence(proj[idx].contiguous(), None if low is None else low[idx].contiguous(), L.mixer, batch, kv, gi,
+                                    self.cfg.rms_norm_eps, None, state_only=True)
+                continue
             mixed, b, a = rec
             ba = torch.stack([b[idx], a[idx]]).contiguous()      # one buffer: the kernels take a common row stride
             self.ops.gdn(mixed[idx].contiguous(), None, ba[0], ba[1], L.gdn, self, batch, kv, gi, state_only=True)
@@ -832,6 +895,8 @@ class Model:
     def weight_bytes(self) -> int:
         n = 0
         for L in {id(L): L for L in self.layers}.values():       # layers may share their tensors
+            if L.mixer is not None:
+                n += sum(l.nbytes() for l in L.mixer.linears())
             for obj in (L.attn, L.gdn, L.mlp):
                 if obj is None:
                     continue

@@ -33,8 +33,8 @@ class StaticStreams:
 
 
 class Sevevik(Model):
-    kernel_sources = ("host", "fused_ops", "gemm_tc", "gemm_sk", "gemm_wide", "moe_gemm", "gemm_simple", "streams", "attn_diff",
-                      "attn_diff_tc", "sampling")
+    kernel_sources = ("host", "fused_ops", "gemm_tc", "gemm_sk", "gemm_wide", "moe_gemm", "gemm_simple", "streams", "attn_maps",
+                      "attn_maps_tc", "sampling")
     cuda_dtypes = (torch.bfloat16, torch.float32)
     fp8_pages = False
 

@@ -163,6 +163,7 @@ class CudaOps:
         # static residual streams, differential attention, 32-bit products
         lib.blz_streams.argtypes = [VP, VP, VP, _c.c_int, _c.c_float, VP, VP, VP, VP, VP, _c.c_float, VP, VP, _c.c_int, _c.c_int, _c.c_int,
                                     _c.c_int, _c.c_int, _c.c_int, VP]
+        lib.blz_residual_norm.argtypes = [VP, _c.c_int, _c.c_float, VP, VP, _c.c_float, VP, VP, _c.c_int, _c.c_int, _c.c_int, VP]
         lib.blz_norm_rows.argtypes = [VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_float, _c.c_int, VP]
         lib.blz_gemm_simple.argtypes = [VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_int, _c.c_int, _c.c_int, _c.c_int,
                                         _c.c_int, VP]
@@ -173,6 +174,19 @@ class CudaOps:
         lib.blz_diff_plain.argtypes = common + [VP] + shape + [_c.c_int, VP]
         lib.blz_diff_tc.argtypes = common + shape + [_c.c_int, _c.c_int, VP]
         lib.blz_diff_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
+
+        # one softmax map with sink and gate; recurrences
+        LL = _c.c_longlong
+        lib.blz_attn_prep_pages.argtypes = [VP] + [LL] * 4 + [VP, VP, LL, LL, VP, VP, VP] + [_c.c_int] * 8 + [_c.c_float, _c.c_int, VP]
+        common = [VP, LL, VP, LL, VP, LL, LL, VP, _c.c_int, VP, VP, VP, VP, VP, LL]
+        shape = [_c.c_int] * 7 + [_c.c_float] * 2
+        lib.blz_soft_plain.argtypes = common + [VP] + shape + [_c.c_int, VP]
+        lib.blz_soft_tc.argtypes = common + shape + [_c.c_int, _c.c_int, VP]
+        lib.blz_soft_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
+        lib.blz_short_conv.argtypes = [VP, LL] + [VP] * 8 + [_c.c_int] * 5 + [VP]
+        lib.blz_delta_rule.argtypes = [VP, LL, VP, LL, VP, LL] + [VP] * 8 + [_c.c_int] * 7 + [VP]
+        lib.blz_state_space.argtypes = [VP, LL, VP, LL] + [VP] * 9 + [_c.c_int] * 7 + [VP]
+        lib.blz_group_norm.argtypes = [VP, VP, LL, VP, VP, LL] + [_c.c_int] * 4 + [_c.c_float] * 2 + [_c.c_int] * 3 + [VP]
 
     # ------------------------------------------------------------------ plumbing
     def _stream(self) -> VP:
@@ -359,8 +373,9 @@ class CudaOps:
     # ------------------------------------------------------------------ basics
     def embed(self, table, tokens):
         T, H = tokens.numel(), table.shape[1]
-        out = torch.empty(T, H, dtype=torch.bfloat16, device=self.device)
-        self._check(self.lib.blz_embed(_ptr(table), _ptr(tokens), _ptr(out), T, H, table.shape[0], self._stream()), "embed")
+        out = torch.empty(T, H, dtype=table.dtype, device=self.device)
+        self._check(self.lib.blz_embed(_ptr(table), _ptr(tokens), _ptr(out), T, H * table.element_size() // 2, table.shape[0],
+                                       self._stream()), "embed")
         return out
 
     def norm(self, x, residual, w, eps, zero_centered=False, quant_for: Optional[Linear] = None, zero_src: bool = False):
@@ -383,6 +398,8 @@ class CudaOps:
         """``silu(x @ Wg^T) * (x @ Wu^T)`` for a stacked ``[gate; up]`` weight with the activation computed in the GEMM's
         epilogue (the ``[T, 2I]`` intermediate never reaches memory); quantised for ``quant_for`` when that GEMM wants it."""
         exact8 = lin.fmt == Format.FP8_BLOCK and (lin.cuda_pack["kind"] == 4 if lin.cuda_pack is not None else self._fp8_block_exact)
+        if lin.fmt == Format.DENSE and (lin.w.dtype == torch.float32 or lin.N % 32 or lin.K % 16):
+            return self._glu(self.linear(lin, x), -1.0)
         if lin.N % 32 or (lin.N // 2) % 8 or exact8:
             return self.silu_mul(self.linear(lin, x), quant_for=quant_for)
         act = self.linear(lin, x, swiglu=True)
@@ -393,14 +410,15 @@ class CudaOps:
         in32 = pk["kind"] == 5
         if x.dtype != (torch.float32 if in32 else torch.bfloat16):
             raise CudaError(f"{x.dtype} activations for {pk['w'].dtype} weights")
-        x = x.contiguous()
+        if x.stride(1) != 1:
+            x = x.contiguous()
         M = x.shape[0]
         if out is None:
             out = torch.empty(M, lin.N, dtype=torch.float32 if f32 else torch.bfloat16, device=self.device)
         if M == 0:
             return out
         bias = pk["bias"].float() if pk["bias"] is not None else None
-        self._check(self.lib.blz_gemm_simple(_ptr(x), lin.K, _ptr(pk["w"]), lin.K, _ptr(out), out.stride(0), _ptr(bias), M, lin.N, lin.K,
+        self._check(self.lib.blz_gemm_simple(_ptr(x), x.stride(0), _ptr(pk["w"]), lin.K, _ptr(out), out.stride(0), _ptr(bias), M, lin.N, lin.K,
                                              int(in32), int(f32), self._stream()), "gemm_simple")
         return out
 
@@ -409,8 +427,11 @@ class CudaOps:
         stacked ``[gate; up]`` weight: in the GEMM's epilogue (fp32 accumulators) where the shape allows."""
         if lin.w.dtype != torch.float32 and lin.N % 32 == 0 and lin.K % 16 == 0:
             return self.linear(lin, x, swiglu=True, glu_limit=limit)
-        gu = self.linear(lin, x)
-        T, I = gu.shape[0], lin.N // 2
+        return self._glu(self.linear(lin, x), limit)
+
+    def _glu(self, gu, limit: float):
+        """The gated activation as an op of its own (``limit`` < 0: SwiGLU)."""
+        T, I = gu.shape[0], gu.shape[1] // 2
         out = torch.empty(T, I, dtype=gu.dtype, device=self.device)
         if T:
             self._check(self.lib.blz_clamped_glu(_ptr(gu), _ptr(out), T, I, limit, int(gu.dtype == torch.float32), self._stream()), "clamped_glu")
@@ -487,8 +508,9 @@ class CudaOps:
             a, rs, M = q.view(torch.uint8).contiguous(), s.float().contiguous(), xt.shape[0]
             lda = a.shape[1]
         else:
-            a = x.contiguous()
-            M, lda = a.shape[0], a.shape[1] * 2
+            # rows may be a run of columns of a wider matrix where TMA can start and step on 16 bytes
+            a = x if x.stride(1) == 1 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 else x.contiguous()
+            M, lda = a.shape[0], a.stride(0) * 2
         if argmax_parts is not None:
             out = argmax_parts[0]            # the logits are not written; any valid pointer will do
             ld_out = n_out
@@ -768,7 +790,7 @@ class CudaOps:
         return out
 
     # ------------------------------------------------------------------ differential attention
-    DIFF_SHORT_ROWS = 64       # sequences with new tokens * group up to this take the short-row kernel
+    SHORT_ROWS = 64            # sequences with new tokens * group up to this take the short-row kernel
 
     def diff_store(self, qkv, A, batch, kv, layer_idx):
         """The rows' keys and values into their pages."""
@@ -797,26 +819,121 @@ class CudaOps:
         if f32 or a.dim > 128 or a.vdim > 128 or group > 128 or a.scale <= 0:
             self._check(self.lib.blz_diff_plain(*common, _ptr(batch.seq_of_row), *shape, int(f32), st), "diff_plain")
             return out
-        lens = [b - s for s, b in zip(batch.h_q_start, batch.h_q_start[1:])]
-        limit = self.DIFF_SHORT_ROWS
-        small = [n * group for n in lens if 0 < n * group <= limit]
-        items = sum(-(-n // (128 // group)) for n in lens if n * group > limit)
+        items, small = self._split_rows(batch, a)
         if items:
-            self._check(self.lib.blz_diff_tc(*common, *shape, limit, items, st), "diff_tc")
+            self._check(self.lib.blz_diff_tc(*common, *shape, self.SHORT_ROWS, items, st), "diff_tc")
         if small:
-            rb = (max(small) + 15) // 16
-            toks = (max(small) + group - 1) // group
-            keys = min(batch.max_ctx, a.window + toks - 1) if a.window else batch.max_ctx
-            work = len(small) * a.kv_heads * rb
-            sp = max(1, min(4 * self._sm // work, (keys + 127) // 128, 32))
-            po = pm = None
-            if sp > 1:
-                n = B * a.kv_heads * rb * sp * 32
-                po = self._buf("diff_part_o", n * 128 * 4).view(torch.float32)
-                pm = self._buf("diff_part_ml", n * 2 * 4).view(torch.float32)
-                self.launches += 1
-            self._check(self.lib.blz_diff_short(*common, *shape, limit, rb, sp, _ptr(po), _ptr(pm), st), "diff_short")
+            self._check(self.lib.blz_diff_short(*common, *shape, self.SHORT_ROWS, *small, st), "diff_short")
         return out
+
+    def _split_rows(self, batch, a):
+        """How a step's sequences are shared out between the page attention kernels: row blocks for the prompt kernel, and (row
+        blocks, key splits, workspaces) of the short-row kernel or None."""
+        group, B, limit = a.group, batch.slots.numel(), self.SHORT_ROWS
+        lens = [b - s for s, b in zip(batch.h_q_start, batch.h_q_start[1:])]
+        small = [n * group for n in lens if 0 < n * group <= limit]
+        per = (128 // group) * (1 if a.maps == 2 else 2)
+        items = sum(-(-n // per) for n in lens if n * group > limit)
+        if not small:
+            return items, None
+        rb = (max(small) + 15) // 16
+        toks = (max(small) + group - 1) // group
+        keys = min(batch.max_ctx, a.window + toks - 1) if a.window else batch.max_ctx
+        work = len(small) * a.kv_heads * rb
+        sp = max(1, min(4 * self._sm // work, (keys + 127) // 128, 32))
+        po = pm = None
+        if sp > 1:
+            n = B * a.kv_heads * rb * sp * 16 * a.maps
+            po = self._buf("maps_part_o", n * 128 * 4).view(torch.float32)
+            pm = self._buf("maps_part_ml", n * 2 * 4).view(torch.float32)
+            self.launches += 1
+        return items, (rb, sp, _ptr(po), _ptr(pm))
+
+    # ------------------------------------------------------------------ post-norm residual, gated softmax attention, recurrences
+    def residual_norm(self, x, alpha: float, y, w, eps):
+        """``norm(alpha * x + y)`` in fp32 (in place of an fp32 ``x``), and the same in y's type."""
+        T, W = y.shape
+        f32 = y.dtype == torch.float32
+        dst = torch.empty(T, W, dtype=torch.float32, device=self.device) if x.dtype != torch.float32 else x
+        h = dst if f32 else torch.empty_like(y)
+        if T:
+            self._check(self.lib.blz_residual_norm(_ptr(x), int(x.dtype != torch.float32), alpha, _ptr(y), _ptr(w), eps, _ptr(dst),
+                                                   VP(0) if f32 else _ptr(h), T, W, int(f32), self._stream()), "residual_norm")
+        return dst, h
+
+    def attn_prep_pages(self, proj, M, batch, kv, layer_idx, eps):
+        """Rotated and normalised queries ``[T, heads * dim]`` of a mixer; its keys and values go to their pages."""
+        A, a, pool, c = M.attn, M.attn.spec, kv.kv[layer_idx], M.cols
+        if kv.layout != "tiles" or pool.dtype != proj.dtype:
+            raise CudaError(f"attention of {proj.dtype} rows needs 'tiles' pages of that type")
+        T = proj.shape[0]
+        q = torch.empty(T, a.heads * a.dim, dtype=proj.dtype, device=self.device)
+        rot = a.rot.dims if a.rot is not None else 0
+        self._check(self.lib.blz_attn_prep_pages(_ptr(proj), proj.stride(0), c["q"], c["k"], c["v"], _ptr(q), _ptr(pool), pool.stride(0),
+                                                 pool.stride(1), _ptr(batch.positions), _ptr(batch.slot_mapping), _ptr(A.freq), T, a.heads,
+                                                 a.kv_heads, a.dim, a.vdim, rot, int(rot > 0 and a.rot.interleaved), int(a.unit_rms), eps,
+                                                 int(proj.dtype == torch.float32), self._stream()), "attn_prep_pages")
+        return q
+
+    def soft_attention(self, proj, M, batch, kv, layer_idx, eps, out):
+        """Softmax attention of a mixer (page write included), gated and scaled, into ``out`` (columns of a wider matrix)."""
+        self.soft_attend(self.attn_prep_pages(proj, M, batch, kv, layer_idx, eps), proj, M, batch, kv, layer_idx, out)
+
+    def soft_attend(self, q, proj, M, batch, kv, layer_idx, out):
+        A, a, pool, bt = M.attn, M.attn.spec, kv.kv[layer_idx], kv.block_table
+        T, B, f32, st = q.shape[0], batch.slots.numel(), q.dtype == torch.float32, self._stream()
+        gate = VP(proj.data_ptr() + M.cols["gate"] * proj.element_size()) if a.gate else VP(0)
+        common = (_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(pool), pool.stride(0), pool.stride(1), _ptr(bt), bt.stride(0),
+                  _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(A.sink), gate, proj.stride(0))
+        shape = (T, B, a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.scale, a.out_scale)
+        if f32 or a.dim > 128 or a.vdim > 128 or a.group > 128 or a.scale <= 0:
+            self._check(self.lib.blz_soft_plain(*common, _ptr(batch.seq_of_row), *shape, int(f32), st), "soft_plain")
+            return
+        items, small = self._split_rows(batch, a)
+        if items:
+            self._check(self.lib.blz_soft_tc(*common, *shape, self.SHORT_ROWS, items, st), "soft_tc")
+        if small:
+            self._check(self.lib.blz_soft_short(*common, *shape, self.SHORT_ROWS, *small, st), "soft_short")
+
+    def short_conv(self, proj, M, batch, kv, layer_idx):
+        """Causal convolution and SiLU of a mixer's recurrent inputs ``[T, conv_dim]``; advances its history."""
+        R, r, T = M.rec, M.rec.spec, proj.shape[0]
+        y = torch.empty(T, r.conv_dim, dtype=proj.dtype, device=self.device)
+        src = VP(proj.data_ptr() + M.cols["conv"] * proj.element_size())
+        self._check(self.lib.blz_short_conv(src, proj.stride(0), _ptr(y), _ptr(kv.conv_state[layer_idx]), _ptr(R.conv_w), _ptr(R.conv_b),
+                                            _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(batch.gdn_defer),
+                                            batch.slots.numel(), r.conv_dim, r.conv, int(batch.max_q_len), int(proj.dtype == torch.float32),
+                                            self._stream()), "short_conv")
+        return y
+
+    def recurrence(self, proj, low, M, batch, kv, layer_idx, eps, out, state_only: bool = False):
+        """The recurrent mixer of a layer: convolution, recurrence, gated norm into ``out`` (columns of a wider matrix).  Sequences
+        flagged in ``batch.gdn_defer`` leave their state untouched; ``state_only`` advances the states and writes nothing."""
+        R, r, T, es, st = M.rec, M.rec.spec, proj.shape[0], proj.element_size(), self._stream()
+        y = self.short_conv(proj, M, batch, kv, layer_idx)
+        o = None if state_only else torch.empty(T, r.heads * r.vdim, dtype=torch.float32, device=self.device)
+        self.recur(y, proj, low, M, batch, kv, layer_idx, o)
+        if state_only:
+            return
+        delta = R.kind == "delta"
+        z, ldz = (low.data_ptr() + r.heads * r.dim * es, low.stride(0)) if delta else (proj.data_ptr() + M.cols["z"] * es, proj.stride(0))
+        self._check(self.lib.blz_group_norm(_ptr(o), VP(z), ldz, _ptr(R.norm_w), _ptr(out), out.stride(0), T, R.norm_groups,
+                                            o.shape[1] // R.norm_groups, R.norm_w.numel(), eps, r.out_scale, int(delta), int(not delta),
+                                            int(es == 4), st), "group_norm")
+
+    def recur(self, y, proj, low, M, batch, kv, layer_idx, o):
+        """The recurrence alone: convolved inputs ``y`` to fp32 rows ``o`` (None: the state only)."""
+        R, r, es, f32 = M.rec, M.rec.spec, proj.element_size(), int(proj.dtype == torch.float32)
+        seqs = (_ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(batch.gdn_defer), batch.slots.numel())
+        state, st, longest = kv.rec_state[layer_idx], self._stream(), int(batch.max_q_len)
+        if R.kind == "delta":
+            self._check(self.lib.blz_delta_rule(_ptr(y), y.stride(0), _ptr(low), low.stride(0), VP(proj.data_ptr() + M.cols["beta"] * es),
+                                                proj.stride(0), _ptr(R.A), _ptr(R.dt_bias), _ptr(state), _ptr(o), *seqs, r.heads,
+                                                r.kv_heads, r.dim, r.vdim, longest, f32, st), "delta_rule")
+        else:
+            self._check(self.lib.blz_state_space(_ptr(y), y.stride(0), VP(proj.data_ptr() + M.cols["dt"] * es), proj.stride(0), _ptr(R.A),
+                                                 _ptr(R.dt_bias), _ptr(R.D), _ptr(state), _ptr(o), *seqs, r.heads, r.groups, r.state,
+                                                 r.vdim, longest, f32, st), "state_space")
 
     # ------------------------------------------------------------------ head
     def argmax(self, logits, index_offset: int = 0, want_values: bool = False):

@@ -71,6 +71,17 @@ def apply_rope_neox(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> to
     return torch.cat([x1 * c - x2 * s, x2 * c + x1 * s, rest], dim=-1)
 
 
+def rotate_heads(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, interleaved: bool) -> torch.Tensor:
+    """x ``[T, H, D]``: the first ``2 * len(freq)`` dimensions of each head turned by position * frequency (fp32)."""
+    n, xf = freq.numel(), x.float()
+    ang = positions.double().view(-1, 1, 1) * freq.double()
+    c, s = torch.cos(ang).float(), torch.sin(ang).float()
+    a, b = (xf[..., 0:2 * n:2], xf[..., 1:2 * n:2]) if interleaved else (xf[..., :n], xf[..., n:2 * n])
+    ra, rb = a * c - b * s, b * c + a * s
+    turned = torch.stack([ra, rb], -1).flatten(-2) if interleaved else torch.cat([ra, rb], -1)
+    return torch.cat([turned, xf[..., 2 * n:]], -1)
+
+
 def hadamard_rotate(x: torch.Tensor) -> torch.Tensor:
     """Randomised Hadamard rotation of the last dimension (a power of two): element i changes sign when bit 15 of
     ``i * 2654435761 mod 2**32`` is set, then a Walsh-Hadamard transform scaled by 1/sqrt(D).  Orthogonal, so the dot
@@ -134,8 +145,10 @@ def kv_write(k_pool: torch.Tensor, v_pool: torch.Tensor, k: torch.Tensor, v: tor
 
 def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                     slots: Sequence[int], q_start: Sequence[int], ctx_len: Sequence[int], scale: float,
-                    tree_mask: Optional[torch.Tensor] = None, allowed: Optional[Sequence] = None) -> torch.Tensor:
-    """Causal GQA attention of q ``[T, H, D]`` over the paged pools.
+                    tree_mask: Optional[torch.Tensor] = None, allowed: Optional[Sequence] = None, window: int = 0,
+                    sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal GQA attention of q ``[T, H, D]`` over the paged pools.  ``window`` > 0: over the last ``window`` positions; ``sink``
+    ``[H]``: one more term ``exp(sink)`` in the denominators.
 
     Sequence ``b`` owns rows ``q_start[b]:q_start[b+1]``; its KV length *including* those rows is
     ``ctx_len[b]``; row i attends to positions ``<= ctx_len - q_len + i``.  With ``tree_mask`` (``[T]`` int32) row i
@@ -143,9 +156,9 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     ``allowed[b]`` (bool ``[q_len, ctx_len]`` or None) further restricts what sequence b's rows see (a sparse selection).
     """
     T, H, D = q.shape
-    KH = k_pool.shape[1]
+    KH, E = k_pool.shape[1], v_pool.shape[3]
     group = H // KH
-    out = torch.empty(T, H, D, dtype=torch.float32, device=q.device)
+    out = torch.empty(T, H, E, dtype=torch.float32, device=q.device)
     for b, slot in enumerate(slots):
         r0, r1 = q_start[b], q_start[b + 1]
         ql, n = r1 - r0, ctx_len[b]
@@ -154,12 +167,14 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
         npg = (n + PAGE - 1) // PAGE
         pages = block_table[slot, :npg].long()
         K = k_pool[pages].float().permute(1, 0, 2, 3).reshape(KH, npg * PAGE, D)[:, :n]
-        V = v_pool[pages].float().permute(1, 0, 2, 3).reshape(KH, npg * PAGE, D)[:, :n]
+        V = v_pool[pages].float().permute(1, 0, 2, 3).reshape(KH, npg * PAGE, E)[:, :n]
         qq = q[r0:r1].float().view(ql, KH, group, D).permute(1, 2, 0, 3)       # [KH, g, ql, D]
         s = torch.einsum("hgqd,hnd->hgqn", qq, K) * scale
         pos_q = torch.arange(n - ql, n, device=q.device).view(ql, 1)
         pos_k = torch.arange(n, device=q.device).view(1, n)
         mask = pos_k <= pos_q
+        if window:
+            mask = mask & (pos_k > pos_q - window)
         if tree_mask is not None:
             words = tree_mask[r0:r1].to(torch.int64).view(ql, 1) & 0xFFFFFFFF
             own = ((words >> torch.arange(min(ql, 32), device=q.device).view(1, -1)) & 1).bool()      # [ql, min(ql, 32)]
@@ -168,9 +183,11 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
         if allowed is not None and allowed[b] is not None:
             mask = mask & allowed[b]
         s = s.masked_fill(~mask, float("-inf"))
-        p = torch.softmax(s, dim=-1)
-        o = torch.einsum("hgqn,hnd->hgqd", p, V)                               # [KH, g, ql, D]
-        out[r0:r1] = o.permute(2, 0, 1, 3).reshape(ql, H, D)
+        if sink is not None:
+            s = torch.cat([s, sink.float().view(KH, group, 1, 1).expand(KH, group, ql, 1)], dim=-1)
+        p = torch.softmax(s, dim=-1)[..., :n]
+        o = torch.einsum("hgqn,hnd->hgqd", p, V)                               # [KH, g, ql, E]
+        out[r0:r1] = o.permute(2, 0, 1, 3).reshape(ql, H, E)
     return out.to(q.dtype)
 
 
@@ -251,17 +268,22 @@ def moe_forward(x: torch.Tensor, topk_w: torch.Tensor, topk_id: torch.Tensor, ex
 
 
 # ----------------------------------------------------------------------------------- Gated DeltaNet
-def gdn_conv(x: torch.Tensor, conv_state: torch.Tensor, w: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+def gdn_conv(x: torch.Tensor, conv_state: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
+             round_sum: bool = True) -> Tuple[torch.Tensor, torch.Tensor]:
     """Causal depthwise conv + SiLU over one sequence.
 
-    ``x [T, C]``, ``conv_state [C, k-1]`` (the last k-1 inputs), ``w [C, k]``.  The conv result is
-    rounded to the activation dtype before SiLU.  Returns (y [T, C], new_state).
+    ``x [T, C]``, ``conv_state [C, k-1]`` (the last k-1 inputs), ``w [C, k]``, optional ``bias [C]``.  The conv result is
+    rounded to the activation dtype before SiLU (``round_sum``).  Returns (y [T, C], new_state).
     """
     T, C = x.shape
     k = w.shape[1]
     hist = torch.cat([conv_state.t().to(x.dtype), x], dim=0)          # [k-1+T, C]
     win = hist.float().unfold(0, k, 1)                                 # [T, C, k]
-    y = (win * w.float().unsqueeze(0)).sum(-1).to(x.dtype)
+    y = (win * w.float().unsqueeze(0)).sum(-1)
+    if bias is not None:
+        y = y + bias.float()
+    if round_sum:
+        y = y.to(x.dtype)
     y = F.silu(y.float()).to(x.dtype)
     new_state = hist[-(k - 1):].t().contiguous().to(conv_state.dtype) if k > 1 else conv_state
     return y, new_state
@@ -331,6 +353,49 @@ def gdn_chunked(q, k, v, g, beta, state, chunk: int = 64):
         S = S * torch.exp(GL).view(Hv, 1, 1) + torch.einsum(
             "hjk,hjv->hkv", K * torch.exp(GL.unsqueeze(1) - G).unsqueeze(2), U)
     return out.to(v.dtype), S
+
+
+# ----------------------------------------------------------------------------------- recurrences with an fp32 state
+def delta_rule(q, k, v, a, b, A, dt_bias, state):
+    """Gated delta rule with a decay per head and key channel, one sequence: q, k ``[T, G, dk]``, v ``[T, H, dv]``, decay inputs a
+    ``[T, H, dk]``, write strengths b ``[T, H]`` (before their sigmoid), A ``[H]`` > 0, state ``[H, dk, dv]``.  fp32."""
+    T, G, dk = q.shape
+    H = v.shape[1]
+    unit = lambda x: x.float() * torch.rsqrt(x.float().pow(2).sum(-1, keepdim=True) + 1e-6)      # noqa: E731
+    q, k = [unit(x).repeat_interleave(H // G, 1) for x in (q, k)]
+    g = torch.exp(-A.view(1, H, 1) * F.softplus(a.float() + dt_bias.view(1, H, dk)))
+    beta, v, S = torch.sigmoid(b.float()), v.float(), state.clone()
+    out = torch.empty(T, H, v.shape[2], device=q.device)
+    for t in range(T):
+        S = S * g[t].unsqueeze(-1)
+        u = beta[t].unsqueeze(-1) * (v[t] - torch.einsum("hkv,hk->hv", S, k[t]))
+        S = S + k[t].unsqueeze(-1) * u.unsqueeze(1)
+        out[t] = torch.einsum("hkv,hk->hv", S, q[t]) * dk ** -0.5
+    return out, S
+
+
+def state_space(x, B, C, dt, A, dt_bias, D, state):
+    """State-space duality, one sequence: x ``[T, H, dv]``, B, C ``[T, G, N]``, dt ``[T, H]`` before its softplus, A ``[H]`` > 0,
+    state ``[H, N, dv]``.  fp32."""
+    T, H, _ = x.shape
+    x, dt, S = x.float(), F.softplus(dt.float() + dt_bias), state.clone()
+    B, C = [y.float().repeat_interleave(H // B.shape[1], 1) for y in (B, C)]
+    decay = torch.exp(-A * dt)
+    out = torch.empty_like(x)
+    for t in range(T):
+        S = S * decay[t].view(H, 1, 1) + (dt[t].view(H, 1) * B[t]).unsqueeze(-1) * x[t].unsqueeze(1)
+        out[t] = torch.einsum("hnv,hn->hv", S, C[t]) + D.view(H, 1) * x[t]
+    return out, S
+
+
+def group_norm(o, z, w, groups: int, eps: float, sigmoid: bool, gate_first: bool, post: float = 1.0):
+    """RMS norm of each of ``groups`` equal parts of fp32 rows ``[T, C]`` with a gate (``silu(z)`` or ``sigmoid(z)``) before or after
+    it and a weight that repeats over the columns.  fp32."""
+    gate = torch.sigmoid(z.float()) if sigmoid else F.silu(z.float())
+    x = o * gate if gate_first else o
+    x = x.view(x.shape[0], groups, -1)
+    x = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)).flatten(1) * w.repeat(o.shape[1] // w.numel())
+    return (x if gate_first else x * gate) * post
 
 
 # ----------------------------------------------------------------------------------- head

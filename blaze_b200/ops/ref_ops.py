@@ -112,6 +112,62 @@ class RefOps:
                                batch.h_q_start, batch.h_ctx_len, a.scale, a.window, A.lam, 1.0 - a.diff, eps)
         return o.reshape(T, -1).to(qkv.dtype)
 
+    # -------------------------------------------------------------- post-norm residual, gated softmax attention, recurrences
+    def residual_norm(self, x, alpha: float, y, w, eps):
+        """(fp32 ``norm(alpha * x + y)``, the same in y's type)."""
+        x = self.norm_rows(alpha * x.float() + y.float(), None, w, eps, torch.float32)
+        return x, x.to(y.dtype)
+
+    def soft_attention(self, proj, M, batch, kv, layer_idx, eps, out):
+        A, a, T = M.attn, M.attn.spec, proj.shape[0]
+        q = proj[:, M.cols["q"]:][:, :a.heads * a.dim].reshape(T, a.heads, a.dim)
+        k = proj[:, M.cols["k"]:][:, :a.kv_heads * a.dim].reshape(T, a.kv_heads, a.dim)
+        v = proj[:, M.cols["v"]:][:, :a.kv_heads * a.vdim].reshape(T, a.kv_heads, a.vdim)
+        if a.rot is not None:
+            q, k = [ref.rotate_heads(x, batch.positions, A.freq.double().sum(0), a.rot.interleaved) for x in (q, k)]
+        if a.unit_rms:
+            q, k = [x.float() * torch.rsqrt(x.float().pow(2).mean(-1, keepdim=True) + eps) for x in (q, k)]
+        q, valid = q.to(proj.dtype), batch.slot_mapping >= 0
+        ref.kv_write(kv.k[layer_idx], kv.v[layer_idx], k[valid], v[valid], batch.slot_mapping[valid])
+        o = ref.paged_attention(q.float(), kv.k[layer_idx], kv.v[layer_idx], kv.block_table, batch.h_slots, batch.h_q_start, batch.h_ctx_len,
+                                a.scale, window=a.window, sink=A.sink).reshape(T, -1)
+        if a.gate:
+            o = o * torch.sigmoid(proj[:, M.cols["gate"]:][:, :o.shape[1]].float())
+        out.copy_(o * a.out_scale)
+
+    def recurrence(self, proj, low, M, batch, kv, layer_idx, eps, out, state_only: bool = False):
+        """The recurrent mixer of a layer, one sequence at a time.  Sequences flagged in ``batch.h_gdn_defer`` leave their state
+        untouched; ``state_only`` advances the states and writes nothing."""
+        R, r = M.rec, M.rec.spec
+        conv_state, rec_state, defer = kv.conv_state[layer_idx], kv.rec_state[layer_idx], getattr(batch, "h_gdn_defer", None)
+        C, dt, H, dv = r.conv_dim, proj.dtype, r.heads, r.vdim
+        for b, slot in enumerate(batch.h_slots):
+            r0, r1 = batch.h_q_start[b], batch.h_q_start[b + 1]
+            n = r1 - r0
+            if n <= 0:
+                continue
+            if batch.h_ctx_len[b] == n:
+                conv_state[slot].zero_()
+                rec_state[slot].zero_()
+            y, cs = ref.gdn_conv(proj[r0:r1, M.cols["conv"]:][:, :C], conv_state[slot], R.conv_w, R.conv_b, round_sum=False)
+            if R.kind == "delta":
+                nk, hd = r.kv_heads * r.dim, H * r.dim
+                o, S = ref.delta_rule(y[:, :nk].view(n, -1, r.dim), y[:, nk:2 * nk].view(n, -1, r.dim), y[:, 2 * nk:].view(n, H, dv),
+                                      low[r0:r1, :hd].reshape(n, H, r.dim), proj[r0:r1, M.cols["beta"]:][:, :H], R.A, R.dt_bias, rec_state[slot])
+                z = low[r0:r1, hd:]
+            else:
+                ng = r.groups * r.state
+                o, S = ref.state_space(y[:, :r.inner].view(n, H, dv), y[:, r.inner:r.inner + ng].view(n, -1, r.state),
+                                       y[:, r.inner + ng:].view(n, -1, r.state), proj[r0:r1, M.cols["dt"]:][:, :H], R.A, R.dt_bias, R.D,
+                                       rec_state[slot])
+                z = proj[r0:r1, M.cols["z"]:][:, :r.inner]
+            if not (defer is not None and defer[b]):
+                conv_state[slot].copy_(cs)
+                rec_state[slot].copy_(S)
+            if not state_only:
+                out[r0:r1] = ref.group_norm(o.reshape(n, -1), z, R.norm_w, R.norm_groups, eps, R.kind == "delta", R.kind != "delta",
+                                            r.out_scale).to(dt)
+
     # -------------------------------------------------------------- MoE
     def router_topk(self, logits, k, renorm=True):
         return ref.router_topk(logits, k, renorm)

@@ -29,7 +29,7 @@ class Leader:
             return ct(items)
 
         def commit_state(items):
-            if engine.kv.gdn_layers and items:
+            if engine.kv.state_layers and items:
                 self.call("commit_state", [(s.row, keep) for s, keep in items])
             return cs(items)
         engine.commit_tree, engine.commit_state = commit_tree, commit_state

@@ -1043,7 +1043,7 @@ class Scheduler:
                 self.stats.accepted_tokens += min(accepted, real)
                 # KV of rejected draft rows is dropped; the last emitted token's KV is computed next step
                 a.computed = a.computed - len(toks) + 1 + accepted
-                if eng.kv.gdn_layers:
+                if eng.kv.state_layers:
                     eng.commit_state([(a.seq, 1 + accepted)])     # recurrent layers advance over the accepted rows only
                 eng.truncate(a.seq, a.computed)
             self._append(a, new, lps)
@@ -1232,7 +1232,7 @@ class Scheduler:
             if why in (Finish.STOP, Finish.LENGTH) and not a.req.embed_only:
                 # keep the finished conversation for follow-up turns
                 n = a.seq.length - a.seq.length % PAGE
-                if n >= PAGE and not self.engine.kv.gdn_layers:
+                if n >= PAGE and not self.engine.kv.state_layers:
                     self.cache.remember(self._key_tokens(a, n), a.seq, SnapKind.FINISH)
             self.engine.close(a.seq)
             a.seq = None

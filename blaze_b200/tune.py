@@ -142,6 +142,8 @@ def tune_model(model, rows: Iterable[int] = (256,), tuning: Optional[Tuning] = N
             lins += [L.attn.qkv, L.attn.o]
         if L.gdn is not None:
             lins += [L.gdn.in_proj, L.gdn.out_proj]
+        if L.mixer is not None:
+            lins += L.mixer.linears()
         mlp = L.mlp
         if hasattr(mlp, "down") and hasattr(mlp, "gate_up") and not hasattr(mlp, "experts"):
             lins += [mlp.down]          # gate_up runs with the SwiGLU epilogue, which has one variant

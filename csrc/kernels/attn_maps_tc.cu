@@ -1,26 +1,28 @@
-// Differential attention with an optional sliding window for long prompt portions, on tcgen05.
+// Softmax attention of one or two maps per head (attn_maps.cuh) for long prompt portions, on tcgen05.
 //
-// A CTA takes up to 128 query rows (tokens x group) of one key/value head.  The two maps of a head are the two halves of a
+// Two maps: a CTA takes up to 128 query rows (tokens x group) of one key/value head.  The two maps of a head are the two halves of a
 // ping-pong: warpgroup 0 runs the softmax of map 1, warpgroup 1 that of map 2, while the tensor core works on the other map.
+// One map: a CTA takes two blocks of up to 128 query rows; the blocks are the two halves, and share keys and values.
 //   S_m = Q_m K_m^T   A = Q_m [128 x dim], B = K_m [128 keys x dim], both K-major in shared memory
 //   O_m += P_m V      A = P_m in tensor memory, B = V [keys x vdim], the pages' token-major blocks read as an MN-major operand
 // Tensor memory (512 columns): S_1 | S_2 | O_1 | O_2, 128 each.  A map's weights overwrite its scores as two bf16 halves, value
 // and remainder (64 columns each), and both enter the value product, so a weight is not rounded to 8 bits.  O accumulates in
 // tensor memory over the key tiles; a row's running maximum moves only when its scores outgrow it by 2^8, and then the row's
 // thread rescales O there (QK of a tile is issued behind PV of the tile before, so O is quiet while scores are looked at).
-// At the end each thread joins one half of a row's columns: a1 - lam a2, the head's RMS norm, the output.
+// At the end, with two maps each thread joins one half of a row's columns: a1 - lam a2, the head's RMS norm, the output; with one
+// each thread divides its row by the sum of its weights (and the sink), gates it and writes it.
 //
-// Roles (three warpgroups): warps 0-3 / 4-7 softmax of map 1 / 2 (one row per thread), warp 8 loads pages with bulk copies,
+// Roles (three warpgroups): warps 0-3 / 4-7 softmax of half 1 / 2 (one row per thread), warp 8 loads pages with bulk copies,
 // warp 9 issues the MMAs.  setmaxnreg moves registers from the last warpgroup to the softmax ones (216 / 216 / 72 of 3 x 168).
 #include "blaze/attn.cuh"
-#include "blaze/attn_diff.cuh"
+#include "blaze/attn_maps.cuh"
 #include "blaze/host.h"
 
 namespace blz {
 
 static constexpr int kTcThreads = 384;
-template <int N> __device__ __forceinline__ void diff_reg_inc() { asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(N)); }
-template <int N> __device__ __forceinline__ void diff_reg_dec() { asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(N)); }
+template <int N> __device__ __forceinline__ void maps_reg_inc() { asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(N)); }
+template <int N> __device__ __forceinline__ void maps_reg_dec() { asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(N)); }
 static constexpr float kTcLazy = 8.f;
 
 // D += A (tensor memory) x B (shared memory)
@@ -39,18 +41,19 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16
       : "memory");
 }
 
-struct DiffTc {
+struct MapsTc {
   int ks, vs;                  // K and V ring depths
 };
 
-__global__ void __launch_bounds__(kTcThreads, 1) diff_tc_kernel(DiffParams p, DiffTc c, int vec_q, int vec_o) {
+template <int MAPS>
+__global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, MapsTc c, int vec_q, int vec_o) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~uintptr_t(127));
-  const int dp = p.dp(), vp = p.vp(), group = p.group(), tpb = 128 / group;
-  const int q_bytes = 128 * dp * 2, k_bytes = 128 * dp * 2, v_bytes = 128 * vp * 2;     // one map's operands; one tile of values
+  const int dp = p.dp(), vp = p.vp(), group = p.group(), tph = 128 / group, tpb = MAPS == 1 ? 2 * tph : tph;   // tokens per half, per CTA
+  const int q_bytes = 128 * dp * 2, k_bytes = 128 * dp * 2, v_bytes = 128 * vp * 2;     // one half's queries, one map's keys; one tile of values
   uint8_t* sQ = smem;                                  // [2]
-  uint8_t* sK = sQ + 2 * q_bytes;                      // [ks][2]
-  uint8_t* sV = sK + c.ks * 2 * k_bytes;               // [vs]
+  uint8_t* sK = sQ + 2 * q_bytes;                      // [ks][MAPS]
+  uint8_t* sV = sK + c.ks * MAPS * k_bytes;               // [vs]
   float* s_l = reinterpret_cast<float*>(sV + c.vs * v_bytes);   // [2][128] sums of the weights
   float* s_ss = s_l + 256;                             // [2][128] sums of squares of a row's halves
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_ss + 256);
@@ -102,11 +105,11 @@ __global__ void __launch_bounds__(kTcThreads, 1) diff_tc_kernel(DiffParams p, Di
   const int b = s_item[0], q0 = s_item[1];
   const int g = blockIdx.y, bb = max(b, 0);
   const int r0 = p.q_start[bb], qlen = p.q_start[bb + 1] - r0, pos0 = p.ctx_len[bb] - qlen;
-  const int ntok = b < 0 ? 0 : min(qlen - q0, tpb), nrows = ntok * group;
+  const int ntok = b < 0 ? 0 : min(qlen - q0, tpb);
   const int pg_lo = first_key(pos0 + q0, p.window) >> 4, pg_hi = (pos0 + q0 + ntok - 1) >> 4;
   const int n = b < 0 ? 0 : (pg_hi - pg_lo + 8) / 8;               // tiles of 8 pages
   if (warp >= 8) {
-    diff_reg_dec<72>();
+    maps_reg_dec<72>();
     if (warp == 8) {
       // -------------------------------------------------------------- page loader
       const int* bt = p.block_table + (size_t)p.slots[b] * p.bt_stride;
@@ -116,12 +119,12 @@ __global__ void __launch_bounds__(kTcThreads, 1) diff_tc_kernel(DiffParams p, Di
       for (; i < n; ++i) {
         const int ks = i % c.ks, vs = i % c.vs;
         const int pidx = pg_lo + i * 8 + pg;
-        const int page = (lane < 24 && pidx <= pg_hi) ? bt[pidx] : 0;        // page 0: zeros
+        const int page = (lane < 8 * (MAPS + 1) && pidx <= pg_hi) ? bt[pidx] : 0;        // page 0: zeros
         const __nv_bfloat16* src = pool + (size_t)page * p.page_stride;
         if (!__all_sync(0xffffffffu, mbar_wait(&k_empty[ks], (uint32_t)(((i / c.ks) & 1) ^ 1), abort_flag, p.status))) break;
-        if (lane == 0) mbar_expect_tx(&k_full[ks], 2 * k_bytes);
+        if (lane == 0) mbar_expect_tx(&k_full[ks], MAPS * k_bytes);
         __syncwarp();
-        if (part < 2) bulk_load(sK + (ks * 2 + part) * k_bytes + pg * 32 * dp, src + part * 16 * dp, 32 * dp, &k_full[ks]);
+        if (part < MAPS) bulk_load(sK + (ks * MAPS + part) * k_bytes + pg * 32 * dp, src + part * 16 * dp, 32 * dp, &k_full[ks]);
         if (!__all_sync(0xffffffffu, mbar_wait(&v_empty[vs], (uint32_t)(((i / c.vs) & 1) ^ 1), abort_flag, p.status))) {
           // this tile's keys are on their way: they land before the block may end
           const long long t0 = clock64();
@@ -130,7 +133,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) diff_tc_kernel(DiffParams p, Di
         }
         if (lane == 0) mbar_expect_tx(&v_full[vs], v_bytes);
         __syncwarp();
-        if (part == 2) bulk_load(sV + vs * v_bytes + pg * 32 * vp, src + 2 * 16 * dp, 32 * vp, &v_full[vs]);
+        if (part == MAPS) bulk_load(sV + vs * v_bytes + pg * 32 * vp, src + MAPS * 16 * dp, 32 * vp, &v_full[vs]);
         __syncwarp();
       }
       if (i < n) {
@@ -146,7 +149,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) diff_tc_kernel(DiffParams p, Di
       if (lane == 0) {
         const uint32_t id_s = make_idesc(1, 1, 128, 128), id_o = make_idesc(1, 1, 128, (uint32_t)vp, 0, 1);
         auto qk = [&](int m, int i) {
-          const uint32_t qa = smem_u32(sQ + m * q_bytes), ka = smem_u32(sK + ((i % c.ks) * 2 + m) * k_bytes);
+          const uint32_t qa = smem_u32(sQ + m * q_bytes), ka = smem_u32(sK + ((i % c.ks) * MAPS + (MAPS == 2 ? m : 0)) * k_bytes);
           for (int s = 0; s < dp / 16; ++s)
             mma_f16(tmem + m * 128, make_smem_desc(qa + s * 256, 128, dp * 16, kSwzNone),
                     make_smem_desc(ka + s * 256, 128, dp * 16, kSwzNone), id_s, s > 0);
@@ -182,16 +185,17 @@ __global__ void __launch_bounds__(kTcThreads, 1) diff_tc_kernel(DiffParams p, Di
       }
     }
   } else {
-    diff_reg_inc<216>();
+    maps_reg_inc<216>();
     if (n > 0) {
-      // -------------------------------------------------------------- softmax of one map (one row per thread)
+      // -------------------------------------------------------------- softmax of one half (one row per thread)
       const int m = warp >> 2, r = threadIdx.x & 127;
       const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
-      const bool live = r < nrows;
-      const int tq = q0 + r / group, head = g * group + r % group;
+      const int t0 = q0 + (MAPS == 1 ? m * tph : 0);               // this half's first token
+      const bool live = r < tph * group && t0 + r / group < q0 + ntok;
+      const int tq = t0 + r / group, head = g * group + r % group;
       const int pos = live ? pos0 + tq : -1, lo = first_key(pos, p.window);
       {
-        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.qkv) + (size_t)(r0 + tq) * p.ld + (size_t)(head * 2 + m) * p.dim;
+        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)(r0 + tq) * p.ld + (size_t)(MAPS == 2 ? head * 2 + m : head) * p.dim;
         __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(sQ + m * q_bytes);
         for (int j = 0; j < dp; j += 8) {
           uint4 u = make_uint4(0, 0, 0, 0);
@@ -209,7 +213,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) diff_tc_kernel(DiffParams p, Di
         __syncwarp();
         if (lane == 0) mbar_arrive(q_full);
       }
-      const float sc = p.scale * 1.4426950408889634f;
+      const float sc = p.scale * kLog2e;
       const uint32_t s_addr = tmem + m * 128 + lanes, o_addr = tmem + 256 + m * 128 + lanes;
       float mx = -INFINITY, l = 0.f;
       bool ok = true;
@@ -275,49 +279,86 @@ __global__ void __launch_bounds__(kTcThreads, 1) diff_tc_kernel(DiffParams p, Di
         __syncwarp();
         if (lane == 0) mbar_arrive(&p_full[m]);
       }
-      s_l[m * 128 + r] = l;
-      // both maps are done: this thread joins columns [m * half, ...) of its row
-      if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&o_full[0], 0, abort_flag, p.status) && mbar_wait(&o_full[1], 0, abort_flag, p.status));
-      bar_sync(1, 256);
-      tc_fence_after();
-      const float i1 = 1.f / s_l[r], i2 = p.lam / s_l[128 + r];
-      const int h16 = (vp / 16 + 1) / 2 * 16, c0 = m * h16, c1 = m ? vp : h16;     // 16-column groups of this half: at most 4
-      float o[64];
-      float ss = 0.f;
-#pragma unroll
-      for (int k = 0; k < 4; ++k) {
-        if (c0 + k * 16 < c1 && ok) {
-          uint32_t x[16], y[16];
-          tmem_ld16(tmem + 256 + lanes + c0 + k * 16, x);
-          tmem_ld16(tmem + 384 + lanes + c0 + k * 16, y);
+      if constexpr (MAPS == 1) {
+        if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&o_full[m], 0, abort_flag, p.status));
+        tc_fence_after();
+        const float f = 1.f / (l + (p.sink ? ex2(p.sink[head] * kLog2e - mx) : 0.f));
+        __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(r0 + tq) * p.ld_out + (size_t)head * p.vdim;
+        const __nv_bfloat16* gate =
+            p.gate ? reinterpret_cast<const __nv_bfloat16*>(p.gate) + (size_t)(r0 + tq) * p.ld_gate + (size_t)head * p.vdim : nullptr;
+        for (int k = 0; k < vp && ok; k += 16) {
+          uint32_t x[16];
+          tmem_ld16(o_addr + k, x);
           tmem_ld_wait();
+          if (live) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) {
-            const float d = __uint_as_float(x[j]) * i1 - __uint_as_float(y[j]) * i2;   // padded columns are zero in both
-            o[k * 16 + j] = d;
-            ss = fmaf(d, d, ss);
+            for (int h = 0; h < 16; h += 8) {
+              const int col = k + h;
+              float y[8];
+#pragma unroll
+              for (int j = 0; j < 8; ++j) y[j] = __uint_as_float(x[h + j]) * f * p.post;
+              if (vec_o && col + 8 <= p.vdim) {
+                if (gate) {
+                  const uint4 u = *reinterpret_cast<const uint4*>(gate + col);
+                  const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&u);
+#pragma unroll
+                  for (int j = 0; j < 8; ++j) y[j] = __fdividef(y[j], 1.f + __expf(-bf2f(e[j])));
+                }
+                *reinterpret_cast<uint4*>(out + col) = make_uint4(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]),
+                                                                  pack_bf16x2(y[4], y[5]), pack_bf16x2(y[6], y[7]));
+              } else {
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                  if (col + j < p.vdim) out[col + j] = __float2bfloat16(gate ? y[j] / (1.f + __expf(-bf2f(gate[col + j]))) : y[j]);
+              }
+            }
           }
         }
-      }
-      s_ss[m * 128 + r] = ss;
-      bar_sync(1, 256);
-      if (ok && live) {
-        const float f = p.post / sqrtf((s_ss[r] + s_ss[128 + r]) / (float)p.vdim + p.eps);
-        __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + ((size_t)(r0 + tq) * p.heads + head) * p.vdim;
+      } else {
+        s_l[m * 128 + r] = l;
+        // both maps are done: this thread joins columns [m * half, ...) of its row
+        if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&o_full[0], 0, abort_flag, p.status) && mbar_wait(&o_full[1], 0, abort_flag, p.status));
+        bar_sync(1, 256);
+        tc_fence_after();
+        const float i1 = 1.f / s_l[r], i2 = p.lam / s_l[128 + r];
+        const int h16 = (vp / 16 + 1) / 2 * 16, c0 = m * h16, c1 = m ? vp : h16;     // 16-column groups of this half: at most 4
+        float o[64];
+        float ss = 0.f;
 #pragma unroll
-        for (int k = 0; k < 64; k += 8) {
-          const int col = c0 + k;
-          if (col >= c1) break;
-          if (vec_o && col + 8 <= p.vdim) {
-            *reinterpret_cast<uint4*>(out + col) = make_uint4(pack_bf16x2(o[k] * f, o[k + 1] * f), pack_bf16x2(o[k + 2] * f, o[k + 3] * f),
-                                                              pack_bf16x2(o[k + 4] * f, o[k + 5] * f), pack_bf16x2(o[k + 6] * f, o[k + 7] * f));
-          } else {
+        for (int k = 0; k < 4; ++k) {
+          if (c0 + k * 16 < c1 && ok) {
+            uint32_t x[16], y[16];
+            tmem_ld16(tmem + 256 + lanes + c0 + k * 16, x);
+            tmem_ld16(tmem + 384 + lanes + c0 + k * 16, y);
+            tmem_ld_wait();
 #pragma unroll
-            for (int j = 0; j < 8; ++j)
-              if (col + j < p.vdim) out[col + j] = __float2bfloat16(o[k + j] * f);
+            for (int j = 0; j < 16; ++j) {
+              const float d = __uint_as_float(x[j]) * i1 - __uint_as_float(y[j]) * i2;   // padded columns are zero in both
+              o[k * 16 + j] = d;
+              ss = fmaf(d, d, ss);
+            }
           }
         }
-      }
+        s_ss[m * 128 + r] = ss;
+        bar_sync(1, 256);
+        if (ok && live) {
+          const float f = p.post / sqrtf((s_ss[r] + s_ss[128 + r]) / (float)p.vdim + p.eps);
+          __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(r0 + tq) * p.ld_out + (size_t)head * p.vdim;
+#pragma unroll
+          for (int k = 0; k < 64; k += 8) {
+            const int col = c0 + k;
+            if (col >= c1) break;
+            if (vec_o && col + 8 <= p.vdim) {
+              *reinterpret_cast<uint4*>(out + col) = make_uint4(pack_bf16x2(o[k] * f, o[k + 1] * f), pack_bf16x2(o[k + 2] * f, o[k + 3] * f),
+                                                                pack_bf16x2(o[k + 4] * f, o[k + 5] * f), pack_bf16x2(o[k + 6] * f, o[k + 7] * f));
+            } else {
+#pragma unroll
+              for (int j = 0; j < 8; ++j)
+                if (col + j < p.vdim) out[col + j] = __float2bfloat16(o[k + j] * f);
+            }
+          }
+        }
+  }
     }
   }
   tc_fence_before();
@@ -328,34 +369,57 @@ __global__ void __launch_bounds__(kTcThreads, 1) diff_tc_kernel(DiffParams p, Di
   }
 }
 
+template <int MAPS>
+static int run_tc(const MapsParams& p, int items, cudaStream_t s) {
+  if (p.T <= 0 || p.B <= 0 || p.heads < 1 || p.kv_heads < 1 || p.kv_heads > 65535 || p.heads % p.kv_heads || p.group() > 128 || p.dim < 1 ||
+      p.dim > 128 || p.vdim < 1 || p.vdim > 128 || p.window < 0 || items < 1)
+    return (int)cudaErrorInvalidValue;
+  if ((p.page_stride * 2) % 16 || (p.head_stride * 2) % 16 || (reinterpret_cast<uintptr_t>(p.pool) & 15)) return (int)cudaErrorInvalidValue;
+  const int q_bytes = 256 * p.dp() * 2, k_bytes = MAPS * 128 * p.dp() * 2, v_bytes = 128 * p.vp() * 2, fixed = 128 + 2048 + 256;
+  MapsTc c = {2, 2};
+  auto total = [&]() { return fixed + q_bytes + c.ks * k_bytes + c.vs * v_bytes; };
+  if (total() > 227 * 1024) c.ks = 1;
+  if (total() > 227 * 1024) return (int)cudaErrorInvalidValue;
+  const int vec_q = (reinterpret_cast<uintptr_t>(p.q) & 15) == 0 && p.ld % 8 == 0 && p.dim % 8 == 0;
+  const int vec_o = (reinterpret_cast<uintptr_t>(p.out) & 15) == 0 && p.ld_out % 8 == 0 && p.vdim % 8 == 0 &&
+                    (!p.gate || ((reinterpret_cast<uintptr_t>(p.gate) & 15) == 0 && p.ld_gate % 8 == 0));
+  static PerDeviceOnce once;
+  cudaError_t e = once.smem_limit(maps_tc_kernel<MAPS>, 227 * 1024);
+  if (e != cudaSuccess) return (int)e;
+  return (int)launch_pdl(maps_tc_kernel<MAPS>, dim3(items, p.kv_heads), dim3(kTcThreads), total(), s, p, c, vec_q, vec_o);
+}
+
 }  // namespace blz
 
-// bf16; the sequences with more than max_rows = new tokens * group rows, `items` row blocks of 128 / group tokens in all.
-// dim, vdim <= 128, group <= 128.
+// Differential attention, bf16; the sequences with more than max_rows = new tokens * group rows, `items` row blocks of 128 / group
+// tokens in all.  dim, vdim <= 128, group <= 128.
 BLZ_API int blz_diff_tc(const void* qkv, long long ld, void* out, void* pool, long long page_stride, long long head_stride,
                         const int* block_table, int bt_stride, const int* slots, const int* q_start, const int* ctx_len, int T, int B,
                         int heads, int kv_heads, int dim, int vdim, int window, float scale, float lam, float post, float eps,
                         int max_rows, int items, cudaStream_t s) {
   using namespace blz;
-  if (T <= 0 || B <= 0 || heads < 1 || kv_heads < 1 || kv_heads > 65535 || heads % kv_heads || heads / kv_heads > 128 || dim < 1 ||
-      dim > 128 || vdim < 1 || vdim > 128 || window < 0 || items < 1)
-    return (int)cudaErrorInvalidValue;
-  if ((page_stride * 2) % 16 || (head_stride * 2) % 16 || (reinterpret_cast<uintptr_t>(pool) & 15)) return (int)cudaErrorInvalidValue;
-  DiffParams p = {};
-  p.qkv = qkv; p.ld = ld; p.out = out; p.pool = pool; p.page_stride = page_stride; p.head_stride = head_stride;
+  MapsParams p = {};
+  p.q = qkv; p.ld = ld; p.out = out; p.ld_out = (long long)heads * vdim; p.pool = pool; p.page_stride = page_stride; p.head_stride = head_stride;
   p.block_table = block_table; p.bt_stride = bt_stride; p.slots = slots; p.q_start = q_start; p.ctx_len = ctx_len;
-  p.T = T; p.B = B; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window;
+  p.T = T; p.B = B; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.maps = 2;
   p.scale = scale; p.lam = lam; p.post = post; p.eps = eps; p.max_rows = max_rows;
   p.status = status_word();
-  const int q_bytes = 256 * p.dp() * 2, k_bytes = 256 * p.dp() * 2, v_bytes = 128 * p.vp() * 2, fixed = 128 + 2048 + 256;
-  DiffTc c = {2, 2};
-  auto total = [&]() { return fixed + q_bytes + c.ks * k_bytes + c.vs * v_bytes; };
-  if (total() > 227 * 1024) c.ks = 1;
-  if (total() > 227 * 1024) return (int)cudaErrorInvalidValue;
-  const int vec_q = (reinterpret_cast<uintptr_t>(qkv) & 15) == 0 && ld % 8 == 0 && dim % 8 == 0;
-  const int vec_o = (reinterpret_cast<uintptr_t>(out) & 15) == 0 && vdim % 8 == 0;
-  static PerDeviceOnce once;
-  cudaError_t e = once.smem_limit(diff_tc_kernel, 227 * 1024);
-  if (e != cudaSuccess) return (int)e;
-  return (int)launch_pdl(diff_tc_kernel, dim3(items, kv_heads), dim3(kTcThreads), total(), s, p, c, vec_q, vec_o);
+  return run_tc<2>(p, items, s);
+}
+
+// One softmax map per head with optional sink and gate (see blz_soft_plain), bf16; the sequences with more than max_rows rows,
+// `items` row blocks of 2 * (128 / group) tokens in all.  dim, vdim <= 128, group <= 128.
+BLZ_API int blz_soft_tc(const void* q, long long ld, void* out, long long ld_out, void* pool, long long page_stride, long long head_stride,
+                        const int* block_table, int bt_stride, const int* slots, const int* q_start, const int* ctx_len, const float* sink,
+                        const void* gate, long long ld_gate, int T, int B, int heads, int kv_heads, int dim, int vdim, int window,
+                        float scale, float post, int max_rows, int items, cudaStream_t s) {
+  using namespace blz;
+  MapsParams p = {};
+  p.q = q; p.ld = ld; p.out = out; p.ld_out = ld_out; p.pool = pool; p.page_stride = page_stride; p.head_stride = head_stride;
+  p.block_table = block_table; p.bt_stride = bt_stride; p.slots = slots; p.q_start = q_start; p.ctx_len = ctx_len;
+  p.sink = sink; p.gate = gate; p.ld_gate = ld_gate;
+  p.T = T; p.B = B; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.maps = 1;
+  p.scale = scale; p.post = post; p.max_rows = max_rows;
+  p.status = status_word();
+  return run_tc<1>(p, items, s);
 }

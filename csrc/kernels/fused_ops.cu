@@ -50,6 +50,10 @@ __global__ void embed_kernel(const __nv_bfloat16* __restrict__ table, const int*
   const int t = blockIdx.x;
   int tok = tokens[t];
   tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);
+  if (H % 8) {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)t * H + i] = table[(size_t)tok * H + i];
+    return;
+  }
   const uint4* src = reinterpret_cast<const uint4*>(table + (size_t)tok * H);
   uint4* dst = reinterpret_cast<uint4*>(out + (size_t)t * H);
   for (int i = threadIdx.x; i < H / 8; i += blockDim.x) dst[i] = src[i];
@@ -740,7 +744,6 @@ static inline int norm_threads(int H) {
 }
 
 BLZ_API int blz_embed(const void* table, const int* tokens, void* out, int T, int H, int vocab, cudaStream_t s) {
-  if (H % 8) return (int)cudaErrorInvalidValue;
   if (T == 0) return 0;
   launch_pdl(embed_kernel, dim3(T), dim3(256), 0, s, (const bf16*)table, tokens, (bf16*)out, H, vocab);
   return (int)cudaGetLastError();

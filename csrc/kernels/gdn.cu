@@ -1,91 +1,119 @@
 // Gated DeltaNet (linear-attention) layer kernels:
-//   conv      : causal depthwise conv (kernel <= 8) + SiLU over variable-length sequences with a per-sequence state of the
-//               last k-1 inputs (reference: kernels/src/cuda/ops_basic.cu gdn_conv_kernel :319)
+//   conv      : causal depthwise conv (kernel <= 8, optional bias, bf16 or fp32) + SiLU over variable-length sequences with a
+//               per-sequence state of the last k-1 inputs (reference: kernels/src/cuda/ops_basic.cu gdn_conv_kernel :319)
 //   recurrent : the gated delta rule, token by token, with the gates computed in the kernel
 //               g = -exp(A_log) * softplus(a + dt_bias), beta = bf16(sigmoid(b))      (ops_basic.cu gdn_gate :301)
 //               S <- S * exp(g);  delta = (v - S^T k) * beta;  S <- S + k delta^T;  o = S^T q
 //               with q, k L2-normalised and q scaled by dk^-1/2               (kernels/src/cuda/gdn_recurrent.cu:27-92)
 //   gated norm: per-head RMSNorm of o times silu(z)                           (ops_basic.cu gated_rmsnorm_kernel :70)
-// State layout: conv_state [rows, C, k-1] bf16, rec_state [rows, Hv, dk, dv] fp32; rows are sequence slots.
+// State layout: conv_state [rows, C, k-1] in the activation type, rec_state [rows, Hv, dk, dv] fp32; rows are sequence slots.
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
 
 namespace blz {
 
+__device__ __forceinline__ float cv_ld(const float* p) { return *p; }
+__device__ __forceinline__ float cv_ld(const __nv_bfloat16* p) { return bf2f(*p); }
+__device__ __forceinline__ void cv_st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void cv_st(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+template <typename T>
+struct ConvParams {
+  const T* x;                  // [T, ldx]
+  T* y;                        // [T, C]
+  T* conv_state;               // [rows, C, k - 1]
+  const T* w;                  // [C, k]
+  const float* bias;           // [C] or null
+  const int *slots, *q_start, *ctx_len, *no_store;
+  long long ldx;
+  int C;
+  int round;                   // the sum is rounded to the activation type before the activation
+};
+
+template <typename T>
+__device__ __forceinline__ float conv_act(float acc, int round) {
+  if constexpr (sizeof(T) == 4) return acc / (1.f + expf(-acc));
+  const float r = round ? bf2f(__float2bfloat16(acc)) : acc;
+  return r / (1.f + __expf(-r));
+}
+
 // grid (ceil(C / 128), B); thread = channel; walks the sequence's tokens in order
-template <int KW>
-__global__ void gdn_conv_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat16* __restrict__ y,
-                                __nv_bfloat16* __restrict__ conv_state, const __nv_bfloat16* __restrict__ w,
-                                const int* __restrict__ slots, const int* __restrict__ q_start, const int* __restrict__ ctx_len,
-                                const int* __restrict__ no_store, int C, int max_rows) {
+template <typename T, int KW>
+__global__ void gdn_conv_kernel(ConvParams<T> p, int max_rows) {
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   const int b = blockIdx.y;
-  if (c >= C) return;
-  const int r0 = q_start[b], n = q_start[b + 1] - r0;
+  if (c >= p.C) return;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
   if (n <= 0 || n > max_rows) return;
-  const bool fresh = ctx_len[b] - n == 0;
-  __nv_bfloat16* st = conv_state + ((size_t)slots[b] * C + c) * (KW - 1);
+  const bool fresh = p.ctx_len[b] - n == 0;
+  T* st = p.conv_state + ((size_t)p.slots[b] * p.C + c) * (KW - 1);
+  const float b0 = p.bias ? p.bias[c] : 0.f;
   float h[KW];
   float wt[KW];
 #pragma unroll
-  for (int j = 0; j < KW - 1; ++j) h[j] = fresh ? 0.f : bf2f(st[j]);
+  for (int j = 0; j < KW - 1; ++j) h[j] = fresh ? 0.f : cv_ld(st + j);
 #pragma unroll
-  for (int j = 0; j < KW; ++j) wt[j] = bf2f(w[(size_t)c * KW + j]);
+  for (int j = 0; j < KW; ++j) wt[j] = cv_ld(p.w + (size_t)c * KW + j);
   for (int t = 0; t < n; ++t) {
-    h[KW - 1] = bf2f(x[(size_t)(r0 + t) * ldx + c]);
-    float acc = 0.f;
+    h[KW - 1] = cv_ld(p.x + (size_t)(r0 + t) * p.ldx + c);
+    float acc = b0;
 #pragma unroll
     for (int j = 0; j < KW; ++j) acc += h[j] * wt[j];
-    const float r = bf2f(__float2bfloat16(acc));
-    y[(size_t)(r0 + t) * C + c] = __float2bfloat16(r / (1.f + __expf(-r)));
+    cv_st(p.y + (size_t)(r0 + t) * p.C + c, conv_act<T>(acc, p.round));
 #pragma unroll
     for (int j = 0; j < KW - 1; ++j) h[j] = h[j + 1];
   }
-  if (no_store != nullptr && no_store[b]) return;      // speculative rows: the state advances when they are replayed
+  if (p.no_store != nullptr && p.no_store[b]) return;      // speculative rows: the state advances when they are replayed
 #pragma unroll
-  for (int j = 0; j < KW - 1; ++j) st[j] = __float2bfloat16(h[j]);
+  for (int j = 0; j < KW - 1; ++j) cv_st(st + j, h[j]);
 }
 
 // Long token runs (prompts): the same convolution with the tokens spread over the grid.  grid (ceil(C / 128), B, segments):
 // segment z handles tokens [z * SEG, (z + 1) * SEG) of the sequence; the k-1 inputs before its first token come from the input
-// itself (or from the state for the run's first tokens); the CTA that holds the run's last token writes the new state.
-template <int KW>
-__global__ void gdn_conv_par_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat16* __restrict__ y,
-                                    __nv_bfloat16* __restrict__ conv_state, const __nv_bfloat16* __restrict__ w,
-                                    const int* __restrict__ slots, const int* __restrict__ q_start, const int* __restrict__ ctx_len,
-                                    const int* __restrict__ no_store, int C, int seg, int min_rows) {
+// itself (or from the state for the run's first tokens).  The new state is a kernel of its own (the first segment reads the old).
+template <typename T, int KW>
+__global__ void gdn_conv_par_kernel(ConvParams<T> p, int seg, int min_rows) {
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   const int b = blockIdx.y;
-  if (c >= C) return;
-  const int r0 = q_start[b], n = q_start[b + 1] - r0;
+  if (c >= p.C) return;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
   if (n < min_rows) return;                        // short runs belong to the sequential kernel
   const int t0 = blockIdx.z * seg, t1 = min(n, t0 + seg);
   if (t0 >= n) return;
-  const bool fresh = ctx_len[b] - n == 0;
-  __nv_bfloat16* st = conv_state + ((size_t)slots[b] * C + c) * (KW - 1);
+  const bool fresh = p.ctx_len[b] - n == 0;
+  const T* st = p.conv_state + ((size_t)p.slots[b] * p.C + c) * (KW - 1);
+  const float b0 = p.bias ? p.bias[c] : 0.f;
   float h[KW];
   float wt[KW];
 #pragma unroll
   for (int j = 0; j < KW - 1; ++j) {
     const int t = t0 - (KW - 1) + j;              // input position of history slot j (negative: before this run)
-    h[j] = t >= 0 ? bf2f(x[(size_t)(r0 + t) * ldx + c]) : (fresh ? 0.f : bf2f(st[KW - 1 + t]));
+    h[j] = t >= 0 ? cv_ld(p.x + (size_t)(r0 + t) * p.ldx + c) : (fresh ? 0.f : cv_ld(st + (KW - 1) + t));
   }
 #pragma unroll
-  for (int j = 0; j < KW; ++j) wt[j] = bf2f(w[(size_t)c * KW + j]);
+  for (int j = 0; j < KW; ++j) wt[j] = cv_ld(p.w + (size_t)c * KW + j);
+#pragma unroll 4
   for (int t = t0; t < t1; ++t) {
-    h[KW - 1] = bf2f(x[(size_t)(r0 + t) * ldx + c]);
-    float acc = 0.f;
+    h[KW - 1] = cv_ld(p.x + (size_t)(r0 + t) * p.ldx + c);
+    float acc = b0;
 #pragma unroll
     for (int j = 0; j < KW; ++j) acc += h[j] * wt[j];
-    const float r = bf2f(__float2bfloat16(acc));
-    y[(size_t)(r0 + t) * C + c] = __float2bfloat16(r / (1.f + __expf(-r)));
+    cv_st(p.y + (size_t)(r0 + t) * p.C + c, conv_act<T>(acc, p.round));
 #pragma unroll
     for (int j = 0; j < KW - 1; ++j) h[j] = h[j + 1];
   }
-  if (t1 == n && !(no_store != nullptr && no_store[b])) {
+}
+// the state after a long run: its last k-1 inputs (such a run has at least that many)
+template <typename T, int KW>
+__global__ void gdn_conv_state_kernel(ConvParams<T> p, int min_rows) {
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int b = blockIdx.y;
+  if (c >= p.C) return;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
+  if (n < min_rows || (p.no_store != nullptr && p.no_store[b])) return;
+  T* st = p.conv_state + ((size_t)p.slots[b] * p.C + c) * (KW - 1);
 #pragma unroll
-    for (int j = 0; j < KW - 1; ++j) st[j] = __float2bfloat16(h[j]);
-  }
+  for (int j = 0; j < KW - 1; ++j) st[j] = p.x[(size_t)(r0 + n - (KW - 1) + j) * p.ldx + c];
 }
 
 // grid (B, Hv, DV / 32), 128 threads: thread = (dv column c = tid % 32, dk quarter qt = tid / 32); the state slice
@@ -184,41 +212,47 @@ typedef __nv_bfloat16 bf16;
 // blz_gdn_recurrent: out may be null (state advance only, used when accepted rows are replayed).
 // max_q: the longest token run of the batch (host knowledge).  Runs of at least 64 tokens are convolved with the tokens
 // spread over the grid (64-token segments), the others by one thread per channel walking the run.
-static int gdn_conv_impl(const void* x, long long ldx, void* y, void* conv_state, const void* w, const int* slots,
-                         const int* q_start, const int* ctx_len, const int* no_store, int B, int C, int kw, int max_q,
-                         cudaStream_t s) {
-  if (B == 0) return 0;
+template <typename T, int KW>
+static void launch_conv(const ConvParams<T>& p, int B, int max_q, cudaStream_t s) {
   constexpr int SEG = 64, LONG = 64;
   const bool par = max_q >= LONG;
-  dim3 grid((C + 127) / 128, B);
-  dim3 grid_par((C + 127) / 128, B, par ? (max_q + SEG - 1) / SEG : 1);
-#define BLZ_CONV(K)                                                                                                         \
-  do {                                                                                                                      \
-    if (par)                                                                                                                \
-      gdn_conv_par_kernel<K><<<grid_par, 128, 0, s>>>((const bf16*)x, ldx, (bf16*)y, (bf16*)conv_state, (const bf16*)w, slots, \
-                                                      q_start, ctx_len, no_store, C, SEG, LONG);                            \
-    if (!par || B > 1)                                                                                                      \
-      gdn_conv_kernel<K><<<grid, 128, 0, s>>>((const bf16*)x, ldx, (bf16*)y, (bf16*)conv_state, (const bf16*)w, slots,      \
-                                              q_start, ctx_len, no_store, C, par ? LONG - 1 : 0x7fffffff);                  \
-  } while (0)
+  const dim3 grid((p.C + 127) / 128, B);
+  if (par) {
+    gdn_conv_par_kernel<T, KW><<<dim3(grid.x, B, (max_q + SEG - 1) / SEG), 128, 0, s>>>(p, SEG, LONG);
+    if (KW > 1) gdn_conv_state_kernel<T, KW><<<grid, 128, 0, s>>>(p, LONG);
+  }
+  if (!par || B > 1) gdn_conv_kernel<T, KW><<<grid, 128, 0, s>>>(p, par ? LONG - 1 : 0x7fffffff);
+}
+template <typename T>
+static int gdn_conv_impl(const void* x, long long ldx, void* y, void* conv_state, const void* w, const float* bias, const int* slots,
+                         const int* q_start, const int* ctx_len, const int* no_store, int B, int C, int kw, int max_q, int round,
+                         cudaStream_t s) {
+  if (B == 0) return 0;
+  if (B > 65535 || C < 1) return (int)cudaErrorInvalidValue;
+  const ConvParams<T> p = {(const T*)x, (T*)y, (T*)conv_state, (const T*)w, bias, slots, q_start, ctx_len, no_store, ldx, C, round};
   switch (kw) {
-    case 2: BLZ_CONV(2); break;
-    case 3: BLZ_CONV(3); break;
-    case 4: BLZ_CONV(4); break;
-    case 8: BLZ_CONV(8); break;
+#define BLZ_CONV(K) case K: launch_conv<T, K>(p, B, max_q, s); break
+    BLZ_CONV(1); BLZ_CONV(2); BLZ_CONV(3); BLZ_CONV(4); BLZ_CONV(5); BLZ_CONV(6); BLZ_CONV(7); BLZ_CONV(8);
+#undef BLZ_CONV
     default: return (int)cudaErrorInvalidValue;
   }
-#undef BLZ_CONV
   return (int)cudaGetLastError();
 }
 BLZ_API int blz_gdn_conv(const void* x, long long ldx, void* y, void* conv_state, const void* w, const int* slots,
                          const int* q_start, const int* ctx_len, const int* no_store, int B, int C, int kw, cudaStream_t s) {
-  return gdn_conv_impl(x, ldx, y, conv_state, w, slots, q_start, ctx_len, no_store, B, C, kw, 0, s);
+  return gdn_conv_impl<bf16>(x, ldx, y, conv_state, w, nullptr, slots, q_start, ctx_len, no_store, B, C, kw, 0, 1, s);
 }
 BLZ_API int blz_gdn_conv_runs(const void* x, long long ldx, void* y, void* conv_state, const void* w, const int* slots,
                               const int* q_start, const int* ctx_len, const int* no_store, int B, int C, int kw, int max_q,
                               cudaStream_t s) {
-  return gdn_conv_impl(x, ldx, y, conv_state, w, slots, q_start, ctx_len, no_store, B, C, kw, max_q, s);
+  return gdn_conv_impl<bf16>(x, ldx, y, conv_state, w, nullptr, slots, q_start, ctx_len, no_store, B, C, kw, max_q, 1, s);
+}
+// The same with an optional bias ([C] fp32), the sum kept in 32 bits up to the activation, kw <= 8; f32 = 1: everything is fp32.
+BLZ_API int blz_short_conv(const void* x, long long ldx, void* y, void* conv_state, const void* w, const float* bias, const int* slots,
+                           const int* q_start, const int* ctx_len, const int* no_store, int B, int C, int kw, int max_q, int f32,
+                           cudaStream_t s) {
+  if (f32) return gdn_conv_impl<float>(x, ldx, y, conv_state, w, bias, slots, q_start, ctx_len, no_store, B, C, kw, max_q, 0, s);
+  return gdn_conv_impl<bf16>(x, ldx, y, conv_state, w, bias, slots, q_start, ctx_len, no_store, B, C, kw, max_q, 0, s);
 }
 
 static int gdn_recurrent_impl(const void* conv, const void* a_in, const void* b_in, long long ld_ab, const float* A_log,

@@ -1,6 +1,6 @@
 // Matrix products on the CUDA cores: C[M,N] = A[M,K] B[N,K]^T (+ bias) for fp32 operands (a model served in true 32-bit; the
 // tensor cores have no such mode) and for bf16 shapes that the TMA kernels do not take (a row length that is not a multiple
-// of 16).  fp32 accumulation, no reduced-precision mode.  Also the clamped gated activation as an op of its own.
+// of 16).  fp32 accumulation, no reduced-precision mode.  Also the gated activations as ops of their own.
 #include "blaze/glu.cuh"
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
@@ -53,15 +53,16 @@ __global__ void __launch_bounds__(256) gemm_simple_kernel(const T* __restrict__ 
   }
 }
 
-// gu [T, 2I] = [gate | up] -> out [T, I]
+// gu [T, 2I] = [gate | up] -> out [T, I]; limit < 0: silu(gate) * up, else the clamped activation
 template <typename T>
-__global__ void clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ out, long long total, int I, float limit) {
+__global__ void glu_kernel(const T* __restrict__ gu, T* __restrict__ out, long long total, int I, float limit) {
   pdl_trigger();
   pdl_wait();
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
     const long long t = i / I;
     const int c = (int)(i - t * I);
-    gs_st(out + i, clamped_glu(gs_ld(gu + t * 2 * I + c), gs_ld(gu + t * 2 * I + I + c), limit));
+    const float g = gs_ld(gu + t * 2 * I + c), u = gs_ld(gu + t * 2 * I + I + c);
+    gs_st(out + i, limit < 0.f ? g / (1.f + expf(-g)) * u : clamped_glu(g, u, limit));
   }
 }
 
@@ -84,12 +85,13 @@ BLZ_API int blz_gemm_simple(const void* A, long long lda, const void* B, long lo
   return (int)launch_simple<__nv_bfloat16, __nv_bfloat16>(A, lda, B, ldb, C, ldc, bias, M, N, K, s);
 }
 
+// limit < 0: silu(gate) * up
 BLZ_API int blz_clamped_glu(const void* gu, void* out, int T, int I, float limit, int f32, cudaStream_t s) {
   using namespace blz;
   if (T <= 0 || I <= 0) return (int)cudaErrorInvalidValue;
   const long long total = (long long)T * I;
   const int blocks = (int)((total + 1023) / 1024 < 4LL * sm_count() ? (total + 1023) / 1024 : 4LL * sm_count());
-  if (f32) return (int)launch_pdl(clamped_glu_kernel<float>, dim3(blocks), dim3(256), 0, s, (const float*)gu, (float*)out, total, I, limit);
-  return (int)launch_pdl(clamped_glu_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out,
+  if (f32) return (int)launch_pdl(glu_kernel<float>, dim3(blocks), dim3(256), 0, s, (const float*)gu, (float*)out, total, I, limit);
+  return (int)launch_pdl(glu_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out,
                          total, I, limit);
 }

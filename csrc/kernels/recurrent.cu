@@ -1,0 +1,499 @@
+// Recurrent mixers with an fp32 state per sequence and head, token by token, for decode rows and prompt runs alike:
+//   delta rule with a decay per key channel:  S <- g * S (rows);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//       g = exp(-A softplus(a + dt_bias)), beta = sigmoid(b), q and k made unit vectors, q times dim^-1/2
+//   state-space duality:  S <- exp(-A dt) S + dt B x^T;  y = S^T C + D x,  dt = softplus(dt_raw + dt_bias)
+// and the norm over groups of columns with a gate before or after it that follows either of them.
+// State: [rows, heads, keys (or state size), vdim] fp32; rows are sequence slots; a sequence without earlier tokens starts at zero.
+//
+// A warp holds 4 * VPT columns of a head's state in registers: 8 lanes share a column's rows (R each), so that a token costs R * VPT
+// multiply-adds per lane and product, and one reduction over 8 lanes.  The delta rule takes both of its products from the decayed
+// state at once (o = S^T q + (k . q) u), which leaves a single reduction on the path from token to token.  What a token needs
+// besides the state (unit vectors, decays, steps: all fp32) is computed once per block into shared memory, 8 tokens at a time;
+// blocks of long runs have four warps of their own for that, working one group of 8 ahead.
+#include "blaze/host.h"
+#include "blaze/sm100.cuh"
+
+namespace blz {
+
+static constexpr int kRecTok = 8;            // tokens per group
+static constexpr int kRecWarps = 4;          // warps that hold state
+
+struct RecParams {
+  const void* conv;            // [T, ld_conv] convolved inputs: delta q | k | v, state space x | B | C
+  const void* a;               // delta: decay inputs [T, ld_a], heads * dk columns; state space: dt_raw [T, ld_a], heads columns
+  const void* b;               // delta: beta inputs [T, ld_b], heads columns
+  const float* A;              // [heads], positive
+  const float* dt_bias;        // delta [heads * dk], state space [heads]
+  const float* D;              // [heads] or null
+  float* state;
+  float* out;                  // [T, heads * dv] or null (the state only)
+  const int *slots, *q_start, *ctx_len, *no_store;
+  long long ld_conv, ld_a, ld_b;
+  int heads, groups, dk, dv;   // groups: key heads (delta) or B / C groups (state space)
+};
+
+__device__ __forceinline__ float rc_ld(const float* p) { return *p; }
+__device__ __forceinline__ float rc_ld(const __nv_bfloat16* p) { return bf2f(*p); }
+template <typename T>
+__device__ __forceinline__ float rc_exp(float x) {
+  if constexpr (sizeof(T) == 4) return expf(x);
+  return __expf(x);
+}
+template <typename T>
+__device__ __forceinline__ float rc_softplus(float x) { return x > 20.f ? x : log1pf(rc_exp<T>(x)); }
+template <typename T>
+__device__ __forceinline__ float rc_sigmoid(float x) { return 1.f / (1.f + rc_exp<T>(-x)); }
+
+// lane (row group kl, column group cg) of a warp: rows kl * 4 + 32 * (i / 4) + i % 4, i < R; columns col .. col + VPT
+template <int R, int VPT>
+__device__ __forceinline__ void load_state(float (&S)[R][VPT], const float* st, int kl, int col, int dk, int dv, bool zero, bool vec) {
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int r = kl * 4 + 32 * (i / 4) + (i & 3);
+#pragma unroll
+    for (int c = 0; c < VPT; ++c) S[i][c] = 0.f;
+    if (zero || r >= dk) continue;
+    const float* p = st + (size_t)r * dv + col;
+    if (VPT == 4 && vec && col < dv) {
+      const float4 f = *reinterpret_cast<const float4*>(p);
+      S[i][0] = f.x; S[i][1 % VPT] = f.y; S[i][2 % VPT] = f.z; S[i][3 % VPT] = f.w;
+    } else {
+#pragma unroll
+      for (int c = 0; c < VPT; ++c)
+        if (col + c < dv) S[i][c] = p[c];
+    }
+  }
+}
+template <int R, int VPT>
+__device__ __forceinline__ void store_state(const float (&S)[R][VPT], float* st, int kl, int col, int dk, int dv, bool vec) {
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int r = kl * 4 + 32 * (i / 4) + (i & 3);
+    if (r >= dk) continue;
+    float* p = st + (size_t)r * dv + col;
+    if (VPT == 4 && vec && col < dv) {
+      *reinterpret_cast<float4*>(p) = make_float4(S[i][0], S[i][1 % VPT], S[i][2 % VPT], S[i][3 % VPT]);
+    } else {
+#pragma unroll
+      for (int c = 0; c < VPT; ++c)
+        if (col + c < dv) p[c] = S[i][c];
+    }
+  }
+}
+
+// grid (B * slices, heads); 128 threads, or 256 with warps 4..7 preparing the next group of tokens
+template <typename T, int R, int VPT>
+__global__ void __launch_bounds__(256, R * VPT <= 64 ? 2 : 1) delta_rule_kernel(RecParams p, int slices) {
+  constexpr int DKP = R * 8, COLS = kRecWarps * 4 * VPT, TOK = 3 * DKP + COLS + 4, NV = DKP / 32;
+  extern __shared__ float sm[];              // [2][kRecTok][q | k | g | v | beta | k . q]; a token is a multiple of 16 bytes
+  const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
+  if (n <= 0) return;
+  const bool ahead = blockDim.x > kRecWarps * 32, holds = warp < kRecWarps;
+  const int dk = p.dk, dv = p.dv, hk = h / (p.heads / p.groups);
+  const int col = slice * COLS + warp * 4 * VPT + (lane >> 3) * VPT;
+  float* st = p.state + ((size_t)p.slots[b] * p.heads + h) * dk * dv;
+  const bool vec = dv % 4 == 0;
+  float S[R][VPT];
+  if (holds) load_state<R, VPT>(S, st, kl, col, dk, dv, p.ctx_len[b] == n, vec);
+  const float A = p.A[h], qs = rsqrtf((float)dk);
+
+  auto stage = [&](int t0, float* buf) {
+    for (int j = ahead ? warp - kRecWarps : warp; j < kRecTok && t0 + j < n; j += kRecWarps) {
+      const size_t row = (size_t)(r0 + t0 + j);
+      float* s = buf + j * TOK;
+      const T* cv = reinterpret_cast<const T*>(p.conv) + row * p.ld_conv;
+      const T* av = reinterpret_cast<const T*>(p.a) + row * p.ld_a + (size_t)h * dk;
+      float q[NV], k[NV], qq = 0.f, kk = 0.f, kq = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int d = lane + i * 32;
+        q[i] = d < dk ? rc_ld(cv + (size_t)hk * dk + d) : 0.f;
+        k[i] = d < dk ? rc_ld(cv + (size_t)(p.groups + hk) * dk + d) : 0.f;
+        qq = fmaf(q[i], q[i], qq);
+        kk = fmaf(k[i], k[i], kk);
+        kq = fmaf(k[i], q[i], kq);
+      }
+      const float qn = qs / sqrtf(warp_sum(qq) + 1e-6f), kn = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
+      kq = warp_sum(kq) * qn * kn;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int d = lane + i * 32;
+        s[d] = q[i] * qn;
+        s[DKP + d] = k[i] * kn;
+        s[2 * DKP + d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d])) : 1.f;
+      }
+      for (int c = lane; c < COLS; c += 32) {
+        const int e = slice * COLS + c;
+        s[3 * DKP + c] = e < dv ? rc_ld(cv + (size_t)2 * p.groups * dk + (size_t)h * dv + e) : 0.f;
+      }
+      if (lane == 0) {
+        s[3 * DKP + COLS] = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + row * p.ld_b + h));
+        s[3 * DKP + COLS + 1] = kq;
+      }
+    }
+  };
+
+  const int lc = warp * 4 * VPT + (lane >> 3) * VPT;       // this lane's columns inside the block
+  if (!ahead || !holds) stage(0, sm);
+  __syncthreads();
+  for (int t0 = 0, c = 0; t0 < n; t0 += kRecTok, ++c) {
+    if (holds) {
+      const float* buf = sm + (c & 1) * kRecTok * TOK;
+      const int m = min(kRecTok, n - t0);
+      for (int j = 0; j < m; ++j) {
+        const float* s = buf + j * TOK;
+        float part[VPT], po[VPT], kr[R <= 16 ? R : 1];
+#pragma unroll
+        for (int v = 0; v < VPT; ++v) part[v] = po[v] = 0.f;
+#pragma unroll
+        for (int i4 = 0; i4 < R / 4; ++i4) {
+          const float4 q4 = *reinterpret_cast<const float4*>(s + kl * 4 + 32 * i4);
+          const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 32 * i4);
+          const float4 g4 = *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 32 * i4);
+          const float qa[4] = {q4.x, q4.y, q4.z, q4.w}, ka[4] = {k4.x, k4.y, k4.z, k4.w}, ga[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            if constexpr (R <= 16) kr[i4 * 4 + i] = ka[i];
+#pragma unroll
+            for (int v = 0; v < VPT; ++v) {
+              float& x = S[i4 * 4 + i][v];
+              x *= ga[i];
+              part[v] = fmaf(x, ka[i], part[v]);
+              po[v] = fmaf(x, qa[i], po[v]);
+            }
+          }
+        }
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+          for (int v = 0; v < VPT; ++v) part[v] += __shfl_xor_sync(0xffffffffu, part[v], o);
+        const float beta = s[3 * DKP + COLS], kq = s[3 * DKP + COLS + 1];
+        float u[VPT];
+#pragma unroll
+        for (int v = 0; v < VPT; ++v) u[v] = beta * (s[3 * DKP + lc + v] - part[v]);
+#pragma unroll
+        for (int i4 = 0; i4 < R / 4; ++i4) {
+          float ka[4];
+          if constexpr (R <= 16) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) ka[i] = kr[i4 * 4 + i];
+          } else {
+            const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 32 * i4);
+            ka[0] = k4.x; ka[1] = k4.y; ka[2] = k4.z; ka[3] = k4.w;
+          }
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int v = 0; v < VPT; ++v) S[i4 * 4 + i][v] = fmaf(ka[i], u[v], S[i4 * 4 + i][v]);
+        }
+        if (p.out) {
+          // sums over the 8 lanes, the columns spread over them
+          int v0 = 0;
+          float o1 = po[0], u1 = u[0];
+          if constexpr (VPT == 4) {
+            const bool up = kl & 4, up2 = kl & 2;
+            const float x0 = (up ? po[2] : po[0]) + __shfl_xor_sync(0xffffffffu, up ? po[0] : po[2], 4);
+            const float x1 = (up ? po[3] : po[1]) + __shfl_xor_sync(0xffffffffu, up ? po[1] : po[3], 4);
+            o1 = (up2 ? x1 : x0) + __shfl_xor_sync(0xffffffffu, up2 ? x0 : x1, 2);
+            v0 = (up ? 2 : 0) + (up2 ? 1 : 0);
+            u1 = up ? (up2 ? u[3] : u[2]) : (up2 ? u[1] : u[0]);
+          } else if constexpr (VPT == 2) {
+            const bool up = kl & 4;
+            o1 = (up ? po[1] : po[0]) + __shfl_xor_sync(0xffffffffu, up ? po[0] : po[1], 4);
+            o1 += __shfl_xor_sync(0xffffffffu, o1, 2);
+            v0 = up ? 1 : 0;
+            u1 = up ? u[1] : u[0];
+          } else {
+            o1 += __shfl_xor_sync(0xffffffffu, o1, 4);
+            o1 += __shfl_xor_sync(0xffffffffu, o1, 2);
+          }
+          o1 += __shfl_xor_sync(0xffffffffu, o1, 1);
+          constexpr int SAME = VPT == 4 ? 1 : (VPT == 2 ? 3 : 7);      // lanes that hold the same column
+          if ((kl & SAME) == 0 && col + v0 < dv) p.out[((size_t)(r0 + t0 + j) * p.heads + h) * dv + col + v0] = fmaf(kq, u1, o1);
+        }
+      }
+    }
+    if (!ahead) __syncthreads();
+    if ((!ahead || !holds) && t0 + kRecTok < n) stage(t0 + kRecTok, sm + ((c + 1) & 1) * kRecTok * TOK);
+    __syncthreads();
+  }
+  if (holds && !(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, dk, dv, vec);
+}
+
+template <typename T, int R, int VPT>
+__global__ void __launch_bounds__(256, R * VPT <= 64 ? 2 : 1) state_space_kernel(RecParams p, int slices) {
+  constexpr int NP = R * 8, COLS = kRecWarps * 4 * VPT, TOK = 2 * NP + COLS + 4;
+  extern __shared__ float sm[];              // [2][kRecTok][B | C | x | dt | decay]
+  const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
+  if (n <= 0) return;
+  const bool ahead = blockDim.x > kRecWarps * 32, holds = warp < kRecWarps;
+  const int N = p.dk, dv = p.dv, g = h / (p.heads / p.groups);
+  const int col = slice * COLS + warp * 4 * VPT + (lane >> 3) * VPT;
+  float* st = p.state + ((size_t)p.slots[b] * p.heads + h) * N * dv;
+  const bool vec = dv % 4 == 0;
+  float S[R][VPT];
+  if (holds) load_state<R, VPT>(S, st, kl, col, N, dv, p.ctx_len[b] == n, vec);
+  const float A = p.A[h], bias = p.dt_bias[h], D = p.D ? p.D[h] : 0.f;
+
+  auto stage = [&](int t0, float* buf) {
+    for (int j = ahead ? warp - kRecWarps : warp; j < kRecTok; j += kRecWarps) {
+      float* s = buf + j * TOK;
+      if (t0 + j >= n) {                     // beyond the run: a step that changes nothing
+        for (int d = lane; d < TOK; d += 32) s[d] = d == 2 * NP + COLS + 1 ? 1.f : 0.f;
+        continue;
+      }
+      const size_t row = (size_t)(r0 + t0 + j);
+      const T* cv = reinterpret_cast<const T*>(p.conv) + row * p.ld_conv;
+      const T* bc = cv + (size_t)p.heads * dv + (size_t)g * N;
+#pragma unroll
+      for (int i = 0; i < NP / 32; ++i) {
+        const int d = lane + i * 32;
+        s[d] = d < N ? rc_ld(bc + d) : 0.f;
+        s[NP + d] = d < N ? rc_ld(bc + (size_t)p.groups * N + d) : 0.f;
+      }
+      for (int c = lane; c < COLS; c += 32) {
+        const int e = slice * COLS + c;
+        s[2 * NP + c] = e < dv ? rc_ld(cv + (size_t)h * dv + e) : 0.f;
+      }
+      if (lane == 0) {
+        const float dt = rc_softplus<T>(rc_ld(reinterpret_cast<const T*>(p.a) + row * p.ld_a + h) + bias);
+        s[2 * NP + COLS] = dt;
+        s[2 * NP + COLS + 1] = rc_exp<T>(-A * dt);
+      }
+    }
+  };
+
+  const int lc = warp * 4 * VPT + (lane >> 3) * VPT;
+  if (!ahead || !holds) stage(0, sm);
+  __syncthreads();
+  for (int t0 = 0, c = 0; t0 < n; t0 += kRecTok, ++c) {
+    if (holds) {
+      const float* buf = sm + (c & 1) * kRecTok * TOK;
+      float y[kRecTok][VPT];
+#pragma unroll
+      for (int j = 0; j < kRecTok; ++j) {
+        const float* s = buf + j * TOK;
+        const float dt = s[2 * NP + COLS], dec = s[2 * NP + COLS + 1];
+        float x[VPT];
+#pragma unroll
+        for (int v = 0; v < VPT; ++v) { x[v] = dt * s[2 * NP + lc + v]; y[j][v] = 0.f; }
+        if (t0 + j < n) {
+#pragma unroll
+          for (int i4 = 0; i4 < R / 4; ++i4) {
+            const float4 b4 = *reinterpret_cast<const float4*>(s + kl * 4 + 32 * i4);
+            const float4 c4 = *reinterpret_cast<const float4*>(s + NP + kl * 4 + 32 * i4);
+            const float ba[4] = {b4.x, b4.y, b4.z, b4.w}, ca[4] = {c4.x, c4.y, c4.z, c4.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+              for (int v = 0; v < VPT; ++v) {
+                float& z = S[i4 * 4 + i][v];
+                z = fmaf(z, dec, ba[i] * x[v]);
+                y[j][v] = fmaf(z, ca[i], y[j][v]);
+              }
+          }
+        }
+      }
+      if (p.out) {
+        // sums over the 8 lanes of a column, the 8 tokens spread over them: lane kl ends with token kl
+#pragma unroll
+        for (int v = 0; v < VPT; ++v) {
+          float z4[4], z2[2];
+          const bool u4 = kl & 4, u2 = kl & 2, u1 = kl & 1;
+#pragma unroll
+          for (int j = 0; j < 4; ++j) z4[j] = (u4 ? y[j + 4][v] : y[j][v]) + __shfl_xor_sync(0xffffffffu, u4 ? y[j][v] : y[j + 4][v], 4);
+#pragma unroll
+          for (int j = 0; j < 2; ++j) z2[j] = (u2 ? z4[j + 2] : z4[j]) + __shfl_xor_sync(0xffffffffu, u2 ? z4[j] : z4[j + 2], 2);
+          y[0][v] = (u1 ? z2[1] : z2[0]) + __shfl_xor_sync(0xffffffffu, u1 ? z2[0] : z2[1], 1);
+        }
+        if (t0 + kl < n) {
+          const float* s = buf + kl * TOK + 2 * NP + lc;
+          float* o = p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col;
+          if (VPT == 4 && vec && col < dv) {
+            *reinterpret_cast<float4*>(o) = make_float4(fmaf(D, s[0], y[0][0]), fmaf(D, s[1 % VPT], y[0][1 % VPT]),
+                                                        fmaf(D, s[2 % VPT], y[0][2 % VPT]), fmaf(D, s[3 % VPT], y[0][3 % VPT]));
+          } else {
+#pragma unroll
+            for (int v = 0; v < VPT; ++v)
+              if (col + v < dv) o[v] = fmaf(D, s[v], y[0][v]);
+          }
+        }
+      }
+    }
+    if (!ahead) __syncthreads();
+    if ((!ahead || !holds) && t0 + kRecTok < n) stage(t0 + kRecTok, sm + ((c + 1) & 1) * kRecTok * TOK);
+    __syncthreads();
+  }
+  if (holds && !(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, N, dv, vec);
+}
+
+// ------------------------------------------------------------------------------------------ norm over groups with a gate
+struct GroupNormParams {
+  const float* o;              // [T, groups * n]
+  const void* z;               // gate inputs [T, ldz] or null
+  const float* w;              // [w_period]: the weight of a column is w[column % w_period]
+  void* out;                   // [T, ld_out]
+  long long ldz, ld_out;
+  int T, groups, n, w_period;
+  int sigmoid;                 // gate: sigmoid(z), else silu(z)
+  int gate_first;              // the gate multiplies before the norm, else after it
+  int vec;                     // rows and pointers allow 4 columns at a time
+  float eps, post;             // everything times post at the end
+};
+
+template <typename T>
+__device__ __forceinline__ float gate_of(float z, int sigmoid) {
+  const float s = rc_sigmoid<T>(z);
+  return sigmoid ? s : z * s;
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void gn_load(const GroupNormParams& p, const float* o, const T* z, int c, float (&x)[VEC], float (&g)[VEC]) {
+  if constexpr (VEC == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(o + c);
+    x[0] = f.x; x[1] = f.y; x[2] = f.z; x[3] = f.w;
+  } else {
+    x[0] = o[c];
+  }
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) g[j] = 1.f;
+  if (z) {
+    T e[VEC];
+    if constexpr (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(e) = *reinterpret_cast<const uint2*>(z + c);
+    else if constexpr (VEC == 4) *reinterpret_cast<float4*>(e) = *reinterpret_cast<const float4*>(z + c);
+    else e[0] = z[c];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) g[j] = gate_of<T>(rc_ld(e + j), p.sigmoid);
+  }
+}
+
+// a group of columns per WARPS warps
+template <typename T, int WARPS, int VEC>
+__global__ void __launch_bounds__(256) group_norm_kernel(GroupNormParams p) {
+  __shared__ float red[8];
+  pdl_trigger();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long unit = WARPS == 1 ? (long long)blockIdx.x * 8 + warp : blockIdx.x;
+  if (unit >= (long long)p.T * p.groups) return;
+  const int t = (int)(unit / p.groups), g = (int)(unit % p.groups), i0 = (WARPS == 1 ? lane : (int)threadIdx.x) * VEC;
+  constexpr int STEP = WARPS * 32 * VEC;
+  const float* o = p.o + (size_t)unit * p.n;
+  const T* z = p.z ? reinterpret_cast<const T*>(p.z) + (size_t)t * p.ldz + (size_t)g * p.n : nullptr;
+  float ss = 0.f;
+  for (int c = i0; c < p.n; c += STEP) {
+    float x[VEC], gt[VEC];
+    gn_load<T, VEC>(p, o, p.gate_first ? z : nullptr, c, x, gt);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) { x[j] *= gt[j]; ss = fmaf(x[j], x[j], ss); }
+  }
+  ss = warp_sum(ss);
+  if constexpr (WARPS > 1) {
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < WARPS; ++i) ss += red[i];
+  }
+  const float f = p.post / sqrtf(ss / (float)p.n + p.eps);
+  T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + (size_t)g * p.n;
+  for (int c = i0; c < p.n; c += STEP) {
+    float x[VEC], gt[VEC];
+    gn_load<T, VEC>(p, o, z, c, x, gt);
+    const int wc = (int)(((long long)g * p.n + c) % p.w_period);
+    T e[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      x[j] *= f * gt[j] * p.w[VEC == 1 ? wc : wc + j];
+      if constexpr (sizeof(T) == 4) e[j] = x[j];
+      else e[j] = __float2bfloat16(x[j]);
+    }
+    if constexpr (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(out + c) = *reinterpret_cast<uint2*>(e);
+    else if constexpr (VEC == 4) *reinterpret_cast<float4*>(out + c) = *reinterpret_cast<float4*>(e);
+    else out[c] = e[0];
+  }
+}
+
+template <typename T, int R, int VPT, bool DELTA>
+static int launch_rec(const RecParams& p, int B, int ahead, cudaStream_t s) {
+  constexpr int DKP = R * 8, COLS = kRecWarps * 4 * VPT;
+  const int slices = (p.dv + COLS - 1) / COLS;
+  const size_t smem = (size_t)2 * kRecTok * ((DELTA ? 3 : 2) * DKP + COLS + 4) * 4;
+  auto kern = DELTA ? delta_rule_kernel<T, R, VPT> : state_space_kernel<T, R, VPT>;
+  static PerDeviceOnce once;
+  cudaError_t e = once.smem_limit(kern, 200 * 1024);
+  if (e != cudaSuccess) return (int)e;
+  kern<<<dim3(B * slices, p.heads), ahead ? 256 : 128, smem, s>>>(p, slices);
+  return (int)cudaGetLastError();
+}
+
+// columns per lane: 4 keeps the reductions and the shared-memory reads few; runs with too few warps to fill the GPU take fewer
+template <typename T, int R, bool DELTA>
+static int pick_cols(const RecParams& p, int B, int max_q, cudaStream_t s) {
+  const int ahead = max_q > 2 * kRecTok;
+  if constexpr (R > 32) return launch_rec<T, R, 1, DELTA>(p, B, ahead, s);
+  else if constexpr (sizeof(T) == 4 || R > 16) return launch_rec<T, R, 2, DELTA>(p, B, ahead, s);
+  else {
+    const long long warps = (long long)B * p.heads * ((p.dv + 15) / 16), room = 4LL * sm_count();
+    if (!ahead || warps >= room) return launch_rec<T, R, 4, DELTA>(p, B, ahead, s);
+    if (2 * warps >= room) return launch_rec<T, R, 2, DELTA>(p, B, ahead, s);
+    return launch_rec<T, R, 1, DELTA>(p, B, ahead, s);
+  }
+}
+
+template <typename T, bool DELTA>
+static int run_rec(const RecParams& p, int B, int max_q, cudaStream_t s) {
+  if (B == 0) return 0;
+  if (B < 0 || p.heads < 1 || p.heads > 65535 || p.groups < 1 || p.heads % p.groups || p.dk < 1 || p.dk > 512 || p.dv < 1)
+    return (int)cudaErrorInvalidValue;
+  if (p.dk <= 32) return pick_cols<T, 4, DELTA>(p, B, max_q, s);
+  if (p.dk <= 64) return pick_cols<T, 8, DELTA>(p, B, max_q, s);
+  if (p.dk <= 128) return pick_cols<T, 16, DELTA>(p, B, max_q, s);
+  if (p.dk <= 256) return pick_cols<T, 32, DELTA>(p, B, max_q, s);
+  return pick_cols<T, 64, DELTA>(p, B, max_q, s);
+}
+
+}  // namespace blz
+
+// Delta rule with channel decays over every sequence of the batch (see RecParams; leading dimensions in elements; conv channels
+// [q key_heads * dk | k key_heads * dk | v heads * dv]).  out fp32 [T, heads * dv] or null.  no_store: optional [B], 1 = leave the
+// state as it was.  dk <= 512.
+BLZ_API int blz_delta_rule(const void* conv, long long ld_conv, const void* a, long long ld_a, const void* b, long long ld_b, const float* A,
+                           const float* dt_bias, float* state, float* out, const int* slots, const int* q_start, const int* ctx_len,
+                           const int* no_store, int B, int heads, int key_heads, int dk, int dv, int max_q, int f32, cudaStream_t s) {
+  using namespace blz;
+  const RecParams p = {conv, a, b, A, dt_bias, nullptr, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_a, ld_b, heads, key_heads, dk, dv};
+  return f32 ? run_rec<float, true>(p, B, max_q, s) : run_rec<__nv_bfloat16, true>(p, B, max_q, s);
+}
+
+// State-space duality (conv channels [x heads * dv | B groups * N | C groups * N]); other arguments as above.  N <= 512.
+BLZ_API int blz_state_space(const void* conv, long long ld_conv, const void* dt, long long ld_dt, const float* A, const float* dt_bias,
+                            const float* D, float* state, float* out, const int* slots, const int* q_start, const int* ctx_len,
+                            const int* no_store, int B, int heads, int groups, int N, int dv, int max_q, int f32, cudaStream_t s) {
+  using namespace blz;
+  const RecParams p = {conv, dt, nullptr, A, dt_bias, D, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_dt, 0, heads, groups, N, dv};
+  return f32 ? run_rec<float, false>(p, B, max_q, s) : run_rec<__nv_bfloat16, false>(p, B, max_q, s);
+}
+
+// RMS norm of each of `groups` runs of n columns of fp32 rows, with a gate (GroupNormParams), to the activation type.
+BLZ_API int blz_group_norm(const float* o, const void* z, long long ldz, const float* w, void* out, long long ld_out, int T, int groups,
+                           int n, int w_period, float eps, float post, int sigmoid, int gate_first, int f32, cudaStream_t s) {
+  using namespace blz;
+  if (T <= 0 || groups < 1 || n < 1 || w_period < 1) return (int)cudaErrorInvalidValue;
+  const int esz = f32 ? 4 : 2;
+  auto ok = [&](const void* q, long long ld) { return (reinterpret_cast<uintptr_t>(q) % (4 * esz)) == 0 && ld % 4 == 0; };
+  const int vec = n % 4 == 0 && w_period % 4 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0 && (!z || ok(z, ldz)) && ok(out, ld_out);
+  const GroupNormParams p = {o, z, w, out, ldz, ld_out, T, groups, n, w_period, sigmoid, gate_first, vec, eps, post};
+  const long long units = (long long)T * groups;
+  const bool wide = n > 512;
+  const dim3 grid((unsigned)(wide ? units : (units + 7) / 8));
+#define BLZ_GN(TT, V) return (int)(wide ? launch_pdl(group_norm_kernel<TT, 8, V>, grid, dim3(256), 0, s, p) \
+                                        : launch_pdl(group_norm_kernel<TT, 1, V>, grid, dim3(256), 0, s, p))
+  if (f32) { if (vec) { BLZ_GN(float, 4); } BLZ_GN(float, 1); }
+  if (vec) { BLZ_GN(__nv_bfloat16, 4); }
+  BLZ_GN(__nv_bfloat16, 1);
+#undef BLZ_GN
+}

@@ -6,6 +6,7 @@
 // the next sublayer's input from the new streams and RMS-normalises it, so that the fp32 streams make one trip through HBM
 // per sublayer.  Before the first sublayer all streams equal the scaled embedding row, which is read from the table
 // (`from_embed`) instead of being copied S times; after the last one only the sum of the streams is written.
+// Beside them: the norm of fp32 rows, and the residual sum of a post-norm decoder (residual_norm_kernel).
 // One CTA per row; the row's columns stay with their thread (float4 where the width allows), so the update is in place.
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
@@ -198,6 +199,40 @@ __global__ void __launch_bounds__(512) norm_rows_kernel(const float* __restrict_
   }
 }
 
+// The residual of a post-norm decoder: x <- norm(alpha * x + y), kept in fp32, with a copy in the activation type for the next
+// sublayer.  `from` holds the old x: fp32 rows (may be x itself), or rows of the activation type.
+template <typename T, typename X, int VEC>
+__global__ void __launch_bounds__(512) residual_norm_kernel(const X* __restrict__ from, float alpha, const T* __restrict__ y,
+                                                            const float* __restrict__ w, float eps, float* x, T* h, int W) {
+  extern __shared__ float u_row[];                   // [W]
+  __shared__ float red[16];
+  pdl_trigger();
+  pdl_wait();
+  const size_t at = (size_t)blockIdx.x * W;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float u[VEC], v[VEC];
+    ld_vec<VEC>(from + at + c, u);
+    ld_vec<VEC>(y + at + c, v);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      u[j] = fmaf(alpha, u[j], v[j]);
+      ss = fmaf(u[j], u[j], ss);
+    }
+    st_vec<VEC>(u_row + c, u);
+  }
+  const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float u[VEC], g[VEC];
+    ld_vec<VEC>(u_row + c, u);
+    ld_vec<VEC>(w + c, g);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) u[j] = u[j] * rs * g[j];
+    st_vec<VEC>(x + at + c, u);
+    if (h) st_vec<VEC>(h + at + c, u);
+  }
+}
+
 static int row_threads(int W, int vec) {
   int n = (W / vec + 1) / 2;
   n = (n + 31) / 32 * 32;
@@ -223,6 +258,16 @@ static cudaError_t pick_streams(const StreamsParams& p, int rows, cudaStream_t s
   if (p.S <= 8) { BLZ_STREAMS(8); }
   BLZ_STREAMS(16);
 #undef BLZ_STREAMS
+}
+
+template <typename T, typename X, int VEC>
+static cudaError_t launch_residual(const void* from, float alpha, const void* y, const float* w, float eps, float* x, void* h, int rows,
+                                   int W, cudaStream_t s) {
+  auto kern = residual_norm_kernel<T, X, VEC>;
+  static PerDeviceOnce once;
+  cudaError_t e = once.smem_limit(kern, 200 * 1024);
+  if (e != cudaSuccess) return e;
+  return launch_pdl(kern, dim3(rows), dim3(row_threads(W, VEC)), (size_t)W * 4, s, (const X*)from, alpha, (const T*)y, w, eps, x, (T*)h, W);
 }
 
 }  // namespace blz
@@ -253,4 +298,19 @@ BLZ_API int blz_norm_rows(const float* x, const int* rows, const float* w, void*
                            : launch_pdl(norm_rows_kernel<float, 1>, g, b, 0, s, x, rows, w, (float*)out, W, eps));
   return (int)(v4 ? launch_pdl(norm_rows_kernel<__nv_bfloat16, 4>, g, b, 0, s, x, rows, w, (__nv_bfloat16*)out, W, eps)
                   : launch_pdl(norm_rows_kernel<__nv_bfloat16, 1>, g, b, 0, s, x, rows, w, (__nv_bfloat16*)out, W, eps));
+}
+
+// x [T, W] fp32 <- norm(alpha * from + y) with the norm's weight w; h [T, W] (activation type, or null) gets a copy.  from_act: `from`
+// is of the activation type (else fp32; x itself may stand there).  f32 = 1: the activation type is fp32.  W <= 51200.
+BLZ_API int blz_residual_norm(const void* from, int from_act, float alpha, const void* y, const float* w, float eps, float* x, void* h,
+                              int T, int W, int f32, cudaStream_t s) {
+  using namespace blz;
+  if (T <= 0 || W < 1 || W > 51200 || !from || !y || !w || !x) return (int)cudaErrorInvalidValue;
+  const bool v4 = W % 4 == 0;
+#define BLZ_RN(TT, XX) return (int)(v4 ? launch_residual<TT, XX, 4>(from, alpha, y, w, eps, x, h, T, W, s) \
+                                       : launch_residual<TT, XX, 1>(from, alpha, y, w, eps, x, h, T, W, s))
+  if (f32) { BLZ_RN(float, float); }
+  if (from_act) { BLZ_RN(__nv_bfloat16, __nv_bfloat16); }
+  BLZ_RN(__nv_bfloat16, float);
+#undef BLZ_RN
 }
