@@ -92,7 +92,7 @@ def main():
     ap.add_argument("--draft-k", type=int, default=4)
     ap.add_argument("--shared-prefix", type=int, default=0)
     ap.add_argument("--out-tokens", type=int, default=0, help="output tokens per request of the --spec run (0 = 512)")
-    ap.add_argument("--design", default=None, choices=["sevevik"],
+    ap.add_argument("--design", default=None, choices=["sevevik", "niletar"],
                     help="instead of the headline run: throughput and kernels of a model design beside the closest other model at equal "
                          "size (one GPU; see blaze_b200/benchmarks/design.py)")
     ap.add_argument("--design-sizes", default="2048,4096", help="widths of the --design run")
@@ -120,7 +120,7 @@ def main():
         from blaze_b200.benchmarks import design
         clk_path = os.path.join(tempfile.gettempdir(), "blaze_clocks_design.csv")
         sampler = clocks_sampler(clk_path, 0)
-        line = design.run(args.design_sizes.split(","), args.steps, args.warmup, layers=args.layers or 8, kernels_only=args.kernels_only)
+        line = design.run(args.design, args.design_sizes.split(","), args.steps, args.warmup, layers=args.layers or 8, kernels_only=args.kernels_only)
         if sampler is not None:
             sampler.terminate()
         print(json.dumps({"metric": "design throughput", **line, "steps": args.steps, "warmup": max(args.warmup, 3), "clocks": clocks_summary(clk_path)}))

@@ -184,8 +184,11 @@ class CudaOps:
         lib.blz_soft_tc.argtypes = common + shape + [_c.c_int, _c.c_int, VP]
         lib.blz_soft_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
         lib.blz_short_conv.argtypes = [VP, LL] + [VP] * 8 + [_c.c_int] * 5 + [VP]
-        lib.blz_delta_rule.argtypes = [VP, LL, VP, LL, VP, LL] + [VP] * 8 + [_c.c_int] * 7 + [VP]
-        lib.blz_state_space.argtypes = [VP, LL, VP, LL] + [VP] * 9 + [_c.c_int] * 7 + [VP]
+        runs = [_c.c_int] * 5 + [VP] + [_c.c_int] * 3 + [VP, LL, _c.c_int, VP]
+        lib.blz_delta_rule.argtypes = [VP, LL, VP, LL, VP, LL] + [VP] * 8 + runs
+        lib.blz_state_space.argtypes = [VP, LL, VP, LL] + [VP] * 9 + runs
+        lib.blz_rec_ws_bytes.restype = LL
+        lib.blz_rec_ws_bytes.argtypes = [_c.c_int] * 5
         lib.blz_group_norm.argtypes = [VP, VP, LL, VP, VP, LL] + [_c.c_int] * 4 + [_c.c_float] * 2 + [_c.c_int] * 3 + [VP]
 
     # ------------------------------------------------------------------ plumbing
@@ -909,31 +912,50 @@ class CudaOps:
     def recurrence(self, proj, low, M, batch, kv, layer_idx, eps, out, state_only: bool = False):
         """The recurrent mixer of a layer: convolution, recurrence, gated norm into ``out`` (columns of a wider matrix).  Sequences
         flagged in ``batch.gdn_defer`` leave their state untouched; ``state_only`` advances the states and writes nothing."""
-        R, r, T, es, st = M.rec, M.rec.spec, proj.shape[0], proj.element_size(), self._stream()
+        R, r, T = M.rec, M.rec.spec, proj.shape[0]
         y = self.short_conv(proj, M, batch, kv, layer_idx)
         o = None if state_only else torch.empty(T, r.heads * r.vdim, dtype=torch.float32, device=self.device)
         self.recur(y, proj, low, M, batch, kv, layer_idx, o)
         if state_only:
             return
+        self.gated_norm(o, low if R.kind == "delta" else proj, M, eps, out)
+
+    def gated_norm(self, o, gates, M, eps, out):
+        """The norm and gate of a recurrence's rows ``o``; ``gates`` holds the gate's columns: the low-rank outputs (delta rule), or
+        the input projection (state space)."""
+        R, r, es = M.rec, M.rec.spec, gates.element_size()
         delta = R.kind == "delta"
-        z, ldz = (low.data_ptr() + r.heads * r.dim * es, low.stride(0)) if delta else (proj.data_ptr() + M.cols["z"] * es, proj.stride(0))
-        self._check(self.lib.blz_group_norm(_ptr(o), VP(z), ldz, _ptr(R.norm_w), _ptr(out), out.stride(0), T, R.norm_groups,
+        z = VP(gates.data_ptr() + (r.heads * r.dim if delta else M.cols["z"]) * es)
+        self._check(self.lib.blz_group_norm(_ptr(o), z, gates.stride(0), _ptr(R.norm_w), _ptr(out), out.stride(0), o.shape[0], R.norm_groups,
                                             o.shape[1] // R.norm_groups, R.norm_w.numel(), eps, r.out_scale, int(delta), int(not delta),
-                                            int(es == 4), st), "group_norm")
+                                            int(es == 4), self._stream()), "group_norm")
+
+    REC_MAX_WS = 4 << 30       # workspace of the streaming recurrences; steps that need more run without it
 
     def recur(self, y, proj, low, M, batch, kv, layer_idx, o):
         """The recurrence alone: convolved inputs ``y`` to fp32 rows ``o`` (None: the state only)."""
         R, r, es, f32 = M.rec, M.rec.spec, proj.element_size(), int(proj.dtype == torch.float32)
         seqs = (_ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(batch.gdn_defer), batch.slots.numel())
-        state, st, longest = kv.rec_state[layer_idx], self._stream(), int(batch.max_q_len)
-        if R.kind == "delta":
+        state, st, longest, T, delta = kv.rec_state[layer_idx], self._stream(), int(batch.max_q_len), y.shape[0], R.kind == "delta"
+        groups = r.kv_heads if delta else r.groups
+        ws, ws_bytes, short = None, 0, True
+        long_rows = int(self.lib.blz_rec_long_rows())
+        if o is not None and longest >= long_rows:
+            # long runs take the streaming kernels, which read what a token needs from a workspace filled for all tokens at once
+            ws_bytes = int(self.lib.blz_rec_ws_bytes(int(delta), T, r.heads, groups, r.state))
+            if ws_bytes <= self.REC_MAX_WS:
+                ws = torch.empty(ws_bytes, dtype=torch.uint8, device=self.device)
+                short = any(0 < e - s < long_rows for s, e in zip(batch.h_q_start, batch.h_q_start[1:]))
+                self.launches += 2 if short else 1
+        runs = (_ptr(batch.seq_of_row), T, longest, int(short), _ptr(ws), ws_bytes, f32, st)
+        if delta:
             self._check(self.lib.blz_delta_rule(_ptr(y), y.stride(0), _ptr(low), low.stride(0), VP(proj.data_ptr() + M.cols["beta"] * es),
                                                 proj.stride(0), _ptr(R.A), _ptr(R.dt_bias), _ptr(state), _ptr(o), *seqs, r.heads,
-                                                r.kv_heads, r.dim, r.vdim, longest, f32, st), "delta_rule")
+                                                r.kv_heads, r.dim, r.vdim, *runs), "delta_rule")
         else:
             self._check(self.lib.blz_state_space(_ptr(y), y.stride(0), VP(proj.data_ptr() + M.cols["dt"] * es), proj.stride(0), _ptr(R.A),
                                                  _ptr(R.dt_bias), _ptr(R.D), _ptr(state), _ptr(o), *seqs, r.heads, r.groups, r.state,
-                                                 r.vdim, longest, f32, st), "state_space")
+                                                 r.vdim, *runs), "state_space")
 
     # ------------------------------------------------------------------ head
     def argmax(self, logits, index_offset: int = 0, want_values: bool = False):
@@ -1095,18 +1117,27 @@ class CudaOps:
     def gdn(self, mixed_qkv, z, b, a, gdn, model, batch, kv, layer_idx, state_only: bool = False):
         """Causal conv + SiLU → gated delta rule (gates computed in the kernel) → gated RMSNorm.  Sequences flagged in
         ``batch.gdn_defer`` leave their state untouched; ``state_only`` advances the states and returns nothing."""
-        cfg = model.cfg
-        dk, dv = cfg.linear_key_head_dim, cfg.linear_value_head_dim
-        hk, hv = gdn.k_heads, gdn.v_heads
-        T = mixed_qkv.shape[0]
-        C = 2 * hk * dk + hv * dv
-        B = batch.slots.numel()
+        conv = self.gdn_conv(mixed_qkv, gdn, batch, kv, layer_idx)
+        o = None if state_only else torch.empty(mixed_qkv.shape[0], gdn.v_heads, model.cfg.linear_value_head_dim, dtype=torch.bfloat16,
+                                                device=self.device)
+        self.gdn_rule(conv, b, a, gdn, model, batch, kv, layer_idx, o)
+        return None if state_only else self.gdn_norm(o, z, gdn, model.cfg)
+
+    def gdn_conv(self, mixed_qkv, gdn, batch, kv, layer_idx):
+        T, C = mixed_qkv.shape[0], gdn.conv_w.shape[0]
         conv = torch.empty(T, C, dtype=torch.bfloat16, device=self.device)
         self._check(self.lib.blz_gdn_conv_runs(_ptr(mixed_qkv), mixed_qkv.stride(0), _ptr(conv), _ptr(kv.conv_state[layer_idx]),
                                                _ptr(gdn.conv_w), _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len),
-                                               _ptr(batch.gdn_defer), B, C, gdn.conv_w.shape[1], int(batch.max_q_len),
+                                               _ptr(batch.gdn_defer), batch.slots.numel(), C, gdn.conv_w.shape[1], int(batch.max_q_len),
                                                self._stream()), "gdn_conv")
-        o = None if state_only else torch.empty(T, hv, dv, dtype=torch.bfloat16, device=self.device)
+        return conv
+
+    def gdn_rule(self, conv, b, a, gdn, model, batch, kv, layer_idx, o):
+        """The gated delta rule on convolved inputs; ``o`` None: the states only."""
+        cfg = model.cfg
+        dk, dv = cfg.linear_key_head_dim, cfg.linear_value_head_dim
+        hk, hv = gdn.k_heads, gdn.v_heads
+        T, B, state_only = conv.shape[0], batch.slots.numel(), o is None
         # long token runs (prompt chunks) go through the chunked tensor-core kernel, short ones (decode, verify, replay)
         # through the token-by-token kernel; both walk the same batch and each takes its own sequences
         chunked = (self.GDN_CHUNK_MIN > 0 and not state_only and dk == 128 and dv == 128 and batch.max_q_len >= self.GDN_CHUNK_MIN)
@@ -1130,8 +1161,9 @@ class CudaOps:
                                                         _ptr(batch.ctx_len), _ptr(batch.gdn_defer), B, hk, hv, dk, dv,
                                                         self.GDN_CHUNK_MIN - 1 if chunked else 0x7fffffff, self._stream()),
                         "gdn_recurrent")
-        if state_only:
-            return None
+
+    def gdn_norm(self, o, z, gdn, cfg):
+        T, hv, dv = o.shape
         y = torch.empty(T, hv * dv, dtype=torch.bfloat16, device=self.device)
         self._check(self.lib.blz_gated_rmsnorm(_ptr(o), _ptr(z), z.stride(0), _ptr(gdn.norm_w), _ptr(y), T, hv, dv,
                                                cfg.rms_norm_eps, 2 if cfg.gdn_output_gate == "sigmoid" else 0, self._stream()),

@@ -608,6 +608,7 @@ struct PrepParams {
   const float* freq;           // [2][rot_dims / 2]: frequencies, and what their rounding to 32 bits left over
   long long ld, q_off, k_off, v_off, page_stride, head_stride;
   int T, heads, kv_heads, dim, vdim, rot_dims, interleaved, unit_rms;
+  int pairs;                   // bf16: neighbouring dimensions can be read and written as 32-bit words
   float eps;
 };
 
@@ -635,7 +636,15 @@ __global__ void __launch_bounds__(128) attn_prep_pages_kernel(PrepParams p) {
     if (u < u1 && u < p.heads + p.kv_heads && p.unit_rms) {
       const T* src = row + (u < p.heads ? p.q_off + (size_t)u * p.dim : p.k_off + (size_t)(u - p.heads) * p.dim);
       float ss = 0.f;
-      for (int j = lane; j < p.dim; j += 32) { const float v = ad_ld(src + j); ss = fmaf(v, v, ss); }
+      if (sizeof(T) == 2 && p.pairs) {
+        for (int j = lane; j < p.dim / 2; j += 32) {
+          const uint32_t w = *reinterpret_cast<const uint32_t*>(src + 2 * j);
+          const float x = __uint_as_float(w << 16), y = __uint_as_float(w & 0xffff0000u);
+          ss = fmaf(x, x, fmaf(y, y, ss));
+        }
+      } else {
+        for (int j = lane; j < p.dim; j += 32) { const float v = ad_ld(src + j); ss = fmaf(v, v, ss); }
+      }
       f[k] = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);         // a rotation leaves the sum of squares as it is
     }
   }
@@ -658,6 +667,17 @@ __global__ void __launch_bounds__(128) attn_prep_pages_kernel(PrepParams p) {
         if (u >= u1 || u >= p.heads + p.kv_heads) continue;
         const bool is_q = u < p.heads;
         const T* src = row + (is_q ? p.q_off + (size_t)u * p.dim : p.k_off + (size_t)(u - p.heads) * p.dim);
+        if (sizeof(T) == 2 && p.pairs && b == a + 1) {             // a pair is one 32-bit word everywhere
+          const uint32_t w = a < p.dim ? *reinterpret_cast<const uint32_t*>(src + a) : 0u;
+          const float x = __uint_as_float(w << 16), y = __uint_as_float(w & 0xffff0000u);
+          const uint32_t r = pack_bf16x2((x * c - y * s) * f[k], (y * c + x * s) * f[k]);
+          if (!is_q) {
+            if (page) *reinterpret_cast<uint32_t*>(page + (size_t)(u - p.heads) * p.head_stride + core_off(slot & 15, a, dp)) = r;
+          } else if (a < p.dim) {
+            *reinterpret_cast<uint32_t*>(reinterpret_cast<T*>(p.q_out) + ((size_t)t * p.heads + u) * p.dim + a) = r;
+          }
+          continue;
+        }
         const float x = a < p.dim ? ad_ld(src + a) : 0.f, y = b < p.dim ? ad_ld(src + b) : 0.f;
         const float xr = (x * c - y * s) * f[k], yr = (y * c + x * s) * f[k];
         if (is_q) {
@@ -679,7 +699,12 @@ __global__ void __launch_bounds__(128) attn_prep_pages_kernel(PrepParams p) {
       if (u0 + k >= u1 || g < 0) continue;
       const T* src = row + p.v_off + (size_t)g * p.vdim;
       T* dst = page + (size_t)g * p.head_stride + 16 * dp;
-      for (int j = lane; j < vp; j += 32) ad_st(dst + core_off(slot & 15, j, vp), j < p.vdim ? ad_ld(src + j) : 0.f);
+      if (sizeof(T) == 2 && p.pairs) {
+        for (int j = 2 * lane; j < vp; j += 64)
+          *reinterpret_cast<uint32_t*>(dst + core_off(slot & 15, j, vp)) = j < p.vdim ? *reinterpret_cast<const uint32_t*>(src + j) : 0u;
+      } else {
+        for (int j = lane; j < vp; j += 32) ad_st(dst + core_off(slot & 15, j, vp), j < p.vdim ? ad_ld(src + j) : 0.f);
+      }
     }
   }
 }
@@ -710,6 +735,7 @@ BLZ_API int blz_attn_prep_pages(const void* qkv, long long ld, long long q_off, 
   p.page_stride = page_stride; p.head_stride = head_stride; p.positions = positions; p.slot_mapping = slot_mapping; p.freq = freq;
   p.T = T; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.rot_dims = rot_dims; p.interleaved = interleaved;
   p.unit_rms = unit_rms; p.eps = eps;
+  p.pairs = !f32 && (reinterpret_cast<uintptr_t>(qkv) & 3) == 0 && ld % 2 == 0 && (q_off | k_off | v_off) % 2 == 0 && dim % 2 == 0 && vdim % 2 == 0;
   const long long warps = (long long)T * ((heads + 2 * kv_heads + kPrepHeads - 1) / kPrepHeads);
   const dim3 grid((unsigned)((warps + 3) / 4));
   if (f32) return (int)launch_pdl(attn_prep_pages_kernel<float>, grid, dim3(128), 0, s, p);

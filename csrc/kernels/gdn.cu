@@ -37,6 +37,27 @@ __device__ __forceinline__ float conv_act(float acc, int round) {
   return r / (1.f + __expf(-r));
 }
 
+template <typename T, int CV>
+__device__ __forceinline__ void cv_ldv(const T* p, float (&v)[CV]) {
+  if constexpr (CV == 4 && sizeof(T) == 2) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
+    v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
+  } else {
+#pragma unroll
+    for (int i = 0; i < CV; ++i) v[i] = cv_ld(p + i);
+  }
+}
+template <typename T, int CV>
+__device__ __forceinline__ void cv_stv(T* p, const float (&v)[CV]) {
+  if constexpr (CV == 4 && sizeof(T) == 2) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  } else {
+#pragma unroll
+    for (int i = 0; i < CV; ++i) cv_st(p + i, v[i]);
+  }
+}
+
 // grid (ceil(C / 128), B); thread = channel; walks the sequence's tokens in order
 template <typename T, int KW>
 __global__ void gdn_conv_kernel(ConvParams<T> p, int max_rows) {
@@ -68,12 +89,13 @@ __global__ void gdn_conv_kernel(ConvParams<T> p, int max_rows) {
   for (int j = 0; j < KW - 1; ++j) cv_st(st + j, h[j]);
 }
 
-// Long token runs (prompts): the same convolution with the tokens spread over the grid.  grid (ceil(C / 128), B, segments):
+// Long token runs (prompts): the same convolution with the tokens spread over the grid, CV channels per thread.
+// grid (ceil(C / (128 CV)), B, segments):
 // segment z handles tokens [z * SEG, (z + 1) * SEG) of the sequence; the k-1 inputs before its first token come from the input
 // itself (or from the state for the run's first tokens).  The new state is a kernel of its own (the first segment reads the old).
-template <typename T, int KW>
+template <typename T, int KW, int CV>
 __global__ void gdn_conv_par_kernel(ConvParams<T> p, int seg, int min_rows) {
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * CV;
   const int b = blockIdx.y;
   if (c >= p.C) return;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
@@ -82,25 +104,49 @@ __global__ void gdn_conv_par_kernel(ConvParams<T> p, int seg, int min_rows) {
   if (t0 >= n) return;
   const bool fresh = p.ctx_len[b] - n == 0;
   const T* st = p.conv_state + ((size_t)p.slots[b] * p.C + c) * (KW - 1);
-  const float b0 = p.bias ? p.bias[c] : 0.f;
-  float h[KW];
-  float wt[KW];
+  float h[KW][CV], wt[KW][CV], b0[CV];
+#pragma unroll
+  for (int i = 0; i < CV; ++i) {
+    b0[i] = p.bias ? p.bias[c + i] : 0.f;
+#pragma unroll
+    for (int j = 0; j < KW; ++j) wt[j][i] = cv_ld(p.w + (size_t)(c + i) * KW + j);
+  }
+  const T* x = p.x + (size_t)(r0 + t0) * p.ldx + c;
 #pragma unroll
   for (int j = 0; j < KW - 1; ++j) {
-    const int t = t0 - (KW - 1) + j;              // input position of history slot j (negative: before this run)
-    h[j] = t >= 0 ? cv_ld(p.x + (size_t)(r0 + t) * p.ldx + c) : (fresh ? 0.f : cv_ld(st + (KW - 1) + t));
+    const int back = KW - 1 - j, t = t0 - back;   // input position of history slot j (negative: before this run)
+    if (t >= 0) {
+      cv_ldv<T, CV>(x - (size_t)back * p.ldx, h[j]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < CV; ++i) h[j][i] = fresh ? 0.f : cv_ld(st + (size_t)i * (KW - 1) + (KW - 1) + t);
+    }
   }
+  T* y = p.y + (size_t)(r0 + t0) * p.C + c;
+  constexpr int AHEAD = 8;                         // tokens in flight
+  for (int t = t0; t < t1; t += AHEAD) {
+    float in[AHEAD][CV];
 #pragma unroll
-  for (int j = 0; j < KW; ++j) wt[j] = cv_ld(p.w + (size_t)c * KW + j);
-#pragma unroll 4
-  for (int t = t0; t < t1; ++t) {
-    h[KW - 1] = cv_ld(p.x + (size_t)(r0 + t) * p.ldx + c);
-    float acc = b0;
+    for (int k = 0; k < AHEAD; ++k)
+      if (t + k < t1) cv_ldv<T, CV>(x + (size_t)k * p.ldx, in[k]);
 #pragma unroll
-    for (int j = 0; j < KW; ++j) acc += h[j] * wt[j];
-    cv_st(p.y + (size_t)(r0 + t) * p.C + c, conv_act<T>(acc, p.round));
+    for (int k = 0; k < AHEAD; ++k) {
+      if (t + k >= t1) break;
+      float o[CV];
 #pragma unroll
-    for (int j = 0; j < KW - 1; ++j) h[j] = h[j + 1];
+      for (int i = 0; i < CV; ++i) {
+        h[KW - 1][i] = in[k][i];
+        float acc = b0[i];
+#pragma unroll
+        for (int j = 0; j < KW; ++j) acc += h[j][i] * wt[j][i];
+        o[i] = conv_act<T>(acc, p.round);
+#pragma unroll
+        for (int j = 0; j < KW - 1; ++j) h[j][i] = h[j + 1][i];
+      }
+      cv_stv<T, CV>(y + (size_t)k * p.C, o);
+    }
+    x += (size_t)AHEAD * p.ldx;
+    y += (size_t)AHEAD * p.C;
   }
 }
 // the state after a long run: its last k-1 inputs (such a run has at least that many)
@@ -218,7 +264,11 @@ static void launch_conv(const ConvParams<T>& p, int B, int max_q, cudaStream_t s
   const bool par = max_q >= LONG;
   const dim3 grid((p.C + 127) / 128, B);
   if (par) {
-    gdn_conv_par_kernel<T, KW><<<dim3(grid.x, B, (max_q + SEG - 1) / SEG), 128, 0, s>>>(p, SEG, LONG);
+    const int segs = (max_q + SEG - 1) / SEG;
+    if (sizeof(T) == 2 && p.C % 4 == 0 && p.ldx % 4 == 0 && ((reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.y)) & 7) == 0)
+      gdn_conv_par_kernel<T, KW, 4><<<dim3((p.C + 511) / 512, B, segs), 128, 0, s>>>(p, SEG, LONG);
+    else
+      gdn_conv_par_kernel<T, KW, 1><<<dim3(grid.x, B, segs), 128, 0, s>>>(p, SEG, LONG);
     if (KW > 1) gdn_conv_state_kernel<T, KW><<<grid, 128, 0, s>>>(p, LONG);
   }
   if (!par || B > 1) gdn_conv_kernel<T, KW><<<grid, 128, 0, s>>>(p, par ? LONG - 1 : 0x7fffffff);

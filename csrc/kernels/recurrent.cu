@@ -8,8 +8,10 @@
 // A warp holds 4 * VPT columns of a head's state in registers: 8 lanes share a column's rows (R each), so that a token costs R * VPT
 // multiply-adds per lane and product, and one reduction over 8 lanes.  The delta rule takes both of its products from the decayed
 // state at once (o = S^T q + (k . q) u), which leaves a single reduction on the path from token to token.  What a token needs
-// besides the state (unit vectors, decays, steps: all fp32) is computed once per block into shared memory, 8 tokens at a time;
-// blocks of long runs have four warps of their own for that, working one group of 8 ahead.
+// besides the state (unit vectors, decays, steps: all fp32) does not depend on the state:
+//   runs of a few tokens (decode, verify rows) prepare it in shared memory, 8 tokens at a time;
+//   long runs have it prepared for all tokens at once by a kernel of its own, as one record per token and head (or group) in a
+//   workspace, and the kernel that holds the state streams the records of 8 tokens at a time through a ring of bulk copies.
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
 
@@ -30,6 +32,10 @@ struct RecParams {
   const int *slots, *q_start, *ctx_len, *no_store;
   long long ld_conv, ld_a, ld_b;
   int heads, groups, dk, dv;   // groups: key heads (delta) or B / C groups (state space)
+  const int* seq_of_row;       // [T], -1 = padding
+  float* records;              // workspace of the long runs
+  int T, long_rows;            // sequences with at least long_rows new tokens are long runs
+  int* status;
 };
 
 __device__ __forceinline__ float rc_ld(const float* p) { return *p; }
@@ -81,26 +87,50 @@ __device__ __forceinline__ void store_state(const float (&S)[R][VPT], float* st,
   }
 }
 
-// grid (B * slices, heads); 128 threads, or 256 with warps 4..7 preparing the next group of tokens
+// sums of y[token][column] over the 8 lanes of a column, the 8 tokens spread over them: lane kl ends with token kl in y[0]
+template <int VPT>
+__device__ __forceinline__ void spread_tokens(float (&y)[kRecTok][VPT], int kl) {
+  const bool u4 = kl & 4, u2 = kl & 2, u1 = kl & 1;
+#pragma unroll
+  for (int v = 0; v < VPT; ++v) {
+    float z4[4], z2[2];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) z4[j] = (u4 ? y[j + 4][v] : y[j][v]) + __shfl_xor_sync(0xffffffffu, u4 ? y[j][v] : y[j + 4][v], 4);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) z2[j] = (u2 ? z4[j + 2] : z4[j]) + __shfl_xor_sync(0xffffffffu, u2 ? z4[j] : z4[j + 2], 2);
+    y[0][v] = (u1 ? z2[1] : z2[0]) + __shfl_xor_sync(0xffffffffu, u1 ? z2[0] : z2[1], 1);
+  }
+}
+template <int VPT>
+__device__ __forceinline__ void store_cols(float* o, const float (&y)[VPT], int col, int dv, bool vec) {
+  if (VPT == 4 && vec) {
+    if (col < dv) *reinterpret_cast<float4*>(o) = make_float4(y[0], y[1 % VPT], y[2 % VPT], y[3 % VPT]);
+  } else {
+#pragma unroll
+    for (int v = 0; v < VPT; ++v)
+      if (col + v < dv) o[v] = y[v];
+  }
+}
+
+// grid (B * slices, heads), 128 threads
 template <typename T, int R, int VPT>
-__global__ void __launch_bounds__(256, R * VPT <= 64 ? 2 : 1) delta_rule_kernel(RecParams p, int slices) {
+__global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_rule_kernel(RecParams p, int slices) {
   constexpr int DKP = R * 8, COLS = kRecWarps * 4 * VPT, TOK = 3 * DKP + COLS + 4, NV = DKP / 32;
   extern __shared__ float sm[];              // [2][kRecTok][q | k | g | v | beta | k . q]; a token is a multiple of 16 bytes
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7;
-  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
-  if (n <= 0) return;
-  const bool ahead = blockDim.x > kRecWarps * 32, holds = warp < kRecWarps;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
+  if (n <= 0 || n >= p.long_rows) return;
   const int dk = p.dk, dv = p.dv, hk = h / (p.heads / p.groups);
   const int col = slice * COLS + warp * 4 * VPT + (lane >> 3) * VPT;
-  float* st = p.state + ((size_t)p.slots[b] * p.heads + h) * dk * dv;
+  float* st = p.state + ((size_t)slot * p.heads + h) * dk * dv;
   const bool vec = dv % 4 == 0;
   float S[R][VPT];
-  if (holds) load_state<R, VPT>(S, st, kl, col, dk, dv, p.ctx_len[b] == n, vec);
+  load_state<R, VPT>(S, st, kl, col, dk, dv, ctx == n, vec);
   const float A = p.A[h], qs = rsqrtf((float)dk);
 
   auto stage = [&](int t0, float* buf) {
-    for (int j = ahead ? warp - kRecWarps : warp; j < kRecTok && t0 + j < n; j += kRecWarps) {
+    for (int j = warp; j < kRecTok && t0 + j < n; j += kRecWarps) {
       const size_t row = (size_t)(r0 + t0 + j);
       float* s = buf + j * TOK;
       const T* cv = reinterpret_cast<const T*>(p.conv) + row * p.ld_conv;
@@ -136,10 +166,10 @@ __global__ void __launch_bounds__(256, R * VPT <= 64 ? 2 : 1) delta_rule_kernel(
   };
 
   const int lc = warp * 4 * VPT + (lane >> 3) * VPT;       // this lane's columns inside the block
-  if (!ahead || !holds) stage(0, sm);
+  stage(0, sm);
   __syncthreads();
   for (int t0 = 0, c = 0; t0 < n; t0 += kRecTok, ++c) {
-    if (holds) {
+    {
       const float* buf = sm + (c & 1) * kRecTok * TOK;
       const int m = min(kRecTok, n - t0);
       for (int j = 0; j < m; ++j) {
@@ -215,32 +245,30 @@ __global__ void __launch_bounds__(256, R * VPT <= 64 ? 2 : 1) delta_rule_kernel(
         }
       }
     }
-    if (!ahead) __syncthreads();
-    if ((!ahead || !holds) && t0 + kRecTok < n) stage(t0 + kRecTok, sm + ((c + 1) & 1) * kRecTok * TOK);
+    if (t0 + kRecTok < n) stage(t0 + kRecTok, sm + ((c + 1) & 1) * kRecTok * TOK);
     __syncthreads();
   }
-  if (holds && !(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, dk, dv, vec);
+  if (!(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, dk, dv, vec);
 }
 
 template <typename T, int R, int VPT>
-__global__ void __launch_bounds__(256, R * VPT <= 64 ? 2 : 1) state_space_kernel(RecParams p, int slices) {
+__global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) state_space_kernel(RecParams p, int slices) {
   constexpr int NP = R * 8, COLS = kRecWarps * 4 * VPT, TOK = 2 * NP + COLS + 4;
   extern __shared__ float sm[];              // [2][kRecTok][B | C | x | dt | decay]
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7;
-  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
-  if (n <= 0) return;
-  const bool ahead = blockDim.x > kRecWarps * 32, holds = warp < kRecWarps;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
+  if (n <= 0 || n >= p.long_rows) return;
   const int N = p.dk, dv = p.dv, g = h / (p.heads / p.groups);
   const int col = slice * COLS + warp * 4 * VPT + (lane >> 3) * VPT;
-  float* st = p.state + ((size_t)p.slots[b] * p.heads + h) * N * dv;
+  float* st = p.state + ((size_t)slot * p.heads + h) * N * dv;
   const bool vec = dv % 4 == 0;
   float S[R][VPT];
-  if (holds) load_state<R, VPT>(S, st, kl, col, N, dv, p.ctx_len[b] == n, vec);
+  load_state<R, VPT>(S, st, kl, col, N, dv, ctx == n, vec);
   const float A = p.A[h], bias = p.dt_bias[h], D = p.D ? p.D[h] : 0.f;
 
   auto stage = [&](int t0, float* buf) {
-    for (int j = ahead ? warp - kRecWarps : warp; j < kRecTok; j += kRecWarps) {
+    for (int j = warp; j < kRecTok; j += kRecWarps) {
       float* s = buf + j * TOK;
       if (t0 + j >= n) {                     // beyond the run: a step that changes nothing
         for (int d = lane; d < TOK; d += 32) s[d] = d == 2 * NP + COLS + 1 ? 1.f : 0.f;
@@ -268,10 +296,10 @@ __global__ void __launch_bounds__(256, R * VPT <= 64 ? 2 : 1) state_space_kernel
   };
 
   const int lc = warp * 4 * VPT + (lane >> 3) * VPT;
-  if (!ahead || !holds) stage(0, sm);
+  stage(0, sm);
   __syncthreads();
   for (int t0 = 0, c = 0; t0 < n; t0 += kRecTok, ++c) {
-    if (holds) {
+    {
       const float* buf = sm + (c & 1) * kRecTok * TOK;
       float y[kRecTok][VPT];
 #pragma unroll
@@ -299,36 +327,375 @@ __global__ void __launch_bounds__(256, R * VPT <= 64 ? 2 : 1) state_space_kernel
         }
       }
       if (p.out) {
-        // sums over the 8 lanes of a column, the 8 tokens spread over them: lane kl ends with token kl
-#pragma unroll
-        for (int v = 0; v < VPT; ++v) {
-          float z4[4], z2[2];
-          const bool u4 = kl & 4, u2 = kl & 2, u1 = kl & 1;
-#pragma unroll
-          for (int j = 0; j < 4; ++j) z4[j] = (u4 ? y[j + 4][v] : y[j][v]) + __shfl_xor_sync(0xffffffffu, u4 ? y[j][v] : y[j + 4][v], 4);
-#pragma unroll
-          for (int j = 0; j < 2; ++j) z2[j] = (u2 ? z4[j + 2] : z4[j]) + __shfl_xor_sync(0xffffffffu, u2 ? z4[j] : z4[j + 2], 2);
-          y[0][v] = (u1 ? z2[1] : z2[0]) + __shfl_xor_sync(0xffffffffu, u1 ? z2[0] : z2[1], 1);
-        }
+        spread_tokens<VPT>(y, kl);
         if (t0 + kl < n) {
           const float* s = buf + kl * TOK + 2 * NP + lc;
-          float* o = p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col;
-          if (VPT == 4 && vec && col < dv) {
-            *reinterpret_cast<float4*>(o) = make_float4(fmaf(D, s[0], y[0][0]), fmaf(D, s[1 % VPT], y[0][1 % VPT]),
-                                                        fmaf(D, s[2 % VPT], y[0][2 % VPT]), fmaf(D, s[3 % VPT], y[0][3 % VPT]));
-          } else {
 #pragma unroll
-            for (int v = 0; v < VPT; ++v)
-              if (col + v < dv) o[v] = fmaf(D, s[v], y[0][v]);
-          }
+          for (int v = 0; v < VPT; ++v) y[0][v] = fmaf(D, s[v], y[0][v]);
+          store_cols<VPT>(p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col, y[0], col, dv, vec);
         }
       }
     }
-    if (!ahead) __syncthreads();
-    if ((!ahead || !holds) && t0 + kRecTok < n) stage(t0 + kRecTok, sm + ((c + 1) & 1) * kRecTok * TOK);
+    if (t0 + kRecTok < n) stage(t0 + kRecTok, sm + ((c + 1) & 1) * kRecTok * TOK);
     __syncthreads();
   }
-  if (holds && !(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, N, dv, vec);
+  if (!(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, N, dv, vec);
+}
+
+// ------------------------------------------------------------------------------------------ long runs
+// Records: delta [heads][T][q | k | g | beta, k . q, 0, 0], state space [groups][T][B | C] and [heads][T][dt, decay, 0, 0];
+// vectors padded to R * 8 floats.
+__device__ __forceinline__ bool in_long_run(const RecParams& p, int t) {
+  const int b = p.seq_of_row[t];
+  return b >= 0 && p.q_start[b + 1] - p.q_start[b] >= p.long_rows;
+}
+
+// a warp per (row, head)
+template <typename T, int R>
+__global__ void __launch_bounds__(128) delta_records_kernel(RecParams p) {
+  constexpr int DKP = R * 8, REC = 3 * DKP + 4, NV = DKP / 32;
+  const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int t = (int)(w / p.heads), h = (int)(w % p.heads), lane = threadIdx.x & 31;
+  if (t >= p.T || !in_long_run(p, t)) return;
+  const int dk = p.dk, hk = h / (p.heads / p.groups);
+  const T* cv = reinterpret_cast<const T*>(p.conv) + (size_t)t * p.ld_conv;
+  const T* av = reinterpret_cast<const T*>(p.a) + (size_t)t * p.ld_a + (size_t)h * dk;
+  float q[NV], k[NV], a[NV], qq = 0.f, kk = 0.f, kq = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = lane + i * 32;
+    q[i] = d < dk ? rc_ld(cv + (size_t)hk * dk + d) : 0.f;
+    k[i] = d < dk ? rc_ld(cv + (size_t)(p.groups + hk) * dk + d) : 0.f;
+    a[i] = d < dk ? rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d] : 0.f;
+  }
+  const float beta = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + (size_t)t * p.ld_b + h)), A = p.A[h];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    qq = fmaf(q[i], q[i], qq);
+    kk = fmaf(k[i], k[i], kk);
+    kq = fmaf(k[i], q[i], kq);
+  }
+  const float qn = rsqrtf((float)dk) / sqrtf(warp_sum(qq) + 1e-6f), kn = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
+  kq = warp_sum(kq) * qn * kn;
+  float* s = p.records + ((size_t)h * p.T + t) * REC;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = lane + i * 32;
+    s[d] = q[i] * qn;
+    s[DKP + d] = k[i] * kn;
+    s[2 * DKP + d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(a[i])) : 1.f;
+  }
+  if (lane == 0) *reinterpret_cast<float4*>(s + 3 * DKP) = make_float4(beta, kq, 0.f, 0.f);
+}
+
+// a block per row
+template <typename T, int R>
+__global__ void __launch_bounds__(128) state_space_records_kernel(RecParams p) {
+  constexpr int NP = R * 8;
+  const int t = blockIdx.x, N = p.dk;
+  if (!in_long_run(p, t)) return;
+  const T* bc = reinterpret_cast<const T*>(p.conv) + (size_t)t * p.ld_conv + (size_t)p.heads * p.dv;
+  for (int i = threadIdx.x; i < p.groups * 2 * NP; i += 128) {
+    const int g = i / (2 * NP), which = i / NP & 1, d = i % NP;
+    p.records[((size_t)g * p.T + t) * 2 * NP + which * NP + d] = d < N ? rc_ld(bc + (size_t)(which * p.groups + g) * N + d) : 0.f;
+  }
+  float4* steps = reinterpret_cast<float4*>(p.records + (size_t)p.groups * p.T * 2 * NP);
+  for (int h = threadIdx.x; h < p.heads; h += 128) {
+    const float dt = rc_softplus<T>(rc_ld(reinterpret_cast<const T*>(p.a) + (size_t)t * p.ld_a + h) + p.dt_bias[h]);
+    steps[(size_t)h * p.T + t] = make_float4(dt, rc_exp<T>(-p.A[h] * dt), 0.f, 0.f);
+  }
+}
+
+// Ring of record groups: warp kRecWarps sends the copies, warps 0 .. kRecWarps - 1 wait for them and give the stages back.
+static constexpr int kRecStages = 4;
+struct RecRing {
+  uint64_t *full, *empty;
+  volatile int* abort_flag;
+  int* status;
+  __device__ __forceinline__ void init(uint8_t* sm, int* st) {
+    full = reinterpret_cast<uint64_t*>(sm);
+    empty = full + kRecStages;
+    abort_flag = reinterpret_cast<volatile int*>(empty + kRecStages);
+    status = st;
+    if (threadIdx.x == 0) {
+      for (int i = 0; i < kRecStages; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], kRecWarps); }
+      *abort_flag = 0;
+      mbar_fence_init();
+    }
+    __syncthreads();
+  }
+  __device__ __forceinline__ bool wait_full(int c) {
+    return __all_sync(0xffffffffu, mbar_wait(&full[c % kRecStages], (uint32_t)((c / kRecStages) & 1), abort_flag, status));
+  }
+  __device__ __forceinline__ void release(int c) {
+    __syncwarp();
+    if ((threadIdx.x & 31) == 0) mbar_arrive(&empty[c % kRecStages]);
+  }
+  // one thread; send(c) puts group c on its way (expect_tx included)
+  template <typename F>
+  __device__ __forceinline__ void produce(int groups, F&& send) {
+    int c = 0;
+    for (; c < groups; ++c) {
+      if (c >= kRecStages && !mbar_wait(&empty[c % kRecStages], (uint32_t)((c / kRecStages - 1) & 1), abort_flag, status)) break;
+      send(c);
+    }
+    if (c < groups)          // given up: what is on its way lands before the block may end
+      for (int k = max(c - kRecStages, 0); k < c; ++k) {
+        const long long t0 = clock64();
+        while (!mbar_try_sleep(&full[k % kRecStages], (uint32_t)((k / kRecStages) & 1), 20000u) && clock64() - t0 < kSpinLimit) {}
+      }
+  }
+};
+
+// what a lane holds of a group's v (x) columns: token kl of the group, its own VPT columns
+template <typename T, int VPT>
+__device__ __forceinline__ void load_cols(float (&v)[VPT], const T* src, bool live, int col, int dv, bool vec) {
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) v[i] = 0.f;
+  if (!live) return;
+  if (VPT == 4 && sizeof(T) == 2 && vec) {
+    if (col < dv) {
+      const uint2 u = *reinterpret_cast<const uint2*>(src);
+      v[0] = __uint_as_float(u.x << 16); v[1 % VPT] = __uint_as_float(u.x & 0xffff0000u);
+      v[2 % VPT] = __uint_as_float(u.y << 16); v[3 % VPT] = __uint_as_float(u.y & 0xffff0000u);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i)
+      if (col + i < dv) v[i] = rc_ld(src + i);
+  }
+}
+
+static constexpr int kRecHead = 128;         // barriers in front of the ring
+
+template <typename T, int R, int VPT>
+__global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) delta_stream_kernel(RecParams p, int slices, int vec_v) {
+  constexpr int DKP = R * 8, COLS = kRecWarps * 4 * VPT, REC = 3 * DKP + 4, STAGE = kRecTok * REC;
+  constexpr int PART = VPT == 1 ? 4 : (VPT == 2 ? 2 : 1);            // independent chains per sum
+  extern __shared__ __align__(128) uint8_t sm8[];
+  __shared__ __align__(16) float s_v[kRecWarps][kRecTok][4 * VPT];
+  const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
+  if (n < p.long_rows) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7, cg = lane >> 3;
+  const int groups = (n + kRecTok - 1) / kRecTok;
+  float* ring = reinterpret_cast<float*>(sm8 + kRecHead);
+  RecRing rr;
+  rr.init(sm8, p.status);
+  if (warp == kRecWarps) {
+    if (lane == 0) {
+      const float* src = p.records + ((size_t)h * p.T + r0) * REC;
+      rr.produce(groups, [&](int c) {
+        const uint32_t bytes = (uint32_t)min(kRecTok, n - c * kRecTok) * REC * 4;
+        mbar_expect_tx(&rr.full[c % kRecStages], bytes);
+        bulk_load(ring + (c % kRecStages) * STAGE, src + (size_t)c * STAGE, bytes, &rr.full[c % kRecStages]);
+      });
+    }
+    return;
+  }
+  const int dk = p.dk, dv = p.dv, col = slice * COLS + warp * 4 * VPT + cg * VPT;
+  float* st = p.state + ((size_t)slot * p.heads + h) * dk * dv;
+  const bool vec = dv % 4 == 0;
+  float S[R][VPT];
+  load_state<R, VPT>(S, st, kl, col, dk, dv, ctx == n, vec);
+  const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + kl) * p.ld_conv + (size_t)2 * p.groups * dk + (size_t)h * dv + col;
+  float vn[VPT];
+  load_cols<T, VPT>(vn, vsrc, kl < n, col, dv, vec_v);
+  bool ok = true;
+  for (int c = 0; c < groups; ++c) {
+    const int t0 = c * kRecTok, m = min(kRecTok, n - t0);
+    __syncwarp();                            // the last group's columns have been read
+#pragma unroll
+    for (int v = 0; v < VPT; ++v) s_v[warp][kl][cg * VPT + v] = vn[v];
+    vsrc += (size_t)kRecTok * p.ld_conv;
+    load_cols<T, VPT>(vn, vsrc, t0 + kRecTok + kl < n, col, dv, vec_v);
+    ok = rr.wait_full(c);
+    if (!ok) break;
+    __syncwarp();
+    const float* buf = ring + (c % kRecStages) * STAGE;
+    float y[VPT <= 2 ? kRecTok : 1][VPT];
+    auto token = [&](int j, float (&po)[VPT]) {
+      const float* s = buf + j * REC;
+      float part[VPT][PART], pq[VPT][PART], kr[R <= 16 ? R : 1];
+#pragma unroll
+      for (int v = 0; v < VPT; ++v)
+#pragma unroll
+        for (int i = 0; i < PART; ++i) part[v][i] = pq[v][i] = 0.f;
+#pragma unroll
+      for (int i4 = 0; i4 < R / 4; ++i4) {
+        const float4 q4 = *reinterpret_cast<const float4*>(s + kl * 4 + 32 * i4);
+        const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 32 * i4);
+        const float4 g4 = *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 32 * i4);
+        const float qa[4] = {q4.x, q4.y, q4.z, q4.w}, ka[4] = {k4.x, k4.y, k4.z, k4.w}, ga[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          if constexpr (R <= 16) kr[i4 * 4 + i] = ka[i];
+#pragma unroll
+          for (int v = 0; v < VPT; ++v) {
+            float& x = S[i4 * 4 + i][v];
+            x *= ga[i];
+            part[v][i % PART] = fmaf(x, ka[i], part[v][i % PART]);
+            pq[v][i % PART] = fmaf(x, qa[i], pq[v][i % PART]);
+          }
+        }
+      }
+      float sum[VPT];
+#pragma unroll
+      for (int v = 0; v < VPT; ++v) {
+        sum[v] = part[v][0];
+        po[v] = pq[v][0];
+#pragma unroll
+        for (int i = 1; i < PART; ++i) { sum[v] += part[v][i]; po[v] += pq[v][i]; }
+      }
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+        for (int v = 0; v < VPT; ++v) sum[v] += __shfl_xor_sync(0xffffffffu, sum[v], o);
+      const float2 bk = *reinterpret_cast<const float2*>(s + 3 * DKP);        // beta, k . q
+      float u[VPT];
+#pragma unroll
+      for (int v = 0; v < VPT; ++v) u[v] = bk.x * (s_v[warp][j][cg * VPT + v] - sum[v]);
+#pragma unroll
+      for (int i4 = 0; i4 < R / 4; ++i4) {
+        float ka[4];
+        if constexpr (R <= 16) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) ka[i] = kr[i4 * 4 + i];
+        } else {
+          const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 32 * i4);
+          ka[0] = k4.x; ka[1] = k4.y; ka[2] = k4.z; ka[3] = k4.w;
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int v = 0; v < VPT; ++v) S[i4 * 4 + i][v] = fmaf(ka[i], u[v], S[i4 * 4 + i][v]);
+      }
+#pragma unroll
+      for (int v = 0; v < VPT; ++v) po[v] = kl == 0 ? fmaf(bk.y, u[v], po[v]) : po[v];
+      if constexpr (VPT == 4) {
+        // the four columns spread over the lanes
+        const bool up = kl & 4, up2 = kl & 2;
+        const float x0 = (up ? po[2 % VPT] : po[0]) + __shfl_xor_sync(0xffffffffu, up ? po[0] : po[2 % VPT], 4);
+        const float x1 = (up ? po[3 % VPT] : po[1 % VPT]) + __shfl_xor_sync(0xffffffffu, up ? po[1 % VPT] : po[3 % VPT], 4);
+        float o1 = (up2 ? x1 : x0) + __shfl_xor_sync(0xffffffffu, up2 ? x0 : x1, 2);
+        o1 += __shfl_xor_sync(0xffffffffu, o1, 1);
+        const int v0 = (up ? 2 : 0) + (up2 ? 1 : 0);
+        if ((kl & 1) == 0 && col + v0 < dv) p.out[((size_t)(r0 + t0 + j) * p.heads + h) * dv + col + v0] = o1;
+      }
+    };
+    if (m == kRecTok) {
+#pragma unroll
+      for (int j = 0; j < kRecTok; ++j) token(j, y[VPT <= 2 ? j : 0]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < kRecTok; ++j) {
+        if (j < m) token(j, y[VPT <= 2 ? j : 0]);
+        else if constexpr (VPT <= 2) {
+#pragma unroll
+          for (int v = 0; v < VPT; ++v) y[VPT <= 2 ? j : 0][v] = 0.f;
+        }
+      }
+    }
+    rr.release(c);
+    if constexpr (VPT <= 2) {
+      spread_tokens<VPT>(y, kl);
+      if (kl < m) store_cols<VPT>(p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col, y[0], col, dv, vec);
+    }
+  }
+  if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, dk, dv, vec);
+}
+
+template <typename T, int R, int VPT>
+__global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) state_space_stream_kernel(RecParams p, int slices, int vec_v) {
+  constexpr int NP = R * 8, COLS = kRecWarps * 4 * VPT, REC = 2 * NP, STAGE = kRecTok * (REC + 4);
+  extern __shared__ __align__(128) uint8_t sm8[];
+  __shared__ __align__(16) float s_v[kRecWarps][kRecTok][4 * VPT];
+  const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
+  if (n < p.long_rows) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7, cg = lane >> 3;
+  const int groups = (n + kRecTok - 1) / kRecTok;
+  float* ring = reinterpret_cast<float*>(sm8 + kRecHead);
+  RecRing rr;
+  rr.init(sm8, p.status);
+  if (warp == kRecWarps) {
+    if (lane == 0) {
+      const float* src = p.records + ((size_t)(h / (p.heads / p.groups)) * p.T + r0) * REC;
+      const float* steps = p.records + (size_t)p.groups * p.T * REC + ((size_t)h * p.T + r0) * 4;
+      rr.produce(groups, [&](int c) {
+        const uint32_t m = (uint32_t)min(kRecTok, n - c * kRecTok);
+        float* dst = ring + (c % kRecStages) * STAGE;
+        mbar_expect_tx(&rr.full[c % kRecStages], m * (REC + 4) * 4);
+        bulk_load(dst, src + (size_t)c * kRecTok * REC, m * REC * 4, &rr.full[c % kRecStages]);
+        bulk_load(dst + kRecTok * REC, steps + (size_t)c * kRecTok * 4, m * 16, &rr.full[c % kRecStages]);
+      });
+    }
+    return;
+  }
+  const int N = p.dk, dv = p.dv, col = slice * COLS + warp * 4 * VPT + cg * VPT;
+  float* st = p.state + ((size_t)slot * p.heads + h) * N * dv;
+  const bool vec = dv % 4 == 0;
+  float S[R][VPT];
+  load_state<R, VPT>(S, st, kl, col, N, dv, ctx == n, vec);
+  const float D = p.D ? p.D[h] : 0.f;
+  const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + kl) * p.ld_conv + (size_t)h * dv + col;
+  float vn[VPT];
+  load_cols<T, VPT>(vn, vsrc, kl < n, col, dv, vec_v);
+  bool ok = true;
+  for (int c = 0; c < groups; ++c) {
+    const int t0 = c * kRecTok, m = min(kRecTok, n - t0);
+    __syncwarp();
+    float x_own[VPT];
+#pragma unroll
+    for (int v = 0; v < VPT; ++v) s_v[warp][kl][cg * VPT + v] = x_own[v] = vn[v];
+    vsrc += (size_t)kRecTok * p.ld_conv;
+    load_cols<T, VPT>(vn, vsrc, t0 + kRecTok + kl < n, col, dv, vec_v);
+    ok = rr.wait_full(c);
+    if (!ok) break;
+    __syncwarp();
+    const float* buf = ring + (c % kRecStages) * STAGE;
+    float y[kRecTok][VPT];
+    auto token = [&](int j) {
+      const float* s = buf + j * REC;
+      const float2 step = *reinterpret_cast<const float2*>(buf + kRecTok * REC + j * 4);      // dt, decay
+      float x[VPT];
+#pragma unroll
+      for (int v = 0; v < VPT; ++v) { x[v] = step.x * s_v[warp][j][cg * VPT + v]; y[j][v] = 0.f; }
+#pragma unroll
+      for (int i4 = 0; i4 < R / 4; ++i4) {
+        const float4 b4 = *reinterpret_cast<const float4*>(s + kl * 4 + 32 * i4);
+        const float4 c4 = *reinterpret_cast<const float4*>(s + NP + kl * 4 + 32 * i4);
+        const float ba[4] = {b4.x, b4.y, b4.z, b4.w}, ca[4] = {c4.x, c4.y, c4.z, c4.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int v = 0; v < VPT; ++v) {
+            float& z = S[i4 * 4 + i][v];
+            z = fmaf(z, step.y, ba[i] * x[v]);
+            y[j][v] = fmaf(z, ca[i], y[j][v]);
+          }
+      }
+    };
+    if (m == kRecTok) {
+#pragma unroll
+      for (int j = 0; j < kRecTok; ++j) token(j);
+    } else {
+#pragma unroll
+      for (int j = 0; j < kRecTok; ++j) {
+        if (j < m) token(j);
+        else {
+#pragma unroll
+          for (int v = 0; v < VPT; ++v) y[j][v] = 0.f;
+        }
+      }
+    }
+    rr.release(c);
+    spread_tokens<VPT>(y, kl);
+#pragma unroll
+    for (int v = 0; v < VPT; ++v) y[0][v] = fmaf(D, x_own[v], y[0][v]);
+    if (kl < m) store_cols<VPT>(p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col, y[0], col, dv, vec);
+  }
+  if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, N, dv, vec);
 }
 
 // ------------------------------------------------------------------------------------------ norm over groups with a gate
@@ -384,11 +751,29 @@ __global__ void __launch_bounds__(256) group_norm_kernel(GroupNormParams p) {
   const float* o = p.o + (size_t)unit * p.n;
   const T* z = p.z ? reinterpret_cast<const T*>(p.z) + (size_t)t * p.ldz + (size_t)g * p.n : nullptr;
   float ss = 0.f;
-  for (int c = i0; c < p.n; c += STEP) {
-    float x[VEC], gt[VEC];
-    gn_load<T, VEC>(p, o, p.gate_first ? z : nullptr, c, x, gt);
+  constexpr int KEEP = VEC == 4 ? 4 : 1;             // columns of this many turns stay in registers
+  float kx[KEEP][VEC], kg[KEEP][VEC];
+  if (p.n <= KEEP * STEP) {
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) { x[j] *= gt[j]; ss = fmaf(x[j], x[j], ss); }
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = i0 + i * STEP;
+      if (c < p.n) gn_load<T, VEC>(p, o, z, c, kx[i], kg[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+      if (i0 + i * STEP < p.n)
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          const float x = p.gate_first ? kx[i][j] * kg[i][j] : kx[i][j];
+          ss = fmaf(x, x, ss);
+        }
+  } else {
+    for (int c = i0; c < p.n; c += STEP) {
+      float x[VEC], gt[VEC];
+      gn_load<T, VEC>(p, o, p.gate_first ? z : nullptr, c, x, gt);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) { x[j] *= gt[j]; ss = fmaf(x[j], x[j], ss); }
+    }
   }
   ss = warp_sum(ss);
   if constexpr (WARPS > 1) {
@@ -400,82 +785,139 @@ __global__ void __launch_bounds__(256) group_norm_kernel(GroupNormParams p) {
   }
   const float f = p.post / sqrtf(ss / (float)p.n + p.eps);
   T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + (size_t)g * p.n;
-  for (int c = i0; c < p.n; c += STEP) {
-    float x[VEC], gt[VEC];
-    gn_load<T, VEC>(p, o, z, c, x, gt);
+  auto put = [&](int c, const float (&x)[VEC], const float (&gt)[VEC]) {
     const int wc = (int)(((long long)g * p.n + c) % p.w_period);
     T e[VEC];
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
-      x[j] *= f * gt[j] * p.w[VEC == 1 ? wc : wc + j];
-      if constexpr (sizeof(T) == 4) e[j] = x[j];
-      else e[j] = __float2bfloat16(x[j]);
+      const float v = x[j] * (f * gt[j] * p.w[VEC == 1 ? wc : wc + j]);
+      if constexpr (sizeof(T) == 4) e[j] = v;
+      else e[j] = __float2bfloat16(v);
     }
     if constexpr (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(out + c) = *reinterpret_cast<uint2*>(e);
     else if constexpr (VEC == 4) *reinterpret_cast<float4*>(out + c) = *reinterpret_cast<float4*>(e);
     else out[c] = e[0];
+  };
+  if (p.n <= KEEP * STEP) {
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+      if (i0 + i * STEP < p.n) put(i0 + i * STEP, kx[i], kg[i]);
+  } else {
+    for (int c = i0; c < p.n; c += STEP) {
+      float x[VEC], gt[VEC];
+      gn_load<T, VEC>(p, o, z, c, x, gt);
+      put(c, x, gt);
+    }
   }
 }
 
 template <typename T, int R, int VPT, bool DELTA>
-static int launch_rec(const RecParams& p, int B, int ahead, cudaStream_t s) {
-  constexpr int DKP = R * 8, COLS = kRecWarps * 4 * VPT;
+static int launch_short_runs(const RecParams& p, int B, cudaStream_t s) {
+  constexpr int COLS = kRecWarps * 4 * VPT;
   const int slices = (p.dv + COLS - 1) / COLS;
-  const size_t smem = (size_t)2 * kRecTok * ((DELTA ? 3 : 2) * DKP + COLS + 4) * 4;
+  const size_t smem = (size_t)2 * kRecTok * ((DELTA ? 3 : 2) * R * 8 + COLS + 4) * 4;
   auto kern = DELTA ? delta_rule_kernel<T, R, VPT> : state_space_kernel<T, R, VPT>;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(kern, 200 * 1024);
   if (e != cudaSuccess) return (int)e;
-  kern<<<dim3(B * slices, p.heads), ahead ? 256 : 128, smem, s>>>(p, slices);
+  kern<<<dim3(B * slices, p.heads), kRecWarps * 32, smem, s>>>(p, slices);
+  return (int)cudaGetLastError();
+}
+template <typename T, int R, int VPT, bool DELTA>
+static int launch_long_runs(const RecParams& p, int B, cudaStream_t s) {
+  constexpr int COLS = kRecWarps * 4 * VPT;
+  const int slices = (p.dv + COLS - 1) / COLS;
+  const size_t smem = kRecHead + (size_t)kRecStages * kRecTok * ((DELTA ? 3 : 2) * R * 8 + 4) * 4;
+  auto kern = DELTA ? delta_stream_kernel<T, R, VPT> : state_space_stream_kernel<T, R, VPT>;
+  static PerDeviceOnce once;
+  cudaError_t e = once.smem_limit(kern, 220 * 1024);
+  if (e != cudaSuccess) return (int)e;
+  const long long off = DELTA ? 2LL * p.groups * p.dk : 0;             // first v (x) channel
+  const int vec_v = (reinterpret_cast<uintptr_t>(p.conv) & 7) == 0 && p.ld_conv % 4 == 0 && off % 4 == 0 && p.dv % 4 == 0;
+  kern<<<dim3(B * slices, p.heads), (kRecWarps + 1) * 32, smem, s>>>(p, slices, vec_v);
   return (int)cudaGetLastError();
 }
 
-// columns per lane: 4 keeps the reductions and the shared-memory reads few; runs with too few warps to fill the GPU take fewer
+template <int R, bool DELTA>
+static long long record_floats(int T, int heads, int groups) {
+  if (DELTA) return (long long)heads * T * (3 * R * 8 + 4);
+  return (long long)groups * T * 2 * R * 8 + (long long)heads * T * 4;
+}
+
+// Columns per lane: 4 keeps the reductions and the shared-memory reads few; long runs with too few warps to fill the GPU take fewer.
 template <typename T, int R, bool DELTA>
-static int pick_cols(const RecParams& p, int B, int max_q, cudaStream_t s) {
-  const int ahead = max_q > 2 * kRecTok;
-  if constexpr (R > 32) return launch_rec<T, R, 1, DELTA>(p, B, ahead, s);
-  else if constexpr (sizeof(T) == 4 || R > 16) return launch_rec<T, R, 2, DELTA>(p, B, ahead, s);
-  else {
+static int run_width(RecParams p, int B, int max_q, int short_runs, long long ws_bytes, cudaStream_t s) {
+  constexpr int V = R > 32 ? 1 : (sizeof(T) == 4 || R > 16 ? 2 : 4);
+  const bool stream = p.records != nullptr && max_q >= p.long_rows && p.out != nullptr;
+  if (stream) {
+    if (ws_bytes < record_floats<R, DELTA>(p.T, p.heads, p.groups) * 4 || (reinterpret_cast<uintptr_t>(p.records) & 15) || !p.seq_of_row)
+      return (int)cudaErrorInvalidValue;
+    if constexpr (DELTA) delta_records_kernel<T, R><<<(unsigned)(((long long)p.T * p.heads + 3) / 4), 128, 0, s>>>(p);
+    else state_space_records_kernel<T, R><<<p.T, 128, 0, s>>>(p);
+    int e = (int)cudaGetLastError();
+    if (e) return e;
     const long long warps = (long long)B * p.heads * ((p.dv + 15) / 16), room = 4LL * sm_count();
-    if (!ahead || warps >= room) return launch_rec<T, R, 4, DELTA>(p, B, ahead, s);
-    if (2 * warps >= room) return launch_rec<T, R, 2, DELTA>(p, B, ahead, s);
-    return launch_rec<T, R, 1, DELTA>(p, B, ahead, s);
+    if constexpr (V == 4) {
+      e = warps >= room ? launch_long_runs<T, R, 4, DELTA>(p, B, s) : 2 * warps >= room ? launch_long_runs<T, R, 2, DELTA>(p, B, s)
+                                                                                        : launch_long_runs<T, R, 1, DELTA>(p, B, s);
+    } else {
+      e = launch_long_runs<T, R, V, DELTA>(p, B, s);
+    }
+    if (e || !short_runs) return e;
+  } else {
+    p.long_rows = 0x7fffffff;
   }
+  return launch_short_runs<T, R, V, DELTA>(p, B, s);
 }
 
 template <typename T, bool DELTA>
-static int run_rec(const RecParams& p, int B, int max_q, cudaStream_t s) {
+static int run_rec(const RecParams& p, int B, int max_q, int short_runs, long long ws_bytes, cudaStream_t s) {
   if (B == 0) return 0;
   if (B < 0 || p.heads < 1 || p.heads > 65535 || p.groups < 1 || p.heads % p.groups || p.dk < 1 || p.dk > 512 || p.dv < 1)
     return (int)cudaErrorInvalidValue;
-  if (p.dk <= 32) return pick_cols<T, 4, DELTA>(p, B, max_q, s);
-  if (p.dk <= 64) return pick_cols<T, 8, DELTA>(p, B, max_q, s);
-  if (p.dk <= 128) return pick_cols<T, 16, DELTA>(p, B, max_q, s);
-  if (p.dk <= 256) return pick_cols<T, 32, DELTA>(p, B, max_q, s);
-  return pick_cols<T, 64, DELTA>(p, B, max_q, s);
+#define BLZ_REC(R) return run_width<T, R, DELTA>(p, B, max_q, short_runs, ws_bytes, s)
+  if (p.dk <= 32) BLZ_REC(4);
+  if (p.dk <= 64) BLZ_REC(8);
+  if (p.dk <= 128) BLZ_REC(16);
+  if (p.dk <= 256) BLZ_REC(32);
+  BLZ_REC(64);
+#undef BLZ_REC
 }
 
 }  // namespace blz
 
+// Runs of at least this many new tokens are long runs where the caller gives a workspace.
+static constexpr int kLongRows = 32;
+BLZ_API int blz_rec_long_rows() { return kLongRows; }
+// Workspace bytes of a step of T rows (delta: 1 = blz_delta_rule, 0 = blz_state_space).
+BLZ_API long long blz_rec_ws_bytes(int delta, int T, int heads, int groups, int dk) {
+  const int R = dk <= 32 ? 4 : dk <= 64 ? 8 : dk <= 128 ? 16 : dk <= 256 ? 32 : 64;
+  return 4 * (delta ? (long long)heads * T * (3 * R * 8 + 4) : (long long)groups * T * 2 * R * 8 + (long long)heads * T * 4);
+}
+
 // Delta rule with channel decays over every sequence of the batch (see RecParams; leading dimensions in elements; conv channels
 // [q key_heads * dk | k key_heads * dk | v heads * dv]).  out fp32 [T, heads * dv] or null.  no_store: optional [B], 1 = leave the
-// state as it was.  dk <= 512.
+// state as it was.  max_q: the longest run; ws (or null: every run is taken as a short one): blz_rec_ws_bytes; short_runs: there
+// are runs below blz_rec_long_rows.  dk <= 512.
 BLZ_API int blz_delta_rule(const void* conv, long long ld_conv, const void* a, long long ld_a, const void* b, long long ld_b, const float* A,
                            const float* dt_bias, float* state, float* out, const int* slots, const int* q_start, const int* ctx_len,
-                           const int* no_store, int B, int heads, int key_heads, int dk, int dv, int max_q, int f32, cudaStream_t s) {
+                           const int* no_store, int B, int heads, int key_heads, int dk, int dv, const int* seq_of_row, int T, int max_q,
+                           int short_runs, float* ws, long long ws_bytes, int f32, cudaStream_t s) {
   using namespace blz;
-  const RecParams p = {conv, a, b, A, dt_bias, nullptr, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_a, ld_b, heads, key_heads, dk, dv};
-  return f32 ? run_rec<float, true>(p, B, max_q, s) : run_rec<__nv_bfloat16, true>(p, B, max_q, s);
+  const RecParams p = {conv, a, b, A, dt_bias, nullptr, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_a, ld_b, heads, key_heads,
+                       dk, dv, seq_of_row, ws, T, kLongRows, status_word()};
+  return f32 ? run_rec<float, true>(p, B, max_q, short_runs, ws_bytes, s) : run_rec<__nv_bfloat16, true>(p, B, max_q, short_runs, ws_bytes, s);
 }
 
 // State-space duality (conv channels [x heads * dv | B groups * N | C groups * N]); other arguments as above.  N <= 512.
 BLZ_API int blz_state_space(const void* conv, long long ld_conv, const void* dt, long long ld_dt, const float* A, const float* dt_bias,
                             const float* D, float* state, float* out, const int* slots, const int* q_start, const int* ctx_len,
-                            const int* no_store, int B, int heads, int groups, int N, int dv, int max_q, int f32, cudaStream_t s) {
+                            const int* no_store, int B, int heads, int groups, int N, int dv, const int* seq_of_row, int T, int max_q,
+                            int short_runs, float* ws, long long ws_bytes, int f32, cudaStream_t s) {
   using namespace blz;
-  const RecParams p = {conv, dt, nullptr, A, dt_bias, D, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_dt, 0, heads, groups, N, dv};
-  return f32 ? run_rec<float, false>(p, B, max_q, s) : run_rec<__nv_bfloat16, false>(p, B, max_q, s);
+  const RecParams p = {conv, dt, nullptr, A, dt_bias, D, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_dt, 0, heads, groups,
+                       N, dv, seq_of_row, ws, T, kLongRows, status_word()};
+  return f32 ? run_rec<float, false>(p, B, max_q, short_runs, ws_bytes, s) : run_rec<__nv_bfloat16, false>(p, B, max_q, short_runs, ws_bytes, s);
 }
 
 // RMS norm of each of `groups` runs of n columns of fp32 rows, with a gate (GroupNormParams), to the activation type.
@@ -488,7 +930,7 @@ BLZ_API int blz_group_norm(const float* o, const void* z, long long ldz, const f
   const int vec = n % 4 == 0 && w_period % 4 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0 && (!z || ok(z, ldz)) && ok(out, ld_out);
   const GroupNormParams p = {o, z, w, out, ldz, ld_out, T, groups, n, w_period, sigmoid, gate_first, vec, eps, post};
   const long long units = (long long)T * groups;
-  const bool wide = n > 512;
+  const bool wide = n > 1024;
   const dim3 grid((unsigned)(wide ? units : (units + 7) / 8));
 #define BLZ_GN(TT, V) return (int)(wide ? launch_pdl(group_norm_kernel<TT, 8, V>, grid, dim3(256), 0, s, p) \
                                         : launch_pdl(group_norm_kernel<TT, 1, V>, grid, dim3(256), 0, s, p))
