@@ -184,7 +184,7 @@ class CudaOps:
         lib.blz_soft_tc.argtypes = common + shape + [_c.c_int, _c.c_int, VP]
         lib.blz_soft_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
         lib.blz_short_conv.argtypes = [VP, LL] + [VP] * 8 + [_c.c_int] * 5 + [VP]
-        runs = [_c.c_int] * 5 + [VP] + [_c.c_int] * 3 + [VP, LL, _c.c_int, VP]
+        runs = [_c.c_int] * 5 + [VP] + [_c.c_int] * 2 + [VP, LL, _c.c_int, VP]
         lib.blz_delta_rule.argtypes = [VP, LL, VP, LL, VP, LL] + [VP] * 8 + runs
         lib.blz_state_space.argtypes = [VP, LL, VP, LL] + [VP] * 9 + runs
         lib.blz_rec_ws_bytes.restype = LL
@@ -938,16 +938,20 @@ class CudaOps:
         seqs = (_ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(batch.gdn_defer), batch.slots.numel())
         state, st, longest, T, delta = kv.rec_state[layer_idx], self._stream(), int(batch.max_q_len), y.shape[0], R.kind == "delta"
         groups = r.kv_heads if delta else r.groups
-        ws, ws_bytes, short = None, 0, True
-        long_rows = int(self.lib.blz_rec_long_rows())
-        if o is not None and longest >= long_rows:
-            # long runs take the streaming kernels, which read what a token needs from a workspace filled for all tokens at once
+        # which kernels the step needs: single tokens, short runs, and long runs, which read what a token needs from a workspace
+        # filled for all tokens at once
+        lens = [e - s for s, e in zip(batch.h_q_start, batch.h_q_start[1:])]
+        long_rows, ws, ws_bytes = int(self.lib.blz_rec_long_rows()), None, 0
+        kinds = (1 if 1 in lens else 0) | (2 if any(1 < n < long_rows for n in lens) else 0)
+        if longest >= long_rows:
             ws_bytes = int(self.lib.blz_rec_ws_bytes(int(delta), T, r.heads, groups, r.state))
-            if ws_bytes <= self.REC_MAX_WS:
+            if o is not None and ws_bytes <= self.REC_MAX_WS:
                 ws = torch.empty(ws_bytes, dtype=torch.uint8, device=self.device)
-                short = any(0 < e - s < long_rows for s, e in zip(batch.h_q_start, batch.h_q_start[1:]))
-                self.launches += 2 if short else 1
-        runs = (_ptr(batch.seq_of_row), T, longest, int(short), _ptr(ws), ws_bytes, f32, st)
+                kinds |= 4
+            else:
+                kinds |= 2
+        self.launches += (0, 0, 0, 1, 1, 2, 2, 3)[kinds]
+        runs = (_ptr(batch.seq_of_row), T, kinds, _ptr(ws), ws_bytes, f32, st)
         if delta:
             self._check(self.lib.blz_delta_rule(_ptr(y), y.stride(0), _ptr(low), low.stride(0), VP(proj.data_ptr() + M.cols["beta"] * es),
                                                 proj.stride(0), _ptr(R.A), _ptr(R.dt_bias), _ptr(state), _ptr(o), *seqs, r.heads,

@@ -9,7 +9,7 @@
 // multiply-adds per lane and product, and one reduction over 8 lanes.  The delta rule takes both of its products from the decayed
 // state at once (o = S^T q + (k . q) u), which leaves a single reduction on the path from token to token.  What a token needs
 // besides the state (unit vectors, decays, steps: all fp32) does not depend on the state:
-//   runs of a few tokens (decode, verify rows) prepare it in shared memory, 8 tokens at a time;
+//   single tokens (decode) take it straight from memory; runs of a few (verify rows) prepare it in shared memory, 8 tokens at a time;
 //   long runs have it prepared for all tokens at once by a kernel of its own, as one record per token and head (or group) in a
 //   workspace, and the kernel that holds the state streams the records of 8 tokens at a time through a ring of bulk copies.
 #include "blaze/host.h"
@@ -50,12 +50,12 @@ __device__ __forceinline__ float rc_softplus(float x) { return x > 20.f ? x : lo
 template <typename T>
 __device__ __forceinline__ float rc_sigmoid(float x) { return 1.f / (1.f + rc_exp<T>(-x)); }
 
-// lane (row group kl, column group cg) of a warp: rows kl * 4 + 32 * (i / 4) + i % 4, i < R; columns col .. col + VPT
-template <int R, int VPT>
+// lane (row group kl < KL, column group cg) of a warp: rows kl * 4 + 4 KL * (i / 4) + i % 4, i < R; columns col .. col + VPT
+template <int KL, int R, int VPT>
 __device__ __forceinline__ void load_state(float (&S)[R][VPT], const float* st, int kl, int col, int dk, int dv, bool zero, bool vec) {
 #pragma unroll
   for (int i = 0; i < R; ++i) {
-    const int r = kl * 4 + 32 * (i / 4) + (i & 3);
+    const int r = kl * 4 + 4 * KL * (i / 4) + (i & 3);
 #pragma unroll
     for (int c = 0; c < VPT; ++c) S[i][c] = 0.f;
     if (zero || r >= dk) continue;
@@ -70,11 +70,11 @@ __device__ __forceinline__ void load_state(float (&S)[R][VPT], const float* st, 
     }
   }
 }
-template <int R, int VPT>
+template <int KL, int R, int VPT>
 __device__ __forceinline__ void store_state(const float (&S)[R][VPT], float* st, int kl, int col, int dk, int dv, bool vec) {
 #pragma unroll
   for (int i = 0; i < R; ++i) {
-    const int r = kl * 4 + 32 * (i / 4) + (i & 3);
+    const int r = kl * 4 + 4 * KL * (i / 4) + (i & 3);
     if (r >= dk) continue;
     float* p = st + (size_t)r * dv + col;
     if (VPT == 4 && vec && col < dv) {
@@ -87,8 +87,8 @@ __device__ __forceinline__ void store_state(const float (&S)[R][VPT], float* st,
   }
 }
 
-// sums of y[token][column] over the 8 lanes of a column, the 8 tokens spread over them: lane kl ends with token kl in y[0]
-template <int VPT>
+// sums of y[token][column] over the KL (8 or 16) lanes of a column, the 8 tokens spread over them: lane kl ends with token kl % 8 in y[0]
+template <int KL, int VPT>
 __device__ __forceinline__ void spread_tokens(float (&y)[kRecTok][VPT], int kl) {
   const bool u4 = kl & 4, u2 = kl & 2, u1 = kl & 1;
 #pragma unroll
@@ -99,6 +99,7 @@ __device__ __forceinline__ void spread_tokens(float (&y)[kRecTok][VPT], int kl) 
 #pragma unroll
     for (int j = 0; j < 2; ++j) z2[j] = (u2 ? z4[j + 2] : z4[j]) + __shfl_xor_sync(0xffffffffu, u2 ? z4[j] : z4[j + 2], 2);
     y[0][v] = (u1 ? z2[1] : z2[0]) + __shfl_xor_sync(0xffffffffu, u1 ? z2[0] : z2[1], 1);
+    if constexpr (KL == 16) y[0][v] += __shfl_xor_sync(0xffffffffu, y[0][v], 8);
   }
 }
 template <int VPT>
@@ -120,13 +121,13 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_r
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
-  if (n <= 0 || n >= p.long_rows) return;
+  if (n <= 1 || n >= p.long_rows) return;          // single tokens and long runs have kernels of their own
   const int dk = p.dk, dv = p.dv, hk = h / (p.heads / p.groups);
   const int col = slice * COLS + warp * 4 * VPT + (lane >> 3) * VPT;
   float* st = p.state + ((size_t)slot * p.heads + h) * dk * dv;
   const bool vec = dv % 4 == 0;
   float S[R][VPT];
-  load_state<R, VPT>(S, st, kl, col, dk, dv, ctx == n, vec);
+  load_state<8, R, VPT>(S, st, kl, col, dk, dv, ctx == n, vec);
   const float A = p.A[h], qs = rsqrtf((float)dk);
 
   auto stage = [&](int t0, float* buf) {
@@ -248,7 +249,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_r
     if (t0 + kRecTok < n) stage(t0 + kRecTok, sm + ((c + 1) & 1) * kRecTok * TOK);
     __syncthreads();
   }
-  if (!(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, dk, dv, vec);
+  if (!(p.no_store != nullptr && p.no_store[b])) store_state<8, R, VPT>(S, st, kl, col, dk, dv, vec);
 }
 
 template <typename T, int R, int VPT>
@@ -258,13 +259,13 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) state_s
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
-  if (n <= 0 || n >= p.long_rows) return;
+  if (n <= 1 || n >= p.long_rows) return;          // single tokens and long runs have kernels of their own
   const int N = p.dk, dv = p.dv, g = h / (p.heads / p.groups);
   const int col = slice * COLS + warp * 4 * VPT + (lane >> 3) * VPT;
   float* st = p.state + ((size_t)slot * p.heads + h) * N * dv;
   const bool vec = dv % 4 == 0;
   float S[R][VPT];
-  load_state<R, VPT>(S, st, kl, col, N, dv, ctx == n, vec);
+  load_state<8, R, VPT>(S, st, kl, col, N, dv, ctx == n, vec);
   const float A = p.A[h], bias = p.dt_bias[h], D = p.D ? p.D[h] : 0.f;
 
   auto stage = [&](int t0, float* buf) {
@@ -327,7 +328,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) state_s
         }
       }
       if (p.out) {
-        spread_tokens<VPT>(y, kl);
+        spread_tokens<8, VPT>(y, kl);
         if (t0 + kl < n) {
           const float* s = buf + kl * TOK + 2 * NP + lc;
 #pragma unroll
@@ -339,21 +340,150 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) state_s
     if (t0 + kRecTok < n) stage(t0 + kRecTok, sm + ((c + 1) & 1) * kRecTok * TOK);
     __syncthreads();
   }
-  if (!(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, N, dv, vec);
+  if (!(p.no_store != nullptr && p.no_store[b])) store_state<8, R, VPT>(S, st, kl, col, N, dv, vec);
+}
+
+// ------------------------------------------------------------------------------------------ single tokens
+// A decode row's state is read, changed and written back once; every lane takes what it needs of the token straight from memory, so
+// that all of a warp's reads are under way together and no warp waits for another.
+// KL lanes per column; elements of a vector as in load_state
+template <typename T, int KL, int R>
+__device__ __forceinline__ void load_vec_rows(float (&x)[R], const T* src, int kl, int n, bool vec) {
+#pragma unroll
+  for (int i4 = 0; i4 < R / 4; ++i4) {
+    const int r = kl * 4 + 4 * KL * i4;
+    if (vec && sizeof(T) == 2) {
+      uint2 u = make_uint2(0u, 0u);
+      if (r < n) u = *reinterpret_cast<const uint2*>(src + r);
+      x[i4 * 4] = __uint_as_float(u.x << 16); x[i4 * 4 + 1] = __uint_as_float(u.x & 0xffff0000u);
+      x[i4 * 4 + 2] = __uint_as_float(u.y << 16); x[i4 * 4 + 3] = __uint_as_float(u.y & 0xffff0000u);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[i4 * 4 + i] = r + i < n ? rc_ld(src + r + i) : 0.f;
+    }
+  }
+}
+template <int KL>
+__device__ __forceinline__ float lanes_sum(float x) {
+#pragma unroll
+  for (int o = KL / 2; o > 0; o >>= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
+  return x;
+}
+
+template <typename T, int KL, int R, int VPT>
+__global__ void __launch_bounds__(kRecWarps * 32, 3) delta_step_kernel(RecParams p, int slices, int vec_t) {
+  constexpr int CG = 32 / KL;
+  __shared__ __align__(16) float s_g[KL * R];
+  const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
+  if (n != 1) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane % KL;
+  const int dk = p.dk, dv = p.dv, hk = h / (p.heads / p.groups);
+  const int col = slice * kRecWarps * CG * VPT + warp * CG * VPT + lane / KL * VPT;
+  float* st = p.state + ((size_t)slot * p.heads + h) * dk * dv;
+  const bool vec = dv % 4 == 0;
+  float S[R][VPT], q[R], k[R];
+  alignas(16) float g[R];
+  load_state<KL, R, VPT>(S, st, kl, col, dk, dv, ctx == 1, vec);
+  const T* cv = reinterpret_cast<const T*>(p.conv) + (size_t)r0 * p.ld_conv;
+  load_vec_rows<T, KL, R>(q, cv + (size_t)hk * dk, kl, dk, vec_t);
+  load_vec_rows<T, KL, R>(k, cv + (size_t)(p.groups + hk) * dk, kl, dk, vec_t);
+  float v[VPT];
+#pragma unroll
+  for (int c = 0; c < VPT; ++c) v[c] = col + c < dv ? rc_ld(cv + (size_t)2 * p.groups * dk + (size_t)h * dv + col + c) : 0.f;
+  const float beta = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + (size_t)r0 * p.ld_b + h)), A = p.A[h];
+  // the decays, one per thread
+  const T* av = reinterpret_cast<const T*>(p.a) + (size_t)r0 * p.ld_a + (size_t)h * dk;
+  for (int d = threadIdx.x; d < KL * R; d += kRecWarps * 32)
+    s_g[d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d])) : 1.f;
+  float qq = 0.f, kk = 0.f, kq = 0.f;
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    qq = fmaf(q[i], q[i], qq);
+    kk = fmaf(k[i], k[i], kk);
+    kq = fmaf(k[i], q[i], kq);
+  }
+  const float qn = rsqrtf((float)dk) / sqrtf(lanes_sum<KL>(qq) + 1e-6f), kn = 1.f / sqrtf(lanes_sum<KL>(kk) + 1e-6f);
+  kq = lanes_sum<KL>(kq) * qn * kn;
+  __syncthreads();
+#pragma unroll
+  for (int i4 = 0; i4 < R / 4; ++i4) *reinterpret_cast<float4*>(&g[i4 * 4]) = *reinterpret_cast<const float4*>(s_g + kl * 4 + 4 * KL * i4);
+  float part[VPT], po[VPT];
+#pragma unroll
+  for (int c = 0; c < VPT; ++c) part[c] = po[c] = 0.f;
+#pragma unroll
+  for (int i = 0; i < R; ++i)
+#pragma unroll
+    for (int c = 0; c < VPT; ++c) {
+      S[i][c] *= g[i];
+      part[c] = fmaf(S[i][c], k[i], part[c]);
+      po[c] = fmaf(S[i][c], q[i], po[c]);
+    }
+#pragma unroll
+  for (int c = 0; c < VPT; ++c) {
+    const float u = beta * (v[c] - lanes_sum<KL>(part[c]) * kn);
+    po[c] = fmaf(kq, u, lanes_sum<KL>(po[c]) * qn);
+    part[c] = u * kn;
+  }
+#pragma unroll
+  for (int i = 0; i < R; ++i)
+#pragma unroll
+    for (int c = 0; c < VPT; ++c) S[i][c] = fmaf(k[i], part[c], S[i][c]);
+  if (p.out && kl == 0) store_cols<VPT>(p.out + ((size_t)r0 * p.heads + h) * dv + col, po, col, dv, vec);
+  if (!(p.no_store != nullptr && p.no_store[b])) store_state<KL, R, VPT>(S, st, kl, col, dk, dv, vec);
+}
+
+template <typename T, int KL, int R, int VPT>
+__global__ void __launch_bounds__(kRecWarps * 32, 4) state_space_step_kernel(RecParams p, int slices, int vec_t) {
+  constexpr int CG = 32 / KL;
+  const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
+  if (n != 1) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane % KL;
+  const int N = p.dk, dv = p.dv, grp = h / (p.heads / p.groups);
+  const int col = slice * kRecWarps * CG * VPT + warp * CG * VPT + lane / KL * VPT;
+  float* st = p.state + ((size_t)slot * p.heads + h) * N * dv;
+  const bool vec = dv % 4 == 0;
+  float S[R][VPT], B[R], C[R];
+  load_state<KL, R, VPT>(S, st, kl, col, N, dv, ctx == 1, vec);
+  const T* cv = reinterpret_cast<const T*>(p.conv) + (size_t)r0 * p.ld_conv;
+  const T* bc = cv + (size_t)p.heads * dv + (size_t)grp * N;
+  load_vec_rows<T, KL, R>(B, bc, kl, N, vec_t);
+  load_vec_rows<T, KL, R>(C, bc + (size_t)p.groups * N, kl, N, vec_t);
+  float x[VPT], y[VPT];
+#pragma unroll
+  for (int c = 0; c < VPT; ++c) x[c] = col + c < dv ? rc_ld(cv + (size_t)h * dv + col + c) : 0.f;
+  const float dt = rc_softplus<T>(rc_ld(reinterpret_cast<const T*>(p.a) + (size_t)r0 * p.ld_a + h) + p.dt_bias[h]);
+  const float dec = rc_exp<T>(-p.A[h] * dt), D = p.D ? p.D[h] : 0.f;
+#pragma unroll
+  for (int c = 0; c < VPT; ++c) y[c] = 0.f;
+#pragma unroll
+  for (int i = 0; i < R; ++i)
+#pragma unroll
+    for (int c = 0; c < VPT; ++c) {
+      S[i][c] = fmaf(S[i][c], dec, B[i] * (dt * x[c]));
+      y[c] = fmaf(S[i][c], C[i], y[c]);
+    }
+  if (!(p.no_store != nullptr && p.no_store[b])) store_state<KL, R, VPT>(S, st, kl, col, N, dv, vec);
+  if (p.out) {
+#pragma unroll
+    for (int c = 0; c < VPT; ++c) y[c] = fmaf(D, x[c], lanes_sum<KL>(y[c]));
+    if (kl == 0) store_cols<VPT>(p.out + ((size_t)r0 * p.heads + h) * dv + col, y, col, dv, vec);
+  }
 }
 
 // ------------------------------------------------------------------------------------------ long runs
 // Records: delta [heads][T][q | k | g | beta, k . q, 0, 0], state space [groups][T][B | C] and [heads][T][dt, decay, 0, 0];
-// vectors padded to R * 8 floats.
+// vectors padded to 32, 64, 128, 256 or 512 floats.
 __device__ __forceinline__ bool in_long_run(const RecParams& p, int t) {
   const int b = p.seq_of_row[t];
   return b >= 0 && p.q_start[b + 1] - p.q_start[b] >= p.long_rows;
 }
 
 // a warp per (row, head)
-template <typename T, int R>
+template <typename T, int DKP>
 __global__ void __launch_bounds__(128) delta_records_kernel(RecParams p) {
-  constexpr int DKP = R * 8, REC = 3 * DKP + 4, NV = DKP / 32;
+  constexpr int REC = 3 * DKP + 4, NV = DKP / 32;
   const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
   const int t = (int)(w / p.heads), h = (int)(w % p.heads), lane = threadIdx.x & 31;
   if (t >= p.T || !in_long_run(p, t)) return;
@@ -389,9 +519,9 @@ __global__ void __launch_bounds__(128) delta_records_kernel(RecParams p) {
 }
 
 // a block per row
-template <typename T, int R>
+template <typename T, int DKP>
 __global__ void __launch_bounds__(128) state_space_records_kernel(RecParams p) {
-  constexpr int NP = R * 8;
+  constexpr int NP = DKP;
   const int t = blockIdx.x, N = p.dk;
   if (!in_long_run(p, t)) return;
   const T* bc = reinterpret_cast<const T*>(p.conv) + (size_t)t * p.ld_conv + (size_t)p.heads * p.dv;
@@ -447,37 +577,37 @@ struct RecRing {
   }
 };
 
-// what a lane holds of a group's v (x) columns: token kl of the group, its own VPT columns
+// v (x) columns of a group of tokens on their way into a warp's shared memory, kColsAhead groups ahead of their use; lane kl < 8
+// brings token kl's VPT columns.  vec: they can be copied as one word of sizeof(T) * VPT bytes.
+static constexpr int kColsAhead = 3;
 template <typename T, int VPT>
-__device__ __forceinline__ void load_cols(float (&v)[VPT], const T* src, bool live, int col, int dv, bool vec) {
+__device__ __forceinline__ void send_cols(T* dst, const T* src, bool live, int col, int dv, bool vec) {
+  if (live) {
+    if (vec) {
+      if (col < dv)
+        asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"((int)sizeof(T) * VPT) : "memory");
+    } else {
 #pragma unroll
-  for (int i = 0; i < VPT; ++i) v[i] = 0.f;
-  if (!live) return;
-  if (VPT == 4 && sizeof(T) == 2 && vec) {
-    if (col < dv) {
-      const uint2 u = *reinterpret_cast<const uint2*>(src);
-      v[0] = __uint_as_float(u.x << 16); v[1 % VPT] = __uint_as_float(u.x & 0xffff0000u);
-      v[2 % VPT] = __uint_as_float(u.y << 16); v[3 % VPT] = __uint_as_float(u.y & 0xffff0000u);
+      for (int i = 0; i < VPT; ++i)
+        if (col + i < dv) dst[i] = src[i];
     }
-  } else {
-#pragma unroll
-    for (int i = 0; i < VPT; ++i)
-      if (col + i < dv) v[i] = rc_ld(src + i);
   }
+  asm volatile("cp.async.commit_group;" ::: "memory");
 }
+__device__ __forceinline__ void wait_cols() { asm volatile("cp.async.wait_group %0;" ::"n"(kColsAhead) : "memory"); }
 
 static constexpr int kRecHead = 128;         // barriers in front of the ring
 
-template <typename T, int R, int VPT>
+template <typename T, int KL, int R, int VPT>
 __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) delta_stream_kernel(RecParams p, int slices, int vec_v) {
-  constexpr int DKP = R * 8, COLS = kRecWarps * 4 * VPT, REC = 3 * DKP + 4, STAGE = kRecTok * REC;
-  constexpr int PART = VPT == 1 ? 4 : (VPT == 2 ? 2 : 1);            // independent chains per sum
+  constexpr int DKP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, REC = 3 * DKP + 4, STAGE = kRecTok * REC;
+  constexpr int PART = VPT == 2 ? 2 : 1;            // independent chains per sum
   extern __shared__ __align__(128) uint8_t sm8[];
-  __shared__ __align__(16) float s_v[kRecWarps][kRecTok][4 * VPT];
+  __shared__ __align__(16) T s_v[kRecWarps][kColsAhead + 1][kRecTok][CG * VPT];
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
   if (n < p.long_rows) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7, cg = lane >> 3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane % KL, cg = lane / KL;
   const int groups = (n + kRecTok - 1) / kRecTok;
   float* ring = reinterpret_cast<float*>(sm8 + kRecHead);
   RecRing rr;
@@ -493,52 +623,64 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
     }
     return;
   }
-  const int dk = p.dk, dv = p.dv, col = slice * COLS + warp * 4 * VPT + cg * VPT;
+  const int dk = p.dk, dv = p.dv, col = slice * COLS + warp * CG * VPT + cg * VPT;
   float* st = p.state + ((size_t)slot * p.heads + h) * dk * dv;
   const bool vec = dv % 4 == 0;
   float S[R][VPT];
-  load_state<R, VPT>(S, st, kl, col, dk, dv, ctx == n, vec);
-  const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + kl) * p.ld_conv + (size_t)2 * p.groups * dk + (size_t)h * dv + col;
-  float vn[VPT];
-  load_cols<T, VPT>(vn, vsrc, kl < n, col, dv, vec_v);
+  load_state<KL, R, VPT>(S, st, kl, col, dk, dv, ctx == n, vec);
+  const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + (kl & 7)) * p.ld_conv + (size_t)2 * p.groups * dk + (size_t)h * dv + col;
+  auto send_group = [&](int c) {
+    send_cols<T, VPT>(&s_v[warp][c % (kColsAhead + 1)][kl & 7][cg * VPT], vsrc + (size_t)c * kRecTok * p.ld_conv,
+                      kl < kRecTok && c * kRecTok + kl < n, col, dv, vec_v);
+  };
+#pragma unroll
+  for (int c = 0; c < kColsAhead; ++c) send_group(c);
   bool ok = true;
   for (int c = 0; c < groups; ++c) {
     const int t0 = c * kRecTok, m = min(kRecTok, n - t0);
     __syncwarp();                            // the last group's columns have been read
-#pragma unroll
-    for (int v = 0; v < VPT; ++v) s_v[warp][kl][cg * VPT + v] = vn[v];
-    vsrc += (size_t)kRecTok * p.ld_conv;
-    load_cols<T, VPT>(vn, vsrc, t0 + kRecTok + kl < n, col, dv, vec_v);
+    send_group(c + kColsAhead);
+    wait_cols();
+    const T(*cols)[CG * VPT] = s_v[warp][c % (kColsAhead + 1)];
     ok = rr.wait_full(c);
     if (!ok) break;
     __syncwarp();
     const float* buf = ring + (c % kRecStages) * STAGE;
     float y[VPT <= 2 ? kRecTok : 1][VPT];
-    auto token = [&](int j, float (&po)[VPT]) {
+    // what a token brings: the lane's rows of q, k and g, its v, beta and k . q
+    struct Tok {
+      float q[R], k[R], g[R], v[VPT];
+      float2 bk;
+    };
+    auto fetch = [&](int j, Tok& o) {
       const float* s = buf + j * REC;
-      float part[VPT][PART], pq[VPT][PART], kr[R <= 16 ? R : 1];
+#pragma unroll
+      for (int i4 = 0; i4 < R / 4; ++i4) {
+        const float4 q4 = *reinterpret_cast<const float4*>(s + kl * 4 + 4 * KL * i4);
+        const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 4 * KL * i4);
+        const float4 g4 = *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 4 * KL * i4);
+        o.q[i4 * 4] = q4.x; o.q[i4 * 4 + 1] = q4.y; o.q[i4 * 4 + 2] = q4.z; o.q[i4 * 4 + 3] = q4.w;
+        o.k[i4 * 4] = k4.x; o.k[i4 * 4 + 1] = k4.y; o.k[i4 * 4 + 2] = k4.z; o.k[i4 * 4 + 3] = k4.w;
+        o.g[i4 * 4] = g4.x; o.g[i4 * 4 + 1] = g4.y; o.g[i4 * 4 + 2] = g4.z; o.g[i4 * 4 + 3] = g4.w;
+      }
+      o.bk = *reinterpret_cast<const float2*>(s + 3 * DKP);
+#pragma unroll
+      for (int v = 0; v < VPT; ++v) o.v[v] = rc_ld(&cols[j][cg * VPT + v]);
+    };
+    auto token = [&](int j, const Tok& x, float (&po)[VPT]) {
+      float part[VPT][PART], pq[VPT][PART];
 #pragma unroll
       for (int v = 0; v < VPT; ++v)
 #pragma unroll
         for (int i = 0; i < PART; ++i) part[v][i] = pq[v][i] = 0.f;
 #pragma unroll
-      for (int i4 = 0; i4 < R / 4; ++i4) {
-        const float4 q4 = *reinterpret_cast<const float4*>(s + kl * 4 + 32 * i4);
-        const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 32 * i4);
-        const float4 g4 = *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 32 * i4);
-        const float qa[4] = {q4.x, q4.y, q4.z, q4.w}, ka[4] = {k4.x, k4.y, k4.z, k4.w}, ga[4] = {g4.x, g4.y, g4.z, g4.w};
+      for (int i = 0; i < R; ++i)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          if constexpr (R <= 16) kr[i4 * 4 + i] = ka[i];
-#pragma unroll
-          for (int v = 0; v < VPT; ++v) {
-            float& x = S[i4 * 4 + i][v];
-            x *= ga[i];
-            part[v][i % PART] = fmaf(x, ka[i], part[v][i % PART]);
-            pq[v][i % PART] = fmaf(x, qa[i], pq[v][i % PART]);
-          }
+        for (int v = 0; v < VPT; ++v) {
+          S[i][v] *= x.g[i];
+          part[v][i % PART] = fmaf(S[i][v], x.k[i], part[v][i % PART]);
+          pq[v][i % PART] = fmaf(S[i][v], x.q[i], pq[v][i % PART]);
         }
-      }
       float sum[VPT];
 #pragma unroll
       for (int v = 0; v < VPT; ++v) {
@@ -548,31 +690,20 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
         for (int i = 1; i < PART; ++i) { sum[v] += part[v][i]; po[v] += pq[v][i]; }
       }
 #pragma unroll
-      for (int o = 4; o > 0; o >>= 1)
+      for (int o = KL / 2; o > 0; o >>= 1)
 #pragma unroll
         for (int v = 0; v < VPT; ++v) sum[v] += __shfl_xor_sync(0xffffffffu, sum[v], o);
-      const float2 bk = *reinterpret_cast<const float2*>(s + 3 * DKP);        // beta, k . q
       float u[VPT];
 #pragma unroll
-      for (int v = 0; v < VPT; ++v) u[v] = bk.x * (s_v[warp][j][cg * VPT + v] - sum[v]);
+      for (int v = 0; v < VPT; ++v) u[v] = x.bk.x * (x.v[v] - sum[v]);
 #pragma unroll
-      for (int i4 = 0; i4 < R / 4; ++i4) {
-        float ka[4];
-        if constexpr (R <= 16) {
+      for (int i = 0; i < R; ++i)
 #pragma unroll
-          for (int i = 0; i < 4; ++i) ka[i] = kr[i4 * 4 + i];
-        } else {
-          const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 32 * i4);
-          ka[0] = k4.x; ka[1] = k4.y; ka[2] = k4.z; ka[3] = k4.w;
-        }
+        for (int v = 0; v < VPT; ++v) S[i][v] = fmaf(x.k[i], u[v], S[i][v]);
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-          for (int v = 0; v < VPT; ++v) S[i4 * 4 + i][v] = fmaf(ka[i], u[v], S[i4 * 4 + i][v]);
-      }
-#pragma unroll
-      for (int v = 0; v < VPT; ++v) po[v] = kl == 0 ? fmaf(bk.y, u[v], po[v]) : po[v];
+      for (int v = 0; v < VPT; ++v) po[v] = kl == 0 ? fmaf(x.bk.y, u[v], po[v]) : po[v];
       if constexpr (VPT == 4) {
+        static_assert(VPT != 4 || KL == 8);
         // the four columns spread over the lanes
         const bool up = kl & 4, up2 = kl & 2;
         const float x0 = (up ? po[2 % VPT] : po[0]) + __shfl_xor_sync(0xffffffffu, up ? po[0] : po[2 % VPT], 4);
@@ -583,14 +714,24 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
         if ((kl & 1) == 0 && col + v0 < dv) p.out[((size_t)(r0 + t0 + j) * p.heads + h) * dv + col + v0] = o1;
       }
     };
+    constexpr bool FETCH_AHEAD = R * VPT <= 16;          // registers for the next token's operands
     if (m == kRecTok) {
+      Tok tok[2];
+      if (FETCH_AHEAD) fetch(0, tok[0]);
 #pragma unroll
-      for (int j = 0; j < kRecTok; ++j) token(j, y[VPT <= 2 ? j : 0]);
+      for (int j = 0; j < kRecTok; ++j) {
+        if (!FETCH_AHEAD) fetch(j, tok[j & 1]);
+        else if (j + 1 < kRecTok) fetch(j + 1, tok[(j + 1) & 1]);
+        token(j, tok[j & 1], y[VPT <= 2 ? j : 0]);
+      }
     } else {
 #pragma unroll
       for (int j = 0; j < kRecTok; ++j) {
-        if (j < m) token(j, y[VPT <= 2 ? j : 0]);
-        else if constexpr (VPT <= 2) {
+        if (j < m) {
+          Tok tok;
+          fetch(j, tok);
+          token(j, tok, y[VPT <= 2 ? j : 0]);
+        } else if constexpr (VPT <= 2) {
 #pragma unroll
           for (int v = 0; v < VPT; ++v) y[VPT <= 2 ? j : 0][v] = 0.f;
         }
@@ -598,22 +739,22 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
     }
     rr.release(c);
     if constexpr (VPT <= 2) {
-      spread_tokens<VPT>(y, kl);
+      spread_tokens<KL, VPT>(y, kl);
       if (kl < m) store_cols<VPT>(p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col, y[0], col, dv, vec);
     }
   }
-  if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, dk, dv, vec);
+  if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<KL, R, VPT>(S, st, kl, col, dk, dv, vec);
 }
 
-template <typename T, int R, int VPT>
+template <typename T, int KL, int R, int VPT>
 __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) state_space_stream_kernel(RecParams p, int slices, int vec_v) {
-  constexpr int NP = R * 8, COLS = kRecWarps * 4 * VPT, REC = 2 * NP, STAGE = kRecTok * (REC + 4);
+  constexpr int NP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, REC = 2 * NP, STAGE = kRecTok * (REC + 4);
   extern __shared__ __align__(128) uint8_t sm8[];
-  __shared__ __align__(16) float s_v[kRecWarps][kRecTok][4 * VPT];
+  __shared__ __align__(16) T s_v[kRecWarps][kColsAhead + 1][kRecTok][CG * VPT];
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
   if (n < p.long_rows) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7, cg = lane >> 3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane % KL, cg = lane / KL;
   const int groups = (n + kRecTok - 1) / kRecTok;
   float* ring = reinterpret_cast<float*>(sm8 + kRecHead);
   RecRing rr;
@@ -632,70 +773,87 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) s
     }
     return;
   }
-  const int N = p.dk, dv = p.dv, col = slice * COLS + warp * 4 * VPT + cg * VPT;
+  const int N = p.dk, dv = p.dv, col = slice * COLS + warp * CG * VPT + cg * VPT;
   float* st = p.state + ((size_t)slot * p.heads + h) * N * dv;
   const bool vec = dv % 4 == 0;
   float S[R][VPT];
-  load_state<R, VPT>(S, st, kl, col, N, dv, ctx == n, vec);
+  load_state<KL, R, VPT>(S, st, kl, col, N, dv, ctx == n, vec);
   const float D = p.D ? p.D[h] : 0.f;
-  const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + kl) * p.ld_conv + (size_t)h * dv + col;
-  float vn[VPT];
-  load_cols<T, VPT>(vn, vsrc, kl < n, col, dv, vec_v);
+  const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + (kl & 7)) * p.ld_conv + (size_t)h * dv + col;
+  auto send_group = [&](int c) {
+    send_cols<T, VPT>(&s_v[warp][c % (kColsAhead + 1)][kl & 7][cg * VPT], vsrc + (size_t)c * kRecTok * p.ld_conv,
+                      kl < kRecTok && c * kRecTok + kl < n, col, dv, vec_v);
+  };
+#pragma unroll
+  for (int c = 0; c < kColsAhead; ++c) send_group(c);
   bool ok = true;
   for (int c = 0; c < groups; ++c) {
     const int t0 = c * kRecTok, m = min(kRecTok, n - t0);
-    __syncwarp();
-    float x_own[VPT];
-#pragma unroll
-    for (int v = 0; v < VPT; ++v) s_v[warp][kl][cg * VPT + v] = x_own[v] = vn[v];
-    vsrc += (size_t)kRecTok * p.ld_conv;
-    load_cols<T, VPT>(vn, vsrc, t0 + kRecTok + kl < n, col, dv, vec_v);
+    __syncwarp();                            // the last group's columns have been read
+    send_group(c + kColsAhead);
+    wait_cols();
+    const T(*cols)[CG * VPT] = s_v[warp][c % (kColsAhead + 1)];
     ok = rr.wait_full(c);
     if (!ok) break;
     __syncwarp();
     const float* buf = ring + (c % kRecStages) * STAGE;
     float y[kRecTok][VPT];
-    auto token = [&](int j) {
+    struct Tok {
+      float b[R], c[R], x[VPT], dec;
+    };
+    auto fetch = [&](int j, Tok& o) {
       const float* s = buf + j * REC;
-      const float2 step = *reinterpret_cast<const float2*>(buf + kRecTok * REC + j * 4);      // dt, decay
-      float x[VPT];
-#pragma unroll
-      for (int v = 0; v < VPT; ++v) { x[v] = step.x * s_v[warp][j][cg * VPT + v]; y[j][v] = 0.f; }
 #pragma unroll
       for (int i4 = 0; i4 < R / 4; ++i4) {
-        const float4 b4 = *reinterpret_cast<const float4*>(s + kl * 4 + 32 * i4);
-        const float4 c4 = *reinterpret_cast<const float4*>(s + NP + kl * 4 + 32 * i4);
-        const float ba[4] = {b4.x, b4.y, b4.z, b4.w}, ca[4] = {c4.x, c4.y, c4.z, c4.w};
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-          for (int v = 0; v < VPT; ++v) {
-            float& z = S[i4 * 4 + i][v];
-            z = fmaf(z, step.y, ba[i] * x[v]);
-            y[j][v] = fmaf(z, ca[i], y[j][v]);
-          }
+        const float4 b4 = *reinterpret_cast<const float4*>(s + kl * 4 + 4 * KL * i4);
+        const float4 c4 = *reinterpret_cast<const float4*>(s + NP + kl * 4 + 4 * KL * i4);
+        o.b[i4 * 4] = b4.x; o.b[i4 * 4 + 1] = b4.y; o.b[i4 * 4 + 2] = b4.z; o.b[i4 * 4 + 3] = b4.w;
+        o.c[i4 * 4] = c4.x; o.c[i4 * 4 + 1] = c4.y; o.c[i4 * 4 + 2] = c4.z; o.c[i4 * 4 + 3] = c4.w;
       }
+      const float2 step = *reinterpret_cast<const float2*>(buf + kRecTok * REC + j * 4);      // dt, decay
+      o.dec = step.y;
+#pragma unroll
+      for (int v = 0; v < VPT; ++v) o.x[v] = step.x * rc_ld(&cols[j][cg * VPT + v]);
+    };
+    auto token = [&](int j, const Tok& k) {
+#pragma unroll
+      for (int v = 0; v < VPT; ++v) y[j][v] = 0.f;
+#pragma unroll
+      for (int i = 0; i < R; ++i)
+#pragma unroll
+        for (int v = 0; v < VPT; ++v) {
+          S[i][v] = fmaf(S[i][v], k.dec, k.b[i] * k.x[v]);
+          y[j][v] = fmaf(S[i][v], k.c[i], y[j][v]);
+        }
     };
     if (m == kRecTok) {
+      Tok tok[2];                            // the next token's operands are fetched before this one's are used
+      fetch(0, tok[0]);
 #pragma unroll
-      for (int j = 0; j < kRecTok; ++j) token(j);
+      for (int j = 0; j < kRecTok; ++j) {
+        if (j + 1 < kRecTok) fetch(j + 1, tok[(j + 1) & 1]);
+        token(j, tok[j & 1]);
+      }
     } else {
 #pragma unroll
       for (int j = 0; j < kRecTok; ++j) {
-        if (j < m) token(j);
-        else {
+        if (j < m) {
+          Tok tok;
+          fetch(j, tok);
+          token(j, tok);
+        } else {
 #pragma unroll
           for (int v = 0; v < VPT; ++v) y[j][v] = 0.f;
         }
       }
     }
     rr.release(c);
-    spread_tokens<VPT>(y, kl);
+    spread_tokens<KL, VPT>(y, kl);
 #pragma unroll
-    for (int v = 0; v < VPT; ++v) y[0][v] = fmaf(D, x_own[v], y[0][v]);
+    for (int v = 0; v < VPT; ++v) y[0][v] = fmaf(D, rc_ld(&cols[kl & 7][cg * VPT + v]), y[0][v]);
     if (kl < m) store_cols<VPT>(p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col, y[0], col, dv, vec);
   }
-  if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<R, VPT>(S, st, kl, col, N, dv, vec);
+  if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<KL, R, VPT>(S, st, kl, col, N, dv, vec);
 }
 
 // ------------------------------------------------------------------------------------------ norm over groups with a gate
@@ -811,11 +969,25 @@ __global__ void __launch_bounds__(256) group_norm_kernel(GroupNormParams p) {
   }
 }
 
-template <typename T, int R, int VPT, bool DELTA>
-static int launch_short_runs(const RecParams& p, int B, cudaStream_t s) {
-  constexpr int COLS = kRecWarps * 4 * VPT;
+// bf16: 4 neighbouring elements of the token's vectors can be read as one 64-bit word
+static int words_of_four(const RecParams& p, bool delta) {
+  auto ok = [](const void* q, long long ld) { return (reinterpret_cast<uintptr_t>(q) & 7) == 0 && ld % 4 == 0; };
+  return ok(p.conv, p.ld_conv) && p.dk % 4 == 0 && p.dv % 4 == 0 && (!delta || ok(p.a, p.ld_a));
+}
+
+template <typename T, int DKP, bool DELTA>
+static int launch_steps(const RecParams& p, int B, cudaStream_t s) {
+  constexpr int KL = DKP <= 128 ? 8 : DKP / 16, R = DKP / KL, COLS = kRecWarps * (32 / KL) * 4;
   const int slices = (p.dv + COLS - 1) / COLS;
-  const size_t smem = (size_t)2 * kRecTok * ((DELTA ? 3 : 2) * R * 8 + COLS + 4) * 4;
+  auto kern = DELTA ? delta_step_kernel<T, KL, R, 4> : state_space_step_kernel<T, KL, R, 4>;
+  kern<<<dim3(B * slices, p.heads), kRecWarps * 32, 0, s>>>(p, slices, words_of_four(p, DELTA));
+  return (int)cudaGetLastError();
+}
+template <typename T, int DKP, bool DELTA>
+static int launch_short_runs(const RecParams& p, int B, cudaStream_t s) {
+  constexpr int R = DKP / 8, VPT = R > 32 ? 1 : (sizeof(T) == 4 || R > 16 ? 2 : 4), COLS = kRecWarps * 4 * VPT;
+  const int slices = (p.dv + COLS - 1) / COLS;
+  const size_t smem = (size_t)2 * kRecTok * ((DELTA ? 3 : 2) * DKP + COLS + 4) * 4;
   auto kern = DELTA ? delta_rule_kernel<T, R, VPT> : state_space_kernel<T, R, VPT>;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(kern, 200 * 1024);
@@ -823,65 +995,67 @@ static int launch_short_runs(const RecParams& p, int B, cudaStream_t s) {
   kern<<<dim3(B * slices, p.heads), kRecWarps * 32, smem, s>>>(p, slices);
   return (int)cudaGetLastError();
 }
-template <typename T, int R, int VPT, bool DELTA>
-static int launch_long_runs(const RecParams& p, int B, cudaStream_t s) {
-  constexpr int COLS = kRecWarps * 4 * VPT;
+template <typename T, int KL, int R, int VPT, bool DELTA>
+static int launch_stream(const RecParams& p, int B, cudaStream_t s) {
+  constexpr int COLS = kRecWarps * (32 / KL) * VPT;
   const int slices = (p.dv + COLS - 1) / COLS;
-  const size_t smem = kRecHead + (size_t)kRecStages * kRecTok * ((DELTA ? 3 : 2) * R * 8 + 4) * 4;
-  auto kern = DELTA ? delta_stream_kernel<T, R, VPT> : state_space_stream_kernel<T, R, VPT>;
+  const size_t smem = kRecHead + (size_t)kRecStages * kRecTok * ((DELTA ? 3 : 2) * R * KL + 4) * 4;
+  void (*kern)(RecParams, int, int);
+  if constexpr (DELTA) kern = delta_stream_kernel<T, KL, R, VPT>;
+  else kern = state_space_stream_kernel<T, KL, R, VPT>;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(kern, 220 * 1024);
   if (e != cudaSuccess) return (int)e;
-  const long long off = DELTA ? 2LL * p.groups * p.dk : 0;             // first v (x) channel
-  const int vec_v = (reinterpret_cast<uintptr_t>(p.conv) & 7) == 0 && p.ld_conv % 4 == 0 && off % 4 == 0 && p.dv % 4 == 0;
-  kern<<<dim3(B * slices, p.heads), (kRecWarps + 1) * 32, smem, s>>>(p, slices, vec_v);
+  kern<<<dim3(B * slices, p.heads), (kRecWarps + 1) * 32, smem, s>>>(p, slices, words_of_four(p, DELTA));
   return (int)cudaGetLastError();
 }
-
-template <int R, bool DELTA>
-static long long record_floats(int T, int heads, int groups) {
-  if (DELTA) return (long long)heads * T * (3 * R * 8 + 4);
-  return (long long)groups * T * 2 * R * 8 + (long long)heads * T * 4;
+// 16 columns per warp keep the reductions and the shared-memory reads few; where that gives too few warps to fill the GPU, 4 columns
+template <typename T, int DKP, bool DELTA>
+static int launch_long_runs(const RecParams& p, int B, cudaStream_t s) {
+  if constexpr (DELTA) delta_records_kernel<T, DKP><<<(unsigned)(((long long)p.T * p.heads + 3) / 4), 128, 0, s>>>(p);
+  else state_space_records_kernel<T, DKP><<<p.T, 128, 0, s>>>(p);
+  const int e = (int)cudaGetLastError();
+  if (e) return e;
+  if constexpr (sizeof(T) == 2 && DKP <= 128)
+    if ((long long)B * p.heads * ((p.dv + 15) / 16) >= 4LL * sm_count()) return launch_stream<T, 8, DKP / 8, 4, DELTA>(p, B, s);
+  constexpr int KL = DKP >= 64 ? 16 : 8;
+  if constexpr (sizeof(T) == 2 && !DELTA && DKP <= 128)     // no reduction between tokens: 8 columns already at half the warps
+    if ((long long)B * p.heads * ((p.dv + 7) / 8) >= 2LL * sm_count()) return launch_stream<T, KL, DKP / KL, 4, DELTA>(p, B, s);
+  return launch_stream<T, KL, DKP / KL, 2, DELTA>(p, B, s);
 }
 
-// Columns per lane: 4 keeps the reductions and the shared-memory reads few; long runs with too few warps to fill the GPU take fewer.
-template <typename T, int R, bool DELTA>
-static int run_width(RecParams p, int B, int max_q, int short_runs, long long ws_bytes, cudaStream_t s) {
-  constexpr int V = R > 32 ? 1 : (sizeof(T) == 4 || R > 16 ? 2 : 4);
-  const bool stream = p.records != nullptr && max_q >= p.long_rows && p.out != nullptr;
-  if (stream) {
-    if (ws_bytes < record_floats<R, DELTA>(p.T, p.heads, p.groups) * 4 || (reinterpret_cast<uintptr_t>(p.records) & 15) || !p.seq_of_row)
-      return (int)cudaErrorInvalidValue;
-    if constexpr (DELTA) delta_records_kernel<T, R><<<(unsigned)(((long long)p.T * p.heads + 3) / 4), 128, 0, s>>>(p);
-    else state_space_records_kernel<T, R><<<p.T, 128, 0, s>>>(p);
-    int e = (int)cudaGetLastError();
-    if (e) return e;
-    const long long warps = (long long)B * p.heads * ((p.dv + 15) / 16), room = 4LL * sm_count();
-    if constexpr (V == 4) {
-      e = warps >= room ? launch_long_runs<T, R, 4, DELTA>(p, B, s) : 2 * warps >= room ? launch_long_runs<T, R, 2, DELTA>(p, B, s)
-                                                                                        : launch_long_runs<T, R, 1, DELTA>(p, B, s);
-    } else {
-      e = launch_long_runs<T, R, V, DELTA>(p, B, s);
-    }
-    if (e || !short_runs) return e;
-  } else {
-    p.long_rows = 0x7fffffff;
-  }
-  return launch_short_runs<T, R, V, DELTA>(p, B, s);
+// kinds: which sequences the step has, bit 0 = single tokens, 1 = short runs, 2 = long runs (with a workspace)
+template <typename T, int DKP, bool DELTA>
+static int run_width(RecParams p, int B, int kinds, cudaStream_t s) {
+  int e = 0;
+  if (kinds & 1) e = launch_steps<T, DKP, DELTA>(p, B, s);
+  if (!e && (kinds & 4)) e = launch_long_runs<T, DKP, DELTA>(p, B, s);
+  else p.long_rows = 0x7fffffff;
+  if (!e && (kinds & 2)) e = launch_short_runs<T, DKP, DELTA>(p, B, s);
+  return e;
+}
+
+static int padded_dk(int dk) { return dk <= 32 ? 32 : dk <= 64 ? 64 : dk <= 128 ? 128 : dk <= 256 ? 256 : 512; }
+static long long record_bytes(bool delta, long long T, int heads, int groups, int dk) {
+  const long long n = padded_dk(dk);
+  return 4 * (delta ? heads * T * (3 * n + 4) : groups * T * 2 * n + heads * T * 4);
 }
 
 template <typename T, bool DELTA>
-static int run_rec(const RecParams& p, int B, int max_q, int short_runs, long long ws_bytes, cudaStream_t s) {
+static int run_rec(const RecParams& p, int B, int kinds, long long ws_bytes, cudaStream_t s) {
   if (B == 0) return 0;
   if (B < 0 || p.heads < 1 || p.heads > 65535 || p.groups < 1 || p.heads % p.groups || p.dk < 1 || p.dk > 512 || p.dv < 1)
     return (int)cudaErrorInvalidValue;
-#define BLZ_REC(R) return run_width<T, R, DELTA>(p, B, max_q, short_runs, ws_bytes, s)
-  if (p.dk <= 32) BLZ_REC(4);
-  if (p.dk <= 64) BLZ_REC(8);
-  if (p.dk <= 128) BLZ_REC(16);
-  if (p.dk <= 256) BLZ_REC(32);
-  BLZ_REC(64);
-#undef BLZ_REC
+  if ((kinds & 4) && (!p.records || !p.out || !p.seq_of_row || p.T < 1 || ws_bytes < record_bytes(DELTA, p.T, p.heads, p.groups, p.dk) ||
+                      (reinterpret_cast<uintptr_t>(p.records) & 15)))
+    return (int)cudaErrorInvalidValue;
+  switch (padded_dk(p.dk)) {
+    case 32: return run_width<T, 32, DELTA>(p, B, kinds, s);
+    case 64: return run_width<T, 64, DELTA>(p, B, kinds, s);
+    case 128: return run_width<T, 128, DELTA>(p, B, kinds, s);
+    case 256: return run_width<T, 256, DELTA>(p, B, kinds, s);
+    default: return run_width<T, 512, DELTA>(p, B, kinds, s);
+  }
 }
 
 }  // namespace blz
@@ -891,33 +1065,32 @@ static constexpr int kLongRows = 32;
 BLZ_API int blz_rec_long_rows() { return kLongRows; }
 // Workspace bytes of a step of T rows (delta: 1 = blz_delta_rule, 0 = blz_state_space).
 BLZ_API long long blz_rec_ws_bytes(int delta, int T, int heads, int groups, int dk) {
-  const int R = dk <= 32 ? 4 : dk <= 64 ? 8 : dk <= 128 ? 16 : dk <= 256 ? 32 : 64;
-  return 4 * (delta ? (long long)heads * T * (3 * R * 8 + 4) : (long long)groups * T * 2 * R * 8 + (long long)heads * T * 4);
+  return blz::record_bytes(delta != 0, T, heads, groups, dk);
 }
 
 // Delta rule with channel decays over every sequence of the batch (see RecParams; leading dimensions in elements; conv channels
 // [q key_heads * dk | k key_heads * dk | v heads * dv]).  out fp32 [T, heads * dv] or null.  no_store: optional [B], 1 = leave the
-// state as it was.  max_q: the longest run; ws (or null: every run is taken as a short one): blz_rec_ws_bytes; short_runs: there
-// are runs below blz_rec_long_rows.  dk <= 512.
+// state as it was.  kinds: the sequences with one new token (bit 0), with up to blz_rec_long_rows (bit 1), with more (bit 2, which
+// needs out and the workspace ws of blz_rec_ws_bytes; without that bit they count as bit 1's).  dk <= 512.
 BLZ_API int blz_delta_rule(const void* conv, long long ld_conv, const void* a, long long ld_a, const void* b, long long ld_b, const float* A,
                            const float* dt_bias, float* state, float* out, const int* slots, const int* q_start, const int* ctx_len,
-                           const int* no_store, int B, int heads, int key_heads, int dk, int dv, const int* seq_of_row, int T, int max_q,
-                           int short_runs, float* ws, long long ws_bytes, int f32, cudaStream_t s) {
+                           const int* no_store, int B, int heads, int key_heads, int dk, int dv, const int* seq_of_row, int T, int kinds,
+                           float* ws, long long ws_bytes, int f32, cudaStream_t s) {
   using namespace blz;
   const RecParams p = {conv, a, b, A, dt_bias, nullptr, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_a, ld_b, heads, key_heads,
                        dk, dv, seq_of_row, ws, T, kLongRows, status_word()};
-  return f32 ? run_rec<float, true>(p, B, max_q, short_runs, ws_bytes, s) : run_rec<__nv_bfloat16, true>(p, B, max_q, short_runs, ws_bytes, s);
+  return f32 ? run_rec<float, true>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, true>(p, B, kinds, ws_bytes, s);
 }
 
 // State-space duality (conv channels [x heads * dv | B groups * N | C groups * N]); other arguments as above.  N <= 512.
 BLZ_API int blz_state_space(const void* conv, long long ld_conv, const void* dt, long long ld_dt, const float* A, const float* dt_bias,
                             const float* D, float* state, float* out, const int* slots, const int* q_start, const int* ctx_len,
-                            const int* no_store, int B, int heads, int groups, int N, int dv, const int* seq_of_row, int T, int max_q,
-                            int short_runs, float* ws, long long ws_bytes, int f32, cudaStream_t s) {
+                            const int* no_store, int B, int heads, int groups, int N, int dv, const int* seq_of_row, int T, int kinds,
+                            float* ws, long long ws_bytes, int f32, cudaStream_t s) {
   using namespace blz;
   const RecParams p = {conv, dt, nullptr, A, dt_bias, D, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_dt, 0, heads, groups,
                        N, dv, seq_of_row, ws, T, kLongRows, status_word()};
-  return f32 ? run_rec<float, false>(p, B, max_q, short_runs, ws_bytes, s) : run_rec<__nv_bfloat16, false>(p, B, max_q, short_runs, ws_bytes, s);
+  return f32 ? run_rec<float, false>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, false>(p, B, kinds, ws_bytes, s);
 }
 
 // RMS norm of each of `groups` runs of n columns of fp32 rows, with a gate (GroupNormParams), to the activation type.
