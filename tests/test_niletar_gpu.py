@@ -115,7 +115,7 @@ def test_products_with_biases_and_of_some_columns(ops, dtype):
 
 @pytest.mark.parametrize("dtype", TYPES)
 @pytest.mark.parametrize("T,groups,n,period,first", [(3, 4, 24, 96, True), (5, 7, 20, 20, False), (2, 1, 4096, 4096, True), (9, 3, 33, 33, False),
-                                                     (40, 16, 128, 128, False), (1, 2, 1000, 2000, True)])
+                                                     (40, 16, 128, 128, False), (1, 2, 1000, 2000, True), (300, 8, 256, 2048, True), (2, 3, 5000, 15000, True)])
 def test_group_norm(ops, T, groups, n, period, first, dtype):
     from blaze_b200.ops.cuda_ops import VP, _ptr
     g = torch.Generator().manual_seed(n)
