@@ -1103,7 +1103,7 @@ BLZ_API int blz_group_norm(const float* o, const void* z, long long ldz, const f
   const int vec = n % 4 == 0 && w_period % 4 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0 && (!z || ok(z, ldz)) && ok(out, ld_out);
   const GroupNormParams p = {o, z, w, out, ldz, ld_out, T, groups, n, w_period, sigmoid, gate_first, vec, eps, post};
   const long long units = (long long)T * groups;
-  const bool wide = n > 512 || (n > 128 && units < 8LL * sm_count());        // a block per group, else a warp
+  const bool wide = n > 1024 || (n > 128 && units < 8LL * sm_count());        // a block per group, else a warp
   const dim3 grid((unsigned)(wide ? units : (units + 7) / 8));
 #define BLZ_GN(TT, V) return (int)(wide ? launch_pdl(group_norm_kernel<TT, 8, V>, grid, dim3(256), 0, s, p) \
                                         : launch_pdl(group_norm_kernel<TT, 1, V>, grid, dim3(256), 0, s, p))
