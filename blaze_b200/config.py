@@ -106,6 +106,43 @@ class SoftAttnSpec:
 
 
 @dataclass
+class LatentAttnSpec:
+    """Softmax attention whose keys and values are linear maps of one cached vector per token (a normed latent of ``kv_rank``
+    numbers), beside a rotated key part that all heads share; queries come through a latent of their own."""
+    heads: int
+    dim: int                    # per head, queries and keys without rotation
+    rot_dim: int                # rotated query / key columns
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float                # of the scores
+    rot: Optional[RotarySpec] = None
+    sink: bool = False          # as in SoftAttnSpec
+    window: int = 0             # as in DiffAttnSpec
+    kv_from: Optional[int] = None          # the layer whose latents and rotated key parts this one reads instead of its own
+    maps = 1
+    kv_heads = 1                # what is cached is one key / value head of kv_rank + rot_dim columns
+
+    @property
+    def group(self) -> int:
+        return self.heads
+
+
+@dataclass
+class GatedLinearSpec:
+    """Linear attention whose forget gate, one per head and query channel, also decides what is written (HGRN2); normed per head."""
+    heads: int
+    dim: int
+    vdim: int
+    conv = 0                    # no convolution of its own
+    out_scale = 1.0
+
+    @property
+    def state(self) -> int:
+        return self.dim
+
+
+@dataclass
 class DeltaSpec:
     """Gated delta rule with one decay per head and key channel, and a gated norm per head."""
     heads: int
@@ -152,18 +189,33 @@ class GluSpec:
 
 
 @dataclass
+class PolyNormSpec:
+    """Dense feed-forward without a gate, activated by a sum of normed powers (``a N(z) + b N(z^2) + c N(z^3) + e``)."""
+    ff: int
+
+
+@dataclass
+class MoeSpec:
+    """Routed experts ``down(relu(up h)^2)`` weighted by their softmax scores, renormalised over the chosen ones, and a shared one."""
+    experts: int
+    top: int
+    ff: int                     # per expert
+    shared_ff: int = 0          # 0: no shared expert
+
+
+@dataclass
 class LayerSpec:
     """One entry of a configuration that describes its layers one by one: an attention, a recurrence, or both side by side."""
-    attn: Union[DiffAttnSpec, SoftAttnSpec, None] = None
-    mlp: Optional[GluSpec] = None          # None: the layer has no feed-forward
+    attn: Union[DiffAttnSpec, SoftAttnSpec, LatentAttnSpec, None] = None
+    mlp: Union[GluSpec, PolyNormSpec, MoeSpec, None] = None        # None: the layer has no feed-forward
     weights_of: Optional[int] = None       # the layer whose tensors this one uses (with a cache and a state of its own)
-    rec: Union[DeltaSpec, StateSpaceSpec, None] = None
+    rec: Union[DeltaSpec, StateSpaceSpec, GatedLinearSpec, None] = None
 
     @property
     def kind(self) -> str:
-        a = None if self.attn is None else "diff_attention" if self.attn.maps == 2 else "soft_attention"
-        r = None if self.rec is None else "state_space" if isinstance(self.rec, StateSpaceSpec) else "delta_rule"
-        return "+".join(k for k in (a, r) if k)
+        names = {DiffAttnSpec: "diff_attention", SoftAttnSpec: "soft_attention", LatentAttnSpec: "latent_attention", DeltaSpec: "delta_rule",
+                 StateSpaceSpec: "state_space", GatedLinearSpec: "gated_linear"}
+        return "+".join(names[type(m)] for m in (self.attn, self.rec) if m is not None)
 
 
 @dataclass
@@ -216,13 +268,14 @@ class ModelConfig:
     indexer_head_dim: int = 0
     indexer_budget: int = 0
     indexer_compress_ratio: int = 0
-    # models whose configuration lists its layers one by one, each with sizes of its own (Sevevik, Niletar); the sizes above then
-    # hold those of the first layer
+    # models whose configuration lists its layers one by one, each with sizes of its own (Sevevik, Niletar, Rapisun); the sizes above
+    # then hold those of the first layer
     layer_specs: List[LayerSpec] = field(default_factory=list)
     streams: int = 1                        # residual streams joined by learned static mixes
     residual_mult: float = 1.0              # of every sublayer's output
     embed_scale: float = 1.0
     residual_alpha: float = 1.0             # post-norm residual: x <- norm(alpha * x + sublayer)
+    input_conv: int = 0                     # taps of a causal convolution that is added to every mixer's input (0: none)
     # tokens
     eos_token_ids: List[int] = field(default_factory=list)
     bos_token_id: Optional[int] = None
@@ -302,6 +355,8 @@ class ModelConfig:
             return cls._from_sevevik(raw)
         if raw.get("architecture") == "Niletar":
             return cls._from_niletar(raw)
+        if raw.get("architecture") == "Rapisun":
+            return cls._from_rapisun(raw)
         archs = raw.get("architectures") or ["Qwen3ForCausalLM"]
         t = raw.get("text_config", raw)
         g = lambda k, d=None: t.get(k, raw.get(k, d))  # noqa: E731
@@ -439,6 +494,31 @@ class ModelConfig:
                              torch_dtype=str(raw.get("torch_dtype", "bfloat16")))
 
     @classmethod
+    def _from_rapisun(cls, raw: Dict[str, Any]) -> "ModelConfig":
+        """The layer-by-layer configuration of the Rapisun design."""
+        specs: List[LayerSpec] = []
+        for i, e in enumerate(raw["layers"]):
+            m, attn, rec = e["mixer"], None, None
+            if e["type"] == "hgrn2":
+                rec = GatedLinearSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]))
+            elif e["type"] == "latent_attention":
+                src = m.get("kv_from")
+                attn = LatentAttnSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
+                                      q_rank=int(m["q_rank"]), kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), rot=_rotary(m.get("rot")),
+                                      sink=True, window=int((m.get("mask") or {}).get("size") or 0), kv_from=None if src is None else int(src))
+                if attn.rot is not None:
+                    attn.rot.interleaved = False
+            else:
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+            specs.append(LayerSpec(attn, _norm_or_moe(i, e), None, rec))
+        _check_layers(specs)
+        taps = int((raw.get("canon") or {}).get("taps") or 0)
+        if taps < 0:
+            raise ValueError(f"an input convolution of {taps} taps")
+        return cls.of_layers(specs, architecture="Rapisun", model_type="rapisun", vocab_size=int(raw["vocab"]), hidden_size=int(raw["width"]),
+                             rms_norm_eps=float(raw["norm"]["eps"]), input_conv=taps, torch_dtype=str(raw.get("torch_dtype", "bfloat16")))
+
+    @classmethod
     def of_layers(cls, specs: List[LayerSpec], **kw) -> "ModelConfig":
         """A configuration from its layer list; the model-wide sizes that other parts read are those of the first layer."""
         a = next((s.attn for s in specs if s.attn is not None), None)
@@ -462,6 +542,19 @@ def _dense_mlp(i: int, entry: Dict[str, Any], limit: bool) -> Optional[GluSpec]:
     return GluSpec(ff=int(m["ff"]), limit=float(m["limit"]) if limit else None)
 
 
+def _norm_or_moe(i: int, entry: Dict[str, Any]) -> Union[PolyNormSpec, MoeSpec, None]:
+    m = entry.get("mlp")
+    if m is None:
+        return None
+    if m.get("kind") == "dense":
+        return PolyNormSpec(ff=int(m["ff"]))
+    if m.get("kind") != "moe":
+        raise ValueError(f"layer {i}: unknown feed-forward {m.get('kind')!r}")
+    shared = m.get("shared")
+    return MoeSpec(experts=int(m["router"]["experts"]), top=int(m["router"]["top"]), ff=int(m["expert"]["ff"]),
+                   shared_ff=int(shared["ff"]) if shared else 0)
+
+
 def _rotary(rot: Optional[Dict[str, Any]]) -> Optional[RotarySpec]:
     if not rot:
         return None
@@ -482,15 +575,27 @@ def _check_layers(specs: List[LayerSpec]) -> None:
                 raise ValueError(f"layer {i}: {a.heads} query heads over {a.kv_heads} key/value heads of {a.dim} / {a.vdim}")
             if a.window < 0:
                 raise ValueError(f"layer {i}: a window of {a.window}")
-            rot = getattr(a, "rot", None)
-            if rot is not None and (rot.dims % 2 or not 0 <= rot.dims <= a.dim):
-                raise ValueError(f"layer {i}: rotary positions on {rot.dims} of {a.dim} dimensions")
+            rot, turned = getattr(a, "rot", None), a.rot_dim if isinstance(a, LatentAttnSpec) else a.dim
+            if rot is not None and (rot.dims % 2 or not 0 <= rot.dims <= turned):
+                raise ValueError(f"layer {i}: rotary positions on {rot.dims} of {turned} dimensions")
+            if isinstance(a, LatentAttnSpec):
+                if min(a.rot_dim, a.q_rank, a.kv_rank) < 1:
+                    raise ValueError(f"layer {i}: latents of {a.q_rank} / {a.kv_rank} and a rotated part of {a.rot_dim} columns")
+                if a.kv_from is not None:
+                    src = specs[a.kv_from].attn if 0 <= a.kv_from < i else None
+                    if not isinstance(src, LatentAttnSpec) or src.kv_from is not None:
+                        raise ValueError(f"layer {i} reads the latents of layer {a.kv_from}, which has none of its own before it")
+                    if (src.kv_rank, src.rot_dim, src.rot) != (a.kv_rank, a.rot_dim, a.rot):
+                        raise ValueError(f"layer {i} reads latents of layer {a.kv_from} that have another size or rotation")
         if r is not None:
-            groups = r.groups if isinstance(r, StateSpaceSpec) else r.kv_heads
-            if min(r.heads, groups, r.state, r.vdim, r.conv) < 1 or r.heads % groups:
+            groups = r.groups if isinstance(r, StateSpaceSpec) else r.kv_heads if isinstance(r, DeltaSpec) else r.heads
+            taps = r.conv if not isinstance(r, GatedLinearSpec) else 1
+            if min(r.heads, groups, r.state, r.vdim, taps) < 1 or r.heads % groups:
                 raise ValueError(f"layer {i}: {r.heads} recurrent heads over {groups} groups, state {r.state} x {r.vdim}, {r.conv} taps")
             if isinstance(r, StateSpaceSpec) and (r.norm_groups < 1 or r.inner % r.norm_groups):
                 raise ValueError(f"layer {i}: {r.inner} columns in {r.norm_groups} norm groups")
+        if isinstance(s.mlp, MoeSpec) and (not 1 <= s.mlp.top <= s.mlp.experts or s.mlp.ff < 1):
+            raise ValueError(f"layer {i}: {s.mlp.top} of {s.mlp.experts} experts of {s.mlp.ff}")
         if s.weights_of is not None:
             src = specs[s.weights_of] if 0 <= s.weights_of < len(specs) else None
             if src is None or src.weights_of is not None:
@@ -568,6 +673,14 @@ def named_config(name: str) -> ModelConfig:
         layers = [LayerSpec(a, GluSpec(320), None, d), LayerSpec(None, None, None, mamba()), LayerSpec(a, GluSpec(320), 0, d)]
         return ModelConfig.of_layers(layers, architecture="Niletar", model_type="niletar", vocab_size=1024, hidden_size=192,
                                      zero_centered_norm=True, residual_alpha=1.8)
+    elif n in ("tiny-rapisun",):
+        # the Rapisun layer kinds in miniature: both mixers, both feed-forwards and none, latents read by a later layer
+        def latent(**kw):
+            return LatentAttnSpec(**{**dict(heads=4, dim=24, rot_dim=16, vdim=40, q_rank=48, kv_rank=64, scale=0.16,
+                                            rot=RotarySpec(16, 1.0e4, False), sink=True, window=40), **kw})
+        layers = [LayerSpec(None, PolyNormSpec(320), None, GatedLinearSpec(4, 32, 48)), LayerSpec(latent(), MoeSpec(8, 2, 64, 96)),
+                  LayerSpec(latent(heads=6, window=24, kv_from=1)), LayerSpec(None, MoeSpec(8, 2, 64), None, GatedLinearSpec(2, 48, 32))]
+        return ModelConfig.of_layers(layers, architecture="Rapisun", model_type="rapisun", vocab_size=1024, hidden_size=192, input_conv=4)
     elif n in ("qwen3-8b",):
         c = ModelConfig(vocab_size=151936, hidden_size=4096, num_layers=36, num_heads=32, num_kv_heads=8,
                         head_dim=128, intermediate_size=12288, rope=RopeConfig(theta=1e6))

@@ -15,8 +15,13 @@ Pages hold 16 tokens.  Two pool layouts exist:
   in a row is what ``ldmatrix`` and the tensor core's unswizzled operands both take.  The ``logical`` form of such a layer is
   ``k [pages, maps * kv_heads, 16, dim]`` (two maps: key head g's at 2g and 2g + 1) and ``v [pages, kv_heads, 16, vdim]``.
 
+  A latent attention caches one vector per token, ``[latent | rotated key part]`` (each padded to 16), which is key and value at
+  once: a page block is one such part of ``pad16(kv_rank) + pad16(rot_dim)`` columns.  Its ``logical`` form is ``k [pages, 1, 16,
+  kv_rank]`` (the latents) and ``v [pages, 1, 16, rot_dim]``.  A layer that reads another's latents has no pages of its own.
+
 Recurrent layers (Gated DeltaNet, and the recurrences of a layer-by-layer configuration) keep one state row per sequence row: the
-last inputs of their convolution in the activation type and the recurrent state in fp32, of each layer's own sizes.
+last inputs of their convolution in the activation type and the recurrent state in fp32, of each layer's own sizes.  A
+configuration whose mixers' inputs are convolved (``input_conv``) keeps the last inputs of every layer there too, in fp32.
 
 The reference keeps one-token pages and several KV dtypes (``crates/blaze/src/model.rs:499-583``,
 ``alloc_kv`` :517); its page bookkeeping is in ``engine.rs:1083-1164``.
@@ -30,7 +35,7 @@ from typing import Tuple, Sequence, Dict, List, Optional
 import numpy as np
 import torch
 
-from .config import ModelConfig
+from .config import LatentAttnSpec, ModelConfig
 
 PAGE = 16
 
@@ -41,12 +46,14 @@ def pad16(n: int) -> int:
 
 def page_elems(spec) -> int:
     """Elements of one (page, key/value head) block of the ``tiles`` layout."""
+    if isinstance(spec, LatentAttnSpec):
+        return PAGE * (pad16(spec.kv_rank) + pad16(spec.rot_dim))
     return PAGE * (spec.maps * pad16(spec.dim) + pad16(spec.vdim))
 
 
 def kv_bytes_per_token(cfg: ModelConfig, kv_dtype: str, tp_world: int = 1) -> int:
     if cfg.layer_specs:
-        attn = [s.attn for s in cfg.layer_specs if s.attn is not None]
+        attn = [s.attn for s in cfg.layer_specs if s.attn is not None and getattr(s.attn, "kv_from", None) is None]
         return sum(a.kv_heads * page_elems(a) for a in attn) // PAGE * (4 if kv_dtype == "fp32" else 2)
     n_attn = sum(1 for i in range(cfg.num_layers) if cfg.layer_type(i) == "full_attention")
     kvh = max(cfg.num_kv_heads // tp_world, 1)
@@ -99,8 +106,16 @@ class KVCache:
                 raise ValueError(f"{cfg.architecture} keeps its keys and values in bf16 or fp32, not {kv_dtype}")
             if a is None:
                 continue
-            if layout == "tiles":
+            src = getattr(a, "kv_from", None)
+            if src is not None:
+                for d in (self.kv, self.k, self.v):
+                    if src in d:
+                        d[i] = d[src]
+            elif layout == "tiles":
                 self.kv[i] = torch.zeros(num_pages, a.kv_heads, page_elems(a), dtype=tdt, device=device)
+            elif isinstance(a, LatentAttnSpec):
+                self.k[i] = torch.zeros(num_pages, 1, PAGE, a.kv_rank, dtype=tdt, device=device)
+                self.v[i] = torch.zeros(num_pages, 1, PAGE, a.rot_dim, dtype=tdt, device=device)
             else:
                 self.k[i] = torch.zeros(num_pages, a.maps * a.kv_heads, PAGE, a.dim, dtype=tdt, device=device)
                 self.v[i] = torch.zeros(num_pages, a.kv_heads, PAGE, a.vdim, dtype=tdt, device=device)
@@ -137,9 +152,14 @@ class KVCache:
 
         rec = {i: cfg.layer_specs[i].rec for i in (range(lo, hi) if cfg.layer_specs else ()) if cfg.layer_specs[i].rec is not None}
         for i, r in rec.items():
-            self.conv_state[i] = torch.zeros(self.state_rows, r.conv_dim, r.conv - 1, dtype=tdt, device=device)
+            if r.conv:
+                self.conv_state[i] = torch.zeros(self.state_rows, r.conv_dim, r.conv - 1, dtype=tdt, device=device)
             self.rec_state[i] = torch.zeros(self.state_rows, r.heads, r.state, r.vdim, dtype=torch.float32, device=device)
-        self.state_layers = self.gdn_layers + list(rec)     # every layer with a recurrent state
+        self.input_state: Dict[int, torch.Tensor] = {}      # last inputs of the mixers, where those are convolved
+        if cfg.input_conv > 1:
+            for i in range(lo, hi):
+                self.input_state[i] = torch.zeros(self.state_rows, cfg.input_conv - 1, cfg.hidden_size, dtype=torch.float32, device=device)
+        self.state_layers = sorted({*self.gdn_layers, *rec, *self.input_state})       # every layer with a state row
 
         # sparse-attention indexer: the raw index key of every token, paged like K and V (shared prefixes share them)
         self.idx_k: Dict[int, torch.Tensor] = {}
@@ -194,23 +214,23 @@ class KVCache:
 
     def nbytes(self) -> int:
         n = 0
-        for d in (self.k, self.v, self.kv, self.conv_state, self.rec_state, self.idx_k):
-            n += sum(t.numel() * t.element_size() for t in d.values())
+        for d in (self.k, self.v, self.kv, self.conv_state, self.rec_state, self.input_state, self.idx_k):
+            n += sum(t.numel() * t.element_size() for t in {id(t): t for t in d.values()}.values())      # layers may share pages
         return n + (self.ple.nbytes() if self.ple is not None else 0)
 
     # ------------------------------------------------------------------ recurrent state rows
     def copy_state(self, src: int, dst: int) -> None:
         """Copy the conv + recurrent state of row ``src`` to row ``dst`` (``model.rs:2718``)."""
-        for i in self.state_layers:
-            self.conv_state[i][dst].copy_(self.conv_state[i][src])
-            self.rec_state[i][dst].copy_(self.rec_state[i][src])
+        for d in (self.conv_state, self.rec_state, self.input_state):
+            for t in d.values():
+                t[dst].copy_(t[src])
         if self.ple is not None:
             self.ple.copy(src, dst)
 
     def zero_state(self, row: int) -> None:
-        for i in self.state_layers:
-            self.conv_state[i][row].zero_()
-            self.rec_state[i][row].zero_()
+        for d in (self.conv_state, self.rec_state, self.input_state):
+            for t in d.values():
+                t[row].zero_()
         if self.ple is not None:
             self.ple.zero(row)
 

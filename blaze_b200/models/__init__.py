@@ -10,5 +10,8 @@ def model_class(cfg):
     if cfg.architecture == "Niletar":
         from .niletar import Niletar
         return Niletar
+    if cfg.architecture == "Rapisun":
+        from .rapisun import Rapisun
+        return Rapisun
     from .qwen3 import Model
     return Model

@@ -71,13 +71,44 @@ class SoftAttn:
         self.sink = None if sink is None else sink.to(device, torch.float32).contiguous()
         self.freq = None
         if spec.rot is not None:
-            f = torch.tensor(spec.rot.frequencies(), dtype=torch.float64)
-            self.freq = torch.stack([f.float(), (f - f.float().double()).float()]).to(device)
+            self.freq = _two_floats(spec.rot.frequencies(), device)
+
+
+class LatentAttn:
+    """Attention of a :class:`Mixer` over cached latents (config.LatentAttnSpec).  The input projection gives the queries' latent
+    (normed by ``q_norm``, then ``uq``) and, unless the layer reads another's, the keys' latent (``c_norm``) and rotated part.
+    ``uk [heads, dim, kv_rank]`` and ``uv [heads, vdim, kv_rank]`` make a head's keys and values out of a latent."""
+
+    def __init__(self, spec, device):
+        self.spec = spec
+        self.uq: Linear = None
+        self.q_norm: torch.Tensor = None
+        self.c_norm: Optional[torch.Tensor] = None
+        self.uk: torch.Tensor = None
+        self.uv: torch.Tensor = None
+        self.expand: Linear = None       # rows [uk | uv], one product for the keys and values of a run of latents
+        self.uk_t: torch.Tensor = None   # uk as [heads, kv_rank, dim]
+        self.sink: Optional[torch.Tensor] = None
+        self.freq = None if spec.rot is None else _two_floats(spec.rot.frequencies(), device)
+
+    def set_maps(self, uk: torch.Tensor, uv: torch.Tensor, dtype) -> None:
+        a = self.spec
+        self.expand = Linear.from_dense(torch.cat([uk, uv]).to(dtype), dtype=dtype)
+        self.uk = self.expand.w[:uk.shape[0]].view(a.heads, a.dim, a.kv_rank)
+        self.uv = self.expand.w[uk.shape[0]:].view(a.heads, a.vdim, a.kv_rank)
+        self.uk_t = self.uk.transpose(1, 2).contiguous()
+
+
+def _two_floats(f, device) -> torch.Tensor:
+    """``[2, n]`` fp32: numbers, and what rounding them to 32 bits left over."""
+    f = torch.tensor(f, dtype=torch.float64)
+    return torch.stack([f.float(), (f - f.float().double()).float()]).to(device)
 
 
 class Recurrence:
-    """Recurrent part of a :class:`Mixer`, ``kind`` "delta" (config.DeltaSpec) or "ssm" (config.StateSpaceSpec).  ``A`` is the positive
-    decay rate; decay, step and norm weights are fp32.  ``low`` (delta): from the low-rank inputs to [decay inputs | norm gates]."""
+    """Recurrent part of a :class:`Mixer`, ``kind`` "delta" (config.DeltaSpec), "ssm" (config.StateSpaceSpec) or "gated"
+    (config.GatedLinearSpec).  ``A`` is the positive decay rate, or (gated) the lower bound of the forget gates, whose bias is
+    ``dt_bias``; decay, step and norm weights are fp32.  ``low`` (delta): from the low-rank inputs to [decay inputs | norm gates]."""
 
     def __init__(self, spec, kind: str, norm_groups: int):
         self.spec, self.kind, self.norm_groups = spec, kind, norm_groups
@@ -96,11 +127,12 @@ class Mixer:
         self.o: Linear = None
         self.cols: Dict[str, int] = {}
         self.low_width = 0               # columns of the low-rank inputs
-        self.attn: Optional[SoftAttn] = None
+        self.attn: Optional[SoftAttn] = None             # or a LatentAttn
         self.rec: Optional[Recurrence] = None
 
     def linears(self) -> List[Linear]:
-        return [l for l in (self.in_proj, self.o, self.rec.low if self.rec is not None else None) if l is not None]
+        latent = [self.attn.uq, self.attn.expand] if isinstance(self.attn, LatentAttn) else []
+        return [l for l in (self.in_proj, self.o, self.rec.low if self.rec is not None else None, *latent) if l is not None]
 
 
 class DenseMlp:
@@ -118,8 +150,20 @@ class ClampedGlu:
         self.limit = limit
 
 
+class PlainMlp:
+    """Dense feed-forward without a gate: ``down(act(up x))``, act the squared ReLU, or (``poly``: its four numbers)
+    the sum of normed powers."""
+
+    def __init__(self, poly: Optional[torch.Tensor] = None):
+        self.up: Linear = None
+        self.down: Linear = None
+        self.poly = poly
+
+
 class Experts:
     """Routed experts of one layer (this rank's share under expert parallelism)."""
+
+    act = "swiglu"                       # or "relu2": no gate, ``gate_up`` holds the up projections alone
 
     def __init__(self):
         self.gate_up: List[Linear] = []
@@ -132,14 +176,16 @@ class Experts:
     def forward_one(self, e: int, x: torch.Tensor) -> torch.Tensor:
         from ..ops import ref
         le = e - self.first
-        return self.down[le].ref(ref.silu_mul(self.gate_up[le].ref(x)))
+        up = self.gate_up[le].ref(x)
+        return self.down[le].ref(ref.silu_mul(up) if self.act == "swiglu" else ref.relu2(up))
 
 
 class MoeMlp:
     def __init__(self):
         self.router: Linear = None
         self.experts: Experts = None
-        self.shared: Optional[DenseMlp] = None
+        self.shared: Optional[DenseMlp] = None           # or a PlainMlp
+        self.rows_out = False            # the result stays as routed rows: the residual op that follows sums them up
         self.shared_gate: Optional[Linear] = None
         self.top_k = 0
         self.renorm = True
@@ -159,6 +205,7 @@ class Layer:
         # post-norm designs: the mixers as one object, and the norms of the sums after them and after the feed-forward
         self.mixer: Optional[Mixer] = None
         self.mixer_norm = self.mlp_norm = None
+        self.in_conv: Optional[torch.Tensor] = None      # [taps, hidden] fp32: convolution added to the mixer's input
 
 
 _PROFILE_PHASES = os.environ.get("BLAZE_PROFILE_PHASES", "0") == "1"
@@ -255,6 +302,7 @@ class Model:
         self.capture_layers: List[int] = []                   # hidden states kept for drafters
         self.captured: Dict[int, torch.Tensor] = {}
         self.gdn_records: Dict[int, tuple] = {}               # per GDN layer: inputs of the last step that deferred state
+        self.conv_records: Dict[int, torch.Tensor] = {}       # per layer with an input convolution: the same
         self.ple_records: Dict = {}                           # per n-gram embedding layer: the same for its convolution
         self.hc_final = None                                  # hyper-connection that reads the streams out (last stage)
         if cfg.has_hc and (self.tp.world > 1 or first_layer != 0 or self.last_layer != cfg.num_layers):
@@ -760,7 +808,9 @@ class Model:
         proj = ops.linear(M.in_proj, h)
         n_attn = M.attn.spec.heads * M.attn.spec.vdim if M.attn is not None else 0
         y = torch.empty(proj.shape[0], M.o.K, dtype=proj.dtype, device=proj.device)
-        if M.attn is not None:
+        if isinstance(M.attn, LatentAttn):
+            ops.latent_attention(proj, M, batch, kv, gi, eps, y[:, :n_attn])
+        elif M.attn is not None:
             ops.soft_attention(proj, M, batch, kv, gi, eps, y[:, :n_attn])
         if M.rec is not None:
             low = ops.linear(M.rec.low, proj[:, M.cols["low"]:M.cols["low"] + M.low_width]) if M.rec.low is not None else None
@@ -791,6 +841,8 @@ class Model:
         idx = rows.long()
         for li, L in enumerate(self.layers):
             gi = self.first_layer + li
+            if gi in self.conv_records:
+                self.ops.input_conv(self.conv_records[gi][idx].contiguous(), L.in_conv, batch, kv, gi, self.dtype, state_only=True)
             if L.gdn is None and (L.mixer is None or L.mixer.rec is None):
                 continue
             rec = self.gdn_records.get(gi)
@@ -827,6 +879,9 @@ class Model:
         tp = self.tp.world > 1
         if isinstance(M, ClampedGlu):
             return ops.linear(M.down, ops.linear_glu(M.gate_up, h, M.limit)), "full"
+        if isinstance(M, PlainMlp):
+            a = ops.linear_relu2(M.up, h) if M.poly is None else ops.poly_norm(ops.linear(M.up, h), M.poly, self.cfg.rms_norm_eps)
+            return ops.linear(M.down, a), "full"
         if isinstance(M, DenseMlp):
             a = ops.linear_swiglu(M.gate_up, h, quant_for=M.down)
             return self._row_cut(M.down, a, a.rows if hasattr(a, "rows") else a.shape[0], fused)
@@ -845,6 +900,8 @@ class Model:
                 self.heat.observe(layer, ids)
         # Tokens are replicated across the ranks, so expert parallelism needs no dispatch: every rank runs the routed
         # pairs whose expert it holds and the partial outputs are summed by the reduce + norm that follows.
+        if M.rows_out:
+            return ops.moe_rows(hd, w, ids, M.experts, self._mlp(M.shared, hd)[0] if M.shared is not None else None), "full"
         y = ops.moe(hd, w, ids, M.experts)
         routed_partial = tp
         if M.shared is not None:
@@ -903,8 +960,8 @@ class Model:
                 for v in vars(obj).values():
                     if isinstance(v, Linear):
                         n += v.nbytes()
-                    elif isinstance(v, DenseMlp):
-                        n += v.gate_up.nbytes() + v.down.nbytes()
+                    elif isinstance(v, (DenseMlp, PlainMlp)):
+                        n += (v.gate_up if isinstance(v, DenseMlp) else v.up).nbytes() + v.down.nbytes()
                     elif isinstance(v, Experts):
                         n += sum(l.nbytes() for l in v.gate_up) + sum(l.nbytes() for l in v.down)
         if self.lm_head is not None:

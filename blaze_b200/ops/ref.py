@@ -235,6 +235,17 @@ def clamped_glu(gu: torch.Tensor, limit: float) -> torch.Tensor:
     return g * torch.sigmoid(1.702 * g) * (u + 1)
 
 
+def relu2(z: torch.Tensor) -> torch.Tensor:
+    return z.float().clamp(min=0).square().to(z.dtype)
+
+
+def poly_norm(z: torch.Tensor, act: torch.Tensor, eps: float) -> torch.Tensor:
+    """``a N(z) + b N(z^2) + c N(z^3) + e``, N dividing a row by its root mean square; ``act`` holds a, b, c, e.  fp32."""
+    z = z.float()
+    n = lambda x: x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)      # noqa: E731
+    return act[0] * n(z) + act[1] * n(z * z) + act[2] * n(z * z * z) + act[3]
+
+
 def silu_mul(gu: torch.Tensor) -> torch.Tensor:
     """``[T, 2I]`` laid out as ``[gate | up]`` → ``silu(gate) * up`` in the input dtype."""
     I = gu.shape[-1] // 2
@@ -388,10 +399,34 @@ def state_space(x, B, C, dt, A, dt_bias, D, state):
     return out, S
 
 
+def gated_linear(q, f, v, lower, bias, state):
+    """Linear attention whose forget gates also decide what is written, one sequence: q and the gates' inputs f ``[T, H, dk]`` before
+    their activations, v ``[T, H, dv]``, lower bounds and biases ``[H * dk]``, state ``[H, dk, dv]``.  fp32."""
+    T, H, dk = q.shape
+    lo = lower.view(1, H, dk)
+    z = f.float() + bias.view(1, H, dk)
+    keep, write = lo + (1 - lo) * torch.sigmoid(z), (1 - lo) * torch.sigmoid(-z)
+    q, v, S = F.silu(q.float()), v.float(), state.clone()
+    out = torch.empty(T, H, v.shape[2], device=q.device)
+    for t in range(T):
+        S = S * keep[t].unsqueeze(-1) + write[t].unsqueeze(-1) * v[t].unsqueeze(1)
+        out[t] = torch.einsum("hkv,hk->hv", S, q[t])
+    return out, S
+
+
+def input_conv(x, state, w):
+    """``x + conv(x)`` over one sequence, ``x [T, C]`` fp32, ``w [taps, C]``, ``state [taps - 1, C]`` the inputs before; (y, new state)."""
+    hist = torch.cat([state, x])
+    y = x.clone()
+    for j in range(w.shape[0]):
+        y += hist[j:j + x.shape[0]] * w[j]
+    return y, hist[x.shape[0]:]
+
+
 def group_norm(o, z, w, groups: int, eps: float, sigmoid: bool, gate_first: bool, post: float = 1.0):
-    """RMS norm of each of ``groups`` equal parts of fp32 rows ``[T, C]`` with a gate (``silu(z)`` or ``sigmoid(z)``) before or after
-    it and a weight that repeats over the columns.  fp32."""
-    gate = torch.sigmoid(z.float()) if sigmoid else F.silu(z.float())
+    """RMS norm of each of ``groups`` equal parts of fp32 rows ``[T, C]`` with a gate (``silu(z)`` or ``sigmoid(z)``; z None: none)
+    before or after it and a weight that repeats over the columns.  fp32."""
+    gate = torch.ones_like(o) if z is None else torch.sigmoid(z.float()) if sigmoid else F.silu(z.float())
     x = o * gate if gate_first else o
     x = x.view(x.shape[0], groups, -1)
     x = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)).flatten(1) * w.repeat(o.shape[1] // w.numel())

@@ -97,8 +97,11 @@ class RefOps:
     def streams_sum(self, src, y, prev):
         return (ref.streams_write(src, prev.mix, prev.out, y) if y is not None else src).sum(1)
 
-    def norm_rows(self, x, rows, w, eps, dtype):
+    def norm_rows(self, x, rows, w, eps, dtype, centre: bool = False):
+        """RMS norm (``centre``: layer norm) of fp32 rows, those named by ``rows``, to ``dtype``."""
         x = x if rows is None else x[rows.long()]
+        if centre:
+            x = x - x.mean(-1, keepdim=True)
         return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w).to(dtype)
 
     def diff_attention(self, qkv, A, batch, kv, layer_idx, eps):
@@ -139,18 +142,25 @@ class RefOps:
         """The recurrent mixer of a layer, one sequence at a time.  Sequences flagged in ``batch.h_gdn_defer`` leave their state
         untouched; ``state_only`` advances the states and writes nothing."""
         R, r = M.rec, M.rec.spec
-        conv_state, rec_state, defer = kv.conv_state[layer_idx], kv.rec_state[layer_idx], getattr(batch, "h_gdn_defer", None)
-        C, dt, H, dv = r.conv_dim, proj.dtype, r.heads, r.vdim
+        conv_state, rec_state, defer = kv.conv_state.get(layer_idx), kv.rec_state[layer_idx], getattr(batch, "h_gdn_defer", None)
+        gated = R.kind == "gated"
+        dt, H, dv = proj.dtype, r.heads, r.vdim
         for b, slot in enumerate(batch.h_slots):
             r0, r1 = batch.h_q_start[b], batch.h_q_start[b + 1]
             n = r1 - r0
             if n <= 0:
                 continue
             if batch.h_ctx_len[b] == n:
-                conv_state[slot].zero_()
+                if not gated:
+                    conv_state[slot].zero_()
                 rec_state[slot].zero_()
-            y, cs = ref.gdn_conv(proj[r0:r1, M.cols["conv"]:][:, :C], conv_state[slot], R.conv_w, R.conv_b, round_sum=False)
-            if R.kind == "delta":
+            if not gated:
+                y, cs = ref.gdn_conv(proj[r0:r1, M.cols["conv"]:][:, :r.conv_dim], conv_state[slot], R.conv_w, R.conv_b, round_sum=False)
+            z = None
+            if gated:
+                cols = {c: proj[r0:r1, M.cols[c]:][:, :H * d].reshape(n, H, d) for c, d in (("q", r.dim), ("f", r.dim), ("v", dv))}
+                o, S = ref.gated_linear(cols["q"], cols["f"], cols["v"], R.A, R.dt_bias, rec_state[slot])
+            elif R.kind == "delta":
                 nk, hd = r.kv_heads * r.dim, H * r.dim
                 o, S = ref.delta_rule(y[:, :nk].view(n, -1, r.dim), y[:, nk:2 * nk].view(n, -1, r.dim), y[:, 2 * nk:].view(n, H, dv),
                                       low[r0:r1, :hd].reshape(n, H, r.dim), proj[r0:r1, M.cols["beta"]:][:, :H], R.A, R.dt_bias, rec_state[slot])
@@ -162,11 +172,67 @@ class RefOps:
                                        rec_state[slot])
                 z = proj[r0:r1, M.cols["z"]:][:, :r.inner]
             if not (defer is not None and defer[b]):
-                conv_state[slot].copy_(cs)
+                if not gated:
+                    conv_state[slot].copy_(cs)
                 rec_state[slot].copy_(S)
             if not state_only:
                 out[r0:r1] = ref.group_norm(o.reshape(n, -1), z, R.norm_w, R.norm_groups, eps, R.kind == "delta", R.kind != "delta",
                                             r.out_scale).to(dt)
+
+    # -------------------------------------------------------------- residual with normed branches, input convolution, latent attention
+    def embed_norm(self, table, tokens, w, eps):
+        """Layer-normed embedding rows, fp32."""
+        return self.norm_rows(table[tokens.long()].float(), None, w, eps, torch.float32, centre=True)
+
+    def branch_norm(self, x, y, w, eps, copy: bool = True):
+        """(fp32 ``x + layer_norm(y)``, the same in y's type or None)."""
+        x = x + self.norm_rows(y.float(), None, w, eps, torch.float32, centre=True)
+        return x, x.to(y.dtype) if copy else None
+
+    def input_conv(self, x, w, batch, kv, layer_idx, dtype, state_only: bool = False):
+        """``x + conv(x)`` of fp32 rows in ``dtype``, with the inputs before each sequence's rows from its state row, which advances
+        (not for sequences flagged in ``batch.h_gdn_defer``)."""
+        out, state = torch.empty(x.shape, dtype=dtype, device=x.device), kv.input_state.get(layer_idx)
+        defer = getattr(batch, "h_gdn_defer", None)
+        for b, slot in enumerate(batch.h_slots):
+            r0, r1 = batch.h_q_start[b], batch.h_q_start[b + 1]
+            if r1 <= r0:
+                continue
+            fresh = batch.h_ctx_len[b] == r1 - r0
+            before = x.new_zeros(w.shape[0] - 1, x.shape[1]) if state is None or fresh else state[slot]
+            y, after = ref.input_conv(x[r0:r1], before, w)
+            out[r0:r1] = y.to(dtype)
+            if state is not None and not (defer is not None and defer[b]):
+                state[slot].copy_(after)
+        return None if state_only else out
+
+    def linear_relu2(self, lin: Linear, x):
+        return ref.relu2(self.linear(lin, x))
+
+    def poly_norm(self, z, act, eps):
+        return ref.poly_norm(z, act, eps).to(z.dtype)
+
+    def latent_attention(self, proj, M, batch, kv, layer_idx, eps, out):
+        """Latent attention of a mixer: its own latents go to their pages, heads' outputs (before the output projection) to ``out``."""
+        A, a, T, dt = M.attn, M.attn.spec, proj.shape[0], proj.dtype
+        turn = lambda x: x.float() if A.freq is None else ref.rotate_heads(x, batch.positions, A.freq.double().sum(0), False)   # noqa: E731
+        if a.kv_from is None:
+            c = self.norm_rows(proj[:, M.cols["kv"]:][:, :a.kv_rank].float(), None, A.c_norm, eps, dt)
+            kr = turn(proj[:, M.cols["kv"] + a.kv_rank:][:, :a.rot_dim].reshape(T, 1, -1))
+            valid = batch.slot_mapping >= 0
+            ref.kv_write(kv.k[layer_idx], kv.v[layer_idx], c[valid][:, None], kr[valid], batch.slot_mapping[valid])
+        q = self.linear(A.uq, self.norm_rows(proj[:, M.cols["q"]:][:, :a.q_rank].float(), None, A.q_norm, eps, dt)).view(T, a.heads, -1)
+        # keys and values by head: the score of a latent is (uk^T q) . c, the output uv (sum of weighted latents)
+        ql = torch.einsum("thd,hdr->thr", q[..., :a.dim].float(), A.uk.float())
+        q = torch.cat([ql, turn(q[..., a.dim:])], -1)
+        keys = torch.cat([kv.k[layer_idx], kv.v[layer_idx]], -1)
+        o = ref.paged_attention(q, keys, kv.k[layer_idx], kv.block_table, batch.h_slots, batch.h_q_start, batch.h_ctx_len, a.scale,
+                                window=a.window, sink=A.sink)
+        out.copy_(torch.einsum("thr,her->the", o.float(), A.uv.float()).reshape(T, -1))
+
+    def moe_rows(self, x, topk_w, topk_id, experts, shared=None):
+        y = self.moe(x, topk_w, topk_id, experts)
+        return y if shared is None else self.add(y, shared)
 
     # -------------------------------------------------------------- MoE
     def router_topk(self, logits, k, renorm=True):
