@@ -70,6 +70,7 @@ class StepBatch:
     max_q_len: int = 1
     max_ctx: int = 0
     h2d_bytes: int = 0
+    visible: dict = field(default_factory=dict)       # page lists that the layers of one step share (CudaOps._visible_pages)
 
     @property
     def num_seqs(self) -> int:

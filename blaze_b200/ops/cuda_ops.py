@@ -48,6 +48,14 @@ class _Symbols:
             return self._Missing()
 
 
+class RoutedRows:
+    """What routed experts leave behind: ``rows`` in the padded row space, the ``row_map [T, k]`` of each token's rows with their
+    ``weights``, and rows that are added to the sums (``extra``, may be None)."""
+
+    def __init__(self, rows, row_map, weights, extra):
+        self.rows, self.row_map, self.weights, self.extra = rows, row_map, weights, extra
+
+
 class CudaOps:
     is_cuda = True
     name = "sm100a"
@@ -164,7 +172,7 @@ class CudaOps:
         lib.blz_streams.argtypes = [VP, VP, VP, _c.c_int, _c.c_float, VP, VP, VP, VP, VP, _c.c_float, VP, VP, _c.c_int, _c.c_int, _c.c_int,
                                     _c.c_int, _c.c_int, _c.c_int, VP]
         lib.blz_residual_norm.argtypes = [VP, _c.c_int, _c.c_float, VP, VP, _c.c_float, VP, VP, _c.c_int, _c.c_int, _c.c_int, VP]
-        lib.blz_norm_rows.argtypes = [VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_float, _c.c_int, VP]
+        lib.blz_norm_rows.argtypes = [VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_float, _c.c_int, _c.c_int, VP]
         lib.blz_gemm_simple.argtypes = [VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_int, _c.c_int, _c.c_int, _c.c_int,
                                         _c.c_int, VP]
         lib.blz_clamped_glu.argtypes = [VP, VP, _c.c_int, _c.c_int, _c.c_float, _c.c_int, VP]
@@ -181,7 +189,7 @@ class CudaOps:
         common = [VP, LL, VP, LL, VP, LL, LL, VP, _c.c_int, VP, VP, VP, VP, VP, LL]
         shape = [_c.c_int] * 7 + [_c.c_float] * 2
         lib.blz_soft_plain.argtypes = common + [VP] + shape + [_c.c_int, VP]
-        lib.blz_soft_tc.argtypes = common + shape + [_c.c_int, _c.c_int, VP]
+        lib.blz_soft_tc.argtypes = common + shape + [_c.c_int, _c.c_int, VP, VP]
         lib.blz_soft_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
         lib.blz_short_conv.argtypes = [VP, LL] + [VP] * 8 + [_c.c_int] * 5 + [VP]
         runs = [_c.c_int] * 5 + [VP] + [_c.c_int] * 2 + [VP, LL, _c.c_int, VP]
@@ -189,6 +197,24 @@ class CudaOps:
         lib.blz_state_space.argtypes = [VP, LL, VP, LL] + [VP] * 9 + runs
         lib.blz_rec_ws_bytes.restype = LL
         lib.blz_rec_ws_bytes.argtypes = [_c.c_int] * 5
+        lib.blz_gated_linear.argtypes = [VP, LL, VP, LL, VP, LL] + [VP] * 8 + [_c.c_int] * 4 + [VP] + [_c.c_int] * 2 + [VP, LL, _c.c_int, VP]
+        # residual with normed branches, input convolution, feed-forwards without a gate
+        lib.blz_branch_norm.argtypes = [VP, LL, VP, VP, _c.c_int, VP, VP, _c.c_float, VP, VP] + [_c.c_int] * 3 + [VP]
+        lib.blz_embed_norm.argtypes = [VP, VP, _c.c_int, VP, _c.c_float, VP] + [_c.c_int] * 3 + [VP]
+        lib.blz_input_conv.argtypes = [VP] * 8 + [_c.c_int] * 5 + [VP]
+        lib.blz_relu2.argtypes = [VP, _c.c_int, VP, LL, _c.c_int, VP]
+        lib.blz_poly_norm.argtypes = [VP, VP, VP, _c.c_int, _c.c_int, _c.c_float, _c.c_int, VP]
+        lib.blz_gemm_simple_experts.argtypes = [VP, LL, VP, VP, LL] + [_c.c_int] * 3 + [VP, VP, _c.c_int, VP]
+        # latent attention
+        lib.blz_latent_prep.argtypes = [VP, LL, LL, LL, VP, VP, LL, VP, VP, VP, VP, VP] + [_c.c_int] * 5 + [_c.c_float, _c.c_int, VP]
+        lib.blz_latent_rot.argtypes = [VP] * 6 + [_c.c_int] * 8 + [VP]
+        lib.blz_head_gemm.argtypes = [VP, LL, LL, VP, VP, LL, LL] + [_c.c_int] * 4 + [VP, VP, _c.c_int, _c.c_int, VP]
+        lib.blz_latent_rows_block.restype = _c.c_int
+        lib.blz_latent_rows_block.argtypes = [_c.c_int] * 3
+        lib.blz_latent_rows.argtypes = [VP, VP, VP, LL, VP, _c.c_int, VP, VP, VP, VP] + [_c.c_int] * 5 + [_c.c_float] + [_c.c_int] * 5 + [VP, VP, VP]
+        lib.blz_latent_gather.argtypes = [VP, LL, VP, _c.c_int, VP, _c.c_int, _c.c_int, VP]
+        lib.blz_expand_store.argtypes = [VP, LL, VP, LL, VP, VP] + [_c.c_int] * 6 + [VP]
+        lib.blz_shared_plain.argtypes = [VP, LL, VP, LL, VP, LL, VP, _c.c_int, VP, VP, VP, VP, VP] + [_c.c_int] * 6 + [_c.c_float, _c.c_int, VP]
         lib.blz_group_norm.argtypes = [VP, VP, LL, VP, VP, LL] + [_c.c_int] * 4 + [_c.c_float] * 2 + [_c.c_int] * 3 + [VP]
 
     # ------------------------------------------------------------------ plumbing
@@ -782,14 +808,14 @@ class CudaOps:
         T, W = (src[1].numel(), src[0].shape[1]) if isinstance(src, tuple) else (src.shape[0], src.shape[2])
         return self._streams(src, y, prev, None, None, 0.0, T, W, True, False)[2]
 
-    def norm_rows(self, x, rows, w, eps, dtype):
-        """RMS norm of fp32 rows (those named by ``rows``) to ``dtype``."""
+    def norm_rows(self, x, rows, w, eps, dtype, centre: bool = False):
+        """RMS norm (``centre``: layer norm) of fp32 rows (those named by ``rows``) to ``dtype``."""
         R = x.shape[0] if rows is None else rows.numel()
         out = torch.empty(R, x.shape[1], dtype=dtype, device=self.device)
         if R:
             rows = None if rows is None else rows.to(torch.int32)
-            self._check(self.lib.blz_norm_rows(_ptr(x), _ptr(rows), _ptr(w), _ptr(out), R, x.shape[1], eps, int(dtype == torch.float32),
-                                               self._stream()), "norm_rows")
+            self._check(self.lib.blz_norm_rows(_ptr(x), _ptr(rows), _ptr(w), _ptr(out), R, x.shape[1], eps, int(centre),
+                                               int(dtype == torch.float32), self._stream()), "norm_rows")
         return out
 
     # ------------------------------------------------------------------ differential attention
@@ -894,7 +920,7 @@ class CudaOps:
             return
         items, small = self._split_rows(batch, a)
         if items:
-            self._check(self.lib.blz_soft_tc(*common, *shape, self.SHORT_ROWS, items, st), "soft_tc")
+            self._check(self.lib.blz_soft_tc(*common, *shape, self.SHORT_ROWS, items, VP(0), st), "soft_tc")
         if small:
             self._check(self.lib.blz_soft_short(*common, *shape, self.SHORT_ROWS, *small, st), "soft_short")
 
@@ -913,7 +939,7 @@ class CudaOps:
         """The recurrent mixer of a layer: convolution, recurrence, gated norm into ``out`` (columns of a wider matrix).  Sequences
         flagged in ``batch.gdn_defer`` leave their state untouched; ``state_only`` advances the states and writes nothing."""
         R, r, T = M.rec, M.rec.spec, proj.shape[0]
-        y = self.short_conv(proj, M, batch, kv, layer_idx)
+        y = self.short_conv(proj, M, batch, kv, layer_idx) if r.conv else None
         o = None if state_only else torch.empty(T, r.heads * r.vdim, dtype=torch.float32, device=self.device)
         self.recur(y, proj, low, M, batch, kv, layer_idx, o)
         if state_only:
@@ -922,10 +948,10 @@ class CudaOps:
 
     def gated_norm(self, o, gates, M, eps, out):
         """The norm and gate of a recurrence's rows ``o``; ``gates`` holds the gate's columns: the low-rank outputs (delta rule), or
-        the input projection (state space)."""
+        the input projection (state space; gated linear attention has none)."""
         R, r, es = M.rec, M.rec.spec, gates.element_size()
         delta = R.kind == "delta"
-        z = VP(gates.data_ptr() + (r.heads * r.dim if delta else M.cols["z"]) * es)
+        z = VP(0) if R.kind == "gated" else VP(gates.data_ptr() + (r.heads * r.dim if delta else M.cols["z"]) * es)
         self._check(self.lib.blz_group_norm(_ptr(o), z, gates.stride(0), _ptr(R.norm_w), _ptr(out), out.stride(0), o.shape[0], R.norm_groups,
                                             o.shape[1] // R.norm_groups, R.norm_w.numel(), eps, r.out_scale, int(delta), int(not delta),
                                             int(es == 4), self._stream()), "group_norm")
@@ -933,18 +959,19 @@ class CudaOps:
     REC_MAX_WS = 4 << 30       # workspace of the streaming recurrences; steps that need more run without it
 
     def recur(self, y, proj, low, M, batch, kv, layer_idx, o):
-        """The recurrence alone: convolved inputs ``y`` to fp32 rows ``o`` (None: the state only)."""
+        """The recurrence alone: convolved inputs ``y`` (gated linear attention: None) to fp32 rows ``o`` (None: the state only)."""
         R, r, es, f32 = M.rec, M.rec.spec, proj.element_size(), int(proj.dtype == torch.float32)
         seqs = (_ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(batch.gdn_defer), batch.slots.numel())
-        state, st, longest, T, delta = kv.rec_state[layer_idx], self._stream(), int(batch.max_q_len), y.shape[0], R.kind == "delta"
-        groups = r.kv_heads if delta else r.groups
+        state, st, longest, T = kv.rec_state[layer_idx], self._stream(), int(batch.max_q_len), proj.shape[0]
+        delta, gated = R.kind == "delta", R.kind == "gated"
+        groups = r.kv_heads if delta else r.heads if gated else r.groups
         # which kernels the step needs: single tokens, short runs, and long runs, which read what a token needs from a workspace
         # filled for all tokens at once
         lens = [e - s for s, e in zip(batch.h_q_start, batch.h_q_start[1:])]
         long_rows, ws, ws_bytes = int(self.lib.blz_rec_long_rows()), None, 0
         kinds = (1 if 1 in lens else 0) | (2 if any(1 < n < long_rows for n in lens) else 0)
         if longest >= long_rows:
-            ws_bytes = int(self.lib.blz_rec_ws_bytes(int(delta), T, r.heads, groups, r.state))
+            ws_bytes = int(self.lib.blz_rec_ws_bytes(2 if gated else int(delta), T, r.heads, groups, r.state))
             if o is not None and ws_bytes <= self.REC_MAX_WS:
                 ws = torch.empty(ws_bytes, dtype=torch.uint8, device=self.device)
                 kinds |= 4
@@ -952,7 +979,12 @@ class CudaOps:
                 kinds |= 2
         self.launches += (0, 0, 0, 1, 1, 2, 2, 3)[kinds]
         runs = (_ptr(batch.seq_of_row), T, kinds, _ptr(ws), ws_bytes, f32, st)
-        if delta:
+        if gated:
+            at = [VP(proj.data_ptr() + M.cols[c] * es) for c in ("q", "f", "v")]
+            ld = proj.stride(0)
+            self._check(self.lib.blz_gated_linear(at[0], ld, at[1], ld, at[2], ld, _ptr(R.A), _ptr(R.dt_bias), _ptr(state), _ptr(o), *seqs,
+                                                  r.heads, r.dim, r.vdim, *runs), "gated_linear")
+        elif delta:
             self._check(self.lib.blz_delta_rule(_ptr(y), y.stride(0), _ptr(low), low.stride(0), VP(proj.data_ptr() + M.cols["beta"] * es),
                                                 proj.stride(0), _ptr(R.A), _ptr(R.dt_bias), _ptr(state), _ptr(o), *seqs, r.heads,
                                                 r.kv_heads, r.dim, r.vdim, *runs), "delta_rule")
@@ -960,6 +992,164 @@ class CudaOps:
             self._check(self.lib.blz_state_space(_ptr(y), y.stride(0), VP(proj.data_ptr() + M.cols["dt"] * es), proj.stride(0), _ptr(R.A),
                                                  _ptr(R.dt_bias), _ptr(R.D), _ptr(state), _ptr(o), *seqs, r.heads, r.groups, r.state,
                                                  r.vdim, *runs), "state_space")
+
+    # ------------------------------------------------------------------ residual with normed branches, input convolution
+    def embed_norm(self, table, tokens, w, eps):
+        """Layer-normed embedding rows, fp32."""
+        T, W = tokens.numel(), table.shape[1]
+        x = torch.empty(T, W, dtype=torch.float32, device=self.device)
+        if T:
+            self._check(self.lib.blz_embed_norm(_ptr(table), _ptr(tokens), table.shape[0], _ptr(w), eps, _ptr(x), T, W,
+                                                int(table.dtype == torch.float32), self._stream()), "embed_norm")
+        return x
+
+    def branch_norm(self, x, y, w, eps, copy: bool = True):
+        """``x + layer_norm(y)`` in place of the fp32 rows ``x``, and the same in y's type (``copy``; else None).  ``y`` may be routed
+        rows (:meth:`moe_rows`), which are summed up on the way."""
+        T, W = x.shape
+        routed = isinstance(y, RoutedRows)
+        rows = y.rows if routed else y
+        f32 = rows.dtype == torch.float32
+        h = None if not copy else x if f32 else torch.empty(T, W, dtype=rows.dtype, device=self.device)
+        if T:
+            how = (_ptr(y.weights), _ptr(y.row_map), y.row_map.shape[1], _ptr(y.extra)) if routed else (VP(0), VP(0), 0, VP(0))
+            self._check(self.lib.blz_branch_norm(_ptr(rows), rows.stride(0), *how, _ptr(w), eps, _ptr(x), VP(0) if f32 else _ptr(h), T, W,
+                                                 int(f32), self._stream()), "branch_norm")
+        return x, h
+
+    def input_conv(self, x, w, batch, kv, layer_idx, dtype, state_only: bool = False):
+        """``x + conv(x)`` of fp32 rows in ``dtype``, with the inputs before each sequence's rows from its state row, which advances
+        (not for sequences flagged in ``batch.gdn_defer``)."""
+        T, W = x.shape
+        h = None if state_only else torch.empty(T, W, dtype=dtype, device=self.device)
+        if h is not None and T > batch.h_q_start[-1]:
+            h[batch.h_q_start[-1]:].zero_()                  # padding rows
+        if T:
+            self._check(self.lib.blz_input_conv(_ptr(x), _ptr(h), _ptr(kv.input_state.get(layer_idx)), _ptr(w), _ptr(batch.slots),
+                                                _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(batch.gdn_defer), batch.slots.numel(), W,
+                                                w.shape[0], int(batch.max_q_len), int(dtype == torch.float32), self._stream()), "input_conv")
+            if batch.max_q_len > 32:
+                self.launches += 1
+        return h
+
+    # ------------------------------------------------------------------ feed-forwards without a gate
+    def relu2_(self, z, row_list=None):
+        """``relu(z)^2`` in place, of all rows or of those named by ``row_list`` (-1: none)."""
+        n = z.shape[0] if row_list is None else row_list.numel()
+        if n:
+            self._check(self.lib.blz_relu2(_ptr(z), z.shape[1], _ptr(row_list), n, int(z.dtype == torch.float32), self._stream()), "relu2")
+        return z
+
+    def linear_relu2(self, lin: Linear, x):
+        return self.relu2_(self.linear(lin, x))
+
+    def poly_norm(self, z, act, eps):
+        out = torch.empty_like(z)
+        if z.shape[0]:
+            self._check(self.lib.blz_poly_norm(_ptr(z), _ptr(act), _ptr(out), z.shape[0], z.shape[1], eps, int(z.dtype == torch.float32),
+                                               self._stream()), "poly_norm")
+        return out
+
+    # ------------------------------------------------------------------ latent attention
+    LATENT_SHORT = 16          # new tokens up to which a sequence's queries are mapped to the latents instead of the latents to keys
+
+    def latent_attention(self, proj, M, batch, kv, layer_idx, eps, out):
+        """Latent attention of a mixer: its own latents go to their pages, the heads' outputs (before the output projection) to ``out``."""
+        q = self.latent_queries(proj, M, batch, kv, layer_idx, eps)
+        self.latent_attend(q, M, batch, kv, layer_idx, out)
+
+    def latent_queries(self, proj, M, batch, kv, layer_idx, eps):
+        """Page write, and the queries ``[T, heads * (dim + rot_dim)]`` before their rotation."""
+        A, a, T, pool = M.attn, M.attn.spec, proj.shape[0], kv.kv[layer_idx]
+        if kv.layout != "tiles" or pool.dtype != proj.dtype:
+            raise CudaError(f"latent attention of {proj.dtype} rows needs 'tiles' pages of that type")
+        own = a.kv_from is None
+        lat = torch.empty(T, a.q_rank, dtype=proj.dtype, device=self.device)
+        self._check(self.lib.blz_latent_prep(_ptr(proj), proj.stride(0), M.cols["q"], M.cols.get("kv", 0), _ptr(lat),
+                                             _ptr(pool) if own else VP(0), pool.stride(0), _ptr(A.q_norm), _ptr(A.c_norm), _ptr(A.freq),
+                                             _ptr(batch.positions), _ptr(batch.slot_mapping), T, a.q_rank, a.kv_rank, a.rot_dim,
+                                             a.rot.dims if a.rot is not None else 0, eps, int(proj.dtype == torch.float32), self._stream()),
+                    "latent_prep")
+        return self.linear(A.uq, lat)
+
+    def latent_attend(self, q, M, batch, kv, layer_idx, out):
+        A, a, pool, bt = M.attn, M.attn.spec, kv.kv[layer_idx], kv.block_table
+        T, H, B, f32, st = q.shape[0], a.heads, batch.slots.numel(), q.dtype == torch.float32, self._stream()
+        lens = [e - s for s, e in zip(batch.h_q_start, batch.h_q_start[1:])]
+        # which way: many tokens by head where the prompt kernel covers the sizes, all the others over the latents
+        block = 0 if f32 or a.scale <= 0 else int(self.lib.blz_latent_rows_block(a.kv_rank, a.rot_dim, H))
+        wide = not f32 and a.scale > 0 and a.vdim <= 128 and a.dim + a.rot_dim <= 192
+        most = self.LATENT_SHORT if wide else max(batch.max_q_len, 1)
+        short = [n for n in lens if 0 < n <= most]
+        D = (a.kv_rank + 15) // 16 * 16 + (a.rot_dim + 15) // 16 * 16
+        qe = torch.empty(T, H, D, dtype=q.dtype, device=self.device) if short else None
+        rows = (_ptr(batch.seq_of_row), _ptr(batch.q_start))
+        rot = a.rot.dims if a.rot is not None else 0
+        self._check(self.lib.blz_latent_rot(_ptr(q), _ptr(qe), _ptr(A.freq), _ptr(batch.positions), *rows, T, H, a.dim, a.rot_dim, rot,
+                                            a.kv_rank, most, int(f32), st), "latent_rot")
+        if short:
+            self._check(self.lib.blz_head_gemm(_ptr(q), q.stride(0), a.dim + a.rot_dim, _ptr(A.uk_t), _ptr(qe), H * D, D, T, a.kv_rank, a.dim,
+                                               H, *rows, most, int(f32), st), "head_gemm")
+            lat = torch.empty(T, H, a.kv_rank, dtype=q.dtype, device=self.device)
+            seqs = (_ptr(bt), bt.stride(0), _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(A.sink))
+            if block:
+                longest = max(short)
+                R = int(self.lib.blz_latent_rows_block(a.kv_rank, a.rot_dim, longest * H))
+                rb = (longest * H + R - 1) // R
+                keys = min(batch.max_ctx, a.window + (R + H - 1) // H) if a.window else batch.max_ctx
+                sp = max(1, min(self._sm // (len(short) * rb), (keys + 127) // 128, 32))
+                po = pm = None
+                if sp > 1:
+                    n = B * rb * sp * R
+                    po, pm = self._buf("latent_part_o", n * a.kv_rank * 4), self._buf("latent_part_ml", n * 8)
+                    self.launches += 1
+                self._check(self.lib.blz_latent_rows(_ptr(qe), _ptr(lat), _ptr(pool), pool.stride(0), *seqs, B, H, a.kv_rank, a.rot_dim, a.window,
+                                                     a.scale, most, longest, R, rb, sp, _ptr(po), _ptr(pm), st), "latent_rows")
+            else:
+                self._check(self.lib.blz_shared_plain(_ptr(qe), H * D, _ptr(lat), H * a.kv_rank, _ptr(pool), pool.stride(0), *seqs,
+                                                      _ptr(batch.seq_of_row), T, B, H, D, a.kv_rank, a.window, a.scale, int(f32), st),
+                            "shared_plain")
+            self._check(self.lib.blz_head_gemm(_ptr(lat), H * a.kv_rank, a.kv_rank, _ptr(A.uv), _ptr(out), out.stride(0), a.vdim, T, a.vdim,
+                                               a.kv_rank, H, *rows, most, int(f32), st), "head_gemm")
+        if any(n > most for n in lens):
+            self._latent_expanded(q, M, batch, kv, layer_idx, most, out)
+
+    def _latent_expanded(self, q, M, batch, kv, layer_idx, most: int, out):
+        """Prompt portions: keys and values by head of all tokens that the sequences with more than ``most`` new tokens see."""
+        A, a, pool, st = M.attn, M.attn.spec, kv.kv[layer_idx], self._stream()
+        T, H, B = q.shape[0], a.heads, batch.slots.numel()
+        pages, base, n_pages, items = self._visible_pages(batch, kv, a.window, most)
+        lat = torch.empty(n_pages * 16, a.kv_rank, dtype=q.dtype, device=self.device)
+        self._check(self.lib.blz_latent_gather(_ptr(pool), pool.stride(0), _ptr(pages), n_pages, _ptr(lat), a.kv_rank, a.rot_dim, st), "latent_gather")
+        kx = self.linear(A.expand, lat)
+        up = lambda n: (n + 15) // 16 * 16       # noqa: E731
+        be = 16 * (up(a.dim + a.rot_dim) + up(a.vdim))
+        scratch = torch.empty(n_pages, H, be, dtype=q.dtype, device=self.device)
+        self._check(self.lib.blz_expand_store(_ptr(kx), kx.stride(0), _ptr(pool), pool.stride(0), _ptr(pages), _ptr(scratch), n_pages, H, a.dim,
+                                              a.rot_dim, a.vdim, a.kv_rank, st), "expand_store")
+        bt = kv.block_table
+        self._check(self.lib.blz_soft_tc(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(scratch), scratch.stride(0), scratch.stride(1),
+                                         _ptr(bt), bt.stride(0), _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(A.sink), VP(0), 0,
+                                         T, B, H, H, a.dim + a.rot_dim, a.vdim, a.window, a.scale, 1.0, most, items, _ptr(base), st), "soft_tc")
+
+    def _visible_pages(self, batch, kv, window: int, most: int):
+        """(pages, page base of each sequence, number of pages, row blocks) of the sequences with more than ``most`` new tokens: the pages
+        any of their rows sees, one sequence after the other.  Kept with the batch: its layers share them."""
+        key = (window, most)
+        hit = batch.visible.get(key)
+        if hit is not None:
+            return hit
+        pages, base, items = [], [], 0
+        for b, slot in enumerate(batch.h_slots):
+            n, ctx = batch.h_q_start[b + 1] - batch.h_q_start[b], batch.h_ctx_len[b]
+            lo = (max(ctx - n - window + 1, 0) if window else 0) // 16
+            base.append(len(pages) - lo)
+            if n > most:
+                pages.extend(kv.block_table_host[slot, lo:(ctx + 15) // 16].tolist())
+                items += -(-n // 256)
+        dev = torch.tensor(base + pages, dtype=torch.int32).to(self.device)
+        batch.visible[key] = hit = (dev[len(base):], dev[:len(base)], len(pages), items)
+        return hit
 
     # ------------------------------------------------------------------ head
     def argmax(self, logits, index_offset: int = 0, want_values: bool = False):
@@ -988,6 +1178,28 @@ class CudaOps:
         if ex.cuda_pack is not None:
             return ex.cuda_pack
 
+        relu2 = ex.act == "relu2"
+        if relu2 and (ex.gate_up[0].w.dtype == torch.float32 or ex.gate_up[0].K % 16):
+            # 32-bit, or rows too ragged for TMA: the CUDA-core product
+            def plain(lins):
+                w = torch.stack([l.w for l in lins]).to(self.device).contiguous()
+                return {"kind": 5, "w": w, "N": lins[0].N, "K": lins[0].K, "fmt": Format.DENSE, "act_quant": False}
+            ex.cuda_pack = {"gate_up": plain(ex.gate_up), "down": plain(ex.down)}
+            return ex.cuda_pack
+
+        def padded(lins, n128, k128):
+            """The grouped product's tiles are 128 rows of one expert's weight: pad those that are not (zeros stay zeros)."""
+            N, K = lins[0].N, lins[0].K
+            NP, KP = (N + 127) // 128 * 128 if n128 else N, (K + 127) // 128 * 128 if k128 else K
+            if (NP, KP) == (N, K):
+                return lins
+            out = []
+            for l in lins:
+                w = l.w.new_zeros(NP, KP)
+                w[:N, :K] = l.w
+                out.append(Linear.from_dense(w, dtype=l.w.dtype))
+            return out
+
         def stack(lins):
             pk0 = self.pack(lins[0], tiled=False, exact_fp8=False)
             kind = pk0["kind"]
@@ -1011,7 +1223,8 @@ class CudaOps:
                 l.cuda_pack = None          # the stacked copy replaces the per-expert ones
             return {"kind": kind, "w": w.contiguous(), "sf": sf, "alpha": alpha, "N": lins[0].N, "K": lins[0].K,
                     "fmt": lins[0].fmt, "act_quant": lins[0].act_quant}
-        ex.cuda_pack = {"gate_up": stack(ex.gate_up), "down": stack(ex.down)}
+        up, down = (padded(ex.gate_up, True, False), padded(ex.down, True, True)) if relu2 else (ex.gate_up, ex.down)
+        ex.cuda_pack = {"gate_up": stack(up), "down": stack(down)}
         return ex.cuda_pack
 
     def _grouped_gemm(self, pk, a, M_pad, tile_expert, n_exp, out):
@@ -1031,6 +1244,15 @@ class CudaOps:
     def moe(self, x, topk_w, topk_id, experts):
         """Routed experts held by this rank: scatter rows by expert → grouped gate_up GEMM → SwiGLU → grouped down GEMM →
         weighted combine.  ``x`` is bf16 ``[T, H]``.  Under expert parallelism the result is a partial sum."""
+        r = self.moe_rows(x, topk_w, topk_id, experts)
+        T, H, k = x.shape[0], x.shape[1], topk_id.shape[1]
+        out = torch.empty(T, H, dtype=torch.bfloat16, device=self.device)
+        self._check(self.lib.blz_moe_combine(_ptr(r.rows), _ptr(r.weights), _ptr(r.row_map), _ptr(out), T, H, k, self._stream()),
+                    "moe_combine")
+        return out
+
+    def moe_rows(self, x, topk_w, topk_id, experts, shared=None) -> RoutedRows:
+        """The routed experts' outputs as rows (:meth:`branch_norm` sums them up, with ``shared`` added)."""
         pk = self.pack_experts(experts)
         gu, dn = pk["gate_up"], pk["down"]
         T, H = x.shape
@@ -1063,11 +1285,26 @@ class CudaOps:
                                                  _ptr(a.row_scale), _ptr(topk_id), _ptr(offsets), _ptr(fill), _ptr(row_map), T, H, k,
                                                  first, n_exp, self._stream()), "moe_scatter")
         else:
-            a = torch.empty(M_pad, H, dtype=torch.bfloat16, device=dev)
+            a = torch.empty(M_pad, H, dtype=x.dtype, device=dev)
             self._check(self.lib.blz_moe_scatter(0, _ptr(x.contiguous()), VP(0), VP(0), _ptr(a), VP(0), VP(0), _ptr(topk_id),
-                                                 _ptr(offsets), _ptr(fill), _ptr(row_map), T, H, k, first, n_exp, self._stream()),
-                        "moe_scatter")
-        g = torch.empty(M_pad, gu["N"], dtype=torch.bfloat16, device=dev)
+                                                 _ptr(offsets), _ptr(fill), _ptr(row_map), T, H * x.element_size() // 2, k, first, n_exp,
+                                                 self._stream()), "moe_scatter")
+        self._route_counts = None
+        g = torch.empty(M_pad, gu["N"], dtype=x.dtype, device=dev)
+        if experts.act == "relu2":
+            y = torch.empty(M_pad, dn["N"], dtype=x.dtype, device=dev)
+            for w, src, dst in ((gu, a, g), (dn, g, y)):
+                if w["kind"] == 5:
+                    self._check(self.lib.blz_gemm_simple_experts(_ptr(src), src.stride(0), _ptr(w["w"]), _ptr(dst), dst.stride(0), max_tiles, w["N"],
+                                                                 w["K"], _ptr(tile_expert), _ptr(tile_rows), int(x.dtype == torch.float32),
+                                                                 self._stream()), "gemm_simple_experts")
+                elif narrow:
+                    self._moe_gemm(w, src, max_tiles, tile_expert, tile_rows, n_exp, dst)
+                else:
+                    self._grouped_gemm(w, src, M_pad, tile_expert, n_exp, dst)
+                if dst is g:
+                    self.relu2_(g, row_map)
+            return RoutedRows(y, row_map, topk_w.contiguous(), shared)
         proxy_d = Linear(dn["fmt"], dn["N"], dn["K"])
         proxy_d.act_quant = dn["act_quant"]
         y = torch.empty(M_pad, dn["N"], dtype=torch.bfloat16, device=dev)
@@ -1080,11 +1317,7 @@ class CudaOps:
             # only the routed rows: the padded row space is up to (1 + experts * 128 / routed rows) times larger
             act = self._silu_mul_live(g, proxy_d if dn["kind"] in (1, 2) else None, row_map)
             self._grouped_gemm(dn, act, M_pad, tile_expert, n_exp, y)
-        out = torch.empty(T, H, dtype=torch.bfloat16, device=dev)
-        self._check(self.lib.blz_moe_combine(_ptr(y), _ptr(topk_w.contiguous()), _ptr(row_map), _ptr(out), T, H, k, self._stream()),
-                    "moe_combine")
-        self._route_counts = None
-        return out
+        return RoutedRows(y, row_map, topk_w.contiguous(), shared)
 
     def _moe_gemm(self, pk, a, row_tiles, tile_expert, tile_rows, n_exp, out):
         """Expert GEMM over the padded row space with the features on the MMA lanes and only each tile's live rows on its columns."""

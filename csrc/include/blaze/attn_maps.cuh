@@ -33,6 +33,8 @@ struct MapsParams {
   int max_rows;                // rows (new tokens * group) up to which a sequence belongs to the short-row kernel
   int row_blocks, splits, stages;
   int* status;
+  const int* page_base;        // [B] or null: the pages of sequence b are page_base[b] + page index, not block_table's
+  int shared_kv;               // one map: a block is its key part alone, whose first vdim columns are the values
 
   __host__ __device__ int group() const { return heads / kv_heads; }
   __host__ __device__ int dp() const { return (dim + 15) / 16 * 16; }

@@ -60,7 +60,7 @@ __global__ void __launch_bounds__(128) maps_plain_kernel(MapsParams p) {
   const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int b = p.seq_of_row[t];
   if (b < 0) return;
-  const int g = h / p.group(), dp = p.dp(), vp = p.vp();
+  const int g = h / p.group(), dp = p.dp(), vp = p.shared_kv ? dp : p.vp(), v_at = p.shared_kv ? 0 : MAPS * 16 * dp;
   const int pos = p.ctx_len[b] - (p.q_start[b + 1] - t);
   const int lo = first_key(pos, p.window);
   const T* q = reinterpret_cast<const T*>(p.q) + (size_t)t * p.ld + (size_t)h * MAPS * p.dim;
@@ -109,7 +109,7 @@ __global__ void __launch_bounds__(128) maps_plain_kernel(MapsParams p) {
     __syncthreads();
     const int k_end = min(128, pos - k0 + 1);
     for (int kk = max(lo - k0, 0); kk < k_end; ++kk) {
-      const T* vr = pool + (size_t)s_page[kk >> 4] * p.page_stride + MAPS * 16 * dp;
+      const T* vr = pool + (size_t)s_page[kk >> 4] * p.page_stride + v_at;
 #pragma unroll
       for (int c = 0; c < VC; ++c) {
         const int e = tid + c * 128;
@@ -754,7 +754,20 @@ BLZ_API int blz_soft_plain(const void* q, long long ld, void* out, long long ld_
   return blz::run_plain(p, f32, s);
 }
 
-// The same for the short sequences of a bf16 step; see blz_diff_short (one map: part_o [...][1][16][VP]).
+// Every head against the one vector a token has in its page (dim columns, a multiple of 16, of which the first vdim are the value), with an
+// optional sink; otherwise as above.
+BLZ_API int blz_shared_plain(const void* q, long long ld, void* out, long long ld_out, void* pool, long long page_stride, const int* block_table,
+                             int bt_stride, const int* slots, const int* q_start, const int* ctx_len, const float* sink, const int* seq_of_row,
+                             int T, int B, int heads, int dim, int vdim, int window, float scale, int f32, cudaStream_t s) {
+  if (dim % 16 || vdim > dim) return (int)cudaErrorInvalidValue;
+  blz::MapsParams p = blz::soft_params(q, ld, out, ld_out, pool, page_stride, 0, block_table, bt_stride, slots, q_start, ctx_len, sink, nullptr, 0,
+                                       T, B, heads, 1, dim, vdim, window, scale, 1.f);
+  p.seq_of_row = seq_of_row;
+  p.shared_kv = 1;
+  return blz::run_plain(p, f32, s);
+}
+
+// One softmax map (blz_soft_plain) for the short sequences of a bf16 step; see blz_diff_short (one map: part_o [...][1][16][VP]).
 BLZ_API int blz_soft_short(const void* q, long long ld, void* out, long long ld_out, void* pool, long long page_stride, long long head_stride,
                            const int* block_table, int bt_stride, const int* slots, const int* q_start, const int* ctx_len,
                            const float* sink, const void* gate, long long ld_gate, int T, int B, int heads, int kv_heads, int dim, int vdim,

@@ -33,14 +33,6 @@ __device__ __forceinline__ void mma_f16_ts(uint32_t d_tmem, uint32_t a_tmem, uin
       ::"r"(d_tmem), "r"(a_tmem), "l"(b), "r"(idesc), "r"(acc)
       : "memory");
 }
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
-      ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
-        "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-      : "memory");
-}
-
 struct MapsTc {
   int ks, vs;                  // K and V ring depths
 };
@@ -119,7 +111,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
       for (; i < n; ++i) {
         const int ks = i % c.ks, vs = i % c.vs;
         const int pidx = pg_lo + i * 8 + pg;
-        const int page = (lane < 8 * (MAPS + 1) && pidx <= pg_hi) ? bt[pidx] : 0;        // page 0: zeros
+        int page = 0;                                    // page 0: finite numbers, masked
+        if (lane < 8 * (MAPS + 1) && pidx <= pg_hi) page = p.page_base ? p.page_base[b] + pidx : bt[pidx];
         const __nv_bfloat16* src = pool + (size_t)page * p.page_stride;
         if (!__all_sync(0xffffffffu, mbar_wait(&k_empty[ks], (uint32_t)(((i / c.ks) & 1) ^ 1), abort_flag, p.status))) break;
         if (lane == 0) mbar_expect_tx(&k_full[ks], MAPS * k_bytes);
@@ -372,13 +365,14 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
 template <int MAPS>
 static int run_tc(const MapsParams& p, int items, cudaStream_t s) {
   if (p.T <= 0 || p.B <= 0 || p.heads < 1 || p.kv_heads < 1 || p.kv_heads > 65535 || p.heads % p.kv_heads || p.group() > 128 || p.dim < 1 ||
-      p.dim > 128 || p.vdim < 1 || p.vdim > 128 || p.window < 0 || items < 1)
+      p.dim > 256 || p.vdim < 1 || p.vdim > 128 || p.window < 0 || items < 1)
     return (int)cudaErrorInvalidValue;
   if ((p.page_stride * 2) % 16 || (p.head_stride * 2) % 16 || (reinterpret_cast<uintptr_t>(p.pool) & 15)) return (int)cudaErrorInvalidValue;
   const int q_bytes = 256 * p.dp() * 2, k_bytes = MAPS * 128 * p.dp() * 2, v_bytes = 128 * p.vp() * 2, fixed = 128 + 2048 + 256;
   MapsTc c = {2, 2};
   auto total = [&]() { return fixed + q_bytes + c.ks * k_bytes + c.vs * v_bytes; };
   if (total() > 227 * 1024) c.ks = 1;
+  if (total() > 227 * 1024) c.vs = 1;
   if (total() > 227 * 1024) return (int)cudaErrorInvalidValue;
   const int vec_q = (reinterpret_cast<uintptr_t>(p.q) & 15) == 0 && p.ld % 8 == 0 && p.dim % 8 == 0;
   const int vec_o = (reinterpret_cast<uintptr_t>(p.out) & 15) == 0 && p.ld_out % 8 == 0 && p.vdim % 8 == 0 &&
@@ -408,13 +402,15 @@ BLZ_API int blz_diff_tc(const void* qkv, long long ld, void* out, void* pool, lo
 }
 
 // One softmax map per head with optional sink and gate (see blz_soft_plain), bf16; the sequences with more than max_rows rows,
-// `items` row blocks of 2 * (128 / group) tokens in all.  dim, vdim <= 128, group <= 128.
+// `items` row blocks of 2 * (128 / group) tokens in all.  vdim <= 128, group <= 128, dim as far as shared memory goes (192 at least).
+// page_base ([B] or null): the pages of sequence b lie one after the other from page_base[b] (of position 0, which need not exist) on.
 BLZ_API int blz_soft_tc(const void* q, long long ld, void* out, long long ld_out, void* pool, long long page_stride, long long head_stride,
                         const int* block_table, int bt_stride, const int* slots, const int* q_start, const int* ctx_len, const float* sink,
                         const void* gate, long long ld_gate, int T, int B, int heads, int kv_heads, int dim, int vdim, int window,
-                        float scale, float post, int max_rows, int items, cudaStream_t s) {
+                        float scale, float post, int max_rows, int items, const int* page_base, cudaStream_t s) {
   using namespace blz;
   MapsParams p = {};
+  p.page_base = page_base;
   p.q = q; p.ld = ld; p.out = out; p.ld_out = ld_out; p.pool = pool; p.page_stride = page_stride; p.head_stride = head_stride;
   p.block_table = block_table; p.bt_stride = bt_stride; p.slots = slots; p.q_start = q_start; p.ctx_len = ctx_len;
   p.sink = sink; p.gate = gate; p.ld_gate = ld_gate;

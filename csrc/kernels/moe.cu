@@ -97,7 +97,7 @@ __global__ void moe_plan_kernel(const int* __restrict__ counts, int* __restrict_
   }
 }
 
-// One block per token.  QK: 0 = bf16 rows [T, K]; 1 = NVFP4 (data [T, K/2], tiled e4m3 scales, row scale); 2 = MXFP8.
+// One block per token.  QK: 0 = bf16 rows [T, K] (32-bit rows of K / 2); 1 = NVFP4 (data [T, K/2], tiled e4m3 scales, row scale); 2 = MXFP8.
 template <int QK>
 __global__ void moe_scatter_kernel(const uint8_t* __restrict__ src, const uint8_t* __restrict__ src_sf,
                                    const float* __restrict__ src_rs, uint8_t* __restrict__ dst, uint8_t* __restrict__ dst_sf,
@@ -119,6 +119,12 @@ __global__ void moe_scatter_kernel(const uint8_t* __restrict__ src, const uint8_
   for (int j = 0; j < k; ++j) {
     const int row = s_row[j];
     if (row < 0) continue;
+    if (QK == 0 && row_bytes % 16) {                 // ragged rows: element by element
+      const uint16_t* s2 = reinterpret_cast<const uint16_t*>(src + (size_t)t * row_bytes);
+      uint16_t* d2 = reinterpret_cast<uint16_t*>(dst + (size_t)row * row_bytes);
+      for (int i = threadIdx.x; i < K; i += blockDim.x) d2[i] = s2[i];
+      continue;
+    }
     const uint4* s4 = reinterpret_cast<const uint4*>(src + (size_t)t * row_bytes);
     uint4* d4 = reinterpret_cast<uint4*>(dst + (size_t)row * row_bytes);
     for (int i = threadIdx.x; i < row_bytes / 16; i += blockDim.x) d4[i] = s4[i];

@@ -2,6 +2,8 @@
 //   delta rule with a decay per key channel:  S <- g * S (rows);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //       g = exp(-A softplus(a + dt_bias)), beta = sigmoid(b), q and k made unit vectors, q times dim^-1/2
 //   state-space duality:  S <- exp(-A dt) S + dt B x^T;  y = S^T C + D x,  dt = softplus(dt_raw + dt_bias)
+//   gated linear (HGRN2): S <- f * S + (1 - f) v^T (f acts on rows);  o = S^T silu(q),  f = lo + (1 - lo) sigmoid(f_raw + bias)
+//       (rows beyond dk have f = 0 and q = 0)
 // and the norm over groups of columns with a gate before or after it that follows either of them.
 // State: [rows, heads, keys (or state size), vdim] fp32; rows are sequence slots; a sequence without earlier tokens starts at zero.
 //
@@ -21,17 +23,18 @@ static constexpr int kRecTok = 8;            // tokens per group
 static constexpr int kRecWarps = 4;          // warps that hold state
 
 struct RecParams {
-  const void* conv;            // [T, ld_conv] convolved inputs: delta q | k | v, state space x | B | C
-  const void* a;               // delta: decay inputs [T, ld_a], heads * dk columns; state space: dt_raw [T, ld_a], heads columns
-  const void* b;               // delta: beta inputs [T, ld_b], heads columns
-  const float* A;              // [heads], positive
-  const float* dt_bias;        // delta [heads * dk], state space [heads]
+  const void* conv;            // [T, ld_conv] convolved inputs: delta q | k | v, state space x | B | C; gated linear: v
+  const void* a;               // delta: decay inputs [T, ld_a], heads * dk columns; state space: dt_raw [T, ld_a], heads columns;
+                               // gated linear: f_raw, heads * dk columns
+  const void* b;               // delta: beta inputs [T, ld_b], heads columns; gated linear: q before its activation, heads * dk columns
+  const float* A;              // [heads], positive; gated linear: lower bounds [heads * dk]
+  const float* dt_bias;        // delta and gated linear [heads * dk], state space [heads]
   const float* D;              // [heads] or null
   float* state;
   float* out;                  // [T, heads * dv] or null (the state only)
   const int *slots, *q_start, *ctx_len, *no_store;
   long long ld_conv, ld_a, ld_b;
-  int heads, groups, dk, dv;   // groups: key heads (delta) or B / C groups (state space)
+  int heads, groups, dk, dv;   // groups: key heads (delta), B / C groups (state space), heads (gated linear)
   const int* seq_of_row;       // [T], -1 = padding
   float* records;              // workspace of the long runs
   int T, long_rows;            // sequences with at least long_rows new tokens are long runs
@@ -49,6 +52,13 @@ template <typename T>
 __device__ __forceinline__ float rc_softplus(float x) { return x > 20.f ? x : log1pf(rc_exp<T>(x)); }
 template <typename T>
 __device__ __forceinline__ float rc_sigmoid(float x) { return 1.f / (1.f + rc_exp<T>(-x)); }
+
+// the three recurrences; GATED shares the kernels of SSM, which have no reduction between tokens
+enum RecKind { DELTA, SSM, GATED };
+template <typename T>
+__device__ __forceinline__ float rc_silu(float x) { return x * rc_sigmoid<T>(x); }
+template <typename T>
+__device__ __forceinline__ float forget_gate(float z, float lo) { return fmaf(1.f - lo, rc_sigmoid<T>(z), lo); }
 
 // lane (row group kl < KL, column group cg) of a warp: rows kl * 4 + 4 KL * (i / 4) + i % 4, i < R; columns col .. col + VPT
 template <int KL, int R, int VPT>
@@ -252,10 +262,10 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_r
   if (!(p.no_store != nullptr && p.no_store[b])) store_state<8, R, VPT>(S, st, kl, col, dk, dv, vec);
 }
 
-template <typename T, int R, int VPT>
+template <typename T, int R, int VPT, bool G>
 __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) state_space_kernel(RecParams p, int slices) {
   constexpr int NP = R * 8, COLS = kRecWarps * 4 * VPT, TOK = 2 * NP + COLS + 4;
-  extern __shared__ float sm[];              // [2][kRecTok][B | C | x | dt | decay]
+  extern __shared__ float sm[];              // [2][kRecTok][B | C | x | dt | decay]; G: [f | q | v | ..]
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
@@ -266,11 +276,28 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) state_s
   const bool vec = dv % 4 == 0;
   float S[R][VPT];
   load_state<8, R, VPT>(S, st, kl, col, N, dv, ctx == n, vec);
-  const float A = p.A[h], bias = p.dt_bias[h], D = p.D ? p.D[h] : 0.f;
+  const float A = G ? 0.f : p.A[h], bias = G ? 0.f : p.dt_bias[h], D = !G && p.D ? p.D[h] : 0.f;
 
   auto stage = [&](int t0, float* buf) {
     for (int j = warp; j < kRecTok; j += kRecWarps) {
       float* s = buf + j * TOK;
+      if constexpr (G) {
+        if (t0 + j >= n) continue;
+        const size_t row = (size_t)(r0 + t0 + j), hd = (size_t)h * N;
+        const T* fr = reinterpret_cast<const T*>(p.a) + row * p.ld_a + hd;
+        const T* qr = reinterpret_cast<const T*>(p.b) + row * p.ld_b + hd;
+#pragma unroll
+        for (int i = 0; i < NP / 32; ++i) {
+          const int d = lane + i * 32;
+          s[d] = d < N ? forget_gate<T>(rc_ld(fr + d) + p.dt_bias[hd + d], p.A[hd + d]) : 0.f;
+          s[NP + d] = d < N ? rc_silu<T>(rc_ld(qr + d)) : 0.f;
+        }
+        for (int c = lane; c < COLS; c += 32) {
+          const int e = slice * COLS + c;
+          s[2 * NP + c] = e < dv ? rc_ld(reinterpret_cast<const T*>(p.conv) + row * p.ld_conv + (size_t)h * dv + e) : 0.f;
+        }
+        continue;
+      }
       if (t0 + j >= n) {                     // beyond the run: a step that changes nothing
         for (int d = lane; d < TOK; d += 32) s[d] = d == 2 * NP + COLS + 1 ? 1.f : 0.f;
         continue;
@@ -306,7 +333,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) state_s
 #pragma unroll
       for (int j = 0; j < kRecTok; ++j) {
         const float* s = buf + j * TOK;
-        const float dt = s[2 * NP + COLS], dec = s[2 * NP + COLS + 1];
+        const float dt = G ? 1.f : s[2 * NP + COLS], dec = G ? 0.f : s[2 * NP + COLS + 1];
         float x[VPT];
 #pragma unroll
         for (int v = 0; v < VPT; ++v) { x[v] = dt * s[2 * NP + lc + v]; y[j][v] = 0.f; }
@@ -321,7 +348,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) state_s
 #pragma unroll
               for (int v = 0; v < VPT; ++v) {
                 float& z = S[i4 * 4 + i][v];
-                z = fmaf(z, dec, ba[i] * x[v]);
+                z = G ? fmaf(z, ba[i], (1.f - ba[i]) * x[v]) : fmaf(z, dec, ba[i] * x[v]);
                 y[j][v] = fmaf(z, ca[i], y[j][v]);
               }
           }
@@ -332,7 +359,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) state_s
         if (t0 + kl < n) {
           const float* s = buf + kl * TOK + 2 * NP + lc;
 #pragma unroll
-          for (int v = 0; v < VPT; ++v) y[0][v] = fmaf(D, s[v], y[0][v]);
+          for (int v = 0; v < VPT && !G; ++v) y[0][v] = fmaf(D, s[v], y[0][v]);
           store_cols<VPT>(p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col, y[0], col, dv, vec);
         }
       }
@@ -472,9 +499,56 @@ __global__ void __launch_bounds__(kRecWarps * 32, 4) state_space_step_kernel(Rec
   }
 }
 
+// The gates and queries of a row, one per thread, meet in shared memory.
+template <typename T, int KL, int R, int VPT>
+__global__ void __launch_bounds__(kRecWarps * 32, 4) gated_step_kernel(RecParams p, int slices, int) {
+  constexpr int CG = 32 / KL, NP = KL * R;
+  __shared__ __align__(16) float s_f[NP], s_q[NP];
+  const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
+  if (n != 1) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane % KL, N = p.dk, dv = p.dv;
+  const int col = slice * kRecWarps * CG * VPT + warp * CG * VPT + lane / KL * VPT;
+  float* st = p.state + ((size_t)slot * p.heads + h) * N * dv;
+  const bool vec = dv % 4 == 0;
+  float S[R][VPT], v[VPT], y[VPT];
+  load_state<KL, R, VPT>(S, st, kl, col, N, dv, ctx == 1, vec);
+  const size_t hd = (size_t)h * N;
+  const T* fr = reinterpret_cast<const T*>(p.a) + (size_t)r0 * p.ld_a + hd;
+  const T* qr = reinterpret_cast<const T*>(p.b) + (size_t)r0 * p.ld_b + hd;
+  const T* vr = reinterpret_cast<const T*>(p.conv) + (size_t)r0 * p.ld_conv + (size_t)h * dv + col;
+#pragma unroll
+  for (int c = 0; c < VPT; ++c) { v[c] = col + c < dv ? rc_ld(vr + c) : 0.f; y[c] = 0.f; }
+  for (int d = threadIdx.x; d < NP; d += kRecWarps * 32) {
+    s_f[d] = d < N ? forget_gate<T>(rc_ld(fr + d) + p.dt_bias[hd + d], p.A[hd + d]) : 0.f;
+    s_q[d] = d < N ? rc_silu<T>(rc_ld(qr + d)) : 0.f;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i4 = 0; i4 < R / 4; ++i4) {
+    const float4 f4 = *reinterpret_cast<const float4*>(s_f + kl * 4 + 4 * KL * i4);
+    const float4 q4 = *reinterpret_cast<const float4*>(s_q + kl * 4 + 4 * KL * i4);
+    const float fa[4] = {f4.x, f4.y, f4.z, f4.w}, qa[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int c = 0; c < VPT; ++c) {
+        float& z = S[i4 * 4 + i][c];
+        z = fmaf(z, fa[i], (1.f - fa[i]) * v[c]);
+        y[c] = fmaf(z, qa[i], y[c]);
+      }
+  }
+  if (!(p.no_store != nullptr && p.no_store[b])) store_state<KL, R, VPT>(S, st, kl, col, N, dv, vec);
+  if (p.out) {
+#pragma unroll
+    for (int c = 0; c < VPT; ++c) y[c] = lanes_sum<KL>(y[c]);
+    if (kl == 0) store_cols<VPT>(p.out + ((size_t)r0 * p.heads + h) * dv + col, y, col, dv, vec);
+  }
+}
+
 // ------------------------------------------------------------------------------------------ long runs
-// Records: delta [heads][T][q | k | g | beta, k . q, 0, 0], state space [groups][T][B | C] and [heads][T][dt, decay, 0, 0];
-// vectors padded to 32, 64, 128, 256 or 512 floats.
+// Records: delta [heads][T][q | k | g | beta, k . q, 0, 0], state space [groups][T][B | C] and [heads][T][dt, decay, 0, 0], gated
+// linear [heads][T][f | q]; vectors padded to 32, 64, 128, 256 or 512 floats.
 __device__ __forceinline__ bool in_long_run(const RecParams& p, int t) {
   const int b = p.seq_of_row[t];
   return b >= 0 && p.q_start[b + 1] - p.q_start[b] >= p.long_rows;
@@ -533,6 +607,24 @@ __global__ void __launch_bounds__(128) state_space_records_kernel(RecParams p) {
   for (int h = threadIdx.x; h < p.heads; h += 128) {
     const float dt = rc_softplus<T>(rc_ld(reinterpret_cast<const T*>(p.a) + (size_t)t * p.ld_a + h) + p.dt_bias[h]);
     steps[(size_t)h * p.T + t] = make_float4(dt, rc_exp<T>(-p.A[h] * dt), 0.f, 0.f);
+  }
+}
+
+// a warp per (row, head)
+template <typename T, int DKP>
+__global__ void __launch_bounds__(128) gated_records_kernel(RecParams p) {
+  const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int t = (int)(w / p.heads), h = (int)(w % p.heads), lane = threadIdx.x & 31, N = p.dk;
+  if (t >= p.T || !in_long_run(p, t)) return;
+  const size_t hd = (size_t)h * N;
+  const T* fr = reinterpret_cast<const T*>(p.a) + (size_t)t * p.ld_a + hd;
+  const T* qr = reinterpret_cast<const T*>(p.b) + (size_t)t * p.ld_b + hd;
+  float* s = p.records + ((size_t)h * p.T + t) * 2 * DKP;
+#pragma unroll
+  for (int i = 0; i < DKP / 32; ++i) {
+    const int d = lane + i * 32;
+    s[d] = d < N ? forget_gate<T>(rc_ld(fr + d) + p.dt_bias[hd + d], p.A[hd + d]) : 0.f;
+    s[DKP + d] = d < N ? rc_silu<T>(rc_ld(qr + d)) : 0.f;
   }
 }
 
@@ -746,9 +838,9 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
   if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<KL, R, VPT>(S, st, kl, col, dk, dv, vec);
 }
 
-template <typename T, int KL, int R, int VPT>
+template <typename T, int KL, int R, int VPT, bool G>
 __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) state_space_stream_kernel(RecParams p, int slices, int vec_v) {
-  constexpr int NP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, REC = 2 * NP, STAGE = kRecTok * (REC + 4);
+  constexpr int NP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, REC = 2 * NP, STEPS = G ? 0 : 4, STAGE = kRecTok * (REC + STEPS);
   extern __shared__ __align__(128) uint8_t sm8[];
   __shared__ __align__(16) T s_v[kRecWarps][kColsAhead + 1][kRecTok][CG * VPT];
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
@@ -766,9 +858,9 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) s
       rr.produce(groups, [&](int c) {
         const uint32_t m = (uint32_t)min(kRecTok, n - c * kRecTok);
         float* dst = ring + (c % kRecStages) * STAGE;
-        mbar_expect_tx(&rr.full[c % kRecStages], m * (REC + 4) * 4);
+        mbar_expect_tx(&rr.full[c % kRecStages], m * (REC + STEPS) * 4);
         bulk_load(dst, src + (size_t)c * kRecTok * REC, m * REC * 4, &rr.full[c % kRecStages]);
-        bulk_load(dst + kRecTok * REC, steps + (size_t)c * kRecTok * 4, m * 16, &rr.full[c % kRecStages]);
+        if constexpr (!G) bulk_load(dst + kRecTok * REC, steps + (size_t)c * kRecTok * 4, m * 16, &rr.full[c % kRecStages]);
       });
     }
     return;
@@ -778,7 +870,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) s
   const bool vec = dv % 4 == 0;
   float S[R][VPT];
   load_state<KL, R, VPT>(S, st, kl, col, N, dv, ctx == n, vec);
-  const float D = p.D ? p.D[h] : 0.f;
+  const float D = !G && p.D ? p.D[h] : 0.f;
   const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + (kl & 7)) * p.ld_conv + (size_t)h * dv + col;
   auto send_group = [&](int c) {
     send_cols<T, VPT>(&s_v[warp][c % (kColsAhead + 1)][kl & 7][cg * VPT], vsrc + (size_t)c * kRecTok * p.ld_conv,
@@ -810,7 +902,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) s
         o.b[i4 * 4] = b4.x; o.b[i4 * 4 + 1] = b4.y; o.b[i4 * 4 + 2] = b4.z; o.b[i4 * 4 + 3] = b4.w;
         o.c[i4 * 4] = c4.x; o.c[i4 * 4 + 1] = c4.y; o.c[i4 * 4 + 2] = c4.z; o.c[i4 * 4 + 3] = c4.w;
       }
-      const float2 step = *reinterpret_cast<const float2*>(buf + kRecTok * REC + j * 4);      // dt, decay
+      const float2 step = G ? make_float2(1.f, 0.f) : *reinterpret_cast<const float2*>(buf + kRecTok * REC + j * 4);      // dt, decay
       o.dec = step.y;
 #pragma unroll
       for (int v = 0; v < VPT; ++v) o.x[v] = step.x * rc_ld(&cols[j][cg * VPT + v]);
@@ -822,7 +914,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) s
       for (int i = 0; i < R; ++i)
 #pragma unroll
         for (int v = 0; v < VPT; ++v) {
-          S[i][v] = fmaf(S[i][v], k.dec, k.b[i] * k.x[v]);
+          S[i][v] = G ? fmaf(S[i][v], k.b[i], (1.f - k.b[i]) * k.x[v]) : fmaf(S[i][v], k.dec, k.b[i] * k.x[v]);
           y[j][v] = fmaf(S[i][v], k.c[i], y[j][v]);
         }
     };
@@ -850,7 +942,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) s
     rr.release(c);
     spread_tokens<KL, VPT>(y, kl);
 #pragma unroll
-    for (int v = 0; v < VPT; ++v) y[0][v] = fmaf(D, rc_ld(&cols[kl & 7][cg * VPT + v]), y[0][v]);
+    for (int v = 0; v < VPT && !G; ++v) y[0][v] = fmaf(D, rc_ld(&cols[kl & 7][cg * VPT + v]), y[0][v]);
     if (kl < m) store_cols<VPT>(p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col, y[0], col, dv, vec);
   }
   if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<KL, R, VPT>(S, st, kl, col, N, dv, vec);
@@ -970,91 +1062,97 @@ __global__ void __launch_bounds__(256) group_norm_kernel(GroupNormParams p) {
 }
 
 // bf16: 4 neighbouring elements of the token's vectors can be read as one 64-bit word
-static int words_of_four(const RecParams& p, bool delta) {
+static int words_of_four(const RecParams& p, RecKind kind) {
   auto ok = [](const void* q, long long ld) { return (reinterpret_cast<uintptr_t>(q) & 7) == 0 && ld % 4 == 0; };
-  return ok(p.conv, p.ld_conv) && p.dk % 4 == 0 && p.dv % 4 == 0 && (!delta || ok(p.a, p.ld_a));
+  return ok(p.conv, p.ld_conv) && (kind == GATED || p.dk % 4 == 0) && p.dv % 4 == 0 && (kind != DELTA || ok(p.a, p.ld_a));
 }
 
-template <typename T, int DKP, bool DELTA>
+template <typename T, int DKP, RecKind K>
 static int launch_steps(const RecParams& p, int B, cudaStream_t s) {
   constexpr int KL = DKP <= 128 ? 8 : DKP / 16, R = DKP / KL, COLS = kRecWarps * (32 / KL) * 4;
   const int slices = (p.dv + COLS - 1) / COLS;
-  auto kern = DELTA ? delta_step_kernel<T, KL, R, 4> : state_space_step_kernel<T, KL, R, 4>;
-  kern<<<dim3(B * slices, p.heads), kRecWarps * 32, 0, s>>>(p, slices, words_of_four(p, DELTA));
+  auto kern = delta_step_kernel<T, KL, R, 4>;
+  if constexpr (K == SSM) kern = state_space_step_kernel<T, KL, R, 4>;
+  if constexpr (K == GATED) kern = gated_step_kernel<T, KL, R, 4>;
+  kern<<<dim3(B * slices, p.heads), kRecWarps * 32, 0, s>>>(p, slices, words_of_four(p, K));
   return (int)cudaGetLastError();
 }
-template <typename T, int DKP, bool DELTA>
+template <typename T, int DKP, RecKind K>
 static int launch_short_runs(const RecParams& p, int B, cudaStream_t s) {
   constexpr int R = DKP / 8, VPT = R > 32 ? 1 : (sizeof(T) == 4 || R > 16 ? 2 : 4), COLS = kRecWarps * 4 * VPT;
   const int slices = (p.dv + COLS - 1) / COLS;
-  const size_t smem = (size_t)2 * kRecTok * ((DELTA ? 3 : 2) * DKP + COLS + 4) * 4;
-  auto kern = DELTA ? delta_rule_kernel<T, R, VPT> : state_space_kernel<T, R, VPT>;
+  const size_t smem = (size_t)2 * kRecTok * ((K == DELTA ? 3 : 2) * DKP + COLS + 4) * 4;
+  void (*kern)(RecParams, int);
+  if constexpr (K == DELTA) kern = delta_rule_kernel<T, R, VPT>;
+  else kern = state_space_kernel<T, R, VPT, K == GATED>;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(kern, 200 * 1024);
   if (e != cudaSuccess) return (int)e;
   kern<<<dim3(B * slices, p.heads), kRecWarps * 32, smem, s>>>(p, slices);
   return (int)cudaGetLastError();
 }
-template <typename T, int KL, int R, int VPT, bool DELTA>
+template <typename T, int KL, int R, int VPT, RecKind K>
 static int launch_stream(const RecParams& p, int B, cudaStream_t s) {
   constexpr int COLS = kRecWarps * (32 / KL) * VPT;
   const int slices = (p.dv + COLS - 1) / COLS;
-  const size_t smem = kRecHead + (size_t)kRecStages * kRecTok * ((DELTA ? 3 : 2) * R * KL + 4) * 4;
+  const size_t smem = kRecHead + (size_t)kRecStages * kRecTok * ((K == DELTA ? 3 : 2) * R * KL + (K == GATED ? 0 : 4)) * 4;
   void (*kern)(RecParams, int, int);
-  if constexpr (DELTA) kern = delta_stream_kernel<T, KL, R, VPT>;
-  else kern = state_space_stream_kernel<T, KL, R, VPT>;
+  if constexpr (K == DELTA) kern = delta_stream_kernel<T, KL, R, VPT>;
+  else kern = state_space_stream_kernel<T, KL, R, VPT, K == GATED>;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(kern, 220 * 1024);
   if (e != cudaSuccess) return (int)e;
-  kern<<<dim3(B * slices, p.heads), (kRecWarps + 1) * 32, smem, s>>>(p, slices, words_of_four(p, DELTA));
+  kern<<<dim3(B * slices, p.heads), (kRecWarps + 1) * 32, smem, s>>>(p, slices, words_of_four(p, K));
   return (int)cudaGetLastError();
 }
 // 16 columns per warp keep the reductions and the shared-memory reads few; where that gives too few warps to fill the GPU, 4 columns
-template <typename T, int DKP, bool DELTA>
+template <typename T, int DKP, RecKind K>
 static int launch_long_runs(const RecParams& p, int B, cudaStream_t s) {
-  if constexpr (DELTA) delta_records_kernel<T, DKP><<<(unsigned)(((long long)p.T * p.heads + 3) / 4), 128, 0, s>>>(p);
+  const unsigned warps4 = (unsigned)(((long long)p.T * p.heads + 3) / 4);
+  if constexpr (K == DELTA) delta_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
+  else if constexpr (K == GATED) gated_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
   else state_space_records_kernel<T, DKP><<<p.T, 128, 0, s>>>(p);
   const int e = (int)cudaGetLastError();
   if (e) return e;
   if constexpr (sizeof(T) == 2 && DKP <= 128)
-    if ((long long)B * p.heads * ((p.dv + 15) / 16) >= 4LL * sm_count()) return launch_stream<T, 8, DKP / 8, 4, DELTA>(p, B, s);
+    if ((long long)B * p.heads * ((p.dv + 15) / 16) >= 4LL * sm_count()) return launch_stream<T, 8, DKP / 8, 4, K>(p, B, s);
   constexpr int KL = DKP >= 64 ? 16 : 8;
-  if constexpr (sizeof(T) == 2 && !DELTA && DKP <= 128)     // no reduction between tokens: 8 columns already at half the warps
-    if ((long long)B * p.heads * ((p.dv + 7) / 8) >= 2LL * sm_count()) return launch_stream<T, KL, DKP / KL, 4, DELTA>(p, B, s);
-  return launch_stream<T, KL, DKP / KL, 2, DELTA>(p, B, s);
+  if constexpr (sizeof(T) == 2 && K != DELTA && DKP <= 128)     // no reduction between tokens: 8 columns already at half the warps
+    if ((long long)B * p.heads * ((p.dv + 7) / 8) >= 2LL * sm_count()) return launch_stream<T, KL, DKP / KL, 4, K>(p, B, s);
+  return launch_stream<T, KL, DKP / KL, 2, K>(p, B, s);
 }
 
 // kinds: which sequences the step has, bit 0 = single tokens, 1 = short runs, 2 = long runs (with a workspace)
-template <typename T, int DKP, bool DELTA>
+template <typename T, int DKP, RecKind K>
 static int run_width(RecParams p, int B, int kinds, cudaStream_t s) {
   int e = 0;
-  if (kinds & 1) e = launch_steps<T, DKP, DELTA>(p, B, s);
-  if (!e && (kinds & 4)) e = launch_long_runs<T, DKP, DELTA>(p, B, s);
+  if (kinds & 1) e = launch_steps<T, DKP, K>(p, B, s);
+  if (!e && (kinds & 4)) e = launch_long_runs<T, DKP, K>(p, B, s);
   else p.long_rows = 0x7fffffff;
-  if (!e && (kinds & 2)) e = launch_short_runs<T, DKP, DELTA>(p, B, s);
+  if (!e && (kinds & 2)) e = launch_short_runs<T, DKP, K>(p, B, s);
   return e;
 }
 
 static int padded_dk(int dk) { return dk <= 32 ? 32 : dk <= 64 ? 64 : dk <= 128 ? 128 : dk <= 256 ? 256 : 512; }
-static long long record_bytes(bool delta, long long T, int heads, int groups, int dk) {
+static long long record_bytes(RecKind kind, long long T, int heads, int groups, int dk) {
   const long long n = padded_dk(dk);
-  return 4 * (delta ? heads * T * (3 * n + 4) : groups * T * 2 * n + heads * T * 4);
+  return 4 * (kind == DELTA ? heads * T * (3 * n + 4) : kind == GATED ? heads * T * 2 * n : groups * T * 2 * n + heads * T * 4);
 }
 
-template <typename T, bool DELTA>
+template <typename T, RecKind K>
 static int run_rec(const RecParams& p, int B, int kinds, long long ws_bytes, cudaStream_t s) {
   if (B == 0) return 0;
   if (B < 0 || p.heads < 1 || p.heads > 65535 || p.groups < 1 || p.heads % p.groups || p.dk < 1 || p.dk > 512 || p.dv < 1)
     return (int)cudaErrorInvalidValue;
-  if ((kinds & 4) && (!p.records || !p.out || !p.seq_of_row || p.T < 1 || ws_bytes < record_bytes(DELTA, p.T, p.heads, p.groups, p.dk) ||
+  if ((kinds & 4) && (!p.records || !p.out || !p.seq_of_row || p.T < 1 || ws_bytes < record_bytes(K, p.T, p.heads, p.groups, p.dk) ||
                       (reinterpret_cast<uintptr_t>(p.records) & 15)))
     return (int)cudaErrorInvalidValue;
   switch (padded_dk(p.dk)) {
-    case 32: return run_width<T, 32, DELTA>(p, B, kinds, s);
-    case 64: return run_width<T, 64, DELTA>(p, B, kinds, s);
-    case 128: return run_width<T, 128, DELTA>(p, B, kinds, s);
-    case 256: return run_width<T, 256, DELTA>(p, B, kinds, s);
-    default: return run_width<T, 512, DELTA>(p, B, kinds, s);
+    case 32: return run_width<T, 32, K>(p, B, kinds, s);
+    case 64: return run_width<T, 64, K>(p, B, kinds, s);
+    case 128: return run_width<T, 128, K>(p, B, kinds, s);
+    case 256: return run_width<T, 256, K>(p, B, kinds, s);
+    default: return run_width<T, 512, K>(p, B, kinds, s);
   }
 }
 
@@ -1063,9 +1161,9 @@ static int run_rec(const RecParams& p, int B, int kinds, long long ws_bytes, cud
 // Runs of at least this many new tokens are long runs where the caller gives a workspace.
 static constexpr int kLongRows = 32;
 BLZ_API int blz_rec_long_rows() { return kLongRows; }
-// Workspace bytes of a step of T rows (delta: 1 = blz_delta_rule, 0 = blz_state_space).
-BLZ_API long long blz_rec_ws_bytes(int delta, int T, int heads, int groups, int dk) {
-  return blz::record_bytes(delta != 0, T, heads, groups, dk);
+// Workspace bytes of a step of T rows (kind: 0 = blz_state_space, 1 = blz_delta_rule, 2 = blz_gated_linear).
+BLZ_API long long blz_rec_ws_bytes(int kind, int T, int heads, int groups, int dk) {
+  return blz::record_bytes(kind == 1 ? blz::DELTA : kind == 2 ? blz::GATED : blz::SSM, T, heads, groups, dk);
 }
 
 // Delta rule with channel decays over every sequence of the batch (see RecParams; leading dimensions in elements; conv channels
@@ -1079,7 +1177,7 @@ BLZ_API int blz_delta_rule(const void* conv, long long ld_conv, const void* a, l
   using namespace blz;
   const RecParams p = {conv, a, b, A, dt_bias, nullptr, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_a, ld_b, heads, key_heads,
                        dk, dv, seq_of_row, ws, T, kLongRows, status_word()};
-  return f32 ? run_rec<float, true>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, true>(p, B, kinds, ws_bytes, s);
+  return f32 ? run_rec<float, DELTA>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, DELTA>(p, B, kinds, ws_bytes, s);
 }
 
 // State-space duality (conv channels [x heads * dv | B groups * N | C groups * N]); other arguments as above.  N <= 512.
@@ -1090,7 +1188,19 @@ BLZ_API int blz_state_space(const void* conv, long long ld_conv, const void* dt,
   using namespace blz;
   const RecParams p = {conv, dt, nullptr, A, dt_bias, D, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_dt, 0, heads, groups,
                        N, dv, seq_of_row, ws, T, kLongRows, status_word()};
-  return f32 ? run_rec<float, false>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, false>(p, B, kinds, ws_bytes, s);
+  return f32 ? run_rec<float, SSM>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, SSM>(p, B, kinds, ws_bytes, s);
+}
+
+// Gated linear attention: q and f_raw [T, heads * dk], v [T, heads * dv] (runs of columns), lower bounds and biases [heads * dk] fp32;
+// other arguments as above.  dk <= 512.
+BLZ_API int blz_gated_linear(const void* q, long long ld_q, const void* f, long long ld_f, const void* v, long long ld_v, const float* lower,
+                             const float* bias, float* state, float* out, const int* slots, const int* q_start, const int* ctx_len,
+                             const int* no_store, int B, int heads, int dk, int dv, const int* seq_of_row, int T, int kinds, float* ws,
+                             long long ws_bytes, int f32, cudaStream_t s) {
+  using namespace blz;
+  const RecParams p = {v, f, q, lower, bias, nullptr, state, out, slots, q_start, ctx_len, no_store, ld_v, ld_f, ld_q, heads, heads,
+                       dk, dv, seq_of_row, ws, T, kLongRows, status_word()};
+  return f32 ? run_rec<float, GATED>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, GATED>(p, B, kinds, ws_bytes, s);
 }
 
 // RMS norm of each of `groups` runs of n columns of fp32 rows, with a gate (GroupNormParams), to the activation type.

@@ -6,7 +6,8 @@
 // the next sublayer's input from the new streams and RMS-normalises it, so that the fp32 streams make one trip through HBM
 // per sublayer.  Before the first sublayer all streams equal the scaled embedding row, which is read from the table
 // (`from_embed`) instead of being copied S times; after the last one only the sum of the streams is written.
-// Beside them: the norm of fp32 rows, and the residual sum of a post-norm decoder (residual_norm_kernel).
+// Beside them: the norm of fp32 rows, the residual sum of a post-norm decoder (residual_norm_kernel), the residual that takes
+// normed branches (branch_norm_kernel), and the causal convolution of a residual over time (input_conv_kernel).
 // One CTA per row; the row's columns stay with their thread (float4 where the width allows), so the update is in place.
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
@@ -172,20 +173,29 @@ __global__ void __launch_bounds__(512) streams_kernel(StreamsParams p) {
   }
 }
 
-// RMS norm of fp32 rows (the rows named by `rows`, or all) to the activation type.
+// RMS norm (centre: layer norm) of fp32 rows (the rows named by `rows`, or all) to the activation type.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(512) norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows,
-                                                        const float* __restrict__ w, T* __restrict__ out, int W, float eps) {
-  __shared__ float red[16];
+                                                        const float* __restrict__ w, T* __restrict__ out, int W, float eps, int centre) {
+  __shared__ float red[16], red1[16];
   pdl_trigger();
   pdl_wait();
   const float* xr = x + (size_t)(rows ? rows[blockIdx.x] : blockIdx.x) * W;
-  float ss = 0.f;
+  float ss = 0.f, mean = 0.f;
+  if (centre) {
+    for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+      float v[VEC];
+      ld_vec<VEC>(xr + c, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) mean += v[j];
+    }
+    mean = block_sum(mean, red1) / (float)W;
+  }
   for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
     float v[VEC];
     ld_vec<VEC>(xr + c, v);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) ss = fmaf(v[j], v[j], ss);
+    for (int j = 0; j < VEC; ++j) ss = fmaf(v[j] - mean, v[j] - mean, ss);
   }
   const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
   T* o = out + (size_t)blockIdx.x * W;
@@ -194,7 +204,7 @@ __global__ void __launch_bounds__(512) norm_rows_kernel(const float* __restrict_
     ld_vec<VEC>(xr + c, v);
     ld_vec<VEC>(w + c, g);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) v[j] = v[j] * rs * g[j];
+    for (int j = 0; j < VEC; ++j) v[j] = (v[j] - mean) * rs * g[j];
     st_vec<VEC>(o + c, v);
   }
 }
@@ -231,6 +241,222 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(const X* __restrict_
     st_vec<VEC>(x + at + c, u);
     if (h) st_vec<VEC>(h + at + c, u);
   }
+}
+
+// A branch into an fp32 residual: x <- x + layer_norm(branch) * w, with a copy in the activation type (h, may be null).  The branch is
+// a row of y; or (ROUTED) the weighted sum of the k rows of y that row_map names (-1: none) plus, if there is one, a row of `extra`;
+// or (EMBED) the token's row of a table, and x is then the normed row alone.
+enum BranchSrc { ROWS, ROUTED, EMBED };
+struct BranchParams {
+  const void* y;               // [.., ldy] activation type
+  const void* extra;           // [T, W]
+  const float* weights;        // [T, k]
+  const int* row_map;          // [T, k], or (EMBED) tokens [T]
+  const float* w;              // [W]
+  float* x;                    // [T, W]
+  void* h;
+  long long ldy;
+  int k, W, vocab;
+  float eps;
+};
+
+template <typename T, int VEC, BranchSrc SRC>
+__global__ void __launch_bounds__(512) branch_norm_kernel(BranchParams p) {
+  extern __shared__ float u_row[];                   // [W]
+  __shared__ float red0[16], red1[16], s_w[32];
+  __shared__ int s_row[32];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, W = p.W;
+  const size_t at = (size_t)t * W;
+  const T* y = reinterpret_cast<const T*>(p.y);
+  if constexpr (SRC == ROUTED) {
+    if (threadIdx.x < p.k) {
+      s_w[threadIdx.x] = p.weights[(size_t)t * p.k + threadIdx.x];
+      s_row[threadIdx.x] = p.row_map[(size_t)t * p.k + threadIdx.x];
+    }
+    __syncthreads();
+  } else if constexpr (SRC == EMBED) {
+    const int tok = p.row_map[t];
+    y += (size_t)(tok < 0 ? 0 : tok >= p.vocab ? p.vocab - 1 : tok) * p.ldy;
+  } else {
+    y += (size_t)t * p.ldy;
+  }
+  float sum = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float u[VEC];
+    if constexpr (SRC == ROUTED) {
+      if (p.extra) {
+        ld_vec<VEC>(reinterpret_cast<const T*>(p.extra) + at + c, u);
+      } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) u[j] = 0.f;
+      }
+      for (int i = 0; i < p.k; ++i) {
+        if (s_row[i] < 0) continue;
+        float v[VEC];
+        ld_vec<VEC>(y + (size_t)s_row[i] * p.ldy + c, v);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) u[j] = fmaf(s_w[i], v[j], u[j]);
+      }
+    } else {
+      ld_vec<VEC>(y + c, u);
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) sum += u[j];
+    st_vec<VEC>(u_row + c, u);
+  }
+  const float mean = block_sum(sum, red0) / (float)W;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float u[VEC];
+    ld_vec<VEC>(u_row + c, u);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) ss = fmaf(u[j] - mean, u[j] - mean, ss);
+  }
+  const float rs = 1.f / sqrtf(block_sum(ss, red1) / (float)W + p.eps);
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float u[VEC], g[VEC], x[VEC];
+    ld_vec<VEC>(u_row + c, u);
+    ld_vec<VEC>(p.w + c, g);
+    if constexpr (SRC != EMBED) ld_vec<VEC>(p.x + at + c, x);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) u[j] = SRC == EMBED ? (u[j] - mean) * rs * g[j] : fmaf((u[j] - mean) * rs, g[j], x[j]);
+    st_vec<VEC>(p.x + at + c, u);
+    if (p.h) st_vec<VEC>(reinterpret_cast<T*>(p.h) + at + c, u);
+  }
+}
+
+// h = x + conv(x): a causal convolution of every column over a sequence's rows, whose earlier inputs are in the sequence's state row.
+// A thread takes VEC columns of up to kConvSeg rows of one sequence; a longer run's state is written by a kernel of its own (its first
+// segment reads the old one).  TAPS = 0: any number, read again for every row.
+static constexpr int kConvSeg = 32;
+struct InputConvParams {
+  const float* x;              // [T, W]
+  void* h;                     // [T, W] activation type, or null (the state only)
+  float* state;                // [rows, taps - 1, W]
+  const float* w;              // [taps, W]
+  const int *slots, *q_start, *ctx_len, *no_store;
+  int W, taps;
+};
+
+template <typename T, int TAPS, int VEC>
+__global__ void __launch_bounds__(128) input_conv_kernel(InputConvParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = (blockIdx.x * 128 + threadIdx.x) * VEC, b = blockIdx.y, W = p.W, taps = TAPS ? TAPS : p.taps;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, t0 = blockIdx.z * kConvSeg, t1 = min(n, t0 + kConvSeg);
+  if (c >= W || t0 >= n) return;
+  const bool fresh = p.ctx_len[b] == n;
+  float* st = p.state + (size_t)p.slots[b] * (taps - 1) * W + c;
+  const float* x = p.x + (size_t)r0 * W + c;
+  auto input = [&](int t, float (&v)[VEC]) {         // input of position t of this run (negative: before it)
+    if (t >= 0) {
+      ld_vec<VEC>(x + (size_t)t * W, v);
+    } else if (!fresh) {
+      ld_vec<VEC>(st + (size_t)(taps - 1 + t) * W, v);
+    } else {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] = 0.f;
+    }
+  };
+  T* h = reinterpret_cast<T*>(p.h) + (size_t)r0 * W + c;
+  if constexpr (TAPS == 0) {
+    for (int t = t0; t < t1 && p.h; ++t) {
+      float y[VEC], v[VEC], g[VEC];
+      input(t, y);
+      for (int i = 0; i < taps; ++i) {
+        input(t - taps + 1 + i, v);
+        ld_vec<VEC>(p.w + (size_t)i * W + c, g);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) y[j] = fmaf(g[j], v[j], y[j]);
+      }
+      st_vec<VEC>(h + (size_t)t * W, y);
+    }
+  } else {
+    float v[TAPS][VEC], g[TAPS][VEC];
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) ld_vec<VEC>(p.w + (size_t)i * W + c, g[i]);
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i) input(t0 - TAPS + 1 + i, v[i]);
+    constexpr int AHEAD = 4;                         // rows in flight
+    for (int t = t0; t < t1; t += AHEAD) {
+      float in[AHEAD][VEC];
+#pragma unroll
+      for (int k = 0; k < AHEAD; ++k)
+        if (t + k < t1) ld_vec<VEC>(x + (size_t)(t + k) * W, in[k]);
+#pragma unroll
+      for (int k = 0; k < AHEAD; ++k) {
+        if (t + k >= t1) break;
+        float y[VEC];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          v[TAPS - 1][j] = y[j] = in[k][j];
+#pragma unroll
+          for (int i = 0; i < TAPS; ++i) y[j] = fmaf(g[i][j], v[i][j], y[j]);
+#pragma unroll
+          for (int i = 0; i < TAPS - 1; ++i) v[i][j] = v[i + 1][j];
+        }
+        if (p.h) st_vec<VEC>(h + (size_t)(t + k) * W, y);
+      }
+    }
+    if (n > kConvSeg || (p.no_store != nullptr && p.no_store[b])) return;
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i) st_vec<VEC>(st + (size_t)i * W, v[i]);
+  }
+}
+
+// the state after a run of more than min_rows rows
+template <int VEC>
+__global__ void __launch_bounds__(128) input_conv_state_kernel(InputConvParams p, int min_rows) {
+  const int c = (blockIdx.x * 128 + threadIdx.x) * VEC, b = blockIdx.y, W = p.W;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
+  if (c >= W || n <= min_rows || (p.no_store != nullptr && p.no_store[b])) return;
+  const bool fresh = p.ctx_len[b] == n;
+  float* st = p.state + (size_t)p.slots[b] * (p.taps - 1) * W + c;
+  for (int i = 0; i < p.taps - 1; ++i) {             // entry i: input n - (taps - 1) + i, an older entry where the run is shorter
+    const int t = n - p.taps + 1 + i;
+    float v[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] = 0.f;
+    if (t >= 0) ld_vec<VEC>(p.x + (size_t)(r0 + t) * W + c, v);
+    else if (!fresh) ld_vec<VEC>(st + (size_t)(i + n) * W, v);
+    st_vec<VEC>(st + (size_t)i * W, v);
+  }
+}
+
+template <typename T, int VEC>
+static int launch_input_conv(const InputConvParams& p, int B, int max_q, cudaStream_t s) {
+  const dim3 grid((p.W + 128 * VEC - 1) / (128 * VEC), B, (max_q + kConvSeg - 1) / kConvSeg);
+  cudaError_t e;
+  switch (p.taps) {
+#define BLZ_IC(K) case K: e = launch_pdl(input_conv_kernel<T, K, VEC>, grid, dim3(128), 0, s, p); break
+    BLZ_IC(1); BLZ_IC(2); BLZ_IC(3); BLZ_IC(4); BLZ_IC(5); BLZ_IC(6); BLZ_IC(7); BLZ_IC(8);
+    default: e = launch_pdl(input_conv_kernel<T, 0, VEC>, grid, dim3(128), 0, s, p);
+#undef BLZ_IC
+  }
+  if (e != cudaSuccess) return (int)e;
+  const int min_rows = p.taps > 8 ? 0 : kConvSeg;
+  if (p.taps > 1 && max_q > min_rows) input_conv_state_kernel<VEC><<<dim3(grid.x, B), 128, 0, s>>>(p, min_rows);
+  return (int)cudaGetLastError();
+}
+
+static int row_threads(int W, int vec);
+template <BranchSrc SRC>
+static int launch_branch(const BranchParams& p, int T, int f32, int vec, cudaStream_t s) {
+  const dim3 block(row_threads(p.W, vec ? 4 : 1));
+  const size_t sm = (size_t)p.W * 4;
+#define BLZ_BN(TT, V)                                                                   \
+  do {                                                                                  \
+    static PerDeviceOnce once;                                                          \
+    const cudaError_t e = once.smem_limit(branch_norm_kernel<TT, V, SRC>, 200 * 1024);  \
+    if (e != cudaSuccess) return (int)e;                                                \
+    return (int)launch_pdl(branch_norm_kernel<TT, V, SRC>, dim3(T), block, sm, s, p);   \
+  } while (0)
+  if (f32) { if (vec) BLZ_BN(float, 4); BLZ_BN(float, 1); }
+  if (vec) BLZ_BN(__nv_bfloat16, 4);
+  BLZ_BN(__nv_bfloat16, 1);
+#undef BLZ_BN
 }
 
 static int row_threads(int W, int vec) {
@@ -289,15 +515,16 @@ BLZ_API int blz_streams(float* streams, const void* table, const int* tokens, in
   return (int)(f32 ? pick_streams<float>(p, T, s) : pick_streams<__nv_bfloat16>(p, T, s));
 }
 
-BLZ_API int blz_norm_rows(const float* x, const int* rows, const float* w, void* out, int R, int W, float eps, int f32, cudaStream_t s) {
+BLZ_API int blz_norm_rows(const float* x, const int* rows, const float* w, void* out, int R, int W, float eps, int centre, int f32,
+                          cudaStream_t s) {
   using namespace blz;
   if (R <= 0 || W < 1) return (int)cudaErrorInvalidValue;
   const bool v4 = W % 4 == 0;
   const dim3 g(R), b(row_threads(W, v4 ? 4 : 1));
-  if (f32) return (int)(v4 ? launch_pdl(norm_rows_kernel<float, 4>, g, b, 0, s, x, rows, w, (float*)out, W, eps)
-                           : launch_pdl(norm_rows_kernel<float, 1>, g, b, 0, s, x, rows, w, (float*)out, W, eps));
-  return (int)(v4 ? launch_pdl(norm_rows_kernel<__nv_bfloat16, 4>, g, b, 0, s, x, rows, w, (__nv_bfloat16*)out, W, eps)
-                  : launch_pdl(norm_rows_kernel<__nv_bfloat16, 1>, g, b, 0, s, x, rows, w, (__nv_bfloat16*)out, W, eps));
+  if (f32) return (int)(v4 ? launch_pdl(norm_rows_kernel<float, 4>, g, b, 0, s, x, rows, w, (float*)out, W, eps, centre)
+                           : launch_pdl(norm_rows_kernel<float, 1>, g, b, 0, s, x, rows, w, (float*)out, W, eps, centre));
+  return (int)(v4 ? launch_pdl(norm_rows_kernel<__nv_bfloat16, 4>, g, b, 0, s, x, rows, w, (__nv_bfloat16*)out, W, eps, centre)
+                  : launch_pdl(norm_rows_kernel<__nv_bfloat16, 1>, g, b, 0, s, x, rows, w, (__nv_bfloat16*)out, W, eps, centre));
 }
 
 // x [T, W] fp32 <- norm(alpha * from + y) with the norm's weight w; h [T, W] (activation type, or null) gets a copy.  from_act: `from`
@@ -313,4 +540,34 @@ BLZ_API int blz_residual_norm(const void* from, int from_act, float alpha, const
   if (from_act) { BLZ_RN(__nv_bfloat16, __nv_bfloat16); }
   BLZ_RN(__nv_bfloat16, float);
 #undef BLZ_RN
+}
+
+// x [T, W] fp32 <- x + layer_norm(branch) * w, h (activation type, or null) a copy; the branch: rows of y [T, ldy], or (row_map) the sums
+// of weights[t, i] * y[row_map[t, i]], i < k <= 32, and of extra [T, W] (or null).  W <= 51200.
+BLZ_API int blz_branch_norm(const void* y, long long ldy, const float* weights, const int* row_map, int k, const void* extra, const float* w,
+                            float eps, float* x, void* h, int T, int W, int f32, cudaStream_t s) {
+  using namespace blz;
+  if (T <= 0 || W < 1 || W > 51200 || !y || !w || !x || (row_map && (!weights || k < 1 || k > 32))) return (int)cudaErrorInvalidValue;
+  BranchParams p = {y, extra, weights, row_map, w, x, h, ldy, k, W, 0, eps};
+  const int vec = W % 4 == 0 && ldy % 4 == 0;
+  return row_map ? launch_branch<ROUTED>(p, T, f32, vec, s) : launch_branch<ROWS>(p, T, f32, vec, s);
+}
+
+// x [T, W] fp32 = layer_norm(table[token]) * w.
+BLZ_API int blz_embed_norm(const void* table, const int* tokens, int vocab, const float* w, float eps, float* x, int T, int W, int f32,
+                           cudaStream_t s) {
+  using namespace blz;
+  if (T <= 0 || W < 1 || W > 51200 || vocab < 1 || !table || !tokens || !w || !x) return (int)cudaErrorInvalidValue;
+  const BranchParams p = {table, nullptr, nullptr, tokens, w, x, nullptr, W, 0, W, vocab, eps};
+  return launch_branch<EMBED>(p, T, f32, W % 4 == 0, s);
+}
+
+// See InputConvParams; max_q: the longest run of the batch.  no_store: optional [B], 1 = leave the sequence's state as it was.
+BLZ_API int blz_input_conv(const float* x, void* h, float* state, const float* w, const int* slots, const int* q_start, const int* ctx_len,
+                           const int* no_store, int B, int W, int taps, int max_q, int f32, cudaStream_t s) {
+  using namespace blz;
+  if (B < 1 || B > 65535 || W < 1 || taps < 1 || max_q < 1 || !x || !w || (taps > 1 && !state)) return (int)cudaErrorInvalidValue;
+  const InputConvParams p = {x, h, state, w, slots, q_start, ctx_len, no_store, W, taps};
+  if (f32) return W % 4 == 0 ? launch_input_conv<float, 4>(p, B, max_q, s) : launch_input_conv<float, 1>(p, B, max_q, s);
+  return W % 4 == 0 ? launch_input_conv<__nv_bfloat16, 4>(p, B, max_q, s) : launch_input_conv<__nv_bfloat16, 1>(p, B, max_q, s);
 }

@@ -1,0 +1,356 @@
+"""The Rapisun design's kernels on a B200 against the independent restatement in ``oracle_rapisun.py``: each mechanism alone over
+many sizes, then whole models in bf16 and fp32 through the engine and the scheduler."""
+import pytest
+import torch
+
+import oracle_rapisun as O
+import rapisun_case as C
+from test_niletar_gpu import LENS, SIZES, Sequences, rel, schedule
+from test_sevevik_cpu import SCHEDULES, mixed_steps
+
+pytestmark = pytest.mark.gpu
+DEV = "cuda"
+TYPES = [torch.float32, torch.bfloat16]
+
+
+@pytest.fixture(scope="module")
+def ops():
+    from blaze_b200.ops import get_ops
+    return get_ops(DEV)
+
+
+def rnd(*s, seed=0):
+    return torch.randn(*s, generator=torch.Generator().manual_seed(seed))
+
+
+# ----------------------------------------------------------------------------------- residual, norms, convolution
+@pytest.mark.parametrize("dtype", TYPES)
+@pytest.mark.parametrize("T,W", [(1, 64), (5, 100), (3, 257), (37, 512), (2, 4096), (300, 2048)])
+def test_normed_branches(ops, T, W, dtype):
+    x, y, w = rnd(T, W) * 3, (rnd(T, W, seed=1) + 2).to(dtype), rnd(W, seed=2)
+    want = x.double() + O.layer_norm(y.double(), w.double(), 1e-3)
+    got, h = ops.branch_norm(x.to(DEV), y.to(DEV), w.to(DEV), 1e-3)
+    assert got.dtype == torch.float32 and h.dtype == dtype and rel(got, want) < 1e-6 and rel(h, want) < (1e-6 if dtype == torch.float32 else 8e-3)
+    assert ops.branch_norm(x.to(DEV), y.to(DEV), w.to(DEV), 1e-3, copy=False)[1] is None
+    rows = torch.tensor([T - 1, 0], dtype=torch.int32)
+    got = ops.norm_rows(x.to(DEV), rows.to(DEV), w.to(DEV), 1e-3, torch.float32, centre=True)
+    assert rel(got, O.layer_norm(x[rows.long()].double(), w.double(), 1e-3)) < 1e-6
+    table, tok = rnd(50, W, seed=3).to(dtype), torch.randint(0, 50, (T,), generator=torch.Generator().manual_seed(T)).int()
+    assert rel(ops.embed_norm(table.to(DEV), tok.to(DEV), w.to(DEV), 1e-3), O.layer_norm(table[tok.long()].double(), w.double(), 1e-3)) < 1e-6
+
+
+@pytest.mark.parametrize("dtype", TYPES)
+@pytest.mark.parametrize("taps,W", [(1, 40), (2, 33), (3, 300), (4, 128), (5, 1024), (8, 65), (11, 36), (40, 24)])
+def test_input_convolution(ops, taps, W, dtype):
+    from blaze_b200.config import LayerSpec, GatedLinearSpec
+    S = Sequences(LayerSpec(rec=GatedLinearSpec(1, 8, 8)), dtype)
+    if taps > 1:
+        S.kv.input_state = {0: torch.full((8, taps - 1, W), 3.0, device=DEV)}
+    w = rnd(W, taps, seed=taps)
+    x = {b: rnd(n, W, seed=b) for b, n in LENS.items()}
+    got = {b: [] for b in LENS}
+    for k, step in enumerate(schedule(LENS, SIZES, late=(2, 5))):
+        ents, rows = [(b, n) for b, _, n in step], torch.cat([x[b][p:p + n] for b, p, n in step]).to(DEV)
+        wt = w.t().contiguous().to(DEV)
+        if k % 2:                            # the same rows once more with the state kept as it was
+            ops.input_conv(rows, wt, S.batch(ents, defer=[b for b, _ in ents]), S.kv, 0, dtype)
+        h = ops.input_conv(rows, wt, S.batch(ents), S.kv, 0, dtype).cpu()
+        for (b, _, _), o in zip(step, h.split([n for _, _, n in step])):
+            got[b].append(o)
+    for b in LENS:
+        assert rel(torch.cat(got[b]), O.input_conv(x[b].double(), w.double())) < (1e-6 if dtype == torch.float32 else 8e-3), b
+
+
+# ----------------------------------------------------------------------------------- feed-forwards
+@pytest.mark.parametrize("dtype", TYPES)
+@pytest.mark.parametrize("T,I", [(1, 96), (5, 40), (70, 512), (3, 33), (2, 6144)])
+def test_activations_without_a_gate(ops, T, I, dtype):
+    z, act = (rnd(T, I) * 1.7 + 0.3).to(dtype), torch.tensor([0.7, -0.4, 1.3, 0.25])
+    tol = 2e-6 if dtype == torch.float32 else 8e-3
+    assert rel(ops.poly_norm(z.to(DEV), act.to(DEV), 1e-2), O.poly_norm(z.double(), act.double(), 1e-2)) < tol
+    assert rel(ops.relu2_(z.to(DEV)), O.squared_relu(z.double())) < tol
+
+
+@pytest.mark.parametrize("dtype", TYPES)
+@pytest.mark.parametrize("T,W,E,top,ff,shared", [(1, 64, 4, 1, 48, 32), (9, 144, 6, 2, 40, 56), (70, 100, 5, 5, 24, 0), (300, 256, 12, 4, 96, 128),
+                                                 (37, 512, 33, 6, 256, 0), (600, 128, 3, 1, 64, 64), (2, 81, 7, 2, 33, 0)])
+def test_routed_experts(ops, T, W, E, top, ff, shared, dtype):
+    from blaze_b200.config import GatedLinearSpec, LayerSpec, ModelConfig, MoeSpec
+    from blaze_b200.models.rapisun import Rapisun
+    L = C.hgrn2(C.moe(E, top, ff, shared), 1, 8, 8)
+    cfg = C.config([L], width=W, vocab=64)
+    w = C.weights(cfg, seed=E)
+    m = Rapisun(ModelConfig.from_json(cfg), DEV, dtype, ops=ops)._assemble(lambda n, s: w[n])
+    h, x, nw = rnd(T, W).to(dtype), rnd(T, W, seed=1), rnd(W, seed=2)
+    y, _ = m._mlp(m.layers[0].mlp, h.to(DEV))
+    got, _ = ops.branch_norm(x.to(DEV), y, nw.to(DEV), 1e-4, copy=False)
+    wd = {n: t.double() for n, t in w.items()}
+    out = O.mixture(h.double(), wd, "l0.mlp.", L["mlp"])
+    want = x.double() + O.layer_norm(out, nw.double(), 1e-4)
+    assert rel(got, want) < (1e-5 if dtype == torch.float32 else 2e-2)
+
+
+# ----------------------------------------------------------------------------------- gated linear attention
+GATED = [(2, 20, 28), (6, 32, 16), (4, 64, 64), (3, 128, 128), (8, 96, 40), (2, 160, 24), (1, 300, 9), (4, 8, 200), (1, 500, 6), (5, 17, 33)]
+
+
+def run_gated(ops, sizes, dtype, lens, sched, late=()):
+    from blaze_b200.config import GatedLinearSpec, LayerSpec
+    from blaze_b200.models.qwen3 import Mixer, Recurrence
+    H, d, e = sizes
+    spec, M = GatedLinearSpec(H, d, e), Mixer()
+    R = M.rec = Recurrence(spec, "gated", H)
+    up = lambda n: (n + 7) // 8 * 8      # noqa: E731
+    M.cols = {"q": 0, "f": up(H * d), "v": 2 * up(H * d)}
+    R.A, R.dt_bias = torch.sigmoid(rnd(H * d, seed=1) * 3).to(DEV), (rnd(H * d, seed=2) * 2 + 2).to(DEV)
+    S = Sequences(LayerSpec(rec=spec), dtype)
+    proj = {b: (rnd(n, 2 * up(H * d) + up(H * e), seed=10 + b) * 1.5).to(dtype) for b, n in lens.items()}
+    got = {b: [] for b in lens}
+    for k, step in enumerate(schedule(lens, sched, late)):
+        ents, rows = [(b, n) for b, _, n in step], torch.cat([proj[b][p:p + n] for b, p, n in step]).to(DEV)
+        out = torch.full((rows.shape[0], H * e), float("nan"), device=DEV)
+        if k % 2:                            # the same rows once more with the state kept as it was
+            ops.recur(None, rows, None, M, S.batch(ents, defer=[b for b, _ in ents]), S.kv, 0, None)
+        ops.recur(None, rows, None, M, S.batch(ents), S.kv, 0, out)
+        for (b, p, n), o in zip(step, out.cpu().split([n for _, _, n in step])):
+            got[b].append(o)
+            if p + n == lens[b]:
+                S.free(b)
+    want = {}
+    for b, n in lens.items():
+        q, f, v = (proj[b].double()[:, M.cols[c]:][:, :H * k].view(n, H, k) for c, k in (("q", d), ("f", d), ("v", e)))
+        f = O.forget_gate(f + R.dt_bias.double().cpu().view(H, d), R.A.double().cpu().view(H, d))
+        want[b] = torch.cat([O.gated_linear(O.silu(q[:, h]), f[:, h], v[:, h]) for h in range(H)], 1)
+    return {b: torch.cat(got[b]) for b in lens}, want
+
+
+@pytest.mark.parametrize("dtype", TYPES)
+@pytest.mark.parametrize("sizes", GATED)
+def test_gated_linear(ops, sizes, dtype):
+    got, want = run_gated(ops, sizes, dtype, LENS, SIZES, late=(2, 5))
+    for b in LENS:
+        assert rel(got[b], want[b]) < 1e-5, b            # fp32 inside for either type: inputs are exact
+
+
+def test_gated_linear_with_many_sequences(ops):
+    for count, n in ((1, 70), (4, 60), (8, 40)):
+        lens = {b: n + 3 * b for b in range(count)}
+        got, want = run_gated(ops, (32, 64, 64), torch.bfloat16, lens, {b: [33, 1, 17] for b in lens})
+        for b in lens:
+            assert rel(got[b], want[b]) < 1e-5, (count, b)
+
+
+# ----------------------------------------------------------------------------------- latent attention alone
+# heads, dim, rotated, vdim, latent, window
+ATTN = [(4, 24, 8, 40, 48, 20), (8, 64, 16, 64, 128, 72), (1, 16, 16, 16, 16, 5), (5, 12, 6, 20, 36, 0), (16, 32, 32, 64, 256, 50), (40, 64, 32, 64, 256, 100),
+        (20, 16, 64, 128, 512, 33), (3, 128, 64, 128, 96, 130), (2, 40, 24, 24, 130, 17), (6, 160, 48, 144, 200, 64), (64, 8, 8, 16, 32, 128), (2, 20, 10, 18, 600, 40)]
+PORTIONS = {"whole": [10 ** 6], "pairs and more": [2, 37, 3, 130, 1, 16, 17], "decode": [190] + [1] * 30, "small": [5, 16, 2, 11, 1]}
+
+
+class LatentLayer:
+    """A latent attention fed rows of [queries | latent | rotated part] (the queries' map is the identity); a second layer reads the
+    first one's latents with maps, sizes and a window of its own."""
+
+    def __init__(self, ops, case, dtype, second=False):
+        from blaze_b200.config import LatentAttnSpec, LayerSpec, ModelConfig, RotarySpec
+        from blaze_b200.linear import Linear
+        from blaze_b200.models.qwen3 import LatentAttn, Mixer
+        H, d, r, e, R, win = case
+        self.rot = {"dims": r, "base": 300.0}
+        spec = lambda **kw: LatentAttnSpec(**{**dict(heads=H, dim=d, rot_dim=r, vdim=e, q_rank=H * (d + r), kv_rank=R, scale=2.0 / (d + r) ** 0.5,     # noqa: E731
+                                                     rot=RotarySpec(r, 300.0, False), sink=True, window=win), **kw})
+        self.a = spec() if not second else spec(heads=H + 1, vdim=e + 8, q_rank=(H + 1) * (d + r), window=win + 7, kv_from=0)
+        a = self.a
+        self.M, self.ops, self.dtype = Mixer(), ops, dtype
+        A = self.M.attn = LatentAttn(a, DEV)
+        self.sink = rnd(a.heads, seed=d) * 2 + 1
+        A.sink, A.q_norm, A.c_norm = self.sink.to(DEV), torch.ones(a.q_rank, device=DEV), (rnd(R, seed=5) * 0.3 + 1).to(DEV)
+        A.uq = Linear.from_dense(torch.eye(a.q_rank, device=DEV), dtype=dtype)
+        uk, uv = [(rnd(a.heads * k, R, seed=6 + k) * R ** -0.5).to(DEV) for k in (d, e)]
+        A.set_maps(uk, uv, dtype)
+        self.at = (a.q_rank + 7) // 8 * 8
+        self.M.cols = {"q": 0, "kv": self.at}
+        self.width = (self.at + R + r + 7) // 8 * 8
+        self.index = 1 if second else 0
+        self.S = Sequences(LayerSpec(spec()), dtype)
+
+    def step(self, entries, batch=None):
+        a = self.a
+        n = a.heads * a.vdim
+        batch = batch or self.S.batch([(s, r.shape[0]) for s, r in entries])
+        out = torch.full((sum(r.shape[0] for _, r in entries), n + 8), 7.0, dtype=self.dtype, device=DEV)
+        self.ops.latent_attention(torch.cat([r for _, r in entries]).to(DEV), self.M, batch, self.S.kv, 0, 1e-5, out[:, :n])
+        assert self.ops.take_status() == 0 and bool((out[:, n:] == 7).all())
+        return torch.split(out[:, :n].cpu(), [r.shape[0] for _, r in entries])
+
+    def rows(self, n, seed, plant=()):
+        """Random rows; ``plant``: (query, key) places whose score is made to stand out, in every head."""
+        a = self.a
+        x = rnd(n, self.width, seed=seed)
+        q, kr = x[:, :a.q_rank].view(n, a.heads, -1), x[:, self.at + a.kv_rank:][:, :a.rot_dim]
+        for k, (i, j) in enumerate(plant):               # undo the rotations, so that the rotated vectors agree
+            u = rnd(a.rot_dim, seed=100 + k)
+            u = u / u.norm() * (a.dim + a.rot_dim) ** 0.5
+            q[i, :, a.dim:], kr[j] = 1.5 * self.turn(u, -i), 1.5 * self.turn(u, -j)
+        return x.to(self.dtype)
+
+    def turn(self, u, p):
+        half, y = self.rot["dims"] // 2, u.clone()
+        for i in range(half):
+            f = torch.tensor(p * self.rot["base"] ** (-2.0 * i / self.rot["dims"]), dtype=torch.float64)
+            c, s = float(torch.cos(f)), float(torch.sin(f))
+            y[i], y[i + half] = u[i] * c - u[i + half] * s, u[i + half] * c + u[i] * s
+        return y
+
+    def oracle(self, rows, keys=None):
+        a, n, A = self.a, rows.shape[0], self.M.attn
+        q = O.rms(rows.double()[:, :a.q_rank], 1e-5).view(n, a.heads, -1)
+        keys = rows if keys is None else keys
+        z = keys.double()[:, -(self.width - self.at):] if keys is rows else keys.double()
+        c, kr = O.rms(z[:, :a.kv_rank], 1e-5) * A.c_norm.double().cpu(), O.rotate_half(z[:, a.kv_rank:a.kv_rank + a.rot_dim], **self.rot)
+        qr = O.rotate_half(q[..., a.dim:], **self.rot)
+        out = []
+        for h in range(a.heads):
+            k, v = c @ A.uk[h].double().cpu().T, c @ A.uv[h].double().cpu().T
+            out.append(O.sink_window_attention(torch.cat([q[:, h, :a.dim], qr[:, h]], 1), torch.cat([k, kr], 1), v, a.scale, a.window, self.sink[h].double()))
+        return torch.cat(out, 1)
+
+
+@pytest.mark.parametrize("portions", PORTIONS)
+@pytest.mark.parametrize("case", ATTN)
+@pytest.mark.parametrize("dtype", TYPES)
+def test_latent_attention(ops, case, portions, dtype):
+    n, win = 220, case[-1]
+    L = LatentLayer(ops, case, dtype)
+    # keys at page borders, at the first tokens, just inside the window's edge (and just outside, where they must not show)
+    plant = [(15, 0), (16, 15), (63, 48), (64, 64), (129, 127), (150, 143), (191, 190), (3, 2)]
+    if win:
+        plant += [(i, i - win + 1) for i in (100, 160, 200, 215) if i >= win - 1] + [(i, i - win) for i in (110, 170, 205, 217) if i >= win]
+    else:
+        plant += [(200, 0), (205, 1), (217, 16)]
+    rows, out, pos = L.rows(n, 7 + sum(case), plant), [], 0
+    for c in C.cut(n, PORTIONS[portions]):
+        out.append(L.step([(0, rows[pos:pos + c])])[0])
+        pos += c
+    want, got = L.oracle(rows), torch.cat(out)
+    err = (got.double() - want).abs().amax(1) / want.abs().max()
+    limit = 3e-2 if dtype == torch.bfloat16 else 1e-5
+    assert err.max() < limit, (int(err.argmax()), float(err.max()))
+    assert err.mean() < limit / 3
+
+
+@pytest.mark.parametrize("case", [ATTN[0], ATTN[1], ATTN[5], ATTN[6]])
+def test_batches_of_unequal_sequences(ops, case):
+    """Long portions, short portions and single rows in one step; a freed sequence's pages serve the next one."""
+    L = LatentLayer(ops, case, torch.bfloat16)
+    rows = {b: L.rows(n, 50 + b, [(n - 1, n - 3)] if n > 3 else []) for b, n in LENS.items()}
+    got = {b: [] for b in LENS}
+    for step in schedule(LENS, SIZES, late=(2, 5)):
+        for (b, p, n), o in zip(step, L.step([(b, rows[b][p:p + n]) for b, p, n in step])):
+            got[b].append(o)
+            if p + n == LENS[b]:
+                L.S.free(b)
+    for b in LENS:
+        assert rel(torch.cat(got[b]), L.oracle(rows[b])) < 3e-2, b
+
+
+@pytest.mark.parametrize("dtype", TYPES)
+def test_a_layer_reads_anothers_latents(ops, dtype):
+    first, second = LatentLayer(ops, ATTN[0], dtype), LatentLayer(ops, ATTN[0], dtype, second=True)
+    second.S, n, pos = first.S, 150, 0
+    rows, own = first.rows(n, 1), second.rows(n, 2, [(90, 64), (91, 65), (100, 99)])
+    out = []
+    for c in C.cut(n, [37, 2, 1, 60, 1]):
+        batch = first.S.batch([(0, c)])
+        first.step([(0, rows[pos:pos + c])], batch)
+        before = first.S.kv.kv[0].clone()
+        out.append(second.step([(0, own[pos:pos + c])], batch)[0])
+        assert torch.equal(before, first.S.kv.kv[0])
+        pos += c
+    want = second.oracle(own, keys=rows[:, first.at:])
+    assert rel(torch.cat(out), want) < (1e-5 if dtype == torch.float32 else 3e-2)
+
+
+@pytest.mark.parametrize("window", [0, 1000])
+def test_long_context_is_split_over_blocks(ops, window):
+    L, n = LatentLayer(ops, (8, 32, 16, 64, 128, window), torch.bfloat16), 1500
+    plant = [(n - 1, 700), (n - 2, n - 1000), (n - 3, 502), (n - 4, n - 4)] + ([] if window else [(n - 5, 0), (n - 6, 5)])
+    rows = L.rows(n, 3, plant)
+    L.step([(0, rows[:n - 6])])
+    got = torch.cat([L.step([(0, rows[i:i + 1])])[0] for i in range(n - 6, n)])
+    want = L.oracle(rows)[-6:]
+    assert rel(got, want) < 3e-2
+
+
+# ----------------------------------------------------------------------------------- whole models
+CONFIGS = {
+    "mixed layers": C.config(),
+    "wider": C.config([C.hgrn2(C.dense(512), 4, 64, 128), C.latent(C.moe(16, 4, 128, 256), None, 64, 8, 64, 32, 64, 192, 256, 0.1, 1e5),
+                       C.hgrn2(C.moe(16, 4, 128, 256), 4, 128, 64), C.latent(C.moe(16, 4, 128, 256), 1, 100, 16, 64, 32, 128, 192, 256, 0.1, 1e5)],
+                      width=512, vocab=1000, taps=3),
+    "ragged": C.config([C.latent(C.moe(5, 3, 36, 20), None, 7, 3, 10, 6, 14, 22, 26, 0.4, 50.0), C.hgrn2(None, 5, 9, 11),
+                        C.latent(C.dense(50), 0, 70, 1, 18, 6, 9, 30, 26, 0.4, 50.0), C.hgrn2(C.moe(3, 1, 28, 0), 1, 40, 7)], width=100, vocab=77, taps=6, eps=1e-4),
+}
+
+
+@pytest.mark.parametrize("name", CONFIGS)
+@pytest.mark.parametrize("dtype", TYPES)
+def test_model_in_every_schedule(tmp_path, name, dtype):
+    from blaze_b200.llm import LLM
+    from test_niletar_cpu import verify_with_rejected_rows
+    cfg = CONFIGS[name]
+    w = C.weights(cfg, seed=2)
+    V = cfg["vocab"]
+    seqs = {"a": C.tokens(150, V, 1), "b": C.tokens(67, V, 2), "c": C.tokens(33, V, 3), "d": C.tokens(1, V, 4), "e": C.tokens(90, V, 5)}
+    want = {i: O.forward(cfg, w, t) for i, t in seqs.items()}
+    llm = LLM(C.save(tmp_path, cfg, w), device=DEV, dtype=dtype, kv_tokens=336, max_seqs=3, max_model_len=512, enable_prefix_caching=False)
+    assert llm.model.ops.is_cuda and llm.engine.kv.layout == "tiles"
+    limit = 1e-4 if dtype == torch.float32 else 0.08
+    for sched, f in SCHEDULES.items():
+        got = C.run(llm.engine, {"a": seqs["a"]}, [[("a", n)] for n in f(150)])["a"]
+        assert C.error(got, want["a"]) < limit, sched
+    for _ in range(2):
+        got = C.run(llm.engine, seqs, mixed_steps(seqs))
+        for i in seqs:
+            assert C.error(got[i], want[i]) < limit, i
+    if V >= 310:
+        got = verify_with_rejected_rows(llm.engine, {i: [t % 300 for t in seqs[i]] for i in ("b", "c")})
+        for i in got:
+            assert C.error(got[i], O.forward(cfg, w, [t % 300 for t in seqs[i]])) < limit, i
+
+
+@pytest.mark.parametrize("graphs", [True, False])
+def test_generation_follows_the_logits(tmp_path, graphs):
+    """Greedy generation through the scheduler (captured decode steps, prefix cache, speculation): every chosen token is the best
+    one of the oracle's logits for that context, up to bf16 rounding."""
+    from blaze_b200.llm import LLM
+    from blaze_b200.sampler import SamplingParams
+    cfg = CONFIGS["wider"]
+    w = C.weights(cfg, seed=6)
+    path = C.save(tmp_path, cfg, w)
+    prompts = [C.tokens(n, 1000, 40 + n) for n in (90, 5, 33, 64)]
+    sp = SamplingParams(temperature=0.0, max_tokens=40, ignore_eos=True)
+    for kw in ({}, {"spec_method": "ngram", "max_draft": 3}):
+        llm = LLM(path, device=DEV, kv_tokens=2048, max_seqs=4, max_model_len=256, chunk=64, use_graphs=graphs, **kw)
+        for outs in (llm.generate(prompts, sp), llm.generate(prompts, sp)):
+            for p, o in zip(prompts, outs):
+                t = p + o.token_ids
+                lg = O.forward(cfg, w, t[:-1], dtype=torch.float32)[len(p) - 1:]
+                chosen = lg[torch.arange(len(o.token_ids)), torch.tensor(o.token_ids)]
+                assert len(o.token_ids) == 40 and float((lg.max(1).values - chosen).max()) < 0.15 * float(lg.std())
+        assert bool(llm.engine._graphs) == graphs
+
+
+def test_32_bit_generation_is_the_oracles(tmp_path):
+    from blaze_b200.llm import LLM
+    from blaze_b200.sampler import SamplingParams
+    cfg = CONFIGS["mixed layers"]
+    w = C.weights(cfg, seed=9)
+    prompts = [C.tokens(n, 320, 60 + n) for n in (40, 7)]
+    llm = LLM(C.save(tmp_path, cfg, w), device=DEV, dtype=torch.float32, kv_tokens=512, max_seqs=2, max_model_len=128)
+    outs = llm.generate(prompts, SamplingParams(temperature=0.0, max_tokens=24, ignore_eos=True))
+    for p, o in zip(prompts, outs):
+        t = list(p)
+        for _ in range(24):
+            t.append(int(O.forward(cfg, w, t)[-1].argmax()))
+        assert o.token_ids == t[len(p):]
