@@ -1060,6 +1060,10 @@ class CudaOps:
 
     def latent_queries(self, proj, M, batch, kv, layer_idx, eps):
         """Page write, and the queries ``[T, heads * (dim + rot_dim)]`` before their rotation."""
+        return self.linear(M.attn.uq, self.latent_prep(proj, M, batch, kv, layer_idx, eps))
+
+    def latent_prep(self, proj, M, batch, kv, layer_idx, eps):
+        """The queries' normed latents; the keys' (where the layer has its own) with their rotated part go to their pages."""
         A, a, T, pool = M.attn, M.attn.spec, proj.shape[0], kv.kv[layer_idx]
         if kv.layout != "tiles" or pool.dtype != proj.dtype:
             raise CudaError(f"latent attention of {proj.dtype} rows needs 'tiles' pages of that type")
@@ -1070,67 +1074,80 @@ class CudaOps:
                                              _ptr(batch.positions), _ptr(batch.slot_mapping), T, a.q_rank, a.kv_rank, a.rot_dim,
                                              a.rot.dims if a.rot is not None else 0, eps, int(proj.dtype == torch.float32), self._stream()),
                     "latent_prep")
-        return self.linear(A.uq, lat)
+        return lat
 
     def latent_attend(self, q, M, batch, kv, layer_idx, out):
-        A, a, pool, bt = M.attn, M.attn.spec, kv.kv[layer_idx], kv.block_table
-        T, H, B, f32, st = q.shape[0], a.heads, batch.slots.numel(), q.dtype == torch.float32, self._stream()
+        """Rotation and attention of the queries.  Sequences with many new tokens go by head where the prompt kernel covers the
+        sizes, all the others over the latents."""
+        A, a = M.attn, M.attn.spec
+        T, H, f32 = q.shape[0], a.heads, q.dtype == torch.float32
         lens = [e - s for s, e in zip(batch.h_q_start, batch.h_q_start[1:])]
-        # which way: many tokens by head where the prompt kernel covers the sizes, all the others over the latents
-        block = 0 if f32 or a.scale <= 0 else int(self.lib.blz_latent_rows_block(a.kv_rank, a.rot_dim, H))
         wide = not f32 and a.scale > 0 and a.vdim <= 128 and a.dim + a.rot_dim <= 192
         most = self.LATENT_SHORT if wide else max(batch.max_q_len, 1)
-        short = [n for n in lens if 0 < n <= most]
+        longest = max((n for n in lens if n <= most), default=0)
         D = (a.kv_rank + 15) // 16 * 16 + (a.rot_dim + 15) // 16 * 16
-        qe = torch.empty(T, H, D, dtype=q.dtype, device=self.device) if short else None
+        qe = torch.empty(T, H, D, dtype=q.dtype, device=self.device) if longest else None
         rows = (_ptr(batch.seq_of_row), _ptr(batch.q_start))
-        rot = a.rot.dims if a.rot is not None else 0
-        self._check(self.lib.blz_latent_rot(_ptr(q), _ptr(qe), _ptr(A.freq), _ptr(batch.positions), *rows, T, H, a.dim, a.rot_dim, rot,
-                                            a.kv_rank, most, int(f32), st), "latent_rot")
-        if short:
-            self._check(self.lib.blz_head_gemm(_ptr(q), q.stride(0), a.dim + a.rot_dim, _ptr(A.uk_t), _ptr(qe), H * D, D, T, a.kv_rank, a.dim,
-                                               H, *rows, most, int(f32), st), "head_gemm")
-            lat = torch.empty(T, H, a.kv_rank, dtype=q.dtype, device=self.device)
-            seqs = (_ptr(bt), bt.stride(0), _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(A.sink))
-            if block:
-                longest = max(short)
-                R = int(self.lib.blz_latent_rows_block(a.kv_rank, a.rot_dim, longest * H))
-                rb = (longest * H + R - 1) // R
-                keys = min(batch.max_ctx, a.window + (R + H - 1) // H) if a.window else batch.max_ctx
-                sp = max(1, min(self._sm // (len(short) * rb), (keys + 127) // 128, 32))
-                po = pm = None
-                if sp > 1:
-                    n = B * rb * sp * R
-                    po, pm = self._buf("latent_part_o", n * a.kv_rank * 4), self._buf("latent_part_ml", n * 8)
-                    self.launches += 1
-                self._check(self.lib.blz_latent_rows(_ptr(qe), _ptr(lat), _ptr(pool), pool.stride(0), *seqs, B, H, a.kv_rank, a.rot_dim, a.window,
-                                                     a.scale, most, longest, R, rb, sp, _ptr(po), _ptr(pm), st), "latent_rows")
-            else:
-                self._check(self.lib.blz_shared_plain(_ptr(qe), H * D, _ptr(lat), H * a.kv_rank, _ptr(pool), pool.stride(0), *seqs,
-                                                      _ptr(batch.seq_of_row), T, B, H, D, a.kv_rank, a.window, a.scale, int(f32), st),
-                            "shared_plain")
-            self._check(self.lib.blz_head_gemm(_ptr(lat), H * a.kv_rank, a.kv_rank, _ptr(A.uv), _ptr(out), out.stride(0), a.vdim, T, a.vdim,
-                                               a.kv_rank, H, *rows, most, int(f32), st), "head_gemm")
+        self._check(self.lib.blz_latent_rot(_ptr(q), _ptr(qe), _ptr(A.freq), _ptr(batch.positions), *rows, T, H, a.dim, a.rot_dim,
+                                            a.rot.dims if a.rot is not None else 0, a.kv_rank, most, int(f32), self._stream()), "latent_rot")
+        if longest:
+            self._head_gemm(q, a.dim + a.rot_dim, A.uk_t, qe.view(T, H * D), D, batch, most)
+            lat = torch.empty(T, H * a.kv_rank, dtype=q.dtype, device=self.device)
+            self.latent_rows(qe, M, batch, kv, layer_idx, longest, most, lat)
+            self._head_gemm(lat, a.kv_rank, A.uv, out, a.vdim, batch, most)
         if any(n > most for n in lens):
-            self._latent_expanded(q, M, batch, kv, layer_idx, most, out)
+            self._expanded_attention(q, M, batch, kv, self._expand_latents(M, batch, kv, layer_idx, most), most, out)
 
-    def _latent_expanded(self, q, M, batch, kv, layer_idx, most: int, out):
-        """Prompt portions: keys and values by head of all tokens that the sequences with more than ``most`` new tokens see."""
+    def _head_gemm(self, x, x_head: int, w, y, y_head: int, batch, most: int):
+        """``y[t, h] = w[h] x[t, h]`` for the sequences with at most ``most`` new tokens; ``*_head``: columns from head to head."""
+        self._check(self.lib.blz_head_gemm(_ptr(x), x.stride(0), x_head, _ptr(w), _ptr(y), y.stride(0), y_head, x.shape[0], w.shape[1], w.shape[2],
+                                           w.shape[0], _ptr(batch.seq_of_row), _ptr(batch.q_start), most, int(x.dtype == torch.float32),
+                                           self._stream()), "head_gemm")
+
+    def latent_rows(self, qe, M, batch, kv, layer_idx, longest: int, most: int, lat):
+        """Weighted sums of the latents for the sequences with at most ``most`` new tokens (the longest has ``longest``)."""
+        A, a, pool, bt = M.attn, M.attn.spec, kv.kv[layer_idx], kv.block_table
+        T, H, D = qe.shape
+        B, f32, st = batch.slots.numel(), qe.dtype == torch.float32, self._stream()
+        seqs = (_ptr(bt), bt.stride(0), _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(A.sink))
+        R = 0 if f32 or a.scale <= 0 else int(self.lib.blz_latent_rows_block(a.kv_rank, a.rot_dim, longest * H))
+        if R == 0:
+            self._check(self.lib.blz_shared_plain(_ptr(qe), H * D, _ptr(lat), H * a.kv_rank, _ptr(pool), pool.stride(0), *seqs,
+                                                  _ptr(batch.seq_of_row), T, B, H, D, a.kv_rank, a.window, a.scale, int(f32), st), "shared_plain")
+            return
+        short = sum(1 for s, e in zip(batch.h_q_start, batch.h_q_start[1:]) if 0 < e - s <= most)
+        rb = (longest * H + R - 1) // R
+        keys = min(batch.max_ctx, a.window + (R + H - 1) // H) if a.window else batch.max_ctx
+        sp = max(1, min(self._sm // (short * rb), (keys + 127) // 128, 32))
+        po = pm = None
+        if sp > 1:
+            n = B * rb * sp * R
+            po, pm = self._buf("latent_part_o", n * a.kv_rank * 4), self._buf("latent_part_ml", n * 8)
+            self.launches += 1
+        self._check(self.lib.blz_latent_rows(_ptr(qe), _ptr(lat), _ptr(pool), pool.stride(0), *seqs, B, H, a.kv_rank, a.rot_dim, a.window, a.scale,
+                                             most, longest, R, rb, sp, _ptr(po), _ptr(pm), st), "latent_rows")
+
+    def _expand_latents(self, M, batch, kv, layer_idx, most: int):
+        """Keys and values by head, as pages, of all tokens that the sequences with more than ``most`` new tokens see."""
         A, a, pool, st = M.attn, M.attn.spec, kv.kv[layer_idx], self._stream()
-        T, H, B = q.shape[0], a.heads, batch.slots.numel()
-        pages, base, n_pages, items = self._visible_pages(batch, kv, a.window, most)
-        lat = torch.empty(n_pages * 16, a.kv_rank, dtype=q.dtype, device=self.device)
-        self._check(self.lib.blz_latent_gather(_ptr(pool), pool.stride(0), _ptr(pages), n_pages, _ptr(lat), a.kv_rank, a.rot_dim, st), "latent_gather")
+        pages, _, n, _ = self._visible_pages(batch, kv, a.window, most)
+        lat = torch.empty(n * 16, a.kv_rank, dtype=pool.dtype, device=self.device)
+        self._check(self.lib.blz_latent_gather(_ptr(pool), pool.stride(0), _ptr(pages), n, _ptr(lat), a.kv_rank, a.rot_dim, st), "latent_gather")
         kx = self.linear(A.expand, lat)
-        up = lambda n: (n + 15) // 16 * 16       # noqa: E731
-        be = 16 * (up(a.dim + a.rot_dim) + up(a.vdim))
-        scratch = torch.empty(n_pages, H, be, dtype=q.dtype, device=self.device)
-        self._check(self.lib.blz_expand_store(_ptr(kx), kx.stride(0), _ptr(pool), pool.stride(0), _ptr(pages), _ptr(scratch), n_pages, H, a.dim,
+        block = 16 * ((a.dim + a.rot_dim + 15) // 16 * 16 + (a.vdim + 15) // 16 * 16)
+        out = torch.empty(n, a.heads, block, dtype=pool.dtype, device=self.device)
+        self._check(self.lib.blz_expand_store(_ptr(kx), kx.stride(0), _ptr(pool), pool.stride(0), _ptr(pages), _ptr(out), n, a.heads, a.dim,
                                               a.rot_dim, a.vdim, a.kv_rank, st), "expand_store")
-        bt = kv.block_table
-        self._check(self.lib.blz_soft_tc(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(scratch), scratch.stride(0), scratch.stride(1),
-                                         _ptr(bt), bt.stride(0), _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(A.sink), VP(0), 0,
-                                         T, B, H, H, a.dim + a.rot_dim, a.vdim, a.window, a.scale, 1.0, most, items, _ptr(base), st), "soft_tc")
+        return out
+
+    def _expanded_attention(self, q, M, batch, kv, pages, most: int, out):
+        """Prompt attention of the sequences with more than ``most`` new tokens over the pages of :meth:`_expand_latents`."""
+        A, a, bt = M.attn, M.attn.spec, kv.block_table
+        _, base, _, items = self._visible_pages(batch, kv, a.window, most)
+        self._check(self.lib.blz_soft_tc(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(pages), pages.stride(0), pages.stride(1), _ptr(bt),
+                                         bt.stride(0), _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(A.sink), VP(0), 0,
+                                         q.shape[0], batch.slots.numel(), a.heads, a.heads, a.dim + a.rot_dim, a.vdim, a.window, a.scale, 1.0, most,
+                                         items, _ptr(base), self._stream()), "soft_tc")
 
     def _visible_pages(self, batch, kv, window: int, most: int):
         """(pages, page base of each sequence, number of pages, row blocks) of the sequences with more than ``most`` new tokens: the pages

@@ -166,7 +166,7 @@ class LatentLayer:
         self.sink = rnd(a.heads, seed=d) * 2 + 1
         A.sink, A.q_norm, A.c_norm = self.sink.to(DEV), torch.ones(a.q_rank, device=DEV), (rnd(R, seed=5) * 0.3 + 1).to(DEV)
         A.uq = Linear.from_dense(torch.eye(a.q_rank, device=DEV), dtype=dtype)
-        uk, uv = [(rnd(a.heads * k, R, seed=6 + k) * R ** -0.5).to(DEV) for k in (d, e)]
+        uk, uv = [(rnd(a.heads * k, R, seed=6 + k) * R ** -0.5).to(DEV) for k in (a.dim, a.vdim)]
         A.set_maps(uk, uv, dtype)
         self.at = (a.q_rank + 7) // 8 * 8
         self.M.cols = {"q": 0, "kv": self.at}
@@ -293,6 +293,16 @@ CONFIGS = {
 }
 
 
+def check(got, want, dtype, what):
+    """Every row close; in bf16 a few rows may differ, those where rounding makes a token choose another expert."""
+    d = got.double() - want
+    err = (d - d.mean(1, keepdim=True)).pow(2).mean(1).sqrt() / want.std()
+    if dtype == torch.float32:
+        assert err.max() < 1e-4, what
+    else:
+        assert err.median() < 0.025 and int((err > 0.05).sum()) <= max(2, 0.05 * err.numel()), (what, err)
+
+
 @pytest.mark.parametrize("name", CONFIGS)
 @pytest.mark.parametrize("dtype", TYPES)
 def test_model_in_every_schedule(tmp_path, name, dtype):
@@ -305,18 +315,16 @@ def test_model_in_every_schedule(tmp_path, name, dtype):
     want = {i: O.forward(cfg, w, t) for i, t in seqs.items()}
     llm = LLM(C.save(tmp_path, cfg, w), device=DEV, dtype=dtype, kv_tokens=336, max_seqs=3, max_model_len=512, enable_prefix_caching=False)
     assert llm.model.ops.is_cuda and llm.engine.kv.layout == "tiles"
-    limit = 1e-4 if dtype == torch.float32 else 0.08
     for sched, f in SCHEDULES.items():
-        got = C.run(llm.engine, {"a": seqs["a"]}, [[("a", n)] for n in f(150)])["a"]
-        assert C.error(got, want["a"]) < limit, sched
+        check(C.run(llm.engine, {"a": seqs["a"]}, [[("a", n)] for n in f(150)])["a"], want["a"], dtype, sched)
     for _ in range(2):
         got = C.run(llm.engine, seqs, mixed_steps(seqs))
         for i in seqs:
-            assert C.error(got[i], want[i]) < limit, i
+            check(got[i], want[i], dtype, i)
     if V >= 310:
         got = verify_with_rejected_rows(llm.engine, {i: [t % 300 for t in seqs[i]] for i in ("b", "c")})
         for i in got:
-            assert C.error(got[i], O.forward(cfg, w, [t % 300 for t in seqs[i]])) < limit, i
+            check(got[i], O.forward(cfg, w, [t % 300 for t in seqs[i]]), dtype, i)
 
 
 @pytest.mark.parametrize("graphs", [True, False])
