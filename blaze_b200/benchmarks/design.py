@@ -203,7 +203,7 @@ def _attention(ops, cfg: ModelConfig, B: int, qlen: int, ctx: int, copies: int):
         heads, kv_heads, q_norm, k_norm = H, G, torch.ones(D, device="cuda").bfloat16(), torch.ones(D, device="cuda").bfloat16()
     M.cfg = cfg
     q = torch.randn(T, H, D, device="cuda").bfloat16()
-    qkv = torch.randn(T, (H + 2 * G) * D, device="cuda").bfloat16()
+    qkv = torch.randn(T, (H * (2 if cfg.attn_output_gate else 1) + 2 * G) * D, device="cuda").bfloat16()
     calls = [lambda kv=kv: ops.attention(q, M, batch, kv, 0, D ** -0.5) for kv in kvs]
     write = [lambda kv=kv: ops.attn_prep_store(qkv, N, M, batch, kv, 0, None) for kv in kvs]
     return calls, write, B * ctx * G * 2.0 * D, 4.0 * B * H * keys * D, T * qkv.shape[1] * 2.0
