@@ -151,7 +151,8 @@ def _feed_forward(own: ModelConfig, rel: ModelConfig, names, W: int, ff: int, ad
                 calls = [lambda m=m: ops.branch_norm(x, m._mlp(m.layers[0].mlp, h)[0], w, 1e-6) for m in ms]
                 nb += T * W * 8.0
             else:
-                calls = [lambda m=m: ops.norm(m._mlp(m.layers[0].mlp, h)[0], h, w.bfloat16(), 1e-6) for m in ms]
+                res = torch.zeros(T, W, device="cuda").bfloat16()
+                calls = [lambda m=m: ops.norm(m._mlp(m.layers[0].mlp, h)[0], res, w.bfloat16(), 1e-6) for m in ms]
                 nb += T * W * 4.0
             add(f"experts + residual + norm, {T} rows", name, graph_ms(calls), nb, fl)
             del ms, calls

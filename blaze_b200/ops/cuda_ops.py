@@ -210,7 +210,7 @@ class CudaOps:
         lib.blz_latent_rot.argtypes = [VP] * 6 + [_c.c_int] * 8 + [VP]
         lib.blz_head_gemm.argtypes = [VP, LL, LL, VP, VP, LL, LL] + [_c.c_int] * 4 + [VP, VP, _c.c_int, _c.c_int, VP]
         lib.blz_latent_rows_block.restype = _c.c_int
-        lib.blz_latent_rows_block.argtypes = [_c.c_int] * 3
+        lib.blz_latent_rows_block.argtypes = [_c.c_int] * 3 + [VP]
         lib.blz_latent_rows.argtypes = [VP, VP, VP, LL, VP, _c.c_int, VP, VP, VP, VP] + [_c.c_int] * 5 + [_c.c_float] + [_c.c_int] * 5 + [VP, VP, VP]
         lib.blz_latent_gather.argtypes = [VP, LL, VP, _c.c_int, VP, _c.c_int, _c.c_int, VP]
         lib.blz_expand_store.argtypes = [VP, LL, VP, LL, VP, VP] + [_c.c_int] * 6 + [VP]
@@ -1051,6 +1051,7 @@ class CudaOps:
         return out
 
     # ------------------------------------------------------------------ latent attention
+    LATENT_BLOCK = 64          # query rows per CTA of the kernel over the latents, at most
     LATENT_SHORT = 16          # new tokens up to which a sequence's queries are mapped to the latents instead of the latents to keys
 
     def latent_attention(self, proj, M, batch, kv, layer_idx, eps, out):
@@ -1110,7 +1111,9 @@ class CudaOps:
         T, H, D = qe.shape
         B, f32, st = batch.slots.numel(), qe.dtype == torch.float32, self._stream()
         seqs = (_ptr(bt), bt.stride(0), _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(A.sink))
-        R = 0 if f32 or a.scale <= 0 else int(self.lib.blz_latent_rows_block(a.kv_rank, a.rot_dim, longest * H))
+        per_sm = _c.c_int(1)
+        R = 0 if f32 or a.scale <= 0 else int(self.lib.blz_latent_rows_block(a.kv_rank, a.rot_dim, min(longest * H, self.LATENT_BLOCK),
+                                                                             _c.byref(per_sm)))
         if R == 0:
             self._check(self.lib.blz_shared_plain(_ptr(qe), H * D, _ptr(lat), H * a.kv_rank, _ptr(pool), pool.stride(0), *seqs,
                                                   _ptr(batch.seq_of_row), T, B, H, D, a.kv_rank, a.window, a.scale, int(f32), st), "shared_plain")
@@ -1118,7 +1121,7 @@ class CudaOps:
         short = sum(1 for s, e in zip(batch.h_q_start, batch.h_q_start[1:]) if 0 < e - s <= most)
         rb = (longest * H + R - 1) // R
         keys = min(batch.max_ctx, a.window + (R + H - 1) // H) if a.window else batch.max_ctx
-        sp = max(1, min(self._sm // (short * rb), (keys + 127) // 128, 32))
+        sp = max(1, min(per_sm.value * self._sm // (short * rb), (keys + 127) // 128, 32))
         po = pm = None
         if sp > 1:
             n = B * rb * sp * R

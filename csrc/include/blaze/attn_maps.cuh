@@ -55,6 +55,21 @@ __device__ __forceinline__ float ad_ld(const __nv_bfloat16* p) { return __bfloat
 __device__ __forceinline__ void ad_st(float* p, float v) { *p = v; }
 __device__ __forceinline__ void ad_st(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
+// R rows (a multiple of 8) of dim columns -> shared memory as core matrices with D padded columns, by n threads with asynchronous copies of
+// 16 bytes, all under way together; src(r): the row in memory, 16-byte aligned, or null (zeros).  dim % 8 == 0.  A warp reads 32 bytes of
+// a row at a time and writes whole core matrices.  The caller waits (copies_wait) and fences.
+template <typename F>
+__device__ __forceinline__ void copy_rows(__nv_bfloat16* dst, int R, int D, int dim, int tid, int n, const void* any, F&& src) {
+  for (int i = tid; i < R * (D / 8); i += n) {
+    const int rest = i >> 4, r = (rest % (R / 8)) * 8 + (i & 7), j = ((rest / (R / 8)) * 2 + (i >> 3 & 1)) * 8;
+    const __nv_bfloat16* row = src(r);
+    const bool live = row != nullptr && j < dim;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + core_off(r, j, D))),
+                 "l"(live ? (const void*)(row + j) : any), "r"(live ? 16 : 0) : "memory");
+  }
+}
+__device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
 // factor of output column e of (row t, head h): sigmoid(gate) * post
 template <typename T>
 __device__ __forceinline__ float gate_factor(const MapsParams& p, int t, int h, int e) {

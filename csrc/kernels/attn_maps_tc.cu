@@ -60,7 +60,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
   pdl_wait();
   if (warp == 8) {
     // which sequence and row block this CTA has: the long sequences' blocks in order
-    int item = blockIdx.x, b = -1, q0 = 0;
+    int item = gridDim.x - 1 - blockIdx.x, b = -1, q0 = 0;         // the last blocks of a sequence see the most keys: they start first
     for (int base = 0; base < p.B; base += 32) {
       const int i = base + lane;
       const int qlen = i < p.B ? p.q_start[i + 1] - p.q_start[i] : 0;
@@ -188,19 +188,25 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
       const int tq = t0 + r / group, head = g * group + r % group;
       const int pos = live ? pos0 + tq : -1, lo = first_key(pos, p.window);
       {
-        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)(r0 + tq) * p.ld + (size_t)(MAPS == 2 ? head * 2 + m : head) * p.dim;
         __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(sQ + m * q_bytes);
-        for (int j = 0; j < dp; j += 8) {
-          uint4 u = make_uint4(0, 0, 0, 0);
-          if (live && vec_q && j + 8 <= p.dim) {
-            u = *reinterpret_cast<const uint4*>(src + j);
-          } else if (live) {
+        auto row_of = [&](int x) -> const __nv_bfloat16* {
+          const int t = t0 + x / group, h = g * group + x % group;
+          if (x >= tph * group || t >= q0 + ntok) return nullptr;
+          return reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)(r0 + t) * p.ld + (size_t)(MAPS == 2 ? h * 2 + m : h) * p.dim;
+        };
+        if (vec_q) {
+          copy_rows(dst, 128, dp, p.dim, r, 128, p.q, row_of);
+          copies_wait();
+        } else {
+          const __nv_bfloat16* src = row_of(r);
+          for (int j = 0; j < dp; j += 8) {
+            uint4 u = make_uint4(0, 0, 0, 0);
             __nv_bfloat16* e = reinterpret_cast<__nv_bfloat16*>(&u);
 #pragma unroll
             for (int k = 0; k < 8; ++k)
-              if (j + k < p.dim) e[k] = src[j + k];
+              if (live && j + k < p.dim) e[k] = src[j + k];
+            *reinterpret_cast<uint4*>(dst + core_off(r, j, dp)) = u;
           }
-          *reinterpret_cast<uint4*>(dst + core_off(r, j, dp)) = u;
         }
         fence_async_smem();
         __syncwarp();

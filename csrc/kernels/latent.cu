@@ -50,9 +50,11 @@ struct LatentPrepParams {
   float eps;
 };
 
-// block (row, 0): the queries' latent, normed; block (row, 1): the keys' latent, normed, and the rotated part, into their page slot
-template <typename T>
+// block (row, 0): the queries' latent, normed; block (row, 1): the keys' latent, normed, and the rotated part, into their page slot.
+// VEC columns per thread and turn; the first KEEP turns stay in registers between the sum of squares and the result.
+template <typename T, int VEC>
 __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepParams p) {
+  constexpr int KEEP = VEC == 8 ? 2 : 1;
   __shared__ float red[4];
   pdl_trigger();
   pdl_wait();
@@ -62,23 +64,65 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepParams p) {
   if (slot < 0) return;
   const T* src = reinterpret_cast<const T*>(p.proj) + (size_t)t * p.ld + (keys ? p.kv_off : p.q_off);
   const int n = keys ? p.rank : p.q_rank;
-  float ss = 0.f;
-  for (int j = tid; j < n; j += 128) { const float v = ad_ld(src + j); ss = fmaf(v, v, ss); }
+  const float* w = keys ? p.c_norm : p.q_norm;
+  auto load = [&](int j, float (&v)[VEC]) {
+    if constexpr (VEC == 8) {
+      const uint4 u = *reinterpret_cast<const uint4*>(src + j);
+      const uint32_t x[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+      for (int k = 0; k < 4; ++k) { v[2 * k] = __uint_as_float(x[k] << 16); v[2 * k + 1] = __uint_as_float(x[k] & 0xffff0000u); }
+    } else {
+      v[0] = ad_ld(src + j);
+    }
+  };
+  float ss = 0.f, kept[KEEP][VEC];
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int j = (i * 128 + tid) * VEC;
+    if (j < n) {
+      load(j, kept[i]);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) ss = fmaf(kept[i][k], kept[i][k], ss);
+    }
+  }
+  for (int j = (KEEP * 128 + tid) * VEC; j < n; j += 128 * VEC) {
+    float v[VEC];
+    load(j, v);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) ss = fmaf(v[k], v[k], ss);
+  }
   ss = warp_sum(ss);
   if (lane == 0) red[warp] = ss;
   __syncthreads();
   const float f = 1.f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)n + p.eps);
-  if (!keys) {
-    T* dst = reinterpret_cast<T*>(p.q_lat) + (size_t)t * n;
-    for (int j = tid; j < n; j += 128) ad_st(dst + j, ad_ld(src + j) * f * p.q_norm[j]);
-    return;
-  }
-  const int rp = up16(p.rank), tp = up16(p.rot), D = rp + tp, half = p.rot_dims / 2;
+  const int rp = up16(p.rank), tp = up16(p.rot), D = rp + tp, half = p.rot_dims / 2, tok = slot & 15;
+  T* q_lat = reinterpret_cast<T*>(p.q_lat) + (size_t)t * p.q_rank;
   T* page = reinterpret_cast<T*>(p.pool) + (size_t)(slot >> 4) * p.page_stride;
-  const int tok = slot & 15;
-  for (int j = tid; j < rp; j += 128) ad_st(page + core_off(tok, j, D), j < n ? ad_ld(src + j) * f * p.c_norm[j] : 0.f);
+  auto put = [&](int j, const float (&v)[VEC]) {
+    T* dst = keys ? page + core_off(tok, j, D) : q_lat + j;
+    if constexpr (VEC == 8) {
+      float y[8];
+      const float4 a = *reinterpret_cast<const float4*>(w + j), b = *reinterpret_cast<const float4*>(w + j + 4);
+      const float g[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int k = 0; k < 8; ++k) y[k] = v[k] * f * g[k];
+      *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]), pack_bf16x2(y[4], y[5]), pack_bf16x2(y[6], y[7]));
+    } else {
+      ad_st(dst, v[0] * f * w[j]);
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i)
+    if ((i * 128 + tid) * VEC < n) put((i * 128 + tid) * VEC, kept[i]);
+  for (int j = (KEEP * 128 + tid) * VEC; j < n; j += 128 * VEC) {
+    float v[VEC];
+    load(j, v);
+    put(j, v);
+  }
+  if (!keys) return;
+  for (int j = n + tid; j < rp; j += 128) ad_st(page + core_off(tok, j, D), 0.f);
   const float pos = (float)p.positions[t];
-  for (int j = tid; j < tp; j += 128) {
+  for (int j = 127 - tid; j < tp; j += 128) {          // the threads with the least of the latent
     float v = j < p.rot ? ad_ld(src + n + j) : 0.f;
     if (j < 2 * half) {
       const bool low = j < half;
@@ -292,6 +336,7 @@ struct LatentRowsParams {
 
 static constexpr int kLrThreads = 192;
 static constexpr float kLrLazy = 8.f;
+static constexpr float kLrNone = -1e30f;       // the maximum of a row that has seen no key
 
 template <bool MAX>
 __device__ __forceinline__ float lr_op(float a, float b) { return MAX ? fmaxf(a, b) : a + b; }
@@ -330,7 +375,7 @@ __device__ __forceinline__ void reduce_lanes(const float (&v)[R], int lane, floa
 }
 
 template <int R>
-__global__ void __launch_bounds__(kLrThreads, 1) latent_rows_kernel(LatentRowsParams p) {
+__global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kernel(LatentRowsParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~uintptr_t(127));
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, H = p.heads, D = p.D, ST = p.stages;
@@ -344,7 +389,7 @@ __global__ void __launch_bounds__(kLrThreads, 1) latent_rows_kernel(LatentRowsPa
   const int s_lo = pg_lo + split * per, s_n = min(per, pg_lo + pages - s_lo), n = s_n > 0 ? (s_n + 7) / 8 : 0;
   const size_t w0 = (((size_t)b * p.row_blocks + rb) * p.splits + split) * R;        // this CTA's rows in the workspace
   if (n == 0) {
-    for (int r = threadIdx.x; r < R; r += kLrThreads) { p.part_ml[(w0 + r) * 2] = -INFINITY; p.part_ml[(w0 + r) * 2 + 1] = 0.f; }
+    for (int r = threadIdx.x; r < R; r += kLrThreads) { p.part_ml[(w0 + r) * 2] = kLrNone; p.part_ml[(w0 + r) * 2 + 1] = 0.f; }
     return;
   }
   const int nvb = (p.rank + 127) / 128, tile = 256 * D;                            // accumulators; bytes of 128 cached vectors
@@ -438,18 +483,14 @@ __global__ void __launch_bounds__(kLrThreads, 1) latent_rows_kernel(LatentRowsPa
     const uint32_t lanes = (uint32_t)(warp * 32) << 16;
     const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + ((size_t)r0 * H + (size_t)rb * R) * D;
     const int live = min(R, rows - rb * R);
-    for (int i = tid; i < R * (D / 8); i += 128) {
-      const int r = i % R, j = i / R * 8;
-      uint4 u = make_uint4(0, 0, 0, 0);
-      if (r < live) u = *reinterpret_cast<const uint4*>(q + (size_t)r * D + j);
-      *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(sQ) + core_off(r, j, D)) = u;
-    }
+    copy_rows(reinterpret_cast<__nv_bfloat16*>(sQ), R, D, D, tid, 128, q, [&](int r) { return r < live ? q + (size_t)r * D : nullptr; });
     const int end = (s_lo + s_n) * 16 - 1;
     if (tid < R) {
       const int pos = tid < live ? pos0 + (rb * R + tid) / H : -1;
       s_vis[tid] = make_int2(first_key(pos, p.window), min(pos, end));
-      s_m[tid] = -INFINITY;
+      s_m[tid] = kLrNone;
     }
+    copies_wait();
     fence_async_smem();
     __syncwarp();
     if (lane == 0) mbar_arrive(q_full);
@@ -464,13 +505,13 @@ __global__ void __launch_bounds__(kLrThreads, 1) latent_rows_kernel(LatentRowsPa
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[i & 1], (uint32_t)((i >> 1) & 1), abort_flag, p.status)) && ok;
       tc_fence_after();
       float v[R];
+      {
+        uint32_t x[R / 16][16];
 #pragma unroll
-      for (int k = 0; k < R; k += 16) {
-        uint32_t x[16];
-        tmem_ld16(tmem + (i & 1) * R + lanes + k, x);
+        for (int k = 0; k < R / 16; ++k) tmem_ld16(tmem + (i & 1) * R + lanes + k * 16, x[k]);
         tmem_ld_wait();
 #pragma unroll
-        for (int j = 0; j < 16; ++j) v[k + j] = __uint_as_float(x[j]) * sc;
+        for (int r = 0; r < R; ++r) v[r] = __uint_as_float(x[r / 16][r % 16]) * sc;
       }
       const int k0 = (s_lo + i * 8) * 16, key = k0 + tid;
       if (k0 < all_lo || k0 + 127 > all_hi) {
@@ -480,16 +521,24 @@ __global__ void __launch_bounds__(kLrThreads, 1) latent_rows_kernel(LatentRowsPa
           if (key < vis.x || key > vis.y) v[r] = -INFINITY;
         }
       }
-      reduce_lanes<R, true>(v, lane, s_red + warp * R);
-      bar_sync(1, 128);
+      // most tiles outgrow no row's maximum: one vote, and the columns are reduced only where it says so
       bool grow = false;
-      if (tid < R) {
-        const float t = fmaxf(fmaxf(s_red[tid], s_red[R + tid]), fmaxf(s_red[2 * R + tid], s_red[3 * R + tid])), m = s_m[tid];
-        grow = t > m + kLrLazy || (m == -INFINITY && t != -INFINITY);
-        s_f[tid] = grow ? (m == -INFINITY ? 0.f : ex2(m - t)) : 1.f;
-        if (grow) s_m[tid] = t;
+#pragma unroll
+      for (int r = 0; r < R; r += 4) {
+        const float4 m = *reinterpret_cast<const float4*>(s_m + r);
+        grow |= v[r] > m.x + kLrLazy || v[r + 1] > m.y + kLrLazy || v[r + 2] > m.z + kLrLazy || v[r + 3] > m.w + kLrLazy;
       }
       const bool calm = bar_red_and(2, 128, !grow);
+      if (!calm) {
+        reduce_lanes<R, true>(v, lane, s_red + warp * R);
+        bar_sync(1, 128);
+        if (tid < R) {
+          const float t = fmaxf(fmaxf(s_red[tid], s_red[R + tid]), fmaxf(s_red[2 * R + tid], s_red[3 * R + tid])), m = s_m[tid];
+          s_f[tid] = t > m + kLrLazy ? ex2(m - t) : 1.f;
+          if (t > m + kLrLazy) s_m[tid] = t;
+        }
+        bar_sync(1, 128);
+      }
       if (i > 0) ok = __all_sync(0xffffffffu, mbar_wait(pv_done, (uint32_t)((i - 1) & 1), abort_flag, p.status)) && ok;
       if (!calm) {
         tc_fence_after();
@@ -516,8 +565,8 @@ __global__ void __launch_bounds__(kLrThreads, 1) latent_rows_kernel(LatentRowsPa
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int r = g * 8 + j * 2;
-          const float m0 = s_m[r], m1 = s_m[r + 1];
-          const float a = ex2(v[r] - (m0 == -INFINITY ? 0.f : m0)), c = ex2(v[r + 1] - (m1 == -INFINITY ? 0.f : m1));
+          const float2 m = *reinterpret_cast<const float2*>(s_m + r);
+          const float a = ex2(v[r] - m.x), c = ex2(v[r + 1] - m.y);
           l[r] += a;
           l[r + 1] += c;
           hi[j] = pack_bf16x2(a, c);
@@ -579,30 +628,31 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(LatentRowsParams p,
   const int b = blockIdx.y, rr = blockIdx.x, r0 = p.q_start[b], qlen = p.q_start[b + 1] - r0;
   if (qlen > p.max_tokens || rr >= qlen * p.heads) return;
   const size_t w = ((size_t)b * p.row_blocks + rr / R) * p.splits * R + rr % R;      // split s at w + s * R
-  float m = -INFINITY, l = 0.f;
+  float m = kLrNone, l = 0.f;
   for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.part_ml[(w + (size_t)s * R) * 2]);
   for (int s = 0; s < p.splits; ++s) {
     const float* ml = p.part_ml + (w + (size_t)s * R) * 2;
-    if (ml[0] != -INFINITY) l = fmaf(ex2(ml[0] - m), ml[1], l);
+    l = fmaf(ex2(ml[0] - m), ml[1], l);
   }
   const float inv = 1.f / (l + (p.sink ? ex2(p.sink[rr % p.heads] * kLog2e - m) : 0.f));
   for (int c = threadIdx.x; c < p.rank; c += 128) {
     float o = 0.f;
     for (int s = 0; s < p.splits; ++s) {
       const float ms = p.part_ml[(w + (size_t)s * R) * 2];
-      if (ms != -INFINITY) o = fmaf(ex2(ms - m), p.part_o[(w + (size_t)s * R) * p.rank + c], o);
+      if (ms != kLrNone) o = fmaf(ex2(ms - m), p.part_o[(w + (size_t)s * R) * p.rank + c], o);
     }
     reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)r0 * p.heads + rr) * p.rank + c] = __float2bfloat16(o * inv);
   }
 }
 
 static int rows_smem(int R, int D, int stages) { return 128 + 128 + 8 * R * 4 + 2 * R * D + 512 * R + stages * 256 * D + 2048; }
-static constexpr int kLrSmem = 227 * 1024;
+static constexpr int kLrSmem = 227 * 1024, kLrSmemHalf = 113 * 1024;      // one CTA per SM, two
 
 template <int R>
 static int launch_rows(LatentRowsParams p, int B, int longest, cudaStream_t s) {
+  const int fit = R <= 32 && rows_smem(R, p.D, 1) <= kLrSmemHalf ? kLrSmemHalf : kLrSmem;
   int st = 4;
-  while (st > 1 && rows_smem(R, p.D, st) > kLrSmem) --st;
+  while (st > 1 && rows_smem(R, p.D, st) > fit) --st;
   const int sm = rows_smem(R, p.D, st);
   if (sm > kLrSmem || (2 + (p.rank + 127) / 128) * R > 512) return (int)cudaErrorInvalidValue;
   p.stages = st;
@@ -689,8 +739,11 @@ BLZ_API int blz_latent_prep(const void* proj, long long ld, long long q_off, lon
   const LatentPrepParams p = {proj, q_lat, pool, q_norm, c_norm, freq, positions, slot_mapping, ld, q_off, kv_off, page_stride, q_rank, rank,
                               rot, rot_dims, eps};
   const dim3 grid(T, pool ? 2 : 1);
-  if (f32) return (int)launch_pdl(latent_prep_kernel<float>, grid, dim3(128), 0, s, p);
-  return (int)launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, p);
+  if (f32) return (int)launch_pdl(latent_prep_kernel<float, 1>, grid, dim3(128), 0, s, p);
+  auto ok = [](const void* q) { return !q || (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  if (ok(proj) && ok(q_lat) && ok(pool) && ok(q_norm) && ok(c_norm) && (ld | q_off | kv_off | (long long)q_rank | (long long)rank | page_stride) % 8 == 0)
+    return (int)launch_pdl(latent_prep_kernel<__nv_bfloat16, 8>, grid, dim3(128), 0, s, p);
+  return (int)launch_pdl(latent_prep_kernel<__nv_bfloat16, 1>, grid, dim3(128), 0, s, p);
 }
 
 // Rotation of the queries q [T, heads, dim + rot]: rows of sequences with at most max_tokens new tokens into q_eff [T, heads, D], from
@@ -718,12 +771,14 @@ BLZ_API int blz_head_gemm(const void* a, long long lda, long long sa, const void
   return (int)launch_pdl(head_gemm_kernel, grid, dim3(128), 0, s, p, vec);
 }
 
-// Query rows per CTA of blz_latent_rows for sequences of up to `rows` (new tokens x heads) rows; 0: not these sizes.
-BLZ_API int blz_latent_rows_block(int rank, int rot, int rows) {
+// Query rows per CTA of blz_latent_rows for sequences of up to `rows` (new tokens x heads) rows; 0: not these sizes.  *per_sm (may be
+// null): how many CTAs share an SM.
+BLZ_API int blz_latent_rows_block(int rank, int rot, int rows, int* per_sm) {
   using namespace blz;
   const int D = up16(rank) + up16(rot), nvb = (rank + 127) / 128;
   int R = rows > 48 ? 64 : rows > 32 ? 48 : rows > 16 ? 32 : 16;
   while (R >= 16 && ((2 + nvb) * R > 512 || rows_smem(R, D, R > 16 ? 2 : 1) > kLrSmem)) R -= 16;
+  if (per_sm) *per_sm = R >= 16 && R <= 32 && rows_smem(R, D, 1) <= kLrSmemHalf ? 2 : 1;
   return R;
 }
 
