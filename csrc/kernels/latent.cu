@@ -191,6 +191,7 @@ struct HeadGemmParams {
   int M, N, K;
   RowFilter rows;
 };
+static constexpr int kHgStages = 4, kHgPitch = 72;             // tiles of 64 columns under way; row pitch: 8 rows cover all banks
 
 __global__ void __launch_bounds__(256) head_gemm_f32_kernel(HeadGemmParams p) {
   __shared__ float sa[16][68], sb[16][68];
@@ -240,10 +241,11 @@ __device__ __forceinline__ void lt_mma(float (&c)[4], const uint32_t (&a)[4], ui
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// bf16: few rows against many small weights, so the products ride on the reads (warp-level MMAs); 4 warps of 32 x 32 outputs
+// bf16: few rows against many small weights, so the products ride on the reads (warp-level MMAs); 4 warps of 32 x 32 outputs, the next
+// tiles of both operands on their way as asynchronous copies
 __global__ void __launch_bounds__(128) head_gemm_kernel(HeadGemmParams p, int vec) {
-  constexpr int LD = 72;                             // row pitch of 64 columns: 8 rows cover all banks
-  __shared__ __align__(16) __nv_bfloat16 sa[64 * LD], sb[64 * LD];
+  constexpr int LD = kHgPitch;
+  extern __shared__ __align__(16) __nv_bfloat16 ring[];          // [stages][A 64 x LD | B 64 x LD]
   __shared__ int any;
   pdl_trigger();
   pdl_wait();
@@ -255,28 +257,32 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(HeadGemmParams p, int ve
   if (!any) return;
   const __nv_bfloat16* A = reinterpret_cast<const __nv_bfloat16*>(p.a) + h * p.sa;
   const __nv_bfloat16* B = reinterpret_cast<const __nv_bfloat16*>(p.b) + (size_t)h * p.N * p.K;
-  const int wm = (warp & 1) * 32, wn = (warp >> 1) * 32;
+  const int wm = (warp & 1) * 32, wn = (warp >> 1) * 32, tiles = (p.K + 63) / 64;
   const bool upper = m0 + 32 < p.M;                  // the second half of the rows exists
-  float acc[2][4][4] = {};
-  for (int k0 = 0; k0 < p.K; k0 += 64) {
-    for (int i = tid; i < 1024; i += 128) {
-      const int which = i >> 9, r = i >> 3 & 63, c = (i & 7) * 8, row = (which ? n0 : m0) + r, lim = which ? p.N : p.M;
-      const __nv_bfloat16* src = (which ? B + (size_t)row * p.K : A + (size_t)row * p.lda) + k0 + c;
-      uint4 u = make_uint4(0, 0, 0, 0);
-      if (row < lim && k0 + c < p.K) {
-        if (vec) {
-          u = *reinterpret_cast<const uint4*>(src);
-        } else {
-          __nv_bfloat16* e = reinterpret_cast<__nv_bfloat16*>(&u);
-          for (int k = 0; k < 8; ++k)
-            if (k0 + c + k < p.K) e[k] = src[k];
-        }
+  auto send = [&](int t) {
+    __nv_bfloat16* dst = ring + (t % kHgStages) * 128 * LD;
+    for (int i = tid; t < tiles && i < 1024; i += 128) {
+      const int which = i >> 9, r = i >> 3 & 63, c = t * 64 + (i & 7) * 8, row = (which ? n0 : m0) + r, lim = which ? p.N : p.M;
+      const __nv_bfloat16* src = (which ? B + (size_t)row * p.K : A + (size_t)row * p.lda) + c;
+      __nv_bfloat16* to = dst + (which * 64 + r) * LD + (i & 7) * 8;
+      const bool live = row < lim && c < p.K;
+      if (vec) {
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(to)), "l"(live ? src : A), "r"(live ? 16 : 0) : "memory");
+      } else {
+        for (int k = 0; k < 8; ++k) to[k] = live && c + k < p.K ? src[k] : __float2bfloat16(0.f);
       }
-      *reinterpret_cast<uint4*>((which ? sb : sa) + r * LD + c) = u;
     }
-    __syncthreads();
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  float acc[2][4][4] = {};
+  for (int t = 0; t < kHgStages - 1; ++t) send(t);
+  for (int t = 0; t < tiles; ++t) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(kHgStages - 2) : "memory");
+    __syncthreads();                                 // tile t is there, and everyone is done with the slot that is filled next
+    send(t + kHgStages - 1);
+    const __nv_bfloat16 *sa = ring + (t % kHgStages) * 128 * LD, *sb = sa + 64 * LD;
     if (wm == 0 || upper) {
-      const int ks = min(64, p.K - k0);
+      const int ks = min(64, p.K - t * 64);
       for (int k = 0; k < ks; k += 16) {
         uint32_t a[2][4], bq[2][4];
 #pragma unroll
@@ -290,7 +296,6 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(HeadGemmParams p, int ve
           for (int j = 0; j < 4; ++j) lt_mma(acc[i][j], a[i], bq[j >> 1][(j & 1) * 2], bq[j >> 1][(j & 1) * 2 + 1]);
       }
     }
-    __syncthreads();
   }
   __nv_bfloat16* C = reinterpret_cast<__nv_bfloat16*>(p.c) + h * p.sc;
 #pragma unroll
@@ -318,7 +323,8 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(HeadGemmParams p, int ve
 //   S^T = C Q'^T     A = the 128 cached vectors (K-major), B = the R queries; 128 keys on the lanes, R columns, two buffers
 //   O^T += C^T P^T   A = 128 latent columns of the same block (MN-major), B = the weights [keys x R]; one accumulator per 128 columns
 // so that with few rows the tensor core spends N = R columns per key and not 128.  A weight enters as two bf16 numbers, value and
-// remainder, so it is not rounded to 8 bits.  Scores, weights and sums are fp32; a row's running maximum moves only when its scores
+// remainder, so it is not rounded to 8 bits: they are columns of their own (N = 2 R), since with few columns an MMA costs what its A
+// operand costs, and the two sums of a row meet at the end.  Scores, weights and sums are fp32; a row's running maximum moves only when its scores
 // outgrow it by 2^8, and then the accumulators are rescaled in tensor memory.
 // Warps 0-3: softmax (a key per thread), warp 4: page loader, warp 5: MMA issuer.
 struct LatentRowsParams {
@@ -393,6 +399,9 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
     return;
   }
   const int nvb = (p.rank + 127) / 128, tile = 256 * D;                            // accumulators; bytes of 128 cached vectors
+  const int* bt = p.block_table + (size_t)p.slots[b] * p.bt_stride;
+  auto page_of = [&](int i) { return lane < 8 ? bt[min(s_lo + i * 8 + lane, s_lo + s_n - 1)] : 0; };      // beyond the range: the last page again, masked
+  int page = warp == 4 ? page_of(0) : 0;
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem);
   uint64_t *k_full = bars, *k_empty = bars + 4, *s_full = bars + 8, *p_full = bars + 10, *pv_done = bars + 11, *q_full = bars + 12;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 13);
@@ -405,7 +414,7 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
   uint8_t* sP = sQ + 2 * R * D;
   uint8_t* ring = sP + 512 * R;
   uint32_t cols = 32;
-  while (cols < (uint32_t)((2 + nvb) * R)) cols *= 2;
+  while (cols < (uint32_t)((2 + 2 * nvb) * R)) cols *= 2;
   if (threadIdx.x == 0) {
     for (int i = 0; i < 4; ++i) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); }
     for (int i = 0; i < 2; ++i) mbar_init(&s_full[i], 1);
@@ -422,17 +431,16 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
   const uint32_t tmem = *tmem_slot;
   if (warp == 4) {
     // -------------------------------------------------------------- page loader
-    const int* bt = p.block_table + (size_t)p.slots[b] * p.bt_stride;
     int i = 0;
     for (; i < n; ++i) {
-      const int st = i % ST;
-      const int page = lane < 8 ? bt[min(s_lo + i * 8 + lane, s_lo + s_n - 1)] : 0;       // beyond the range: the last page again, masked
+      const int st = i % ST, next = i + 1 < n ? page_of(i + 1) : 0;
       if (!__all_sync(0xffffffffu, mbar_wait(&k_empty[st], (uint32_t)(((i / ST) & 1) ^ 1), abort_flag, p.status))) break;
       if (lane == 0) mbar_expect_tx(&k_full[st], tile);
       __syncwarp();
       if (lane < 8)
         bulk_load(ring + st * tile + lane * 32 * D, reinterpret_cast<const __nv_bfloat16*>(p.pool) + (size_t)page * p.page_stride, 32 * D, &k_full[st]);
       __syncwarp();
+      page = next;
     }
     if (i < n)                               // given up: what was sent lands before the block may end
       for (int k = max(i - ST, 0); k < i; ++k) {
@@ -442,7 +450,7 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
   } else if (warp == 5) {
     // -------------------------------------------------------------- MMA issuer
     if (lane == 0) {
-      const uint32_t id_s = make_idesc(1, 1, 128, R), id_o = make_idesc(1, 1, 128, R, 1, 1);
+      const uint32_t id_s = make_idesc(1, 1, 128, R), id_o = make_idesc(1, 1, 128, 2 * R, 1, 1);
       const uint32_t qa = smem_u32(sQ), pa = smem_u32(sP), ra = smem_u32(ring);
       auto qk = [&](int i) {
         const uint32_t ka = ra + (i % ST) * tile;
@@ -465,10 +473,9 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
         tc_fence_after();
         const uint32_t va = ra + (i % ST) * tile;
         for (int v = 0; v < nvb; ++v)
-          for (int half = 0; half < 2; ++half)
-            for (int s = 0; s < 8; ++s)      // a page of 16 keys per MMA
-              mma_f16(tmem + (2 + v) * R, make_smem_desc(va + s * 32 * D + v * 2048, D * 16, 128, kSwzNone),
-                      make_smem_desc(pa + half * 256 * R + s * 32 * R, 16 * R, 128, kSwzNone), id_o, i > 0 || half > 0 || s > 0);
+          for (int s = 0; s < 8; ++s)        // a page of 16 keys per MMA
+            mma_f16(tmem + (2 + 2 * v) * R, make_smem_desc(va + s * 32 * D + v * 2048, D * 16, 128, kSwzNone),
+                    make_smem_desc(pa + s * 64 * R, 32 * R, 128, kSwzNone), id_o, i > 0 || s > 0);
         mma_commit(pv_done);
         mma_commit(&k_empty[i % ST]);
         if (i + ahead < n) {
@@ -545,20 +552,19 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
 #pragma unroll
         for (int r = 0; r < R; ++r) l[r] *= s_f[r];
         if (i > 0) {
-          for (int c = 0; c < nvb; ++c)
+#pragma unroll 1
+          for (int k = 0; k < 2 * nvb * R; k += 16) {
+            uint32_t x[16];
+            tmem_ld16(tmem + 2 * R + lanes + k, x);
+            tmem_ld_wait();
 #pragma unroll
-            for (int k = 0; k < R; k += 16) {
-              uint32_t x[16];
-              tmem_ld16(tmem + (2 + c) * R + lanes + k, x);
-              tmem_ld_wait();
-#pragma unroll
-              for (int j = 0; j < 16; ++j) x[j] = __float_as_uint(__uint_as_float(x[j]) * s_f[k + j]);
-              tmem_st16(tmem + (2 + c) * R + lanes + k, x);
-            }
+            for (int j = 0; j < 16; ++j) x[j] = __float_as_uint(__uint_as_float(x[j]) * s_f[k % R + j]);
+            tmem_st16(tmem + 2 * R + lanes + k, x);
+          }
           tmem_st_wait();
         }
       }
-      uint8_t* dst = sP + (tid >> 3) * (R / 8) * 128 + (tid & 7) * 16;
+      uint8_t* dst = sP + (tid >> 3) * 32 * R + (tid & 7) * 16;
 #pragma unroll
       for (int g = 0; g < R / 8; ++g) {
         uint32_t hi[4], lo[4];
@@ -573,7 +579,7 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
           lo[j] = pack_bf16x2(a - __uint_as_float(hi[j] << 16), c - __uint_as_float(hi[j] & 0xffff0000u));
         }
         *reinterpret_cast<uint4*>(dst + g * 128) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-        *reinterpret_cast<uint4*>(dst + 256 * R + g * 128) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        *reinterpret_cast<uint4*>(dst + 16 * R + g * 128) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
       }
       fence_async_smem();
       tc_fence_before();
@@ -595,22 +601,40 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
       }
     }
     bar_sync(1, 128);
+    __nv_bfloat16* s_out = reinterpret_cast<__nv_bfloat16*>(ring);         // [R][128]: the tiles have been used
+    float* part = p.part_o + w0 * p.rank;
     for (int c = 0; c < nvb; ++c) {
-      const int col = c * 128 + warp * 32 + lane;
-#pragma unroll
-      for (int k = 0; k < R; k += 16) {
-        uint32_t x[16];
-        tmem_ld16(tmem + (2 + c) * R + lanes + k, x);
+      const int at = c * 128, width = min(128, p.rank - at);
+#pragma unroll 1
+      for (int k = 0; k < R; k += 16) {                  // (loops that run once per CTA are kept short: their code is not in the cache)
+        uint32_t x[16], y[16];
+        tmem_ld16(tmem + (2 + 2 * c) * R + lanes + k, x);
+        tmem_ld16(tmem + (3 + 2 * c) * R + lanes + k, y);
         tmem_ld_wait();
-        if (col >= p.rank || !ok) continue;
 #pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          if (k + j >= live) break;
-          const float o = __uint_as_float(x[j]) * s_f[k + j];
-          if (p.splits > 1) p.part_o[(w0 + k + j) * p.rank + col] = o;
-          else reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)r0 * H + (size_t)rb * R + k + j) * p.rank + col] = __float2bfloat16(o);
+        for (int j = 0; j < 16; ++j) x[j] = __float_as_uint((__uint_as_float(x[j]) + __uint_as_float(y[j])) * s_f[k + j]);
+        if (p.splits == 1) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) s_out[(k + j) * 128 + tid] = __float2bfloat16(__uint_as_float(x[j]));
+        } else if (tid < width) {
+          float* dst = part + (size_t)k * p.rank + at + tid;             // rows beyond the live ones have a place too
+#pragma unroll
+          for (int j = 0; j < 16; ++j) dst[j * p.rank] = __uint_as_float(x[j]);
         }
       }
+      if (p.splits > 1) continue;
+      bar_sync(1, 128);
+      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + ((size_t)r0 * H + (size_t)rb * R) * p.rank + at;
+      if (ok && p.rank % 8 == 0) {
+        for (int i = tid; i < live * 16; i += 128) {
+          const int r = i >> 4, j = (i & 15) * 8;
+          if (j < width) *reinterpret_cast<uint4*>(out + (size_t)r * p.rank + j) = *reinterpret_cast<const uint4*>(s_out + r * 128 + j);
+        }
+      } else if (ok) {
+        for (int i = tid; i < live * 128; i += 128)
+          if (tid < width) out[(size_t)(i >> 7) * p.rank + tid] = s_out[i];
+      }
+      bar_sync(1, 128);
     }
   }
   tc_fence_before();
@@ -627,21 +651,25 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(LatentRowsParams p,
   pdl_wait();
   const int b = blockIdx.y, rr = blockIdx.x, r0 = p.q_start[b], qlen = p.q_start[b + 1] - r0;
   if (qlen > p.max_tokens || rr >= qlen * p.heads) return;
+  __shared__ float s_w[32];
   const size_t w = ((size_t)b * p.row_blocks + rr / R) * p.splits * R + rr % R;      // split s at w + s * R
-  float m = kLrNone, l = 0.f;
-  for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.part_ml[(w + (size_t)s * R) * 2]);
-  for (int s = 0; s < p.splits; ++s) {
-    const float* ml = p.part_ml + (w + (size_t)s * R) * 2;
-    l = fmaf(ex2(ml[0] - m), ml[1], l);
-  }
-  const float inv = 1.f / (l + (p.sink ? ex2(p.sink[rr % p.heads] * kLog2e - m) : 0.f));
+  const int lane = threadIdx.x & 31;
+  const bool mine = lane < p.splits;
+  const float m = mine ? p.part_ml[(w + (size_t)lane * R) * 2] : kLrNone, l = mine ? p.part_ml[(w + (size_t)lane * R) * 2 + 1] : 0.f;
+  const float top = warp_max(m), f = m == kLrNone ? 0.f : ex2(m - top);
+  const float inv = 1.f / (warp_sum(f * l) + (p.sink ? ex2(p.sink[rr % p.heads] * kLog2e - top) : 0.f));
+  if (threadIdx.x < 32) s_w[lane] = f * inv;
+  __syncthreads();
   for (int c = threadIdx.x; c < p.rank; c += 128) {
     float o = 0.f;
-    for (int s = 0; s < p.splits; ++s) {
-      const float ms = p.part_ml[(w + (size_t)s * R) * 2];
-      if (ms != kLrNone) o = fmaf(ex2(ms - m), p.part_o[(w + (size_t)s * R) * p.rank + c], o);
+    for (int s0 = 0; s0 < p.splits; s0 += 8) {
+      float x[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) x[k] = s0 + k < p.splits && s_w[s0 + k] != 0.f ? p.part_o[(w + (size_t)(s0 + k) * R) * p.rank + c] : 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) o = fmaf(x[k], s_w[(s0 + k) & 31], o);
     }
-    reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)r0 * p.heads + rr) * p.rank + c] = __float2bfloat16(o * inv);
+    reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)r0 * p.heads + rr) * p.rank + c] = __float2bfloat16(o);
   }
 }
 
@@ -654,7 +682,7 @@ static int launch_rows(LatentRowsParams p, int B, int longest, cudaStream_t s) {
   int st = 4;
   while (st > 1 && rows_smem(R, p.D, st) > fit) --st;
   const int sm = rows_smem(R, p.D, st);
-  if (sm > kLrSmem || (2 + (p.rank + 127) / 128) * R > 512) return (int)cudaErrorInvalidValue;
+  if (sm > kLrSmem || (2 + 2 * ((p.rank + 127) / 128)) * R > 512 || p.splits > 32) return (int)cudaErrorInvalidValue;
   p.stages = st;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(latent_rows_kernel<R>, kLrSmem);
@@ -768,7 +796,11 @@ BLZ_API int blz_head_gemm(const void* a, long long lda, long long sa, const void
   const dim3 grid((N + 63) / 64, (M + 63) / 64, heads);
   if (f32) return (int)launch_pdl(head_gemm_f32_kernel, grid, dim3(256), 0, s, p);
   const int vec = aligned16(a) && aligned16(b) && (reinterpret_cast<uintptr_t>(c) & 3) == 0 && (lda | sa | (long long)K) % 8 == 0 && (ldc | sc | (long long)N) % 2 == 0;
-  return (int)launch_pdl(head_gemm_kernel, grid, dim3(128), 0, s, p, vec);
+  constexpr int sm = kHgStages * 128 * kHgPitch * 2;
+  static PerDeviceOnce once;
+  const cudaError_t e = once.smem_limit(head_gemm_kernel, sm);
+  if (e != cudaSuccess) return (int)e;
+  return (int)launch_pdl(head_gemm_kernel, grid, dim3(128), sm, s, p, vec);
 }
 
 // Query rows per CTA of blz_latent_rows for sequences of up to `rows` (new tokens x heads) rows; 0: not these sizes.  *per_sm (may be
@@ -777,7 +809,7 @@ BLZ_API int blz_latent_rows_block(int rank, int rot, int rows, int* per_sm) {
   using namespace blz;
   const int D = up16(rank) + up16(rot), nvb = (rank + 127) / 128;
   int R = rows > 48 ? 64 : rows > 32 ? 48 : rows > 16 ? 32 : 16;
-  while (R >= 16 && ((2 + nvb) * R > 512 || rows_smem(R, D, R > 16 ? 2 : 1) > kLrSmem)) R -= 16;
+  while (R >= 16 && ((2 + 2 * nvb) * R > 512 || rows_smem(R, D, R > 16 ? 2 : 1) > kLrSmem)) R -= 16;
   if (per_sm) *per_sm = R >= 16 && R <= 32 && rows_smem(R, D, 1) <= kLrSmemHalf ? 2 : 1;
   return R;
 }
