@@ -326,7 +326,7 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(HeadGemmParams p, int ve
 // remainder, so it is not rounded to 8 bits: they are columns of their own (N = 2 R), since with few columns an MMA costs what its A
 // operand costs, and the two sums of a row meet at the end.  Scores, weights and sums are fp32; a row's running maximum moves only when its scores
 // outgrow it by 2^8, and then the accumulators are rescaled in tensor memory.
-// Warps 0-3: softmax (a key per thread), warp 4: page loader, warp 5: MMA issuer.
+// Softmax warps: a key per thread, R / 2 columns (16 rows: all) in each of the two warpgroups; then a page loader and an MMA issuer.
 struct LatentRowsParams {
   const void* q;               // [T, heads, D]
   void* out;                   // [T, heads, rank]
@@ -340,8 +340,10 @@ struct LatentRowsParams {
   int* status;
 };
 
-static constexpr int kLrThreads = 192;
+__host__ __device__ constexpr int lr_groups(int R) { return R >= 32 ? 2 : 1; }      // softmax warpgroups
+__host__ __device__ constexpr int lr_threads(int R) { return lr_groups(R) * 128 + 64; }
 static constexpr float kLrLazy = 8.f;
+static constexpr int kLrRowBytes = 48;         // shared memory per row besides the operands, a multiple of 16
 static constexpr float kLrNone = -1e30f;       // the maximum of a row that has seen no key
 
 template <bool MAX>
@@ -381,7 +383,8 @@ __device__ __forceinline__ void reduce_lanes(const float (&v)[R], int lane, floa
 }
 
 template <int R>
-__global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kernel(LatentRowsParams p) {
+__global__ void __launch_bounds__(lr_threads(R), R <= 32 ? 2 : 1) latent_rows_kernel(LatentRowsParams p) {
+  constexpr int WG = lr_groups(R), RC = R / WG, NT = WG * 128, kLoader = WG * 4, kIssuer = kLoader + 1;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~uintptr_t(127));
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, H = p.heads, D = p.D, ST = p.stages;
@@ -395,13 +398,13 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
   const int s_lo = pg_lo + split * per, s_n = min(per, pg_lo + pages - s_lo), n = s_n > 0 ? (s_n + 7) / 8 : 0;
   const size_t w0 = (((size_t)b * p.row_blocks + rb) * p.splits + split) * R;        // this CTA's rows in the workspace
   if (n == 0) {
-    for (int r = threadIdx.x; r < R; r += kLrThreads) { p.part_ml[(w0 + r) * 2] = kLrNone; p.part_ml[(w0 + r) * 2 + 1] = 0.f; }
+    for (int r = threadIdx.x; r < R; r += lr_threads(R)) { p.part_ml[(w0 + r) * 2] = kLrNone; p.part_ml[(w0 + r) * 2 + 1] = 0.f; }
     return;
   }
   const int nvb = (p.rank + 127) / 128, tile = 256 * D;                            // accumulators; bytes of 128 cached vectors
   const int* bt = p.block_table + (size_t)p.slots[b] * p.bt_stride;
   auto page_of = [&](int i) { return lane < 8 ? bt[min(s_lo + i * 8 + lane, s_lo + s_n - 1)] : 0; };      // beyond the range: the last page again, masked
-  int page = warp == 4 ? page_of(0) : 0;
+  int page = warp == kLoader ? page_of(0) : 0;
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem);
   uint64_t *k_full = bars, *k_empty = bars + 4, *s_full = bars + 8, *p_full = bars + 10, *pv_done = bars + 11, *q_full = bars + 12;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 13);
@@ -409,8 +412,9 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
   float* s_red = reinterpret_cast<float*>(smem + 128);         // [4][R]
   float* s_m = s_red + 4 * R;
   float* s_f = s_m + R;
-  int2* s_vis = reinterpret_cast<int2*>(s_f + R);              // first and last visible key of a row
-  uint8_t* sQ = smem + 128 + 8 * R * 4;
+  float* s_t = s_f + R;                                        // products above which a row's maximum moves
+  int2* s_vis = reinterpret_cast<int2*>(s_t + R);              // first and last visible key of a row
+  uint8_t* sQ = smem + 128 + kLrRowBytes * R;
   uint8_t* sP = sQ + 2 * R * D;
   uint8_t* ring = sP + 512 * R;
   uint32_t cols = 32;
@@ -418,18 +422,18 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
   if (threadIdx.x == 0) {
     for (int i = 0; i < 4; ++i) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); }
     for (int i = 0; i < 2; ++i) mbar_init(&s_full[i], 1);
-    mbar_init(p_full, 4);
+    mbar_init(p_full, WG * 4);
     mbar_init(pv_done, 1);
-    mbar_init(q_full, 4);
+    mbar_init(q_full, WG * 4);
     *abort_flag = 0;
     mbar_fence_init();
   }
-  if (warp == 5) tmem_alloc(tmem_slot, cols);
+  if (warp == kIssuer) tmem_alloc(tmem_slot, cols);
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_slot;
-  if (warp == 4) {
+  if (warp == kLoader) {
     // -------------------------------------------------------------- page loader
     int i = 0;
     for (; i < n; ++i) {
@@ -447,7 +451,7 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
         const long long t0 = clock64();
         while (!mbar_try_sleep(&k_full[k % ST], (uint32_t)((k / ST) & 1), 20000u) && clock64() - t0 < kSpinLimit) {}
       }
-  } else if (warp == 5) {
+  } else if (warp == kIssuer) {
     // -------------------------------------------------------------- MMA issuer
     if (lane == 0) {
       const uint32_t id_s = make_idesc(1, 1, 128, R), id_o = make_idesc(1, 1, 128, 2 * R, 1, 1);
@@ -459,18 +463,7 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
                   id_s, s > 0);
         mma_commit(&s_full[i & 1]);
       };
-      auto have = [&](int i) { return mbar_wait(&k_full[i % ST], (uint32_t)((i / ST) & 1), abort_flag, p.status); };
-      const int ahead = ST > 1 ? 2 : 1;
-      bool ok = mbar_wait(q_full, 0, abort_flag, p.status);
-      tc_fence_after();
-      for (int j = 0; j < min(ahead, n) && ok; ++j) {
-        ok = have(j);
-        if (ok) qk(j);
-      }
-      for (int i = 0; i < n && ok; ++i) {
-        ok = mbar_wait(p_full, (uint32_t)(i & 1), abort_flag, p.status);
-        if (!ok) break;
-        tc_fence_after();
+      auto pv = [&](int i) {
         const uint32_t va = ra + (i % ST) * tile;
         for (int v = 0; v < nvb; ++v)
           for (int s = 0; s < 8; ++s)        // a page of 16 keys per MMA
@@ -478,101 +471,120 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
                     make_smem_desc(pa + s * 64 * R, 32 * R, 128, kSwzNone), id_o, i > 0 || s > 0);
         mma_commit(pv_done);
         mma_commit(&k_empty[i % ST]);
-        if (i + ahead < n) {
-          ok = have(i + ahead);
-          if (ok) qk(i + ahead);
+      };
+      bool ok = mbar_wait(q_full, 0, abort_flag, p.status);
+      tc_fence_after();
+      // whichever is ready: the value product of tile j, or the scores of tile i, at most two tiles ahead of it (two score buffers)
+      long long t0 = clock64();
+      for (int i = 0, j = 0; ok && j < n;) {
+        if (i > j && mbar_try(p_full, (uint32_t)(j & 1))) {
+          tc_fence_after();
+          pv(j++);
+        } else if (i < n && i < j + 2 && mbar_try(&k_full[i % ST], (uint32_t)((i / ST) & 1))) {
+          qk(i++);
+        } else {
+          if (*abort_flag) ok = false;
+          else if (clock64() - t0 > kSpinLimit) {
+            *abort_flag = 1;
+            if (p.status) atomicCAS(p.status, kOk, kErrMbarTimeout);
+            ok = false;
+          }
+          continue;
         }
+        t0 = clock64();
       }
     }
   } else {
     // -------------------------------------------------------------- softmax: this thread's key of every tile
     const int tid = threadIdx.x;
-    const uint32_t lanes = (uint32_t)(warp * 32) << 16;
+    const int quad = warp & 3, c0 = (warp >> 2) * RC, key_of = tid & 127;        // this thread's lane quadrant, first column and key
+    const uint32_t lanes = (uint32_t)(quad * 32) << 16;
     const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + ((size_t)r0 * H + (size_t)rb * R) * D;
     const int live = min(R, rows - rb * R);
-    copy_rows(reinterpret_cast<__nv_bfloat16*>(sQ), R, D, D, tid, 128, q, [&](int r) { return r < live ? q + (size_t)r * D : nullptr; });
+    copy_rows(reinterpret_cast<__nv_bfloat16*>(sQ), R, D, D, tid, NT, q, [&](int r) { return r < live ? q + (size_t)r * D : nullptr; });
     const int end = (s_lo + s_n) * 16 - 1;
     if (tid < R) {
       const int pos = tid < live ? pos0 + (rb * R + tid) / H : -1;
       s_vis[tid] = make_int2(first_key(pos, p.window), min(pos, end));
-      s_m[tid] = kLrNone;
+      s_m[tid] = s_t[tid] = kLrNone;
     }
     copies_wait();
     fence_async_smem();
     __syncwarp();
     if (lane == 0) mbar_arrive(q_full);
-    bar_sync(1, 128);
+    bar_sync(1, NT);
     const int all_lo = first_key(pos0 + tok_hi, p.window), all_hi = min(pos0 + tok_lo, end);        // what every row sees
     const float sc = p.scale * kLog2e;
-    float l[R];
+    float l[RC];
 #pragma unroll
-    for (int r = 0; r < R; ++r) l[r] = 0.f;
+    for (int r = 0; r < RC; ++r) l[r] = 0.f;
     bool ok = true;                          // once a wait has run out the others return at once; the barriers stay matched
     for (int i = 0; i < n; ++i) {
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[i & 1], (uint32_t)((i >> 1) & 1), abort_flag, p.status)) && ok;
       tc_fence_after();
-      float v[R];
+      float v[RC];
       {
-        uint32_t x[R / 16][16];
+        uint32_t x[RC / 16][16];
 #pragma unroll
-        for (int k = 0; k < R / 16; ++k) tmem_ld16(tmem + (i & 1) * R + lanes + k * 16, x[k]);
+        for (int k = 0; k < RC / 16; ++k) tmem_ld16(tmem + (i & 1) * R + lanes + c0 + k * 16, x[k]);
         tmem_ld_wait();
 #pragma unroll
-        for (int r = 0; r < R; ++r) v[r] = __uint_as_float(x[r / 16][r % 16]) * sc;
+        for (int r = 0; r < RC; ++r) v[r] = __uint_as_float(x[r / 16][r % 16]);
       }
-      const int k0 = (s_lo + i * 8) * 16, key = k0 + tid;
+      const int k0 = (s_lo + i * 8) * 16, key = k0 + key_of;
       if (k0 < all_lo || k0 + 127 > all_hi) {
 #pragma unroll
-        for (int r = 0; r < R; ++r) {
-          const int2 vis = s_vis[r];
+        for (int r = 0; r < RC; ++r) {
+          const int2 vis = s_vis[c0 + r];
           if (key < vis.x || key > vis.y) v[r] = -INFINITY;
         }
       }
       // most tiles outgrow no row's maximum: one vote, and the columns are reduced only where it says so
       bool grow = false;
 #pragma unroll
-      for (int r = 0; r < R; r += 4) {
-        const float4 m = *reinterpret_cast<const float4*>(s_m + r);
-        grow |= v[r] > m.x + kLrLazy || v[r + 1] > m.y + kLrLazy || v[r + 2] > m.z + kLrLazy || v[r + 3] > m.w + kLrLazy;
+      for (int r = 0; r < RC; r += 4) {
+        const float4 t = *reinterpret_cast<const float4*>(s_t + c0 + r);
+        grow |= v[r] > t.x || v[r + 1] > t.y || v[r + 2] > t.z || v[r + 3] > t.w;
       }
-      const bool calm = bar_red_and(2, 128, !grow);
+      const bool calm = bar_red_and(2, NT, !grow);
       if (!calm) {
-        reduce_lanes<R, true>(v, lane, s_red + warp * R);
-        bar_sync(1, 128);
+        reduce_lanes<RC, true>(v, lane, s_red + quad * R + c0);
+        bar_sync(1, NT);
         if (tid < R) {
-          const float t = fmaxf(fmaxf(s_red[tid], s_red[R + tid]), fmaxf(s_red[2 * R + tid], s_red[3 * R + tid])), m = s_m[tid];
+          const float t = fmaxf(fmaxf(s_red[tid], s_red[R + tid]), fmaxf(s_red[2 * R + tid], s_red[3 * R + tid])) * sc, m = s_m[tid];
           s_f[tid] = t > m + kLrLazy ? ex2(m - t) : 1.f;
-          if (t > m + kLrLazy) s_m[tid] = t;
+          if (t > m + kLrLazy) { s_m[tid] = t; s_t[tid] = (t + kLrLazy) / sc; }
         }
-        bar_sync(1, 128);
+        bar_sync(1, NT);
       }
       if (i > 0) ok = __all_sync(0xffffffffu, mbar_wait(pv_done, (uint32_t)((i - 1) & 1), abort_flag, p.status)) && ok;
       if (!calm) {
         tc_fence_after();
 #pragma unroll
-        for (int r = 0; r < R; ++r) l[r] *= s_f[r];
+        for (int r = 0; r < RC; ++r) l[r] *= s_f[c0 + r];
         if (i > 0) {
 #pragma unroll 1
-          for (int k = 0; k < 2 * nvb * R; k += 16) {
+          for (int k = 0; k < 2 * nvb * RC; k += 16) {
+            const int at = (2 + k / RC) * R + c0 + k % RC;
             uint32_t x[16];
-            tmem_ld16(tmem + 2 * R + lanes + k, x);
+            tmem_ld16(tmem + at + lanes, x);
             tmem_ld_wait();
 #pragma unroll
-            for (int j = 0; j < 16; ++j) x[j] = __float_as_uint(__uint_as_float(x[j]) * s_f[k % R + j]);
-            tmem_st16(tmem + 2 * R + lanes + k, x);
+            for (int j = 0; j < 16; ++j) x[j] = __float_as_uint(__uint_as_float(x[j]) * s_f[c0 + k % RC + j]);
+            tmem_st16(tmem + at + lanes, x);
           }
           tmem_st_wait();
         }
       }
-      uint8_t* dst = sP + (tid >> 3) * 32 * R + (tid & 7) * 16;
+      uint8_t* dst = sP + (key_of >> 3) * 32 * R + (key_of & 7) * 16 + c0 * 16;
 #pragma unroll
-      for (int g = 0; g < R / 8; ++g) {
+      for (int g = 0; g < RC / 8; ++g) {
         uint32_t hi[4], lo[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int r = g * 8 + j * 2;
-          const float2 m = *reinterpret_cast<const float2*>(s_m + r);
-          const float a = ex2(v[r] - m.x), c = ex2(v[r + 1] - m.y);
+          const float2 m = *reinterpret_cast<const float2*>(s_m + c0 + r);
+          const float a = ex2(fmaf(v[r], sc, -m.x)), c = ex2(fmaf(v[r + 1], sc, -m.y));
           l[r] += a;
           l[r + 1] += c;
           hi[j] = pack_bf16x2(a, c);
@@ -588,8 +600,8 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
     }
     ok = __all_sync(0xffffffffu, mbar_wait(pv_done, (uint32_t)((n - 1) & 1), abort_flag, p.status)) && ok;
     tc_fence_after();
-    reduce_lanes<R, false>(l, lane, s_red + warp * R);
-    bar_sync(1, 128);
+    reduce_lanes<RC, false>(l, lane, s_red + quad * R + c0);
+    bar_sync(1, NT);
     if (tid < R) {
       const float sum = s_red[tid] + s_red[R + tid] + s_red[2 * R + tid] + s_red[3 * R + tid], m = s_m[tid];
       if (p.splits > 1) {
@@ -600,13 +612,13 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
         s_f[tid] = 1.f / (sum + (p.sink && tid < live ? ex2(p.sink[(rb * R + tid) % H] * kLog2e - m) : 0.f));
       }
     }
-    bar_sync(1, 128);
+    bar_sync(1, NT);
     __nv_bfloat16* s_out = reinterpret_cast<__nv_bfloat16*>(ring);         // [R][128]: the tiles have been used
     float* part = p.part_o + w0 * p.rank;
     for (int c = 0; c < nvb; ++c) {
       const int at = c * 128, width = min(128, p.rank - at);
 #pragma unroll 1
-      for (int k = 0; k < R; k += 16) {                  // (loops that run once per CTA are kept short: their code is not in the cache)
+      for (int k = c0; k < c0 + RC; k += 16) {           // (loops that run once per CTA are kept short: their code is not in the cache)
         uint32_t x[16], y[16];
         tmem_ld16(tmem + (2 + 2 * c) * R + lanes + k, x);
         tmem_ld16(tmem + (3 + 2 * c) * R + lanes + k, y);
@@ -615,31 +627,31 @@ __global__ void __launch_bounds__(kLrThreads, R <= 32 ? 2 : 1) latent_rows_kerne
         for (int j = 0; j < 16; ++j) x[j] = __float_as_uint((__uint_as_float(x[j]) + __uint_as_float(y[j])) * s_f[k + j]);
         if (p.splits == 1) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) s_out[(k + j) * 128 + tid] = __float2bfloat16(__uint_as_float(x[j]));
-        } else if (tid < width) {
-          float* dst = part + (size_t)k * p.rank + at + tid;             // rows beyond the live ones have a place too
+          for (int j = 0; j < 16; ++j) s_out[(k + j) * 128 + key_of] = __float2bfloat16(__uint_as_float(x[j]));
+        } else if (key_of < width) {
+          float* dst = part + (size_t)k * p.rank + at + key_of;             // rows beyond the live ones have a place too
 #pragma unroll
           for (int j = 0; j < 16; ++j) dst[j * p.rank] = __uint_as_float(x[j]);
         }
       }
       if (p.splits > 1) continue;
-      bar_sync(1, 128);
+      bar_sync(1, NT);
       __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + ((size_t)r0 * H + (size_t)rb * R) * p.rank + at;
       if (ok && p.rank % 8 == 0) {
-        for (int i = tid; i < live * 16; i += 128) {
+        for (int i = tid; i < live * 16; i += NT) {
           const int r = i >> 4, j = (i & 15) * 8;
           if (j < width) *reinterpret_cast<uint4*>(out + (size_t)r * p.rank + j) = *reinterpret_cast<const uint4*>(s_out + r * 128 + j);
         }
       } else if (ok) {
-        for (int i = tid; i < live * 128; i += 128)
-          if (tid < width) out[(size_t)(i >> 7) * p.rank + tid] = s_out[i];
+        for (int i = tid; i < live * 128; i += NT)
+          if (key_of < width) out[(size_t)(i >> 7) * p.rank + key_of] = s_out[i];
       }
-      bar_sync(1, 128);
+      bar_sync(1, NT);
     }
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 5) {
+  if (warp == kIssuer) {
     tc_fence_after();
     tmem_dealloc(tmem, cols);
   }
@@ -673,7 +685,7 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(LatentRowsParams p,
   }
 }
 
-static int rows_smem(int R, int D, int stages) { return 128 + 128 + 8 * R * 4 + 2 * R * D + 512 * R + stages * 256 * D + 2048; }
+static int rows_smem(int R, int D, int stages) { return 128 + 128 + kLrRowBytes * R + 2 * R * D + 512 * R + stages * 256 * D + 2048; }
 static constexpr int kLrSmem = 227 * 1024, kLrSmemHalf = 113 * 1024;      // one CTA per SM, two
 
 template <int R>
@@ -687,7 +699,7 @@ static int launch_rows(LatentRowsParams p, int B, int longest, cudaStream_t s) {
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(latent_rows_kernel<R>, kLrSmem);
   if (e != cudaSuccess) return (int)e;
-  e = launch_pdl(latent_rows_kernel<R>, dim3(p.row_blocks * p.splits, B), dim3(kLrThreads), sm, s, p);
+  e = launch_pdl(latent_rows_kernel<R>, dim3(p.row_blocks * p.splits, B), dim3(lr_threads(R)), sm, s, p);
   if (e != cudaSuccess || p.splits == 1) return (int)e;
   return (int)launch_pdl(latent_combine_kernel, dim3(longest * p.heads, B), dim3(128), 0, s, p, R);
 }
@@ -808,9 +820,10 @@ BLZ_API int blz_head_gemm(const void* a, long long lda, long long sa, const void
 BLZ_API int blz_latent_rows_block(int rank, int rot, int rows, int* per_sm) {
   using namespace blz;
   const int D = up16(rank) + up16(rot), nvb = (rank + 127) / 128;
-  int R = rows > 48 ? 64 : rows > 32 ? 48 : rows > 16 ? 32 : 16;
-  while (R >= 16 && ((2 + 2 * nvb) * R > 512 || rows_smem(R, D, R > 16 ? 2 : 1) > kLrSmem)) R -= 16;
-  if (per_sm) *per_sm = R >= 16 && R <= 32 && rows_smem(R, D, 1) <= kLrSmemHalf ? 2 : 1;
+  int R = rows > 32 ? 64 : rows > 16 ? 32 : 16;
+  while (R >= 16 && ((2 + 2 * nvb) * R > 512 || rows_smem(R, D, R > 16 ? 2 : 1) > kLrSmem)) R /= 2;
+  if (R < 16) R = 0;
+  if (per_sm) *per_sm = R && R <= 32 && rows_smem(R, D, 1) <= kLrSmemHalf ? 2 : 1;
   return R;
 }
 
@@ -831,7 +844,6 @@ BLZ_API int blz_latent_rows(const void* q, void* out, const void* pool, long lon
   switch (R) {
     case 16: return launch_rows<16>(p, B, longest, s);
     case 32: return launch_rows<32>(p, B, longest, s);
-    case 48: return launch_rows<48>(p, B, longest, s);
     case 64: return launch_rows<64>(p, B, longest, s);
   }
   return (int)cudaErrorInvalidValue;
