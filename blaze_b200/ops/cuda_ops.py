@@ -207,7 +207,8 @@ class CudaOps:
         lib.blz_gemm_simple_experts.argtypes = [VP, LL, VP, VP, LL] + [_c.c_int] * 3 + [VP, VP, _c.c_int, VP]
         # latent attention
         lib.blz_latent_prep.argtypes = [VP, LL, LL, LL, VP, VP, LL, VP, VP, VP, VP, VP] + [_c.c_int] * 5 + [_c.c_float, _c.c_int, VP]
-        lib.blz_latent_rot.argtypes = [VP] * 6 + [_c.c_int] * 8 + [VP]
+        lib.blz_latent_rot.argtypes = [VP] * 5 + [_c.c_int] * 7 + [VP]
+        lib.blz_latent_map.argtypes = [VP] * 5 + [_c.c_int] * 6 + [VP, VP, _c.c_int, _c.c_int, VP]
         lib.blz_head_gemm.argtypes = [VP, LL, LL, VP, VP, LL, LL] + [_c.c_int] * 4 + [VP, VP, _c.c_int, _c.c_int, VP]
         lib.blz_latent_rows_block.restype = _c.c_int
         lib.blz_latent_rows_block.argtypes = [_c.c_int] * 3 + [VP]
@@ -509,14 +510,16 @@ class CudaOps:
 
     def linear(self, lin: Linear, x, out_dtype=None, out: Optional[torch.Tensor] = None, bn: int = 0, max_ctas: int = 0,
                wide: Optional[bool] = None, ksplit: int = 0, swiglu: bool = False, argmax_parts=None, sk=None,
-               glu_limit: Optional[float] = None):
+               glu_limit: Optional[float] = None, relu2: bool = False):
         """``wide``: None = choose; False = the 128-column kernel (needed by the fused all-reduce epilogue); True = insist on
         the wide-N kernel (raises when the shape is not covered).  ``sk``: None = choose; False = never; True or a K-slice
         count 1..8 = the cluster split-K kernel (bf16 output, row-major weights).  ``swiglu`` with ``glu_limit``: the clamped
-        gated activation instead of SwiGLU."""
+        gated activation instead of SwiGLU.  ``relu2``: squared ReLU of the result."""
         pk = self.pack(lin, swiglu=swiglu)
         kind = pk["kind"]
-        act, limit = int(swiglu) if glu_limit is None else 2, float(glu_limit or 0.0)
+        act, limit = (3 if relu2 else int(swiglu)) if glu_limit is None else 2, float(glu_limit or 0.0)
+        if relu2:
+            wide = sk = False
         if kind == 5 or (kind == 0 and lin.K % 16):
             if swiglu or argmax_parts is not None:
                 raise CudaError("the CUDA-core GEMM has the plain epilogue only")
@@ -565,7 +568,7 @@ class CudaOps:
             x.wait = None
         big = self.NARROW_ALWAYS or (lin.N * lin.K >= 6144 * 4096 if M <= 32 else lin.N >= 16384)
         narrow = (M <= self.NARROW_ROWS and big and kind in (0, 1, 2) and lin.N % 128 == 0 and not f32 and argmax_parts is None
-                  and pending is None and not kt and wide is None and bn == 0 and (sk is None or sk is False)
+                  and pending is None and not kt and (wide is None or relu2) and bn == 0 and (sk is None or sk is False)
                   and (not swiglu or ld_out % 8 == 0) and (sfa is None or sfa.numel() >= 512))
         if narrow:
             self._check(self.lib.blz_gemm_narrow(kind, _ptr(a), lda, _ptr(w), ldb, _ptr(out), ld_out, M, lin.N, lin.K, _ptr(rs),
@@ -1041,7 +1044,9 @@ class CudaOps:
         return z
 
     def linear_relu2(self, lin: Linear, x):
-        return self.relu2_(self.linear(lin, x))
+        if lin.fmt != Format.DENSE or lin.w.dtype == torch.float32 or lin.K % 16:
+            return self.relu2_(self.linear(lin, x))
+        return self.linear(lin, x, relu2=True)
 
     def poly_norm(self, z, act, eps):
         out = torch.empty_like(z)
@@ -1087,16 +1092,18 @@ class CudaOps:
         most = self.LATENT_SHORT if wide else max(batch.max_q_len, 1)
         longest = max((n for n in lens if n <= most), default=0)
         D = (a.kv_rank + 15) // 16 * 16 + (a.rot_dim + 15) // 16 * 16
-        qe = torch.empty(T, H, D, dtype=q.dtype, device=self.device) if longest else None
-        rows = (_ptr(batch.seq_of_row), _ptr(batch.q_start))
-        self._check(self.lib.blz_latent_rot(_ptr(q), _ptr(qe), _ptr(A.freq), _ptr(batch.positions), *rows, T, H, a.dim, a.rot_dim,
-                                            a.rot.dims if a.rot is not None else 0, a.kv_rank, most, int(f32), self._stream()), "latent_rot")
+        rows, rot = (_ptr(batch.seq_of_row), _ptr(batch.q_start)), a.rot.dims if a.rot is not None else 0
         if longest:
-            self._head_gemm(q, a.dim + a.rot_dim, A.uk_t, qe.view(T, H * D), D, batch, most)
+            qe = torch.empty(T, H, D, dtype=q.dtype, device=self.device)
+            self._check(self.lib.blz_latent_map(_ptr(q), _ptr(A.uk_t), _ptr(qe), _ptr(A.freq), _ptr(batch.positions), T, H, a.dim, a.rot_dim, rot,
+                                                a.kv_rank, *rows, most, int(f32), self._stream()), "latent_map")
             lat = torch.empty(T, H * a.kv_rank, dtype=q.dtype, device=self.device)
             self.latent_rows(qe, M, batch, kv, layer_idx, longest, most, lat)
             self._head_gemm(lat, a.kv_rank, A.uv, out, a.vdim, batch, most)
         if any(n > most for n in lens):
+            if rot:
+                self._check(self.lib.blz_latent_rot(_ptr(q), _ptr(A.freq), _ptr(batch.positions), *rows, T, H, a.dim, a.rot_dim, rot, most, int(f32),
+                                                    self._stream()), "latent_rot")
             self._expanded_attention(q, M, batch, kv, self._expand_latents(M, batch, kv, layer_idx, most), most, out)
 
     def _head_gemm(self, x, x_head: int, w, y, y_head: int, batch, most: int):
@@ -1247,7 +1254,7 @@ class CudaOps:
         ex.cuda_pack = {"gate_up": stack(up), "down": stack(down)}
         return ex.cuda_pack
 
-    def _grouped_gemm(self, pk, a, M_pad, tile_expert, n_exp, out):
+    def _grouped_gemm(self, pk, a, M_pad, tile_expert, n_exp, out, act: int = 0):
         kind = pk["kind"]
         if kind in (1, 2):
             data, sfa, rs = a.data, a.sf, a.row_scale
@@ -1258,7 +1265,7 @@ class CudaOps:
         w = pk["w"]
         self._check(self.lib.blz_gemm_tc(kind, _ptr(data), lda, _ptr(w), w.shape[1] * w.element_size(), _ptr(out), out.stride(0),
                                          M_pad, pk["N"], pk["K"], _ptr(rs), _ptr(pk["alpha"]), VP(0), _ptr(sfa), _ptr(pk["sf"]),
-                                         0, 128, 0, _ptr(tile_expert), n_exp, 0, 0, 0.0, self._stream()), "grouped gemm")
+                                         0, 128, 0, _ptr(tile_expert), n_exp, 0, act, 0.0, self._stream()), "grouped gemm")
         return out
 
     def moe(self, x, topk_w, topk_id, experts):
@@ -1318,12 +1325,12 @@ class CudaOps:
                     self._check(self.lib.blz_gemm_simple_experts(_ptr(src), src.stride(0), _ptr(w["w"]), _ptr(dst), dst.stride(0), max_tiles, w["N"],
                                                                  w["K"], _ptr(tile_expert), _ptr(tile_rows), int(x.dtype == torch.float32),
                                                                  self._stream()), "gemm_simple_experts")
+                    if dst is g:
+                        self.relu2_(g, row_map)
                 elif narrow:
-                    self._moe_gemm(w, src, max_tiles, tile_expert, tile_rows, n_exp, dst)
+                    self._moe_gemm(w, src, max_tiles, tile_expert, tile_rows, n_exp, dst, act=3 if dst is g else 0)
                 else:
-                    self._grouped_gemm(w, src, M_pad, tile_expert, n_exp, dst)
-                if dst is g:
-                    self.relu2_(g, row_map)
+                    self._grouped_gemm(w, src, M_pad, tile_expert, n_exp, dst, act=3 if dst is g else 0)
             return RoutedRows(y, row_map, topk_w.contiguous(), shared)
         proxy_d = Linear(dn["fmt"], dn["N"], dn["K"])
         proxy_d.act_quant = dn["act_quant"]
@@ -1339,7 +1346,7 @@ class CudaOps:
             self._grouped_gemm(dn, act, M_pad, tile_expert, n_exp, y)
         return RoutedRows(y, row_map, topk_w.contiguous(), shared)
 
-    def _moe_gemm(self, pk, a, row_tiles, tile_expert, tile_rows, n_exp, out):
+    def _moe_gemm(self, pk, a, row_tiles, tile_expert, tile_rows, n_exp, out, act: int = 0):
         """Expert GEMM over the padded row space with the features on the MMA lanes and only each tile's live rows on its columns."""
         kind = pk["kind"]
         if isinstance(a, QuantAct):
@@ -1351,7 +1358,7 @@ class CudaOps:
         w = pk["w"]
         self._check(self.lib.blz_moe_gemm(kind, _ptr(data), lda, _ptr(w), w.shape[1] * w.element_size(), _ptr(out), out.stride(0),
                                           row_tiles, pk["N"], pk["K"], n_exp, _ptr(rs), _ptr(pk["alpha"]), _ptr(sfa), _ptr(pk["sf"]),
-                                          _ptr(tile_expert), _ptr(tile_rows), 0, self._stream()), f"moe_gemm kind {kind}")
+                                          _ptr(tile_expert), _ptr(tile_rows), act, self._stream()), f"moe_gemm kind {kind}")
 
     def _silu_mul_live(self, gu, quant_for, row_list):
         """``silu_mul`` over the padded row space of the routed rows: only the rows named in ``row_list`` (-1 = none) are

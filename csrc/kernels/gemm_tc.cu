@@ -353,7 +353,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                 if (col0 + i + 3 < p.N) dst[i + 3] = o.w;
               }
             }
-          } else if (p.act) {
+          } else if (p.act && p.act != 3) {
             // SwiGLU in the epilogue: columns [0,16) of the group are gate, [16,32) the matching up features
             __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)row * p.ldc + col0 / 2;
             uint32_t pk[8];
@@ -385,10 +385,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
               const float4 a1 = *reinterpret_cast<const float4*>(sal + c * 32 + i + 4);
               const float4 b0 = *reinterpret_cast<const float4*>(sbi + c * 32 + i);
               const float4 b1 = *reinterpret_cast<const float4*>(sbi + c * 32 + i + 4);
-              const float o0 = fmaf(__uint_as_float(r[i]) * rs, a0.x, b0.x), o1 = fmaf(__uint_as_float(r[i + 1]) * rs, a0.y, b0.y);
-              const float o2 = fmaf(__uint_as_float(r[i + 2]) * rs, a0.z, b0.z), o3 = fmaf(__uint_as_float(r[i + 3]) * rs, a0.w, b0.w);
-              const float o4 = fmaf(__uint_as_float(r[i + 4]) * rs, a1.x, b1.x), o5 = fmaf(__uint_as_float(r[i + 5]) * rs, a1.y, b1.y);
-              const float o6 = fmaf(__uint_as_float(r[i + 6]) * rs, a1.z, b1.z), o7 = fmaf(__uint_as_float(r[i + 7]) * rs, a1.w, b1.w);
+              float o0 = fmaf(__uint_as_float(r[i]) * rs, a0.x, b0.x), o1 = fmaf(__uint_as_float(r[i + 1]) * rs, a0.y, b0.y);
+              float o2 = fmaf(__uint_as_float(r[i + 2]) * rs, a0.z, b0.z), o3 = fmaf(__uint_as_float(r[i + 3]) * rs, a0.w, b0.w);
+              float o4 = fmaf(__uint_as_float(r[i + 4]) * rs, a1.x, b1.x), o5 = fmaf(__uint_as_float(r[i + 5]) * rs, a1.y, b1.y);
+              float o6 = fmaf(__uint_as_float(r[i + 6]) * rs, a1.z, b1.z), o7 = fmaf(__uint_as_float(r[i + 7]) * rs, a1.w, b1.w);
+              if (p.act) {
+                o0 = squared_relu(o0); o1 = squared_relu(o1); o2 = squared_relu(o2); o3 = squared_relu(o3);
+                o4 = squared_relu(o4); o5 = squared_relu(o5); o6 = squared_relu(o6); o7 = squared_relu(o7);
+              }
               if (p.push_rows_per > 0) {
                 // staged per warp as plain tile rows (272-byte pitch: the 16-byte stores of eight rows fall on distinct banks)
                 if constexpr (BN == 128)
@@ -622,7 +626,7 @@ BLZ_API int blz_gemm_push_rs(void* const* slots, void* const* flags, void* done_
 // kind: 0 bf16, 1 nvfp4, 2 mxfp8, 3 fp8.  A [M, K] and B [N, K] row-major (packed bytes for 4/8-bit kinds);
 // lda / ldb in BYTES.  out_f32: C is fp32, else bf16; ldc in elements.  bn: 128 or 256 (0 = choose).
 // act = 1: B's rows come in groups of [16 gate | 16 up] features and C is bf16 [M, N/2] = silu(gate) * up (ldc % 8 == 0);
-// act = 2: the clamped form of glu.cuh with act_limit.
+// act = 2: the clamped form of glu.cuh with act_limit; act = 3: the squared ReLU of every column (any N, experts too).
 // b_kt > 0: B is the tile-major repack [ceil(N/128)][b_kt][128][128 bytes] (zero padded), b_kt = ceil(row bytes / 128).
 BLZ_API int blz_gemm_tc(int kind, const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
                         int M, int N, int K, const float* row_scale, const float* alpha, const void* bias,
@@ -658,7 +662,7 @@ BLZ_API int blz_gemm_tc(int kind, const void* A, long long lda, const void* B, l
   p.b_raw = reinterpret_cast<const uint8_t*>(B);
   p.act = act;
   p.act_limit = act_limit;
-  if (act && (out_f32 || N % 32 || (ldc & 7) || tile_expert)) return (int)cudaErrorInvalidValue;
+  if (act && (out_f32 || (act != 3 && (N % 32 || (ldc & 7) || tile_expert)))) return (int)cudaErrorInvalidValue;
   if (b_kt > 0 && tile_expert) return (int)cudaErrorInvalidValue;
   p.mc_out = nullptr; p.done_ctr = nullptr; p.epoch = nullptr; p.spin_limit = 0; p.rank = 0; p.world = 1;
   p.push_rows_per = 0;
@@ -677,7 +681,7 @@ BLZ_API int blz_gemm_tc(int kind, const void* A, long long lda, const void* B, l
   if (p.amax_val && (!out_f32 || tile_expert)) return (int)cudaErrorInvalidValue;
   if (p.amax_val || push.rows_per > 0) bn = 128;
   if (fuse.mc_out) {
-    if (out_f32 || (N % 32)) return (int)cudaErrorInvalidValue;
+    if (out_f32 || act || (N % 32)) return (int)cudaErrorInvalidValue;
     p.mc_out = fuse.mc_out; p.done_ctr = fuse.done_ctr; p.epoch = fuse.epoch; p.spin_limit = fuse.spin_limit;
     p.rank = fuse.rank; p.world = fuse.world;
     for (int r = 0; r < fuse.world; ++r) p.peer_pad[r] = fuse.peer_pad[r];

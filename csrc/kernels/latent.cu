@@ -136,14 +136,14 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepParams p) {
 }
 
 // ------------------------------------------------------------------------------------------ query rotation
-// A block per row.  Rows the filter has: the rotated part goes behind the mapped query in q_eff [T, heads, D] (pads zeroed); the others'
-// is turned in place in q [T, heads, dim + rot].
+// The rotated part of the queries q [T, heads, dim + rot]: turned in place for the rows of long portions (a block per row), or, beside
+// the product that maps a query to the latents, behind the mapped query in q_eff [T, heads, D] (pads zeroed).
 struct LatentRotParams {
   void* q;
-  void* q_eff;                 // or null: no such rows
+  void* q_eff;
   const float* freq;
   const int* positions;
-  RowFilter rows;
+  RowFilter rows;              // which rows are mapped; the others are turned in place
   int heads, dim, rot, rot_dims, rank;
 };
 
@@ -152,33 +152,39 @@ __global__ void __launch_bounds__(128) latent_rot_kernel(LatentRotParams p) {
   extern __shared__ float cs[];                      // [rot_dims / 2][cos, sin]
   pdl_trigger();
   pdl_wait();
-  const int t = blockIdx.x, half = p.rot_dims / 2, n = p.rows.len(t);
-  if (n == 0) return;
+  const int t = blockIdx.x, half = p.rot_dims / 2;
+  if (p.rows.len(t) <= p.rows.max_tokens) return;
   const float pos = (float)p.positions[t];
   for (int i = threadIdx.x; i < half; i += 128) turn_of(p.freq, half, i, pos, cs[2 * i], cs[2 * i + 1]);
   __syncthreads();
   T* q = reinterpret_cast<T*>(p.q) + (size_t)t * p.heads * (p.dim + p.rot);
-  if (n > p.rows.max_tokens) {
-    for (int i = threadIdx.x; i < p.heads * half; i += 128) {
-      T* x = q + (size_t)(i / half) * (p.dim + p.rot) + p.dim + i % half;
-      const float c = cs[2 * (i % half)], s = cs[2 * (i % half) + 1], u = ad_ld(x), v = ad_ld(x + half);
-      ad_st(x, u * c - v * s);
-      ad_st(x + half, v * c + u * s);
-    }
-    return;
+  for (int i = threadIdx.x; i < p.heads * half; i += 128) {
+    T* x = q + (size_t)(i / half) * (p.dim + p.rot) + p.dim + i % half;
+    const float c = cs[2 * (i % half)], s = cs[2 * (i % half) + 1], u = ad_ld(x), v = ad_ld(x + half);
+    ad_st(x, u * c - v * s);
+    ad_st(x + half, v * c + u * s);
   }
-  const int rp = up16(p.rank), D = rp + up16(p.rot), m = D - p.rank;
-  T* e = reinterpret_cast<T*>(p.q_eff) + (size_t)t * p.heads * D;
-  for (int i = threadIdx.x; i < p.heads * m; i += 128) {
-    const int h = i / m, col = p.rank + i % m, j = col - rp;
-    const T* x = q + (size_t)h * (p.dim + p.rot) + p.dim;
-    float v = j >= 0 && j < p.rot ? ad_ld(x + j) : 0.f;
-    if (j >= 0 && j < 2 * half) {
-      const bool low = j < half;
-      const float o = ad_ld(x + (low ? j + half : j - half)), c = cs[2 * (low ? j : j - half)], s = cs[2 * (low ? j : j - half) + 1];
-      v = low ? v * c - o * s : v * c + o * s;
+}
+
+// rows [m0, m0 + 64) of head h, by n threads: columns rank .. D of q_eff
+template <typename T>
+__device__ __forceinline__ void place_rotated(const LatentRotParams& p, int m0, int M, int h, int n) {
+  const int half = p.rot_dims / 2, rp = up16(p.rank), D = rp + up16(p.rot), zeros = D - p.rank - 2 * half, per = half + zeros;
+  for (int i = threadIdx.x; i < 64 * per; i += n) {
+    const int m = m0 + i / per, k = i % per;
+    if (m >= M || !p.rows.has(m)) continue;
+    const T* x = reinterpret_cast<const T*>(p.q) + ((size_t)m * p.heads + h) * (p.dim + p.rot) + p.dim;
+    T* e = reinterpret_cast<T*>(p.q_eff) + ((size_t)m * p.heads + h) * D;
+    if (k < half) {
+      float c, s;
+      turn_of(p.freq, half, k, (float)p.positions[m], c, s);
+      const float u = ad_ld(x + k), v = ad_ld(x + k + half);
+      ad_st(e + rp + k, u * c - v * s);
+      ad_st(e + rp + k + half, v * c + u * s);
+    } else {                                         // the pad of the latent, what is not turned, the pad behind it
+      const int z = k - half, col = z < rp - p.rank ? p.rank + z : z + p.rank + 2 * half, j = col - rp;
+      ad_st(e + col, j >= 0 && j < p.rot ? ad_ld(x + j) : 0.f);
     }
-    ad_st(e + (size_t)h * D + col, v);
   }
 }
 
@@ -190,6 +196,7 @@ struct HeadGemmParams {
   long long lda, sa, ldc, sc;  // elements: row and head strides
   int M, N, K;
   RowFilter rows;
+  LatentRotParams rot;         // q_eff not null: one block more along N places the rotated parts
 };
 static constexpr int kHgStages = 4, kHgPitch = 72;             // tiles of 64 columns under way; row pitch: 8 rows cover all banks
 
@@ -204,6 +211,7 @@ __global__ void __launch_bounds__(256) head_gemm_f32_kernel(HeadGemmParams p) {
   if (threadIdx.x < 64 && m0 + threadIdx.x < p.M && p.rows.has(m0 + threadIdx.x)) any = 1;
   __syncthreads();
   if (!any) return;
+  if (n0 >= p.N) return place_rotated<float>(p.rot, m0, p.M, h, 256);
   const float* A = reinterpret_cast<const float*>(p.a) + h * p.sa;
   const float* B = reinterpret_cast<const float*>(p.b) + (size_t)h * p.N * p.K;
   float acc[4][4] = {};
@@ -255,6 +263,7 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(HeadGemmParams p, int ve
   if (tid < 64 && m0 + tid < p.M && p.rows.has(m0 + tid)) any = 1;
   __syncthreads();
   if (!any) return;
+  if (n0 >= p.N) return place_rotated<__nv_bfloat16>(p.rot, m0, p.M, h, 128);
   const __nv_bfloat16* A = reinterpret_cast<const __nv_bfloat16*>(p.a) + h * p.sa;
   const __nv_bfloat16* B = reinterpret_cast<const __nv_bfloat16*>(p.b) + (size_t)h * p.N * p.K;
   const int wm = (warp & 1) * 32, wn = (warp >> 1) * 32, tiles = (p.K + 63) / 64;
@@ -786,33 +795,50 @@ BLZ_API int blz_latent_prep(const void* proj, long long ld, long long q_off, lon
   return (int)launch_pdl(latent_prep_kernel<__nv_bfloat16, 1>, grid, dim3(128), 0, s, p);
 }
 
-// Rotation of the queries q [T, heads, dim + rot]: rows of sequences with at most max_tokens new tokens into q_eff [T, heads, D], from
-// column rank on, D = up16(rank) + up16(rot); the others in place.
-BLZ_API int blz_latent_rot(void* q, void* q_eff, const float* freq, const int* positions, const int* seq_of_row, const int* q_start, int T,
-                           int heads, int dim, int rot, int rot_dims, int rank, int max_tokens, int f32, cudaStream_t s) {
+// Rotation in place of the queries q [T, heads, dim + rot] of sequences with more than max_tokens new tokens.
+BLZ_API int blz_latent_rot(void* q, const float* freq, const int* positions, const int* seq_of_row, const int* q_start, int T, int heads, int dim,
+                           int rot, int rot_dims, int max_tokens, int f32, cudaStream_t s) {
   using namespace blz;
-  if (T <= 0 || heads < 1 || dim < 1 || rot < 1 || rot_dims < 0 || rot_dims > rot || rot_dims % 2 || rot_dims > 4096 || (rot_dims && !freq))
+  if (T <= 0 || heads < 1 || dim < 1 || rot < 1 || rot_dims < 2 || rot_dims > rot || rot_dims % 2 || rot_dims > 4096 || !freq)
     return (int)cudaErrorInvalidValue;
-  const LatentRotParams p = {q, q_eff, freq, positions, {seq_of_row, q_start, max_tokens}, heads, dim, rot, rot_dims, rank};
+  const LatentRotParams p = {q, nullptr, freq, positions, {seq_of_row, q_start, max_tokens}, heads, dim, rot, rot_dims, 0};
   const size_t sm = rot_dims * sizeof(float);
   if (f32) return (int)launch_pdl(latent_rot_kernel<float>, dim3(T), dim3(128), sm, s, p);
   return (int)launch_pdl(latent_rot_kernel<__nv_bfloat16>, dim3(T), dim3(128), sm, s, p);
 }
 
-// C[m, h, :N] = A[m, h, :K] B[h]^T, B [heads][N][K], for the rows of sequences with at most max_tokens new tokens; strides in elements.
-BLZ_API int blz_head_gemm(const void* a, long long lda, long long sa, const void* b, void* c, long long ldc, long long sc, int M, int N, int K,
-                          int heads, const int* seq_of_row, const int* q_start, int max_tokens, int f32, cudaStream_t s) {
+static int run_head_gemm(blz::HeadGemmParams p, int heads, int f32, cudaStream_t s) {
   using namespace blz;
-  if (M <= 0 || N < 1 || K < 1 || heads < 1 || heads > 65535 || (M + 63) / 64 > 65535) return (int)cudaErrorInvalidValue;
-  const HeadGemmParams p = {a, b, c, lda, sa, ldc, sc, M, N, K, {seq_of_row, q_start, max_tokens}};
-  const dim3 grid((N + 63) / 64, (M + 63) / 64, heads);
+  if (p.M <= 0 || p.N < 1 || p.K < 1 || heads < 1 || heads > 65535 || (p.M + 63) / 64 > 65535) return (int)cudaErrorInvalidValue;
+  const dim3 grid((p.N + 63) / 64 + (p.rot.q_eff ? 1 : 0), (p.M + 63) / 64, heads);
   if (f32) return (int)launch_pdl(head_gemm_f32_kernel, grid, dim3(256), 0, s, p);
-  const int vec = aligned16(a) && aligned16(b) && (reinterpret_cast<uintptr_t>(c) & 3) == 0 && (lda | sa | (long long)K) % 8 == 0 && (ldc | sc | (long long)N) % 2 == 0;
+  const int vec = aligned16(p.a) && aligned16(p.b) && (reinterpret_cast<uintptr_t>(p.c) & 3) == 0 && (p.lda | p.sa | (long long)p.K) % 8 == 0 &&
+                  (p.ldc | p.sc | (long long)p.N) % 2 == 0;
   constexpr int sm = kHgStages * 128 * kHgPitch * 2;
   static PerDeviceOnce once;
   const cudaError_t e = once.smem_limit(head_gemm_kernel, sm);
   if (e != cudaSuccess) return (int)e;
   return (int)launch_pdl(head_gemm_kernel, grid, dim3(128), sm, s, p, vec);
+}
+
+// C[m, h, :N] = A[m, h, :K] B[h]^T, B [heads][N][K], for the rows of sequences with at most max_tokens new tokens; strides in elements.
+BLZ_API int blz_head_gemm(const void* a, long long lda, long long sa, const void* b, void* c, long long ldc, long long sc, int M, int N, int K,
+                          int heads, const int* seq_of_row, const int* q_start, int max_tokens, int f32, cudaStream_t s) {
+  const blz::HeadGemmParams p = {a, b, c, lda, sa, ldc, sc, M, N, K, {seq_of_row, q_start, max_tokens}, {}};
+  return run_head_gemm(p, heads, f32, s);
+}
+
+// Queries q [T, heads, dim + rot] of the same rows mapped to the latents: q_eff [T, heads, D] = [map_h q_nope (rank) | rotated part], both
+// padded to 16 columns with zeros; map [heads][rank][dim].
+BLZ_API int blz_latent_map(void* q, const void* map, void* q_eff, const float* freq, const int* positions, int T, int heads, int dim, int rot,
+                           int rot_dims, int rank, const int* seq_of_row, const int* q_start, int max_tokens, int f32, cudaStream_t s) {
+  using namespace blz;
+  if (rot < 1 || rot_dims < 0 || rot_dims > rot || rot_dims % 2 || (rot_dims && !freq) || !q_eff) return (int)cudaErrorInvalidValue;
+  const long long D = up16(rank) + up16(rot);
+  const RowFilter rows = {seq_of_row, q_start, max_tokens};
+  const HeadGemmParams p = {q, map, q_eff, (long long)heads * (dim + rot), dim + rot, heads * D, D, T, rank, dim, rows,
+                            {q, q_eff, freq, positions, rows, heads, dim, rot, rot_dims, rank}};
+  return run_head_gemm(p, heads, f32, s);
 }
 
 // Query rows per CTA of blz_latent_rows for sequences of up to `rows` (new tokens x heads) rows; 0: not these sizes.  *per_sm (may be

@@ -247,7 +247,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__
     // finished sums of this thread's feature for the row columns [c0, c0 + n): scales, bias, activation, store.
     // Called by all lanes of a warp with the same c0 and n.
     auto finish = [&](const float* v, int c0, int n) {
-      if (p.act) {
+      if (p.act && p.act != 3) {
         // lanes 0-15 hold the gate, lanes 16-31 the up value of 16 features: one exchange joins them
         const int fo = (ft * 128 + q * 32) / 2 + (lane & 15);
 #pragma unroll
@@ -262,7 +262,10 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__
         const int f = ft * 128 + fl;
 #pragma unroll
         for (int j = 0; j < 32; ++j)
-          if (j < n && c0 + j < rows) p.C[((size_t)mt * 128 + c0 + j) * p.ldc + f] = __float2bfloat16(fmaf(v[j] * al, s_rs[c0 + j], bs));
+          if (j < n && c0 + j < rows) {
+            const float x = fmaf(v[j] * al, s_rs[c0 + j], bs);
+            p.C[((size_t)mt * 128 + c0 + j) * p.ldc + f] = __float2bfloat16(p.act ? squared_relu(x) : x);
+          }
       }
     };
     if (ks == 1) {
@@ -392,7 +395,7 @@ static cudaError_t launch_moe_gemm(const CUtensorMap& tmW, const CUtensorMap& tm
 
 // kind: 0 bf16, 1 nvfp4, 2 mxfp8.  X: routed rows [row_tiles * 128, K] in the padded row space (packed bytes for 4/8-bit
 // kinds, ldx in bytes); W: stacked expert weights [experts * N, K] (ldw in bytes); C bf16 [row_tiles * 128, ldc].
-// N % 128 == 0.  act = 1: SwiGLU on [16 gate | 16 up] interleaved weight rows, C is [rows, N / 2].
+// N % 128 == 0.  act = 1: SwiGLU on [16 gate | 16 up] interleaved weight rows, C is [rows, N / 2]; act = 3: the squared ReLU.
 BLZ_API int blz_moe_gemm(int kind, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc,
                          int row_tiles, int N, int K, int experts, const float* row_scale, const float* alpha, const void* sfx,
                          const void* sfw, const int* tile_expert, const int* tile_rows, int act, cudaStream_t stream) {
