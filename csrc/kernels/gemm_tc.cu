@@ -353,7 +353,24 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                 if (col0 + i + 3 < p.N) dst[i + 3] = o.w;
               }
             }
-          } else if (p.act && p.act != 3) {
+          } else if (p.act == 3) {
+            __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)row * p.ldc + col0;
+#pragma unroll
+            for (int i = 0; i < 32; i += 8) {
+              uint32_t pk[4];
+#pragma unroll
+              for (int j = 0; j < 8; j += 2)
+                pk[j / 2] = pack_bf16x2(squared_relu(fmaf(__uint_as_float(r[i + j]) * rs, sal[c * 32 + i + j], sbi[c * 32 + i + j])),
+                                        squared_relu(fmaf(__uint_as_float(r[i + j + 1]) * rs, sal[c * 32 + i + j + 1], sbi[c * 32 + i + j + 1])));
+              if (whole) {
+                *reinterpret_cast<uint4*>(dst + i) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+              } else {
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                  if (col0 + i + j < p.N) dst[i + j] = reinterpret_cast<const __nv_bfloat16*>(pk)[j];
+              }
+            }
+          } else if (p.act) {
             // SwiGLU in the epilogue: columns [0,16) of the group are gate, [16,32) the matching up features
             __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)row * p.ldc + col0 / 2;
             uint32_t pk[8];
@@ -385,14 +402,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
               const float4 a1 = *reinterpret_cast<const float4*>(sal + c * 32 + i + 4);
               const float4 b0 = *reinterpret_cast<const float4*>(sbi + c * 32 + i);
               const float4 b1 = *reinterpret_cast<const float4*>(sbi + c * 32 + i + 4);
-              float o0 = fmaf(__uint_as_float(r[i]) * rs, a0.x, b0.x), o1 = fmaf(__uint_as_float(r[i + 1]) * rs, a0.y, b0.y);
-              float o2 = fmaf(__uint_as_float(r[i + 2]) * rs, a0.z, b0.z), o3 = fmaf(__uint_as_float(r[i + 3]) * rs, a0.w, b0.w);
-              float o4 = fmaf(__uint_as_float(r[i + 4]) * rs, a1.x, b1.x), o5 = fmaf(__uint_as_float(r[i + 5]) * rs, a1.y, b1.y);
-              float o6 = fmaf(__uint_as_float(r[i + 6]) * rs, a1.z, b1.z), o7 = fmaf(__uint_as_float(r[i + 7]) * rs, a1.w, b1.w);
-              if (p.act) {
-                o0 = squared_relu(o0); o1 = squared_relu(o1); o2 = squared_relu(o2); o3 = squared_relu(o3);
-                o4 = squared_relu(o4); o5 = squared_relu(o5); o6 = squared_relu(o6); o7 = squared_relu(o7);
-              }
+              const float o0 = fmaf(__uint_as_float(r[i]) * rs, a0.x, b0.x), o1 = fmaf(__uint_as_float(r[i + 1]) * rs, a0.y, b0.y);
+              const float o2 = fmaf(__uint_as_float(r[i + 2]) * rs, a0.z, b0.z), o3 = fmaf(__uint_as_float(r[i + 3]) * rs, a0.w, b0.w);
+              const float o4 = fmaf(__uint_as_float(r[i + 4]) * rs, a1.x, b1.x), o5 = fmaf(__uint_as_float(r[i + 5]) * rs, a1.y, b1.y);
+              const float o6 = fmaf(__uint_as_float(r[i + 6]) * rs, a1.z, b1.z), o7 = fmaf(__uint_as_float(r[i + 7]) * rs, a1.w, b1.w);
               if (p.push_rows_per > 0) {
                 // staged per warp as plain tile rows (272-byte pitch: the 16-byte stores of eight rows fall on distinct banks)
                 if constexpr (BN == 128)

@@ -254,15 +254,10 @@ __device__ __forceinline__ void lt_mma(float (&c)[4], const uint32_t (&a)[4], ui
 __global__ void __launch_bounds__(128) head_gemm_kernel(HeadGemmParams p, int vec) {
   constexpr int LD = kHgPitch;
   extern __shared__ __align__(16) __nv_bfloat16 ring[];          // [stages][A 64 x LD | B 64 x LD]
-  __shared__ int any;
+  __shared__ uint8_t live[64];                       // rows the filter has
   pdl_trigger();
   pdl_wait();
   const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64, h = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  if (tid == 0) any = 0;
-  __syncthreads();
-  if (tid < 64 && m0 + tid < p.M && p.rows.has(m0 + tid)) any = 1;
-  __syncthreads();
-  if (!any) return;
   if (n0 >= p.N) return place_rotated<__nv_bfloat16>(p.rot, m0, p.M, h, 128);
   const __nv_bfloat16* A = reinterpret_cast<const __nv_bfloat16*>(p.a) + h * p.sa;
   const __nv_bfloat16* B = reinterpret_cast<const __nv_bfloat16*>(p.b) + (size_t)h * p.N * p.K;
@@ -285,6 +280,12 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(HeadGemmParams p, int ve
   };
   float acc[2][4][4] = {};
   for (int t = 0; t < kHgStages - 1; ++t) send(t);
+  const bool mine = tid < 64 && m0 + tid < p.M && p.rows.has(m0 + tid);
+  if (tid < 64) live[tid] = mine;
+  if (!__syncthreads_or(mine)) {                     // none of them
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    return;
+  }
   for (int t = 0; t < tiles; ++t) {
     asm volatile("cp.async.wait_group %0;" ::"n"(kHgStages - 2) : "memory");
     __syncthreads();                                 // tile t is there, and everyone is done with the slot that is filled next
@@ -312,7 +313,7 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(HeadGemmParams p, int ve
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int m = m0 + wm + i * 16 + (lane >> 2) + half * 8;
-      if (m >= p.M || !p.rows.has(m)) continue;
+      if (!live[m - m0]) continue;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int n = n0 + wn + j * 8 + (lane & 3) * 2;
@@ -814,9 +815,9 @@ static int run_head_gemm(blz::HeadGemmParams p, int heads, int f32, cudaStream_t
   if (f32) return (int)launch_pdl(head_gemm_f32_kernel, grid, dim3(256), 0, s, p);
   const int vec = aligned16(p.a) && aligned16(p.b) && (reinterpret_cast<uintptr_t>(p.c) & 3) == 0 && (p.lda | p.sa | (long long)p.K) % 8 == 0 &&
                   (p.ldc | p.sc | (long long)p.N) % 2 == 0;
-  constexpr int sm = kHgStages * 128 * kHgPitch * 2;
+  const int tiles = (p.K + 63) / 64, sm = (tiles < kHgStages ? tiles : kHgStages) * 128 * kHgPitch * 2;
   static PerDeviceOnce once;
-  const cudaError_t e = once.smem_limit(head_gemm_kernel, sm);
+  const cudaError_t e = once.smem_limit(head_gemm_kernel, kHgStages * 128 * kHgPitch * 2);
   if (e != cudaSuccess) return (int)e;
   return (int)launch_pdl(head_gemm_kernel, grid, dim3(128), sm, s, p, vec);
 }
