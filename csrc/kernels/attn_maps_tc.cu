@@ -100,13 +100,6 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
   const int ntok = b < 0 ? 0 : min(qlen - q0, tpb);
   const int pg_lo = first_key(pos0 + q0, p.window) >> 4, pg_hi = (pos0 + q0 + ntok - 1) >> 4;
   const int n = b < 0 ? 0 : (pg_hi - pg_lo + 8) / 8;               // tiles of 8 pages
-  // the tiles a half's rows see (two maps: the same rows, all of them)
-  auto first_tile = [&](int m) {
-    return MAPS == 2 ? 0 : m * tph >= ntok ? 0 : ((first_key(pos0 + q0 + m * tph, p.window) >> 4) - pg_lo) >> 3;
-  };
-  auto last_tile = [&](int m) {
-    return MAPS == 2 ? n - 1 : m * tph >= ntok ? -1 : (((pos0 + q0 + min(ntok, (m + 1) * tph) - 1) >> 4) - pg_lo) >> 3;
-  };
   if (warp >= 8) {
     maps_reg_dec<72>();
     if (warp == 8) {
@@ -148,41 +141,37 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
       // -------------------------------------------------------------- MMA issuer
       if (lane == 0) {
         const uint32_t id_s = make_idesc(1, 1, 128, 128), id_o = make_idesc(1, 1, 128, (uint32_t)vp, 0, 1);
-        const int f[2] = {first_tile(0), first_tile(1)}, e[2] = {last_tile(0), last_tile(1)};
         auto qk = [&](int m, int i) {
-          if (i < f[m] || i > e[m]) return;
           const uint32_t qa = smem_u32(sQ + m * q_bytes), ka = smem_u32(sK + ((i % c.ks) * MAPS + (MAPS == 2 ? m : 0)) * k_bytes);
           for (int s = 0; s < dp / 16; ++s)
             mma_f16(tmem + m * 128, make_smem_desc(qa + s * 256, 128, dp * 16, kSwzNone),
                     make_smem_desc(ka + s * 256, 128, dp * 16, kSwzNone), id_s, s > 0);
           mma_commit(&s_full[m]);
+          if (m == 1) mma_commit(&k_empty[i % c.ks]);
         };
         bool ok = mbar_wait(q_full, 0, abort_flag, p.status) && mbar_wait(&k_full[0], 0, abort_flag, p.status);
         if (ok) {
           tc_fence_after();
           qk(0, 0);
           qk(1, 0);
-          mma_commit(&k_empty[0]);
         }
         for (int i = 0; i < n && ok; ++i) {
           ok = mbar_wait(&v_full[i % c.vs], (uint32_t)((i / c.vs) & 1), abort_flag, p.status);
           for (int m = 0; m < 2 && ok; ++m) {
-            if (i >= f[m] && i <= e[m]) {
-              if (!mbar_wait(&p_full[m], (uint32_t)((i - f[m]) & 1), abort_flag, p.status)) { ok = false; break; }
-              tc_fence_after();
-              const uint32_t va = smem_u32(sV + (i % c.vs) * v_bytes);
-              for (int half = 0; half < 2; ++half)
-                for (int s = 0; s < 8; ++s)          // a page of 16 keys per MMA
-                  mma_f16_ts(tmem + 256 + m * 128, tmem + m * 128 + half * 64 + s * 8,
-                             make_smem_desc(va + s * 32 * vp, vp * 16, 128, kSwzNone), id_o, i > f[m] || half > 0 || s > 0);
-              if (i == e[m]) mma_commit(&o_full[m]);
-            }
+            if (!mbar_wait(&p_full[m], (uint32_t)(i & 1), abort_flag, p.status)) { ok = false; break; }
+            tc_fence_after();
+            const uint32_t va = smem_u32(sV + (i % c.vs) * v_bytes);
+            for (int half = 0; half < 2; ++half)
+              for (int s = 0; s < 8; ++s)            // a page of 16 keys per MMA
+                mma_f16_ts(tmem + 256 + m * 128, tmem + m * 128 + half * 64 + s * 8,
+                           make_smem_desc(va + s * 32 * vp, vp * 16, 128, kSwzNone), id_o, i > 0 || half > 0 || s > 0);
             if (m == 1) mma_commit(&v_empty[i % c.vs]);
             if (i + 1 < n) {
               if (m == 0 && !mbar_wait(&k_full[(i + 1) % c.ks], (uint32_t)(((i + 1) / c.ks) & 1), abort_flag, p.status)) { ok = false; break; }
               tc_fence_after();
               qk(m, i + 1);
-              if (m == 1) mma_commit(&k_empty[(i + 1) % c.ks]);
+            } else {
+              mma_commit(&o_full[m]);
             }
           }
         }
@@ -227,9 +216,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
       const uint32_t s_addr = tmem + m * 128 + lanes, o_addr = tmem + 256 + m * 128 + lanes;
       float mx = -INFINITY, l = 0.f;
       bool ok = true;
-      const int i0 = first_tile(m), i1 = last_tile(m);
-      for (int i = i0; i <= i1; ++i) {
-        ok = __all_sync(0xffffffffu, mbar_wait(&s_full[m], (uint32_t)((i - i0) & 1), abort_flag, p.status));
+      for (int i = 0; i < n; ++i) {
+        ok = __all_sync(0xffffffffu, mbar_wait(&s_full[m], (uint32_t)(i & 1), abort_flag, p.status));
         if (!ok) break;
         tc_fence_after();
         uint32_t v[4][32];
@@ -256,7 +244,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
           const float f = grow ? (mx == -INFINITY ? 0.f : ex2(mx - mn)) : 1.f;
           mx = mn;
           l *= f;
-          if (i > i0) {
+          if (i > 0) {
             for (int k = 0; k < vp; k += 16) {
               uint32_t w[16];
               tmem_ld16(o_addr + k, w);
@@ -291,7 +279,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
         if (lane == 0) mbar_arrive(&p_full[m]);
       }
       if constexpr (MAPS == 1) {
-        ok = ok && i1 >= i0 && __all_sync(0xffffffffu, mbar_wait(&o_full[m], 0, abort_flag, p.status));
+        if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&o_full[m], 0, abort_flag, p.status));
         tc_fence_after();
         const float f = 1.f / (l + (p.sink ? ex2(p.sink[head] * kLog2e - mx) : 0.f));
         __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(r0 + tq) * p.ld_out + (size_t)head * p.vdim;
