@@ -465,20 +465,25 @@ __global__ void __launch_bounds__(lr_threads(R), R <= 32 ? 2 : 1) latent_rows_ke
     // -------------------------------------------------------------- MMA issuer
     if (lane == 0) {
       const uint32_t id_s = make_idesc(1, 1, 128, R), id_o = make_idesc(1, 1, 128, 2 * R, 1, 1);
-      const uint32_t qa = smem_u32(sQ), pa = smem_u32(sP), ra = smem_u32(ring);
+      // descriptors once, then steps of their address field (16 bytes): an MMA with few columns takes less time than its descriptors
+      const uint64_t q_desc = make_smem_desc(smem_u32(sQ), 128, D * 16, kSwzNone), p_desc = make_smem_desc(smem_u32(sP), 32 * R, 128, kSwzNone);
+      const uint32_t ra = smem_u32(ring);
       auto qk = [&](int i) {
-        const uint32_t ka = ra + (i % ST) * tile;
-        for (int s = 0; s < D / 16; ++s)
-          mma_f16(tmem + (i & 1) * R, make_smem_desc(ka + s * 256, 128, D * 16, kSwzNone), make_smem_desc(qa + s * 256, 128, D * 16, kSwzNone),
-                  id_s, s > 0);
+        const uint64_t k_desc = make_smem_desc(ra + (i % ST) * tile, 128, D * 16, kSwzNone);
+        const uint32_t d = tmem + (i & 1) * R;
+#pragma unroll 6
+        for (int s = 0; s < D / 16; ++s) mma_f16(d, k_desc + s * 16, q_desc + s * 16, id_s, s > 0);
         mma_commit(&s_full[i & 1]);
       };
       auto pv = [&](int i) {
-        const uint32_t va = ra + (i % ST) * tile;
-        for (int v = 0; v < nvb; ++v)
+        uint64_t v_desc = make_smem_desc(ra + (i % ST) * tile, D * 16, 128, kSwzNone);
+        const uint32_t acc = i > 0;
+        for (int v = 0; v < nvb; ++v, v_desc += 128) {
+          const uint32_t d = tmem + (2 + 2 * v) * R;
+#pragma unroll
           for (int s = 0; s < 8; ++s)        // a page of 16 keys per MMA
-            mma_f16(tmem + (2 + 2 * v) * R, make_smem_desc(va + s * 32 * D + v * 2048, D * 16, 128, kSwzNone),
-                    make_smem_desc(pa + s * 64 * R, 32 * R, 128, kSwzNone), id_o, i > 0 || s > 0);
+            mma_f16(d, v_desc + s * 2 * D, p_desc + s * 4 * R, id_o, s > 0 ? 1u : acc);
+        }
         mma_commit(pv_done);
         mma_commit(&k_empty[i % ST]);
       };
