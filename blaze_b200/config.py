@@ -130,7 +130,8 @@ class LatentAttnSpec:
 
 @dataclass
 class GatedLinearSpec:
-    """Linear attention whose forget gate, one per head and query channel, also decides what is written (HGRN2); normed per head."""
+    """Linear attention with a forget gate per head and query channel, whose complement weighs the incoming value (HGRN2); normed per
+    head."""
     heads: int
     dim: int
     vdim: int
@@ -678,7 +679,7 @@ def named_config(name: str) -> ModelConfig:
         def latent(**kw):
             return LatentAttnSpec(**{**dict(heads=4, dim=24, rot_dim=16, vdim=40, q_rank=48, kv_rank=64, scale=0.16,
                                             rot=RotarySpec(16, 1.0e4, False), sink=True, window=40), **kw})
-        layers = [LayerSpec(None, PolyNormSpec(320), None, GatedLinearSpec(4, 32, 48)), LayerSpec(latent(), MoeSpec(8, 2, 64, 96)),
+        layers = [LayerSpec(None, PolyNormSpec(288), None, GatedLinearSpec(4, 32, 48)), LayerSpec(latent(), MoeSpec(8, 2, 64, 96)),
                   LayerSpec(latent(heads=6, window=24, kv_from=1)), LayerSpec(None, MoeSpec(8, 2, 64), None, GatedLinearSpec(2, 48, 32))]
         return ModelConfig.of_layers(layers, architecture="Rapisun", model_type="rapisun", vocab_size=1024, hidden_size=192, input_conv=4)
     elif n in ("qwen3-8b",):

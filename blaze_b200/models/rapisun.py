@@ -1,8 +1,8 @@
 """Rapisun: a decoder that adds the layer-normed output of every sublayer to its residual, described layer by layer in its
 configuration (``ModelConfig.layer_specs``).
 
-Mixers are a linear attention whose forget gate also decides what is written (HGRN2) and a windowed latent attention with a sink,
-whose latents a later layer may read; a causal convolution over time is added to what a mixer reads.  Feed-forwards have no gate: a
+Mixers are a linear attention with forget gates whose complements weigh the incoming values (HGRN2) and a windowed latent attention
+with a sink, whose latents a later layer may read; a causal convolution over time is added to what a mixer reads.  Feed-forwards have no gate: a
 dense one activated by a sum of normed powers, or routed experts with squared ReLUs and a shared one.  The residual, the norms, the
 inputs of the convolutions and the recurrent states are fp32.  Tensor names: ``embed[.norm]``, ``l<i>.{norm1,norm2,canon1}``,
 ``l<i>.mix.{q,f,f.b,lower,v,norm,o}`` or ``l<i>.mix.{dq,dq.norm,uq,dkv,dkv.norm,uk,uv,sink,o}``, ``l<i>.mlp.{up,down,act}`` or

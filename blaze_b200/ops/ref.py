@@ -400,7 +400,7 @@ def state_space(x, B, C, dt, A, dt_bias, D, state):
 
 
 def gated_linear(q, f, v, lower, bias, state):
-    """Linear attention whose forget gates also decide what is written, one sequence: q and the gates' inputs f ``[T, H, dk]`` before
+    """Gated linear attention (state rows keep a share f and take 1 - f of the value), one sequence: q and the gates' inputs f ``[T, H, dk]`` before
     their activations, v ``[T, H, dv]``, lower bounds and biases ``[H * dk]``, state ``[H, dk, dv]``.  fp32."""
     T, H, dk = q.shape
     lo = lower.view(1, H, dk)

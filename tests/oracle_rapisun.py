@@ -74,8 +74,8 @@ def rotate_half(x, dims, base):
 
 
 def sink_window_attention(q, k, v, scale, window, sink):
-    """One head, ``q, k [T, d]``, ``v [T, e]``: a row sees itself and the window - 1 tokens before it (window 0: all of them); the
-    denominator has one more term ``exp(sink)``."""
+    """One head, ``q, k [T, d]``, ``v [T, e]``: keys lie at most window - 1 positions back (window 0: anywhere before);
+    the denominator has one more term ``exp(sink)``."""
     T = q.shape[0]
     out = torch.zeros(T, v.shape[1], dtype=q.dtype)
     for i in range(T):

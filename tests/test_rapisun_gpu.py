@@ -72,7 +72,7 @@ def test_activations_without_a_gate(ops, T, I, dtype):
 
 
 @pytest.mark.parametrize("dtype", TYPES)
-@pytest.mark.parametrize("T,W,E,top,ff,shared", [(1, 64, 4, 1, 48, 32), (9, 144, 6, 2, 40, 56), (70, 100, 5, 5, 24, 0), (300, 256, 12, 4, 96, 128),
+@pytest.mark.parametrize("T,W,E,top,ff,shared", [(1, 64, 4, 1, 48, 32), (9, 144, 6, 2, 40, 56), (70, 100, 5, 5, 24, 0), (300, 256, 10, 3, 104, 136),
                                                  (37, 512, 33, 6, 256, 0), (600, 128, 3, 1, 64, 64), (2, 81, 7, 2, 33, 0)])
 def test_routed_experts(ops, T, W, E, top, ff, shared, dtype):
     from blaze_b200.config import GatedLinearSpec, LayerSpec, ModelConfig, MoeSpec
@@ -142,7 +142,7 @@ def test_gated_linear_with_many_sequences(ops):
 
 # ----------------------------------------------------------------------------------- latent attention alone
 # heads, dim, rotated, vdim, latent, window
-ATTN = [(4, 24, 8, 40, 48, 20), (8, 64, 16, 64, 128, 72), (1, 16, 16, 16, 16, 5), (5, 12, 6, 20, 36, 0), (16, 32, 32, 64, 256, 50), (40, 64, 32, 64, 256, 100),
+ATTN = [(4, 24, 8, 40, 48, 20), (8, 72, 16, 56, 144, 70), (1, 16, 16, 16, 16, 5), (5, 12, 6, 20, 36, 0), (16, 32, 32, 64, 256, 50), (40, 64, 32, 64, 256, 100),
         (20, 16, 64, 128, 512, 33), (3, 128, 64, 128, 96, 130), (2, 40, 24, 24, 130, 17), (6, 160, 48, 144, 200, 64), (64, 8, 8, 16, 32, 128), (2, 20, 10, 18, 600, 40)]
 PORTIONS = {"whole": [10 ** 6], "pairs and more": [2, 37, 3, 130, 1, 16, 17], "decode": [190] + [1] * 30, "small": [5, 16, 2, 11, 1]}
 
@@ -273,7 +273,7 @@ def test_a_layer_reads_anothers_latents(ops, dtype):
 
 @pytest.mark.parametrize("window", [0, 1000])
 def test_long_context_is_split_over_blocks(ops, window):
-    L, n = LatentLayer(ops, (8, 32, 16, 64, 128, window), torch.bfloat16), 1500
+    L, n = LatentLayer(ops, (8, 32, 24, 48, 160, window), torch.bfloat16), 1500
     plant = [(n - 1, 700), (n - 2, n - 1000), (n - 3, 502), (n - 4, n - 4)] + ([] if window else [(n - 5, 0), (n - 6, 5)])
     rows = L.rows(n, 3, plant)
     L.step([(0, rows[:n - 6])])
