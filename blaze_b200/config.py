@@ -11,7 +11,7 @@ from __future__ import annotations
 import json
 import math
 import os
-from dataclasses import dataclass, field, asdict
+from dataclasses import asdict, dataclass, field, replace
 from typing import Any, Dict, List, Optional, Union
 
 
@@ -106,6 +106,43 @@ class SoftAttnSpec:
 
 
 @dataclass
+class SigmoidAttnSpec:
+    """Attention of one layer whose weights are sigmoids of the scores, not shares of a sum, with the options of its designs; scores have
+    a learned term per head and distance bucket (a table of the checkpoint) and one per head."""
+    heads: int
+    kv_heads: int
+    dim: int                    # queries and keys
+    vdim: int                   # values
+    scale: float                # of the scores, before the learned terms
+    far: float                  # distance from which all keys share the table's last row
+    bias: bool = False          # q, k, v and output projections have biases
+    conv: int = 0               # taps of a causal convolution of the projected q, k and v over time (0: none)
+    unit_v: bool = False        # value heads divided by their root mean square
+    temp_coef: float = 0.0      # queries at position p times 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)
+    temp_every: float = 1.0
+    window = 0                  # as in DiffAttnSpec
+    out_scale = 1.0
+    maps = 1
+
+    @property
+    def group(self) -> int:
+        return self.heads // self.kv_heads
+
+    @property
+    def conv_dim(self) -> int:
+        return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
+
+    def bucket(self, n: int, rows: int) -> int:
+        """Row of a table of ``rows`` rows for a key ``n`` tokens back: the first half of the rows for one distance each, the others
+        for ranges that grow logarithmically up to ``far``."""
+        near = rows // 2
+        if n < near:
+            return n
+        # distances where the logarithms' ratio is a whole number fall into the upper bucket, whatever the rounding
+        return min(rows - 1, near + math.floor(math.log(n / near) / math.log(self.far / near) * (rows - near) + 1e-9))
+
+
+@dataclass
 class LatentAttnSpec:
     """Softmax attention whose keys and values are linear maps of one cached vector per token (a normed latent of ``kv_rank``
     numbers), beside a rotated key part that all heads share; queries come through a latent of their own."""
@@ -145,13 +182,16 @@ class GatedLinearSpec:
 
 @dataclass
 class DeltaSpec:
-    """Gated delta rule with one decay per head and key channel, and a gated norm per head."""
+    """Gated delta rule with one decay per head and key channel (or one per head), and a gated norm per head."""
     heads: int
     kv_heads: int               # heads of q and k
     dim: int
     vdim: int
     conv: int                   # taps of the convolution before it
     out_scale: float = 1.0
+    head_decay: bool = False    # one decay per head, its input and the gate's projected from the layer's input as they are; else one per
+                                # key channel, both inputs through low-rank maps
+    gate: str = "sigmoid"       # of the normed output: "sigmoid" | "silu"
 
     @property
     def conv_dim(self) -> int:
@@ -160,6 +200,19 @@ class DeltaSpec:
     @property
     def state(self) -> int:
         return self.dim
+
+
+@dataclass
+class MinGruSpec:
+    """Gated recurrence, element by element, whose gates read the current token only (minGRU), with a gated output."""
+    width: int
+    conv = 0                    # no convolution of its own
+    heads = state = 1
+    out_scale = 1.0
+
+    @property
+    def vdim(self) -> int:
+        return self.width
 
 
 @dataclass
@@ -197,25 +250,34 @@ class PolyNormSpec:
 
 @dataclass
 class MoeSpec:
-    """Routed experts ``down(relu(up h)^2)`` weighted by their softmax scores, renormalised over the chosen ones, and a shared one."""
+    """Routed experts weighted by their scores, and a shared one.  An expert is ``down(relu(up h)^2)`` or
+    ``down(silu(gate h) * up h)``."""
     experts: int
     top: int
     ff: int                     # per expert
     shared_ff: int = 0          # 0: no shared expert
+    act: str = "relu2"          # or "swiglu"
+    scores: str = "softmax"     # or "sigmoid"
+    renorm: bool = True         # weights divided by their sum over the chosen experts
+    weigh_input: bool = False   # the weight multiplies an expert's input, not its output
+    shared_gate: bool = False   # the shared expert's output times sigmoid of a projection to one number
 
 
 @dataclass
 class LayerSpec:
     """One entry of a configuration that describes its layers one by one: an attention, a recurrence, or both side by side."""
-    attn: Union[DiffAttnSpec, SoftAttnSpec, LatentAttnSpec, None] = None
+    attn: Union[DiffAttnSpec, SoftAttnSpec, SigmoidAttnSpec, LatentAttnSpec, None] = None
     mlp: Union[GluSpec, PolyNormSpec, MoeSpec, None] = None        # None: the layer has no feed-forward
     weights_of: Optional[int] = None       # the layer whose tensors this one uses (with a cache and a state of its own)
-    rec: Union[DeltaSpec, StateSpaceSpec, GatedLinearSpec, None] = None
+    rec: Union[DeltaSpec, StateSpaceSpec, GatedLinearSpec, MinGruSpec, None] = None
+    number: Optional[int] = None           # of the layer in the checkpoint, where that is not its place in the list (looped layers)
+    joins: bool = False         # a pass of a loop starts here: the residual is first mapped from itself beside the embedding
 
     @property
     def kind(self) -> str:
-        names = {DiffAttnSpec: "diff_attention", SoftAttnSpec: "soft_attention", LatentAttnSpec: "latent_attention", DeltaSpec: "delta_rule",
-                 StateSpaceSpec: "state_space", GatedLinearSpec: "gated_linear"}
+        names = {DiffAttnSpec: "diff_attention", SoftAttnSpec: "soft_attention", SigmoidAttnSpec: "sigmoid_attention",
+                 LatentAttnSpec: "latent_attention", DeltaSpec: "delta_rule", StateSpaceSpec: "state_space", GatedLinearSpec: "gated_linear",
+                 MinGruSpec: "min_gru"}
         return "+".join(names[type(m)] for m in (self.attn, self.rec) if m is not None)
 
 
@@ -269,7 +331,7 @@ class ModelConfig:
     indexer_head_dim: int = 0
     indexer_budget: int = 0
     indexer_compress_ratio: int = 0
-    # models whose configuration lists its layers one by one, each with sizes of its own (Sevevik, Niletar, Rapisun); the sizes above
+    # models whose configuration lists its layers one by one, each with sizes of its own (Sevevik, Niletar, Rapisun, Medodra); the sizes above
     # then hold those of the first layer
     layer_specs: List[LayerSpec] = field(default_factory=list)
     streams: int = 1                        # residual streams joined by learned static mixes
@@ -358,6 +420,8 @@ class ModelConfig:
             return cls._from_niletar(raw)
         if raw.get("architecture") == "Rapisun":
             return cls._from_rapisun(raw)
+        if raw.get("architecture") == "Medodra":
+            return cls._from_medodra(raw)
         archs = raw.get("architectures") or ["Qwen3ForCausalLM"]
         t = raw.get("text_config", raw)
         g = lambda k, d=None: t.get(k, raw.get(k, d))  # noqa: E731
@@ -520,6 +584,30 @@ class ModelConfig:
                              rms_norm_eps=float(raw["norm"]["eps"]), input_conv=taps, torch_dtype=str(raw.get("torch_dtype", "bfloat16")))
 
     @classmethod
+    def _from_medodra(cls, raw: Dict[str, Any]) -> "ModelConfig":
+        """The layer-by-layer configuration of the Medodra design."""
+        specs: List[LayerSpec] = []
+        for i, e in enumerate(raw["layers"]):
+            m, attn = e["mixer"], None
+            if e["type"] == "delta":
+                rec = DeltaSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), conv=int(m["conv"]),
+                                head_decay=True, gate="silu")
+            elif e["type"] == "parallel":
+                l, t = m["left"], m["left"]["q_temp"]
+                attn = SigmoidAttnSpec(heads=int(l["heads"]), kv_heads=int(l["kv_heads"]), dim=int(l["dim"]), vdim=int(l["vdim"]),
+                                       scale=float(l["scale"]), far=float(l["bias_max"]), bias=True, conv=int(l["conv"]), unit_v=True,
+                                       temp_coef=float(t["coef"]), temp_every=float(t["every"]))
+                rec = MinGruSpec(int(m["right"]["width"]))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+            specs.append(LayerSpec(attn, _gated_moe(i, e), None, rec))
+        specs = _unrolled(specs, raw.get("loop"))
+        _check_layers(specs)
+        return cls.of_layers(specs, architecture="Medodra", model_type="medodra", vocab_size=int(raw["vocab"]), hidden_size=int(raw["width"]),
+                             rms_norm_eps=float(raw["norm"]["eps"]), zero_centered_norm=True, residual_mult=float(raw["residual_mult"]),
+                             embed_scale=float(raw["embedding"]["scale"]), torch_dtype=str(raw.get("torch_dtype", "bfloat16")))
+
+    @classmethod
     def of_layers(cls, specs: List[LayerSpec], **kw) -> "ModelConfig":
         """A configuration from its layer list; the model-wide sizes that other parts read are those of the first layer."""
         a = next((s.attn for s in specs if s.attn is not None), None)
@@ -556,6 +644,32 @@ def _norm_or_moe(i: int, entry: Dict[str, Any]) -> Union[PolyNormSpec, MoeSpec, 
                    shared_ff=int(shared["ff"]) if shared else 0)
 
 
+def _gated_moe(i: int, entry: Dict[str, Any]) -> Optional[MoeSpec]:
+    m = entry.get("mlp")
+    if m is None:
+        return None
+    if m.get("kind") != "moe":
+        raise ValueError(f"layer {i}: unknown feed-forward {m.get('kind')!r}")
+    shared = m.get("shared")
+    return MoeSpec(experts=int(m["router"]["experts"]), top=int(m["router"]["top"]), ff=int(m["expert"]["ff"]),
+                   shared_ff=int(shared["ff"]) if shared else 0, act="swiglu", scores="sigmoid", renorm=False, weigh_input=True,
+                   shared_gate=bool(shared))
+
+
+def _unrolled(specs: List[LayerSpec], loop: Optional[Dict[str, Any]]) -> List[LayerSpec]:
+    """The layers in the order they run: those of ``loop`` (start, stop, times) stand there once per pass, later passes with the tensors
+    of the first."""
+    if not loop:
+        return specs
+    start, stop, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not 0 <= start < stop <= len(specs) or times < 1:
+        raise ValueError(f"a loop over layers {start} .. {stop - 1} of {len(specs)}, {times} times")
+    out = specs[:start]
+    for k in range(times):
+        out += [replace(s, number=i, joins=i == start, weights_of=i if k else None) for i, s in enumerate(specs[start:stop], start)]
+    return out + [replace(s, number=i) for i, s in enumerate(specs[stop:], stop)]
+
+
 def _rotary(rot: Optional[Dict[str, Any]]) -> Optional[RotarySpec]:
     if not rot:
         return None
@@ -576,6 +690,8 @@ def _check_layers(specs: List[LayerSpec]) -> None:
                 raise ValueError(f"layer {i}: {a.heads} query heads over {a.kv_heads} key/value heads of {a.dim} / {a.vdim}")
             if a.window < 0:
                 raise ValueError(f"layer {i}: a window of {a.window}")
+            if isinstance(a, SigmoidAttnSpec) and (a.conv < 0 or a.temp_every <= 0 or a.far <= 0):
+                raise ValueError(f"layer {i}: a convolution of {a.conv} taps, distances up to {a.far}, query temperature steps of {a.temp_every}")
             rot, turned = getattr(a, "rot", None), a.rot_dim if isinstance(a, LatentAttnSpec) else a.dim
             if rot is not None and (rot.dims % 2 or not 0 <= rot.dims <= turned):
                 raise ValueError(f"layer {i}: rotary positions on {rot.dims} of {turned} dimensions")
@@ -590,7 +706,7 @@ def _check_layers(specs: List[LayerSpec]) -> None:
                         raise ValueError(f"layer {i} reads latents of layer {a.kv_from} that have another size or rotation")
         if r is not None:
             groups = r.groups if isinstance(r, StateSpaceSpec) else r.kv_heads if isinstance(r, DeltaSpec) else r.heads
-            taps = r.conv if not isinstance(r, GatedLinearSpec) else 1
+            taps = r.conv if not isinstance(r, (GatedLinearSpec, MinGruSpec)) else 1
             if min(r.heads, groups, r.state, r.vdim, taps) < 1 or r.heads % groups:
                 raise ValueError(f"layer {i}: {r.heads} recurrent heads over {groups} groups, state {r.state} x {r.vdim}, {r.conv} taps")
             if isinstance(r, StateSpaceSpec) and (r.norm_groups < 1 or r.inner % r.norm_groups):
@@ -682,6 +798,14 @@ def named_config(name: str) -> ModelConfig:
         layers = [LayerSpec(None, PolyNormSpec(288), None, GatedLinearSpec(4, 32, 48)), LayerSpec(latent(), MoeSpec(8, 2, 64, 96)),
                   LayerSpec(latent(heads=6, window=24, kv_from=1)), LayerSpec(None, MoeSpec(8, 2, 64), None, GatedLinearSpec(2, 48, 32))]
         return ModelConfig.of_layers(layers, architecture="Rapisun", model_type="rapisun", vocab_size=1024, hidden_size=192, input_conv=4)
+    elif n in ("tiny-medodra",):
+        # the Medodra layer kinds in miniature, one without a feed-forward, with a loop over two of three layers
+        a = SigmoidAttnSpec(4, 2, 32, 48, 0.2, 100.0, True, 4, True, 0.2, 64.0)
+        d = DeltaSpec(4, 2, 32, 40, 3, head_decay=True, gate="silu")
+        moe = MoeSpec(8, 2, 64, 96, "swiglu", "sigmoid", False, True, True)
+        layers = [LayerSpec(a, moe, None, MinGruSpec(160)), LayerSpec(None, moe, None, d), LayerSpec(a, None, None, MinGruSpec(192))]
+        return ModelConfig.of_layers(_unrolled(layers, {"start": 0, "stop": 2, "times": 2}), architecture="Medodra", model_type="medodra",
+                                     vocab_size=1024, hidden_size=192, zero_centered_norm=True, residual_mult=0.8, embed_scale=0.5)
     elif n in ("qwen3-8b",):
         c = ModelConfig(vocab_size=151936, hidden_size=4096, num_layers=36, num_heads=32, num_kv_heads=8,
                         head_dim=128, intermediate_size=12288, rope=RopeConfig(theta=1e6))

@@ -20,8 +20,8 @@ Pages hold 16 tokens.  Two pool layouts exist:
   kv_rank]`` (the latents) and ``v [pages, 1, 16, rot_dim]``.  A layer that reads another's latents has no pages of its own.
 
 Recurrent layers (Gated DeltaNet, and the recurrences of a layer-by-layer configuration) keep one state row per sequence row: the
-last inputs of their convolution in the activation type and the recurrent state in fp32, of each layer's own sizes.  A
-configuration whose mixers' inputs are convolved (``input_conv``) keeps the last inputs of every layer there too, in fp32.
+last inputs of their convolution in the activation type and the recurrent state in fp32, of each layer's own sizes.  An attention
+whose projected queries, keys and values are convolved keeps their last rows there, in the activation type.  A configuration whose mixers' inputs are convolved (``input_conv``) keeps the last inputs of every layer there too, in fp32.
 
 The reference keeps one-token pages and several KV dtypes (``crates/blaze/src/model.rs:499-583``,
 ``alloc_kv`` :517); its page bookkeeping is in ``engine.rs:1083-1164``.
@@ -155,11 +155,16 @@ class KVCache:
             if r.conv:
                 self.conv_state[i] = torch.zeros(self.state_rows, r.conv_dim, r.conv - 1, dtype=tdt, device=device)
             self.rec_state[i] = torch.zeros(self.state_rows, r.heads, r.state, r.vdim, dtype=torch.float32, device=device)
+        self.qkv_state: Dict[int, torch.Tensor] = {}        # [rows, taps - 1, conv_dim]: last projected queries, keys and values
+        for i in (range(lo, hi) if cfg.layer_specs else ()):
+            a = cfg.layer_specs[i].attn
+            if getattr(a, "conv", 0) > 1:
+                self.qkv_state[i] = torch.zeros(self.state_rows, a.conv - 1, a.conv_dim, dtype=tdt, device=device)
         self.input_state: Dict[int, torch.Tensor] = {}      # last inputs of the mixers, where those are convolved
         if cfg.input_conv > 1:
             for i in range(lo, hi):
                 self.input_state[i] = torch.zeros(self.state_rows, cfg.input_conv - 1, cfg.hidden_size, dtype=torch.float32, device=device)
-        self.state_layers = sorted({*self.gdn_layers, *rec, *self.input_state})       # every layer with a state row
+        self.state_layers = sorted({*self.gdn_layers, *rec, *self.qkv_state, *self.input_state})       # every layer with a state row
 
         # sparse-attention indexer: the raw index key of every token, paged like K and V (shared prefixes share them)
         self.idx_k: Dict[int, torch.Tensor] = {}
@@ -214,21 +219,21 @@ class KVCache:
 
     def nbytes(self) -> int:
         n = 0
-        for d in (self.k, self.v, self.kv, self.conv_state, self.rec_state, self.input_state, self.idx_k):
+        for d in (self.k, self.v, self.kv, self.conv_state, self.rec_state, self.qkv_state, self.input_state, self.idx_k):
             n += sum(t.numel() * t.element_size() for t in {id(t): t for t in d.values()}.values())      # layers may share pages
         return n + (self.ple.nbytes() if self.ple is not None else 0)
 
     # ------------------------------------------------------------------ recurrent state rows
     def copy_state(self, src: int, dst: int) -> None:
         """Copy the conv + recurrent state of row ``src`` to row ``dst`` (``model.rs:2718``)."""
-        for d in (self.conv_state, self.rec_state, self.input_state):
+        for d in (self.conv_state, self.rec_state, self.qkv_state, self.input_state):
             for t in d.values():
                 t[dst].copy_(t[src])
         if self.ple is not None:
             self.ple.copy(src, dst)
 
     def zero_state(self, row: int) -> None:
-        for d in (self.conv_state, self.rec_state, self.input_state):
+        for d in (self.conv_state, self.rec_state, self.qkv_state, self.input_state):
             for t in d.values():
                 t[row].zero_()
         if self.ple is not None:

@@ -13,5 +13,8 @@ def model_class(cfg):
     if cfg.architecture == "Rapisun":
         from .rapisun import Rapisun
         return Rapisun
+    if cfg.architecture == "Medodra":
+        from .medodra import Medodra
+        return Medodra
     from .qwen3 import Model
     return Model

@@ -74,6 +74,29 @@ class SoftAttn:
             self.freq = _two_floats(spec.rot.frequencies(), device)
 
 
+class SigmoidAttn:
+    """Sigmoid attention of a :class:`Mixer` (config.SigmoidAttnSpec).  ``bias [heads, PAD + n + PAD]`` fp32 holds what is added to the
+    score of a key, by its distance (at PAD + distance): the learned terms per distance and head, those of the last distance ``n - 1``
+    again for every one beyond, and -inf for keys that come later.  ``conv_w [taps, conv_dim]`` fp32."""
+
+    PAD = 128                            # a kernel may read the entries of a whole tile of keys around a row's own position
+
+    def __init__(self, spec, device, rel, shift, conv_w=None):
+        self.spec = spec                 # config.SigmoidAttnSpec
+        rows, near = rel.shape[0], rel.shape[0] // 2
+        if near < 1 or spec.far <= near:
+            raise ValueError(f"distances up to {spec.far} in a table of {rows} rows")
+        buckets, n = [], 0
+        while not buckets or buckets[-1] < rows - 1:
+            buckets.append(spec.bucket(n, rows))
+            n += 1
+        idx = torch.tensor(buckets + [rows - 1] * self.PAD)
+        table = rel.float().cpu()[idx].t() + shift.float().cpu()[:, None]
+        self.reach = n                   # distances listed one by one
+        self.bias = torch.cat([torch.full((spec.heads, self.PAD), -math.inf), table], 1).contiguous().to(device)
+        self.conv_w = None if conv_w is None else conv_w.t().to(device, torch.float32).contiguous()
+
+
 class LatentAttn:
     """Attention of a :class:`Mixer` over cached latents (config.LatentAttnSpec).  The input projection gives the queries' latent
     (normed by ``q_norm``, then ``uq``) and, unless the layer reads another's, the keys' latent (``c_norm``) and rotated part.
@@ -106,8 +129,8 @@ def _two_floats(f, device) -> torch.Tensor:
 
 
 class Recurrence:
-    """Recurrent part of a :class:`Mixer`, ``kind`` "delta" (config.DeltaSpec), "ssm" (config.StateSpaceSpec) or "gated"
-    (config.GatedLinearSpec).  ``A`` is the positive decay rate, or (gated) the lower bound of the forget gates, whose bias is
+    """Recurrent part of a :class:`Mixer`, ``kind`` "delta" (config.DeltaSpec), "ssm" (config.StateSpaceSpec), "gated"
+    (config.GatedLinearSpec) or "mingru" (config.MinGruSpec).  ``A`` is the positive decay rate, or (gated) the lower bound of the forget gates, whose bias is
     ``dt_bias``; decay, step and norm weights are fp32.  ``low`` (delta): from the low-rank inputs to [decay inputs | norm gates]."""
 
     def __init__(self, spec, kind: str, norm_groups: int):
@@ -120,19 +143,30 @@ class Recurrence:
 
 class Mixer:
     """The mixers of a layer on one input: a stacked input projection (``cols``: first column of each part), an attention and / or a
-    recurrence whose results lie side by side (scaled), and one output projection over both."""
+    recurrence whose results lie side by side (scaled), and one output projection over both; or (``o_rec``) one each, whose results are
+    RMS-normed with the weights ``out_norms`` and averaged."""
 
     def __init__(self):
         self.in_proj: Linear = None
         self.o: Linear = None
         self.cols: Dict[str, int] = {}
         self.low_width = 0               # columns of the low-rank inputs
-        self.attn: Optional[SoftAttn] = None             # or a LatentAttn
+        self.attn: Optional[SoftAttn] = None             # or a SigmoidAttn or LatentAttn
         self.rec: Optional[Recurrence] = None
+        self.o_rec: Optional[Linear] = None
+        self.out_norms: Optional[tuple] = None           # fp32 [hidden], attention's and recurrence's
 
     def linears(self) -> List[Linear]:
         latent = [self.attn.uq, self.attn.expand] if isinstance(self.attn, LatentAttn) else []
-        return [l for l in (self.in_proj, self.o, self.rec.low if self.rec is not None else None, *latent) if l is not None]
+        return [l for l in (self.in_proj, self.o, self.o_rec, self.rec.low if self.rec is not None else None, *latent) if l is not None]
+
+
+class Branches:
+    """What a layer adds to its residual: ``mult`` times the sum of its mixer's rows (``rows``: one tensor, or two that are RMS-normed with
+    ``norms`` and averaged) and of its feed-forward (``ffn``: rows, or what ``ops.moe_rows`` gives; None: there is none)."""
+
+    def __init__(self, rows, norms, ffn, mult: float):
+        self.rows, self.norms, self.ffn, self.mult = rows, norms, ffn, mult
 
 
 class DenseMlp:
@@ -164,6 +198,7 @@ class Experts:
     """Routed experts of one layer (this rank's share under expert parallelism)."""
 
     act = "swiglu"                       # or "relu2": no gate, ``gate_up`` holds the up projections alone
+    weigh_input = False                  # an expert's weight multiplies its input instead of its output
 
     def __init__(self):
         self.gate_up: List[Linear] = []
@@ -187,6 +222,8 @@ class MoeMlp:
         self.shared: Optional[DenseMlp] = None           # or a PlainMlp
         self.rows_out = False            # the result stays as routed rows: the residual op that follows sums them up
         self.shared_gate: Optional[Linear] = None
+        self.gate_row: Optional[int] = None              # the shared expert's gate as a row of ``router``
+        self.sigmoid = False             # scores are sigmoids of the router's logits, not a softmax
         self.top_k = 0
         self.renorm = True
 
@@ -810,13 +847,20 @@ class Model:
         y = torch.empty(proj.shape[0], M.o.K, dtype=proj.dtype, device=proj.device)
         if isinstance(M.attn, LatentAttn):
             ops.latent_attention(proj, M, batch, kv, gi, eps, y[:, :n_attn])
+        elif isinstance(M.attn, SigmoidAttn):
+            if batch.gdn_defer is not None and M.attn.spec.conv > 1:
+                self.gdn_records[gi] = (proj, None)
+            ops.sigmoid_attention(proj, M, batch, kv, gi, eps, y[:, :n_attn])
         elif M.attn is not None:
             ops.soft_attention(proj, M, batch, kv, gi, eps, y[:, :n_attn])
         if M.rec is not None:
             low = ops.linear(M.rec.low, proj[:, M.cols["low"]:M.cols["low"] + M.low_width]) if M.rec.low is not None else None
             if batch.gdn_defer is not None:
                 self.gdn_records[gi] = (proj, low)      # what the recurrence consumed (see _gdn)
-            ops.recurrence(proj, low, M, batch, kv, gi, eps, y[:, n_attn:])
+            z = y[:, n_attn:] if M.o_rec is None else torch.empty(proj.shape[0], M.o_rec.K, dtype=proj.dtype, device=proj.device)
+            ops.recurrence(proj, low, M, batch, kv, gi, eps, z)
+            if M.o_rec is not None:
+                return ops.linear(M.o, y), ops.linear(M.o_rec, z)
         return ops.linear(M.o, y)
 
     def _gdn(self, G: Gdn, h, batch, kv, gi, fused=None):
@@ -843,15 +887,18 @@ class Model:
             gi = self.first_layer + li
             if gi in self.conv_records:
                 self.ops.input_conv(self.conv_records[gi][idx].contiguous(), L.in_conv, batch, kv, gi, self.dtype, state_only=True)
-            if L.gdn is None and (L.mixer is None or L.mixer.rec is None):
+            attn_conv = gi in kv.qkv_state
+            if L.gdn is None and (L.mixer is None or L.mixer.rec is None) and not attn_conv:
                 continue
             rec = self.gdn_records.get(gi)
             if rec is None:
                 raise RuntimeError("no deferred step to replay")
             if L.mixer is not None:
-                proj, low = rec
-                self.ops.recurrence(proj[idx].contiguous(), None if low is None else low[idx].contiguous(), L.mixer, batch, kv, gi,
-                                    self.cfg.rms_norm_eps, None, state_only=True)
+                proj, low = rec[0][idx].contiguous(), None if rec[1] is None else rec[1][idx].contiguous()
+                if attn_conv:
+                    self.ops.sigmoid_attention(proj, L.mixer, batch, kv, gi, self.cfg.rms_norm_eps, None, state_only=True)
+                if L.mixer.rec is not None:
+                    self.ops.recurrence(proj, low, L.mixer, batch, kv, gi, self.cfg.rms_norm_eps, None, state_only=True)
                 continue
             mixed, b, a = rec
             ba = torch.stack([b[idx], a[idx]]).contiguous()      # one buffer: the kernels take a common row stride
@@ -887,10 +934,11 @@ class Model:
             return self._row_cut(M.down, a, a.rows if hasattr(a, "rows") else a.shape[0], fused)
         hd = h.dense if hasattr(h, "dense") and h.dense is not None else h
         logits = ops.linear(M.router, hd, out_dtype=torch.float32)
+        n_exp = None if M.gate_row is None else M.experts.num_experts
         if ops.is_cuda:
-            w, ids = ops.router_topk(logits, M.top_k, M.renorm, M.experts.first, M.experts.count)
+            w, ids = ops.router_topk(logits, M.top_k, M.renorm, M.experts.first, M.experts.count, sigmoid=M.sigmoid, n_exp=n_exp)
         else:
-            w, ids = ops.router_topk(logits, M.top_k, M.renorm)
+            w, ids = ops.router_topk(logits, M.top_k, M.renorm, sigmoid=M.sigmoid, n_exp=n_exp)
         if self.heat is not None:
             if self.tp.expert_order is not None:
                 if self._order_dev is None:
@@ -901,7 +949,8 @@ class Model:
         # Tokens are replicated across the ranks, so expert parallelism needs no dispatch: every rank runs the routed
         # pairs whose expert it holds and the partial outputs are summed by the reduce + norm that follows.
         if M.rows_out:
-            return ops.moe_rows(hd, w, ids, M.experts, self._mlp(M.shared, hd)[0] if M.shared is not None else None), "full"
+            return ops.moe_rows(hd, w, ids, M.experts, self._mlp(M.shared, hd)[0] if M.shared is not None else None,
+                                logits[:, M.gate_row] if M.gate_row is not None else None), "full"
         y = ops.moe(hd, w, ids, M.experts)
         routed_partial = tp
         if M.shared is not None:

@@ -222,6 +222,48 @@ def diff_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
     return out
 
 
+def position_vectors(positions: torch.Tensor, freq: torch.Tensor, width: int) -> torch.Tensor:
+    """Sines (even columns) and cosines (odd ones) of position * frequency of the column pair, fp32 ``[T, width]``."""
+    ang = positions.double().view(-1, 1) * freq.double()
+    return torch.stack([torch.sin(ang), torch.cos(ang)], -1).flatten(1)[:, :width].float()
+
+
+def query_temperature(positions: torch.Tensor, coef: float, every: float) -> torch.Tensor:
+    return 1 + coef * torch.log(torch.floor((positions.float() + 1) / every) + 1)
+
+
+def causal_conv(u: torch.Tensor, before: torch.Tensor, w: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Causal convolution of each channel over one sequence's rows, ``u [T, C]``, ``w [taps, C]``, ``before [taps - 1, C]`` the rows ahead
+    of them; (fp32 rows, the last taps - 1 inputs)."""
+    hist = torch.cat([before.to(u.dtype), u])
+    return sum(hist[j:j + u.shape[0]].float() * w[j] for j in range(w.shape[0])), hist[u.shape[0]:]
+
+
+def sigmoid_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor, slots, q_start, ctx_len,
+                      scale: float, bias: torch.Tensor, pad: int, window: int = 0) -> torch.Tensor:
+    """Causal attention of q ``[T, H, d]`` over paged keys and values, whose weights are sigmoids of the scores: ``bias [H, pad + n + ..]``
+    holds what is added to the score of a key by its distance (from ``pad`` on; the n-th for every one beyond).  fp32 ``[T, H, e]``."""
+    T, H, d = q.shape
+    G, e, n_dist = k_pool.shape[1], v_pool.shape[3], bias.shape[1] - 2 * pad
+    out = torch.zeros(T, H, e, dtype=torch.float32, device=q.device)
+    for b, slot in enumerate(slots):
+        r0, r1 = q_start[b], q_start[b + 1]
+        ql, n = r1 - r0, ctx_len[b]
+        if ql <= 0:
+            continue
+        pages = block_table[slot, :(n + PAGE - 1) // PAGE].long()
+        K = k_pool[pages].float().permute(1, 0, 2, 3).reshape(G, -1, d)[:, :n]
+        V = v_pool[pages].float().permute(1, 0, 2, 3).reshape(G, -1, e)[:, :n]
+        s = torch.einsum("qghd,gnd->ghqn", q[r0:r1].float().view(ql, G, H // G, d), K) * scale
+        dist = torch.arange(n - ql, n, device=q.device).view(ql, 1) - torch.arange(n, device=q.device).view(1, n)
+        add = bias[:, pad + dist.clamp(0, n_dist - 1)].masked_fill(dist < 0, float("-inf"))
+        if window:
+            add = add.masked_fill(dist >= window, float("-inf"))
+        o = torch.einsum("ghqn,gne->qghe", torch.sigmoid(s + add.view(G, H // G, ql, n)), V)
+        out[r0:r1] = o.reshape(ql, H, e)
+    return out
+
+
 def streams_write(x: torch.Tensor, mix: torch.Tensor, out: torch.Tensor, y: torch.Tensor) -> torch.Tensor:
     """Residual streams ``[T, S, W]`` after a sublayer: ``mix[from, to]`` of the old ones plus ``out[to] * y``."""
     return torch.einsum("ab,taw->tbw", mix, x) + out.view(1, -1, 1) * y.float()[:, None]
@@ -252,9 +294,9 @@ def silu_mul(gu: torch.Tensor) -> torch.Tensor:
     return (F.silu(gu[..., :I].float()) * gu[..., I:].float()).to(gu.dtype)
 
 
-def router_topk(logits: torch.Tensor, k: int, renorm: bool = True):
-    """Softmax over all experts (fp32), top-k by probability, lowest id wins ties."""
-    p = torch.softmax(logits.float(), dim=-1)
+def router_topk(logits: torch.Tensor, k: int, renorm: bool = True, sigmoid: bool = False):
+    """Softmax over all experts (or their sigmoids; fp32), top-k by score, lowest id wins ties."""
+    p = torch.sigmoid(logits.float()) if sigmoid else torch.softmax(logits.float(), dim=-1)
     E = p.shape[-1]
     # stable lowest-id tie break: sort by (-p, id)
     order = torch.argsort(-p, dim=-1, stable=True)[..., :k]
@@ -264,8 +306,9 @@ def router_topk(logits: torch.Tensor, k: int, renorm: bool = True):
     return w, order.to(torch.int32)
 
 
-def moe_forward(x: torch.Tensor, topk_w: torch.Tensor, topk_id: torch.Tensor, expert_fn, num_experts: int):
-    """Reference mixture: ``out[t] = sum_j w[t,j] * expert_fn(e_j, x[t])`` evaluated per expert."""
+def moe_forward(x: torch.Tensor, topk_w: torch.Tensor, topk_id: torch.Tensor, expert_fn, num_experts: int, weigh_input: bool = False):
+    """Reference mixture: ``out[t] = sum_j w[t,j] * expert_fn(e_j, x[t])`` evaluated per expert (``weigh_input``:
+    ``sum_j expert_fn(e_j, w[t,j] * x[t])``)."""
     out = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
     first = getattr(getattr(expert_fn, "__self__", None), "first", 0)
     count = getattr(getattr(expert_fn, "__self__", None), "count", num_experts)
@@ -273,8 +316,12 @@ def moe_forward(x: torch.Tensor, topk_w: torch.Tensor, topk_id: torch.Tensor, ex
         tok, slot = (topk_id == e).nonzero(as_tuple=True)
         if tok.numel() == 0:
             continue
+        w = topk_w[tok, slot].float().unsqueeze(-1)
+        if weigh_input:
+            out.index_add_(0, tok, expert_fn(e, (x[tok].float() * w).to(x.dtype)).float())
+            continue
         y = expert_fn(e, x[tok]).float()
-        out.index_add_(0, tok, y * topk_w[tok, slot].float().unsqueeze(-1))
+        out.index_add_(0, tok, y * w)
     return out.to(x.dtype)
 
 
@@ -369,12 +416,12 @@ def gdn_chunked(q, k, v, g, beta, state, chunk: int = 64):
 # ----------------------------------------------------------------------------------- recurrences with an fp32 state
 def delta_rule(q, k, v, a, b, A, dt_bias, state):
     """Gated delta rule with a decay per head and key channel, one sequence: q, k ``[T, G, dk]``, v ``[T, H, dv]``, decay inputs a
-    ``[T, H, dk]``, write strengths b ``[T, H]`` (before their sigmoid), A ``[H]`` > 0, state ``[H, dk, dv]``.  fp32."""
+    ``[T, H, dk]`` (``[T, H, 1]``: one per head), write strengths b ``[T, H]`` (before their sigmoid), A ``[H]`` > 0, state ``[H, dk, dv]``.  fp32."""
     T, G, dk = q.shape
     H = v.shape[1]
     unit = lambda x: x.float() * torch.rsqrt(x.float().pow(2).sum(-1, keepdim=True) + 1e-6)      # noqa: E731
     q, k = [unit(x).repeat_interleave(H // G, 1) for x in (q, k)]
-    g = torch.exp(-A.view(1, H, 1) * F.softplus(a.float() + dt_bias.view(1, H, dk)))
+    g = torch.exp(-A.view(1, H, 1) * F.softplus(a.float() + dt_bias.view(1, H, -1)))
     beta, v, S = torch.sigmoid(b.float()), v.float(), state.clone()
     out = torch.empty(T, H, v.shape[2], device=q.device)
     for t in range(T):
@@ -411,6 +458,17 @@ def gated_linear(q, f, v, lower, bias, state):
     for t in range(T):
         S = S * keep[t].unsqueeze(-1) + write[t].unsqueeze(-1) * v[t].unsqueeze(1)
         out[t] = torch.einsum("hkv,hk->hv", S, q[t])
+    return out, S
+
+
+def min_gru(z, u, state):
+    """minGRU over one sequence: gate inputs z and candidates u ``[T, n]`` before their activations, state ``[n]``.  fp32."""
+    z, u, S = torch.sigmoid(z.float()), u.float(), state.clone()
+    cand = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+    out = torch.empty_like(z)
+    for t in range(z.shape[0]):
+        S = (1 - z[t]) * S + z[t] * cand[t]
+        out[t] = S
     return out, S
 
 

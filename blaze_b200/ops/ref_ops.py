@@ -143,7 +143,7 @@ class RefOps:
         untouched; ``state_only`` advances the states and writes nothing."""
         R, r = M.rec, M.rec.spec
         conv_state, rec_state, defer = kv.conv_state.get(layer_idx), kv.rec_state[layer_idx], getattr(batch, "h_gdn_defer", None)
-        gated = R.kind == "gated"
+        gated, plain = R.kind == "gated", R.kind in ("gated", "mingru")
         dt, H, dv = proj.dtype, r.heads, r.vdim
         for b, slot in enumerate(batch.h_slots):
             r0, r1 = batch.h_q_start[b], batch.h_q_start[b + 1]
@@ -151,15 +151,27 @@ class RefOps:
             if n <= 0:
                 continue
             if batch.h_ctx_len[b] == n:
-                if not gated:
+                if not plain:
                     conv_state[slot].zero_()
                 rec_state[slot].zero_()
-            if not gated:
+            if not plain:
                 y, cs = ref.gdn_conv(proj[r0:r1, M.cols["conv"]:][:, :r.conv_dim], conv_state[slot], R.conv_w, R.conv_b, round_sum=False)
             z = None
             if gated:
                 cols = {c: proj[r0:r1, M.cols[c]:][:, :H * d].reshape(n, H, d) for c, d in (("q", r.dim), ("f", r.dim), ("v", dv))}
                 o, S = ref.gated_linear(cols["q"], cols["f"], cols["v"], R.A, R.dt_bias, rec_state[slot])
+            elif R.kind == "mingru":
+                zg, u, g = [proj[r0:r1, M.cols[c]:][:, :r.width] for c in ("zg", "u", "g")]
+                o, S = ref.min_gru(zg, u, rec_state[slot].view(-1))
+                S = S.view(1, 1, -1)
+                if not state_only:
+                    out[r0:r1] = (o * torch.nn.functional.silu(g.float())).to(dt)
+            elif R.kind == "delta" and r.head_decay:
+                nk = r.kv_heads * r.dim
+                a, b_ = [proj[r0:r1, M.cols[c]:][:, :H] for c in ("decay", "beta")]
+                o, S = ref.delta_rule(y[:, :nk].view(n, -1, r.dim), y[:, nk:2 * nk].view(n, -1, r.dim), y[:, 2 * nk:].view(n, H, dv),
+                                      a.reshape(n, H, 1), b_, R.A, R.dt_bias, rec_state[slot])
+                z = proj[r0:r1, M.cols["z"]:][:, :H * dv]
             elif R.kind == "delta":
                 nk, hd = r.kv_heads * r.dim, H * r.dim
                 o, S = ref.delta_rule(y[:, :nk].view(n, -1, r.dim), y[:, nk:2 * nk].view(n, -1, r.dim), y[:, 2 * nk:].view(n, H, dv),
@@ -172,11 +184,12 @@ class RefOps:
                                        rec_state[slot])
                 z = proj[r0:r1, M.cols["z"]:][:, :r.inner]
             if not (defer is not None and defer[b]):
-                if not gated:
+                if not plain:
                     conv_state[slot].copy_(cs)
                 rec_state[slot].copy_(S)
-            if not state_only:
-                out[r0:r1] = ref.group_norm(o.reshape(n, -1), z, R.norm_w, R.norm_groups, eps, R.kind == "delta", R.kind != "delta",
+            if not state_only and R.kind != "mingru":
+                delta = R.kind == "delta"
+                out[r0:r1] = ref.group_norm(o.reshape(n, -1), z, R.norm_w, R.norm_groups, eps, delta and r.gate == "sigmoid", not delta,
                                             r.out_scale).to(dt)
 
     # -------------------------------------------------------------- residual with normed branches, input convolution, latent attention
@@ -230,17 +243,75 @@ class RefOps:
                                 window=a.window, sink=A.sink)
         out.copy_(torch.einsum("thr,her->the", o.float(), A.uv.float()).reshape(T, -1))
 
-    def moe_rows(self, x, topk_w, topk_id, experts, shared=None):
+    def moe_rows(self, x, topk_w, topk_id, experts, shared=None, gate=None):
+        """``gate``: logits ``[T]``, the shared expert's rows are multiplied by their sigmoid."""
         y = self.moe(x, topk_w, topk_id, experts)
+        if shared is not None and gate is not None:
+            shared = shared.float() * torch.sigmoid(gate.float()).unsqueeze(-1)
+            return (y.float() + shared).to(y.dtype)
         return y if shared is None else self.add(y, shared)
 
+    # -------------------------------------------------------------- parallel branches, position vectors, sigmoid attention
+    def embed_positions(self, table, tokens, positions, scale: float, freq, copy=None):
+        """Scaled embedding rows plus their position's vector, fp32; ``copy`` gets them in its own type."""
+        x = table[tokens.long()].float() * scale + ref.position_vectors(positions, freq.double().sum(0), table.shape[1])
+        if copy is not None:
+            copy.copy_(x)
+        return x
+
+    def branch_step(self, x, br, eps, dtype, w1=None, w2=None, copy=None):
+        """Add a layer's branches (None: nothing) to the fp32 rows ``x``; then their RMS norms with the weights ``w1`` and ``w2`` (None: no
+        such norm) in ``dtype``.  ``copy`` gets the rows in its own type.  (rows, norm 1, norm 2)"""
+        if br is not None:
+            if br.norms is not None:
+                y = sum(self.norm_rows(r.float(), None, w, eps, torch.float32) for r, w in zip(br.rows, br.norms)) / len(br.norms)
+            else:
+                y = br.rows.float()
+            if br.ffn is not None:
+                y = y + br.ffn.float()
+            x = x + br.mult * y
+        if copy is not None:
+            copy.copy_(x)
+        return (x,) + tuple(None if w is None else self.norm_rows(x, None, w, eps, dtype) for w in (w1, w2))
+
+    def sigmoid_attention(self, proj, M, batch, kv, layer_idx, eps, out, state_only: bool = False):
+        """Sigmoid attention of a mixer (convolution, norm and page write included) into ``out``.  Sequences flagged in
+        ``batch.h_gdn_defer`` leave their convolution's inputs untouched; ``state_only`` advances those and does nothing else."""
+        A, a, T, dt = M.attn, M.attn.spec, proj.shape[0], proj.dtype
+        nq, nk, nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
+        u = torch.cat([proj[:, M.cols[c]:][:, :n] for c, n in (("q", nq), ("k", nk), ("v", nv))], 1)
+        y, defer = u.float(), getattr(batch, "h_gdn_defer", None)
+        if a.conv:
+            y, state = torch.empty(u.shape, device=u.device), kv.qkv_state.get(layer_idx)
+            for b, slot in enumerate(batch.h_slots):
+                r0, r1 = batch.h_q_start[b], batch.h_q_start[b + 1]
+                if r1 <= r0:
+                    continue
+                fresh = state is None or batch.h_ctx_len[b] == r1 - r0
+                y[r0:r1], after = ref.causal_conv(u[r0:r1], u.new_zeros(a.conv - 1, u.shape[1]) if fresh else state[slot], A.conv_w)
+                if state is not None and not (defer is not None and defer[b]):
+                    state[slot].copy_(after)
+        if state_only:
+            return
+        q, k, v = y[:, :nq].view(T, -1, a.dim), y[:, nq:nq + nk].view(T, -1, a.dim), y[:, nq + nk:].view(T, -1, a.vdim)
+        if a.temp_coef:
+            q = q * ref.query_temperature(batch.positions, a.temp_coef, a.temp_every).view(T, 1, 1)
+        if a.unit_v:
+            v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)
+        valid = batch.slot_mapping >= 0
+        ref.kv_write(kv.k[layer_idx], kv.v[layer_idx], k[valid], v[valid], batch.slot_mapping[valid])
+        o = ref.sigmoid_attention(q.to(dt), kv.k[layer_idx], kv.v[layer_idx], kv.block_table, batch.h_slots, batch.h_q_start,
+                                  batch.h_ctx_len, a.scale, A.bias, A.PAD, a.window)
+        out.copy_(o.reshape(T, -1) * a.out_scale)
+
     # -------------------------------------------------------------- MoE
-    def router_topk(self, logits, k, renorm=True):
-        return ref.router_topk(logits, k, renorm)
+    def router_topk(self, logits, k, renorm=True, sigmoid=False, n_exp=None):
+        """``n_exp``: the experts' logits are the first ``n_exp`` columns."""
+        return ref.router_topk(logits if n_exp is None else logits[:, :n_exp], k, renorm, sigmoid)
 
     def moe(self, x, topk_w, topk_id, experts):
         """experts: an object with ``num_experts`` and ``forward_one(e, x)``."""
-        return ref.moe_forward(x, topk_w, topk_id, experts.forward_one, experts.num_experts)
+        return ref.moe_forward(x, topk_w, topk_id, experts.forward_one, experts.num_experts, experts.weigh_input)
 
     # -------------------------------------------------------------- GDN
     def gdn(self, mixed_qkv, z, b, a, gdn, model, batch, kv, layer_idx, state_only: bool = False):
