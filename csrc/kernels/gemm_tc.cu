@@ -639,7 +639,7 @@ BLZ_API int blz_gemm_push_rs(void* const* slots, void* const* flags, void* done_
 // kind: 0 bf16, 1 nvfp4, 2 mxfp8, 3 fp8.  A [M, K] and B [N, K] row-major (packed bytes for 4/8-bit kinds);
 // lda / ldb in BYTES.  out_f32: C is fp32, else bf16; ldc in elements.  bn: 128 or 256 (0 = choose).
 // act = 1: B's rows come in groups of [16 gate | 16 up] features and C is bf16 [M, N/2] = silu(gate) * up (ldc % 8 == 0);
-// act = 2: the clamped form of glu.cuh with act_limit; act = 3: the squared ReLU of every column (any N, experts too).
+// act = 2: the clamped form of glu.cuh with act_limit; act = 3: the squared ReLU of every column (any N).  All of them by expert too.
 // b_kt > 0: B is the tile-major repack [ceil(N/128)][b_kt][128][128 bytes] (zero padded), b_kt = ceil(row bytes / 128).
 BLZ_API int blz_gemm_tc(int kind, const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
                         int M, int N, int K, const float* row_scale, const float* alpha, const void* bias,
@@ -675,7 +675,7 @@ BLZ_API int blz_gemm_tc(int kind, const void* A, long long lda, const void* B, l
   p.b_raw = reinterpret_cast<const uint8_t*>(B);
   p.act = act;
   p.act_limit = act_limit;
-  if (act && (out_f32 || (act != 3 && (N % 32 || (ldc & 7) || tile_expert)))) return (int)cudaErrorInvalidValue;
+  if (act && (out_f32 || (act != 3 && (N % 32 || (ldc & 7))))) return (int)cudaErrorInvalidValue;
   if (b_kt > 0 && tile_expert) return (int)cudaErrorInvalidValue;
   p.mc_out = nullptr; p.done_ctr = nullptr; p.epoch = nullptr; p.spin_limit = 0; p.rank = 0; p.world = 1;
   p.push_rows_per = 0;

@@ -1,8 +1,8 @@
 // Mixture-of-experts routing and token movement around the grouped tcgen05 GEMM:
-//   route   : softmax over all experts → top-k (lowest id wins ties) → optional renormalisation, plus a histogram of
+//   route   : softmax over all experts (or their sigmoids) → top-k (lowest id wins ties) → optional renormalisation, plus a histogram of
 //             the experts this rank holds (reference semantics: kernels/src/cuda/ops_basic.cu router_topk_kernel :196)
 //   plan    : prefix sums of the 128-row padded per-expert counts → row offsets and the expert of every M tile
-//   scatter : copies each routed token's (quantised) activation row into its expert's row range
+//   scatter : copies each routed token's (quantised) activation row into its expert's row range, times its weight where that is asked for
 //   combine : out[token] = sum_k w[token,k] * y[row_of(token,k)]
 // Experts not held by this rank (expert parallelism) are skipped: the result is this rank's partial sum, which the
 // fused reduce + norm kernel adds across ranks — tokens are already replicated, so no dispatch traffic is needed.
@@ -15,7 +15,8 @@ namespace blz {
 
 // One warp per token.  E <= 512, k <= 32.
 __global__ void moe_route_kernel(const float* __restrict__ logits, float* __restrict__ topk_w, int* __restrict__ topk_id,
-                                 int* __restrict__ counts, int T, int E, int k, int renorm, int first, int local_n) {
+                                 int* __restrict__ counts, int T, int E, int k, int renorm, int first, int local_n, long long ld,
+                                 int sigmoid) {
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T) return;
@@ -25,18 +26,19 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, float* __rest
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
     const int e = j * 32 + lane;
-    v[j] = e < E ? logits[(size_t)t * E + e] : -INFINITY;
+    v[j] = e < E ? logits[(size_t)t * ld + e] : -INFINITY;
     mx = fmaxf(mx, v[j]);
   }
   mx = warp_max(mx);
   float sum = 0.f;
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
-    v[j] = (j * 32 + lane) < E ? __expf(v[j] - mx) : -1.f;      // -1 marks "absent / taken"
+    if (sigmoid) v[j] = (j * 32 + lane) < E ? 1.f / (1.f + expf(-v[j])) : -1.f;
+    else v[j] = (j * 32 + lane) < E ? __expf(v[j] - mx) : -1.f;      // -1 marks "absent / taken"
     if (v[j] > 0.f) sum += v[j];
   }
   sum = warp_sum(sum);
-  const float inv = 1.f / sum;
+  const float inv = sigmoid ? 1.f : 1.f / sum;
   float wsum = 0.f;
   float my_w = 0.f;
   int my_id = 0;
@@ -52,7 +54,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, float* __rest
       const int oi = __shfl_xor_sync(0xffffffffu, bid, o);
       if (ob > best || (ob == best && oi < bid)) { best = ob; bid = oi; }
     }
-    if ((bid & 31) == lane) v[bid >> 5] = -1.f;
+    if ((bid & 31) == lane && bid < E) v[bid >> 5] = -1.f;      // no candidate left (scores that are not numbers): nothing to take
     if (lane == i) { my_w = best * inv; my_id = bid; }
     wsum += best * inv;
   }
@@ -103,7 +105,7 @@ __global__ void moe_scatter_kernel(const uint8_t* __restrict__ src, const uint8_
                                    const float* __restrict__ src_rs, uint8_t* __restrict__ dst, uint8_t* __restrict__ dst_sf,
                                    float* __restrict__ dst_rs, const int* __restrict__ topk_id, const int* __restrict__ offsets,
                                    int* __restrict__ fill, int* __restrict__ row_map, int K, int k, int first, int local_n,
-                                   int sf_tiles) {
+                                   int sf_tiles, const float* __restrict__ weights, int f32) {
   const int t = blockIdx.x;
   __shared__ int s_row[32];
   if (threadIdx.x < k) {
@@ -119,6 +121,28 @@ __global__ void moe_scatter_kernel(const uint8_t* __restrict__ src, const uint8_
   for (int j = 0; j < k; ++j) {
     const int row = s_row[j];
     if (row < 0) continue;
+    if (QK == 0 && weights) {                        // rows times the token's weight for this expert
+      const float w = weights[(size_t)t * k + j];
+      if (f32) {
+        const float* sf = reinterpret_cast<const float*>(src + (size_t)t * row_bytes);
+        float* df = reinterpret_cast<float*>(dst + (size_t)row * row_bytes);
+        for (int i = threadIdx.x; i < K / 2; i += blockDim.x) df[i] = w * sf[i];
+        continue;
+      }
+      const __nv_bfloat16* sb = reinterpret_cast<const __nv_bfloat16*>(src + (size_t)t * row_bytes);
+      __nv_bfloat16* db = reinterpret_cast<__nv_bfloat16*>(dst + (size_t)row * row_bytes);
+      if (row_bytes % 16) {
+        for (int i = threadIdx.x; i < K; i += blockDim.x) db[i] = __float2bfloat16(w * bf2f(sb[i]));
+      } else {
+        for (int i = threadIdx.x; i < row_bytes / 16; i += blockDim.x) {
+          const uint4 u = reinterpret_cast<const uint4*>(sb)[i];
+          const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&u);
+          reinterpret_cast<uint4*>(db)[i] = make_uint4(pack_bf16x2(w * bf2f(e[0]), w * bf2f(e[1])), pack_bf16x2(w * bf2f(e[2]), w * bf2f(e[3])),
+                                                       pack_bf16x2(w * bf2f(e[4]), w * bf2f(e[5])), pack_bf16x2(w * bf2f(e[6]), w * bf2f(e[7])));
+        }
+      }
+      continue;
+    }
     if (QK == 0 && row_bytes % 16) {                 // ragged rows: element by element
       const uint16_t* s2 = reinterpret_cast<const uint16_t*>(src + (size_t)t * row_bytes);
       uint16_t* d2 = reinterpret_cast<uint16_t*>(dst + (size_t)row * row_bytes);
@@ -168,12 +192,13 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const fl
 
 using namespace blz;
 
-BLZ_API int blz_moe_route(const float* logits, float* topk_w, int* topk_id, int* counts, int T, int E, int k, int renorm,
-                          int first, int local_n, cudaStream_t s) {
-  if (E > 512 || k > 32 || k < 1 || local_n > 512) return (int)cudaErrorInvalidValue;
+// logits [T, ld], the experts' in the first E columns.  sigmoid: scores are sigmoids of the logits, else a softmax over them.
+BLZ_API int blz_moe_route(const float* logits, long long ld, float* topk_w, int* topk_id, int* counts, int T, int E, int k, int renorm,
+                          int sigmoid, int first, int local_n, cudaStream_t s) {
+  if (E > 512 || k > 32 || k < 1 || k > E || local_n > 512) return (int)cudaErrorInvalidValue;
   cudaMemsetAsync(counts, 0, sizeof(int) * (local_n > 0 ? local_n : 1), s);
   if (T == 0) return 0;
-  moe_route_kernel<<<(T + 3) / 4, 128, 0, s>>>(logits, topk_w, topk_id, counts, T, E, k, renorm, first, local_n);
+  moe_route_kernel<<<(T + 3) / 4, 128, 0, s>>>(logits, topk_w, topk_id, counts, T, E, k, renorm, first, local_n, ld, sigmoid);
   return (int)cudaGetLastError();
 }
 
@@ -183,13 +208,15 @@ BLZ_API int blz_moe_plan(const int* counts, int* offsets, int* fill, int* tile_e
   return (int)cudaGetLastError();
 }
 
+// weights (qk 0 only; [T, k] or null): a row is multiplied by its weight on the way; f32: the rows are fp32 (K counts 16-bit elements).
 BLZ_API int blz_moe_scatter(int qk, const void* src, const void* src_sf, const float* src_rs, void* dst, void* dst_sf,
                             float* dst_rs, const int* topk_id, const int* offsets, int* fill, int* row_map, int T, int K, int k,
-                            int first, int local_n, cudaStream_t s) {
+                            int first, int local_n, const float* weights, int f32, cudaStream_t s) {
   if (T == 0) return 0;
+  if (weights && qk) return (int)cudaErrorInvalidValue;
   const int sf_tiles = qk == 1 ? (K + 63) / 64 : (K + 127) / 128;
 #define BLZ_SC(Q) moe_scatter_kernel<Q><<<T, 128, 0, s>>>((const uint8_t*)src, (const uint8_t*)src_sf, src_rs, (uint8_t*)dst, \
-    (uint8_t*)dst_sf, dst_rs, topk_id, offsets, fill, row_map, K, k, first, local_n, sf_tiles)
+    (uint8_t*)dst_sf, dst_rs, topk_id, offsets, fill, row_map, K, k, first, local_n, sf_tiles, weights, f32)
   if (qk == 0) BLZ_SC(0); else if (qk == 1) BLZ_SC(1); else BLZ_SC(2);
 #undef BLZ_SC
   return (int)cudaGetLastError();

@@ -7,7 +7,8 @@
 // per sublayer.  Before the first sublayer all streams equal the scaled embedding row, which is read from the table
 // (`from_embed`) instead of being copied S times; after the last one only the sum of the streams is written.
 // Beside them: the norm of fp32 rows, the residual sum of a post-norm decoder (residual_norm_kernel), the residual that takes
-// normed branches (branch_norm_kernel), and the causal convolution of a residual over time (input_conv_kernel).
+// normed branches (branch_norm_kernel), the residual that takes a mixer and a feed-forward side by side (branch_step_kernel), embedding
+// rows with position vectors (embed_positions_kernel), and the causal convolution of a residual over time (input_conv_kernel).
 // One CTA per row; the row's columns stay with their thread (float4 where the width allows), so the update is in place.
 #include "blaze/host.h"
 #include "blaze/sm100.cuh"
@@ -327,6 +328,161 @@ __global__ void __launch_bounds__(512) branch_norm_kernel(BranchParams p) {
   }
 }
 
+// sums of two numbers over the block
+__device__ __forceinline__ float2 block_sum2(float2 v, float2* red) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+  v.x = warp_sum(v.x);
+  v.y = warp_sum(v.y);
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  float2 r = make_float2(0.f, 0.f);
+  for (int i = 0; i < nw; ++i) { r.x += red[i].x; r.y += red[i].y; }
+  return r;
+}
+
+// What stands between two layers whose mixer and feed-forward read the same residual:
+//   x <- x + mult * (mixer + ffn), in fp32; then up to two RMS norms of it, for the next mixer and feed-forward, and a copy (activation type).
+// mixer: a row of y1, or (m1) the mean of the rows of y1 and y2, each RMS-normed with a weight; or nothing (y1 null: x stays as it is).
+// ffn: the sum of the k rows of routed that row_map names (-1: none), times weights where there are any, and of a row of extra times
+// sigmoid(gate) where there is a gate.
+struct BranchStepParams {
+  float* x;                    // [T, W]
+  const void *y1, *y2;         // [T, W] activation type
+  const float *m1, *m2;        // [W]
+  const void* routed;          // [.., ld_routed]
+  const float* weights;        // [T, k] or null
+  const int* row_map;          // [T, k]
+  const void* extra;           // [T, W] or null
+  const float* gate;           // gate[t * ld_gate], or null
+  const float *w1, *w2;        // [W] or null
+  void *h1, *h2, *copy;        // [T, W], [T, W], [T, ld_copy] activation type, or null
+  long long ld_routed, ld_gate, ld_copy;
+  int k, W;
+  float mult, eps;
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(512) branch_step_kernel(BranchStepParams p) {
+  extern __shared__ float u_row[];                   // [W]
+  __shared__ float2 red0[16];
+  __shared__ float red1[16], s_w[32];
+  __shared__ int s_row[32];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, W = p.W;
+  const size_t at = (size_t)t * W;
+  const T *y1 = reinterpret_cast<const T*>(p.y1) + at, *y2 = reinterpret_cast<const T*>(p.y2) + at;
+  const T *routed = reinterpret_cast<const T*>(p.routed), *extra = reinterpret_cast<const T*>(p.extra);
+  const bool add = p.y1 != nullptr, normed = p.m1 != nullptr;
+  float f1 = 1.f, f2 = 0.f, sg = 1.f;
+  if (add) {
+    if (threadIdx.x < p.k) {
+      s_w[threadIdx.x] = p.weights ? p.weights[(size_t)t * p.k + threadIdx.x] : 1.f;
+      s_row[threadIdx.x] = p.row_map[(size_t)t * p.k + threadIdx.x];
+    }
+    if (p.gate) sg = 1.f / (1.f + expf(-p.gate[(size_t)t * p.ld_gate]));
+    float2 ss = make_float2(0.f, 0.f);
+    if (normed) {
+      for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+        float a[VEC], b[VEC];
+        ld_vec<VEC>(y1 + c, a);
+        ld_vec<VEC>(y2 + c, b);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) { ss.x = fmaf(a[j], a[j], ss.x); ss.y = fmaf(b[j], b[j], ss.y); }
+      }
+    }
+    ss = block_sum2(ss, red0);                       // also makes s_w and s_row visible
+    if (normed) {
+      f1 = 0.5f / sqrtf(ss.x / (float)W + p.eps);
+      f2 = 0.5f / sqrtf(ss.y / (float)W + p.eps);
+    }
+  }
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float x[VEC];
+    ld_vec<VEC>(p.x + at + c, x);
+    if (add) {
+      float u[VEC], v[VEC];
+      ld_vec<VEC>(y1 + c, u);
+      if (normed) {
+        float g[VEC], w[VEC];
+        ld_vec<VEC>(y2 + c, v);
+        ld_vec<VEC>(p.m1 + c, g);
+        ld_vec<VEC>(p.m2 + c, w);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) u[j] = fmaf(u[j] * f1, g[j], v[j] * f2 * w[j]);
+      }
+      if (extra) {
+        ld_vec<VEC>(extra + at + c, v);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) u[j] = fmaf(sg, v[j], u[j]);
+      }
+      for (int i = 0; i < p.k; ++i) {
+        if (s_row[i] < 0) continue;
+        ld_vec<VEC>(routed + (size_t)s_row[i] * p.ld_routed + c, v);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) u[j] = fmaf(s_w[i], v[j], u[j]);
+      }
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) x[j] = fmaf(p.mult, u[j], x[j]);
+      st_vec<VEC>(p.x + at + c, x);
+    }
+    if (p.copy) st_vec<VEC>(reinterpret_cast<T*>(p.copy) + (size_t)t * p.ld_copy + c, x);
+    if (p.w1 || p.w2) {
+      st_vec<VEC>(u_row + c, x);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) ss = fmaf(x[j], x[j], ss);
+    }
+  }
+  if (!p.w1 && !p.w2) return;
+  const float rs = 1.f / sqrtf(block_sum(ss, red1) / (float)W + p.eps);
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float u[VEC], w[VEC], h[VEC];
+    ld_vec<VEC>(u_row + c, u);
+    if (p.w1) {
+      ld_vec<VEC>(p.w1 + c, w);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) h[j] = u[j] * rs * w[j];
+      st_vec<VEC>(reinterpret_cast<T*>(p.h1) + at + c, h);
+    }
+    if (p.w2) {
+      ld_vec<VEC>(p.w2 + c, w);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) h[j] = u[j] * rs * w[j];
+      st_vec<VEC>(reinterpret_cast<T*>(p.h2) + at + c, h);
+    }
+  }
+}
+
+// x = scale * table[token] + position vector: sine (even columns) and cosine (odd ones) of position * freq[column / 2], with freq given as
+// two floats so that far positions keep their angle; copy (activation type, or null) gets the row too.
+template <typename T>
+__global__ void __launch_bounds__(256) embed_positions_kernel(const T* __restrict__ table, const int* __restrict__ tokens,
+                                                              const int* __restrict__ positions, const float* __restrict__ freq, int vocab,
+                                                              float scale, float* __restrict__ x, T* __restrict__ copy, long long ld_copy, int W) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, half = (W + 1) / 2;
+  int tok = tokens[t];
+  tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);
+  const T* row = table + (size_t)tok * W;
+  const float pos = (float)positions[t];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    const float hi = freq[i], ang = pos * hi, rest = fmaf(pos, hi, -ang) + pos * freq[half + i];
+    float s, c;
+    sincosf(ang, &s, &c);
+    const float v[2] = {fmaf(rest, c, s), fmaf(-rest, s, c)};
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int col = 2 * i + j;
+      if (col >= W) break;
+      const float y = fmaf(scale, ld_act(row + col), v[j]);
+      x[(size_t)t * W + col] = y;
+      if (copy) st_act(copy + (size_t)t * ld_copy + col, y);
+    }
+  }
+}
+
 // h = x + conv(x): a causal convolution of every column over a sequence's rows, whose earlier inputs are in the sequence's state row.
 // A thread takes VEC columns of up to kConvSeg rows of one sequence; a longer run's state is written by a kernel of its own (its first
 // segment reads the old one).  TAPS = 0: any number, read again for every row.
@@ -560,6 +716,44 @@ BLZ_API int blz_embed_norm(const void* table, const int* tokens, int vocab, cons
   if (T <= 0 || W < 1 || W > 51200 || vocab < 1 || !table || !tokens || !w || !x) return (int)cudaErrorInvalidValue;
   const BranchParams p = {table, nullptr, nullptr, tokens, w, x, nullptr, W, 0, W, vocab, eps};
   return launch_branch<EMBED>(p, T, f32, W % 4 == 0, s);
+}
+
+// See BranchStepParams; f32 = 1: the activation type is fp32.  k <= 32, W <= 51200.
+BLZ_API int blz_branch_step(float* x, const void* y1, const void* y2, const float* m1, const float* m2, const void* routed, long long ld_routed,
+                            const float* weights, const int* row_map, int k, const void* extra, const float* gate, long long ld_gate,
+                            const float* w1, const float* w2, void* h1, void* h2, void* copy, long long ld_copy, float mult, float eps, int T,
+                            int W, int f32, cudaStream_t s) {
+  using namespace blz;
+  if (T <= 0 || W < 1 || W > 51200 || !x || k < 0 || k > 32 || (k && (!routed || !row_map)) || (m1 && (!m2 || !y1 || !y2)) ||
+      (w1 && !h1) || (w2 && !h2))
+    return (int)cudaErrorInvalidValue;
+  const BranchStepParams p = {x, y1, y2, m1, m2, routed, weights, row_map, extra, gate, w1, w2, h1, h2, copy, ld_routed, ld_gate, ld_copy,
+                              k, W, mult, eps};
+  const bool vec = W % 4 == 0 && ld_routed % 4 == 0 && ld_copy % 4 == 0;
+  const dim3 block(row_threads(W, vec ? 4 : 1));
+#define BLZ_BS(TT, V)                                                                                \
+  do {                                                                                               \
+    static PerDeviceOnce once;                                                                       \
+    const cudaError_t e = once.smem_limit(branch_step_kernel<TT, V>, 200 * 1024);                    \
+    if (e != cudaSuccess) return (int)e;                                                             \
+    return (int)launch_pdl(branch_step_kernel<TT, V>, dim3(T), block, (size_t)W * 4, s, p);          \
+  } while (0)
+  if (f32) { if (vec) BLZ_BS(float, 4); BLZ_BS(float, 1); }
+  if (vec) BLZ_BS(__nv_bfloat16, 4);
+  BLZ_BS(__nv_bfloat16, 1);
+#undef BLZ_BS
+}
+
+// x [T, W] fp32 = scale * table[token] + sines and cosines (embed_positions_kernel); freq [2][(W + 1) / 2].
+BLZ_API int blz_embed_positions(const void* table, const int* tokens, const int* positions, const float* freq, int vocab, float scale, float* x,
+                                void* copy, long long ld_copy, int T, int W, int f32, cudaStream_t s) {
+  using namespace blz;
+  if (T <= 0 || W < 1 || vocab < 1 || !table || !tokens || !positions || !freq || !x) return (int)cudaErrorInvalidValue;
+  if (f32)
+    return (int)launch_pdl(embed_positions_kernel<float>, dim3(T), dim3(256), 0, s, (const float*)table, tokens, positions, freq, vocab, scale, x,
+                           (float*)copy, ld_copy, W);
+  return (int)launch_pdl(embed_positions_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, s, (const __nv_bfloat16*)table, tokens, positions, freq,
+                         vocab, scale, x, (__nv_bfloat16*)copy, ld_copy, W);
 }
 
 // See InputConvParams; max_q: the longest run of the batch.  no_store: optional [B], 1 = leave the sequence's state as it was.
