@@ -3,14 +3,18 @@
 // A head has one or two query / key maps of `dim` and one value of `vdim`; a map is a softmax attention of its own.
 //   two maps (differential attention): the head's output is rms(a1 - lam * a2) * post over its vdim values;
 //   one map: a * sigmoid(gate) * post, where the softmax may have a sink: one more term exp(sink) in the denominator, without a
-//   key and a value; sink and gate are optional.
+//   key and a value; sink and gate are optional;
+//   sigmoid (one map): a key's weight is sigmoid(score + bias), not its share of a sum; the bias is a number per head and distance.
 // Query head h reads key/value head h / group.  A row sees the keys at most window - 1 positions before it (window 0: all).
 // A page block (one page, one key/value head) is [K map 1 | (K map 2) | V] of 16 tokens each, as 8 x 8 core matrices:
 // element (token t, column j) of a part with D padded columns sits at (t / 8) * 8 D + (j / 8) * 64 + (t % 8) * 8 + j % 8.
 #pragma once
+#include "blaze/attn.cuh"
 #include "blaze/sm100.cuh"
 
 namespace blz {
+
+static constexpr int kBiasPad = 128;
 
 struct MapsParams {
   const void* q;               // [T, ld]: q [heads][maps][dim] of every row
@@ -34,11 +38,16 @@ struct MapsParams {
   int row_blocks, splits, stages;
   int* status;
   const int* page_base;        // [B] or null: the pages of sequence b are page_base[b] + page index, not block_table's
+  const float* bias;           // sigmoid: [heads][bias_len()], entry kBiasPad + distance, see bias_len
+  int reach;                   // sigmoid: distances listed one by one; keys farther away have the last one's bias
   int shared_kv;               // one map: a block is its key part alone, whose first vdim columns are the values
 
   __host__ __device__ int group() const { return heads / kv_heads; }
   __host__ __device__ int dp() const { return (dim + 15) / 16 * 16; }
   __host__ __device__ int vp() const { return (vdim + 15) / 16 * 16; }
+  // a row's entries around its own position can be read for a whole tile: those of keys that come later are -inf, those beyond
+  // the last listed distance equal it.  The tensor-core kernels take the table times -log2(e).
+  __host__ __device__ int bias_len() const { return reach + 2 * kBiasPad; }
   __host__ __device__ int block_elems() const { return 16 * (maps * dp() + vp()); }
 };
 
@@ -69,6 +78,13 @@ __device__ __forceinline__ void copy_rows(__nv_bfloat16* dst, int R, int D, int 
   }
 }
 __device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
+// 1 / (1 + 2^t): the sigmoid of a score s for t = -s log2(e)
+__device__ __forceinline__ float sigmoid_ex2(float t) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + ex2(t)));
+  return r;
+}
 
 // factor of output column e of (row t, head h): sigmoid(gate) * post
 template <typename T>

@@ -1,5 +1,5 @@
 // Softmax attention of one or two maps per head (attn_maps.cuh) over paged bf16 / fp32 keys and values: the page write, a plain
-// kernel for any size and for fp32, and the short-row kernel (decode, verify rows, short prompt portions).  Long prompt portions
+// kernel for any size and for fp32, the same with sigmoid weights, and the short-row kernel (decode, verify rows, short prompt portions).  Long prompt portions
 // are attn_maps_tc.cu's.
 //
 // Short rows: a CTA takes 16 query rows (new tokens x group) of one key/value head and a range of pages; its four warps take
@@ -47,7 +47,7 @@ __global__ void __launch_bounds__(256) maps_store_kernel(MapsParams p, int vec) 
 
 // ------------------------------------------------------------------------------------------ any size, either type
 // One CTA (128 threads) per (row, head): 128 keys at a time, a key per thread for the scores, value columns over the threads.
-template <typename T, int MAPS>
+template <typename T, int MAPS, bool SIG = false>
 __global__ void __launch_bounds__(128) maps_plain_kernel(MapsParams p) {
   constexpr int VC = 8;                                // value columns per thread: vdim <= 128 * VC
   extern __shared__ float sh[];
@@ -86,8 +86,12 @@ __global__ void __launch_bounds__(128) maps_plain_kernel(MapsParams p) {
         float d = 0.f;
         for (int j = 0; j < p.dim; ++j) d = fmaf(s_q[mp * p.dim + j], ad_ld(kr + core_off(key & 15, j, dp)), d);
         s[mp] = d * p.scale;
+        if constexpr (SIG) s[mp] += p.bias[(size_t)h * p.bias_len() + kBiasPad + min(pos - key, p.reach - 1)];
       }
     }
+    if constexpr (SIG) {
+      s_p[tid] = s[0] == -INFINITY ? 0.f : 1.f / (1.f + expf(-s[0]));
+    } else {
 #pragma unroll
     for (int mp = 0; mp < MAPS; ++mp) {
       const float v = warp_max(s[mp]);
@@ -106,6 +110,7 @@ __global__ void __launch_bounds__(128) maps_plain_kernel(MapsParams p) {
 #pragma unroll
       for (int c = 0; c < VC; ++c) acc[mp][c] *= f;
     }
+    }
     __syncthreads();
     const int k_end = min(128, pos - k0 + 1);
     for (int kk = max(lo - k0, 0); kk < k_end; ++kk) {
@@ -121,6 +126,13 @@ __global__ void __launch_bounds__(128) maps_plain_kernel(MapsParams p) {
       }
     }
   }
+  T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + (size_t)h * p.vdim;
+  if constexpr (SIG) {
+#pragma unroll
+    for (int c = 0; c < VC; ++c)
+      if (tid + c * 128 < p.vdim) ad_st(out + tid + c * 128, acc[0][c] * gate_factor<T>(p, t, h, tid + c * 128));
+    return;
+  }
   __syncthreads();
 #pragma unroll
   for (int mp = 0; mp < MAPS; ++mp) {
@@ -128,7 +140,6 @@ __global__ void __launch_bounds__(128) maps_plain_kernel(MapsParams p) {
     if (lane == 0) red[mp][warp] = v;
   }
   __syncthreads();
-  T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + (size_t)h * p.vdim;
   const float l0 = red[0][0] + red[0][1] + red[0][2] + red[0][3];
   if constexpr (MAPS == 1) {
     const float sink = p.sink ? p.sink[h] : -INFINITY, mx = fmaxf(m[0], sink), f = expf(m[0] - mx);
@@ -178,13 +189,13 @@ static constexpr float kLazy = 8.f;      // log2 of how far a row's weights may 
 
 // what a CTA's finished rows become: the head's output (one key range) or an entry of the workspace.
 // 8 threads per row; o holds this thread's columns, relative to the maxima m (log2), with sums l.
-template <int MAPS, int VP>
+template <int MAPS, int VP, bool SIG>
 __device__ __forceinline__ void finish_rows(const MapsParams& p, float (&o)[MAPS][VP / 8], const float (&m)[MAPS], const float (&l)[MAPS],
                                             int row_t, int head, int sub) {
   float f;
   if constexpr (MAPS == 1) {
     if (row_t < 0) return;
-    f = 1.f / (l[0] + (p.sink ? ex2(p.sink[head] * kLog2e - m[0]) : 0.f));
+    f = SIG ? 1.f : 1.f / (l[0] + (p.sink ? ex2(p.sink[head] * kLog2e - m[0]) : 0.f));
   } else {
     const float i0 = 1.f / l[0], i1 = p.lam / l[1];
     float ss = 0.f;
@@ -206,7 +217,7 @@ __device__ __forceinline__ void finish_rows(const MapsParams& p, float (&o)[MAPS
   }
 }
 
-template <int MAPS, int VP>
+template <int MAPS, int VP, bool SIG>
 __global__ void __launch_bounds__(kShortWarps * 32) maps_short_kernel(MapsParams p) {
   extern __shared__ __align__(128) uint8_t smem_raw[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -276,6 +287,17 @@ __global__ void __launch_bounds__(kShortWarps * 32) maps_short_kernel(MapsParams
   const int row_a = rb * 16 + (lane >> 2);
   const int pos_a = row_a < rows ? pos0 + row_a / group : -1, pos_b = row_a + 8 < rows ? pos0 + (row_a + 8) / group : -1;
   const int lo_a = first_key(pos_a, p.window), lo_b = first_key(pos_b, p.window);
+  // sigmoid: this thread's two rows of the bias table, and their last entries
+  const float *ba = nullptr, *bb = nullptr;
+  float far_a = 0.f, far_b = 0.f;
+  int far_key = -1;                             // pages that end at or before it are beyond the listed distances for every row
+  if constexpr (SIG) {
+    ba = p.bias + (size_t)(g * group + row_a % group) * p.bias_len() + kBiasPad;
+    bb = p.bias + (size_t)(g * group + (row_a + 8) % group) * p.bias_len() + kBiasPad;
+    far_a = ba[p.reach - 1];
+    far_b = bb[p.reach - 1];
+    far_key = pos0 + tok_lo - (p.reach - 1);
+  }
   const int mat = lane >> 3, mrow = lane & 7;
   const uint32_t q_addr = smem_u32(sQ) + ((mat & 1) * 8 * dp + (mat >> 1) * 64 + mrow * 8) * 2;
   bool ok = true;
@@ -302,6 +324,26 @@ __global__ void __launch_bounds__(kShortWarps * 32) maps_short_kernel(MapsParams
       }
     }
     const int key = k0 + 2 * (lane & 3);
+    uint32_t hi[MAPS][4], lo[MAPS][4];
+    if constexpr (SIG) {
+      const bool far = k0 + 15 <= far_key && p.window == 0;
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          float t = k < 2 ? far_a : far_b;
+          if (!far) {
+            const int pos = k < 2 ? pos_a : pos_b, kk = key + h * 8 + (k & 1);
+            const bool vis = kk <= pos && kk >= (k < 2 ? lo_a : lo_b);
+            t = vis ? (k < 2 ? ba : bb)[min(pos - kk, p.reach - 1)] : INFINITY;
+          }
+          s[0][h][k] = sigmoid_ex2(fmaf(s[0][h][k], -sc, t));
+        }
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) split_bf16x2(s[0][h][2 * r], s[0][h][2 * r + 1], hi[0][h * 2 + r], lo[0][h * 2 + r]);
+    } else {
     float mx[MAPS][2];
 #pragma unroll
     for (int mp = 0; mp < MAPS; ++mp) {
@@ -342,7 +384,6 @@ __global__ void __launch_bounds__(kShortWarps * 32) maps_short_kernel(MapsParams
         for (int c = 0; c < VP / 8; ++c) { o[mp][c][0] *= f[0]; o[mp][c][1] *= f[0]; o[mp][c][2] *= f[1]; o[mp][c][3] *= f[1]; }
       }
     }
-    uint32_t hi[MAPS][4], lo[MAPS][4];
 #pragma unroll
     for (int mp = 0; mp < MAPS; ++mp) {
       float w[2][4];
@@ -357,6 +398,7 @@ __global__ void __launch_bounds__(kShortWarps * 32) maps_short_kernel(MapsParams
       for (int h = 0; h < 2; ++h)
 #pragma unroll
         for (int r = 0; r < 2; ++r) split_bf16x2(w[h][2 * r], w[h][2 * r + 1], hi[mp][h * 2 + r], lo[mp][h * 2 + r]);
+    }
     }
     const uint32_t va = blk + (MAPS * 16 * dp + (mat & 1) * 8 * vp + (mat >> 1) * 64 + mrow * 8) * 2;
 #pragma unroll
@@ -422,6 +464,7 @@ __global__ void __launch_bounds__(kShortWarps * 32) maps_short_kernel(MapsParams
     for (int w = 0; w < kShortWarps; ++w) mm[mp] = fmaxf(mm[mp], s_ml[((w * MAPS + mp) * 16 + r) * 2]);
 #pragma unroll
     for (int w = 0; w < kShortWarps; ++w) {
+      if constexpr (SIG) { f[mp][w] = rb * 16 + r < rows ? 1.f : 0.f; continue; }
       const float mw = s_ml[((w * MAPS + mp) * 16 + r) * 2];
       f[mp][w] = mw == -INFINITY ? 0.f : ex2(mw - mm[mp]);
       ll[mp] = fmaf(f[mp][w], s_ml[((w * MAPS + mp) * 16 + r) * 2 + 1], ll[mp]);
@@ -440,7 +483,7 @@ __global__ void __launch_bounds__(kShortWarps * 32) maps_short_kernel(MapsParams
       }
     }
   if (p.splits == 1) {
-    finish_rows<MAPS, VP>(p, res, mm, ll, rr < rows ? r0 + rr / group : -1, g * group + rr % group, sub);
+    finish_rows<MAPS, VP, SIG>(p, res, mm, ll, rr < rows ? r0 + rr / group : -1, g * group + rr % group, sub);
   } else if (rr < rows) {
     const size_t w = (((size_t)b * p.kv_heads + g) * p.row_blocks + rb) * p.splits + split;
 #pragma unroll
@@ -454,7 +497,7 @@ __global__ void __launch_bounds__(kShortWarps * 32) maps_short_kernel(MapsParams
 }
 
 // joins the split key ranges of one (sequence, key/value head, 16 rows)
-template <int MAPS, int VP>
+template <int MAPS, int VP, bool SIG>
 __global__ void __launch_bounds__(128) maps_combine_kernel(MapsParams p) {
   pdl_trigger();
   pdl_wait();
@@ -476,8 +519,8 @@ __global__ void __launch_bounds__(128) maps_combine_kernel(MapsParams p) {
     for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, p.part_ml[(((w0 + s) * MAPS + mp) * 16 + r) * 2]);
     for (int s = 0; s < p.splits; ++s) {
       const float* ml = p.part_ml + (((w0 + s) * MAPS + mp) * 16 + r) * 2;
-      if (ml[0] == -INFINITY) continue;
-      const float f = ex2(ml[0] - mm);
+      if (!SIG && ml[0] == -INFINITY) continue;
+      const float f = SIG ? 1.f : ex2(ml[0] - mm);
       l[mp] = fmaf(f, ml[1], l[mp]);
       const float* po = p.part_o + (((w0 + s) * MAPS + mp) * 16 + r) * VP + sub;
 #pragma unroll
@@ -486,12 +529,12 @@ __global__ void __launch_bounds__(128) maps_combine_kernel(MapsParams p) {
     }
     mx[mp] = mm;
   }
-  finish_rows<MAPS, VP>(p, o, mx, l, rr < rows ? r0 + rr / p.group() : -1, g * p.group() + rr % p.group(), sub);
+  finish_rows<MAPS, VP, SIG>(p, o, mx, l, rr < rows ? r0 + rr / p.group() : -1, g * p.group() + rr % p.group(), sub);
 }
 
 static constexpr int kShortSmemTarget = 110 * 1024;      // two CTAs per SM
 
-template <int MAPS, int VP>
+template <int MAPS, int VP, bool SIG = false>
 static cudaError_t launch_short(MapsParams p, cudaStream_t s) {
   const int be = p.block_elems() * 2, fixed = 512 + MAPS * 16 * p.dp() * 2;
   const int merge = (kShortWarps * MAPS * 16 * (VP + 4) + kShortWarps * MAPS * 16 * 2) * 4;
@@ -501,13 +544,13 @@ static cudaError_t launch_short(MapsParams p, cudaStream_t s) {
   if (ring < merge) ring = merge;
   if (fixed + ring > 227 * 1024) return cudaErrorInvalidValue;
   p.stages = st;
-  auto kern = maps_short_kernel<MAPS, VP>;
+  auto kern = maps_short_kernel<MAPS, VP, SIG>;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(kern, 227 * 1024);
   if (e != cudaSuccess) return e;
   e = launch_pdl(kern, dim3(p.row_blocks * p.splits, p.kv_heads, p.B), dim3(kShortWarps * 32), fixed + ring, s, p);
   if (e != cudaSuccess || p.splits == 1) return e;
-  return launch_pdl(maps_combine_kernel<MAPS, VP>, dim3(p.row_blocks, p.kv_heads, p.B), dim3(128), 0, s, p);
+  return launch_pdl(maps_combine_kernel<MAPS, VP, SIG>, dim3(p.row_blocks, p.kv_heads, p.B), dim3(128), 0, s, p);
 }
 
 static cudaError_t check_maps(const MapsParams& p, int esz) {
@@ -521,6 +564,11 @@ static int run_plain(const MapsParams& p, int f32, cudaStream_t s) {
   if (check_maps(p, f32 ? 4 : 2) != cudaSuccess || p.vdim > 1024 || p.dim > 4096 || p.heads > 65535 || !p.seq_of_row) return (int)cudaErrorInvalidValue;
   const size_t sm = p.maps * (p.dim + 128) * sizeof(float);
   const dim3 grid(p.T, p.heads);
+  if (p.bias) {
+    if (p.maps != 1 || p.reach < 1) return (int)cudaErrorInvalidValue;
+    if (f32) return (int)launch_pdl(maps_plain_kernel<float, 1, true>, grid, dim3(128), sm, s, p);
+    return (int)launch_pdl(maps_plain_kernel<__nv_bfloat16, 1, true>, grid, dim3(128), sm, s, p);
+  }
   if (p.maps == 1) {
     if (f32) return (int)launch_pdl(maps_plain_kernel<float, 1>, grid, dim3(128), sm, s, p);
     return (int)launch_pdl(maps_plain_kernel<__nv_bfloat16, 1>, grid, dim3(128), sm, s, p);
@@ -533,6 +581,10 @@ static int run_short(const MapsParams& p, cudaStream_t s) {
   if (check_maps(p, 2) != cudaSuccess || p.dim > 128 || p.vdim > 128) return (int)cudaErrorInvalidValue;
   if (p.max_rows < 1 || p.row_blocks < 1 || p.splits < 1 || p.B > 65535 || p.kv_heads > 65535 || (p.splits > 1 && (!p.part_o || !p.part_ml)))
     return (int)cudaErrorInvalidValue;
+  if (p.bias) {
+    if (p.maps != 1 || p.reach < 1) return (int)cudaErrorInvalidValue;
+    return (int)(p.vdim <= 32 ? launch_short<1, 32, true>(p, s) : p.vdim <= 64 ? launch_short<1, 64, true>(p, s) : launch_short<1, 128, true>(p, s));
+  }
 #define BLZ_SHORT(M) return (int)(p.vdim <= 32 ? launch_short<M, 32>(p, s) : p.vdim <= 64 ? launch_short<M, 64>(p, s) : launch_short<M, 128>(p, s))
   if (p.maps == 1) { BLZ_SHORT(1); }
   BLZ_SHORT(2);
@@ -709,6 +761,155 @@ __global__ void __launch_bounds__(128) attn_prep_pages_kernel(PrepParams p) {
   }
 }
 
+// ------------------------------------------------------------------------------------------ convolution, value norm, page write
+struct ConvPrepParams {
+  PrepParams a;                // sizes, offsets, query buffer, pages
+  const float* w;              // [taps][C], C = q | k | v columns
+  void* state;                 // [rows][taps - 1][C]: the last projected rows of each sequence
+  const int *slots, *q_start, *ctx_len, *no_store;
+  int taps, unit_v, state_only;
+  float temp_coef, temp_every;
+};
+static constexpr int kConvPrepTok = 8;     // tokens per warp, at least the taps before the current one
+
+// A warp per (8 tokens of a sequence, head): a causal convolution over time of each projected channel, then queries (times their position's
+// temperature) to their buffer, keys and values (divided by their root mean square: unit_v) to their page.  The rows before the sequence's
+// new ones come from its state, which only the first 8 tokens' warp of a channel reads, and then writes.  TAPS: the real ones rounded up.
+template <typename T, int TAPS, int VEC>
+__global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) {
+  pdl_trigger();
+  pdl_wait();
+  const PrepParams& p = q.a;
+  const int lane = threadIdx.x & 31, u = blockIdx.y * 4 + (threadIdx.x >> 5), b = blockIdx.z, t0 = blockIdx.x * kConvPrepTok;
+  const int r0 = q.q_start[b], n = q.q_start[b + 1] - r0;
+  if (u >= p.heads + 2 * p.kv_heads || t0 >= n) return;
+  const bool is_q = u < p.heads, is_v = u >= p.heads + p.kv_heads;
+  const int D = is_v ? p.vdim : p.dim, g = is_v ? u - p.heads - p.kv_heads : u - p.heads, taps = q.taps, m = min(kConvPrepTok, n - t0);
+  const int C = p.heads * p.dim + p.kv_heads * (p.dim + p.vdim);
+  const int ch = is_q ? u * p.dim : is_v ? p.heads * p.dim + p.kv_heads * p.dim + g * p.vdim : p.heads * p.dim + g * p.dim;     // first channel
+  const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)r0 * p.ld + (is_q ? p.q_off + (size_t)u * p.dim
+                                                                          : is_v ? p.v_off + (size_t)g * p.vdim : p.k_off + (size_t)g * p.dim);
+  const bool fresh = q.ctx_len[b] == n;
+  T* st = reinterpret_cast<T*>(q.state) + (size_t)q.slots[b] * (taps - 1) * C + ch;
+  const int dp = (p.dim + 15) / 16 * 16, vp = (p.vdim + 15) / 16 * 16;
+  auto load = [&](const T* at, float (&v)[VEC]) {
+    if constexpr (VEC == 4 && sizeof(T) == 2) {
+      const uint2 w = *reinterpret_cast<const uint2*>(at);
+      v[0] = __uint_as_float(w.x << 16); v[1] = __uint_as_float(w.x & 0xffff0000u);
+      v[2] = __uint_as_float(w.y << 16); v[3] = __uint_as_float(w.y & 0xffff0000u);
+    } else if constexpr (VEC == 4) {
+      const float4 w = *reinterpret_cast<const float4*>(at);
+      v[0] = w.x; v[1] = w.y; v[2] = w.z; v[3] = w.w;
+    } else {
+      v[0] = ad_ld(at);
+    }
+  };
+  auto input = [&](int t, int c, float (&v)[VEC]) {     // projected columns c.. of the sequence's new token t (negative: before them)
+    if (t >= 0) {
+      load(src + (size_t)t * p.ld + c, v);
+    } else if (!fresh && t > -taps) {
+      load(st + (size_t)(taps - 1 + t) * C + c, v);
+    } else {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] = 0.f;
+    }
+  };
+  float y[kConvPrepTok][VEC];
+  auto conv = [&](int c) {
+    float in[TAPS - 1 + kConvPrepTok][VEC], w[TAPS][VEC];
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) {
+      const int r = i - (TAPS - taps);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) w[i][j] = r >= 0 ? q.w[(size_t)r * C + ch + c + j] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < TAPS - 1 + kConvPrepTok; ++i) {
+      if (i < TAPS - 1 + m) {
+        input(t0 + i - (TAPS - 1), c, in[i]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) in[i][j] = 0.f;
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < kConvPrepTok; ++k) {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        y[k][j] = 0.f;
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) y[k][j] = fmaf(w[i][j], in[k + i][j], y[k][j]);
+      }
+    }
+  };
+  if (!q.state_only) {
+    const bool once = D <= 32 * VEC;
+    float f[kConvPrepTok];
+#pragma unroll
+    for (int k = 0; k < kConvPrepTok; ++k) f[k] = 1.f;
+    if (once && lane * VEC < D) conv(lane * VEC);
+    if (is_v && q.unit_v) {
+      float ss[kConvPrepTok];
+#pragma unroll
+      for (int k = 0; k < kConvPrepTok; ++k) ss[k] = 0.f;
+      for (int c = lane * VEC; c < D; c += 32 * VEC) {
+        if (!once) conv(c);
+#pragma unroll
+        for (int k = 0; k < kConvPrepTok; ++k)
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) ss[k] = fmaf(y[k][j], y[k][j], ss[k]);
+      }
+#pragma unroll
+      for (int k = 0; k < kConvPrepTok; ++k)
+        if (k < m) f[k] = 1.f / sqrtf(warp_sum(ss[k]) / (float)D + p.eps);
+    } else if (is_q && q.temp_coef != 0.f) {
+#pragma unroll
+      for (int k = 0; k < kConvPrepTok; ++k)
+        if (k < m) f[k] = fmaf(q.temp_coef, logf(floorf(__fdiv_rn((float)(p.positions[r0 + t0 + k] + 1), q.temp_every)) + 1.f), 1.f);
+    }
+    for (int c = lane * VEC; c < D; c += 32 * VEC) {
+      if (!once) conv(c);
+#pragma unroll
+      for (int k = 0; k < kConvPrepTok; ++k) {
+        if (k >= m) break;
+        const int row = r0 + t0 + k;
+        T* dst;
+        if (is_q) {
+          dst = reinterpret_cast<T*>(p.q_out) + ((size_t)row * p.heads + u) * p.dim + c;
+        } else {
+          const int slot = p.slot_mapping[row];
+          if (slot < 0) continue;
+          dst = reinterpret_cast<T*>(p.pool) + (size_t)(slot >> 4) * p.page_stride + (size_t)g * p.head_stride +
+                (is_v ? 16 * dp + core_off(slot & 15, c, vp) : core_off(slot & 15, c, dp));
+        }
+        if constexpr (VEC == 4 && sizeof(T) == 2)
+          *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(y[k][0] * f[k], y[k][1] * f[k]), pack_bf16x2(y[k][2] * f[k], y[k][3] * f[k]));
+        else if constexpr (VEC == 4)
+          *reinterpret_cast<float4*>(dst) = make_float4(y[k][0] * f[k], y[k][1] * f[k], y[k][2] * f[k], y[k][3] * f[k]);
+        else
+          ad_st(dst, y[k][0] * f[k]);
+      }
+    }
+  }
+  if (t0 > 0 || taps < 2 || (q.no_store != nullptr && q.no_store[b])) return;
+  for (int c = lane * VEC; c < D; c += 32 * VEC) {
+    for (int i = 0; i < taps - 1; ++i) {               // entry i: the row taps - 1 - i before the next token; an older entry moves up
+      float v[VEC];
+      input(n - (taps - 1) + i, c, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) ad_st(st + (size_t)i * C + c + j, v[j]);
+    }
+  }
+}
+
+template <typename T, int TAPS>
+static int launch_conv_prep(const ConvPrepParams& q, bool vec, int B, int max_q, cudaStream_t s) {
+  const PrepParams& p = q.a;
+  const dim3 grid((max_q + kConvPrepTok - 1) / kConvPrepTok, (p.heads + 2 * p.kv_heads + 3) / 4, B);
+  if (vec) return (int)launch_pdl(conv_prep_pages_kernel<T, TAPS, 4>, grid, dim3(128), 0, s, q);
+  return (int)launch_pdl(conv_prep_pages_kernel<T, TAPS, 1>, grid, dim3(128), 0, s, q);
+}
+
 static MapsParams soft_params(const void* q, long long ld, void* out, long long ld_out, void* pool, long long page_stride, long long head_stride,
                               const int* block_table, int bt_stride, const int* slots, const int* q_start, const int* ctx_len,
                               const float* sink, const void* gate, long long ld_gate, int T, int B, int heads, int kv_heads, int dim,
@@ -740,6 +941,33 @@ BLZ_API int blz_attn_prep_pages(const void* qkv, long long ld, long long q_off, 
   const dim3 grid((unsigned)((warps + 3) / 4));
   if (f32) return (int)launch_pdl(attn_prep_pages_kernel<float>, grid, dim3(128), 0, s, p);
   return (int)launch_pdl(attn_prep_pages_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, p);
+}
+
+// q, k and v of the T rows (element offsets into a row of qkv) through a causal convolution over time (w [taps][C] fp32, taps <= 8, C the
+// columns q | k | v; state [rows][taps - 1][C], activation type, which advances unless no_store): q times 1 + temp_coef ln(floor((position
+// + 1) / temp_every) + 1) to q_out, k and v (divided by their root mean square: unit_v) to their page slots (-1: skip).  max_q: the longest
+// run of the batch.  state_only: the state advances and nothing else is written.
+BLZ_API int blz_conv_prep_pages(const void* qkv, long long ld, long long q_off, long long k_off, long long v_off, void* q_out, void* pool,
+                                long long page_stride, long long head_stride, const int* positions, const int* slot_mapping, const float* w,
+                                void* state, const int* slots, const int* q_start, const int* ctx_len, const int* no_store, int B, int max_q,
+                                int T, int heads, int kv_heads, int dim, int vdim, int taps, int unit_v, float temp_coef, float temp_every,
+                                float eps, int state_only, int f32, cudaStream_t s) {
+  using namespace blz;
+  if (T <= 0 || B < 1 || B > 65535 || max_q < 1 || heads < 1 || kv_heads < 1 || heads + 2 * kv_heads > 4 * 65535 || dim < 1 || vdim < 1 ||
+      taps < 1 || taps > kConvPrepTok || !w || (taps > 1 && !state) || temp_every <= 0.f)
+    return (int)cudaErrorInvalidValue;
+  ConvPrepParams q = {};
+  PrepParams& p = q.a;
+  p.qkv = qkv; p.ld = ld; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.q_out = q_out; p.pool = pool;
+  p.page_stride = page_stride; p.head_stride = head_stride; p.positions = positions; p.slot_mapping = slot_mapping;
+  p.T = T; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.eps = eps;
+  q.w = w; q.state = state; q.slots = slots; q.q_start = q_start; q.ctx_len = ctx_len; q.no_store = no_store;
+  q.taps = taps; q.unit_v = unit_v; q.state_only = state_only; q.temp_coef = temp_coef; q.temp_every = temp_every;
+  const int unit = f32 ? 16 : 8;                       // bytes of four columns
+  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && (ld | q_off | k_off | v_off) % 4 == 0 && reinterpret_cast<uintptr_t>(qkv) % unit == 0 &&
+                   reinterpret_cast<uintptr_t>(state) % unit == 0;
+  if (f32) return taps <= 4 ? launch_conv_prep<float, 4>(q, vec, B, max_q, s) : launch_conv_prep<float, 8>(q, vec, B, max_q, s);
+  return taps <= 4 ? launch_conv_prep<__nv_bfloat16, 4>(q, vec, B, max_q, s) : launch_conv_prep<__nv_bfloat16, 8>(q, vec, B, max_q, s);
 }
 
 // One softmax map per head with an optional sink ([heads] fp32) and an optional output gate ([T, ld_gate], columns like out's);
@@ -776,5 +1004,29 @@ BLZ_API int blz_soft_short(const void* q, long long ld, void* out, long long ld_
   blz::MapsParams p = blz::soft_params(q, ld, out, ld_out, pool, page_stride, head_stride, block_table, bt_stride, slots, q_start, ctx_len,
                                        sink, gate, ld_gate, T, B, heads, kv_heads, dim, vdim, window, scale, post);
   p.max_rows = max_rows; p.row_blocks = row_blocks; p.splits = splits; p.part_o = part_o; p.part_ml = part_ml;
+  return blz::run_short(p, s);
+}
+
+// Sigmoid attention (attn_maps.cuh): bias [heads][reach + 256] fp32, every row of the step; otherwise as blz_soft_plain.
+BLZ_API int blz_sigmoid_plain(const void* q, long long ld, void* out, long long ld_out, void* pool, long long page_stride, long long head_stride,
+                              const int* block_table, int bt_stride, const int* slots, const int* q_start, const int* ctx_len,
+                              const float* bias, int reach, const int* seq_of_row, int T, int B, int heads, int kv_heads, int dim, int vdim,
+                              int window, float scale, float post, int f32, cudaStream_t s) {
+  blz::MapsParams p = blz::soft_params(q, ld, out, ld_out, pool, page_stride, head_stride, block_table, bt_stride, slots, q_start, ctx_len,
+                                       nullptr, nullptr, 0, T, B, heads, kv_heads, dim, vdim, window, scale, post);
+  if (!bias) return (int)cudaErrorInvalidValue;
+  p.seq_of_row = seq_of_row; p.bias = bias; p.reach = reach;
+  return blz::run_plain(p, f32, s);
+}
+
+// The same for the short sequences of a bf16 step (see blz_soft_short); bias times -log2(e).
+BLZ_API int blz_sigmoid_short(const void* q, long long ld, void* out, long long ld_out, void* pool, long long page_stride, long long head_stride,
+                              const int* block_table, int bt_stride, const int* slots, const int* q_start, const int* ctx_len,
+                              const float* bias, int reach, int T, int B, int heads, int kv_heads, int dim, int vdim, int window, float scale,
+                              float post, int max_rows, int row_blocks, int splits, float* part_o, float* part_ml, cudaStream_t s) {
+  blz::MapsParams p = blz::soft_params(q, ld, out, ld_out, pool, page_stride, head_stride, block_table, bt_stride, slots, q_start, ctx_len,
+                                       nullptr, nullptr, 0, T, B, heads, kv_heads, dim, vdim, window, scale, post);
+  if (!bias) return (int)cudaErrorInvalidValue;
+  p.max_rows = max_rows; p.row_blocks = row_blocks; p.splits = splits; p.part_o = part_o; p.part_ml = part_ml; p.bias = bias; p.reach = reach;
   return blz::run_short(p, s);
 }

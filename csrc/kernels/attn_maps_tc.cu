@@ -3,6 +3,8 @@
 // Two maps: a CTA takes up to 128 query rows (tokens x group) of one key/value head.  The two maps of a head are the two halves of a
 // ping-pong: warpgroup 0 runs the softmax of map 1, warpgroup 1 that of map 2, while the tensor core works on the other map.
 // One map: a CTA takes two blocks of up to 128 query rows; the blocks are the two halves, and share keys and values.
+// Sigmoid (one map): a weight needs no maximum and no sum, so O is never rescaled; the biases of a row's listed distances are read from a
+// table in shared memory, and beyond them a tile has one number per row.  The table also masks what a row may not see.
 //   S_m = Q_m K_m^T   A = Q_m [128 x dim], B = K_m [128 keys x dim], both K-major in shared memory
 //   O_m += P_m V      A = P_m in tensor memory, B = V [keys x vdim], the pages' token-major blocks read as an MN-major operand
 // Tensor memory (512 columns): S_1 | S_2 | O_1 | O_2, 128 each.  A map's weights overwrite its scores as two bf16 halves, value
@@ -35,9 +37,10 @@ __device__ __forceinline__ void mma_f16_ts(uint32_t d_tmem, uint32_t a_tmem, uin
 }
 struct MapsTc {
   int ks, vs;                  // K and V ring depths
+  int tab_ld;                  // sigmoid: floats per head of the bias table in shared memory (0: it stays in global memory)
 };
 
-template <int MAPS>
+template <int MAPS, bool SIG>
 __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, MapsTc c, int vec_q, int vec_o) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~uintptr_t(127));
@@ -54,6 +57,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 16);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   int* s_item = reinterpret_cast<int*>(tmem_slot + 2);          // sequence, first token of the row block
+  float* s_tab = reinterpret_cast<float*>(s_item + 2);          // [group][tab_ld]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_trigger();
@@ -89,6 +93,12 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
     *abort_flag = 0;
     mbar_fence_init();
   }
+  if constexpr (SIG) {
+    if (c.tab_ld)
+      for (int i = threadIdx.x; i < group * p.bias_len(); i += kTcThreads)
+        s_tab[i / p.bias_len() * c.tab_ld + i % p.bias_len()] = p.bias[(size_t)blockIdx.y * group * p.bias_len() + i];
+  }
+  __syncwarp();
   if (warp == 9) tmem_alloc(tmem_slot, 512);
   tc_fence_before();
   __syncthreads();
@@ -216,6 +226,12 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
       const uint32_t s_addr = tmem + m * 128 + lanes, o_addr = tmem + 256 + m * 128 + lanes;
       float mx = -INFINITY, l = 0.f;
       bool ok = true;
+      const float* tab = nullptr;                      // this row's biases by distance
+      float far = 0.f;
+      if constexpr (SIG) {
+        tab = (c.tab_ld ? s_tab + (r % group) * c.tab_ld : p.bias + (size_t)head * p.bias_len()) + kBiasPad;
+        far = tab[p.reach - 1];
+      }
       for (int i = 0; i < n; ++i) {
         ok = __all_sync(0xffffffffu, mbar_wait(&s_full[m], (uint32_t)(i & 1), abort_flag, p.status));
         if (!ok) break;
@@ -225,6 +241,41 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
         for (int k = 0; k < 4; ++k) tmem_ld32(s_addr + k * 32, v[k]);
         tmem_ld_wait();
         const int k0 = (pg_lo + i * 8) * 16, a = lo - k0, z = pos - k0;       // columns a..z are visible
+        if constexpr (SIG) {
+          const float nsc = -sc;
+          if (__all_sync(0xffffffffu, z - 127 >= p.reach - 1)) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+#pragma unroll
+              for (int j = 0; j < 32; ++j) v[k][j] = __float_as_uint(fmaf(__uint_as_float(v[k][j]), nsc, far));
+          } else {
+            const float* at = tab + max(min(z, p.reach + 126), -1);
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+#pragma unroll
+              for (int j = 0; j < 32; ++j) v[k][j] = __float_as_uint(fmaf(__uint_as_float(v[k][j]), nsc, at[-(k * 32 + j)]));
+          }
+          if (__any_sync(0xffffffffu, a > 0)) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (k * 32 + j < a) v[k][j] = 0x7f800000u;                     // weight 0
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            uint32_t hi[16], rm[16];
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              const float w0 = sigmoid_ex2(__uint_as_float(v[k][2 * j])), w1 = sigmoid_ex2(__uint_as_float(v[k][2 * j + 1]));
+              const __nv_bfloat162 h = __floats2bfloat162_rn(w0, w1);
+              hi[j] = *reinterpret_cast<const uint32_t*>(&h);
+              rm[j] = pack_bf16x2(w0 - __uint_as_float(hi[j] << 16), w1 - __uint_as_float(hi[j] & 0xffff0000u));
+            }
+            tmem_st16(s_addr + k * 16, hi);
+            tmem_st16(s_addr + 64 + k * 16, rm);
+          }
+        } else {
         if (!__all_sync(0xffffffffu, a <= 0 && z >= 127)) {
 #pragma unroll
           for (int k = 0; k < 4; ++k)
@@ -273,6 +324,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
           tmem_st16(s_addr + 64 + k * 16, rm);
         }
         l += l0 + l1;
+        }
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
@@ -281,7 +333,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
       if constexpr (MAPS == 1) {
         if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&o_full[m], 0, abort_flag, p.status));
         tc_fence_after();
-        const float f = 1.f / (l + (p.sink ? ex2(p.sink[head] * kLog2e - mx) : 0.f));
+        const float f = SIG ? 1.f : 1.f / (l + (p.sink ? ex2(p.sink[head] * kLog2e - mx) : 0.f));
         __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(r0 + tq) * p.ld_out + (size_t)head * p.vdim;
         const __nv_bfloat16* gate =
             p.gate ? reinterpret_cast<const __nv_bfloat16*>(p.gate) + (size_t)(r0 + tq) * p.ld_gate + (size_t)head * p.vdim : nullptr;
@@ -368,15 +420,24 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
   }
 }
 
-template <int MAPS>
+template <int MAPS, bool SIG = false>
 static int run_tc(const MapsParams& p, int items, cudaStream_t s) {
   if (p.T <= 0 || p.B <= 0 || p.heads < 1 || p.kv_heads < 1 || p.kv_heads > 65535 || p.heads % p.kv_heads || p.group() > 128 || p.dim < 1 ||
       p.dim > 256 || p.vdim < 1 || p.vdim > 128 || p.window < 0 || items < 1)
     return (int)cudaErrorInvalidValue;
   if ((p.page_stride * 2) % 16 || (p.head_stride * 2) % 16 || (reinterpret_cast<uintptr_t>(p.pool) & 15)) return (int)cudaErrorInvalidValue;
   const int q_bytes = 256 * p.dp() * 2, k_bytes = MAPS * 128 * p.dp() * 2, v_bytes = 128 * p.vp() * 2, fixed = 128 + 2048 + 256;
-  MapsTc c = {2, 2};
-  auto total = [&]() { return fixed + q_bytes + c.ks * k_bytes + c.vs * v_bytes; };
+  if (SIG && (!p.bias || p.reach < 1)) return (int)cudaErrorInvalidValue;
+  MapsTc c = {2, 2, 0};
+  int tab = 0;
+  auto total = [&]() { return fixed + q_bytes + c.ks * k_bytes + c.vs * v_bytes + tab; };
+  if (SIG && p.bias_len() <= 16384) {
+    // neighbouring tokens of a head read neighbouring entries; the heads of a warp's rows are set apart by as many banks as it has tokens
+    const int ld = (p.bias_len() + 31) / 32 * 32 + (p.group() < 32 ? 32 / p.group() : 1);
+    tab = p.group() * ld * 4;
+    if (total() <= 227 * 1024) c.tab_ld = ld;
+    else tab = 0;
+  }
   if (total() > 227 * 1024) c.ks = 1;
   if (total() > 227 * 1024) c.vs = 1;
   if (total() > 227 * 1024) return (int)cudaErrorInvalidValue;
@@ -384,9 +445,9 @@ static int run_tc(const MapsParams& p, int items, cudaStream_t s) {
   const int vec_o = (reinterpret_cast<uintptr_t>(p.out) & 15) == 0 && p.ld_out % 8 == 0 && p.vdim % 8 == 0 &&
                     (!p.gate || ((reinterpret_cast<uintptr_t>(p.gate) & 15) == 0 && p.ld_gate % 8 == 0));
   static PerDeviceOnce once;
-  cudaError_t e = once.smem_limit(maps_tc_kernel<MAPS>, 227 * 1024);
+  cudaError_t e = once.smem_limit(maps_tc_kernel<MAPS, SIG>, 227 * 1024);
   if (e != cudaSuccess) return (int)e;
-  return (int)launch_pdl(maps_tc_kernel<MAPS>, dim3(items, p.kv_heads), dim3(kTcThreads), total(), s, p, c, vec_q, vec_o);
+  return (int)launch_pdl(maps_tc_kernel<MAPS, SIG>, dim3(items, p.kv_heads), dim3(kTcThreads), total(), s, p, c, vec_q, vec_o);
 }
 
 }  // namespace blz
@@ -424,4 +485,20 @@ BLZ_API int blz_soft_tc(const void* q, long long ld, void* out, long long ld_out
   p.scale = scale; p.post = post; p.max_rows = max_rows;
   p.status = status_word();
   return run_tc<1>(p, items, s);
+}
+
+// Sigmoid attention (attn_maps.cuh) of the long sequences of a bf16 step; bias [heads][reach + 256] fp32 times -log2(e); otherwise as
+// blz_soft_tc.
+BLZ_API int blz_sigmoid_tc(const void* q, long long ld, void* out, long long ld_out, void* pool, long long page_stride, long long head_stride,
+                           const int* block_table, int bt_stride, const int* slots, const int* q_start, const int* ctx_len,
+                           const float* bias, int reach, int T, int B, int heads, int kv_heads, int dim, int vdim, int window, float scale,
+                           float post, int max_rows, int items, cudaStream_t s) {
+  using namespace blz;
+  MapsParams p = {};
+  p.q = q; p.ld = ld; p.out = out; p.ld_out = ld_out; p.pool = pool; p.page_stride = page_stride; p.head_stride = head_stride;
+  p.block_table = block_table; p.bt_stride = bt_stride; p.slots = slots; p.q_start = q_start; p.ctx_len = ctx_len;
+  p.T = T; p.B = B; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.maps = 1;
+  p.scale = scale; p.post = post; p.max_rows = max_rows; p.bias = bias; p.reach = reach;
+  p.status = status_word();
+  return run_tc<1, true>(p, items, s);
 }
