@@ -140,7 +140,7 @@ class Medodra(Model):
             return dense(gate_up, p + "gate+up"), dense(tensor(p + "down", W, ff), p + "down")
         M, E = MoeMlp(), Experts()
         M.top_k, M.renorm, M.sigmoid, M.rows_out, M.experts = spec.top, spec.renorm, spec.scores == "sigmoid", True, E
-        E.act, E.weigh_input, E.num_experts, E.count = spec.act, spec.weigh_input, spec.experts, spec.experts
+        E.act, E.weigh_input, E.fused_act, E.num_experts, E.count = spec.act, spec.weigh_input, True, spec.experts, spec.experts
         for e in range(spec.experts):
             gate_up, down = glu(f"{p}e{e}.", spec.ff)
             E.gate_up.append(gate_up)

@@ -94,7 +94,8 @@ class SigmoidAttn:
         table = rel.float().cpu()[idx].t() + shift.float().cpu()[:, None]
         self.reach = n                   # distances listed one by one
         self.bias = torch.cat([torch.full((spec.heads, self.PAD), -math.inf), table], 1).contiguous().to(device)
-        self.conv_w = None if conv_w is None else conv_w.t().to(device, torch.float32).contiguous()
+        self.bias_ex2 = self.bias * -math.log2(math.e)       # what the tensor-core kernels take
+        self.conv_w = torch.ones(1, spec.conv_dim, device=device) if conv_w is None else conv_w.t().to(device, torch.float32).contiguous()
 
 
 class LatentAttn:
@@ -199,6 +200,7 @@ class Experts:
 
     act = "swiglu"                       # or "relu2": no gate, ``gate_up`` holds the up projections alone
     weigh_input = False                  # an expert's weight multiplies its input instead of its output
+    fused_act = False                    # SwiGLU in the grouped product's epilogue (bf16; the packed rows are interleaved for it)
 
     def __init__(self):
         self.gate_up: List[Linear] = []

@@ -50,10 +50,11 @@ class _Symbols:
 
 class RoutedRows:
     """What routed experts leave behind: ``rows`` in the padded row space, the ``row_map [T, k]`` of each token's rows with their
-    ``weights``, and rows that are added to the sums (``extra``, may be None)."""
+    ``weights`` (None: the rows count as they are), and rows that are added to the sums (``extra``, may be None; times the sigmoid of
+    ``gate``, logits ``[T]``, where there is one)."""
 
-    def __init__(self, rows, row_map, weights, extra):
-        self.rows, self.row_map, self.weights, self.extra = rows, row_map, weights, extra
+    def __init__(self, rows, row_map, weights, extra, gate=None):
+        self.rows, self.row_map, self.weights, self.extra, self.gate = rows, row_map, weights, extra, gate
 
 
 class CudaOps:
@@ -124,7 +125,7 @@ class CudaOps:
         lib.blz_add_sigmoid_scaled.argtypes = [VP, VP, VP, VP, _c.c_int, _c.c_int, VP]
         lib.blz_gather_rows.argtypes = [VP, VP, VP, _c.c_int, _c.c_int, VP]
         lib.blz_argmax.argtypes = [VP, VP, VP, _c.c_int, _c.c_int, _c.c_longlong, _c.c_int, VP]
-        lib.blz_moe_route.argtypes = [VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_int, _c.c_int, _c.c_int, _c.c_int, VP]
+        lib.blz_moe_route.argtypes = [VP, _c.c_longlong, VP, VP, VP] + [_c.c_int] * 7 + [VP]
         lib.blz_moe_plan.argtypes = [VP, VP, VP, VP, VP, _c.c_int, _c.c_int, VP]
         lib.blz_moe_gemm.restype = _c.c_int
         lib.blz_moe_gemm.argtypes = [_c.c_int, VP, _c.c_longlong, VP, _c.c_longlong, VP, _c.c_longlong, _c.c_int, _c.c_int, _c.c_int,
@@ -144,7 +145,7 @@ class CudaOps:
         # on its columns (blz_moe_gemm); above it the 128-row tiles of the grouped GEMM are full enough (BLAZE_MOE_NARROW=0: never)
         self.MOE_NARROW_ROWS = 48 if os.environ.get("BLAZE_MOE_NARROW", "1") != "0" else 0
         lib.blz_moe_scatter.argtypes = [_c.c_int, VP, VP, VP, VP, VP, VP, VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_int, _c.c_int,
-                                        _c.c_int, VP]
+                                        _c.c_int, VP, _c.c_int, VP]
         lib.blz_moe_combine.argtypes = [VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_int, VP]
         self._route_counts = None
         lib.blz_gdn_conv.argtypes = [VP, _c.c_longlong, VP, VP, VP, VP, VP, VP, VP, _c.c_int, _c.c_int, _c.c_int, VP]
@@ -193,7 +194,7 @@ class CudaOps:
         lib.blz_soft_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
         lib.blz_short_conv.argtypes = [VP, LL] + [VP] * 8 + [_c.c_int] * 5 + [VP]
         runs = [_c.c_int] * 5 + [VP] + [_c.c_int] * 2 + [VP, LL, _c.c_int, VP]
-        lib.blz_delta_rule.argtypes = [VP, LL, VP, LL, VP, LL] + [VP] * 8 + runs
+        lib.blz_delta_rule.argtypes = [VP, LL, VP, LL, VP, LL] + [VP] * 8 + [_c.c_int] + runs
         lib.blz_state_space.argtypes = [VP, LL, VP, LL] + [VP] * 9 + runs
         lib.blz_rec_ws_bytes.restype = LL
         lib.blz_rec_ws_bytes.argtypes = [_c.c_int] * 5
@@ -205,6 +206,16 @@ class CudaOps:
         lib.blz_relu2.argtypes = [VP, _c.c_int, VP, LL, _c.c_int, VP]
         lib.blz_poly_norm.argtypes = [VP, VP, VP, _c.c_int, _c.c_int, _c.c_float, _c.c_int, VP]
         lib.blz_gemm_simple_experts.argtypes = [VP, LL, VP, VP, LL] + [_c.c_int] * 3 + [VP, VP, _c.c_int, VP]
+        # mixer and feed-forward side by side, position vectors, sigmoid attention, minGRU
+        lib.blz_branch_step.argtypes = [VP] * 6 + [LL, VP, VP, _c.c_int, VP, VP, LL] + [VP] * 5 + [LL] + [_c.c_float] * 2 + [_c.c_int] * 3 + [VP]
+        lib.blz_embed_positions.argtypes = [VP] * 4 + [_c.c_int, _c.c_float, VP, VP, LL] + [_c.c_int] * 3 + [VP]
+        lib.blz_conv_prep_pages.argtypes = ([VP] + [LL] * 4 + [VP, VP, LL, LL] + [VP] * 8 + [_c.c_int] * 9 + [_c.c_float] * 3 +
+                                            [_c.c_int] * 2 + [VP])
+        common = [VP, LL, VP, LL, VP, LL, LL, VP, _c.c_int, VP, VP, VP, VP, _c.c_int]
+        lib.blz_sigmoid_plain.argtypes = common + [VP] + shape + [_c.c_int, VP]
+        lib.blz_sigmoid_tc.argtypes = common + shape + [_c.c_int, _c.c_int, VP]
+        lib.blz_sigmoid_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
+        lib.blz_min_gru.argtypes = [VP, VP, VP, LL, VP, VP, LL, VP, VP, VP, VP] + [_c.c_int] * 4 + [VP]
         # latent attention
         lib.blz_latent_prep.argtypes = [VP, LL, LL, LL, VP, VP, LL, VP, VP, VP, VP, VP] + [_c.c_int] * 5 + [_c.c_float, _c.c_int, VP]
         lib.blz_latent_rot.argtypes = [VP] * 5 + [_c.c_int] * 7 + [VP]
@@ -942,21 +953,37 @@ class CudaOps:
         """The recurrent mixer of a layer: convolution, recurrence, gated norm into ``out`` (columns of a wider matrix).  Sequences
         flagged in ``batch.gdn_defer`` leave their state untouched; ``state_only`` advances the states and writes nothing."""
         R, r, T = M.rec, M.rec.spec, proj.shape[0]
+        if R.kind == "mingru":
+            self.min_gru(proj, M, batch, kv, layer_idx, None if state_only else out)
+            return
         y = self.short_conv(proj, M, batch, kv, layer_idx) if r.conv else None
         o = None if state_only else torch.empty(T, r.heads * r.vdim, dtype=torch.float32, device=self.device)
         self.recur(y, proj, low, M, batch, kv, layer_idx, o)
         if state_only:
             return
-        self.gated_norm(o, low if R.kind == "delta" else proj, M, eps, out)
+        self.gated_norm(o, low if low is not None else proj, M, eps, out)
+
+    def min_gru(self, proj, M, batch, kv, layer_idx, out):
+        """Elementwise gated recurrence with its output gate, into ``out`` (None: the state only)."""
+        r, es = M.rec.spec, proj.element_size()
+        z, u, g = [VP(proj.data_ptr() + M.cols[c] * es) for c in ("zg", "u", "g")]
+        lens = [e - s for s, e in zip(batch.h_q_start, batch.h_q_start[1:])]
+        kinds = (1 if 1 in lens else 0) | (2 if batch.max_q_len > 1 else 0)
+        if kinds == 3:
+            self.launches += 1
+        self._check(self.lib.blz_min_gru(z, u, g, proj.stride(0), _ptr(kv.rec_state[layer_idx]), _ptr(out), out.stride(0) if out is not None else 0,
+                                         _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(batch.gdn_defer),
+                                         batch.slots.numel(), r.width, kinds, int(es == 4), self._stream()), "min_gru")
 
     def gated_norm(self, o, gates, M, eps, out):
-        """The norm and gate of a recurrence's rows ``o``; ``gates`` holds the gate's columns: the low-rank outputs (delta rule), or
-        the input projection (state space; gated linear attention has none)."""
+        """The norm and gate of a recurrence's rows ``o``; ``gates`` holds the gate's columns: the low-rank outputs (delta rule with channel
+        decays), or the input projection (gated linear attention has none)."""
         R, r, es = M.rec, M.rec.spec, gates.element_size()
         delta = R.kind == "delta"
-        z = VP(0) if R.kind == "gated" else VP(gates.data_ptr() + (r.heads * r.dim if delta else M.cols["z"]) * es)
+        z = VP(0) if R.kind == "gated" else VP(gates.data_ptr() + (r.heads * r.dim if delta and not r.head_decay else M.cols["z"]) * es)
         self._check(self.lib.blz_group_norm(_ptr(o), z, gates.stride(0), _ptr(R.norm_w), _ptr(out), out.stride(0), o.shape[0], R.norm_groups,
-                                            o.shape[1] // R.norm_groups, R.norm_w.numel(), eps, r.out_scale, int(delta), int(not delta),
+                                            o.shape[1] // R.norm_groups, R.norm_w.numel(), eps, r.out_scale,
+                                            int(delta and r.gate == "sigmoid"), int(not delta),
                                             int(es == 4), self._stream()), "group_norm")
 
     REC_MAX_WS = 4 << 30       # workspace of the streaming recurrences; steps that need more run without it
@@ -974,7 +1001,7 @@ class CudaOps:
         long_rows, ws, ws_bytes = int(self.lib.blz_rec_long_rows()), None, 0
         kinds = (1 if 1 in lens else 0) | (2 if any(1 < n < long_rows for n in lens) else 0)
         if longest >= long_rows:
-            ws_bytes = int(self.lib.blz_rec_ws_bytes(2 if gated else int(delta), T, r.heads, groups, r.state))
+            ws_bytes = int(self.lib.blz_rec_ws_bytes(2 if gated else 3 if delta and r.head_decay else int(delta), T, r.heads, groups, r.state))
             if o is not None and ws_bytes <= self.REC_MAX_WS:
                 ws = torch.empty(ws_bytes, dtype=torch.uint8, device=self.device)
                 kinds |= 4
@@ -988,9 +1015,10 @@ class CudaOps:
             self._check(self.lib.blz_gated_linear(at[0], ld, at[1], ld, at[2], ld, _ptr(R.A), _ptr(R.dt_bias), _ptr(state), _ptr(o), *seqs,
                                                   r.heads, r.dim, r.vdim, *runs), "gated_linear")
         elif delta:
-            self._check(self.lib.blz_delta_rule(_ptr(y), y.stride(0), _ptr(low), low.stride(0), VP(proj.data_ptr() + M.cols["beta"] * es),
+            decay, ld = (VP(proj.data_ptr() + M.cols["decay"] * es), proj.stride(0)) if r.head_decay else (_ptr(low), low.stride(0))
+            self._check(self.lib.blz_delta_rule(_ptr(y), y.stride(0), decay, ld, VP(proj.data_ptr() + M.cols["beta"] * es),
                                                 proj.stride(0), _ptr(R.A), _ptr(R.dt_bias), _ptr(state), _ptr(o), *seqs, r.heads,
-                                                r.kv_heads, r.dim, r.vdim, *runs), "delta_rule")
+                                                r.kv_heads, r.dim, r.vdim, int(r.head_decay), *runs), "delta_rule")
         else:
             self._check(self.lib.blz_state_space(_ptr(y), y.stride(0), VP(proj.data_ptr() + M.cols["dt"] * es), proj.stride(0), _ptr(R.A),
                                                  _ptr(R.dt_bias), _ptr(R.D), _ptr(state), _ptr(o), *seqs, r.heads, r.groups, r.state,
@@ -1034,6 +1062,74 @@ class CudaOps:
             if batch.max_q_len > 32:
                 self.launches += 1
         return h
+
+    # ------------------------------------------------------------------ mixer and feed-forward side by side, sigmoid attention
+    def embed_positions(self, table, tokens, positions, scale: float, freq, copy=None):
+        """Scaled embedding rows plus their position's vector, fp32; ``copy`` (columns of a wider matrix) gets them in the table's type."""
+        T, W = tokens.numel(), table.shape[1]
+        x = torch.empty(T, W, dtype=torch.float32, device=self.device)
+        if T:
+            self._check(self.lib.blz_embed_positions(_ptr(table), _ptr(tokens), _ptr(positions), _ptr(freq), table.shape[0], scale, _ptr(x),
+                                                     _ptr(copy), copy.stride(0) if copy is not None else 0, T, W,
+                                                     int(table.dtype == torch.float32), self._stream()), "embed_positions")
+        return x
+
+    def branch_step(self, x, br, eps, dtype, w1=None, w2=None, copy=None):
+        """Add a layer's branches (None: nothing) to the fp32 rows ``x`` in place; then their RMS norms with the weights ``w1`` and ``w2``
+        (None: no such norm) in ``dtype``.  ``copy`` (columns of a wider matrix) gets the rows in ``dtype``.  (rows, norm 1, norm 2)"""
+        T, W = x.shape
+        h1, h2 = [None if w is None else torch.empty(T, W, dtype=dtype, device=self.device) for w in (w1, w2)]
+        if not T:
+            return x, h1, h2
+        y1 = y2 = m1 = m2 = ffn = None
+        mult = 0.0
+        if br is not None:
+            mult, ffn = br.mult, br.ffn
+            (y1, y2), (m1, m2) = (br.rows, br.norms) if br.norms is not None else ((br.rows, None), (None, None))
+        routed = (_ptr(ffn.rows), ffn.rows.stride(0), _ptr(ffn.weights), _ptr(ffn.row_map), ffn.row_map.shape[1], _ptr(ffn.extra),
+                  _ptr(ffn.gate), ffn.gate.stride(0) if ffn.gate is not None else 0) if ffn is not None else (VP(0), 0, VP(0), VP(0), 0, VP(0), VP(0), 0)
+        self._check(self.lib.blz_branch_step(_ptr(x), _ptr(y1), _ptr(y2), _ptr(m1), _ptr(m2), *routed, _ptr(w1), _ptr(w2), _ptr(h1), _ptr(h2),
+                                             _ptr(copy), copy.stride(0) if copy is not None else 0, mult, eps, T, W,
+                                             int(dtype == torch.float32), self._stream()), "branch_step")
+        return x, h1, h2
+
+    def conv_prep_pages(self, proj, M, batch, kv, layer_idx, eps, state_only: bool = False):
+        """Convolved queries ``[T, heads * dim]`` of a sigmoid attention (times their position's temperature); its convolved keys and
+        (normed) values go to their pages, and the convolution's history advances.  ``state_only``: only that."""
+        A, a, pool, c, T = M.attn, M.attn.spec, kv.kv[layer_idx], M.cols, proj.shape[0]
+        if kv.layout != "tiles" or pool.dtype != proj.dtype:
+            raise CudaError(f"attention of {proj.dtype} rows needs 'tiles' pages of that type")
+        q = None if state_only else torch.empty(T, a.heads * a.dim, dtype=proj.dtype, device=self.device)
+        self._check(self.lib.blz_conv_prep_pages(_ptr(proj), proj.stride(0), c["q"], c["k"], c["v"], _ptr(q), _ptr(pool), pool.stride(0),
+                                                 pool.stride(1), _ptr(batch.positions), _ptr(batch.slot_mapping), _ptr(A.conv_w),
+                                                 _ptr(kv.qkv_state.get(layer_idx)), _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len),
+                                                 _ptr(batch.gdn_defer), batch.slots.numel(), int(batch.max_q_len), T, a.heads, a.kv_heads,
+                                                 a.dim, a.vdim, max(a.conv, 1), int(a.unit_v), a.temp_coef, a.temp_every, eps, int(state_only),
+                                                 int(proj.dtype == torch.float32), self._stream()), "conv_prep_pages")
+        return q
+
+    def sigmoid_attention(self, proj, M, batch, kv, layer_idx, eps, out, state_only: bool = False):
+        """Sigmoid attention of a mixer (convolution, value norm and page write included) into ``out`` (columns of a wider matrix).
+        ``state_only`` advances the convolution's history and does nothing else."""
+        q = self.conv_prep_pages(proj, M, batch, kv, layer_idx, eps, state_only)
+        if not state_only:
+            self.sigmoid_attend(q, M, batch, kv, layer_idx, out)
+
+    def sigmoid_attend(self, q, M, batch, kv, layer_idx, out):
+        A, a, pool, bt = M.attn, M.attn.spec, kv.kv[layer_idx], kv.block_table
+        T, B, f32, st = q.shape[0], batch.slots.numel(), q.dtype == torch.float32, self._stream()
+        plain = f32 or a.dim > 128 or a.vdim > 128 or a.group > 128 or a.scale <= 0
+        common = (_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(pool), pool.stride(0), pool.stride(1), _ptr(bt), bt.stride(0),
+                  _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(A.bias if plain else A.bias_ex2), A.reach)
+        shape = (T, B, a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.scale, a.out_scale)
+        if plain:
+            self._check(self.lib.blz_sigmoid_plain(*common, _ptr(batch.seq_of_row), *shape, int(f32), st), "sigmoid_plain")
+            return
+        items, small = self._split_rows(batch, a)
+        if items:
+            self._check(self.lib.blz_sigmoid_tc(*common, *shape, self.SHORT_ROWS, items, st), "sigmoid_tc")
+        if small:
+            self._check(self.lib.blz_sigmoid_short(*common, *shape, self.SHORT_ROWS, *small, st), "sigmoid_short")
 
     # ------------------------------------------------------------------ feed-forwards without a gate
     def relu2_(self, z, row_list=None):
@@ -1188,14 +1284,16 @@ class CudaOps:
         return (out, vals) if want_values else out
 
     # ------------------------------------------------------------------ mixture of experts
-    def router_topk(self, logits, k, renorm=True, first: int = 0, local_n: int = -1):
-        """Softmax → top-k → renormalise on the device; also counts the routed rows of each local expert."""
-        T, E = logits.shape
+    def router_topk(self, logits, k, renorm=True, first: int = 0, local_n: int = -1, sigmoid: bool = False, n_exp: Optional[int] = None):
+        """Softmax (or sigmoids) → top-k → renormalise on the device; also counts the routed rows of each local expert.  ``n_exp``: the
+        experts' logits are the first ``n_exp`` columns."""
+        T, E = logits.shape[0], logits.shape[1] if n_exp is None else n_exp
+        logits = logits if logits.stride(1) == 1 else logits.contiguous()
         local_n = E if local_n < 0 else local_n
         w = torch.empty(T, k, dtype=torch.float32, device=self.device)
         ids = torch.empty(T, k, dtype=torch.int32, device=self.device)
         counts = torch.empty(max(local_n, 1), dtype=torch.int32, device=self.device)
-        self._check(self.lib.blz_moe_route(_ptr(logits.contiguous()), _ptr(w), _ptr(ids), _ptr(counts), T, E, k, int(renorm),
+        self._check(self.lib.blz_moe_route(_ptr(logits), logits.stride(0), _ptr(w), _ptr(ids), _ptr(counts), T, E, k, int(renorm), int(sigmoid),
                                            first, local_n, self._stream()), "moe_route")
         self._route_counts = (counts, first, local_n)
         return w, ids
@@ -1205,8 +1303,8 @@ class CudaOps:
         if ex.cuda_pack is not None:
             return ex.cuda_pack
 
-        relu2 = ex.act == "relu2"
-        if relu2 and (ex.gate_up[0].w.dtype == torch.float32 or ex.gate_up[0].K % 16):
+        relu2, fused = ex.act == "relu2", ex.act == "swiglu" and ex.fused_act
+        if (relu2 or fused) and (ex.gate_up[0].w.dtype == torch.float32 or ex.gate_up[0].K % 16):
             # 32-bit, or rows too ragged for TMA: the CUDA-core product
             def plain(lins):
                 w = torch.stack([l.w for l in lins]).to(self.device).contiguous()
@@ -1250,6 +1348,21 @@ class CudaOps:
                 l.cuda_pack = None          # the stacked copy replaces the per-expert ones
             return {"kind": kind, "w": w.contiguous(), "sf": sf, "alpha": alpha, "N": lins[0].N, "K": lins[0].K,
                     "fmt": lins[0].fmt, "act_quant": lins[0].act_quant}
+        if fused:
+            # [gate | up] rows, each half rounded up to 64 features, in the order of the SwiGLU epilogue
+            ff, K = ex.down[0].K, ex.gate_up[0].K
+            fp = (ff + 63) // 64 * 64
+            ws = []
+            for l in ex.gate_up:
+                w = l.w.new_zeros(2 * fp, K)
+                w[:ff], w[fp:fp + ff] = l.w[:ff], l.w[ff:]
+                ws.append(w[self.swiglu_order(2 * fp).to(w.device)])
+            downs = [l.w.new_zeros((l.N + 127) // 128 * 128, fp) for l in ex.down]
+            for w, l in zip(downs, ex.down):
+                w[:l.N, :ff] = l.w
+            ex.cuda_pack = {n: {"kind": 0, "w": torch.cat(w).to(self.device, torch.bfloat16).contiguous(), "sf": None, "alpha": None, "N": w[0].shape[0],
+                                "K": w[0].shape[1], "fmt": Format.DENSE, "act_quant": False} for n, w in (("gate_up", ws), ("down", downs))}
+            return ex.cuda_pack
         up, down = (padded(ex.gate_up, True, False), padded(ex.down, True, True)) if relu2 else (ex.gate_up, ex.down)
         ex.cuda_pack = {"gate_up": stack(up), "down": stack(down)}
         return ex.cuda_pack
@@ -1278,8 +1391,9 @@ class CudaOps:
                     "moe_combine")
         return out
 
-    def moe_rows(self, x, topk_w, topk_id, experts, shared=None) -> RoutedRows:
-        """The routed experts' outputs as rows (:meth:`branch_norm` sums them up, with ``shared`` added)."""
+    def moe_rows(self, x, topk_w, topk_id, experts, shared=None, gate=None) -> RoutedRows:
+        """The routed experts' outputs as rows (:meth:`branch_norm` and :meth:`branch_step` sum them up, with ``shared`` added, there times
+        the sigmoid of the logits ``gate``)."""
         pk = self.pack_experts(experts)
         gu, dn = pk["gate_up"], pk["down"]
         T, H = x.shape
@@ -1310,13 +1424,33 @@ class CudaOps:
             a = self._alloc_qact(Format.NVFP4 if mode == 1 else Format.MXFP8, M_pad, H)
             self._check(self.lib.blz_moe_scatter(mode, _ptr(xq.data), _ptr(xq.sf), _ptr(xq.row_scale), _ptr(a.data), _ptr(a.sf),
                                                  _ptr(a.row_scale), _ptr(topk_id), _ptr(offsets), _ptr(fill), _ptr(row_map), T, H, k,
-                                                 first, n_exp, self._stream()), "moe_scatter")
+                                                 first, n_exp, VP(0), 0, self._stream()), "moe_scatter")
         else:
             a = torch.empty(M_pad, H, dtype=x.dtype, device=dev)
             self._check(self.lib.blz_moe_scatter(0, _ptr(x.contiguous()), VP(0), VP(0), _ptr(a), VP(0), VP(0), _ptr(topk_id),
                                                  _ptr(offsets), _ptr(fill), _ptr(row_map), T, H * x.element_size() // 2, k, first, n_exp,
+                                                 _ptr(topk_w if experts.weigh_input else None), int(x.dtype == torch.float32),
                                                  self._stream()), "moe_scatter")
         self._route_counts = None
+        weights = None if experts.weigh_input else topk_w.contiguous()
+        if experts.act == "swiglu" and experts.fused_act:
+            y = torch.empty(M_pad, dn["N"], dtype=x.dtype, device=dev)
+            if gu["kind"] == 5:
+                g = torch.empty(M_pad, gu["N"], dtype=x.dtype, device=dev)
+                simple = (_ptr(tile_expert), _ptr(tile_rows), int(x.dtype == torch.float32), self._stream())
+                self._check(self.lib.blz_gemm_simple_experts(_ptr(a), a.stride(0), _ptr(gu["w"]), _ptr(g), g.stride(0), max_tiles, gu["N"],
+                                                             gu["K"], *simple), "gemm_simple_experts")
+                g = self._glu(g, -1.0)
+                self._check(self.lib.blz_gemm_simple_experts(_ptr(g), g.stride(0), _ptr(dn["w"]), _ptr(y), y.stride(0), max_tiles, dn["N"],
+                                                             dn["K"], *simple), "gemm_simple_experts")
+            else:
+                g = torch.empty(M_pad, gu["N"] // 2, dtype=x.dtype, device=dev)
+                for w, src, dst in ((gu, a, g), (dn, g, y)):
+                    if narrow:
+                        self._moe_gemm(w, src, max_tiles, tile_expert, tile_rows, n_exp, dst, act=int(dst is g))
+                    else:
+                        self._grouped_gemm(w, src, M_pad, tile_expert, n_exp, dst, act=int(dst is g))
+            return RoutedRows(y, row_map, weights, shared, gate)
         g = torch.empty(M_pad, gu["N"], dtype=x.dtype, device=dev)
         if experts.act == "relu2":
             y = torch.empty(M_pad, dn["N"], dtype=x.dtype, device=dev)
@@ -1331,7 +1465,7 @@ class CudaOps:
                     self._moe_gemm(w, src, max_tiles, tile_expert, tile_rows, n_exp, dst, act=3 if dst is g else 0)
                 else:
                     self._grouped_gemm(w, src, M_pad, tile_expert, n_exp, dst, act=3 if dst is g else 0)
-            return RoutedRows(y, row_map, topk_w.contiguous(), shared)
+            return RoutedRows(y, row_map, weights, shared, gate)
         proxy_d = Linear(dn["fmt"], dn["N"], dn["K"])
         proxy_d.act_quant = dn["act_quant"]
         y = torch.empty(M_pad, dn["N"], dtype=torch.bfloat16, device=dev)
@@ -1344,7 +1478,7 @@ class CudaOps:
             # only the routed rows: the padded row space is up to (1 + experts * 128 / routed rows) times larger
             act = self._silu_mul_live(g, proxy_d if dn["kind"] in (1, 2) else None, row_map)
             self._grouped_gemm(dn, act, M_pad, tile_expert, n_exp, y)
-        return RoutedRows(y, row_map, topk_w.contiguous(), shared)
+        return RoutedRows(y, row_map, weights, shared, gate)
 
     def _moe_gemm(self, pk, a, row_tiles, tile_expert, tile_rows, n_exp, out, act: int = 0):
         """Expert GEMM over the padded row space with the features on the MMA lanes and only each tile's live rows on its columns."""

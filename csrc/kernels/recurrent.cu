@@ -1,7 +1,8 @@
 // Recurrent mixers with an fp32 state per sequence and head, token by token, for decode rows and prompt runs alike:
 //   delta rule with a decay per key channel:  S <- g * S (rows);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
-//       g = exp(-A softplus(a + dt_bias)), beta = sigmoid(b), q and k made unit vectors, q times dim^-1/2
+//       g = exp(-A softplus(a + dt_bias)), beta = sigmoid(b), q and k made unit vectors, q times dim^-1/2; or one decay per head
 //   state-space duality:  S <- exp(-A dt) S + dt B x^T;  y = S^T C + D x,  dt = softplus(dt_raw + dt_bias)
+//   minGRU, element by element:  S <- (1 - z) S + z c;  o = S silu(g),  z = sigmoid(z_raw), c = u + 1/2 (u >= 0) or sigmoid(u)
 //   gated linear (HGRN2): S <- f * S + (1 - f) v^T (f acts on rows);  o = S^T silu(q),  f = lo + (1 - lo) sigmoid(f_raw + bias)
 //       (rows beyond dk have f = 0 and q = 0)
 // and the norm over groups of columns with a gate before or after it that follows either of them.
@@ -24,11 +25,11 @@ static constexpr int kRecWarps = 4;          // warps that hold state
 
 struct RecParams {
   const void* conv;            // [T, ld_conv] convolved inputs: delta q | k | v, state space x | B | C; gated linear: v
-  const void* a;               // delta: decay inputs [T, ld_a], heads * dk columns; state space: dt_raw [T, ld_a], heads columns;
+  const void* a;               // delta: decay inputs [T, ld_a], heads * dk columns (one decay per head: heads columns); state space: dt_raw [T, ld_a], heads columns;
                                // gated linear: f_raw, heads * dk columns
   const void* b;               // delta: beta inputs [T, ld_b], heads columns; gated linear: q before its activation, heads * dk columns
   const float* A;              // [heads], positive; gated linear: lower bounds [heads * dk]
-  const float* dt_bias;        // delta and gated linear [heads * dk], state space [heads]
+  const float* dt_bias;        // delta and gated linear [heads * dk], state space and delta with one decay per head [heads]
   const float* D;              // [heads] or null
   float* state;
   float* out;                  // [T, heads * dv] or null (the state only)
@@ -53,8 +54,13 @@ __device__ __forceinline__ float rc_softplus(float x) { return x > 20.f ? x : lo
 template <typename T>
 __device__ __forceinline__ float rc_sigmoid(float x) { return 1.f / (1.f + rc_exp<T>(-x)); }
 
-// the three recurrences; GATED shares the kernels of SSM, which have no reduction between tokens
-enum RecKind { DELTA, SSM, GATED };
+// the recurrences; GATED shares the kernels of SSM, which have no reduction between tokens, HDELTA (one decay per head) those of DELTA
+enum RecKind { DELTA, SSM, GATED, HDELTA };
+// the decay of a head (HDELTA)
+template <typename T>
+__device__ __forceinline__ float head_decay(const RecParams& p, size_t row, int h) {
+  return rc_exp<T>(-p.A[h] * rc_softplus<T>(rc_ld(reinterpret_cast<const T*>(p.a) + row * p.ld_a + h) + p.dt_bias[h]));
+}
 template <typename T>
 __device__ __forceinline__ float rc_silu(float x) { return x * rc_sigmoid<T>(x); }
 template <typename T>
@@ -124,10 +130,10 @@ __device__ __forceinline__ void store_cols(float* o, const float (&y)[VPT], int 
 }
 
 // grid (B * slices, heads), 128 threads
-template <typename T, int R, int VPT>
+template <typename T, int R, int VPT, bool HD>
 __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_rule_kernel(RecParams p, int slices) {
-  constexpr int DKP = R * 8, COLS = kRecWarps * 4 * VPT, TOK = 3 * DKP + COLS + 4, NV = DKP / 32;
-  extern __shared__ float sm[];              // [2][kRecTok][q | k | g | v | beta | k . q]; a token is a multiple of 16 bytes
+  constexpr int DKP = R * 8, COLS = kRecWarps * 4 * VPT, V0 = (HD ? 2 : 3) * DKP, TOK = V0 + COLS + 4, NV = DKP / 32;
+  extern __shared__ float sm[];              // [2][kRecTok][q | k | (g) | v | beta | k . q | (g)]; a token is a multiple of 16 bytes
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane & 7;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
@@ -145,7 +151,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_r
       const size_t row = (size_t)(r0 + t0 + j);
       float* s = buf + j * TOK;
       const T* cv = reinterpret_cast<const T*>(p.conv) + row * p.ld_conv;
-      const T* av = reinterpret_cast<const T*>(p.a) + row * p.ld_a + (size_t)h * dk;
+      const T* av = reinterpret_cast<const T*>(p.a) + row * p.ld_a + (size_t)(HD ? 0 : h) * dk;
       float q[NV], k[NV], qq = 0.f, kk = 0.f, kq = 0.f;
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
@@ -163,15 +169,16 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_r
         const int d = lane + i * 32;
         s[d] = q[i] * qn;
         s[DKP + d] = k[i] * kn;
-        s[2 * DKP + d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d])) : 1.f;
+        if constexpr (!HD) s[2 * DKP + d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d])) : 1.f;
       }
       for (int c = lane; c < COLS; c += 32) {
         const int e = slice * COLS + c;
-        s[3 * DKP + c] = e < dv ? rc_ld(cv + (size_t)2 * p.groups * dk + (size_t)h * dv + e) : 0.f;
+        s[V0 + c] = e < dv ? rc_ld(cv + (size_t)2 * p.groups * dk + (size_t)h * dv + e) : 0.f;
       }
       if (lane == 0) {
-        s[3 * DKP + COLS] = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + row * p.ld_b + h));
-        s[3 * DKP + COLS + 1] = kq;
+        s[V0 + COLS] = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + row * p.ld_b + h));
+        s[V0 + COLS + 1] = kq;
+        if constexpr (HD) s[V0 + COLS + 2] = head_decay<T>(p, row, h);
       }
     }
   };
@@ -185,6 +192,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_r
       const int m = min(kRecTok, n - t0);
       for (int j = 0; j < m; ++j) {
         const float* s = buf + j * TOK;
+        const float gh = HD ? s[V0 + COLS + 2] : 0.f;
         float part[VPT], po[VPT], kr[R <= 16 ? R : 1];
 #pragma unroll
         for (int v = 0; v < VPT; ++v) part[v] = po[v] = 0.f;
@@ -192,7 +200,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_r
         for (int i4 = 0; i4 < R / 4; ++i4) {
           const float4 q4 = *reinterpret_cast<const float4*>(s + kl * 4 + 32 * i4);
           const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 32 * i4);
-          const float4 g4 = *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 32 * i4);
+          const float4 g4 = HD ? make_float4(gh, gh, gh, gh) : *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 32 * i4);
           const float qa[4] = {q4.x, q4.y, q4.z, q4.w}, ka[4] = {k4.x, k4.y, k4.z, k4.w}, ga[4] = {g4.x, g4.y, g4.z, g4.w};
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
@@ -210,10 +218,10 @@ __global__ void __launch_bounds__(kRecWarps * 32, R * VPT <= 64 ? 4 : 2) delta_r
         for (int o = 4; o > 0; o >>= 1)
 #pragma unroll
           for (int v = 0; v < VPT; ++v) part[v] += __shfl_xor_sync(0xffffffffu, part[v], o);
-        const float beta = s[3 * DKP + COLS], kq = s[3 * DKP + COLS + 1];
+        const float beta = s[V0 + COLS], kq = s[V0 + COLS + 1];
         float u[VPT];
 #pragma unroll
-        for (int v = 0; v < VPT; ++v) u[v] = beta * (s[3 * DKP + lc + v] - part[v]);
+        for (int v = 0; v < VPT; ++v) u[v] = beta * (s[V0 + lc + v] - part[v]);
 #pragma unroll
         for (int i4 = 0; i4 < R / 4; ++i4) {
           float ka[4];
@@ -397,7 +405,7 @@ __device__ __forceinline__ float lanes_sum(float x) {
   return x;
 }
 
-template <typename T, int KL, int R, int VPT>
+template <typename T, int KL, int R, int VPT, bool HD>
 __global__ void __launch_bounds__(kRecWarps * 32, 3) delta_step_kernel(RecParams p, int slices, int vec_t) {
   constexpr int CG = 32 / KL;
   __shared__ __align__(16) float s_g[KL * R];
@@ -420,8 +428,9 @@ __global__ void __launch_bounds__(kRecWarps * 32, 3) delta_step_kernel(RecParams
   for (int c = 0; c < VPT; ++c) v[c] = col + c < dv ? rc_ld(cv + (size_t)2 * p.groups * dk + (size_t)h * dv + col + c) : 0.f;
   const float beta = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + (size_t)r0 * p.ld_b + h)), A = p.A[h];
   // the decays, one per thread
-  const T* av = reinterpret_cast<const T*>(p.a) + (size_t)r0 * p.ld_a + (size_t)h * dk;
-  for (int d = threadIdx.x; d < KL * R; d += kRecWarps * 32)
+  const T* av = reinterpret_cast<const T*>(p.a) + (size_t)r0 * p.ld_a + (size_t)(HD ? 0 : h) * dk;
+  const float gh = HD ? head_decay<T>(p, r0, h) : 0.f;
+  for (int d = threadIdx.x; !HD && d < KL * R; d += kRecWarps * 32)
     s_g[d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d])) : 1.f;
   float qq = 0.f, kk = 0.f, kq = 0.f;
 #pragma unroll
@@ -432,9 +441,9 @@ __global__ void __launch_bounds__(kRecWarps * 32, 3) delta_step_kernel(RecParams
   }
   const float qn = rsqrtf((float)dk) / sqrtf(lanes_sum<KL>(qq) + 1e-6f), kn = 1.f / sqrtf(lanes_sum<KL>(kk) + 1e-6f);
   kq = lanes_sum<KL>(kq) * qn * kn;
-  __syncthreads();
+  if constexpr (!HD) __syncthreads();
 #pragma unroll
-  for (int i4 = 0; i4 < R / 4; ++i4) *reinterpret_cast<float4*>(&g[i4 * 4]) = *reinterpret_cast<const float4*>(s_g + kl * 4 + 4 * KL * i4);
+  for (int i4 = 0; i4 < R / 4 && !HD; ++i4) *reinterpret_cast<float4*>(&g[i4 * 4]) = *reinterpret_cast<const float4*>(s_g + kl * 4 + 4 * KL * i4);
   float part[VPT], po[VPT];
 #pragma unroll
   for (int c = 0; c < VPT; ++c) part[c] = po[c] = 0.f;
@@ -442,7 +451,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, 3) delta_step_kernel(RecParams
   for (int i = 0; i < R; ++i)
 #pragma unroll
     for (int c = 0; c < VPT; ++c) {
-      S[i][c] *= g[i];
+      S[i][c] *= HD ? gh : g[i];
       part[c] = fmaf(S[i][c], k[i], part[c]);
       po[c] = fmaf(S[i][c], q[i], po[c]);
     }
@@ -547,7 +556,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, 4) gated_step_kernel(RecParams
 }
 
 // ------------------------------------------------------------------------------------------ long runs
-// Records: delta [heads][T][q | k | g | beta, k . q, 0, 0], state space [groups][T][B | C] and [heads][T][dt, decay, 0, 0], gated
+// Records: delta [heads][T][q | k | g | beta, k . q, 0, 0], with one decay per head [heads][T][q | k | beta, k . q, g, 0], state space [groups][T][B | C] and [heads][T][dt, decay, 0, 0], gated
 // linear [heads][T][f | q]; vectors padded to 32, 64, 128, 256 or 512 floats.
 __device__ __forceinline__ bool in_long_run(const RecParams& p, int t) {
   const int b = p.seq_of_row[t];
@@ -555,22 +564,22 @@ __device__ __forceinline__ bool in_long_run(const RecParams& p, int t) {
 }
 
 // a warp per (row, head)
-template <typename T, int DKP>
+template <typename T, int DKP, bool HD>
 __global__ void __launch_bounds__(128) delta_records_kernel(RecParams p) {
-  constexpr int REC = 3 * DKP + 4, NV = DKP / 32;
+  constexpr int B0 = (HD ? 2 : 3) * DKP, REC = B0 + 4, NV = DKP / 32;
   const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
   const int t = (int)(w / p.heads), h = (int)(w % p.heads), lane = threadIdx.x & 31;
   if (t >= p.T || !in_long_run(p, t)) return;
   const int dk = p.dk, hk = h / (p.heads / p.groups);
   const T* cv = reinterpret_cast<const T*>(p.conv) + (size_t)t * p.ld_conv;
-  const T* av = reinterpret_cast<const T*>(p.a) + (size_t)t * p.ld_a + (size_t)h * dk;
+  const T* av = reinterpret_cast<const T*>(p.a) + (size_t)t * p.ld_a + (size_t)(HD ? 0 : h) * dk;
   float q[NV], k[NV], a[NV], qq = 0.f, kk = 0.f, kq = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int d = lane + i * 32;
     q[i] = d < dk ? rc_ld(cv + (size_t)hk * dk + d) : 0.f;
     k[i] = d < dk ? rc_ld(cv + (size_t)(p.groups + hk) * dk + d) : 0.f;
-    a[i] = d < dk ? rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d] : 0.f;
+    a[i] = !HD && d < dk ? rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d] : 0.f;
   }
   const float beta = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + (size_t)t * p.ld_b + h)), A = p.A[h];
 #pragma unroll
@@ -587,9 +596,9 @@ __global__ void __launch_bounds__(128) delta_records_kernel(RecParams p) {
     const int d = lane + i * 32;
     s[d] = q[i] * qn;
     s[DKP + d] = k[i] * kn;
-    s[2 * DKP + d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(a[i])) : 1.f;
+    if constexpr (!HD) s[2 * DKP + d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(a[i])) : 1.f;
   }
-  if (lane == 0) *reinterpret_cast<float4*>(s + 3 * DKP) = make_float4(beta, kq, 0.f, 0.f);
+  if (lane == 0) *reinterpret_cast<float4*>(s + B0) = make_float4(beta, kq, HD ? head_decay<T>(p, t, h) : 0.f, 0.f);
 }
 
 // a block per row
@@ -690,9 +699,9 @@ __device__ __forceinline__ void wait_cols() { asm volatile("cp.async.wait_group 
 
 static constexpr int kRecHead = 128;         // barriers in front of the ring
 
-template <typename T, int KL, int R, int VPT>
+template <typename T, int KL, int R, int VPT, bool HD>
 __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) delta_stream_kernel(RecParams p, int slices, int vec_v) {
-  constexpr int DKP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, REC = 3 * DKP + 4, STAGE = kRecTok * REC;
+  constexpr int DKP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, B0 = (HD ? 2 : 3) * DKP, REC = B0 + 4, STAGE = kRecTok * REC;
   constexpr int PART = VPT == 2 ? 2 : 1;            // independent chains per sum
   extern __shared__ __align__(128) uint8_t sm8[];
   __shared__ __align__(16) T s_v[kRecWarps][kColsAhead + 1][kRecTok][CG * VPT];
@@ -741,7 +750,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
     float y[VPT <= 2 ? kRecTok : 1][VPT];
     // what a token brings: the lane's rows of q, k and g, its v, beta and k . q
     struct Tok {
-      float q[R], k[R], g[R], v[VPT];
+      float q[R], k[R], g[HD ? 1 : R], v[VPT];
       float2 bk;
     };
     auto fetch = [&](int j, Tok& o) {
@@ -750,12 +759,15 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
       for (int i4 = 0; i4 < R / 4; ++i4) {
         const float4 q4 = *reinterpret_cast<const float4*>(s + kl * 4 + 4 * KL * i4);
         const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 4 * KL * i4);
-        const float4 g4 = *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 4 * KL * i4);
         o.q[i4 * 4] = q4.x; o.q[i4 * 4 + 1] = q4.y; o.q[i4 * 4 + 2] = q4.z; o.q[i4 * 4 + 3] = q4.w;
         o.k[i4 * 4] = k4.x; o.k[i4 * 4 + 1] = k4.y; o.k[i4 * 4 + 2] = k4.z; o.k[i4 * 4 + 3] = k4.w;
-        o.g[i4 * 4] = g4.x; o.g[i4 * 4 + 1] = g4.y; o.g[i4 * 4 + 2] = g4.z; o.g[i4 * 4 + 3] = g4.w;
+        if constexpr (!HD) {
+          const float4 g4 = *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 4 * KL * i4);
+          o.g[i4 * 4] = g4.x; o.g[i4 * 4 + 1] = g4.y; o.g[i4 * 4 + 2] = g4.z; o.g[i4 * 4 + 3] = g4.w;
+        }
       }
-      o.bk = *reinterpret_cast<const float2*>(s + 3 * DKP);
+      o.bk = *reinterpret_cast<const float2*>(s + B0);
+      if constexpr (HD) o.g[0] = s[B0 + 2];
 #pragma unroll
       for (int v = 0; v < VPT; ++v) o.v[v] = rc_ld(&cols[j][cg * VPT + v]);
     };
@@ -769,7 +781,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
       for (int i = 0; i < R; ++i)
 #pragma unroll
         for (int v = 0; v < VPT; ++v) {
-          S[i][v] *= x.g[i];
+          S[i][v] *= x.g[HD ? 0 : i];
           part[v][i % PART] = fmaf(S[i][v], x.k[i], part[v][i % PART]);
           pq[v][i % PART] = fmaf(S[i][v], x.q[i], pq[v][i % PART]);
         }
@@ -1061,17 +1073,172 @@ __global__ void __launch_bounds__(256) group_norm_kernel(GroupNormParams p) {
   }
 }
 
+// ------------------------------------------------------------------------------------------ minGRU
+struct GruParams {
+  const void *z, *u, *g;       // [T, ld] before their activations
+  float* state;                // [rows, width]
+  void* out;                   // [T, ld_out] or null (the state only)
+  const int *slots, *q_start, *ctx_len, *no_store;
+  long long ld, ld_out;
+  int width;
+};
+static constexpr int kGruWarps = 16, kGruTok = 8;      // a block takes kGruWarps * kGruTok tokens at a time
+
+template <typename T>
+__device__ __forceinline__ void gru_gate(float z, float u, float& keep, float& add) {
+  const float s = rc_sigmoid<T>(z);
+  keep = 1.f - s;
+  add = s * (u >= 0.f ? u + 0.5f : rc_sigmoid<T>(u));
+}
+template <typename T, int VEC> struct alignas(sizeof(T) * VEC) GruVec { T e[VEC]; };
+template <typename T, int VEC>
+__device__ __forceinline__ GruVec<T, VEC> gru_load(const void* base, size_t at) {
+  GruVec<T, VEC> v;
+  const T* p = reinterpret_cast<const T*>(base) + at;
+  if constexpr (sizeof(T) * VEC == 16) *reinterpret_cast<uint4*>(v.e) = *reinterpret_cast<const uint4*>(p);
+  else if constexpr (sizeof(T) * VEC == 8) *reinterpret_cast<uint2*>(v.e) = *reinterpret_cast<const uint2*>(p);
+  else if constexpr (sizeof(T) * VEC == 4) *reinterpret_cast<uint32_t*>(v.e) = *reinterpret_cast<const uint32_t*>(p);
+  else v.e[0] = *p;
+  return v;
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void gru_store(const GruParams& p, size_t row, int c, const GruVec<T, VEC>& g, const float (&S)[VEC]) {
+  T* o = reinterpret_cast<T*>(p.out) + row * p.ld_out + c;
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) {
+    const float y = S[j] * rc_silu<T>(rc_ld(g.e + j));
+    if constexpr (sizeof(T) == 4) o[j] = y;
+    else o[j] = __float2bfloat16(y);
+  }
+}
+
+// single tokens: a thread per VEC elements of a sequence
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) min_gru_step_kernel(GruParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.y, c = (blockIdx.x * 128 + threadIdx.x) * VEC;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
+  if (n != 1 || c >= p.width) return;
+  const size_t at = (size_t)r0 * p.ld + c;
+  const auto z = gru_load<T, VEC>(p.z, at), u = gru_load<T, VEC>(p.u, at);
+  float* st = p.state + (size_t)p.slots[b] * p.width + c;
+  const bool fresh = p.ctx_len[b] == 1;
+  float S[VEC];
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) {
+    float keep, add;
+    gru_gate<T>(rc_ld(z.e + j), rc_ld(u.e + j), keep, add);
+    S[j] = fresh ? add : fmaf(keep, st[j], add);
+  }
+  if (p.out) gru_store<T, VEC>(p, r0, c, gru_load<T, VEC>(p.g, at), S);
+  if (p.no_store != nullptr && p.no_store[b]) return;
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) st[j] = S[j];
+}
+
+// longer runs: a block per 32 * VEC elements of a sequence.  Each warp folds kGruTok tokens into one pair (factor, addend) per element;
+// the pairs of the warps before it and the carry give the state its own tokens start from.  The next tokens are fetched meanwhile.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kGruWarps * 32) min_gru_kernel(GruParams p) {
+  __shared__ float s_a[2][kGruWarps][32 * VEC], s_b[2][kGruWarps][32 * VEC], s_c[2][32 * VEC];
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, c = (blockIdx.x * 32 + lane) * VEC;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
+  if (n <= 1) return;
+  const bool live = c < p.width;
+  float* st = p.state + (size_t)p.slots[b] * p.width + c;
+  const bool fresh = p.ctx_len[b] == n;
+  float S[VEC];
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) S[j] = !fresh && live ? st[j] : 0.f;
+  if (warp == 0)
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) s_c[0][lane * VEC + j] = S[j];
+  GruVec<T, VEC> z[kGruTok], u[kGruTok], g[kGruTok];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int k = 0; k < kGruTok; ++k)
+      if (live && t0 + k < n) {
+        const size_t at = (size_t)(r0 + t0 + k) * p.ld + c;
+        z[k] = gru_load<T, VEC>(p.z, at);
+        u[k] = gru_load<T, VEC>(p.u, at);
+        if (p.out) g[k] = gru_load<T, VEC>(p.g, at);
+      }
+  };
+  constexpr int STEP = kGruWarps * kGruTok;
+  fetch(warp * kGruTok);
+  for (int i = 0, base = 0; base < n; ++i, base += STEP) {
+    const int t0 = base + warp * kGruTok, par = i & 1;
+    float keep[kGruTok][VEC], add[kGruTok][VEC], A[VEC], B[VEC];
+    GruVec<T, VEC> gate[kGruTok];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) { A[j] = 1.f; B[j] = 0.f; }
+#pragma unroll
+    for (int k = 0; k < kGruTok; ++k) {
+      gate[k] = g[k];
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        keep[k][j] = 1.f;
+        add[k][j] = 0.f;
+        if (live && t0 + k < n) gru_gate<T>(rc_ld(z[k].e + j), rc_ld(u[k].e + j), keep[k][j], add[k][j]);
+        A[j] *= keep[k][j];
+        B[j] = fmaf(keep[k][j], B[j], add[k][j]);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) { s_a[par][warp][lane * VEC + j] = A[j]; s_b[par][warp][lane * VEC + j] = B[j]; }
+    fetch(t0 + STEP);
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) S[j] = s_c[par][lane * VEC + j];
+    for (int w = 0; w < warp; ++w)
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) S[j] = fmaf(s_a[par][w][lane * VEC + j], S[j], s_b[par][w][lane * VEC + j]);
+#pragma unroll
+    for (int k = 0; k < kGruTok; ++k) {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) S[j] = fmaf(keep[k][j], S[j], add[k][j]);
+      if (p.out && live && t0 + k < n) gru_store<T, VEC>(p, r0 + t0 + k, c, gate[k], S);
+    }
+    if (warp == kGruWarps - 1)
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) s_c[par ^ 1][lane * VEC + j] = S[j];
+  }
+  if (warp != kGruWarps - 1 || !live || (p.no_store != nullptr && p.no_store[b])) return;
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) st[j] = S[j];          // tokens beyond the run changed nothing
+}
+
+template <typename T>
+static int run_gru(const GruParams& p, int B, int kinds, int vec, cudaStream_t s) {
+  cudaError_t e = cudaSuccess;
+  if (kinds & 1) {
+    constexpr int V = 4;
+    if (vec) e = launch_pdl(min_gru_step_kernel<T, V>, dim3((p.width + 128 * V - 1) / (128 * V), B), dim3(128), 0, s, p);
+    else e = launch_pdl(min_gru_step_kernel<T, 1>, dim3((p.width + 127) / 128, B), dim3(128), 0, s, p);
+  }
+  if (e == cudaSuccess && (kinds & 2)) {
+    // two elements per lane where that still gives every SM a block
+    if (vec && (long long)B * ((p.width + 63) / 64) >= sm_count())
+      e = launch_pdl(min_gru_kernel<T, 2>, dim3((p.width + 63) / 64, B), dim3(kGruWarps * 32), 0, s, p);
+    else e = launch_pdl(min_gru_kernel<T, 1>, dim3((p.width + 31) / 32, B), dim3(kGruWarps * 32), 0, s, p);
+  }
+  return (int)e;
+}
+
 // bf16: 4 neighbouring elements of the token's vectors can be read as one 64-bit word
 static int words_of_four(const RecParams& p, RecKind kind) {
   auto ok = [](const void* q, long long ld) { return (reinterpret_cast<uintptr_t>(q) & 7) == 0 && ld % 4 == 0; };
-  return ok(p.conv, p.ld_conv) && (kind == GATED || p.dk % 4 == 0) && p.dv % 4 == 0 && (kind != DELTA || ok(p.a, p.ld_a));
+  return ok(p.conv, p.ld_conv) && (kind == GATED || p.dk % 4 == 0) && p.dv % 4 == 0 && (kind != DELTA || ok(p.a, p.ld_a));      // HDELTA's are read one by one
 }
 
 template <typename T, int DKP, RecKind K>
 static int launch_steps(const RecParams& p, int B, cudaStream_t s) {
   constexpr int KL = DKP <= 128 ? 8 : DKP / 16, R = DKP / KL, COLS = kRecWarps * (32 / KL) * 4;
   const int slices = (p.dv + COLS - 1) / COLS;
-  auto kern = delta_step_kernel<T, KL, R, 4>;
+  auto kern = delta_step_kernel<T, KL, R, 4, K == HDELTA>;
   if constexpr (K == SSM) kern = state_space_step_kernel<T, KL, R, 4>;
   if constexpr (K == GATED) kern = gated_step_kernel<T, KL, R, 4>;
   kern<<<dim3(B * slices, p.heads), kRecWarps * 32, 0, s>>>(p, slices, words_of_four(p, K));
@@ -1083,7 +1250,7 @@ static int launch_short_runs(const RecParams& p, int B, cudaStream_t s) {
   const int slices = (p.dv + COLS - 1) / COLS;
   const size_t smem = (size_t)2 * kRecTok * ((K == DELTA ? 3 : 2) * DKP + COLS + 4) * 4;
   void (*kern)(RecParams, int);
-  if constexpr (K == DELTA) kern = delta_rule_kernel<T, R, VPT>;
+  if constexpr (K == DELTA || K == HDELTA) kern = delta_rule_kernel<T, R, VPT, K == HDELTA>;
   else kern = state_space_kernel<T, R, VPT, K == GATED>;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(kern, 200 * 1024);
@@ -1097,7 +1264,7 @@ static int launch_stream(const RecParams& p, int B, cudaStream_t s) {
   const int slices = (p.dv + COLS - 1) / COLS;
   const size_t smem = kRecHead + (size_t)kRecStages * kRecTok * ((K == DELTA ? 3 : 2) * R * KL + (K == GATED ? 0 : 4)) * 4;
   void (*kern)(RecParams, int, int);
-  if constexpr (K == DELTA) kern = delta_stream_kernel<T, KL, R, VPT>;
+  if constexpr (K == DELTA || K == HDELTA) kern = delta_stream_kernel<T, KL, R, VPT, K == HDELTA>;
   else kern = state_space_stream_kernel<T, KL, R, VPT, K == GATED>;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(kern, 220 * 1024);
@@ -1109,7 +1276,7 @@ static int launch_stream(const RecParams& p, int B, cudaStream_t s) {
 template <typename T, int DKP, RecKind K>
 static int launch_long_runs(const RecParams& p, int B, cudaStream_t s) {
   const unsigned warps4 = (unsigned)(((long long)p.T * p.heads + 3) / 4);
-  if constexpr (K == DELTA) delta_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
+  if constexpr (K == DELTA || K == HDELTA) delta_records_kernel<T, DKP, K == HDELTA><<<warps4, 128, 0, s>>>(p);
   else if constexpr (K == GATED) gated_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
   else state_space_records_kernel<T, DKP><<<p.T, 128, 0, s>>>(p);
   const int e = (int)cudaGetLastError();
@@ -1117,7 +1284,7 @@ static int launch_long_runs(const RecParams& p, int B, cudaStream_t s) {
   if constexpr (sizeof(T) == 2 && DKP <= 128)
     if ((long long)B * p.heads * ((p.dv + 15) / 16) >= 4LL * sm_count()) return launch_stream<T, 8, DKP / 8, 4, K>(p, B, s);
   constexpr int KL = DKP >= 64 ? 16 : 8;
-  if constexpr (sizeof(T) == 2 && K != DELTA && DKP <= 128)     // no reduction between tokens: 8 columns already at half the warps
+  if constexpr (sizeof(T) == 2 && K != DELTA && K != HDELTA && DKP <= 128)     // no reduction between tokens: 8 columns already at half the warps
     if ((long long)B * p.heads * ((p.dv + 7) / 8) >= 2LL * sm_count()) return launch_stream<T, KL, DKP / KL, 4, K>(p, B, s);
   return launch_stream<T, KL, DKP / KL, 2, K>(p, B, s);
 }
@@ -1136,7 +1303,7 @@ static int run_width(RecParams p, int B, int kinds, cudaStream_t s) {
 static int padded_dk(int dk) { return dk <= 32 ? 32 : dk <= 64 ? 64 : dk <= 128 ? 128 : dk <= 256 ? 256 : 512; }
 static long long record_bytes(RecKind kind, long long T, int heads, int groups, int dk) {
   const long long n = padded_dk(dk);
-  return 4 * (kind == DELTA ? heads * T * (3 * n + 4) : kind == GATED ? heads * T * 2 * n : groups * T * 2 * n + heads * T * 4);
+  return 4 * (kind == DELTA ? heads * T * (3 * n + 4) : kind == HDELTA ? heads * T * (2 * n + 4) : kind == GATED ? heads * T * 2 * n : groups * T * 2 * n + heads * T * 4);
 }
 
 template <typename T, RecKind K>
@@ -1161,22 +1328,25 @@ static int run_rec(const RecParams& p, int B, int kinds, long long ws_bytes, cud
 // Runs of at least this many new tokens are long runs where the caller gives a workspace.
 static constexpr int kLongRows = 32;
 BLZ_API int blz_rec_long_rows() { return kLongRows; }
-// Workspace bytes of a step of T rows (kind: 0 = blz_state_space, 1 = blz_delta_rule, 2 = blz_gated_linear).
+// Workspace bytes of a step of T rows (kind: 0 = blz_state_space, 1 = blz_delta_rule, 2 = blz_gated_linear, 3 = blz_delta_rule with one
+// decay per head).
 BLZ_API long long blz_rec_ws_bytes(int kind, int T, int heads, int groups, int dk) {
-  return blz::record_bytes(kind == 1 ? blz::DELTA : kind == 2 ? blz::GATED : blz::SSM, T, heads, groups, dk);
+  return blz::record_bytes(kind == 1 ? blz::DELTA : kind == 2 ? blz::GATED : kind == 3 ? blz::HDELTA : blz::SSM, T, heads, groups, dk);
 }
 
 // Delta rule with channel decays over every sequence of the batch (see RecParams; leading dimensions in elements; conv channels
 // [q key_heads * dk | k key_heads * dk | v heads * dv]).  out fp32 [T, heads * dv] or null.  no_store: optional [B], 1 = leave the
 // state as it was.  kinds: the sequences with one new token (bit 0), with up to blz_rec_long_rows (bit 1), with more (bit 2, which
-// needs out and the workspace ws of blz_rec_ws_bytes; without that bit they count as bit 1's).  dk <= 512.
+// needs out and the workspace ws of blz_rec_ws_bytes; without that bit they count as bit 1's).  dk <= 512.  per_head: one decay per head.
 BLZ_API int blz_delta_rule(const void* conv, long long ld_conv, const void* a, long long ld_a, const void* b, long long ld_b, const float* A,
                            const float* dt_bias, float* state, float* out, const int* slots, const int* q_start, const int* ctx_len,
-                           const int* no_store, int B, int heads, int key_heads, int dk, int dv, const int* seq_of_row, int T, int kinds,
-                           float* ws, long long ws_bytes, int f32, cudaStream_t s) {
+                           const int* no_store, int B, int heads, int key_heads, int dk, int dv, int per_head, const int* seq_of_row, int T,
+                           int kinds, float* ws, long long ws_bytes, int f32, cudaStream_t s) {
   using namespace blz;
   const RecParams p = {conv, a, b, A, dt_bias, nullptr, state, out, slots, q_start, ctx_len, no_store, ld_conv, ld_a, ld_b, heads, key_heads,
                        dk, dv, seq_of_row, ws, T, kLongRows, status_word()};
+  if (per_head)
+    return f32 ? run_rec<float, HDELTA>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, HDELTA>(p, B, kinds, ws_bytes, s);
   return f32 ? run_rec<float, DELTA>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, DELTA>(p, B, kinds, ws_bytes, s);
 }
 
@@ -1201,6 +1371,19 @@ BLZ_API int blz_gated_linear(const void* q, long long ld_q, const void* f, long 
   const RecParams p = {v, f, q, lower, bias, nullptr, state, out, slots, q_start, ctx_len, no_store, ld_v, ld_f, ld_q, heads, heads,
                        dk, dv, seq_of_row, ws, T, kLongRows, status_word()};
   return f32 ? run_rec<float, GATED>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, GATED>(p, B, kinds, ws_bytes, s);
+}
+
+// minGRU over every sequence of the batch: gate inputs z, candidates u and output gates g [T, ld] (runs of columns, width each), state
+// [rows][width] fp32; out [T, ld_out] (activation type) or null.  kinds: bit 0 = some sequences have one new token, bit 1 = some have more.
+BLZ_API int blz_min_gru(const void* z, const void* u, const void* g, long long ld, float* state, void* out, long long ld_out, const int* slots,
+                        const int* q_start, const int* ctx_len, const int* no_store, int B, int width, int kinds, int f32, cudaStream_t s) {
+  using namespace blz;
+  if (B == 0) return 0;
+  if (B < 0 || B > 65535 || width < 1 || !z || !u || !g || !state) return (int)cudaErrorInvalidValue;
+  const GruParams p = {z, u, g, state, out, slots, q_start, ctx_len, no_store, ld, ld_out, width};
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(u) | reinterpret_cast<uintptr_t>(g);
+  const int vec = bits % (f32 ? 16 : 8) == 0 && ld % 4 == 0 && width % 4 == 0;
+  return f32 ? run_gru<float>(p, B, kinds, vec, s) : run_gru<__nv_bfloat16>(p, B, kinds, vec, s);
 }
 
 // RMS norm of each of `groups` runs of n columns of fp32 rows, with a gate (GroupNormParams), to the activation type.
