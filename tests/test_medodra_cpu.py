@@ -302,7 +302,7 @@ def test_lost_states_and_far_tokens_show(case, reference):
 
 
 @pytest.mark.parametrize("cfg,rows", [
-    (C.config([C.delta(None, 1, 1, 3, 8, 1), C.delta(C.moe(2, 1, 8, 16), 6, 2, 40, 12, 4)], width=96, loop=(0, 2, 3)), 16),
+    (C.config([C.delta(None, 1, 1, 6, 8, 1), C.delta(C.moe(2, 1, 8, 16), 6, 2, 40, 12, 4)], width=96, loop=(0, 2, 3)), 16),
     (C.config([C.parallel(C.moe(3, 3, 16, 24), 1, 1, 8, 40, 1, 1.3, 9, 0.0, 1, 17), C.parallel(None, 5, 5, 12, 7, 5, 0.7, 30.5, 1.0, 3, 200)], vocab=77, width=101,
               eps=1e-3, loop=(1, 2, 1)), 6),
     (C.config([C.parallel(None, 8, 2, 20, 12, 8, 0.2, 2000, 0.1, 7, 33), C.delta(C.moe(9, 4, 12, 30), 4, 4, 16, 16, 8)], width=81, mult=1.0, scale=1.0, loop=None), 32),
