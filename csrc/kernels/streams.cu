@@ -471,7 +471,8 @@ __global__ void __launch_bounds__(256) embed_positions_kernel(const T* __restric
     const float hi = freq[i], ang = pos * hi, rest = fmaf(pos, hi, -ang) + pos * freq[half + i];
     float s, c;
     sincosf(ang, &s, &c);
-    const float v[2] = {fmaf(rest, c, s), fmaf(-rest, s, c)};
+    const float half_sq = 0.5f * rest * rest;        // the rest grows to hundredths of a radian at the farthest positions
+    const float v[2] = {fmaf(rest, c, fmaf(-half_sq, s, s)), fmaf(-rest, s, fmaf(-half_sq, c, c))};
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int col = 2 * i + j;

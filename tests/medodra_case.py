@@ -61,7 +61,7 @@ def weights(cfg, seed=0, sharp=1.0, rows=16):
             w[f"l{i}.norm{n}"] = rnd(W, std=0.2)
         if f:
             p = f"l{i}.mlp."
-            w[p + "router"], w[p + "shared.sg"] = lin(f["router"]["experts"], W, 1.5), lin(1, W)
+            w[p + "router"], w[p + "shared.sg"] = lin(f["router"]["experts"], W, 5.0), lin(1, W)
             parts = {f"e{e}.": f["expert"]["ff"] for e in range(f["router"]["experts"])}
             for n, ff in {**parts, "shared.": f["shared"]["ff"]}.items():
                 w[p + n + "gate"], w[p + n + "up"], w[p + n + "down"] = lin(ff, W, 1.5), lin(ff, W, 1.5), lin(W, ff)

@@ -36,16 +36,16 @@ def causal_conv(x, w):
     return sum(padded[j:j + T] * w[:, j] for j in range(taps))
 
 
-def position_vectors(T, width, dtype):
+def position_vectors(positions, width, dtype):
     """Sines (even columns) and cosines (odd columns) of position * 10000^(-2 i / width), i counting the pairs of columns."""
-    p = torch.arange(T, dtype=torch.float64)
+    p = positions.to(torch.float64)
     cols = [(torch.sin if c % 2 == 0 else torch.cos)(p * 10000.0 ** (-2.0 * (c // 2) / width)) for c in range(width)]
     return torch.stack(cols, 1).to(dtype)
 
 
 def embedding(tokens, table, scale):
     x = table[torch.as_tensor(tokens)] * scale
-    return x + position_vectors(x.shape[0], x.shape[1], x.dtype)
+    return x + position_vectors(torch.arange(x.shape[0]), x.shape[1], x.dtype)
 
 
 def join_input(x, x0, w):
