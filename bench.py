@@ -92,7 +92,7 @@ def main():
     ap.add_argument("--draft-k", type=int, default=4)
     ap.add_argument("--shared-prefix", type=int, default=0)
     ap.add_argument("--out-tokens", type=int, default=0, help="output tokens per request of the --spec run (0 = 512)")
-    ap.add_argument("--design", default=None, choices=["sevevik", "niletar", "rapisun"],
+    ap.add_argument("--design", default=None, choices=["sevevik", "niletar", "rapisun", "medodra"],
                     help="instead of the headline run: throughput and kernels of a model design beside the closest other model at equal "
                          "size (one GPU; see blaze_b200/benchmarks/design.py)")
     ap.add_argument("--design-sizes", default="2048,4096", help="widths of the --design run")

@@ -2,8 +2,8 @@
 weights, bf16), and every kernel that is the design's own beside the like kernel of the relative, with fractions of the measured
 peaks.  ``bench.py --design <name>`` runs it: Sevevik against the Qwen3 decoder (equal width, heads, projections and
 feed-forward), Niletar against the Qwen3-Next hybrid with a dense feed-forward (Gated DeltaNet layers with a state as large as the
-state-space layers', gated attention layers with heads as the parallel ones'), Rapisun against the Qwen3-Next hybrid with experts (see
-:mod:`blaze_b200.benchmarks.rapisun`); the relatives keep FP8 pages, their only format on a GPU.
+state-space layers', gated attention layers with heads as the parallel ones'), Rapisun and Medodra against the Qwen3-Next hybrid with experts
+(see :mod:`blaze_b200.benchmarks.rapisun` and :mod:`blaze_b200.benchmarks.medodra`); the relatives keep FP8 pages, their only format on a GPU.
 
 Device-timed with CUDA events; kernels in captured graphs over buffers that together exceed L2.
 """
@@ -17,7 +17,7 @@ import torch
 
 from ..config import (DeltaSpec, DiffAttnSpec, GluSpec, LayerSpec, ModelConfig, RopeConfig, RotarySpec, SoftAttnSpec,
                       StateSpaceSpec)
-from . import rapisun
+from . import medodra, rapisun
 from .kernels import peaks
 
 # width, query heads, key/value heads, feed-forward
@@ -25,14 +25,15 @@ SIZES = {"2048": (2048, 16, 8, 6144), "4096": (4096, 32, 8, 12288)}
 WINDOW = 1024
 
 
-RELATIVE = {"sevevik": "qwen3", "niletar": "qwen3-next (dense)", "rapisun": "qwen3-next (moe)"}
+RELATIVE = {"sevevik": "qwen3", "niletar": "qwen3-next (dense)", "rapisun": "qwen3-next (moe)", "medodra": "qwen3-next (moe)"}
+OWN = {"rapisun": rapisun, "medodra": medodra}          # designs whose kernels are timed in a module of their own
 
 
 def configs(design: str, size: str, layers: int, vocab: int) -> Dict[str, ModelConfig]:
     """The design's configuration and its relative's."""
     W, H, G, ff = SIZES[size]
-    if design == "rapisun":
-        return rapisun.configs(W, H, G, ff, WINDOW, layers, vocab)
+    if design in OWN:
+        return OWN[design].configs(W, H, G, ff, WINDOW, layers, vocab)
     if design == "niletar":
         attn = SoftAttnSpec(H, G, 128, 128, 128 ** -0.5, RotarySpec(128, 5.0e5, True, 8.0, 1.0, 4.0, 8192.0), True, True, True, True,
                             out_scale=0.7)
@@ -275,7 +276,7 @@ def kernels(design: str, size: str) -> List[Dict]:
         bound = max(nbytes / pk["hbm_gbs"] / 1e6, flops / pk["bf16_tflops"] / 1e9)
         rows.append({"kernel": name, "model": model, "us": round(ms * 1e3, 2), "roofline_frac": round(bound / ms, 3),
                      "bound": "hbm" if nbytes / pk["hbm_gbs"] / 1e6 >= flops / pk["bf16_tflops"] / 1e9 else "bf16 tensor"})
-    if design == "rapisun":
+    if design in OWN:
         def like_attention(label, B, qlen, ctx, cfg, model):
             calls, write, kvb, flops, rowb = _attention(ops, cfg, B, qlen, ctx, 2 if B == 256 else 8 if qlen == 1 else 4)
             add("attention " + label, model, _graph_ms(calls), kvb + B * qlen * H * 128 * 4.0, flops)
@@ -290,7 +291,7 @@ def kernels(design: str, size: str) -> List[Dict]:
                 add(f"{part} {label}", model, _graph_ms(c), nbytes, flops)
             del calls
             torch.cuda.empty_cache()
-        rapisun.kernels(SIZES[size], WINDOW, add, _graph_ms, like_attention, like_recurrence, ops)
+        OWN[design].kernels(SIZES[size], WINDOW, add, _graph_ms, like_attention, like_recurrence, ops)
         assert ops.take_status() == 0
         return rows
     for name, B, qlen, ctx, copies in (("attention decode 256x1024", 256, 1, 1024, 2), ("attention decode 32x1024", 32, 1, 1024, 8),
@@ -357,7 +358,7 @@ def kernels(design: str, size: str) -> List[Dict]:
 
 def run(design: str, sizes, steps: int, warmup: int, layers: int = 8, vocab: int = 32768, kernels_only: bool = False) -> Dict:
     res: Dict = {"design": design, "beside": f"{RELATIVE[design]} (equal size, bf16 weights, FP8 pages)", "layers": layers, "vocab": vocab,
-                 "window": WINDOW if design != "niletar" else None, "data": "synthetic token ids, random-init weights", "throughput": {}, "kernels": {}}
+                 "window": WINDOW if design in ("sevevik", "rapisun") else None, "data": "synthetic token ids, random-init weights", "throughput": {}, "kernels": {}}
     for size in sizes:
         res["kernels"][size] = kernels(design, size)
         if not kernels_only:

@@ -38,7 +38,7 @@ def _sequences(cfg: ModelConfig, B: int, qlen: int, ctx: int, copies: int):
         perm = torch.randperm(B * per, generator=torch.Generator().manual_seed(0)).tolist()
         for b in range(B):
             kv.set_pages(b, [1 + p for p in perm[b * per:(b + 1) * per]])
-        for t in (*kv.kv.values(), *kv.rec_state.values(), *kv.input_state.values()):
+        for t in (*kv.kv.values(), *kv.rec_state.values(), *kv.conv_state.values(), *kv.qkv_state.values(), *kv.input_state.values()):
             t.normal_()
         _ = kv.block_table
     return kvs, build_batch([SeqChunk(b, [0] * qlen, ctx - qlen) for b in range(B)], kvs[0].block_table_host, "cuda")

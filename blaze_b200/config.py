@@ -593,7 +593,7 @@ class ModelConfig:
                 rec = DeltaSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), conv=int(m["conv"]),
                                 head_decay=True, gate="silu")
             elif e["type"] == "parallel":
-                l, t = m["left"], m["left"]["q_temp"]
+                l, t = m["left"], m["left"].get("q_temp") or {"coef": 0.0, "every": 1.0}
                 attn = SigmoidAttnSpec(heads=int(l["heads"]), kv_heads=int(l["kv_heads"]), dim=int(l["dim"]), vdim=int(l["vdim"]),
                                        scale=float(l["scale"]), far=float(l["bias_max"]), bias=True, conv=int(l["conv"]), unit_v=True,
                                        temp_coef=float(t["coef"]), temp_every=float(t["every"]))
