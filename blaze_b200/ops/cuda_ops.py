@@ -215,7 +215,9 @@ class CudaOps:
         lib.blz_sigmoid_plain.argtypes = common + [VP] + shape + [_c.c_int, VP]
         lib.blz_sigmoid_tc.argtypes = common + shape + [_c.c_int, _c.c_int, VP]
         lib.blz_sigmoid_short.argtypes = common + shape + [_c.c_int, _c.c_int, _c.c_int, VP, VP, VP]
-        lib.blz_min_gru.argtypes = [VP, VP, VP, LL, VP, VP, LL, VP, VP, VP, VP] + [_c.c_int] * 4 + [VP]
+        lib.blz_min_gru.argtypes = [VP, VP, VP, LL, VP, VP, LL, VP, VP, VP, VP] + [_c.c_int] * 4 + [VP, _c.c_int, VP]
+        lib.blz_min_gru_ws_bytes.restype = LL
+        lib.blz_min_gru_ws_bytes.argtypes = [_c.c_int] * 3
         # latent attention
         lib.blz_latent_prep.argtypes = [VP, LL, LL, LL, VP, VP, LL, VP, VP, VP, VP, VP] + [_c.c_int] * 5 + [_c.c_float, _c.c_int, VP]
         lib.blz_latent_rot.argtypes = [VP] * 5 + [_c.c_int] * 7 + [VP]
@@ -969,11 +971,13 @@ class CudaOps:
         z, u, g = [VP(proj.data_ptr() + M.cols[c] * es) for c in ("zg", "u", "g")]
         lens = [e - s for s, e in zip(batch.h_q_start, batch.h_q_start[1:])]
         kinds = (1 if 1 in lens else 0) | (2 if batch.max_q_len > 1 else 0)
-        if kinds == 3:
-            self.launches += 1
+        ws_bytes = int(self.lib.blz_min_gru_ws_bytes(len(lens), int(batch.max_q_len), r.width)) if kinds & 2 else 0
+        ws = torch.empty(ws_bytes, dtype=torch.uint8, device=self.device) if ws_bytes else None
+        self.launches += int(kinds == 3) + int(ws is not None)
         self._check(self.lib.blz_min_gru(z, u, g, proj.stride(0), _ptr(kv.rec_state[layer_idx]), _ptr(out), out.stride(0) if out is not None else 0,
                                          _ptr(batch.slots), _ptr(batch.q_start), _ptr(batch.ctx_len), _ptr(batch.gdn_defer),
-                                         batch.slots.numel(), r.width, kinds, int(es == 4), self._stream()), "min_gru")
+                                         batch.slots.numel(), r.width, int(batch.max_q_len), kinds, _ptr(ws), int(es == 4), self._stream()),
+                    "min_gru")
 
     def gated_norm(self, o, gates, M, eps, out):
         """The norm and gate of a recurrence's rows ``o``; ``gates`` holds the gate's columns: the low-rank outputs (delta rule with channel

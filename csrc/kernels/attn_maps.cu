@@ -779,19 +779,28 @@ template <typename T, int TAPS, int VEC>
 __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) {
   pdl_trigger();
   pdl_wait();
+  constexpr int IN = TAPS - 1 + kConvPrepTok;          // rows that the block's tokens need
   const PrepParams& p = q.a;
   const int lane = threadIdx.x & 31, u = blockIdx.y * 4 + (threadIdx.x >> 5), b = blockIdx.z, t0 = blockIdx.x * kConvPrepTok;
   const int r0 = q.q_start[b], n = q.q_start[b + 1] - r0;
   if (u >= p.heads + 2 * p.kv_heads || t0 >= n) return;
+  const bool fresh = q.ctx_len[b] == n;
   const bool is_q = u < p.heads, is_v = u >= p.heads + p.kv_heads;
   const int D = is_v ? p.vdim : p.dim, g = is_v ? u - p.heads - p.kv_heads : u - p.heads, taps = q.taps, m = min(kConvPrepTok, n - t0);
   const int C = p.heads * p.dim + p.kv_heads * (p.dim + p.vdim);
   const int ch = is_q ? u * p.dim : is_v ? p.heads * p.dim + p.kv_heads * p.dim + g * p.vdim : p.heads * p.dim + g * p.dim;     // first channel
   const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)r0 * p.ld + (is_q ? p.q_off + (size_t)u * p.dim
                                                                           : is_v ? p.v_off + (size_t)g * p.vdim : p.k_off + (size_t)g * p.dim);
-  const bool fresh = q.ctx_len[b] == n;
   T* st = reinterpret_cast<T*>(q.state) + (size_t)q.slots[b] * (taps - 1) * C + ch;
   const int dp = (p.dim + 15) / 16 * 16, vp = (p.vdim + 15) / 16 * 16;
+  // lane k has token k's slot, and its query's factor
+  int my_slot = -1;
+  float my_f = 1.f;
+  if (lane < m && !q.state_only) {
+    if (!is_q) my_slot = p.slot_mapping[r0 + t0 + lane];
+    else if (q.temp_coef != 0.f)
+      my_f = fmaf(q.temp_coef, logf(floorf(__fdiv_rn((float)(p.positions[r0 + t0 + lane] + 1), q.temp_every)) + 1.f), 1.f);
+  }
   auto load = [&](const T* at, float (&v)[VEC]) {
     if constexpr (VEC == 4 && sizeof(T) == 2) {
       const uint2 w = *reinterpret_cast<const uint2*>(at);
@@ -804,6 +813,11 @@ __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) 
       v[0] = ad_ld(at);
     }
   };
+  auto store = [&](T* at, const float (&v)[VEC], float f) {
+    if constexpr (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(at) = make_uint2(pack_bf16x2(v[0] * f, v[1 % VEC] * f), pack_bf16x2(v[2 % VEC] * f, v[3 % VEC] * f));
+    else if constexpr (VEC == 4) *reinterpret_cast<float4*>(at) = make_float4(v[0] * f, v[1 % VEC] * f, v[2 % VEC] * f, v[3 % VEC] * f);
+    else ad_st(at, v[0] * f);
+  };
   auto input = [&](int t, int c, float (&v)[VEC]) {     // projected columns c.. of the sequence's new token t (negative: before them)
     if (t >= 0) {
       load(src + (size_t)t * p.ld + c, v);
@@ -814,17 +828,45 @@ __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) 
       for (int j = 0; j < VEC; ++j) v[j] = 0.f;
     }
   };
-  float y[kConvPrepTok][VEC];
+  const bool advance = t0 == 0 && taps > 1 && !(q.no_store != nullptr && q.no_store[b]);
+  // the state after the run, entry i the row taps - 1 - i before the next token; entries of a short run move up.  `in`: rows from
+  // 1 - TAPS on, all that a run of up to kConvPrepTok tokens can leave behind
+  auto leave = [&](int c, const float (&in)[IN][VEC]) {
+    if (n <= kConvPrepTok) {
+#pragma unroll
+      for (int k = 0; k < IN; ++k) {
+        const int i = k - (TAPS - 1) - n + taps - 1;
+        if (i >= 0 && i < taps - 1 && k < TAPS - 1 + n) store(st + (size_t)i * C + c, in[k], 1.f);
+      }
+    } else {
+      float v[TAPS][VEC];
+#pragma unroll
+      for (int i = 0; i < TAPS - 1; ++i)
+        if (i < taps - 1) load(src + (size_t)(n - (taps - 1) + i) * p.ld + c, v[i]);
+#pragma unroll
+      for (int i = 0; i < TAPS - 1; ++i)
+        if (i < taps - 1) store(st + (size_t)i * C + c, v[i], 1.f);
+    }
+  };
+  float y[kConvPrepTok][VEC], in[IN][VEC];
   auto conv = [&](int c) {
-    float in[TAPS - 1 + kConvPrepTok][VEC], w[TAPS][VEC];
+    float w[TAPS][VEC];
 #pragma unroll
     for (int i = 0; i < TAPS; ++i) {
       const int r = i - (TAPS - taps);
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) w[i][j] = r >= 0 ? q.w[(size_t)r * C + ch + c + j] : 0.f;
+      for (int j = 0; j < VEC; ++j) w[i][j] = 0.f;
+      if (r < 0) continue;
+      const float* at = q.w + (size_t)r * C + ch + c;
+      if constexpr (VEC == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(at);
+        w[i][0] = f.x; w[i][1] = f.y; w[i][2] = f.z; w[i][3] = f.w;
+      } else {
+        w[i][0] = *at;
+      }
     }
 #pragma unroll
-    for (int i = 0; i < TAPS - 1 + kConvPrepTok; ++i) {
+    for (int i = 0; i < IN; ++i) {
       if (i < TAPS - 1 + m) {
         input(t0 + i - (TAPS - 1), c, in[i]);
       } else {
@@ -834,6 +876,7 @@ __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) 
     }
 #pragma unroll
     for (int k = 0; k < kConvPrepTok; ++k) {
+      if (k >= m) break;
 #pragma unroll
       for (int j = 0; j < VEC; ++j) {
         y[k][j] = 0.f;
@@ -842,63 +885,55 @@ __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) 
       }
     }
   };
-  if (!q.state_only) {
-    const bool once = D <= 32 * VEC;
-    float f[kConvPrepTok];
-#pragma unroll
-    for (int k = 0; k < kConvPrepTok; ++k) f[k] = 1.f;
-    if (once && lane * VEC < D) conv(lane * VEC);
-    if (is_v && q.unit_v) {
-      float ss[kConvPrepTok];
-#pragma unroll
-      for (int k = 0; k < kConvPrepTok; ++k) ss[k] = 0.f;
-      for (int c = lane * VEC; c < D; c += 32 * VEC) {
-        if (!once) conv(c);
-#pragma unroll
-        for (int k = 0; k < kConvPrepTok; ++k)
-#pragma unroll
-          for (int j = 0; j < VEC; ++j) ss[k] = fmaf(y[k][j], y[k][j], ss[k]);
-      }
-#pragma unroll
-      for (int k = 0; k < kConvPrepTok; ++k)
-        if (k < m) f[k] = 1.f / sqrtf(warp_sum(ss[k]) / (float)D + p.eps);
-    } else if (is_q && q.temp_coef != 0.f) {
-#pragma unroll
-      for (int k = 0; k < kConvPrepTok; ++k)
-        if (k < m) f[k] = fmaf(q.temp_coef, logf(floorf(__fdiv_rn((float)(p.positions[r0 + t0 + k] + 1), q.temp_every)) + 1.f), 1.f);
+  const bool once = D <= 32 * VEC;                     // one turn of the warp takes the whole head
+  if (once && lane * VEC < D) conv(lane * VEC);
+  if (q.state_only) {
+    for (int c = lane * VEC; c < D && advance; c += 32 * VEC) {
+      if (!once) conv(c);
+      leave(c, in);
     }
+    return;
+  }
+  if (is_v && q.unit_v) {
+    float ss[kConvPrepTok];
+#pragma unroll
+    for (int k = 0; k < kConvPrepTok; ++k) ss[k] = 0.f;
     for (int c = lane * VEC; c < D; c += 32 * VEC) {
       if (!once) conv(c);
 #pragma unroll
       for (int k = 0; k < kConvPrepTok; ++k) {
         if (k >= m) break;
-        const int row = r0 + t0 + k;
-        T* dst;
-        if (is_q) {
-          dst = reinterpret_cast<T*>(p.q_out) + ((size_t)row * p.heads + u) * p.dim + c;
-        } else {
-          const int slot = p.slot_mapping[row];
-          if (slot < 0) continue;
-          dst = reinterpret_cast<T*>(p.pool) + (size_t)(slot >> 4) * p.page_stride + (size_t)g * p.head_stride +
-                (is_v ? 16 * dp + core_off(slot & 15, c, vp) : core_off(slot & 15, c, dp));
-        }
-        if constexpr (VEC == 4 && sizeof(T) == 2)
-          *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(y[k][0] * f[k], y[k][1] * f[k]), pack_bf16x2(y[k][2] * f[k], y[k][3] * f[k]));
-        else if constexpr (VEC == 4)
-          *reinterpret_cast<float4*>(dst) = make_float4(y[k][0] * f[k], y[k][1] * f[k], y[k][2] * f[k], y[k][3] * f[k]);
-        else
-          ad_st(dst, y[k][0] * f[k]);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) ss[k] = fmaf(y[k][j], y[k][j], ss[k]);
       }
     }
-  }
-  if (t0 > 0 || taps < 2 || (q.no_store != nullptr && q.no_store[b])) return;
-  for (int c = lane * VEC; c < D; c += 32 * VEC) {
-    for (int i = 0; i < taps - 1; ++i) {               // entry i: the row taps - 1 - i before the next token; an older entry moves up
-      float v[VEC];
-      input(n - (taps - 1) + i, c, v);
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) ad_st(st + (size_t)i * C + c + j, v[j]);
+    for (int k = 0; k < kConvPrepTok; ++k) {
+      if (k >= m) break;
+      const float f = 1.f / sqrtf(warp_sum(ss[k]) / (float)D + p.eps);
+      if (lane == k) my_f = f;
     }
+  }
+  float f[kConvPrepTok];
+  int slot[kConvPrepTok];
+#pragma unroll
+  for (int k = 0; k < kConvPrepTok; ++k) {
+    f[k] = __shfl_sync(0xffffffffu, my_f, k);
+    slot[k] = __shfl_sync(0xffffffffu, my_slot, k);
+  }
+  for (int c = lane * VEC; c < D; c += 32 * VEC) {
+    if (!once) conv(c);
+#pragma unroll
+    for (int k = 0; k < kConvPrepTok; ++k) {
+      if (k >= m) break;
+      if (is_q) {
+        store(reinterpret_cast<T*>(p.q_out) + ((size_t)(r0 + t0 + k) * p.heads + u) * p.dim + c, y[k], f[k]);
+      } else if (slot[k] >= 0) {
+        T* page = reinterpret_cast<T*>(p.pool) + (size_t)(slot[k] >> 4) * p.page_stride + (size_t)g * p.head_stride;
+        store(page + (is_v ? 16 * dp + core_off(slot[k] & 15, c, vp) : core_off(slot[k] & 15, c, dp)), y[k], f[k]);
+      }
+    }
+    if (advance) leave(c, in);
   }
 }
 

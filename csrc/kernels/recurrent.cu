@@ -556,7 +556,7 @@ __global__ void __launch_bounds__(kRecWarps * 32, 4) gated_step_kernel(RecParams
 }
 
 // ------------------------------------------------------------------------------------------ long runs
-// Records: delta [heads][T][q | k | g | beta, k . q, 0, 0], with one decay per head [heads][T][q | k | beta, k . q, g, 0], state space [groups][T][B | C] and [heads][T][dt, decay, 0, 0], gated
+// Records: delta [heads][T][q | k | g | beta, k . q, 0, 0] (one decay per head: see delta_block_records_kernel), state space [groups][T][B | C] and [heads][T][dt, decay, 0, 0], gated
 // linear [heads][T][f | q]; vectors padded to 32, 64, 128, 256 or 512 floats.
 __device__ __forceinline__ bool in_long_run(const RecParams& p, int t) {
   const int b = p.seq_of_row[t];
@@ -564,22 +564,22 @@ __device__ __forceinline__ bool in_long_run(const RecParams& p, int t) {
 }
 
 // a warp per (row, head)
-template <typename T, int DKP, bool HD>
+template <typename T, int DKP>
 __global__ void __launch_bounds__(128) delta_records_kernel(RecParams p) {
-  constexpr int B0 = (HD ? 2 : 3) * DKP, REC = B0 + 4, NV = DKP / 32;
+  constexpr int REC = 3 * DKP + 4, NV = DKP / 32;
   const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
   const int t = (int)(w / p.heads), h = (int)(w % p.heads), lane = threadIdx.x & 31;
   if (t >= p.T || !in_long_run(p, t)) return;
   const int dk = p.dk, hk = h / (p.heads / p.groups);
   const T* cv = reinterpret_cast<const T*>(p.conv) + (size_t)t * p.ld_conv;
-  const T* av = reinterpret_cast<const T*>(p.a) + (size_t)t * p.ld_a + (size_t)(HD ? 0 : h) * dk;
+  const T* av = reinterpret_cast<const T*>(p.a) + (size_t)t * p.ld_a + (size_t)h * dk;
   float q[NV], k[NV], a[NV], qq = 0.f, kk = 0.f, kq = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int d = lane + i * 32;
     q[i] = d < dk ? rc_ld(cv + (size_t)hk * dk + d) : 0.f;
     k[i] = d < dk ? rc_ld(cv + (size_t)(p.groups + hk) * dk + d) : 0.f;
-    a[i] = !HD && d < dk ? rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d] : 0.f;
+    a[i] = d < dk ? rc_ld(av + d) + p.dt_bias[(size_t)h * dk + d] : 0.f;
   }
   const float beta = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + (size_t)t * p.ld_b + h)), A = p.A[h];
 #pragma unroll
@@ -596,9 +596,91 @@ __global__ void __launch_bounds__(128) delta_records_kernel(RecParams p) {
     const int d = lane + i * 32;
     s[d] = q[i] * qn;
     s[DKP + d] = k[i] * kn;
-    if constexpr (!HD) s[2 * DKP + d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(a[i])) : 1.f;
+    s[2 * DKP + d] = d < dk ? rc_exp<T>(-A * rc_softplus<T>(a[i])) : 1.f;
   }
-  if (lane == 0) *reinterpret_cast<float4*>(s + B0) = make_float4(beta, kq, HD ? head_decay<T>(p, t, h) : 0.f, 0.f);
+  if (lane == 0) *reinterpret_cast<float4*>(s + 3 * DKP) = make_float4(beta, kq, 0.f, 0.f);
+}
+
+// One decay per head: four tokens at a time.  With S the state before them, G_i the decay over tokens 0..i and D_ij that over j+1..i,
+//   u_i = beta_i (v_i - G_i S^T k_i) - sum_{j<i} a_ij u_j,  a_ij = beta_i D_ij k_i . k_j
+//   o_i = G_i S^T q_i + sum_{j<=i} c_ij u_j,                c_ij = D_ij q_i . k_j
+//   S <- G_3 S + sum_j D_3j k_j u_j
+// so that the products with the state do not wait for one another.  A warp per (4 tokens, head) writes what does not depend on the
+// state: per token q | k | a_i0..3 | c_i0..3 | beta_i, beta_i G_i, G_i, D_3i | G_3, 0, 0, 0 (a sequence's last tokens: of those there are).
+static constexpr int kBlockTok = 4, kBlockCoef = 16;
+struct Whole { static constexpr bool value = true; };
+struct Part { static constexpr bool value = false; };
+template <typename T, int DKP>
+__global__ void __launch_bounds__(128) delta_block_records_kernel(RecParams p) {
+  constexpr int REC = 2 * DKP + kBlockCoef, NV = DKP / 32;
+  const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int t = (int)(w / p.heads), h = (int)(w % p.heads), lane = threadIdx.x & 31;
+  if (t >= p.T || !in_long_run(p, t)) return;
+  const int seq = p.seq_of_row[t], rest = p.q_start[seq + 1] - t, m = min(kBlockTok, rest);
+  if ((t - p.q_start[seq]) % kBlockTok) return;            // the block's first row has the whole block
+  const int dk = p.dk, hk = h / (p.heads / p.groups);
+  float q[kBlockTok][NV], k[kBlockTok][NV], beta[kBlockTok], g[kBlockTok];
+#pragma unroll
+  for (int j = 0; j < kBlockTok; ++j) {
+    const T* cv = reinterpret_cast<const T*>(p.conv) + (size_t)(t + min(j, m - 1)) * p.ld_conv;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = lane + i * 32;
+      q[j][i] = d < dk && j < m ? rc_ld(cv + (size_t)hk * dk + d) : 0.f;
+      k[j][i] = d < dk && j < m ? rc_ld(cv + (size_t)(p.groups + hk) * dk + d) : 0.f;
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < kBlockTok; ++j) {
+    const size_t row = t + min(j, m - 1);
+    beta[j] = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + row * p.ld_b + h));
+    g[j] = head_decay<T>(p, row, h);
+  }
+  const float qs = rsqrtf((float)dk);
+#pragma unroll
+  for (int j = 0; j < kBlockTok; ++j) {
+    float qq = 0.f, kk = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) { qq = fmaf(q[j][i], q[j][i], qq); kk = fmaf(k[j][i], k[j][i], kk); }
+    const float qn = qs / sqrtf(warp_sum(qq) + 1e-6f), kn = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) { q[j][i] *= qn; k[j][i] *= kn; }
+  }
+  float G = 1.f, D[kBlockTok];                             // D[j]: decay over tokens j + 1 .. i
+#pragma unroll
+  for (int i = 0; i < kBlockTok; ++i) {
+    if (i >= m) break;
+    float* s = p.records + ((size_t)h * p.T + t + i) * REC;
+    G *= g[i];
+    float a[kBlockTok], c[kBlockTok];
+#pragma unroll
+    for (int j = 0; j < kBlockTok; ++j) {
+      a[j] = c[j] = 0.f;
+      if (j > i) continue;
+      D[j] = j == i ? 1.f : D[j] * g[i];
+      float kk = 0.f, qk = 0.f;
+#pragma unroll
+      for (int e = 0; e < NV; ++e) { kk = fmaf(k[i][e], k[j][e], kk); qk = fmaf(q[i][e], k[j][e], qk); }
+      c[j] = D[j] * warp_sum(qk);
+      if (j < i) a[j] = beta[i] * D[j] * warp_sum(kk);
+    }
+#pragma unroll
+    for (int e = 0; e < NV; ++e) {
+      s[lane + e * 32] = q[i][e];
+      s[DKP + lane + e * 32] = k[i][e];
+    }
+    if (lane == 0) {
+      float4* f = reinterpret_cast<float4*>(s + 2 * DKP);
+      f[0] = make_float4(a[0], a[1], a[2], a[3]);
+      f[1] = make_float4(c[0], c[1], c[2], c[3]);
+      float last = 1.f, all = G;                           // decays to the end of the block
+#pragma unroll
+      for (int e = 1; e < kBlockTok; ++e)
+        if (e > i && e < m) { last *= g[e]; all *= g[e]; }
+      f[2] = make_float4(beta[i], beta[i] * G, G, last);
+      f[3] = make_float4(all, 0.f, 0.f, 0.f);
+    }
+  }
 }
 
 // a block per row
@@ -699,9 +781,9 @@ __device__ __forceinline__ void wait_cols() { asm volatile("cp.async.wait_group 
 
 static constexpr int kRecHead = 128;         // barriers in front of the ring
 
-template <typename T, int KL, int R, int VPT, bool HD>
+template <typename T, int KL, int R, int VPT>
 __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) delta_stream_kernel(RecParams p, int slices, int vec_v) {
-  constexpr int DKP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, B0 = (HD ? 2 : 3) * DKP, REC = B0 + 4, STAGE = kRecTok * REC;
+  constexpr int DKP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, REC = 3 * DKP + 4, STAGE = kRecTok * REC;
   constexpr int PART = VPT == 2 ? 2 : 1;            // independent chains per sum
   extern __shared__ __align__(128) uint8_t sm8[];
   __shared__ __align__(16) T s_v[kRecWarps][kColsAhead + 1][kRecTok][CG * VPT];
@@ -750,7 +832,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
     float y[VPT <= 2 ? kRecTok : 1][VPT];
     // what a token brings: the lane's rows of q, k and g, its v, beta and k . q
     struct Tok {
-      float q[R], k[R], g[HD ? 1 : R], v[VPT];
+      float q[R], k[R], g[R], v[VPT];
       float2 bk;
     };
     auto fetch = [&](int j, Tok& o) {
@@ -761,13 +843,10 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
         const float4 k4 = *reinterpret_cast<const float4*>(s + DKP + kl * 4 + 4 * KL * i4);
         o.q[i4 * 4] = q4.x; o.q[i4 * 4 + 1] = q4.y; o.q[i4 * 4 + 2] = q4.z; o.q[i4 * 4 + 3] = q4.w;
         o.k[i4 * 4] = k4.x; o.k[i4 * 4 + 1] = k4.y; o.k[i4 * 4 + 2] = k4.z; o.k[i4 * 4 + 3] = k4.w;
-        if constexpr (!HD) {
-          const float4 g4 = *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 4 * KL * i4);
-          o.g[i4 * 4] = g4.x; o.g[i4 * 4 + 1] = g4.y; o.g[i4 * 4 + 2] = g4.z; o.g[i4 * 4 + 3] = g4.w;
-        }
+        const float4 g4 = *reinterpret_cast<const float4*>(s + 2 * DKP + kl * 4 + 4 * KL * i4);
+        o.g[i4 * 4] = g4.x; o.g[i4 * 4 + 1] = g4.y; o.g[i4 * 4 + 2] = g4.z; o.g[i4 * 4 + 3] = g4.w;
       }
-      o.bk = *reinterpret_cast<const float2*>(s + B0);
-      if constexpr (HD) o.g[0] = s[B0 + 2];
+      o.bk = *reinterpret_cast<const float2*>(s + 3 * DKP);
 #pragma unroll
       for (int v = 0; v < VPT; ++v) o.v[v] = rc_ld(&cols[j][cg * VPT + v]);
     };
@@ -781,7 +860,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
       for (int i = 0; i < R; ++i)
 #pragma unroll
         for (int v = 0; v < VPT; ++v) {
-          S[i][v] *= x.g[HD ? 0 : i];
+          S[i][v] *= x.g[i];
           part[v][i % PART] = fmaf(S[i][v], x.k[i], part[v][i % PART]);
           pq[v][i % PART] = fmaf(S[i][v], x.q[i], pq[v][i % PART]);
         }
@@ -846,6 +925,159 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
       spread_tokens<KL, VPT>(y, kl);
       if (kl < m) store_cols<VPT>(p.out + ((size_t)(r0 + t0 + kl) * p.heads + h) * dv + col, y[0], col, dv, vec);
     }
+  }
+  if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<KL, R, VPT>(S, st, kl, col, dk, dv, vec);
+}
+
+// sums of y[token][column] over the KL (8 or 16) lanes of a column, the 4 tokens spread over them: lane kl ends with token kl % 4 in y[0]
+template <int KL, int VPT>
+__device__ __forceinline__ void spread_block(float (&y)[kBlockTok][VPT], int kl) {
+  const bool u2 = kl & 2, u1 = kl & 1;
+#pragma unroll
+  for (int v = 0; v < VPT; ++v) {
+    float z[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) z[j] = (u2 ? y[j + 2][v] : y[j][v]) + __shfl_xor_sync(0xffffffffu, u2 ? y[j][v] : y[j + 2][v], 2);
+    y[0][v] = (u1 ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, u1 ? z[0] : z[1], 1);
+#pragma unroll
+    for (int o = 4; o < KL; o <<= 1) y[0][v] += __shfl_xor_sync(0xffffffffu, y[0][v], o);
+  }
+}
+
+// long runs with one decay per head, four tokens at a time (see delta_block_records_kernel)
+template <typename T, int KL, int R, int VPT>
+__global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) delta_block_kernel(RecParams p, int slices, int vec_v) {
+  constexpr int DKP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, REC = 2 * DKP + kBlockCoef, STAGE = kRecTok * REC;
+  constexpr bool KEEP_K = R <= 8;                   // registers for the block's keys
+  extern __shared__ __align__(128) uint8_t sm8[];
+  __shared__ __align__(16) T s_v[kRecWarps][kColsAhead + 1][kRecTok][CG * VPT];
+  const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
+  if (n < p.long_rows) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane % KL, cg = lane / KL;
+  const int groups = (n + kRecTok - 1) / kRecTok;
+  float* ring = reinterpret_cast<float*>(sm8 + kRecHead);
+  RecRing rr;
+  rr.init(sm8, p.status);
+  if (warp == kRecWarps) {
+    if (lane == 0) {
+      const float* src = p.records + ((size_t)h * p.T + r0) * REC;
+      rr.produce(groups, [&](int c) {
+        const uint32_t bytes = (uint32_t)min(kRecTok, n - c * kRecTok) * REC * 4;
+        mbar_expect_tx(&rr.full[c % kRecStages], bytes);
+        bulk_load(ring + (c % kRecStages) * STAGE, src + (size_t)c * STAGE, bytes, &rr.full[c % kRecStages]);
+      });
+    }
+    return;
+  }
+  const int dk = p.dk, dv = p.dv, col = slice * COLS + warp * CG * VPT + cg * VPT;
+  float* st = p.state + ((size_t)slot * p.heads + h) * dk * dv;
+  const bool vec = dv % 4 == 0;
+  float S[R][VPT];
+  load_state<KL, R, VPT>(S, st, kl, col, dk, dv, ctx == n, vec);
+  const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + (kl & 7)) * p.ld_conv + (size_t)2 * p.groups * dk + (size_t)h * dv + col;
+  auto send_group = [&](int c) {
+    send_cols<T, VPT>(&s_v[warp][c % (kColsAhead + 1)][kl & 7][cg * VPT], vsrc + (size_t)c * kRecTok * p.ld_conv,
+                      kl < kRecTok && c * kRecTok + kl < n, col, dv, vec_v);
+  };
+#pragma unroll
+  for (int c = 0; c < kColsAhead; ++c) send_group(c);
+  const int mine = kl & (kBlockTok - 1), quad = lane & ~(kBlockTok - 1);
+  bool ok = true;
+  for (int c = 0; c < groups; ++c) {
+    const int t0 = c * kRecTok;
+    __syncwarp();                            // the last group's columns have been read
+    send_group(c + kColsAhead);
+    wait_cols();
+    const T(*cols)[CG * VPT] = s_v[warp][c % (kColsAhead + 1)];
+    ok = rr.wait_full(c);
+    if (!ok) break;
+    __syncwarp();
+    const float* buf = ring + (c % kRecStages) * STAGE;
+    auto block = [&](int j0, int m, auto whole) {
+      constexpr bool WHOLE = decltype(whole)::value;       // m == kBlockTok
+      const float* rec = buf + j0 * REC;
+      float pk[kBlockTok][VPT], pq[kBlockTok][VPT];
+      [[maybe_unused]] float kr[KEEP_K ? kBlockTok : 1][R];
+#pragma unroll
+      for (int j = 0; j < kBlockTok; ++j) {
+#pragma unroll
+        for (int v = 0; v < VPT; ++v) pk[j][v] = pq[j][v] = 0.f;
+        if (!WHOLE && j >= m) continue;
+#pragma unroll
+        for (int i4 = 0; i4 < R / 4; ++i4) {
+          const float4 q4 = *reinterpret_cast<const float4*>(rec + j * REC + kl * 4 + 4 * KL * i4);
+          const float4 k4 = *reinterpret_cast<const float4*>(rec + j * REC + DKP + kl * 4 + 4 * KL * i4);
+          const float qa[4] = {q4.x, q4.y, q4.z, q4.w}, ka[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            if constexpr (KEEP_K) kr[j][i4 * 4 + i] = ka[i];
+#pragma unroll
+            for (int v = 0; v < VPT; ++v) {
+              pk[j][v] = fmaf(S[i4 * 4 + i][v], ka[i], pk[j][v]);
+              pq[j][v] = fmaf(S[i4 * 4 + i][v], qa[i], pq[j][v]);
+            }
+          }
+        }
+      }
+      spread_block<KL, VPT>(pk, kl);
+      spread_block<KL, VPT>(pq, kl);
+      // this lane's token of the block
+      const int my = WHOLE ? mine : min(mine, m - 1);
+      const float* cf = rec + my * REC + 2 * DKP;
+      const float4 a4 = *reinterpret_cast<const float4*>(cf), c4 = *reinterpret_cast<const float4*>(cf + 4), s4 = *reinterpret_cast<const float4*>(cf + 8);
+      const float a[4] = {a4.x, a4.y, a4.z, a4.w}, cc[4] = {c4.x, c4.y, c4.z, c4.w};
+      float u[VPT], o[VPT], uu[kBlockTok][VPT];
+#pragma unroll
+      for (int v = 0; v < VPT; ++v) {
+        u[v] = fmaf(s4.x, rc_ld(&cols[j0 + my][cg * VPT + v]), -s4.y * pk[0][v]);
+        o[v] = s4.z * pq[0][v];
+      }
+#pragma unroll
+      for (int j = 0; j < kBlockTok; ++j) {
+        if (!WHOLE && j >= m) break;
+        const float to_end = rec[j * REC + 2 * DKP + 11];
+#pragma unroll
+        for (int v = 0; v < VPT; ++v) {
+          const float x = __shfl_sync(0xffffffffu, u[v], quad | j);
+          u[v] = fmaf(-a[j], x, u[v]);
+          o[v] = fmaf(cc[j], x, o[v]);
+          uu[j][v] = to_end * x;
+        }
+      }
+      if (kl < m) store_cols<VPT>(p.out + ((size_t)(r0 + t0 + j0 + kl) * p.heads + h) * dv + col, o, col, dv, vec);
+      const float all = rec[2 * DKP + 12];
+#pragma unroll
+      for (int i = 0; i < R; ++i)
+#pragma unroll
+        for (int v = 0; v < VPT; ++v) S[i][v] *= all;
+#pragma unroll
+      for (int j = 0; j < kBlockTok; ++j) {
+        if (!WHOLE && j >= m) break;
+#pragma unroll
+        for (int i4 = 0; i4 < R / 4; ++i4) {
+          float ka[4];
+          if constexpr (KEEP_K) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) ka[i] = kr[j][i4 * 4 + i];
+          } else {
+            const float4 k4 = *reinterpret_cast<const float4*>(rec + j * REC + DKP + kl * 4 + 4 * KL * i4);
+            ka[0] = k4.x; ka[1] = k4.y; ka[2] = k4.z; ka[3] = k4.w;
+          }
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int v = 0; v < VPT; ++v) S[i4 * 4 + i][v] = fmaf(ka[i], uu[j][v], S[i4 * 4 + i][v]);
+        }
+      }
+    };
+    const int m = min(kRecTok, n - t0);
+#pragma unroll
+    for (int j0 = 0; j0 < kRecTok; j0 += kBlockTok) {
+      if (m >= j0 + kBlockTok) block(j0, kBlockTok, Whole{});
+      else if (m > j0) block(j0, m - j0, Part{});
+    }
+    rr.release(c);
   }
   if (ok && !(p.no_store != nullptr && p.no_store[b])) store_state<KL, R, VPT>(S, st, kl, col, dk, dv, vec);
 }
@@ -1081,14 +1313,27 @@ struct GruParams {
   const int *slots, *q_start, *ctx_len, *no_store;
   long long ld, ld_out;
   int width;
+  float2* pairs;               // [B][parts][width]: of each part of a run, the factor of the state before it and the addend; of the first
+                               // part the addend alone, with the state before the run in it; or null (a block takes a whole run)
+  float* before;               // [B][width]: the states before the runs (with pairs)
+  int part, parts;             // tokens per part, parts of the longest run
 };
-static constexpr int kGruWarps = 16, kGruTok = 8;      // a block takes kGruWarps * kGruTok tokens at a time
+static constexpr int kGruWarps = 8, kGruTok = 8;       // a block takes kGruWarps * kGruTok tokens at a time
+static constexpr int kGruPart = 256;
 
+// a gate; bf16: the special function unit's reciprocal (two units in the last place)
+template <typename T>
+__device__ __forceinline__ float gru_sigmoid(float x) {
+  if constexpr (sizeof(T) == 4) return 1.f / (1.f + expf(-x));
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + __expf(-x)));
+  return r;
+}
 template <typename T>
 __device__ __forceinline__ void gru_gate(float z, float u, float& keep, float& add) {
-  const float s = rc_sigmoid<T>(z);
+  const float s = gru_sigmoid<T>(z), c = gru_sigmoid<T>(u);
   keep = 1.f - s;
-  add = s * (u >= 0.f ? u + 0.5f : rc_sigmoid<T>(u));
+  add = s * (u >= 0.f ? u + 0.5f : c);
 }
 template <typename T, int VEC> struct alignas(sizeof(T) * VEC) GruVec { T e[VEC]; };
 template <typename T, int VEC>
@@ -1101,27 +1346,35 @@ __device__ __forceinline__ GruVec<T, VEC> gru_load(const void* base, size_t at) 
   else v.e[0] = *p;
   return v;
 }
+// vec: the output's rows allow VEC elements as one word
 template <typename T, int VEC>
-__device__ __forceinline__ void gru_store(const GruParams& p, size_t row, int c, const GruVec<T, VEC>& g, const float (&S)[VEC]) {
+__device__ __forceinline__ void gru_store(const GruParams& p, size_t row, int c, const GruVec<T, VEC>& g, const float (&S)[VEC], bool vec) {
   T* o = reinterpret_cast<T*>(p.out) + row * p.ld_out + c;
+  GruVec<T, VEC> y;
 #pragma unroll
   for (int j = 0; j < VEC; ++j) {
-    const float y = S[j] * rc_silu<T>(rc_ld(g.e + j));
-    if constexpr (sizeof(T) == 4) o[j] = y;
-    else o[j] = __float2bfloat16(y);
+    const float x = rc_ld(g.e + j), v = S[j] * (x * gru_sigmoid<T>(x));
+    if constexpr (sizeof(T) == 4) y.e[j] = v;
+    else y.e[j] = __float2bfloat16(v);
+  }
+  if (vec) {
+    *reinterpret_cast<GruVec<T, VEC>*>(o) = y;
+  } else {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) o[j] = y.e[j];
   }
 }
 
 // single tokens: a thread per VEC elements of a sequence
 template <typename T, int VEC>
-__global__ void __launch_bounds__(128) min_gru_step_kernel(GruParams p) {
+__global__ void __launch_bounds__(128) min_gru_step_kernel(GruParams p, int vec) {
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.y, c = (blockIdx.x * 128 + threadIdx.x) * VEC;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
   if (n != 1 || c >= p.width) return;
   const size_t at = (size_t)r0 * p.ld + c;
-  const auto z = gru_load<T, VEC>(p.z, at), u = gru_load<T, VEC>(p.u, at);
+  const auto z = gru_load<T, VEC>(p.z, at), u = gru_load<T, VEC>(p.u, at), g = gru_load<T, VEC>(p.g, at);
   float* st = p.state + (size_t)p.slots[b] * p.width + c;
   const bool fresh = p.ctx_len[b] == 1;
   float S[VEC];
@@ -1131,45 +1384,112 @@ __global__ void __launch_bounds__(128) min_gru_step_kernel(GruParams p) {
     gru_gate<T>(rc_ld(z.e + j), rc_ld(u.e + j), keep, add);
     S[j] = fresh ? add : fmaf(keep, st[j], add);
   }
-  if (p.out) gru_store<T, VEC>(p, r0, c, gru_load<T, VEC>(p.g, at), S);
+  if (p.out) gru_store<T, VEC>(p, r0, c, g, S, vec);
   if (p.no_store != nullptr && p.no_store[b]) return;
 #pragma unroll
   for (int j = 0; j < VEC; ++j) st[j] = S[j];
 }
 
-// longer runs: a block per 32 * VEC elements of a sequence.  Each warp folds kGruTok tokens into one pair (factor, addend) per element;
-// the pairs of the warps before it and the carry give the state its own tokens start from.  The next tokens are fetched meanwhile.
+// what a part of a run does to the state, for parts that blocks of their own take (see GruParams::pairs); a thread per VEC elements
 template <typename T, int VEC>
-__global__ void __launch_bounds__(kGruWarps * 32) min_gru_kernel(GruParams p) {
-  __shared__ float s_a[2][kGruWarps][32 * VEC], s_b[2][kGruWarps][32 * VEC], s_c[2][32 * VEC];
+__global__ void __launch_bounds__(64) min_gru_pairs_kernel(GruParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.y, i = blockIdx.z, c = (blockIdx.x * 64 + threadIdx.x) * VEC;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, t0 = i * p.part, t1 = min(n, t0 + p.part);
+  if (n <= 1 || c >= p.width || t0 >= n) return;
+  const bool fresh = p.ctx_len[b] == n;
+  float A[VEC], B[VEC];
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) { A[j] = 1.f; B[j] = 0.f; }
+  if (i == 0) {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      B[j] = fresh ? 0.f : p.state[(size_t)p.slots[b] * p.width + c + j];
+      p.before[(size_t)b * p.width + c + j] = B[j];
+    }
+  }
+  for (int t = t0; t < t1; t += kGruTok) {
+    GruVec<T, VEC> z[kGruTok], u[kGruTok];
+#pragma unroll
+    for (int k = 0; k < kGruTok; ++k)
+      if (t + k < t1) {
+        const size_t at = (size_t)(r0 + t + k) * p.ld + c;
+        z[k] = gru_load<T, VEC>(p.z, at);
+        u[k] = gru_load<T, VEC>(p.u, at);
+      }
+#pragma unroll
+    for (int k = 0; k < kGruTok; ++k)
+      if (t + k < t1)
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          float keep, add;
+          gru_gate<T>(rc_ld(z[k].e + j), rc_ld(u[k].e + j), keep, add);
+          A[j] *= keep;
+          B[j] = fmaf(keep, B[j], add);
+        }
+  }
+  float2* to = p.pairs + ((size_t)b * p.parts + i) * p.width + c;
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) to[j] = make_float2(A[j], B[j]);
+}
+
+// longer runs: a block per 32 * VEC elements of a sequence (and per part of it).  Each warp folds kGruTok tokens into one pair (factor,
+// addend) per element; the pairs of the warps before it and the carry give the state its own tokens start from.  The next tokens are
+// fetched meanwhile.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kGruWarps * 32, 2) min_gru_kernel(GruParams p, int vec) {
+  __shared__ float2 s_p[2][kGruWarps][32 * VEC];
+  __shared__ float s_c[2][32 * VEC];
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, c = (blockIdx.x * 32 + lane) * VEC;
-  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0;
-  if (n <= 1) return;
+  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, from = blockIdx.z * p.part, to = min(n, from + p.part);
+  if (n <= 1 || from >= n) return;
   const bool live = c < p.width;
   float* st = p.state + (size_t)p.slots[b] * p.width + c;
   const bool fresh = p.ctx_len[b] == n;
-  float S[VEC];
-#pragma unroll
-  for (int j = 0; j < VEC; ++j) S[j] = !fresh && live ? st[j] : 0.f;
-  if (warp == 0)
-#pragma unroll
-    for (int j = 0; j < VEC; ++j) s_c[0][lane * VEC + j] = S[j];
   GruVec<T, VEC> z[kGruTok], u[kGruTok], g[kGruTok];
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int k = 0; k < kGruTok; ++k)
-      if (live && t0 + k < n) {
+      if (live && t0 + k < to) {
         const size_t at = (size_t)(r0 + t0 + k) * p.ld + c;
         z[k] = gru_load<T, VEC>(p.z, at);
         u[k] = gru_load<T, VEC>(p.u, at);
         if (p.out) g[k] = gru_load<T, VEC>(p.g, at);
       }
   };
+  fetch(from + warp * kGruTok);
+  float S[VEC];
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) S[j] = 0.f;
+  if (warp == 0) {
+    if (live) {
+      if (!p.pairs) {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) S[j] = fresh ? 0.f : st[j];
+      } else if (blockIdx.z == 0) {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) S[j] = p.before[(size_t)b * p.width + c + j];
+      } else {
+        const float2* pr = p.pairs + (size_t)b * p.parts * p.width + c;
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) S[j] = pr[j].y;
+#pragma unroll 8
+        for (int i = 1; i < blockIdx.z; ++i)
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) {
+            const float2 f = pr[(size_t)i * p.width + j];
+            S[j] = fmaf(f.x, S[j], f.y);
+          }
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) s_c[0][lane * VEC + j] = S[j];
+  }
   constexpr int STEP = kGruWarps * kGruTok;
-  fetch(warp * kGruTok);
-  for (int i = 0, base = 0; base < n; ++i, base += STEP) {
+  for (int i = 0, base = from; base < to; ++i, base += STEP) {
     const int t0 = base + warp * kGruTok, par = i & 1;
     float keep[kGruTok][VEC], add[kGruTok][VEC], A[VEC], B[VEC];
     GruVec<T, VEC> gate[kGruTok];
@@ -1182,48 +1502,56 @@ __global__ void __launch_bounds__(kGruWarps * 32) min_gru_kernel(GruParams p) {
       for (int j = 0; j < VEC; ++j) {
         keep[k][j] = 1.f;
         add[k][j] = 0.f;
-        if (live && t0 + k < n) gru_gate<T>(rc_ld(z[k].e + j), rc_ld(u[k].e + j), keep[k][j], add[k][j]);
+        if (live && t0 + k < to) gru_gate<T>(rc_ld(z[k].e + j), rc_ld(u[k].e + j), keep[k][j], add[k][j]);
         A[j] *= keep[k][j];
         B[j] = fmaf(keep[k][j], B[j], add[k][j]);
       }
     }
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) { s_a[par][warp][lane * VEC + j] = A[j]; s_b[par][warp][lane * VEC + j] = B[j]; }
+    for (int j = 0; j < VEC; ++j) s_p[par][warp][lane * VEC + j] = make_float2(A[j], B[j]);
     fetch(t0 + STEP);
     __syncthreads();
 #pragma unroll
     for (int j = 0; j < VEC; ++j) S[j] = s_c[par][lane * VEC + j];
-    for (int w = 0; w < warp; ++w)
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) S[j] = fmaf(s_a[par][w][lane * VEC + j], S[j], s_b[par][w][lane * VEC + j]);
+    for (int w = 0; w < kGruWarps - 1; ++w)
+      if (w < warp)
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          const float2 f = s_p[par][w][lane * VEC + j];
+          S[j] = fmaf(f.x, S[j], f.y);
+        }
+    if (warp == kGruWarps - 1)               // the state after these tokens, as soon as it is known
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) s_c[par ^ 1][lane * VEC + j] = fmaf(A[j], S[j], B[j]);
 #pragma unroll
     for (int k = 0; k < kGruTok; ++k) {
 #pragma unroll
       for (int j = 0; j < VEC; ++j) S[j] = fmaf(keep[k][j], S[j], add[k][j]);
-      if (p.out && live && t0 + k < n) gru_store<T, VEC>(p, r0 + t0 + k, c, gate[k], S);
+      if (p.out && live && t0 + k < to) gru_store<T, VEC>(p, r0 + t0 + k, c, gate[k], S, vec);
     }
-    if (warp == kGruWarps - 1)
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) s_c[par ^ 1][lane * VEC + j] = S[j];
   }
-  if (warp != kGruWarps - 1 || !live || (p.no_store != nullptr && p.no_store[b])) return;
+  if (to < n || warp != kGruWarps - 1 || !live || (p.no_store != nullptr && p.no_store[b])) return;
 #pragma unroll
   for (int j = 0; j < VEC; ++j) st[j] = S[j];          // tokens beyond the run changed nothing
 }
 
 template <typename T>
-static int run_gru(const GruParams& p, int B, int kinds, int vec, cudaStream_t s) {
+static int run_gru(GruParams p, int B, int kinds, int vec, int vec_o, cudaStream_t s) {
   cudaError_t e = cudaSuccess;
   if (kinds & 1) {
     constexpr int V = 4;
-    if (vec) e = launch_pdl(min_gru_step_kernel<T, V>, dim3((p.width + 128 * V - 1) / (128 * V), B), dim3(128), 0, s, p);
-    else e = launch_pdl(min_gru_step_kernel<T, 1>, dim3((p.width + 127) / 128, B), dim3(128), 0, s, p);
+    if (vec) e = launch_pdl(min_gru_step_kernel<T, V>, dim3((p.width + 128 * V - 1) / (128 * V), B), dim3(128), 0, s, p, vec_o);
+    else e = launch_pdl(min_gru_step_kernel<T, 1>, dim3((p.width + 127) / 128, B), dim3(128), 0, s, p, 0);
   }
   if (e == cudaSuccess && (kinds & 2)) {
-    // two elements per lane where that still gives every SM a block
-    if (vec && (long long)B * ((p.width + 63) / 64) >= sm_count())
-      e = launch_pdl(min_gru_kernel<T, 2>, dim3((p.width + 63) / 64, B), dim3(kGruWarps * 32), 0, s, p);
-    else e = launch_pdl(min_gru_kernel<T, 1>, dim3((p.width + 31) / 32, B), dim3(kGruWarps * 32), 0, s, p);
+    if (p.pairs) {
+      if (vec) e = launch_pdl(min_gru_pairs_kernel<T, 2>, dim3((p.width + 127) / 128, B, p.parts), dim3(64), 0, s, p);
+      else e = launch_pdl(min_gru_pairs_kernel<T, 1>, dim3((p.width + 63) / 64, B, p.parts), dim3(64), 0, s, p);
+      if (e != cudaSuccess) return (int)e;
+    }
+    if (vec) e = launch_pdl(min_gru_kernel<T, 2>, dim3((p.width + 63) / 64, B, p.parts), dim3(kGruWarps * 32), 0, s, p, vec_o);
+    else e = launch_pdl(min_gru_kernel<T, 1>, dim3((p.width + 31) / 32, B, p.parts), dim3(kGruWarps * 32), 0, s, p, 0);
   }
   return (int)e;
 }
@@ -1262,9 +1590,10 @@ template <typename T, int KL, int R, int VPT, RecKind K>
 static int launch_stream(const RecParams& p, int B, cudaStream_t s) {
   constexpr int COLS = kRecWarps * (32 / KL) * VPT;
   const int slices = (p.dv + COLS - 1) / COLS;
-  const size_t smem = kRecHead + (size_t)kRecStages * kRecTok * ((K == DELTA ? 3 : 2) * R * KL + (K == GATED ? 0 : 4)) * 4;
+  const size_t smem = kRecHead + (size_t)kRecStages * kRecTok * ((K == DELTA ? 3 : 2) * R * KL + (K == GATED ? 0 : K == HDELTA ? kBlockCoef : 4)) * 4;
   void (*kern)(RecParams, int, int);
-  if constexpr (K == DELTA || K == HDELTA) kern = delta_stream_kernel<T, KL, R, VPT, K == HDELTA>;
+  if constexpr (K == DELTA) kern = delta_stream_kernel<T, KL, R, VPT>;
+  else if constexpr (K == HDELTA) kern = delta_block_kernel<T, KL, R, VPT>;
   else kern = state_space_stream_kernel<T, KL, R, VPT, K == GATED>;
   static PerDeviceOnce once;
   cudaError_t e = once.smem_limit(kern, 220 * 1024);
@@ -1276,7 +1605,8 @@ static int launch_stream(const RecParams& p, int B, cudaStream_t s) {
 template <typename T, int DKP, RecKind K>
 static int launch_long_runs(const RecParams& p, int B, cudaStream_t s) {
   const unsigned warps4 = (unsigned)(((long long)p.T * p.heads + 3) / 4);
-  if constexpr (K == DELTA || K == HDELTA) delta_records_kernel<T, DKP, K == HDELTA><<<warps4, 128, 0, s>>>(p);
+  if constexpr (K == DELTA) delta_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
+  else if constexpr (K == HDELTA) delta_block_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
   else if constexpr (K == GATED) gated_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
   else state_space_records_kernel<T, DKP><<<p.T, 128, 0, s>>>(p);
   const int e = (int)cudaGetLastError();
@@ -1303,7 +1633,7 @@ static int run_width(RecParams p, int B, int kinds, cudaStream_t s) {
 static int padded_dk(int dk) { return dk <= 32 ? 32 : dk <= 64 ? 64 : dk <= 128 ? 128 : dk <= 256 ? 256 : 512; }
 static long long record_bytes(RecKind kind, long long T, int heads, int groups, int dk) {
   const long long n = padded_dk(dk);
-  return 4 * (kind == DELTA ? heads * T * (3 * n + 4) : kind == HDELTA ? heads * T * (2 * n + 4) : kind == GATED ? heads * T * 2 * n : groups * T * 2 * n + heads * T * 4);
+  return 4 * (kind == DELTA ? heads * T * (3 * n + 4) : kind == HDELTA ? heads * T * (2 * n + kBlockCoef) : kind == GATED ? heads * T * 2 * n : groups * T * 2 * n + heads * T * 4);
 }
 
 template <typename T, RecKind K>
@@ -1373,17 +1703,35 @@ BLZ_API int blz_gated_linear(const void* q, long long ld_q, const void* f, long 
   return f32 ? run_rec<float, GATED>(p, B, kinds, ws_bytes, s) : run_rec<__nv_bfloat16, GATED>(p, B, kinds, ws_bytes, s);
 }
 
+// Workspace bytes of blz_min_gru for B sequences with up to max_q new tokens (0: none is needed): few long runs are cut into parts.
+BLZ_API long long blz_min_gru_ws_bytes(int B, int max_q, int width) {
+  using namespace blz;
+  const long long blocks = (long long)B * ((width + 63) / 64), parts = (max_q + kGruPart - 1) / kGruPart;
+  return parts < 2 || parts > 65535 || blocks >= 4LL * sm_count() ? 0 : (long long)B * width * (parts * 8 + 4);
+}
+
 // minGRU over every sequence of the batch: gate inputs z, candidates u and output gates g [T, ld] (runs of columns, width each), state
-// [rows][width] fp32; out [T, ld_out] (activation type) or null.  kinds: bit 0 = some sequences have one new token, bit 1 = some have more.
+// [rows][width] fp32; out [T, ld_out] (activation type) or null.  kinds: bit 0 = some sequences have one new token, bit 1 = some have more
+// (max_q at most).  ws: blz_min_gru_ws_bytes, or null.
 BLZ_API int blz_min_gru(const void* z, const void* u, const void* g, long long ld, float* state, void* out, long long ld_out, const int* slots,
-                        const int* q_start, const int* ctx_len, const int* no_store, int B, int width, int kinds, int f32, cudaStream_t s) {
+                        const int* q_start, const int* ctx_len, const int* no_store, int B, int width, int max_q, int kinds, void* ws, int f32,
+                        cudaStream_t s) {
   using namespace blz;
   if (B == 0) return 0;
-  if (B < 0 || B > 65535 || width < 1 || !z || !u || !g || !state) return (int)cudaErrorInvalidValue;
-  const GruParams p = {z, u, g, state, out, slots, q_start, ctx_len, no_store, ld, ld_out, width};
+  if (B < 0 || B > 65535 || width < 1 || max_q < 1 || !z || !u || !g || !state || (reinterpret_cast<uintptr_t>(ws) & 7))
+    return (int)cudaErrorInvalidValue;
+  GruParams p = {z, u, g, state, out, slots, q_start, ctx_len, no_store, ld, ld_out, width, nullptr, nullptr, max_q, 1};
+  if (ws) {
+    p.part = kGruPart;
+    p.parts = (max_q + kGruPart - 1) / kGruPart;
+    p.pairs = reinterpret_cast<float2*>(ws);
+    p.before = reinterpret_cast<float*>(p.pairs + (size_t)B * p.parts * width);
+    if (p.parts > 65535) return (int)cudaErrorInvalidValue;
+  }
   const uintptr_t bits = reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(u) | reinterpret_cast<uintptr_t>(g);
-  const int vec = bits % (f32 ? 16 : 8) == 0 && ld % 4 == 0 && width % 4 == 0;
-  return f32 ? run_gru<float>(p, B, kinds, vec, s) : run_gru<__nv_bfloat16>(p, B, kinds, vec, s);
+  const int unit = f32 ? 16 : 8, vec = bits % unit == 0 && ld % 4 == 0 && width % 4 == 0;
+  const int vec_o = reinterpret_cast<uintptr_t>(out) % unit == 0 && ld_out % 4 == 0;
+  return f32 ? run_gru<float>(p, B, kinds, vec, vec_o, s) : run_gru<__nv_bfloat16>(p, B, kinds, vec, vec_o, s);
 }
 
 // RMS norm of each of `groups` runs of n columns of fp32 rows, with a gate (GroupNormParams), to the activation type.

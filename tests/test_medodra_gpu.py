@@ -182,12 +182,12 @@ def test_min_gru(ops, width, dtype):
     from blaze_b200.models.qwen3 import Mixer, Recurrence
     spec, M, f32 = MinGruSpec(width), Mixer(), dtype == torch.float32
     M.rec = Recurrence(spec, "mingru", 1)
-    for pad, seqs in ((0, LENS), (3, LENS), (0, {b: 140 + b for b in range(8)})):
+    for pad, seqs in ((0, LENS), (3, LENS), (0, {b: 140 + b for b in range(8)}), (0, {0: 1600, 1: 700})):
         up = (width + 7) // 8 * 8 + pad
         M.cols = {"zg": pad, "u": up + pad, "g": 2 * up + pad}
         S = Sequences(LayerSpec(rec=spec), dtype)
         x = {b: (rnd(n, 3 * up + 8, seed=b) * 2).to(dtype) for b, n in seqs.items()}
-        got, portions = {b: [] for b in seqs}, SIZES if seqs is LENS else {b: [129, 1, 2] for b in seqs}
+        got, portions = {b: [] for b in seqs}, SIZES if seqs is LENS else {b: [n // 2 + 7, 1, 600 - b] for b, n in seqs.items()}
         for k, step in enumerate(schedule(seqs, portions, late=(2, 5))):
             proj = torch.cat([x[b][p:p + n] for b, p, n in step]).to(DEV)
             wide = torch.full((proj.shape[0], width + 8), 7.0, dtype=dtype, device=DEV)
