@@ -775,11 +775,15 @@ static constexpr int kConvPrepTok = 8;     // tokens per warp, at least the taps
 // A warp per (8 tokens of a sequence, head): a causal convolution over time of each projected channel, then queries (times their position's
 // temperature) to their buffer, keys and values (divided by their root mean square: unit_v) to their page.  The rows before the sequence's
 // new ones come from its state, which only the first 8 tokens' warp of a channel reads, and then writes.  TAPS: the real ones rounded up.
-template <typename T, int TAPS, int VEC>
+// ONCE: one turn of the warp takes a whole head (dim and vdim up to 32 * VEC), whose rows then stay in registers.
+template <typename T, int VEC> struct alignas(sizeof(T) * VEC) PrepVec { T e[VEC]; };
+
+template <typename T, int TAPS, int VEC, bool ONCE>
 __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) {
   pdl_trigger();
   pdl_wait();
   constexpr int IN = TAPS - 1 + kConvPrepTok;          // rows that the block's tokens need
+  using Vec = PrepVec<T, VEC>;
   const PrepParams& p = q.a;
   const int lane = threadIdx.x & 31, u = blockIdx.y * 4 + (threadIdx.x >> 5), b = blockIdx.z, t0 = blockIdx.x * kConvPrepTok;
   const int r0 = q.q_start[b], n = q.q_start[b + 1] - r0;
@@ -789,8 +793,8 @@ __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) 
   const int D = is_v ? p.vdim : p.dim, g = is_v ? u - p.heads - p.kv_heads : u - p.heads, taps = q.taps, m = min(kConvPrepTok, n - t0);
   const int C = p.heads * p.dim + p.kv_heads * (p.dim + p.vdim);
   const int ch = is_q ? u * p.dim : is_v ? p.heads * p.dim + p.kv_heads * p.dim + g * p.vdim : p.heads * p.dim + g * p.dim;     // first channel
-  const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)r0 * p.ld + (is_q ? p.q_off + (size_t)u * p.dim
-                                                                          : is_v ? p.v_off + (size_t)g * p.vdim : p.k_off + (size_t)g * p.dim);
+  const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)(r0 + t0) * p.ld + (is_q ? p.q_off + (size_t)u * p.dim
+                                                                               : is_v ? p.v_off + (size_t)g * p.vdim : p.k_off + (size_t)g * p.dim);
   T* st = reinterpret_cast<T*>(q.state) + (size_t)q.slots[b] * (taps - 1) * C + ch;
   const int dp = (p.dim + 15) / 16 * 16, vp = (p.vdim + 15) / 16 * 16;
   // lane k has token k's slot, and its query's factor
@@ -801,139 +805,125 @@ __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) 
     else if (q.temp_coef != 0.f)
       my_f = fmaf(q.temp_coef, logf(floorf(__fdiv_rn((float)(p.positions[r0 + t0 + lane] + 1), q.temp_every)) + 1.f), 1.f);
   }
-  auto load = [&](const T* at, float (&v)[VEC]) {
-    if constexpr (VEC == 4 && sizeof(T) == 2) {
-      const uint2 w = *reinterpret_cast<const uint2*>(at);
-      v[0] = __uint_as_float(w.x << 16); v[1] = __uint_as_float(w.x & 0xffff0000u);
-      v[2] = __uint_as_float(w.y << 16); v[3] = __uint_as_float(w.y & 0xffff0000u);
-    } else if constexpr (VEC == 4) {
-      const float4 w = *reinterpret_cast<const float4*>(at);
-      v[0] = w.x; v[1] = w.y; v[2] = w.z; v[3] = w.w;
-    } else {
-      v[0] = ad_ld(at);
-    }
-  };
-  auto store = [&](T* at, const float (&v)[VEC], float f) {
-    if constexpr (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(at) = make_uint2(pack_bf16x2(v[0] * f, v[1 % VEC] * f), pack_bf16x2(v[2 % VEC] * f, v[3 % VEC] * f));
-    else if constexpr (VEC == 4) *reinterpret_cast<float4*>(at) = make_float4(v[0] * f, v[1 % VEC] * f, v[2 % VEC] * f, v[3 % VEC] * f);
-    else ad_st(at, v[0] * f);
-  };
-  auto input = [&](int t, int c, float (&v)[VEC]) {     // projected columns c.. of the sequence's new token t (negative: before them)
-    if (t >= 0) {
-      load(src + (size_t)t * p.ld + c, v);
-    } else if (!fresh && t > -taps) {
-      load(st + (size_t)(taps - 1 + t) * C + c, v);
+  // projected columns c.. of the block's row i - (TAPS - 1): a new token's, one before the run's first (from the state), or none
+  auto input = [&](int i, int c) {
+    Vec v;
+    const int k = i - (TAPS - 1);
+    if (t0 + k >= 0) {
+      v = *reinterpret_cast<const Vec*>(src + (long long)k * p.ld + c);
+    } else if (!fresh && k > -taps) {
+      v = *reinterpret_cast<const Vec*>(st + (size_t)(taps - 1 + k) * C + c);
     } else {
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) v[j] = 0.f;
+      for (int j = 0; j < VEC; ++j) ad_st(v.e + j, 0.f);
     }
+    return v;
   };
-  const bool advance = t0 == 0 && taps > 1 && !(q.no_store != nullptr && q.no_store[b]);
-  // the state after the run, entry i the row taps - 1 - i before the next token; entries of a short run move up.  `in`: rows from
-  // 1 - TAPS on, all that a run of up to kConvPrepTok tokens can leave behind
-  auto leave = [&](int c, const float (&in)[IN][VEC]) {
-    if (n <= kConvPrepTok) {
-#pragma unroll
-      for (int k = 0; k < IN; ++k) {
-        const int i = k - (TAPS - 1) - n + taps - 1;
-        if (i >= 0 && i < taps - 1 && k < TAPS - 1 + n) store(st + (size_t)i * C + c, in[k], 1.f);
-      }
-    } else {
-      float v[TAPS][VEC];
-#pragma unroll
-      for (int i = 0; i < TAPS - 1; ++i)
-        if (i < taps - 1) load(src + (size_t)(n - (taps - 1) + i) * p.ld + c, v[i]);
-#pragma unroll
-      for (int i = 0; i < TAPS - 1; ++i)
-        if (i < taps - 1) store(st + (size_t)i * C + c, v[i], 1.f);
-    }
-  };
-  float y[kConvPrepTok][VEC], in[IN][VEC];
-  auto conv = [&](int c) {
-    float w[TAPS][VEC];
+  auto weights = [&](int c, float (&w)[TAPS][VEC]) {
 #pragma unroll
     for (int i = 0; i < TAPS; ++i) {
       const int r = i - (TAPS - taps);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) w[i][j] = 0.f;
       if (r < 0) continue;
-      const float* at = q.w + (size_t)r * C + ch + c;
-      if constexpr (VEC == 4) {
-        const float4 f = *reinterpret_cast<const float4*>(at);
-        w[i][0] = f.x; w[i][1] = f.y; w[i][2] = f.z; w[i][3] = f.w;
-      } else {
-        w[i][0] = *at;
-      }
-    }
+      const PrepVec<float, VEC> f = *reinterpret_cast<const PrepVec<float, VEC>*>(q.w + (size_t)r * C + ch + c);
 #pragma unroll
-    for (int i = 0; i < IN; ++i) {
-      if (i < TAPS - 1 + m) {
-        input(t0 + i - (TAPS - 1), c, in[i]);
-      } else {
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) in[i][j] = 0.f;
-      }
-    }
-#pragma unroll
-    for (int k = 0; k < kConvPrepTok; ++k) {
-      if (k >= m) break;
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) {
-        y[k][j] = 0.f;
-#pragma unroll
-        for (int i = 0; i < TAPS; ++i) y[k][j] = fmaf(w[i][j], in[k + i][j], y[k][j]);
-      }
+      for (int j = 0; j < VEC; ++j) w[i][j] = f.e[j];
     }
   };
-  const bool once = D <= 32 * VEC;                     // one turn of the warp takes the whole head
-  if (once && lane * VEC < D) conv(lane * VEC);
-  if (q.state_only) {
-    for (int c = lane * VEC; c < D && advance; c += 32 * VEC) {
-      if (!once) conv(c);
-      leave(c, in);
+  auto put = [&](int k, int c, const float (&y)[VEC], float f, int slot) {
+    T* dst;
+    if (is_q) {
+      dst = reinterpret_cast<T*>(p.q_out) + ((size_t)(r0 + t0 + k) * p.heads + u) * p.dim + c;
+    } else {
+      if (slot < 0) return;
+      dst = reinterpret_cast<T*>(p.pool) + (size_t)(slot >> 4) * p.page_stride + (size_t)g * p.head_stride +
+            (is_v ? 16 * dp + core_off(slot & 15, c, vp) : core_off(slot & 15, c, dp));
     }
-    return;
-  }
-  if (is_v && q.unit_v) {
-    float ss[kConvPrepTok];
+    Vec o;
 #pragma unroll
-    for (int k = 0; k < kConvPrepTok; ++k) ss[k] = 0.f;
-    for (int c = lane * VEC; c < D; c += 32 * VEC) {
-      if (!once) conv(c);
+    for (int j = 0; j < VEC; ++j) ad_st(o.e + j, y[j] * f);
+    *reinterpret_cast<Vec*>(dst) = o;
+  };
+  const bool advance = t0 == 0 && taps > 1 && !(q.no_store != nullptr && q.no_store[b]);
+  if constexpr (ONCE) {
+    const int c = lane * VEC;
+    const bool live = c < D;
+    Vec in[IN];
+    float w[TAPS][VEC];
+    if (live) {
 #pragma unroll
-      for (int k = 0; k < kConvPrepTok; ++k) {
-        if (k >= m) break;
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) ss[k] = fmaf(y[k][j], y[k][j], ss[k]);
-      }
+      for (int i = 0; i < IN; ++i)
+        if (i < TAPS - 1 + m) in[i] = input(i, c);
+      if (!q.state_only) weights(c, w);
     }
 #pragma unroll
     for (int k = 0; k < kConvPrepTok; ++k) {
-      if (k >= m) break;
-      const float f = 1.f / sqrtf(warp_sum(ss[k]) / (float)D + p.eps);
-      if (lane == k) my_f = f;
+      if (k >= m || q.state_only) break;
+      float y[VEC];
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        y[j] = 0.f;
+        if (live)
+#pragma unroll
+          for (int i = 0; i < TAPS; ++i) y[j] = fmaf(w[i][j], ad_ld(in[k + i].e + j), y[j]);
+      }
+      float f = __shfl_sync(0xffffffffu, my_f, k);
+      if (is_v && q.unit_v) {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) ss = fmaf(y[j], y[j], ss);
+        f = 1.f / sqrtf(warp_sum(ss) / (float)D + p.eps);
+      }
+      const int slot = __shfl_sync(0xffffffffu, my_slot, k);
+      if (live) put(k, c, y, f, slot);
     }
-  }
-  float f[kConvPrepTok];
-  int slot[kConvPrepTok];
+    if (!advance || !live) return;
+    // the state after the run, entry i the row taps - 1 - i before the next token; entries of a short run move up
+    if (n <= kConvPrepTok) {
 #pragma unroll
-  for (int k = 0; k < kConvPrepTok; ++k) {
-    f[k] = __shfl_sync(0xffffffffu, my_f, k);
-    slot[k] = __shfl_sync(0xffffffffu, my_slot, k);
-  }
-  for (int c = lane * VEC; c < D; c += 32 * VEC) {
-    if (!once) conv(c);
+      for (int k = 0; k < IN; ++k) {
+        const int i = k - (TAPS - 1) - n + taps - 1;
+        if (i >= 0 && i < taps - 1) *reinterpret_cast<Vec*>(st + (size_t)i * C + c) = in[k];
+      }
+    } else {
+      for (int i = 0; i < taps - 1; ++i)
+        *reinterpret_cast<Vec*>(st + (size_t)i * C + c) = *reinterpret_cast<const Vec*>(src + (size_t)(n - (taps - 1) + i) * p.ld + c);
+    }
+  } else {
+    auto conv = [&](int k, int c, float (&y)[VEC]) {
+      float w[TAPS][VEC];
+      weights(c, w);
 #pragma unroll
-    for (int k = 0; k < kConvPrepTok; ++k) {
-      if (k >= m) break;
-      if (is_q) {
-        store(reinterpret_cast<T*>(p.q_out) + ((size_t)(r0 + t0 + k) * p.heads + u) * p.dim + c, y[k], f[k]);
-      } else if (slot[k] >= 0) {
-        T* page = reinterpret_cast<T*>(p.pool) + (size_t)(slot[k] >> 4) * p.page_stride + (size_t)g * p.head_stride;
-        store(page + (is_v ? 16 * dp + core_off(slot[k] & 15, c, vp) : core_off(slot[k] & 15, c, dp)), y[k], f[k]);
+      for (int j = 0; j < VEC; ++j) y[j] = 0.f;
+#pragma unroll
+      for (int i = 0; i < TAPS; ++i) {
+        const Vec v = input(k + i, c);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) y[j] = fmaf(w[i][j], ad_ld(v.e + j), y[j]);
+      }
+    };
+    for (int k = 0; k < m && !q.state_only; ++k) {
+      float f = __shfl_sync(0xffffffffu, my_f, k), y[VEC];
+      const int slot = __shfl_sync(0xffffffffu, my_slot, k);
+      if (is_v && q.unit_v) {
+        float ss = 0.f;
+        for (int c = lane * VEC; c < D; c += 32 * VEC) {
+          conv(k, c, y);
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) ss = fmaf(y[j], y[j], ss);
+        }
+        f = 1.f / sqrtf(warp_sum(ss) / (float)D + p.eps);
+      }
+      for (int c = lane * VEC; c < D; c += 32 * VEC) {
+        conv(k, c, y);
+        put(k, c, y, f, slot);
       }
     }
-    if (advance) leave(c, in);
+    if (!advance) return;
+    for (int c = lane * VEC; c < D; c += 32 * VEC)
+      for (int i = 0; i < taps - 1; ++i)               // ascending: an entry is read before it is written over
+        *reinterpret_cast<Vec*>(st + (size_t)i * C + c) = input(TAPS - 1 + n - (taps - 1) + i, c);
   }
 }
 
@@ -941,8 +931,10 @@ template <typename T, int TAPS>
 static int launch_conv_prep(const ConvPrepParams& q, bool vec, int B, int max_q, cudaStream_t s) {
   const PrepParams& p = q.a;
   const dim3 grid((max_q + kConvPrepTok - 1) / kConvPrepTok, (p.heads + 2 * p.kv_heads + 3) / 4, B);
-  if (vec) return (int)launch_pdl(conv_prep_pages_kernel<T, TAPS, 4>, grid, dim3(128), 0, s, q);
-  return (int)launch_pdl(conv_prep_pages_kernel<T, TAPS, 1>, grid, dim3(128), 0, s, q);
+  const int D = p.dim > p.vdim ? p.dim : p.vdim;
+  if (vec && D <= 128) return (int)launch_pdl(conv_prep_pages_kernel<T, TAPS, 4, true>, grid, dim3(128), 0, s, q);
+  if (vec) return (int)launch_pdl(conv_prep_pages_kernel<T, TAPS, 4, false>, grid, dim3(128), 0, s, q);
+  return (int)launch_pdl(conv_prep_pages_kernel<T, TAPS, 1, false>, grid, dim3(128), 0, s, q);
 }
 
 static MapsParams soft_params(const void* q, long long ld, void* out, long long ld_out, void* pool, long long page_stride, long long head_stride,

@@ -614,10 +614,13 @@ template <typename T, int DKP>
 __global__ void __launch_bounds__(128) delta_block_records_kernel(RecParams p) {
   constexpr int REC = 2 * DKP + kBlockCoef, NV = DKP / 32;
   const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-  const int t = (int)(w / p.heads), h = (int)(w % p.heads), lane = threadIdx.x & 31;
-  if (t >= p.T || !in_long_run(p, t)) return;
+  const int h = (int)(w % p.heads), lane = threadIdx.x & 31;
+  // the block that starts in these rows: of a sequence that goes on through all of them exactly one does, and a warp whose rows see
+  // one sequence end and another begin takes both of theirs in turn
+  for (int t = (int)(w / p.heads) * kBlockTok, end = min(t + kBlockTok, p.T); t < end; ++t) {
+  if (!in_long_run(p, t)) continue;
   const int seq = p.seq_of_row[t], rest = p.q_start[seq + 1] - t, m = min(kBlockTok, rest);
-  if ((t - p.q_start[seq]) % kBlockTok) return;            // the block's first row has the whole block
+  if ((t - p.q_start[seq]) % kBlockTok) continue;
   const int dk = p.dk, hk = h / (p.heads / p.groups);
   float q[kBlockTok][NV], k[kBlockTok][NV], beta[kBlockTok], g[kBlockTok];
 #pragma unroll
@@ -680,6 +683,7 @@ __global__ void __launch_bounds__(128) delta_block_records_kernel(RecParams p) {
       f[2] = make_float4(beta[i], beta[i] * G, G, last);
       f[3] = make_float4(all, 0.f, 0.f, 0.f);
     }
+  }
   }
 }
 
@@ -949,8 +953,9 @@ template <typename T, int KL, int R, int VPT>
 __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) delta_block_kernel(RecParams p, int slices, int vec_v) {
   constexpr int DKP = R * KL, CG = 32 / KL, COLS = kRecWarps * CG * VPT, REC = 2 * DKP + kBlockCoef, STAGE = kRecTok * REC;
   constexpr bool KEEP_K = R <= 8;                   // registers for the block's keys
+  constexpr int VC = sizeof(T) * VPT < 4 ? 2 : VPT; // v columns that a lane brings: at least 4 bytes
   extern __shared__ __align__(128) uint8_t sm8[];
-  __shared__ __align__(16) T s_v[kRecWarps][kColsAhead + 1][kRecTok][CG * VPT];
+  __shared__ __align__(16) T s_v[kRecWarps][kColsAhead + 1][kRecTok][CG * VC];
   const int b = blockIdx.x / slices, slice = blockIdx.x % slices, h = blockIdx.y;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, slot = p.slots[b], ctx = p.ctx_len[b];
   if (n < p.long_rows) return;
@@ -975,10 +980,11 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
   const bool vec = dv % 4 == 0;
   float S[R][VPT];
   load_state<KL, R, VPT>(S, st, kl, col, dk, dv, ctx == n, vec);
-  const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + (kl & 7)) * p.ld_conv + (size_t)2 * p.groups * dk + (size_t)h * dv + col;
+  const int vcol = VC > VPT ? col & ~1 : col;
+  const T* vsrc = reinterpret_cast<const T*>(p.conv) + (size_t)(r0 + (kl & 7)) * p.ld_conv + (size_t)2 * p.groups * dk + (size_t)h * dv + vcol;
   auto send_group = [&](int c) {
-    send_cols<T, VPT>(&s_v[warp][c % (kColsAhead + 1)][kl & 7][cg * VPT], vsrc + (size_t)c * kRecTok * p.ld_conv,
-                      kl < kRecTok && c * kRecTok + kl < n, col, dv, vec_v);
+    send_cols<T, VC>(&s_v[warp][c % (kColsAhead + 1)][kl & 7][cg * VC], vsrc + (size_t)c * kRecTok * p.ld_conv,
+                     kl < kRecTok && c * kRecTok + kl < n, vcol, dv, vec_v);
   };
 #pragma unroll
   for (int c = 0; c < kColsAhead; ++c) send_group(c);
@@ -989,7 +995,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
     __syncwarp();                            // the last group's columns have been read
     send_group(c + kColsAhead);
     wait_cols();
-    const T(*cols)[CG * VPT] = s_v[warp][c % (kColsAhead + 1)];
+    const T(*cols)[CG * VC] = s_v[warp][c % (kColsAhead + 1)];
     ok = rr.wait_full(c);
     if (!ok) break;
     __syncwarp();
@@ -1030,7 +1036,7 @@ __global__ void __launch_bounds__((kRecWarps + 1) * 32, R * VPT <= 64 ? 2 : 1) d
       float u[VPT], o[VPT], uu[kBlockTok][VPT];
 #pragma unroll
       for (int v = 0; v < VPT; ++v) {
-        u[v] = fmaf(s4.x, rc_ld(&cols[j0 + my][cg * VPT + v]), -s4.y * pk[0][v]);
+        u[v] = fmaf(s4.x, rc_ld(&cols[j0 + my][cg * VC + (VC > VPT ? col & 1 : v)]), -s4.y * pk[0][v]);
         o[v] = s4.z * pq[0][v];
       }
 #pragma unroll
@@ -1319,14 +1325,15 @@ struct GruParams {
   int part, parts;             // tokens per part, parts of the longest run
 };
 static constexpr int kGruWarps = 8, kGruTok = 8;       // a block takes kGruWarps * kGruTok tokens at a time
-static constexpr int kGruPart = 256;
+static constexpr int kGruPart = 512;
 
 // a gate; bf16: the special function unit's reciprocal (two units in the last place)
 template <typename T>
 __device__ __forceinline__ float gru_sigmoid(float x) {
   if constexpr (sizeof(T) == 4) return 1.f / (1.f + expf(-x));
   float r;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + __expf(-x)));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x * -1.4426950408889634f));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + r));
   return r;
 }
 template <typename T>
@@ -1346,9 +1353,10 @@ __device__ __forceinline__ GruVec<T, VEC> gru_load(const void* base, size_t at) 
   else v.e[0] = *p;
   return v;
 }
-// vec: the output's rows allow VEC elements as one word
+// vec: the output's rows allow VEC elements as one word; left: elements of the row from c on
 template <typename T, int VEC>
-__device__ __forceinline__ void gru_store(const GruParams& p, size_t row, int c, const GruVec<T, VEC>& g, const float (&S)[VEC], bool vec) {
+__device__ __forceinline__ void gru_store(const GruParams& p, size_t row, int c, const GruVec<T, VEC>& g, const float (&S)[VEC], bool vec,
+                                          int left = VEC) {
   T* o = reinterpret_cast<T*>(p.out) + row * p.ld_out + c;
   GruVec<T, VEC> y;
 #pragma unroll
@@ -1357,11 +1365,12 @@ __device__ __forceinline__ void gru_store(const GruParams& p, size_t row, int c,
     if constexpr (sizeof(T) == 4) y.e[j] = v;
     else y.e[j] = __float2bfloat16(v);
   }
-  if (vec) {
+  if (vec && left >= VEC) {
     *reinterpret_cast<GruVec<T, VEC>*>(o) = y;
   } else {
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) o[j] = y.e[j];
+    for (int j = 0; j < VEC; ++j)
+      if (j < left) o[j] = y.e[j];
   }
 }
 
@@ -1390,154 +1399,137 @@ __global__ void __launch_bounds__(128) min_gru_step_kernel(GruParams p, int vec)
   for (int j = 0; j < VEC; ++j) st[j] = S[j];
 }
 
-// what a part of a run does to the state, for parts that blocks of their own take (see GruParams::pairs); a thread per VEC elements
-template <typename T, int VEC>
-__global__ void __launch_bounds__(64) min_gru_pairs_kernel(GruParams p) {
-  pdl_trigger();
-  pdl_wait();
-  const int b = blockIdx.y, i = blockIdx.z, c = (blockIdx.x * 64 + threadIdx.x) * VEC;
-  const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, t0 = i * p.part, t1 = min(n, t0 + p.part);
-  if (n <= 1 || c >= p.width || t0 >= n) return;
-  const bool fresh = p.ctx_len[b] == n;
-  float A[VEC], B[VEC];
-#pragma unroll
-  for (int j = 0; j < VEC; ++j) { A[j] = 1.f; B[j] = 0.f; }
-  if (i == 0) {
-#pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-      B[j] = fresh ? 0.f : p.state[(size_t)p.slots[b] * p.width + c + j];
-      p.before[(size_t)b * p.width + c + j] = B[j];
-    }
-  }
-  for (int t = t0; t < t1; t += kGruTok) {
-    GruVec<T, VEC> z[kGruTok], u[kGruTok];
-#pragma unroll
-    for (int k = 0; k < kGruTok; ++k)
-      if (t + k < t1) {
-        const size_t at = (size_t)(r0 + t + k) * p.ld + c;
-        z[k] = gru_load<T, VEC>(p.z, at);
-        u[k] = gru_load<T, VEC>(p.u, at);
-      }
-#pragma unroll
-    for (int k = 0; k < kGruTok; ++k)
-      if (t + k < t1)
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) {
-          float keep, add;
-          gru_gate<T>(rc_ld(z[k].e + j), rc_ld(u[k].e + j), keep, add);
-          A[j] *= keep;
-          B[j] = fmaf(keep, B[j], add);
-        }
-  }
-  float2* to = p.pairs + ((size_t)b * p.parts + i) * p.width + c;
-#pragma unroll
-  for (int j = 0; j < VEC; ++j) to[j] = make_float2(A[j], B[j]);
-}
+// Runs: a block takes 128 bytes of a row's elements (VEC per lane) over a run, or over a part of it.  Rows come in tiles of kGruWarps *
+// kGruTok tokens through a ring in shared memory.  Each warp folds its kGruTok tokens into one pair (factor, addend) per element; the pairs of
+// the warps before it and the carry give the state its own tokens start from.  PAIRS: the carry is a pair itself and is all that is
+// written (see GruParams::pairs); else the outputs and, by the last part, the state.
+static constexpr int kGruStages = 3, kGruTile = kGruWarps * kGruTok;
 
-// longer runs: a block per 32 * VEC elements of a sequence (and per part of it).  Each warp folds kGruTok tokens into one pair (factor,
-// addend) per element; the pairs of the warps before it and the carry give the state its own tokens start from.  The next tokens are
-// fetched meanwhile.
-template <typename T, int VEC>
-__global__ void __launch_bounds__(kGruWarps * 32, 2) min_gru_kernel(GruParams p, int vec) {
-  __shared__ float2 s_p[2][kGruWarps][32 * VEC];
-  __shared__ float s_c[2][32 * VEC];
+template <typename T, bool PAIRS>
+__global__ void __launch_bounds__(kGruWarps * 32, 3) min_gru_kernel(GruParams p, int vec, int vec_o) {
+  constexpr int VEC = 4 / sizeof(T), COLS = 32 * VEC, ARRS = PAIRS ? 2 : 3, CHUNK = 16 / sizeof(T);
+  extern __shared__ __align__(128) uint8_t sm8[];                // [stages][z | u | g][tile][COLS]
+  __shared__ float2 s_p[kGruWarps][COLS], s_c[2][COLS];
   pdl_trigger();
   pdl_wait();
-  const int b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, c = (blockIdx.x * 32 + lane) * VEC;
+  const int b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, c0 = blockIdx.x * COLS, c = c0 + lane * VEC;
   const int r0 = p.q_start[b], n = p.q_start[b + 1] - r0, from = blockIdx.z * p.part, to = min(n, from + p.part);
   if (n <= 1 || from >= n) return;
+  T* ring = reinterpret_cast<T*>(sm8);
+  const int tiles = (to - from + kGruTile - 1) / kGruTile;
+  auto fill = [&](int i) {
+    if (i < tiles) {
+      T* dst = ring + (size_t)(i % kGruStages) * ARRS * kGruTile * COLS;
+      for (int x = threadIdx.x; x < ARRS * kGruTile * 8; x += kGruWarps * 32) {
+        const int part = x & 7, row = x >> 3, t = from + i * kGruTile + row % kGruTile, a = row / kGruTile, col = c0 + part * CHUNK;
+        const T* src = reinterpret_cast<const T*>(a == 0 ? p.z : a == 1 ? p.u : p.g) + (size_t)(r0 + min(t, to - 1)) * p.ld + col;
+        T* at = dst + row * COLS + part * CHUNK;
+        if (vec) {
+          const int bytes = t < to ? max(min((p.width - col) * (int)sizeof(T), 16), 0) : 0;
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(at)), "l"(bytes ? (const void*)src : p.z), "r"(bytes) : "memory");
+        } else {
+#pragma unroll
+          for (int e = 0; e < CHUNK; ++e)
+            if (t < to && col + e < p.width) at[e] = src[e];
+        }
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+#pragma unroll
+  for (int i = 0; i < kGruStages; ++i) fill(i);
   const bool live = c < p.width;
   float* st = p.state + (size_t)p.slots[b] * p.width + c;
   const bool fresh = p.ctx_len[b] == n;
-  GruVec<T, VEC> z[kGruTok], u[kGruTok], g[kGruTok];
-  auto fetch = [&](int t0) {
-#pragma unroll
-    for (int k = 0; k < kGruTok; ++k)
-      if (live && t0 + k < to) {
-        const size_t at = (size_t)(r0 + t0 + k) * p.ld + c;
-        z[k] = gru_load<T, VEC>(p.z, at);
-        u[k] = gru_load<T, VEC>(p.u, at);
-        if (p.out) g[k] = gru_load<T, VEC>(p.g, at);
-      }
-  };
-  fetch(from + warp * kGruTok);
-  float S[VEC];
-#pragma unroll
-  for (int j = 0; j < VEC; ++j) S[j] = 0.f;
   if (warp == 0) {
-    if (live) {
-      if (!p.pairs) {
+    // the carry: of a part's pair the state before the run in its addend, or nothing; else the state
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) S[j] = fresh ? 0.f : st[j];
-      } else if (blockIdx.z == 0) {
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) S[j] = p.before[(size_t)b * p.width + c + j];
-      } else {
-        const float2* pr = p.pairs + (size_t)b * p.parts * p.width + c;
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) S[j] = pr[j].y;
+    for (int j = 0; j < VEC; ++j) {
+      float S = 0.f;
+      if (c + j < p.width) {
+        if (PAIRS || !p.pairs) {
+          if (blockIdx.z == 0 && !fresh) S = st[j];
+          if (PAIRS && blockIdx.z == 0) p.before[(size_t)b * p.width + c + j] = S;
+        } else if (blockIdx.z == 0) {
+          S = p.before[(size_t)b * p.width + c + j];
+        } else {
+          const float2* pr = p.pairs + (size_t)b * p.parts * p.width + c + j;
+          S = pr->y;
 #pragma unroll 8
-        for (int i = 1; i < blockIdx.z; ++i)
-#pragma unroll
-          for (int j = 0; j < VEC; ++j) {
-            const float2 f = pr[(size_t)i * p.width + j];
-            S[j] = fmaf(f.x, S[j], f.y);
+          for (int i = 1; i < blockIdx.z; ++i) {
+            const float2 f = pr[(size_t)i * p.width];
+            S = fmaf(f.x, S, f.y);
           }
+        }
       }
+      s_c[0][lane * VEC + j] = make_float2(1.f, S);
     }
-#pragma unroll
-    for (int j = 0; j < VEC; ++j) s_c[0][lane * VEC + j] = S[j];
   }
-  constexpr int STEP = kGruWarps * kGruTok;
-  for (int i = 0, base = from; base < to; ++i, base += STEP) {
-    const int t0 = base + warp * kGruTok, par = i & 1;
+  float S[VEC];
+  for (int i = 0; i < tiles; ++i) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(kGruStages - 1) : "memory");
+    __syncthreads();
+    const T* tile = ring + (size_t)(i % kGruStages) * ARRS * kGruTile * COLS + (size_t)warp * kGruTok * COLS + lane * VEC;
+    const int t0 = from + i * kGruTile + warp * kGruTok;
     float keep[kGruTok][VEC], add[kGruTok][VEC], A[VEC], B[VEC];
-    GruVec<T, VEC> gate[kGruTok];
+    GruVec<T, VEC> gate[PAIRS ? 1 : kGruTok];
 #pragma unroll
     for (int j = 0; j < VEC; ++j) { A[j] = 1.f; B[j] = 0.f; }
 #pragma unroll
     for (int k = 0; k < kGruTok; ++k) {
-      gate[k] = g[k];
+      const GruVec<T, VEC> z = *reinterpret_cast<const GruVec<T, VEC>*>(tile + k * COLS), u = *reinterpret_cast<const GruVec<T, VEC>*>(tile + (kGruTile + k) * COLS);
+      if constexpr (!PAIRS) gate[k] = *reinterpret_cast<const GruVec<T, VEC>*>(tile + (2 * kGruTile + k) * COLS);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) {
-        keep[k][j] = 1.f;
-        add[k][j] = 0.f;
-        if (live && t0 + k < to) gru_gate<T>(rc_ld(z[k].e + j), rc_ld(u[k].e + j), keep[k][j], add[k][j]);
+        gru_gate<T>(rc_ld(z.e + j), rc_ld(u.e + j), keep[k][j], add[k][j]);
+        if (t0 + k >= to) { keep[k][j] = 1.f; add[k][j] = 0.f; }          // beyond the run: nothing changes
         A[j] *= keep[k][j];
         B[j] = fmaf(keep[k][j], B[j], add[k][j]);
       }
     }
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) s_p[par][warp][lane * VEC + j] = make_float2(A[j], B[j]);
-    fetch(t0 + STEP);
+    for (int j = 0; j < VEC; ++j) s_p[warp][lane * VEC + j] = make_float2(A[j], B[j]);
     __syncthreads();
+    float2 carry[VEC];
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) S[j] = s_c[par][lane * VEC + j];
+    for (int j = 0; j < VEC; ++j) carry[j] = s_c[i & 1][lane * VEC + j];
 #pragma unroll
     for (int w = 0; w < kGruWarps - 1; ++w)
       if (w < warp)
 #pragma unroll
         for (int j = 0; j < VEC; ++j) {
-          const float2 f = s_p[par][w][lane * VEC + j];
-          S[j] = fmaf(f.x, S[j], f.y);
+          const float2 f = s_p[w][lane * VEC + j];
+          carry[j] = make_float2(f.x * carry[j].x, fmaf(f.x, carry[j].y, f.y));
         }
-    if (warp == kGruWarps - 1)               // the state after these tokens, as soon as it is known
+    if (warp == kGruWarps - 1)               // the carry after these tokens, as soon as it is known
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) s_c[par ^ 1][lane * VEC + j] = fmaf(A[j], S[j], B[j]);
+      for (int j = 0; j < VEC; ++j) s_c[(i + 1) & 1][lane * VEC + j] = make_float2(A[j] * carry[j].x, fmaf(A[j], carry[j].y, B[j]));
+    fill(i + kGruStages);                    // every warp has read this tile
+    if constexpr (!PAIRS) {
 #pragma unroll
-    for (int k = 0; k < kGruTok; ++k) {
+      for (int j = 0; j < VEC; ++j) S[j] = carry[j].y;
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) S[j] = fmaf(keep[k][j], S[j], add[k][j]);
-      if (p.out && live && t0 + k < to) gru_store<T, VEC>(p, r0 + t0 + k, c, gate[k], S, vec);
+      for (int k = 0; k < kGruTok; ++k) {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) S[j] = fmaf(keep[k][j], S[j], add[k][j]);
+        if (p.out && live && t0 + k < to) gru_store<T, VEC>(p, r0 + t0 + k, c, gate[k], S, vec_o, p.width - c);
+      }
     }
   }
-  if (to < n || warp != kGruWarps - 1 || !live || (p.no_store != nullptr && p.no_store[b])) return;
+  if (warp != kGruWarps - 1 || !live) return;
+  if constexpr (PAIRS) {
 #pragma unroll
-  for (int j = 0; j < VEC; ++j) st[j] = S[j];          // tokens beyond the run changed nothing
+    for (int j = 0; j < VEC; ++j)
+      if (c + j < p.width) p.pairs[((size_t)b * p.parts + blockIdx.z) * p.width + c + j] = s_c[tiles & 1][lane * VEC + j];
+  } else if (to == n && !(p.no_store != nullptr && p.no_store[b])) {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j)
+      if (c + j < p.width) st[j] = S[j];     // tokens beyond the run changed nothing
+  }
 }
 
 template <typename T>
-static int run_gru(GruParams p, int B, int kinds, int vec, int vec_o, cudaStream_t s) {
+static int run_gru(const GruParams& p, int B, int kinds, int vec, int vec16, int vec_o, cudaStream_t s) {
   cudaError_t e = cudaSuccess;
   if (kinds & 1) {
     constexpr int V = 4;
@@ -1545,13 +1537,17 @@ static int run_gru(GruParams p, int B, int kinds, int vec, int vec_o, cudaStream
     else e = launch_pdl(min_gru_step_kernel<T, 1>, dim3((p.width + 127) / 128, B), dim3(128), 0, s, p, 0);
   }
   if (e == cudaSuccess && (kinds & 2)) {
+    constexpr int COLS = 128 / sizeof(T);
+    constexpr size_t tile = (size_t)kGruStages * kGruTile * 128;          // per array
+    const dim3 grid((p.width + COLS - 1) / COLS, B, p.parts), block(kGruWarps * 32);
+    static PerDeviceOnce once, once_pairs;
     if (p.pairs) {
-      if (vec) e = launch_pdl(min_gru_pairs_kernel<T, 2>, dim3((p.width + 127) / 128, B, p.parts), dim3(64), 0, s, p);
-      else e = launch_pdl(min_gru_pairs_kernel<T, 1>, dim3((p.width + 63) / 64, B, p.parts), dim3(64), 0, s, p);
+      e = once_pairs.smem_limit(min_gru_kernel<T, true>, 2 * tile);
+      if (e == cudaSuccess) e = launch_pdl(min_gru_kernel<T, true>, grid, block, 2 * tile, s, p, vec16, 0);
       if (e != cudaSuccess) return (int)e;
     }
-    if (vec) e = launch_pdl(min_gru_kernel<T, 2>, dim3((p.width + 63) / 64, B, p.parts), dim3(kGruWarps * 32), 0, s, p, vec_o);
-    else e = launch_pdl(min_gru_kernel<T, 1>, dim3((p.width + 31) / 32, B, p.parts), dim3(kGruWarps * 32), 0, s, p, 0);
+    e = once.smem_limit(min_gru_kernel<T, false>, 3 * tile);
+    if (e == cudaSuccess) e = launch_pdl(min_gru_kernel<T, false>, grid, block, 3 * tile, s, p, vec16, vec_o);
   }
   return (int)e;
 }
@@ -1606,7 +1602,8 @@ template <typename T, int DKP, RecKind K>
 static int launch_long_runs(const RecParams& p, int B, cudaStream_t s) {
   const unsigned warps4 = (unsigned)(((long long)p.T * p.heads + 3) / 4);
   if constexpr (K == DELTA) delta_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
-  else if constexpr (K == HDELTA) delta_block_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
+  else if constexpr (K == HDELTA)
+    delta_block_records_kernel<T, DKP><<<(unsigned)(((long long)((p.T + kBlockTok - 1) / kBlockTok) * p.heads + 3) / 4), 128, 0, s>>>(p);
   else if constexpr (K == GATED) gated_records_kernel<T, DKP><<<warps4, 128, 0, s>>>(p);
   else state_space_records_kernel<T, DKP><<<p.T, 128, 0, s>>>(p);
   const int e = (int)cudaGetLastError();
@@ -1707,7 +1704,7 @@ BLZ_API int blz_gated_linear(const void* q, long long ld_q, const void* f, long 
 BLZ_API long long blz_min_gru_ws_bytes(int B, int max_q, int width) {
   using namespace blz;
   const long long blocks = (long long)B * ((width + 63) / 64), parts = (max_q + kGruPart - 1) / kGruPart;
-  return parts < 2 || parts > 65535 || blocks >= 4LL * sm_count() ? 0 : (long long)B * width * (parts * 8 + 4);
+  return parts < 2 || parts > 65535 || blocks >= sm_count() ? 0 : (long long)B * width * (parts * 8 + 4);
 }
 
 // minGRU over every sequence of the batch: gate inputs z, candidates u and output gates g [T, ld] (runs of columns, width each), state
@@ -1729,9 +1726,9 @@ BLZ_API int blz_min_gru(const void* z, const void* u, const void* g, long long l
     if (p.parts > 65535) return (int)cudaErrorInvalidValue;
   }
   const uintptr_t bits = reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(u) | reinterpret_cast<uintptr_t>(g);
-  const int unit = f32 ? 16 : 8, vec = bits % unit == 0 && ld % 4 == 0 && width % 4 == 0;
+  const int unit = f32 ? 16 : 8, vec = bits % unit == 0 && ld % 4 == 0 && width % 4 == 0, vec16 = bits % 16 == 0 && ld % (f32 ? 4 : 8) == 0;
   const int vec_o = reinterpret_cast<uintptr_t>(out) % unit == 0 && ld_out % 4 == 0;
-  return f32 ? run_gru<float>(p, B, kinds, vec, vec_o, s) : run_gru<__nv_bfloat16>(p, B, kinds, vec, vec_o, s);
+  return f32 ? run_gru<float>(p, B, kinds, vec, vec16, vec_o, s) : run_gru<__nv_bfloat16>(p, B, kinds, vec, vec16, vec_o, s);
 }
 
 // RMS norm of each of `groups` runs of n columns of fp32 rows, with a gate (GroupNormParams), to the activation type.
