@@ -849,34 +849,57 @@ __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) 
   if constexpr (ONCE) {
     const int c = lane * VEC;
     const bool live = c < D;
-    Vec in[IN];
-    float w[TAPS][VEC];
-    if (live) {
+    Vec in[IN];                                        // as they are: all reads go out before the first is used
+    float w[TAPS][VEC], x[IN][VEC];
+    const int cc = live ? c : 0;
+    if (t0 >= TAPS - 1 && m == kConvPrepTok) {         // every row is a new token's
+      const T* at = src - (TAPS - 1) * p.ld + cc;
 #pragma unroll
-      for (int i = 0; i < IN; ++i)
-        if (i < TAPS - 1 + m) in[i] = input(i, c);
-      if (!q.state_only) weights(c, w);
+      for (int i = 0; i < IN; ++i, at += p.ld) in[i] = *reinterpret_cast<const Vec*>(at);
+    } else {
+#pragma unroll
+      for (int i = 0; i < IN; ++i) in[i] = input(min(i, TAPS - 2 + m), cc);
     }
+    if (!q.state_only) weights(cc, w);
+#pragma unroll
+    for (int i = 0; i < IN; ++i)
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) x[i][j] = ad_ld(in[i].e + j);
+    // where this lane's columns of the tokens go: a row of the query buffer, or a place in the page that a token's slot adds to
+    T* base = is_q ? reinterpret_cast<T*>(p.q_out) + ((size_t)(r0 + t0) * p.heads + u) * p.dim + cc
+                   : reinterpret_cast<T*>(p.pool) + (size_t)g * p.head_stride + (is_v ? 16 * dp : 0) + (cc >> 3) * 64 + (cc & 7);
+    const long long row = is_q ? (long long)p.heads * p.dim : 0;
+    // lane k: offset of token k's slot (-1: none)
+    const int pad8 = 8 * (is_v ? vp : dp);
+    const long long my_at = is_q ? (long long)lane * row : my_slot < 0 ? -1 : (my_slot >> 4) * p.page_stride + (my_slot >> 3 & 1) * pad8 + (my_slot & 7) * 8;
 #pragma unroll
     for (int k = 0; k < kConvPrepTok; ++k) {
       if (k >= m || q.state_only) break;
       float y[VEC];
 #pragma unroll
       for (int j = 0; j < VEC; ++j) {
-        y[j] = 0.f;
-        if (live)
+        y[j] = w[0][j] * x[k][j];
 #pragma unroll
-          for (int i = 0; i < TAPS; ++i) y[j] = fmaf(w[i][j], ad_ld(in[k + i].e + j), y[j]);
+        for (int i = 1; i < TAPS; ++i) y[j] = fmaf(w[i][j], x[k + i][j], y[j]);
       }
       float f = __shfl_sync(0xffffffffu, my_f, k);
       if (is_v && q.unit_v) {
         float ss = 0.f;
 #pragma unroll
         for (int j = 0; j < VEC; ++j) ss = fmaf(y[j], y[j], ss);
-        f = 1.f / sqrtf(warp_sum(ss) / (float)D + p.eps);
+        f = 1.f / sqrtf(warp_sum(live ? ss : 0.f) / (float)D + p.eps);
       }
-      const int slot = __shfl_sync(0xffffffffu, my_slot, k);
-      if (live) put(k, c, y, f, slot);
+      const long long at = __shfl_sync(0xffffffffu, my_at, k);
+      if (live && at >= 0) {
+        Vec o;
+        if constexpr (VEC == 4 && sizeof(T) == 2) {
+          reinterpret_cast<uint2&>(o) = make_uint2(pack_bf16x2(y[0] * f, y[1 % VEC] * f), pack_bf16x2(y[2 % VEC] * f, y[3 % VEC] * f));
+        } else {
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) ad_st(o.e + j, y[j] * f);
+        }
+        *reinterpret_cast<Vec*>(base + at) = o;
+      }
     }
     if (!advance || !live) return;
     // the state after the run, entry i the row taps - 1 - i before the next token; entries of a short run move up
