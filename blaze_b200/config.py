@@ -204,7 +204,7 @@ class DeltaSpec:
 
 @dataclass
 class MinGruSpec:
-    """Gated recurrence, element by element, whose gates read the current token only (minGRU), with a gated output."""
+    """Elementwise recurrence with a gated output (minGRU): its gate and its candidate depend on the token's input, not on the state."""
     width: int
     conv = 0                    # no convolution of its own
     heads = state = 1
