@@ -93,23 +93,23 @@ __global__ void __launch_bounds__(128) maps_plain_kernel(MapsParams p) {
       s_p[tid] = s[0] == -INFINITY ? 0.f : 1.f / (1.f + expf(-s[0]));
     } else {
 #pragma unroll
-    for (int mp = 0; mp < MAPS; ++mp) {
-      const float v = warp_max(s[mp]);
-      if (lane == 0) red[mp][warp] = v;
-    }
-    __syncthreads();
+      for (int mp = 0; mp < MAPS; ++mp) {
+        const float v = warp_max(s[mp]);
+        if (lane == 0) red[mp][warp] = v;
+      }
+      __syncthreads();
 #pragma unroll
-    for (int mp = 0; mp < MAPS; ++mp) {
-      const float mt = fmaxf(fmaxf(red[mp][0], red[mp][1]), fmaxf(red[mp][2], red[mp][3]));
-      const float mn = fmaxf(m[mp], mt);
-      const float f = m[mp] == -INFINITY ? 0.f : expf(m[mp] - mn);
-      const float w = s[mp] == -INFINITY ? 0.f : expf(s[mp] - mn);
-      s_p[mp * 128 + tid] = w;
-      l[mp] = l[mp] * f + w;                           // this thread's share of the sum
-      m[mp] = mn;
+      for (int mp = 0; mp < MAPS; ++mp) {
+        const float mt = fmaxf(fmaxf(red[mp][0], red[mp][1]), fmaxf(red[mp][2], red[mp][3]));
+        const float mn = fmaxf(m[mp], mt);
+        const float f = m[mp] == -INFINITY ? 0.f : expf(m[mp] - mn);
+        const float w = s[mp] == -INFINITY ? 0.f : expf(s[mp] - mn);
+        s_p[mp * 128 + tid] = w;
+        l[mp] = l[mp] * f + w;                           // this thread's share of the sum
+        m[mp] = mn;
 #pragma unroll
-      for (int c = 0; c < VC; ++c) acc[mp][c] *= f;
-    }
+        for (int c = 0; c < VC; ++c) acc[mp][c] *= f;
+      }
     }
     __syncthreads();
     const int k_end = min(128, pos - k0 + 1);
@@ -344,61 +344,61 @@ __global__ void __launch_bounds__(kShortWarps * 32) maps_short_kernel(MapsParams
 #pragma unroll
         for (int r = 0; r < 2; ++r) split_bf16x2(s[0][h][2 * r], s[0][h][2 * r + 1], hi[0][h * 2 + r], lo[0][h * 2 + r]);
     } else {
-    float mx[MAPS][2];
-#pragma unroll
-    for (int mp = 0; mp < MAPS; ++mp) {
-      mx[mp][0] = mx[mp][1] = -INFINITY;
-#pragma unroll
-      for (int h = 0; h < 2; ++h)
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const int kk = key + h * 8 + (k & 1);
-          const bool vis = k < 2 ? (kk <= pos_a && kk >= lo_a) : (kk <= pos_b && kk >= lo_b);
-          s[mp][h][k] = vis ? s[mp][h][k] * sc : -INFINITY;
-          mx[mp][k >> 1] = fmaxf(mx[mp][k >> 1], s[mp][h][k]);
-        }
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        mx[mp][r] = fmaxf(mx[mp][r], __shfl_xor_sync(0xffffffffu, mx[mp][r], 1));
-        mx[mp][r] = fmaxf(mx[mp][r], __shfl_xor_sync(0xffffffffu, mx[mp][r], 2));
-      }
-    }
-    // the running maximum moves only when a row has outgrown it by 2^kLazy (or has none yet): weights stay far from overflow
-    bool grow = false;
-#pragma unroll
-    for (int mp = 0; mp < MAPS; ++mp)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) grow |= mx[mp][r] > m[mp][r] + kLazy || (m[mp][r] == -INFINITY && mx[mp][r] != -INFINITY);
-    if (__any_sync(0xffffffffu, grow)) {
+      float mx[MAPS][2];
 #pragma unroll
       for (int mp = 0; mp < MAPS; ++mp) {
-        float f[2];
+        mx[mp][0] = mx[mp][1] = -INFINITY;
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int kk = key + h * 8 + (k & 1);
+            const bool vis = k < 2 ? (kk <= pos_a && kk >= lo_a) : (kk <= pos_b && kk >= lo_b);
+            s[mp][h][k] = vis ? s[mp][h][k] * sc : -INFINITY;
+            mx[mp][k >> 1] = fmaxf(mx[mp][k >> 1], s[mp][h][k]);
+          }
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
-          const float mn = fmaxf(m[mp][r], mx[mp][r]);
-          f[r] = m[mp][r] == -INFINITY ? 0.f : ex2(m[mp][r] - mn);
-          m[mp][r] = mn;
-          l[mp][r] *= f[r];
+          mx[mp][r] = fmaxf(mx[mp][r], __shfl_xor_sync(0xffffffffu, mx[mp][r], 1));
+          mx[mp][r] = fmaxf(mx[mp][r], __shfl_xor_sync(0xffffffffu, mx[mp][r], 2));
         }
-#pragma unroll
-        for (int c = 0; c < VP / 8; ++c) { o[mp][c][0] *= f[0]; o[mp][c][1] *= f[0]; o[mp][c][2] *= f[1]; o[mp][c][3] *= f[1]; }
       }
-    }
+      // the running maximum moves only when a row has outgrown it by 2^kLazy (or has none yet): weights stay far from overflow
+      bool grow = false;
 #pragma unroll
-    for (int mp = 0; mp < MAPS; ++mp) {
-      float w[2][4];
+      for (int mp = 0; mp < MAPS; ++mp)
 #pragma unroll
-      for (int h = 0; h < 2; ++h)
+        for (int r = 0; r < 2; ++r) grow |= mx[mp][r] > m[mp][r] + kLazy || (m[mp][r] == -INFINITY && mx[mp][r] != -INFINITY);
+      if (__any_sync(0xffffffffu, grow)) {
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          w[h][k] = s[mp][h][k] == -INFINITY ? 0.f : ex2(s[mp][h][k] - m[mp][k >> 1]);
-          l[mp][k >> 1] += w[h][k];
+        for (int mp = 0; mp < MAPS; ++mp) {
+          float f[2];
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const float mn = fmaxf(m[mp][r], mx[mp][r]);
+            f[r] = m[mp][r] == -INFINITY ? 0.f : ex2(m[mp][r] - mn);
+            m[mp][r] = mn;
+            l[mp][r] *= f[r];
+          }
+#pragma unroll
+          for (int c = 0; c < VP / 8; ++c) { o[mp][c][0] *= f[0]; o[mp][c][1] *= f[0]; o[mp][c][2] *= f[1]; o[mp][c][3] *= f[1]; }
         }
+      }
 #pragma unroll
-      for (int h = 0; h < 2; ++h)
+      for (int mp = 0; mp < MAPS; ++mp) {
+        float w[2][4];
 #pragma unroll
-        for (int r = 0; r < 2; ++r) split_bf16x2(w[h][2 * r], w[h][2 * r + 1], hi[mp][h * 2 + r], lo[mp][h * 2 + r]);
-    }
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            w[h][k] = s[mp][h][k] == -INFINITY ? 0.f : ex2(s[mp][h][k] - m[mp][k >> 1]);
+            l[mp][k >> 1] += w[h][k];
+          }
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) split_bf16x2(w[h][2 * r], w[h][2 * r + 1], hi[mp][h * 2 + r], lo[mp][h * 2 + r]);
+      }
     }
     const uint32_t va = blk + (MAPS * 16 * dp + (mat & 1) * 8 * vp + (mat >> 1) * 64 + mrow * 8) * 2;
 #pragma unroll
@@ -772,12 +772,12 @@ struct ConvPrepParams {
 };
 static constexpr int kConvPrepTok = 8;     // tokens per warp, at least the taps before the current one
 
+template <typename T, int VEC> struct alignas(sizeof(T) * VEC) PrepVec { T e[VEC]; };
+
 // A warp per (8 tokens of a sequence, head): a causal convolution over time of each projected channel, then queries (times their position's
 // temperature) to their buffer, keys and values (divided by their root mean square: unit_v) to their page.  The rows before the sequence's
 // new ones come from its state, which only the first 8 tokens' warp of a channel reads, and then writes.  TAPS: the real ones rounded up.
 // ONCE: one turn of the warp takes a whole head (dim and vdim up to 32 * VEC), whose rows then stay in registers.
-template <typename T, int VEC> struct alignas(sizeof(T) * VEC) PrepVec { T e[VEC]; };
-
 template <typename T, int TAPS, int VEC, bool ONCE>
 __global__ void __launch_bounds__(128) conv_prep_pages_kernel(ConvPrepParams q) {
   pdl_trigger();

@@ -276,54 +276,54 @@ __global__ void __launch_bounds__(kTcThreads, 1) maps_tc_kernel(MapsParams p, Ma
             tmem_st16(s_addr + 64 + k * 16, rm);
           }
         } else {
-        if (!__all_sync(0xffffffffu, a <= 0 && z >= 127)) {
+          if (!__all_sync(0xffffffffu, a <= 0 && z >= 127)) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (k * 32 + j < a || k * 32 + j > z) v[k][j] = 0xff800000u;     // -inf
+          }
+          float t = -INFINITY;
 #pragma unroll
           for (int k = 0; k < 4; ++k)
 #pragma unroll
-            for (int j = 0; j < 32; ++j)
-              if (k * 32 + j < a || k * 32 + j > z) v[k][j] = 0xff800000u;     // -inf
-        }
-        float t = -INFINITY;
+            for (int j = 0; j < 32; j += 2) t = fmaxf(t, fmaxf(__uint_as_float(v[k][j]), __uint_as_float(v[k][j + 1])));
+          t *= sc;
+          const bool grow = t > mx + kTcLazy || (mx == -INFINITY && t != -INFINITY);
+          if (__any_sync(0xffffffffu, grow)) {
+            const float mn = grow ? t : mx;
+            const float f = grow ? (mx == -INFINITY ? 0.f : ex2(mx - mn)) : 1.f;
+            mx = mn;
+            l *= f;
+            if (i > 0) {
+              for (int k = 0; k < vp; k += 16) {
+                uint32_t w[16];
+                tmem_ld16(o_addr + k, w);
+                tmem_ld_wait();
 #pragma unroll
-        for (int k = 0; k < 4; ++k)
-#pragma unroll
-          for (int j = 0; j < 32; j += 2) t = fmaxf(t, fmaxf(__uint_as_float(v[k][j]), __uint_as_float(v[k][j + 1])));
-        t *= sc;
-        const bool grow = t > mx + kTcLazy || (mx == -INFINITY && t != -INFINITY);
-        if (__any_sync(0xffffffffu, grow)) {
-          const float mn = grow ? t : mx;
-          const float f = grow ? (mx == -INFINITY ? 0.f : ex2(mx - mn)) : 1.f;
-          mx = mn;
-          l *= f;
-          if (i > 0) {
-            for (int k = 0; k < vp; k += 16) {
-              uint32_t w[16];
-              tmem_ld16(o_addr + k, w);
-              tmem_ld_wait();
-#pragma unroll
-              for (int j = 0; j < 16; ++j) w[j] = __float_as_uint(__uint_as_float(w[j]) * f);
-              tmem_st16(o_addr + k, w);
+                for (int j = 0; j < 16; ++j) w[j] = __float_as_uint(__uint_as_float(w[j]) * f);
+                tmem_st16(o_addr + k, w);
+              }
             }
           }
-        }
-        const float off = mx == -INFINITY ? 0.f : -mx;        // a row that has seen no key yet: every weight is 2^-inf
-        float l0 = 0.f, l1 = 0.f;
+          const float off = mx == -INFINITY ? 0.f : -mx;        // a row that has seen no key yet: every weight is 2^-inf
+          float l0 = 0.f, l1 = 0.f;
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          uint32_t hi[16], rm[16];
+          for (int k = 0; k < 4; ++k) {
+            uint32_t hi[16], rm[16];
 #pragma unroll
-          for (int j = 0; j < 16; ++j) {
-            const float w0 = ex2(fmaf(__uint_as_float(v[k][2 * j]), sc, off)), w1 = ex2(fmaf(__uint_as_float(v[k][2 * j + 1]), sc, off));
-            l0 += w0;
-            l1 += w1;
-            const __nv_bfloat162 h = __floats2bfloat162_rn(w0, w1);
-            hi[j] = *reinterpret_cast<const uint32_t*>(&h);
-            rm[j] = pack_bf16x2(w0 - __uint_as_float(hi[j] << 16), w1 - __uint_as_float(hi[j] & 0xffff0000u));
+            for (int j = 0; j < 16; ++j) {
+              const float w0 = ex2(fmaf(__uint_as_float(v[k][2 * j]), sc, off)), w1 = ex2(fmaf(__uint_as_float(v[k][2 * j + 1]), sc, off));
+              l0 += w0;
+              l1 += w1;
+              const __nv_bfloat162 h = __floats2bfloat162_rn(w0, w1);
+              hi[j] = *reinterpret_cast<const uint32_t*>(&h);
+              rm[j] = pack_bf16x2(w0 - __uint_as_float(hi[j] << 16), w1 - __uint_as_float(hi[j] & 0xffff0000u));
+            }
+            tmem_st16(s_addr + k * 16, hi);
+            tmem_st16(s_addr + 64 + k * 16, rm);
           }
-          tmem_st16(s_addr + k * 16, hi);
-          tmem_st16(s_addr + 64 + k * 16, rm);
-        }
-        l += l0 + l1;
+          l += l0 + l1;
         }
         tmem_st_wait();
         tc_fence_before();

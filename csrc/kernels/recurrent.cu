@@ -618,72 +618,72 @@ __global__ void __launch_bounds__(128) delta_block_records_kernel(RecParams p) {
   // the block that starts in these rows: of a sequence that goes on through all of them exactly one does, and a warp whose rows see
   // one sequence end and another begin takes both of theirs in turn
   for (int t = (int)(w / p.heads) * kBlockTok, end = min(t + kBlockTok, p.T); t < end; ++t) {
-  if (!in_long_run(p, t)) continue;
-  const int seq = p.seq_of_row[t], rest = p.q_start[seq + 1] - t, m = min(kBlockTok, rest);
-  if ((t - p.q_start[seq]) % kBlockTok) continue;
-  const int dk = p.dk, hk = h / (p.heads / p.groups);
-  float q[kBlockTok][NV], k[kBlockTok][NV], beta[kBlockTok], g[kBlockTok];
-#pragma unroll
-  for (int j = 0; j < kBlockTok; ++j) {
-    const T* cv = reinterpret_cast<const T*>(p.conv) + (size_t)(t + min(j, m - 1)) * p.ld_conv;
-#pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      const int d = lane + i * 32;
-      q[j][i] = d < dk && j < m ? rc_ld(cv + (size_t)hk * dk + d) : 0.f;
-      k[j][i] = d < dk && j < m ? rc_ld(cv + (size_t)(p.groups + hk) * dk + d) : 0.f;
-    }
-  }
-#pragma unroll
-  for (int j = 0; j < kBlockTok; ++j) {
-    const size_t row = t + min(j, m - 1);
-    beta[j] = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + row * p.ld_b + h));
-    g[j] = head_decay<T>(p, row, h);
-  }
-  const float qs = rsqrtf((float)dk);
-#pragma unroll
-  for (int j = 0; j < kBlockTok; ++j) {
-    float qq = 0.f, kk = 0.f;
-#pragma unroll
-    for (int i = 0; i < NV; ++i) { qq = fmaf(q[j][i], q[j][i], qq); kk = fmaf(k[j][i], k[j][i], kk); }
-    const float qn = qs / sqrtf(warp_sum(qq) + 1e-6f), kn = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
-#pragma unroll
-    for (int i = 0; i < NV; ++i) { q[j][i] *= qn; k[j][i] *= kn; }
-  }
-  float G = 1.f, D[kBlockTok];                             // D[j]: decay over tokens j + 1 .. i
-#pragma unroll
-  for (int i = 0; i < kBlockTok; ++i) {
-    if (i >= m) break;
-    float* s = p.records + ((size_t)h * p.T + t + i) * REC;
-    G *= g[i];
-    float a[kBlockTok], c[kBlockTok];
+    if (!in_long_run(p, t)) continue;
+    const int seq = p.seq_of_row[t], rest = p.q_start[seq + 1] - t, m = min(kBlockTok, rest);
+    if ((t - p.q_start[seq]) % kBlockTok) continue;
+    const int dk = p.dk, hk = h / (p.heads / p.groups);
+    float q[kBlockTok][NV], k[kBlockTok][NV], beta[kBlockTok], g[kBlockTok];
 #pragma unroll
     for (int j = 0; j < kBlockTok; ++j) {
-      a[j] = c[j] = 0.f;
-      if (j > i) continue;
-      D[j] = j == i ? 1.f : D[j] * g[i];
-      float kk = 0.f, qk = 0.f;
+      const T* cv = reinterpret_cast<const T*>(p.conv) + (size_t)(t + min(j, m - 1)) * p.ld_conv;
 #pragma unroll
-      for (int e = 0; e < NV; ++e) { kk = fmaf(k[i][e], k[j][e], kk); qk = fmaf(q[i][e], k[j][e], qk); }
-      c[j] = D[j] * warp_sum(qk);
-      if (j < i) a[j] = beta[i] * D[j] * warp_sum(kk);
+      for (int i = 0; i < NV; ++i) {
+        const int d = lane + i * 32;
+        q[j][i] = d < dk && j < m ? rc_ld(cv + (size_t)hk * dk + d) : 0.f;
+        k[j][i] = d < dk && j < m ? rc_ld(cv + (size_t)(p.groups + hk) * dk + d) : 0.f;
+      }
     }
 #pragma unroll
-    for (int e = 0; e < NV; ++e) {
-      s[lane + e * 32] = q[i][e];
-      s[DKP + lane + e * 32] = k[i][e];
+    for (int j = 0; j < kBlockTok; ++j) {
+      const size_t row = t + min(j, m - 1);
+      beta[j] = rc_sigmoid<T>(rc_ld(reinterpret_cast<const T*>(p.b) + row * p.ld_b + h));
+      g[j] = head_decay<T>(p, row, h);
     }
-    if (lane == 0) {
-      float4* f = reinterpret_cast<float4*>(s + 2 * DKP);
-      f[0] = make_float4(a[0], a[1], a[2], a[3]);
-      f[1] = make_float4(c[0], c[1], c[2], c[3]);
-      float last = 1.f, all = G;                           // decays to the end of the block
+    const float qs = rsqrtf((float)dk);
 #pragma unroll
-      for (int e = 1; e < kBlockTok; ++e)
-        if (e > i && e < m) { last *= g[e]; all *= g[e]; }
-      f[2] = make_float4(beta[i], beta[i] * G, G, last);
-      f[3] = make_float4(all, 0.f, 0.f, 0.f);
+    for (int j = 0; j < kBlockTok; ++j) {
+      float qq = 0.f, kk = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) { qq = fmaf(q[j][i], q[j][i], qq); kk = fmaf(k[j][i], k[j][i], kk); }
+      const float qn = qs / sqrtf(warp_sum(qq) + 1e-6f), kn = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) { q[j][i] *= qn; k[j][i] *= kn; }
     }
-  }
+    float G = 1.f, D[kBlockTok];                             // D[j]: decay over tokens j + 1 .. i
+#pragma unroll
+    for (int i = 0; i < kBlockTok; ++i) {
+      if (i >= m) break;
+      float* s = p.records + ((size_t)h * p.T + t + i) * REC;
+      G *= g[i];
+      float a[kBlockTok], c[kBlockTok];
+#pragma unroll
+      for (int j = 0; j < kBlockTok; ++j) {
+        a[j] = c[j] = 0.f;
+        if (j > i) continue;
+        D[j] = j == i ? 1.f : D[j] * g[i];
+        float kk = 0.f, qk = 0.f;
+#pragma unroll
+        for (int e = 0; e < NV; ++e) { kk = fmaf(k[i][e], k[j][e], kk); qk = fmaf(q[i][e], k[j][e], qk); }
+        c[j] = D[j] * warp_sum(qk);
+        if (j < i) a[j] = beta[i] * D[j] * warp_sum(kk);
+      }
+#pragma unroll
+      for (int e = 0; e < NV; ++e) {
+        s[lane + e * 32] = q[i][e];
+        s[DKP + lane + e * 32] = k[i][e];
+      }
+      if (lane == 0) {
+        float4* f = reinterpret_cast<float4*>(s + 2 * DKP);
+        f[0] = make_float4(a[0], a[1], a[2], a[3]);
+        f[1] = make_float4(c[0], c[1], c[2], c[3]);
+        float last = 1.f, all = G;                           // decays to the end of the block
+#pragma unroll
+        for (int e = 1; e < kBlockTok; ++e)
+          if (e > i && e < m) { last *= g[e]; all *= g[e]; }
+        f[2] = make_float4(beta[i], beta[i] * G, G, last);
+        f[3] = make_float4(all, 0.f, 0.f, 0.f);
+      }
+    }
   }
 }
 
